@@ -1,0 +1,356 @@
+// Helpers around latent attention (one shared cache row per token, [RMS-normed latent | rotary key]) for any head
+// geometry, and a general attention kernel over such rows in 32-bit arithmetic.
+//
+//   latent_prepare_kernel   per token: norm of the latent + rotation of the shared key -> cache row; rotation of every
+//                           head's rotary query part into the caller's query layout
+//   latent_gather_kernel    cache rows of a list of slots -> contiguous latents (what the per-head up-projections read)
+//   latent_pool_kernel      up-projected keys and values + the cached rotary keys -> padded per-head K / V tiles of a
+//                           temporary pool that the prefill attention kernels read
+//   latent_rows_kernel      a warp per (row, head): scores against the cache rows, softmax with window and sink, sum of
+//                           latents.  Runs 32-bit models and geometries outside the tensor-core kernels.
+// Rotation pairs are neighbours: channels (2i, 2i + 1) turn by the angle of frequency i; cos_sin rows are
+// [cos(dims / 2) | sin(dims / 2)].  Positions, angles, norms, scores and weights are 32-bit.
+#include <cuda_bf16.h>
+#include <cuda_fp16.h>
+#include <cuda_runtime.h>
+#include <math_constants.h>
+#include <stdint.h>
+
+#include "../common/launch.cuh"
+
+namespace {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f(__half v) { return __half2float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+template <> __device__ __forceinline__ __half from_f<__half>(float v) { return __float2half_rn(v); }
+
+struct PrepareParams {
+  const void* q;            // [T, ldq]: head h at h * (dim + rot), rotary part last
+  const void* dkv;          // [T, ldkv]: latent (rank) then rotary key (rot)
+  const float* norm_w;      // [rank]
+  const int* positions;     // [T]
+  const float* cos_sin;     // [max_pos, rdims]
+  const int* slot_mapping;  // [T], < 0: no cache row
+  void* cache;              // rows of rank + rot values
+  void* q_out;              // [T, nh, q_pitch]
+  long ldq, ldkv;
+  int T, nh, dim, rot, rdims, rank, q_pitch, nope_off, rot_off, zero_from, max_pos;
+  float eps;
+};
+
+// Block: (token, share of the heads).  The first block of a token also writes its cache row.
+template <typename T>
+__global__ void __launch_bounds__(128) latent_prepare_kernel(const PrepareParams p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  __shared__ float red[4];
+  const int t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int pos = min(max(p.positions[t], 0), p.max_pos - 1);
+  const float* cs = p.cos_sin + static_cast<long>(pos) * p.rdims;
+  const int half = p.rdims / 2;
+  const T* q = reinterpret_cast<const T*>(p.q) + t * p.ldq;
+  if (blockIdx.y == 0) {
+    const T* row = reinterpret_cast<const T*>(p.dkv) + t * p.ldkv;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < p.rank; i += 128) { const float f = to_f(row[i]); ss += f * f; }
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    const float inv = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / static_cast<float>(p.rank) + p.eps);
+    const int slot = p.slot_mapping[t];
+    if (slot >= 0) {
+      T* dst = reinterpret_cast<T*>(p.cache) + static_cast<long>(slot) * (p.rank + p.rot);
+      for (int i = threadIdx.x; i < p.rank; i += 128) dst[i] = from_f<T>(to_f(row[i]) * inv * p.norm_w[i]);
+      for (int i = threadIdx.x; i < p.rot; i += 128) {
+        float v = to_f(row[p.rank + i]);
+        if (i < 2 * half) {
+          const float other = to_f(row[p.rank + (i ^ 1)]);
+          const float c = cs[i >> 1], s = cs[half + (i >> 1)];
+          v = (i & 1) ? v * c + other * s : v * c - other * s;
+        }
+        dst[p.rank + i] = from_f<T>(v);
+      }
+    }
+  }
+  const int hd = p.dim + p.rot;
+  for (int h = blockIdx.y * 4 + warp; h < p.nh; h += 4 * gridDim.y) {
+    const T* src = q + static_cast<long>(h) * hd;
+    T* dst = reinterpret_cast<T*>(p.q_out) + (static_cast<long>(t) * p.nh + h) * p.q_pitch;
+    for (int i = lane; i < p.rot; i += 32) {
+      float v = to_f(src[p.dim + i]);
+      if (i < 2 * half) {
+        const float other = to_f(src[p.dim + (i ^ 1)]);
+        const float c = cs[i >> 1], s = cs[half + (i >> 1)];
+        v = (i & 1) ? v * c + other * s : v * c - other * s;
+      }
+      dst[p.rot_off + i] = from_f<T>(v);
+    }
+    if (p.nope_off >= 0) {
+      for (int i = lane; i < p.dim; i += 32) dst[p.nope_off + i] = src[i];
+      for (int i = p.zero_from + lane; i < p.q_pitch; i += 32) dst[i] = from_f<T>(0.f);
+    }
+  }
+}
+
+// out [n, pitch] (values beyond rank stay zero) from the cache rows of slots[i]; a negative slot gives a zero row.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_gather_kernel(const T* __restrict__ cache, const int* __restrict__ slots,
+                                                            T* __restrict__ out, int n, int rank, int kd, int pitch,
+                                                            int num_rows) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  constexpr int V = 16 / sizeof(T);
+  const int per = (pitch + V - 1) / V;
+  const bool vec = rank % V == 0 && kd % V == 0 && pitch % V == 0;
+  for (long i = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; i < static_cast<long>(n) * per;
+       i += static_cast<long>(gridDim.x) * 256) {
+    const int r = static_cast<int>(i / per), c = static_cast<int>(i % per) * V;
+    const int slot = slots[r];
+    const bool ok = slot >= 0 && slot < num_rows;
+    if (vec) {
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (ok && c < rank) v = *reinterpret_cast<const uint4*>(cache + static_cast<long>(slot) * kd + c);
+      *reinterpret_cast<uint4*>(out + static_cast<long>(r) * pitch + c) = v;
+    } else {
+      for (int e = c; e < min(c + V, pitch); ++e)
+        out[static_cast<long>(r) * pitch + e] = (ok && e < rank) ? cache[static_cast<long>(slot) * kd + e] : from_f<T>(0.f);
+    }
+  }
+}
+
+// Row i of the step's context (block i / 128, row i % 128 of the temporary pool [n / 128, nh, 128, hd]):
+// K = [key (dim) | cached rotary key (rot) | 0], V = [value (vdim) | 0]; rows with a negative slot are zero.
+template <typename T>
+__global__ void __launch_bounds__(256) latent_pool_kernel(const T* __restrict__ cache, const int* __restrict__ slots,
+                                                          const T* __restrict__ kv, long ldkv, T* __restrict__ k_pool,
+                                                          T* __restrict__ v_pool, int nh, int dim, int rot, int vdim,
+                                                          int rank, int hd, int num_rows) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  constexpr int BS = 128;
+  const int r = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int slot = slots[r];
+  const bool ok = slot >= 0 && slot < num_rows;
+  const T* krow = kv + static_cast<long>(r) * ldkv;
+  const T* vrow = krow + static_cast<long>(nh) * dim;
+  const T* rrow = cache + static_cast<long>(ok ? slot : 0) * (rank + rot) + rank;
+  const bool vec = ((dim | rot | vdim | rank) & 7) == 0 && (ldkv & 7) == 0;
+  for (int h = blockIdx.y * 8 + warp; h < nh; h += 8 * gridDim.y) {
+    const long dst = ((static_cast<long>(r / BS) * nh + h) * BS + r % BS) * hd;
+    for (int c8 = lane; c8 < hd / 4; c8 += 32) {        // hd / 8 chunks of K, then of V
+      const bool is_v = c8 >= hd / 8;
+      const int c = (is_v ? c8 - hd / 8 : c8) * 8;
+      T* out = (is_v ? v_pool : k_pool) + dst + c;
+      if (vec) {
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (ok) {
+          if (is_v) {
+            if (c < vdim) v = *reinterpret_cast<const uint4*>(vrow + static_cast<long>(h) * vdim + c);
+          } else if (c < dim) {
+            v = *reinterpret_cast<const uint4*>(krow + static_cast<long>(h) * dim + c);
+          } else if (c < dim + rot) {
+            v = *reinterpret_cast<const uint4*>(rrow + c - dim);
+          }
+        }
+        *reinterpret_cast<uint4*>(out) = v;
+      } else {
+        for (int e = 0; e < 8; ++e) {
+          T v = from_f<T>(0.f);
+          if (ok) {
+            if (is_v) {
+              if (c + e < vdim) v = vrow[static_cast<long>(h) * vdim + c + e];
+            } else if (c + e < dim) {
+              v = krow[static_cast<long>(h) * dim + c + e];
+            } else if (c + e < dim + rot) {
+              v = rrow[c + e - dim];
+            }
+          }
+          out[e] = v;
+        }
+      }
+    }
+  }
+}
+
+struct RowsParams {
+  const void* q_cat;        // [rows, nh, kd]
+  const void* cache;        // rows of kd values; the first vd are the value
+  void* out;                // element (row r, head h, d) at out + h * out_head_stride + r * out_row_stride + d
+  long out_head_stride, out_row_stride;
+  const int* block_tables;
+  const int* row_lens;
+  const int* seq_of_row;    // or null
+  const float* sinks;       // or null
+  int rows, nh, kd, vd, max_blocks, block_size, window, num_rows;
+  float sm_scale;
+};
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  extern __shared__ float smem[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long item = static_cast<long>(blockIdx.x) * 4 + warp;
+  if (item >= static_cast<long>(p.rows) * p.nh) return;
+  const int r = static_cast<int>(item / p.nh), h = static_cast<int>(item % p.nh);
+  float* q = smem + warp * p.kd;
+  const T* qs = reinterpret_cast<const T*>(p.q_cat) + item * p.kd;
+  for (int i = lane; i < p.kd; i += 32) q[i] = to_f(qs[i]) * p.sm_scale;
+  __syncwarp();
+  const int len = min(p.row_lens[r], p.max_blocks * p.block_size);
+  const int lo = p.window > 0 ? max(0, len - p.window) : 0;
+  const int* bt = p.block_tables + static_cast<long>(p.seq_of_row ? p.seq_of_row[r] : r) * p.max_blocks;
+  const T* cache = reinterpret_cast<const T*>(p.cache);
+  float o[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) o[i] = 0.f;
+  float m = -CUDART_INF_F, l = 0.f;
+  for (int k0 = lo; k0 < len; k0 += 32) {
+    const int tok = k0 + lane;
+    long src = 0;
+    float s = -CUDART_INF_F;
+    if (tok < len) {
+      src = (static_cast<long>(bt[tok / p.block_size]) * p.block_size + tok % p.block_size);
+      src = (src < 0 || src >= p.num_rows ? 0 : src) * p.kd;
+      const T* row = cache + src;
+      float a0 = 0.f, a1 = 0.f;
+      int i = 0;
+      for (; i + 1 < p.kd; i += 2) { a0 = fmaf(q[i], to_f(row[i]), a0); a1 = fmaf(q[i + 1], to_f(row[i + 1]), a1); }
+      if (i < p.kd) a0 = fmaf(q[i], to_f(row[i]), a0);
+      s = a0 + a1;
+    }
+    float mx = s;
+    for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+    const float nm = fmaxf(m, mx);            // at least one key of the chunk is visible
+    const float alpha = __expf(m - nm);
+    const float pv = __expf(s - nm);
+    float rs = pv;
+    for (int x = 16; x > 0; x >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, x);
+    l = l * alpha + rs;
+    m = nm;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] *= alpha;
+    const int n = min(32, len - k0);
+    for (int j = 0; j < n; ++j) {
+      const float pj = __shfl_sync(0xffffffffu, pv, j);
+      const T* row = cache + __shfl_sync(0xffffffffu, src, j);
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (i * 32 + lane < p.vd) o[i] = fmaf(pj, to_f(row[i * 32 + lane]), o[i]);
+    }
+  }
+  if (p.sinks != nullptr && m != -CUDART_INF_F) l += __expf(p.sinks[h] - m);
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  T* out = reinterpret_cast<T*>(p.out) + h * p.out_head_stride + r * p.out_row_stride;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (i * 32 + lane < p.vd) out[i * 32 + lane] = from_f<T>(o[i] * inv);
+}
+
+template <typename T>
+int launch_rows(const RowsParams& p, cudaStream_t s) {
+  const long items = static_cast<long>(p.rows) * p.nh;
+  const dim3 grid(static_cast<unsigned>((items + 3) / 4));
+  const int smem = 4 * p.kd * 4;
+#define FI_ROWS(N) return static_cast<int>(fi::launch_kernel(latent_rows_kernel<T, N>, grid, dim3(128), smem, s, 0, p))
+  if (p.vd <= 64) FI_ROWS(2);
+  if (p.vd <= 128) FI_ROWS(4);
+  if (p.vd <= 256) FI_ROWS(8);
+  if (p.vd <= 512) FI_ROWS(16);
+  FI_ROWS(32);
+#undef FI_ROWS
+}
+
+}  // namespace
+
+#define FI_BY_TYPE(dtype, CALL)                 \
+  if (dtype == 0) { CALL(__nv_bfloat16); }      \
+  else if (dtype == 1) { CALL(__half); }        \
+  else if (dtype == 2) { CALL(float); }         \
+  else return -11;
+
+// dtype: 0 bf16, 1 fp16, 2 fp32 (q, dkv, cache, q_out).  nope_off < 0: only the rotary parts of the queries are
+// written; otherwise the other dimensions are copied to nope_off and [zero_from, q_pitch) is cleared.
+extern "C" int fi_latent_prepare(const void* q, long ldq, const void* dkv, long ldkv, const float* norm_w, float eps,
+                                 const int* positions, const float* cos_sin, int max_pos, const int* slot_mapping,
+                                 void* cache, void* q_out, int q_pitch, int nope_off, int rot_off, int zero_from, int T,
+                                 int nh, int dim, int rot, int rdims, int rank, int dtype, void* stream) {
+  if (T <= 0) return 0;
+  if (nh <= 0 || dim < 0 || rot < 0 || rank <= 0 || rdims < 0 || rdims > rot || rdims % 2 != 0 || max_pos <= 0 ||
+      rot_off < 0 || rot_off + rot > q_pitch || (nope_off >= 0 && (nope_off + dim > q_pitch || zero_from < 0)))
+    return -10;
+  PrepareParams p = {};
+  p.q = q; p.dkv = dkv; p.norm_w = norm_w; p.positions = positions; p.cos_sin = cos_sin; p.slot_mapping = slot_mapping;
+  p.cache = cache; p.q_out = q_out; p.ldq = ldq; p.ldkv = ldkv; p.T = T; p.nh = nh; p.dim = dim; p.rot = rot;
+  p.rdims = rdims; p.rank = rank; p.q_pitch = q_pitch; p.nope_off = nope_off; p.rot_off = rot_off;
+  p.zero_from = zero_from; p.max_pos = max_pos; p.eps = eps;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid(T, T >= 256 ? 1 : (nh + 3) / 4);
+#define FI_CALL(TT) return static_cast<int>(fi::launch_kernel(latent_prepare_kernel<TT>, grid, dim3(128), 0, s, 0, p))
+  FI_BY_TYPE(dtype, FI_CALL)
+#undef FI_CALL
+  return 0;
+}
+
+// out [n, pitch] of dtype; cache holds num_rows rows of kd values.
+extern "C" int fi_latent_gather(const void* cache, const int* slots, void* out, int n, int rank, int kd, int pitch,
+                                int num_rows, int dtype, void* stream) {
+  if (n <= 0) return 0;
+  if (rank <= 0 || kd < rank || pitch < rank || num_rows <= 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0 ||
+      (reinterpret_cast<uintptr_t>(cache) & 15) != 0)
+    return -10;
+  const long work = static_cast<long>(n) * ((pitch + 3) / 4);
+  const unsigned grid = static_cast<unsigned>(work / 256 + 1 < 1184 ? work / 256 + 1 : 1184);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define FI_CALL(TT) return static_cast<int>(fi::launch_kernel(latent_gather_kernel<TT>, dim3(grid), dim3(256), 0, s, 0, \
+    (const TT*)cache, slots, (TT*)out, n, rank, kd, pitch, num_rows))
+  FI_BY_TYPE(dtype, FI_CALL)
+#undef FI_CALL
+  return 0;
+}
+
+// n (a multiple of 128) context rows -> pools [n / 128, nh, 128, hd]; kv: [n, ldkv] = [nh * dim | nh * vdim].
+extern "C" int fi_latent_pool(const void* cache, const int* slots, const void* kv, long ldkv, void* k_pool, void* v_pool,
+                              int n, int nh, int dim, int rot, int vdim, int rank, int hd, int num_rows, int dtype,
+                              void* stream) {
+  if (n <= 0) return 0;
+  if (n % 128 != 0 || nh <= 0 || dim + rot > hd || vdim > hd || hd % 8 != 0 || num_rows <= 0) return -10;
+  if ((reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(k_pool) | reinterpret_cast<uintptr_t>(v_pool) |
+       reinterpret_cast<uintptr_t>(cache)) & 15)
+    return -10;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid(n, n >= 1024 ? 1 : (nh + 7) / 8);
+#define FI_CALL(TT) return static_cast<int>(fi::launch_kernel(latent_pool_kernel<TT>, grid, dim3(256), 0, s, 0, \
+    (const TT*)cache, slots, (const TT*)kv, ldkv, (TT*)k_pool, (TT*)v_pool, nh, dim, rot, vdim, rank, hd, num_rows))
+  if (dtype == 0) { FI_CALL(__nv_bfloat16); }
+  if (dtype == 1) { FI_CALL(__half); }
+#undef FI_CALL
+  return -11;
+}
+
+// General attention of flattened rows over latent cache rows, 32-bit arithmetic.  window <= 0: none; sinks may be null.
+extern "C" int fi_latent_rows(const void* q_cat, const void* cache, void* out, long out_head_stride, long out_row_stride,
+                              const int* block_tables, const int* row_lens, const int* seq_of_row, int rows, int nh,
+                              int kd, int vd, int max_blocks, int block_size, int num_rows, int window,
+                              const float* sinks, float sm_scale, int dtype, void* stream) {
+  if (rows <= 0 || nh <= 0) return 0;
+  if (kd <= 0 || vd <= 0 || vd > kd || vd > 1024 || kd > 2048 || block_size <= 0 || max_blocks <= 0 || num_rows <= 0)
+    return -10;
+  RowsParams p = {};
+  p.q_cat = q_cat; p.cache = cache; p.out = out; p.out_head_stride = out_head_stride; p.out_row_stride = out_row_stride;
+  p.block_tables = block_tables; p.row_lens = row_lens; p.seq_of_row = seq_of_row; p.sinks = sinks; p.rows = rows;
+  p.nh = nh; p.kd = kd; p.vd = vd; p.max_blocks = max_blocks; p.block_size = block_size; p.num_rows = num_rows;
+  p.window = window; p.sm_scale = sm_scale;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define FI_CALL(TT) return launch_rows<TT>(p, s)
+  FI_BY_TYPE(dtype, FI_CALL)
+#undef FI_CALL
+  return 0;
+}

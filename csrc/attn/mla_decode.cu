@@ -5,6 +5,10 @@
 //   score(h, t)  = q_cat[h] . row[t]        q_cat[h] = [q_nope[h] W_UK[h] | rope(q_rope[h])]
 //   out_lat[h]   = sum_t softmax(score)[t] * row[t][0:512]          (then out[h] = out_lat[h] W_UV[h]^T)
 //
+// The decode kernel also runs rows of other geometries (a latent of up to 512 values plus any rotary width, the
+// row a multiple of 16 bytes), with a sliding window and with a per-head sink: an extra exp(sink) in the
+// softmax denominator that has no key and no value.
+//
 // The two per-head projections (W_UK before, W_UV after) are batched matrix products outside this file.
 //
 // Kernels
@@ -89,6 +93,13 @@ __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wai
 // Row-major [rows][W] 16-bit tile whose 16-byte chunks are XOR-swizzled by (row & 7) inside every group of 8.
 template <int W>
 __device__ __forceinline__ int tile_off(int row, int chunk) { return row * W + ((chunk ^ (row & 7)) << 3); }
+// The cache-row tile: the fixed geometry swizzles rows of 576 values; other geometries have a pitch of an odd
+// number of 16-byte chunks, which spreads eight rows over all banks without a swizzle.
+template <int KDT>
+__device__ __forceinline__ int row_off(int row, int chunk, int pitch) {
+  if constexpr (KDT > 0) return tile_off<KDT>(row, chunk);
+  return row * pitch + (chunk << 3);
+}
 
 struct MlaParams {
   const void* q_cat;          // [rows, nh, 576]
@@ -102,16 +113,24 @@ struct MlaParams {
   float* ws_ml;               // [rows, nh, splits, 2] partial (max, denominator)
   int nh, max_blocks, block_size, splits;
   float sm_scale;
+  const float* sinks;         // [nh] or null
+  int window;                 // > 0: only the last `window` rows of the visible ones count
+  int kd, vd, pitch;          // run-time geometry: row width, latent width, shared-memory pitch (elements)
 };
 
-template <typename T>
+// KDT = 576: the fixed geometry.  KDT = 0: geometry from the parameters; VB 64-value blocks cover the latent.
+template <typename T, int KDT, int VB>
 __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   extern __shared__ __align__(16) uint8_t smem[];
-  T* sK = reinterpret_cast<T*>(smem);                       // [64][576]
-  T* sQ = sK + CH * KD;                                     // [16][576]
-  T* sP = sQ + 16 * KD;                                     // [16][64]
+  const int kd = KDT > 0 ? KDT : p.kd;                      // values per cache row
+  const int pitch = KDT > 0 ? KDT : p.pitch;
+  const int ksteps = KDT > 0 ? KDT / 16 : (kd + 15) / 16;
+  const int vd = KDT > 0 ? VB * 64 : p.vd;
+  T* sK = reinterpret_cast<T*>(smem);                       // [64][pitch]
+  T* sQ = sK + CH * pitch;                                  // [16][pitch]
+  T* sP = sQ + 16 * pitch;                                  // [16][64]
   float* sMax = reinterpret_cast<float*>(sP + 16 * CH);     // [4 warps][16 rows]
   const int split = blockIdx.x, group = blockIdx.y, r = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -119,34 +138,41 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   const int heads_here = min(16, p.nh - head0);
   const int len = p.row_lens[r];
   const int* bt = p.block_tables + static_cast<long>(p.seq_of_row ? p.seq_of_row[r] : r) * p.max_blocks;
-  const int n_chunks = (len + CH - 1) / CH;
+  const int lo = p.window > 0 ? max(0, len - p.window) : 0;  // first visible row
+  const int c_first = lo / CH;
+  const int n_chunks = max((len + CH - 1) / CH - c_first, 0);
   const int per = (n_chunks + p.splits - 1) / p.splits;
-  const int c_begin = split * per, c_end = min(n_chunks, c_begin + per);
+  const int c_begin = c_first + split * per, c_end = min(c_first + n_chunks, c_begin + per);
 
-  for (int i = threadIdx.x; i < 16 * (KD / 8); i += 128) {
-    const int row = i / (KD / 8), c = i % (KD / 8);
+  if constexpr (KDT == 0) {             // columns between the row width and the pitch are read as zero
+    for (int i = threadIdx.x; i < (CH + 16) * pitch / 8; i += 128)
+      *reinterpret_cast<uint4*>(sK + i * 8) = make_uint4(0, 0, 0, 0);
+    __syncthreads();
+  }
+  for (int i = threadIdx.x; i < 16 * (kd / 8); i += 128) {
+    const int row = i / (kd / 8), c = i % (kd / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
     if (row < heads_here)
       v = *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.q_cat) +
-                                          (static_cast<long>(r) * p.nh + head0 + row) * KD + c * 8);
-    *reinterpret_cast<uint4*>(sQ + tile_off<KD>(row, c)) = v;
+                                          (static_cast<long>(r) * p.nh + head0 + row) * kd + c * 8);
+    *reinterpret_cast<uint4*>(sQ + row_off<KDT>(row, c, pitch)) = v;
   }
-  float o[16][4];                       // 16 rows x this warp's 128 latent channels
+  float o[VB * 2][4];                   // 16 rows x this warp's quarter of the latent channels
 #pragma unroll
-  for (int i = 0; i < 16; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+  for (int i = 0; i < VB * 2; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;   // rows lane/4 and lane/4 + 8; l: this warp's tokens
   const float scale2 = p.sm_scale * kLog2e;
   const T* cache = reinterpret_cast<const T*>(p.cache);
 
   for (int c = c_begin; c < c_end; ++c) {
     // ---- stage 64 cache rows (rows past the visible length are zero)
-    for (int i = threadIdx.x; i < CH * (KD / 8); i += 128) {
-      const int row = i / (KD / 8), ch = i % (KD / 8);
+    for (int i = threadIdx.x; i < CH * (kd / 8); i += 128) {
+      const int row = i / (kd / 8), ch = i % (kd / 8);
       const int tok = c * CH + row;
       const bool valid = tok < len;
       const int blk = valid ? bt[tok / p.block_size] : 0;
-      const long src = (static_cast<long>(blk) * p.block_size + (valid ? tok % p.block_size : 0)) * KD + ch * 8;
-      cp_async16(sK + tile_off<KD>(row, ch), cache + src, valid);
+      const long src = (static_cast<long>(blk) * p.block_size + (valid ? tok % p.block_size : 0)) * kd + ch * 8;
+      cp_async16(sK + row_off<KDT>(row, ch, pitch), cache + src, valid);
     }
     cp_async_commit();
     cp_async_wait_all();
@@ -154,10 +180,10 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
     // ---- scores of this warp's 16 tokens
     float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll 4
-    for (int ks = 0; ks < KD / 16; ++ks) {
+    for (int ks = 0; ks < ksteps; ++ks) {
       uint32_t a[4], kb[4];
-      ldsm_x4(a, smem_addr(sQ + tile_off<KD>((lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4))));
-      ldsm_x4(kb, smem_addr(sK + tile_off<KD>(warp * 16 + (lane & 7) + (lane >> 4) * 8, ks * 2 + ((lane >> 3) & 1))));
+      ldsm_x4(a, smem_addr(sQ + row_off<KDT>((lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4), pitch)));
+      ldsm_x4(kb, smem_addr(sK + row_off<KDT>(warp * 16 + (lane & 7) + (lane >> 4) * 8, ks * 2 + ((lane >> 3) & 1), pitch)));
       Mma<T>::mma(s[0], a, kb);
       Mma<T>::mma(s[1], a, kb + 2);
     }
@@ -168,7 +194,7 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
       for (int e = 0; e < 4; ++e) {
         const int tok = c * CH + warp * 16 + j * 8 + (lane & 3) * 2 + (e & 1);
         float v = s[j][e] * scale2;
-        if (tok >= len) v = -CUDART_INF_F;
+        if (tok >= len || tok < lo) v = -CUDART_INF_F;
         s[j][e] = v;
         if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
       }
@@ -208,18 +234,18 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
     }
     l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
 #pragma unroll
-    for (int i = 0; i < 16; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+    for (int i = 0; i < VB * 2; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
     __syncthreads();
-    // ---- output: this warp's 128 latent channels over all 64 tokens of the chunk
+    // ---- output: this warp's latent channels over all 64 tokens of the chunk
 #pragma unroll
     for (int ks = 0; ks < CH / 16; ++ks) {
       uint32_t pa[4];
       ldsm_x4(pa, smem_addr(sP + tile_off<CH>((lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4))));
 #pragma unroll
-      for (int dp = 0; dp < 8; ++dp) {
+      for (int dp = 0; dp < VB; ++dp) {
         uint32_t vb[4];
-        ldsm_x4_t(vb, smem_addr(sK + tile_off<KD>(ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8,
-                                                    warp * 16 + dp * 2 + (lane >> 4))));
+        ldsm_x4_t(vb, smem_addr(sK + row_off<KDT>(ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8,
+                                                    warp * (VB * 2) + dp * 2 + (lane >> 4), pitch)));
         Mma<T>::mma(o[2 * dp], pa, vb);
         Mma<T>::mma(o[2 * dp + 1], pa, vb + 2);
       }
@@ -239,11 +265,16 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   for (int w = 0; w < 4; ++w) { lt0 += sMax[w * 16 + (lane >> 2)]; lt1 += sMax[w * 16 + (lane >> 2) + 8]; }
   const int r0 = lane >> 2, r1 = r0 + 8;
   if (p.splits == 1) {
+    if (p.sinks != nullptr) {             // scores are in units of log2: so is the sink
+      if (r0 < heads_here && m0 != -CUDART_INF_F) lt0 += exp2f(p.sinks[head0 + r0] * kLog2e - m0);
+      if (r1 < heads_here && m1 != -CUDART_INF_F) lt1 += exp2f(p.sinks[head0 + r1] * kLog2e - m1);
+    }
     const float i0 = lt0 > 0.f ? 1.f / lt0 : 0.f, i1 = lt1 > 0.f ? 1.f / lt1 : 0.f;
     T* out = reinterpret_cast<T*>(p.out);
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      const int d = warp * 128 + i * 8 + (lane & 3) * 2;
+    for (int i = 0; i < VB * 2; ++i) {
+      const int d = warp * (VB * 16) + i * 8 + (lane & 3) * 2;
+      if (KDT == 0 && d >= vd) continue;
       if (r0 < heads_here)
         *reinterpret_cast<uint32_t*>(out + (head0 + r0) * p.out_head_stride + r * p.out_row_stride + d) =
             Mma<T>::pack(o[i][0] * i0, o[i][1] * i0);
@@ -253,14 +284,15 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
     }
   } else {
 #pragma unroll
-    for (int i = 0; i < 16; ++i) {
-      const int d = warp * 128 + i * 8 + (lane & 3) * 2;
+    for (int i = 0; i < VB * 2; ++i) {
+      const int d = warp * (VB * 16) + i * 8 + (lane & 3) * 2;
+      if (KDT == 0 && d >= vd) continue;
       if (r0 < heads_here) {
-        float* w = p.ws_o + ((static_cast<long>(r) * p.nh + head0 + r0) * p.splits + split) * VD + d;
+        float* w = p.ws_o + ((static_cast<long>(r) * p.nh + head0 + r0) * p.splits + split) * vd + d;
         w[0] = o[i][0]; w[1] = o[i][1];
       }
       if (r1 < heads_here) {
-        float* w = p.ws_o + ((static_cast<long>(r) * p.nh + head0 + r1) * p.splits + split) * VD + d;
+        float* w = p.ws_o + ((static_cast<long>(r) * p.nh + head0 + r1) * p.splits + split) * vd + d;
         w[0] = o[i][2]; w[1] = o[i][3];
       }
     }
@@ -287,13 +319,15 @@ __global__ void mla_merge_kernel(const MlaParams p) {
   for (int s = 0; s < p.splits; ++s) m = fmaxf(m, ml[2 * s]);
   float l = 0.f;
   for (int s = 0; s < p.splits; ++s) l += ml[2 * s] == -CUDART_INF_F ? 0.f : ml[2 * s + 1] * exp2f(ml[2 * s] - m);
+  if (p.sinks != nullptr && m != -CUDART_INF_F) l += exp2f(p.sinks[h] * kLog2e - m);
   const float inv = l > 0.f ? 1.f / l : 0.f;
+  const int vd = p.vd;
   T* out = reinterpret_cast<T*>(p.out) + h * p.out_head_stride + r * p.out_row_stride;
-  const float* wo = p.ws_o + (static_cast<long>(r) * p.nh + h) * p.splits * VD;
-  for (int d = threadIdx.x; d < VD; d += blockDim.x) {
+  const float* wo = p.ws_o + (static_cast<long>(r) * p.nh + h) * p.splits * vd;
+  for (int d = threadIdx.x; d < vd; d += blockDim.x) {
     float acc = 0.f;
     for (int s = 0; s < p.splits; ++s)
-      if (ml[2 * s] != -CUDART_INF_F) acc += wo[s * VD + d] * exp2f(ml[2 * s] - m);
+      if (ml[2 * s] != -CUDART_INF_F) acc += wo[s * vd + d] * exp2f(ml[2 * s] - m);
     out[d] = Mma<T>::from_f(acc * inv);
   }
 }
@@ -430,34 +464,53 @@ extern "C" int fi_mla_prepare(const void* kva, long ldkva, const void* norm_w, f
   return static_cast<int>(cudaGetLastError());
 }
 
-// ws_o: rows * nh * splits * 512 floats, ws_ml: rows * nh * splits * 2 floats (splits > 1 only).
+namespace {
+
+template <typename T, int KDT, int VB>
+int launch_decode(const MlaParams& p, int rows, cudaStream_t s) {
+  const int pitch = KDT > 0 ? KDT : p.pitch;
+  const int smem = (CH * pitch + 16 * pitch + 16 * CH) * 2 + 4 * 16 * 4;
+  auto kern = mla_decode_kernel<T, KDT, VB>;
+  cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
+  if (ce != cudaSuccess) return static_cast<int>(ce);
+  fi::launch_kernel(kern, dim3(p.splits, (p.nh + 15) / 16, rows), dim3(128), smem, s, 0, p);
+  if (p.splits > 1) fi::launch_kernel(mla_merge_kernel<T>, dim3(p.nh, rows), dim3(128), 0, s, 0, p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+int dispatch_decode(const MlaParams& p, int rows, cudaStream_t s) {
+  if (p.kd == KD && p.vd == VD) return launch_decode<T, KD, VD / 64>(p, rows, s);
+  if (p.vd <= 64) return launch_decode<T, 0, 1>(p, rows, s);
+  if (p.vd <= 128) return launch_decode<T, 0, 2>(p, rows, s);
+  if (p.vd <= 256) return launch_decode<T, 0, 4>(p, rows, s);
+  return launch_decode<T, 0, 8>(p, rows, s);
+}
+
+}  // namespace
+
+// Attention of flattened rows over the shared cache rows [latent (vd) | rotary key] of kd values.
+// ws_o: rows * nh * splits * vd floats, ws_ml: rows * nh * splits * 2 floats (splits > 1 only).  window <= 0: none;
+// sinks: fp32 [nh] or null.  Returns -12 for a geometry the kernel does not cover (the caller takes the general one).
 extern "C" int fi_mla_decode(const void* q_cat, const void* cache, void* out, long out_head_stride,
                              long out_row_stride, const int* block_tables, const int* row_lens, const int* seq_of_row,
-                             float* ws_o, float* ws_ml, int rows, int nh, int max_blocks, int block_size, int splits,
-                             float sm_scale, int dtype, void* stream) {
+                             float* ws_o, float* ws_ml, int rows, int nh, int kd, int vd, int max_blocks, int block_size,
+                             int splits, int window, const float* sinks, float sm_scale, int dtype, void* stream) {
   if (rows <= 0 || nh <= 0) return 0;
-  if (splits < 1 || block_size <= 0 || (splits > 1 && (ws_o == nullptr || ws_ml == nullptr))) return -10;
+  if (splits < 1 || block_size <= 0 || (splits > 1 && (ws_o == nullptr || ws_ml == nullptr)) || vd > kd) return -10;
+  if (kd % 8 != 0 || vd % 2 != 0 || vd <= 0 || vd > 512 || kd > 640 || rows > 65535) return -12;
   if ((reinterpret_cast<uintptr_t>(q_cat) | reinterpret_cast<uintptr_t>(cache)) & 15) return -10;
-  if (out_head_stride % 2 != 0 || out_row_stride % 2 != 0) return -10;
+  if (out_head_stride % 2 != 0 || out_row_stride % 2 != 0) return -12;
   MlaParams p = {};
   p.q_cat = q_cat; p.cache = cache; p.out = out; p.out_head_stride = out_head_stride; p.out_row_stride = out_row_stride;
   p.block_tables = block_tables; p.row_lens = row_lens; p.seq_of_row = seq_of_row; p.ws_o = ws_o; p.ws_ml = ws_ml;
   p.nh = nh; p.max_blocks = max_blocks; p.block_size = block_size; p.splits = splits; p.sm_scale = sm_scale;
-  const int smem = (CH * KD + 16 * KD + 16 * CH) * 2 + 4 * 16 * 4;
-  const dim3 grid(splits, (nh + 15) / 16, rows);
+  p.window = window; p.sinks = sinks; p.kd = kd; p.vd = vd;
+  const int vcols = vd <= 64 ? 64 : vd <= 128 ? 128 : vd <= 256 ? 256 : 512;
+  const int kcols = (kd + 15) / 16 * 16;
+  p.pitch = (kcols > vcols ? kcols : vcols) + 8;
   cudaStream_t s = FI_STREAM(stream);
-  if (dtype == 0) {
-    cudaError_t ce = fi::ensure_dynamic_smem(mla_decode_kernel<__nv_bfloat16>, smem);
-    if (ce != cudaSuccess) return static_cast<int>(ce);
-    fi::launch_kernel(mla_decode_kernel<__nv_bfloat16>, grid, dim3(128), smem, s, 0, p);
-    if (splits > 1) fi::launch_kernel(mla_merge_kernel<__nv_bfloat16>, dim3(nh, rows), dim3(128), 0, s, 0, p);
-  } else if (dtype == 1) {
-    cudaError_t ce = fi::ensure_dynamic_smem(mla_decode_kernel<__half>, smem);
-    if (ce != cudaSuccess) return static_cast<int>(ce);
-    fi::launch_kernel(mla_decode_kernel<__half>, grid, dim3(128), smem, s, 0, p);
-    if (splits > 1) fi::launch_kernel(mla_merge_kernel<__half>, dim3(nh, rows), dim3(128), 0, s, 0, p);
-  } else {
-    return -11;
-  }
-  return static_cast<int>(cudaGetLastError());
+  if (dtype == 0) return dispatch_decode<__nv_bfloat16>(p, rows, s);
+  if (dtype == 1) return dispatch_decode<__half>(p, rows, s);
+  return -11;
 }

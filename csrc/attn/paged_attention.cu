@@ -114,6 +114,10 @@ struct AttnParams {
   // partials through distributed shared memory at this byte offset of the dynamic shared memory
   // ([16][HD] sums + [16][2] max/denominator per CTA): no global scratch, no tickets, no second launch
   int cluster_off;
+  // prefill: fp32 [nh] or null, one extra exp(sink) per head in the softmax denominator; channels of a head
+  // that are stored (0 = HD)
+  const float* sinks;
+  int out_dim;
 };
 
 // Load `rows` KV tokens starting at token tok0 of sequence b / kv head kvh into a swizzled tile.
@@ -827,18 +831,25 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   cp_async_wait<0>();
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  if (p.sinks != nullptr) {
+    const float sink = p.sinks[head];
+    if (m0 != -CUDART_INF_F) l0 += exp2f((sink - m0) * kLog2e);
+    if (m1 != -CUDART_INF_F) l1 += exp2f((sink - m1) * kLog2e);
+  }
   const float vs = p.kv_fp8 == 1 ? p.v_scale : 1.f;
   const float i0 = l0 > 0.f ? vs / l0 : 0.f, i1 = l1 > 0.f ? vs / l1 : 0.f;
   T* out = reinterpret_cast<T*>(p.out);
+  const int od = p.out_dim > 0 ? p.out_dim : HD;
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) {
     const int d = i * 8 + (lane & 3) * 2;
+    if (d >= od) break;
     if (row0 < q_len) {
-      const long off = (static_cast<long>(q_begin + row0) * p.nh + head) * HD + d;
+      const long off = (static_cast<long>(q_begin + row0) * p.nh + head) * od + d;
       *reinterpret_cast<uint32_t*>(out + off) = MmaT<T>::pack(o[i][0] * i0, o[i][1] * i0);
     }
     if (row0 + 8 < q_len) {
-      const long off = (static_cast<long>(q_begin + row0 + 8) * p.nh + head) * HD + d;
+      const long off = (static_cast<long>(q_begin + row0 + 8) * p.nh + head) * od + d;
       *reinterpret_cast<uint32_t*>(out + off) = MmaT<T>::pack(o[i][2] * i1, o[i][3] * i1);
     }
   }
@@ -1057,7 +1068,7 @@ extern "C" int fi_paged_prefill(const void* q, long q_stride, const void* k_cach
                                 const int* seq_lens, const int* cu_q, int B, int max_q_len, int nh,
                                 int nkv, int hd, int max_blocks, int block_size, int window,
                                 float sm_scale, float softcap, int kv_fp8, float k_scale,
-                                float v_scale, int dtype, void* stream) {
+                                float v_scale, const float* sinks, int out_dim, int dtype, void* stream) {
   if (B <= 0 || max_q_len <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0) return -10;
   AttnParams p = {};
@@ -1065,6 +1076,8 @@ extern "C" int fi_paged_prefill(const void* q, long q_stride, const void* k_cach
   p.block_tables = block_tables; p.seq_lens = seq_lens; p.cu_q = cu_q; p.max_blocks = max_blocks;
   p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window; p.sm_scale = sm_scale;
   p.softcap = softcap; p.k_scale = k_scale; p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = 1;
+  if (out_dim < 0 || out_dim > hd || out_dim % 2 != 0) return -10;
+  p.sinks = sinks; p.out_dim = out_dim;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == 0) {
     if (hd == 64) return launch_prefill<__nv_bfloat16, 64, 64>(p, B, max_q_len, s);

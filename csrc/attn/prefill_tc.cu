@@ -33,7 +33,9 @@ namespace {
 using namespace fi;
 
 struct TcParams {
-  void* out;                 // [T, nh * HD]
+  void* out;                 // [T, nh * out_dim]
+  const float* sinks;        // [nh] or null: one extra exp(sink) per head in the softmax denominator
+  int out_dim;               // output channels per head that are stored (<= HD)
   const int* block_tables;   // [B, max_blocks]
   const int* seq_lens;       // [B]
   const int* cu_q;           // [B + 1]
@@ -389,12 +391,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       half_sum[half * 128 + row] = l;
       ok = pair_sync();
       l += half_sum[(half ^ 1) * 128 + row];
+      if (p.sinks != nullptr) l += fast_exp2(fmaf(p.sinks[head], kLog2e, -m));   // every row sees at least its own key
       if (row < rows && ok) {
         const float inv = l > 0.f ? 1.f / l : 0.f;
         uint16_t* dst = reinterpret_cast<uint16_t*>(p.out) +
-                        (static_cast<long>(q_begin + qt0 + row) * p.nh + head) * HD + half * HH;
+                        (static_cast<long>(q_begin + qt0 + row) * p.nh + head) * p.out_dim + half * HH;
 #pragma unroll
         for (int c = 0; c < HH / 8; ++c) {
+          if (half * HH + c * 8 >= p.out_dim) break;
           uint4 v;
           v.x = pack2(o[c * 8 + 0] * inv, o[c * 8 + 1] * inv, p.is_fp16);
           v.y = pack2(o[c * 8 + 2] * inv, o[c * 8 + 3] * inv, p.is_fp16);
@@ -445,14 +449,16 @@ extern "C" int fi_paged_prefill_tc_set_trace(void* trace) {
 // a multiple of 128 tokens (larger pages mean fewer, larger TMA boxes per tile).  Returns -12 when the arguments are outside what this kernel covers (the caller then uses
 // the general kernel), other negative values for malformed arguments.
 //   q: token t, head h at q + (t * q_stride + h * hd) elements, T_total rows; caches [num_blocks, nkv,
-//   block_size, hd]; out [T_total, nh * hd].
+//   block_size, hd]; out [T_total, nh * out_dim] (out_dim <= hd, a multiple of 8: the leading channels of each
+//   head); sinks: fp32 [nh] or null.
 extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_cache, const void* v_cache, void* out,
                                    const int* block_tables, const int* seq_lens, const int* cu_q, int B,
                                    int T_total, int max_q_len, int nh, int nkv, int hd, long num_blocks,
                                    int max_blocks, int block_size, int window, float sm_scale, float softcap,
-                                   int dtype, int* status, void* stream) {
+                                   const float* sinks, int out_dim, int dtype, int* status, void* stream) {
   if (B <= 0 || max_q_len <= 0 || T_total <= 0) return 0;
-  if (nkv <= 0 || nh <= 0 || nh % nkv != 0) return -10;
+  if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || out_dim <= 0 || out_dim > hd) return -10;
+  if (out_dim % 8 != 0) return -12;
   if ((hd != 64 && hd != 128) || (dtype != 0 && dtype != 1)) return -12;
   if (block_size != 16 && block_size != 32 && block_size != 64 && block_size % 128 != 0) return -12;
   if ((reinterpret_cast<uintptr_t>(q) & 15) != 0 || (q_stride * 2) % 16 != 0 ||
@@ -466,7 +472,7 @@ extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_c
     return -12;
   TcParams p = {};
   p.out = out; p.block_tables = block_tables; p.seq_lens = seq_lens; p.cu_q = cu_q; p.status = status;
-  p.trace = g_tc_trace;
+  p.trace = g_tc_trace; p.sinks = sinks; p.out_dim = out_dim;
   p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window;
   p.sm_scale = sm_scale; p.softcap = softcap; p.is_fp16 = dtype == 1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);

@@ -232,7 +232,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
     asm volatile("bar.sync 1, 128;" ::: "memory");   // the four warps: row_ss complete before it is used
   }
   // ---------------------------------------------------------------- epilogue (epilogue.cuh)
-  if (warp >= 2) epilogue_tmem_to_smem<BN, DUAL>(p, accum_bar, tmem_base, stage_f32, aborted, warp, lane, row_ss);
+  if (warp >= 2) epilogue_tmem_to_smem<BN, DUAL>(p, accum_bar, tmem_base, stage_f32, aborted, warp, lane, row_ss, n0);
   __syncthreads();
   epilogue_reduce_store<BN, DUAL>(p, stage_f32, aborted, n0, t0, epoch_now, p.T, row_ss);
   __syncthreads();

@@ -9,7 +9,7 @@
 // one-tile-per-CTA kernel pays in full; here it overlaps the next main loop.
 //
 //   C[T, N] = act(X[T, K] W[N, K]^T) + bias + residual           (dual_rows == 0)
-//   C[T, I] = act(X Wg^T) * (X Wu^T)   with W = [Wg; Wu]          (dual_rows == I)
+//   C[T, I] = act(X Wg^T + bg) * (X Wu^T + bu)   with W = [Wg; Wu], bias = [bg; bu]   (dual_rows == I)
 //
 // Warp roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer and TMEM owner, warps 2..5 epilogue.
 // Barriers: full/empty per pipeline stage (running across tiles), acc_full/acc_empty per accumulator.
@@ -42,7 +42,7 @@ struct PParams {
   const void* bias;
   const void* residual;
   int T, N, K, ldc;
-  int dual_rows, act, is_fp16;
+  int dual_rows, act, is_fp16, out_fp32;
   int second_off;   // weight rows between the two A tiles of a CTA: dual_rows (gated) or 128 (plain, 256-row tile)
   int rows_per_tile;   // output rows (of N) one tile covers: 128 (gated or single) or 256
   int n_tiles_n, n_tiles;
@@ -55,6 +55,7 @@ __device__ __forceinline__ float act_f(float g, int act) {
     const float inner = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return g / (1.f + __expf(-2.f * inner));
   }
+  if (act == 3) return fmaxf(g, 0.f);
   return g;
 }
 __device__ __forceinline__ float ld16(const void* p, size_t i, int is_fp16) {
@@ -201,12 +202,17 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
       const int vj = lane >> 2;               // tokens vj and vj + 8 of the batch
       // gated: one output row per thread (gate and up combined); plain wide tile: two rows, 128 apart
       const int halves = (DUAL && !gated) ? 2 : 1;
+      float bias_g = 0.f, bias_u = 0.f;       // gated: bias of this thread's weight row in either half
+      if (DUAL && gated && p.bias != nullptr && n0 + n_local < p.N) {
+        bias_g = ld16(p.bias, n0 + n_local, p.is_fp16);
+        bias_u = ld16(p.bias, p.dual_rows + n0 + n_local, p.is_fp16);
+      }
       for (int hh = 0; hh < halves; ++hh) {
         const int nv = n0 + hh * BM + q * 32 + vc * 8;      // first of the 8 rows this lane stores
         const bool nv_ok = nv < p.N;
         float bias8[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) bias8[e] = (p.bias != nullptr && nv_ok) ? ld16(p.bias, nv + e, p.is_fp16) : 0.f;
+        for (int e = 0; e < 8; ++e) bias8[e] = (p.bias != nullptr && nv_ok && !gated) ? ld16(p.bias, nv + e, p.is_fp16) : 0.f;
         // the residual values of a batch are requested one batch ahead, so their latency hides behind
         // the TMEM read and the transposition of the batch in front
         auto load_res = [&](int c0, uint4 (&dst)[2]) {
@@ -231,7 +237,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             float v = __uint_as_float(r[j]);
-            if (DUAL && gated) v = act_f(v, p.act) * __uint_as_float(u[j]);
+            if (DUAL && gated) v = act_f(v + bias_g, p.act) * (__uint_as_float(u[j]) + bias_u);
             else v = act_f(v, p.act);
             patch[j * 32 + lane] = v;
           }
@@ -245,6 +251,12 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
               const float4 a1 = *reinterpret_cast<const float4*>(patch + j * 32 + vc * 8 + 4);
               float v[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
               const size_t off = static_cast<size_t>(t) * p.ldc + nv;
+              if (p.out_fp32) {               // 32-bit output (no residual in this form)
+                float4* dst = reinterpret_cast<float4*>(reinterpret_cast<float*>(p.C) + off);
+                dst[0] = make_float4(v[0] + bias8[0], v[1] + bias8[1], v[2] + bias8[2], v[3] + bias8[3]);
+                dst[1] = make_float4(v[4] + bias8[4], v[5] + bias8[5], v[6] + bias8[6], v[7] + bias8[7]);
+                continue;
+              }
               const uint4 raw = res_cur[rep];
               const uint32_t rw[4] = {raw.x, raw.y, raw.z, raw.w};
               uint32_t ow[4];
@@ -305,16 +317,18 @@ int launch(const CUtensorMap& tw, const CUtensorMap& tx, const PParams& p, cudaS
 }  // namespace
 
 // Prefill-sized dense GEMM (see the top of the file).  dtype: 0 bf16, 1 fp16 for X, W, bias, residual and
-// C.  dual_rows > 0: gated mode, W holds [gate rows; up rows] and N must equal dual_rows.  Nothing is
+// C (C is 32-bit with out_fp32, which takes no residual).  dual_rows > 0: gated mode, W holds [gate rows; up
+// rows], bias (if any) [gate bias; up bias] and N must equal dual_rows.  Nothing is
 // allocated; returns 0, a negative argument error or a positive CUDA error code.
 extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, const void* bias, const void* residual,
                                         int T, int N, int K, int ldx, int ldw, int ldc, int act, int dual_rows,
-                                        int dtype, int* status, void* stream) {
+                                        int out_fp32, int dtype, int* status, void* stream) {
   if (T <= 0 || N <= 0 || K <= 0) return 0;
   if ((K % 8) != 0 || (ldx % 8) != 0 || (ldw % 8) != 0 || (N % 8) != 0 || (ldc % 8) != 0 ||
       (reinterpret_cast<uintptr_t>(C) & 15) != 0 || (residual != nullptr && (reinterpret_cast<uintptr_t>(residual) & 15) != 0))
     return -10;
   if (dual_rows > 0 && N != dual_rows) return -11;
+  if (out_fp32 && residual != nullptr) return -13;
   const int w_rows = dual_rows > 0 ? 2 * dual_rows : N;
   CUtensorMap tw, tx;
   int r = make_tmap_2d_16bit_sw128(&tw, W, w_rows, K, ldw, BM);
@@ -324,7 +338,7 @@ extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, c
   PParams p;
   p.C = C; p.bias = bias; p.residual = residual;
   p.T = T; p.N = N; p.K = K; p.ldc = ldc;
-  p.dual_rows = dual_rows; p.act = act; p.is_fp16 = dtype == 1;
+  p.dual_rows = dual_rows; p.act = act; p.is_fp16 = dtype == 1; p.out_fp32 = out_fp32;
   // plain products use a 256-row tile (two A tiles per stage against one token tile), which halves the
   // L2 -> shared-memory traffic per FLOP; 128 x 128 tiles were L2-bandwidth-bound at ~55 % of peak
   const bool wide = dual_rows == 0 && N > BM;

@@ -34,12 +34,12 @@ constexpr int kXferTwoShot = 3;      // all-reduce in two hops: partials go to t
 constexpr int kPhasePush = 1, kPhaseReduce = 2, kPhaseCollect = 4;
 constexpr int kMaxCommTiles = 8192; // tiles per call that the flag area can describe
 
-enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2 };
+enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2, kActRelu = 3 };
 enum CommMode : int { kCommNone = 0, kCommAllReduce = 1, kCommReduceScatter = 2 };
 
 struct GemmParams {
   void* C;
-  const void* bias;      // [N] or null (same 16-bit type as X)
+  const void* bias;      // [N] or null (same 16-bit type as X); gated mode: [2 * dual_rows], added before the activation
   const void* residual;  // [T, ldc] or null (same type as C when C is 16-bit)
   int T, N, K;
   int ldc;
@@ -111,6 +111,7 @@ __device__ __forceinline__ float apply_act(float g, int act) {
     const float inner = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return g / (1.f + __expf(-2.f * inner));
   }
+  if (act == kActRelu) return fmaxf(g, 0.f);
   return g;
 }
 
@@ -195,7 +196,7 @@ __device__ __forceinline__ void unpack8(const uint4 raw, int is_fp16, float* g) 
 // Bias + residual + store of 8 consecutive outputs of token row `trow` (row index in C).
 __device__ __forceinline__ void finalize_store8(const GemmParams& p, float* g, int trow, int n) {
   const int nvalid = min(8, p.N - n);
-  if (p.bias != nullptr) {
+  if (p.bias != nullptr && p.dual_rows == 0) {
     for (int j = 0; j < nvalid; ++j) g[j] += ld16_as_float(p.bias, n + j, p.is_fp16);
   }
   const size_t off = static_cast<size_t>(trow) * p.ldc + n;
@@ -354,7 +355,7 @@ template <int BN, bool DUAL>
 __device__ __forceinline__ void epilogue_tmem_to_smem(const GemmParams& p, uint64_t* accum_bar,
                                                       uint32_t tmem_base, float* stage_f32,
                                                       volatile int* aborted, int warp, int lane,
-                                                      const float* row_ss = nullptr) {
+                                                      const float* row_ss = nullptr, int gate_row0 = 0) {
   bool ok = mbar_wait(accum_bar, 0);
   if (!ok) {
     set_status(p.status, kStatusTimeoutAccum);
@@ -369,6 +370,11 @@ __device__ __forceinline__ void epilogue_tmem_to_smem(const GemmParams& p, uint6
     const bool fuse_act_now = DUAL && (p.splits == 1);
     const bool norm_now = p.rms_eps > 0.f && p.splits == 1;   // with split-K the scale is applied after the sum
     const float inv_k = 1.f / static_cast<float>(p.K);
+    float bias_g = 0.f, bias_u = 0.f;                          // gated mode: this thread's weight row of each half
+    if (DUAL && p.bias != nullptr && gate_row0 + n_local < p.dual_rows) {
+      bias_g = ld16_as_float(p.bias, gate_row0 + n_local, p.is_fp16);
+      bias_u = ld16_as_float(p.bias, p.dual_rows + gate_row0 + n_local, p.is_fp16);
+    }
 #pragma unroll 1
     for (int c0 = 0; c0 < BN; c0 += 16) {
       uint32_t r[16];
@@ -392,7 +398,7 @@ __device__ __forceinline__ void epilogue_tmem_to_smem(const GemmParams& p, uint6
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             stage_f32[(c0 + j) * BM + n_local] =
-                apply_act(__uint_as_float(r[j]), p.act) * __uint_as_float(u[j]);
+                apply_act(__uint_as_float(r[j]) + bias_g, p.act) * (__uint_as_float(u[j]) + bias_u);
         } else {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -471,7 +477,14 @@ __device__ __forceinline__ void epilogue_reduce_store(const GemmParams& p, float
       }
       if (DUAL && S > 1) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) g[j] = apply_act(g[j], p.act) * u[j];
+        for (int j = 0; j < 8; ++j) {
+          float bg = 0.f, bu = 0.f;
+          if (p.bias != nullptr && n + j < p.N) {
+            bg = ld16_as_float(p.bias, n + j, p.is_fp16);
+            bu = ld16_as_float(p.bias, p.dual_rows + n + j, p.is_fp16);
+          }
+          g[j] = apply_act(g[j] + bg, p.act) * (u[j] + bu);
+        }
       } else if (!DUAL && p.act != kActNone && !comm) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) g[j] = apply_act(g[j], p.act);

@@ -65,6 +65,45 @@ def _compile_one(src: Path, cmd_prefix: list[str], flags: list[str], verbose: bo
     return obj
 
 
+# Kernel sources one model family needs (beside nothing else): a fresh checkout that serves only that family compiles
+# these into a library of their own instead of everything.
+KERNEL_SETS = {
+    "fimodra": ["attn/latent_rows.cu", "attn/mla_decode.cu", "attn/paged_attention.cu", "attn/prefill_tc.cu",
+                "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "linear_attn/hgrn2.cu",
+                "misc/norm_rope_misc.cu", "misc/residual_stream.cu", "misc/sampling.cu"],
+}
+
+
+def set_library(name: str) -> Path:
+    return PKG_DIR / f"libfi_kernels_{name}.so"
+
+
+def full_library_is_current() -> bool:
+    """The full library exists and every kernel source has an object of its present content."""
+    if not KERNEL_LIB.exists():
+        return False
+    objs = [BUILD_DIR / (str(s.relative_to(CSRC)).replace("/", "_") + "." + _stamp(s, NVCC_FLAGS) + ".o")
+            for s in CSRC.rglob("*.cu")]
+    return all(o.exists() and o.stat().st_mtime <= KERNEL_LIB.stat().st_mtime for o in objs)
+
+
+def build_set(name: str, verbose: bool = True) -> Path:
+    """Compile the kernels of one family and link them on their own.  Nothing is done when they are current."""
+    BUILD_DIR.mkdir(parents=True, exist_ok=True)
+    srcs = [CSRC / s for s in KERNEL_SETS[name]]
+    with cf.ThreadPoolExecutor(max_workers=max(1, min(len(srcs), os.cpu_count() or 1))) as ex:
+        objs = list(ex.map(lambda s: _compile_one(s, [_nvcc()], NVCC_FLAGS, verbose), srcs))
+    lib = set_library(name)
+    if not lib.exists() or lib.stat().st_mtime < max(o.stat().st_mtime for o in objs):
+        tmp = lib.with_suffix(f".{os.getpid()}.tmp")
+        res = subprocess.run([_nvcc(), "-shared", "-o", str(tmp)] + [str(o) for o in objs] +
+                             ["-gencode", "arch=compute_100a,code=sm_100a"], capture_output=True, text=True)
+        if res.returncode != 0:
+            raise RuntimeError(f"link failed: {res.stdout}\n{res.stderr}")
+        os.replace(tmp, lib)
+    return lib
+
+
 def build_all(verbose: bool = True, force: bool = False) -> dict[str, Path]:
     BUILD_DIR.mkdir(parents=True, exist_ok=True)
     if force:

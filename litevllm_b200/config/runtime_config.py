@@ -31,6 +31,7 @@ class RuntimeConfig:
     kv_max_model_len: int | None
     kv_max_active_requests: int
     kv_max_active_requests_explicit: bool
+    kv_pool_tokens: int
     fusion_level: int
     policy_mode: str
     enable_decode_priority: bool
@@ -122,6 +123,7 @@ class RuntimeConfig:
             kv_max_model_len=_int("KV_MAX_MODEL_LEN", profile.kv_max_model_len),
             kv_max_active_requests=_int("KV_MAX_ACTIVE_REQUESTS", profile.kv_max_active_requests),
             kv_max_active_requests_explicit=explicit_active or profile.kv_max_active_requests != 4,
+            kv_pool_tokens=_int("KV_POOL_TOKENS", 0),
             fusion_level=_int("FUSION_LEVEL", profile.fusion_level), policy_mode=policy_mode,
             enable_decode_priority=_flag("LITE_DECODE_PRIORITY", profile.enable_decode_priority),
             prefill_chunk_size=_int("LITE_PREFILL_CHUNK", profile.prefill_chunk_size),

@@ -17,7 +17,7 @@ from .errors import ExecutionStepError
 from .executors import TokenDecodeResult, TokenPrefillResult
 from .request_state import RequestState
 from .sampling_driver import SamplingDriver
-from .step_plan import StepPlan
+from .step_plan import PrefillItem, StepPlan
 
 
 class LiteGpuBackend:
@@ -39,6 +39,9 @@ class LiteGpuBackend:
         self.pipeline = None
         self.pipelined_steps = 0
         self.async_decode = getattr(backend_policy, "async_decode", True)
+        # the model takes portions of prompts and decoded tokens in one forward pass
+        self.mixed_batches = bool(getattr(getattr(prefill_executor, "model", None), "supports_mixed_batch", False))
+        self.mixed_steps = 0
 
     # ------------------------------------------------------------------ KV growth
     def ensure_kv_blocks(self, plan: StepPlan) -> None:
@@ -103,6 +106,8 @@ class LiteGpuBackend:
                 items.append(it)
         if not items:
             return outs
+        if self.mixed_batches:
+            items.sort(key=lambda it: -it.chunk_len)       # long portions first: attention splits a step by length
         t0 = time.perf_counter()
         try:
             lora_map = self.lora_registry.mapping_for_prefill(items, states) if self.lora_registry else None
@@ -129,6 +134,67 @@ class LiteGpuBackend:
                 outs.append(self._process_completion(st, tok))
         self.observer.on_prefill_executed(len(items), sum(i.chunk_len for i in items), time.perf_counter() - t0)
         return outs
+
+    def run_mixed(self, plan: StepPlan) -> list:
+        """One forward pass for the step's portions of prompts and its decoding requests."""
+        states = self.scheduler.requests
+        outs = self.drain_pipeline()
+        items = sorted((it for it in plan.prefills if it.chunk_len > 0), key=lambda it: -it.chunk_len)
+        reqs = [states[r] for r in plan.decodes if r in states and not states[r].finished]
+        n_prompt = len(items)
+        for st in reqs:
+            self._flush_pending(st)
+            items.append(PrefillItem(st.request_id, st.seq_len, 1))
+        if not items:
+            return outs
+        t0 = time.perf_counter()
+        try:
+            res = self.prefill_executor.execute(items, states)
+        except Exception as e:
+            raise ExecutionStepError(f"mixed step failed: {e!r}") from e
+        done_reqs, done_rows = [], []
+        for row, it in enumerate(items):
+            st = states[it.request_id]
+            st.seq_len = it.end
+            if st.is_prefill and st.seq_len < st.prompt_len:
+                continue
+            st.is_prefill = False
+            done_reqs.append(st)
+            done_rows.append(row)
+        if done_reqs:
+            rows = res.logits if len(done_rows) == len(items) else res.logits[done_rows]
+            for st, tok in zip(done_reqs, self._sample(rows, done_reqs)):
+                outs.append(self._process_completion(st, tok))
+        self.mixed_steps += 1
+        dt = time.perf_counter() - t0
+        if n_prompt:
+            self.observer.on_prefill_executed(n_prompt, sum(i.chunk_len for i in items[:n_prompt]), dt)
+        if reqs:
+            self.observer.on_decode_executed(len(reqs), dt)
+        return [o for o in outs if o is not None]
+
+    def run_given_tokens(self, items: list, want: list) -> "torch.Tensor | None":
+        """One step over tokens that were given rather than sampled: the same executors as generation, logits of the
+        wanted offsets of each item in the items' order (None when nothing is wanted)."""
+        states = self.scheduler.requests
+        order = sorted(range(len(items)), key=lambda i: -items[i].chunk_len)
+        run = [items[i] for i in order]
+        total = sum(len(w) for w in want)
+        if all(it.chunk_len == 1 and it.start > 0 for it in run):
+            logits = self.decode_executor.execute_batch([states[it.request_id] for it in run], states).logits
+            rows_of = {i: [r] if want[i] else [] for r, i in enumerate(order)}
+        else:
+            logits = self.prefill_executor.execute(run, states, want=[want[i] for i in order]).logits
+            rows_of, r = {}, 0
+            for i in order:
+                rows_of[i] = list(range(r, r + len(want[i])))
+                r += len(want[i])
+        for it in run:
+            states[it.request_id].seq_len = it.end
+        if not total:
+            return None
+        rows = [r for i in range(len(items)) for r in rows_of[i]]
+        return logits.index_select(0, torch.tensor(rows, device=logits.device)).float()
 
     # ------------------------------------------------------------------ pipelined decode
     def _pipeline_ok(self, reqs, plan: StepPlan) -> bool:
@@ -300,7 +366,7 @@ class LiteGpuBackend:
 
     def stats(self) -> dict:
         return {"kv": self.kv.stats(), "greedy_device_steps": self.greedy_device_steps,
-                "pipelined_decode_steps": self.pipelined_steps,
+                "pipelined_decode_steps": self.pipelined_steps, "mixed_steps": self.mixed_steps,
                 "graph_replays": getattr(self.decode_executor, "graph_replays", 0),
                 "eager_decode_steps": getattr(self.decode_executor, "eager_steps", 0),
                 "prefix_cache": self.prefix_cache.stats() if self.prefix_cache else {"enabled": False},

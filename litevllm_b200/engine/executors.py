@@ -42,9 +42,19 @@ class PrefillExecutor:
         self.model, self.kv_cache, self.builder, self.multimodal = model, kv_cache, builder, multimodal
 
     @torch.inference_mode()
-    def execute(self, items: list[PrefillItem], states: dict[str, RequestState], lora_mapping=None) -> LogitsResult:
+    def execute(self, items: list[PrefillItem], states: dict[str, RequestState], lora_mapping=None,
+                want: list[list[int]] | None = None) -> LogitsResult:
+        """``want``: per item the offsets of the tokens whose logits are asked for (default: the last token of each);
+        rows of the result follow the items and, within an item, its offsets."""
         batch = self.builder.build_prefill(items, states)
         batch.lora_mapping = lora_mapping
+        if want is not None:
+            rows, off = [], 0
+            for it, offsets in zip(items, want):
+                rows += [off + o for o in offsets]
+                off += it.chunk_len
+            # at least one row, so that an empty request for logits needs no special case in the models
+            batch.logits_indices = torch.tensor(rows or [0], dtype=torch.int64, device=self.builder.device)
         embeds = None
         if self.multimodal is not None:
             embeds = self.multimodal.embed_for_prefill(self.model, batch, items, states)

@@ -101,6 +101,7 @@ class InputBatchBuilder:
 
     # ------------------------------------------------------------------ prefill
     def build_prefill(self, items: list[PrefillItem], states: dict[str, RequestState]) -> ForwardBatch:
+        """A varlen batch of portions; an item may also be the single next token of a decoding request."""
         B = len(items)
         T = sum(it.chunk_len for it in items)
         if T > self._cap:
@@ -118,7 +119,7 @@ class InputBatchBuilder:
         for i, it in enumerate(items):
             st = states[it.request_id]
             n = it.chunk_len
-            ids[off:off + n] = st.prompt_token_ids[it.start:it.end]
+            ids[off:off + n] = st.token_span(it.start, it.end)
             pos_h[off:off + n] = np.arange(it.start, it.end, dtype=np.int32)
             slot_h[off:off + n] = self._slots_for(self.kv.blocks_of(it.request_id), it.start, n)
             off += n

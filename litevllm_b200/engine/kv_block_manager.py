@@ -24,6 +24,7 @@ class KVBlockManager:
         self.kv_cache = kv_cache
         self._blocks: dict[str, list[int]] = {}
         self._slot_of: dict[str, int] = {}
+        self._reserved: dict[str, int] = {}      # shared pool: blocks a request may come to hold
         pin = device.type == "cuda"
         self.host_table = torch.zeros(max_active, blocks_per_seq, dtype=torch.int32, pin_memory=pin)
         self.block_tables = torch.zeros(max_active, blocks_per_seq, dtype=torch.int32, device=device)
@@ -38,6 +39,14 @@ class KVBlockManager:
 
     def can_grow(self, request_id: str, num_tokens: int) -> bool:
         return self.allocator.can_allocate(self.num_blocks_needed(request_id, num_tokens))
+
+    def reserve(self, request_id: str, num_tokens: int) -> bool:
+        """Set the blocks of ``num_tokens`` tokens aside for a request; False when they could be needed by others."""
+        need = min(cdiv(num_tokens, self.block_size), self.blocks_per_seq)
+        if sum(self._reserved.values()) + need > self.allocator.num_blocks - 1:
+            return False
+        self._reserved[request_id] = need
+        return True
 
     # ------------------------------------------------------------------ lifecycle
     def register(self, request_id: str, slot_idx: int) -> None:
@@ -66,6 +75,7 @@ class KVBlockManager:
     def release(self, request_id: str) -> None:
         blocks = self._blocks.pop(request_id, None)
         slot = self._slot_of.pop(request_id, None)
+        self._reserved.pop(request_id, None)
         if blocks:
             self.allocator.free(blocks)
         if slot is not None:

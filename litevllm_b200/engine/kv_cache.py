@@ -10,6 +10,7 @@ contiguous ``block_size x head_dim`` tile for bulk loads).
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 
 import torch
@@ -22,10 +23,15 @@ class KVLayerSpec:
     num_kv_heads: int
     head_dim: int
     v_head_dim: int | None = None     # MLA-style caches may use another width for V (0 = no V)
+    state_shape: tuple | None = None  # recurrent layers: shape of the fp32 state a request slot owns
 
     @property
     def v_dim(self) -> int:
         return self.head_dim if self.v_head_dim is None else self.v_head_dim
+
+    @property
+    def state_bytes(self) -> int:
+        return 4 * math.prod(self.state_shape) if self.state_shape else 0
 
 
 def kv_torch_dtype(kv_cache_dtype: str, model_dtype: torch.dtype) -> torch.dtype:
@@ -57,7 +63,10 @@ def bytes_per_block(specs: list[KVLayerSpec], block_size: int, dtype: torch.dtyp
 
 class FlatKVCache:
     def __init__(self, specs: list[KVLayerSpec], num_blocks: int, block_size: int,
-                 dtype: torch.dtype, device: torch.device, fmt: int = 0):
+                 dtype: torch.dtype, device: torch.device, fmt: int = 0, num_slots: int = 0):
+        """``num_slots``: request slots of the engine; recurrent layers (``state_shape``) get one fp32 state per slot
+        in ``states[layer]``.  A slot's state is not cleared when it changes hands: a sequence that starts at
+        position 0 starts from a zero state."""
         self.specs, self.num_blocks, self.block_size = specs, num_blocks, block_size
         self.dtype, self.device, self.fmt = dtype, device, fmt
         e = dtype_nbytes(dtype)
@@ -87,6 +96,11 @@ class FlatKVCache:
                     self.scale_bytes += t.fi_scales.numel() * 4
             self.layers.append((k, v))
         self.total_bytes += self.scale_bytes
+        self.states: list[torch.Tensor | None] = [
+            torch.zeros(num_slots, *s.state_shape, dtype=torch.float32, device=device) if s.state_shape else None
+            for s in specs]
+        self.state_bytes = sum(t.numel() * 4 for t in self.states if t is not None)
+        self.total_bytes += self.state_bytes
 
     def __getitem__(self, i: int):
         return self.layers[i]

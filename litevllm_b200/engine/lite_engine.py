@@ -24,8 +24,10 @@ from .errors import EngineFatalError, InvalidRequestError, RequestAbortedError, 
 from .initialization import LiteRuntimeAssembler, MemoryAuditor
 from .observer import InMemoryRuntimeObserver
 from .request_builder import LiteRequestBuilder
+from .request_state import RequestState
 from .runtime_factory import LiteRuntimeFactory
 from .runtime_planner import RuntimePlanner
+from .step_plan import PrefillItem, StepPlan
 
 logger = init_logger(__name__)
 
@@ -179,6 +181,37 @@ class LiteEngine:
             if self.pre_step_hook is not None:
                 self.pre_step_hook()
             return self.controller.step()
+
+    @torch.inference_mode()
+    def replay_step(self, entries: list, end: list = ()):
+        """Run one step over given tokens instead of sampled ones.  ``entries``: ``(request id, tokens, wanted offsets)``;
+        a request is admitted at its first entry and keeps its slot, blocks and state until it is named in ``end``.  All
+        entries form one batch.  Returns the wanted logits, fp32 [wanted, vocab] in the order of the entries, or None."""
+        with self.lock:
+            items, want = [], []
+            for rid, tokens, offsets in entries:
+                st = self.scheduler.get(rid)
+                if st is None:
+                    st = RequestState(rid, None, [], SamplingParams(temperature=0.0, max_tokens=1))
+                    self.scheduler.enqueue_request(st)
+                    self.scheduler.admit(rid)
+                    self.backend.register_admitted(st)
+                bad = [t for t in tokens if not 0 <= t < self.arch.vocab_size]
+                if bad or any(not 0 <= o < len(tokens) for o in offsets):
+                    raise InvalidRequestError(f"request {rid}: token or wanted offset out of range")
+                if not tokens:
+                    continue
+                items.append(PrefillItem(rid, st.seq_len, len(tokens)))
+                want.append(list(offsets))
+                st.prompt_token_ids.extend(tokens)
+            logits = None
+            if items:
+                self.backend.ensure_kv_blocks(StepPlan(prefills=items))
+                logits = self.backend.run_given_tokens(items, want)
+            for rid in end:
+                self.backend.release_request(rid)
+                self.scheduler.pop_sync_outputs(rid)
+            return logits
 
     def handle_background_error(self, exc: BaseException) -> None:
         """Fatal: every stream gets the exception, every request is released, admission closes."""

@@ -65,5 +65,12 @@ class RequestState:
     def total_len(self) -> int:
         return self.prompt_len + self.num_generated
 
+    def token_span(self, start: int, end: int) -> list[int]:
+        """Tokens [start, end) of prompt and generated text (device-resident tokens must have been flushed)."""
+        n = self.prompt_len
+        if end <= n:
+            return self.prompt_token_ids[start:end]
+        return self.prompt_token_ids[start:n] + self.generated_ids[max(0, start - n):end - n]
+
     def last_token(self) -> int:
         return self.generated_ids[-1] if self.generated_ids else self.prompt_token_ids[-1]

@@ -67,6 +67,8 @@ class RuntimeController:
         self.steps += 1
         if plan.fast_path and len(plan.decodes) == 1:
             return self.backend.decode_step_sync(plan.decodes[0])
+        if plan.prefills and plan.decodes and getattr(self.backend, "mixed_batches", False):
+            return self.backend.run_mixed(plan)
         outs = self.backend.run_prefills(plan)
         outs += self.backend.run_decodes(plan)
         return outs

@@ -46,7 +46,7 @@ class LiteRuntimeFactory:
     def build(ctx: RuntimeAssemblyContext) -> RuntimeComponents:
         plan, rc, custom = ctx.plan, ctx.runtime_config, ctx.custom
         kv_cache = FlatKVCache(ctx.kv_specs, plan.num_total_blocks, plan.block_size, ctx.kv_plan.dtype, ctx.device,
-                               fmt=getattr(ctx.kv_plan, "fmt", 0))
+                               fmt=getattr(ctx.kv_plan, "fmt", 0), num_slots=plan.max_active_requests)
         allocator = BlockAllocator(plan.num_total_blocks)
         kv_manager = KVBlockManager(allocator, plan.block_size, plan.max_active_requests, plan.num_blocks_per_seq,
                                     ctx.device, kv_cache)
@@ -72,8 +72,11 @@ class LiteRuntimeFactory:
             plan.step_token_budget, plan.prefill_chunk_size, plan.prefill_microbatch, rc.scheduler_policy,
             rc.enable_decode_priority, rc.prefill_catchup_ratio, rc.prefill_reserved_tokens,
             rc.prefill_reserve_backlog, rc.min_prefill_chunk_size, rc.max_prefill_chunk_size,
-            ctx.model_policy.verified_decode_batch_sizes, plan.max_active_requests)
-        prefix_cache = PrefixCache(rc.backend_policy.max_prefix_cache_entries, rc.backend_policy.max_prefix_cache_bytes)
+            ctx.model_policy.verified_decode_batch_sizes, plan.max_active_requests,
+            kv_manager=kv_manager if plan.shared_pool else None)
+        has_state = any(s.state_shape for s in ctx.kv_specs)      # recurrent state is not part of cached blocks
+        prefix_cache = PrefixCache(0 if has_state else rc.backend_policy.max_prefix_cache_entries,
+                                   rc.backend_policy.max_prefix_cache_bytes)
         sampling_driver = SamplingDriver(ctx.arch.vocab_size)
         output_pipeline = OutputPipeline(None, plan.max_model_len, GenerationPolicies())
         backend = LiteGpuBackend(scheduler, kv_manager, prefill_executor, decode_executor, sampling_driver,

@@ -5,7 +5,8 @@ Differences from the reference planner (vllm/engine/runtime_planner.py:56-158): 
 4096 is kept as the *default* but an explicit ``kv_max_model_len`` / ``max_model_len`` can raise it;
 slot count defaults to 16 on large-memory GPUs and can be raised up to ``max_num_seqs`` because a
 B200 has room for far more than 16 contexts; KV capacity is still ``1 + slots * blocks_per_seq``
-(every admitted request is guaranteed its whole context, no preemption).
+(every admitted request is guaranteed its whole context, no preemption) unless ``kv_pool_tokens`` asks for a smaller
+pool that the requests share; admission then reserves the blocks a request can come to need.
 """
 from __future__ import annotations
 
@@ -29,6 +30,7 @@ class ExecutionPlan:
     step_token_budget: int
     prefill_chunk_size: int
     prefill_microbatch: int
+    shared_pool: bool = False     # the pool is smaller than slots x context: admission reserves blocks per request
 
 
 @dataclass(frozen=True)
@@ -68,8 +70,11 @@ class RuntimePlanner:
             chunk = min(chunk, rc.max_prefill_chunk_size)
         chunk = max(rc.min_prefill_chunk_size, chunk)
         budget = max(rc.max_num_batched_tokens, active)
-        return ExecutionPlan(block_size=bs, max_model_len=max_len, max_active_requests=active,
-                             num_blocks_per_seq=per_seq, num_total_blocks=1 + active * per_seq,
+        total, shared = active * per_seq, False
+        if rc.kv_pool_tokens and cdiv(rc.kv_pool_tokens, bs) < total:
+            total, shared = max(per_seq, cdiv(rc.kv_pool_tokens, bs)), True
+        return ExecutionPlan(block_size=bs, max_model_len=max_len, max_active_requests=active, shared_pool=shared,
+                             num_blocks_per_seq=per_seq, num_total_blocks=1 + total,
                              step_token_budget=budget, prefill_chunk_size=chunk,
                              prefill_microbatch=max(1, rc.prefill_microbatch_size))
 
@@ -81,5 +86,6 @@ class RuntimePlanner:
         if fmt == 3 and any(s.head_dim % 32 or s.v_dim % 32 for s in specs if s.num_kv_heads > 0):
             name, dt, fmt = "fp8", kv_torch_dtype("fp8", model_dtype), 1      # odd head widths cannot be nibble-packed
         total = bytes_per_block(specs, plan.block_size, dt, fmt) * plan.num_total_blocks
+        total += plan.max_active_requests * sum(s.state_bytes for s in specs)
         return KVCachePlan(dtype=dt, dtype_name=name, k_scale=self.rc.k_scale, v_scale=self.rc.v_scale,
                            bytes_total=total, fmt=fmt)

@@ -17,7 +17,8 @@ class StepScheduler:
                  policy: SchedulerRuntimePolicy | None = None, decode_priority: bool = True,
                  catchup_ratio: float = 0.25, reserved_tokens: int = 0, reserve_backlog: int = 2,
                  min_chunk: int = 128, max_chunk: int | None = None,
-                 verified_decode_batch_sizes: tuple[int, ...] | None = None, max_active: int = 16):
+                 verified_decode_batch_sizes: tuple[int, ...] | None = None, max_active: int = 16, kv_manager=None):
+        self.kv_manager = kv_manager      # set when requests share a pool smaller than slots x context
         self.policy = policy or SchedulerRuntimePolicy()
         self.admission = AdmissionPlanner(min(self.policy.max_admit_per_step, max_active) if max_active < 8
                                           else max(self.policy.max_admit_per_step, max_active))
@@ -36,6 +37,12 @@ class StepScheduler:
                 return StepPlan(decodes=[st.request_id], step_token_budget=self.budget.step_token_budget,
                                 fast_path=True, metrics={"fast_path": True})
         admissions = self.admission.plan(sched.queued, len(sched.free_slots))
+        if self.kv_manager is not None:   # first come, first served: the first request that does not fit stops admission
+            for i, rid in enumerate(admissions):
+                st = sched.requests[rid]
+                if not self.kv_manager.reserve(rid, st.prompt_len + int(st.sampling_params.max_tokens or 0)):
+                    admissions = admissions[:i]
+                    break
         prefill, decode = sched.classify_requests()
         # requests admitted this step start prefilling in the same step
         admitted_states = [sched.requests[r] for r in admissions]

@@ -63,7 +63,8 @@ class LiteLinear(nn.Module):
             return self.quant_method.apply(self, x, residual=residual, out=out, out_dtype=out_dtype,
                                            use_bias=use_bias)
         if self.gated_act is not None:
-            return ops.gated_linear(x, self.weight, self.gated_act, out=out, rms_eps=norm_eps)
+            return ops.gated_linear(x, self.weight, self.gated_act, out=out, rms_eps=norm_eps,
+                                    bias=self.bias if use_bias else None)
         return ops.linear(x, self.weight, self.bias if use_bias else None, residual, out=out,
                           out_dtype=out_dtype, rms_eps=norm_eps)
 

@@ -219,3 +219,48 @@ def iter_qwen35_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, dev
             yield p + "mlp.up_proj.weight", w(p + "u", I, H)
             yield p + "mlp.down_proj.weight", w(p + "d", H, I)
     yield "lm_head.weight", w("lm_head", V, H)
+
+
+def iter_fimodra_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, device="cpu") -> Iterator[tuple[str, torch.Tensor]]:
+    """Linear weights ~ N(0, 1 / fan-in); norms near one; sinks, gate biases, lower bounds and depth averages spread so
+    that each of them matters."""
+    W, V = arch.hidden_size, arch.vocab_size
+
+    def lin(name, out_f, in_f):
+        return name, normal(name, (out_f, in_f), seed, in_f ** -0.5, dtype, device)
+
+    def vec(name, n, base=0.0, std=1.0):
+        return name, base + normal(name, (n,), seed, std, torch.float32, device)
+
+    yield "embed", normal("embed", (V, W), seed, 1.0, dtype, device)
+    for i, l in enumerate(arch.extra["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        H = m["heads"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if l.get("mlp") else ()):
+            yield vec(p + n, W, 1.0, 0.1)
+        if l["type"] == "latent_attention":
+            yield lin(p + "mix.q", H * (m["dim"] + m["rot_dim"]), W)
+            yield lin(p + "mix.dkv", m["kv_rank"] + m["rot_dim"], W)
+            yield vec(p + "mix.dkv.norm", m["kv_rank"], 1.0, 0.1)
+            yield lin(p + "mix.uk", H * m["dim"], m["kv_rank"])
+            yield lin(p + "mix.uv", H * m["vdim"], m["kv_rank"])
+            yield vec(p + "mix.sink", H, 1.0, 1.0)
+            yield lin(p + "mix.o", W, H * m["vdim"])
+        else:
+            yield lin(p + "mix.q", H * m["dim"], W)
+            yield lin(p + "mix.f", H * m["dim"], W)
+            yield vec(p + "mix.f.b", H * m["dim"], 2.0, 2.0)
+            yield p + "mix.lower", torch.sigmoid(normal(p + "mix.lower", (H * m["dim"],), seed, 1.5, torch.float32, device)) * 0.9
+            yield lin(p + "mix.v", H * m["vdim"], W)
+            yield vec(p + "mix.norm", m["vdim"], 1.0, 0.1)
+            yield lin(p + "mix.o", W, H * m["vdim"])
+        if l.get("mlp"):
+            ff = l["mlp"]["ff"]
+            for n, o, k in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+                yield lin(p + f"mlp.{n}", o, k)
+                yield vec(p + f"mlp.{n}.b", o, 0.0, 0.1)
+        a = normal(p + "dwa", (i + 2,), seed, 0.3, torch.float32, device)
+        a[-1] += 1.0
+        yield p + "dwa", a
+    yield vec("final.norm", W, 1.0, 0.1)
+    yield lin("head", V, W)

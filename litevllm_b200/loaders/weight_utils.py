@@ -83,6 +83,32 @@ def load_mapped(param_map: dict, weights: Iterable[tuple[str, torch.Tensor]], st
     return consumed
 
 
+def load_exact(dest: dict, weights: Iterable[tuple[str, torch.Tensor]]) -> set[str]:
+    """Fill destinations by full checkpoint name: a parameter, or ``(LiteLinear, piece, "weight" | "bias")``.  Shapes
+    must match; a tensor without a destination and a destination without a tensor are both errors."""
+    seen: set[str] = set()
+    for name, tensor in weights:
+        d = dest.get(name)
+        if d is None:
+            raise KeyError(f"no destination for checkpoint tensor {name!r}")
+        if isinstance(d, tuple):
+            lin, piece, which = d
+            want = (lin.out_splits[piece], lin.full_in) if which == "weight" else (lin.out_splits[piece],)
+        else:
+            want = tuple(d.shape)
+        if tuple(tensor.shape) != tuple(want):
+            raise ValueError(f"checkpoint tensor {name!r} has shape {tuple(tensor.shape)}, the configuration asks for {tuple(want)}")
+        if isinstance(d, tuple):
+            lin.load_piece(piece, tensor, which)
+        else:
+            d.data.copy_(tensor.to(d.dtype))
+        seen.add(name)
+    missing = sorted(set(dest) - seen)
+    if missing:
+        raise KeyError(f"checkpoint lacks {len(missing)} tensors, e.g. {missing[:4]}")
+    return seen
+
+
 def load_llama_style(model, weights) -> set[str]:
     consumed = load_mapped(llama_param_map(model), weights)
     finalize_quantized(model)

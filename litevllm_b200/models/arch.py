@@ -41,7 +41,7 @@ class MLASpec:
 
 @dataclass
 class ModelArch:
-    family: str                      # llama | qwen2 | qwen3_5 | gemma4 | deepseek_mla | qwen2_vl
+    family: str                      # llama | qwen2 | qwen3_5 | gemma4 | deepseek_mla | qwen2_vl | fimodra
     architecture: str
     hidden_size: int
     num_layers: int
@@ -122,8 +122,50 @@ def _quant_from_hf(cfg: dict) -> QuantSpec:
     return QuantSpec()
 
 
+def _sizes(entry: dict, names: tuple, where: str) -> None:
+    for n in names:
+        if not isinstance(entry.get(n), int) or entry[n] <= 0:
+            raise ValueError(f"{where}: {n!r} must be a positive integer, got {entry.get(n)!r}")
+
+
+def arch_from_fimodra_config(cfg: dict) -> ModelArch:
+    """Fimodra configurations list their layers one by one (mixer type and sizes, feed-forward or null)."""
+    layers = cfg["layers"]
+    if not layers:
+        raise ValueError("the configuration lists no layers")
+    for i, l in enumerate(layers):
+        m, where = l["mixer"], f"layers[{i}]"
+        if l["type"] == "latent_attention":
+            _sizes(m, ("heads", "dim", "rot_dim", "vdim", "kv_rank"), where)
+            dims = (m.get("rot") or {}).get("dims", m["rot_dim"])
+            if dims % 2 or dims > m["rot_dim"]:
+                raise ValueError(f"{where}: cannot rotate {dims} of {m['rot_dim']} dimensions")
+        elif l["type"] == "hgrn2":
+            _sizes(m, ("heads", "dim", "vdim"), where)
+        else:
+            raise ValueError(f"{where}: unknown mixer {l['type']!r}")
+        if l.get("mlp"):
+            _sizes(l["mlp"], ("ff",), where)
+    width, groups = int(cfg["width"]), int(cfg["norm"].get("groups", 1))
+    if width % groups:
+        raise ValueError(f"a width of {width} does not split into {groups} equal parts")
+    heads = max(l["mixer"]["heads"] for l in layers)
+    arch = ModelArch(
+        family="fimodra", architecture="Fimodra", hidden_size=width, num_layers=len(layers), num_heads=heads,
+        num_kv_heads=1, head_dim=max(l["mixer"]["dim"] for l in layers),
+        intermediate_size=max((l["mlp"]["ff"] for l in layers if l.get("mlp")), default=0),
+        vocab_size=int(cfg["vocab"]), rms_eps=float(cfg["norm"]["eps"]), act="relu",
+        max_position=int(cfg.get("max_position_embeddings", 1 << 20)), eos_token_ids=_eos_list(cfg),
+        bos_token_id=cfg.get("bos_token_id"))
+    arch.layer_types = ["linear" if l["type"] == "hgrn2" else "sliding" for l in layers]
+    arch.extra.update(layers=layers, norm_groups=groups)
+    return arch
+
+
 def arch_from_hf_config(cfg: dict) -> ModelArch:
     """Build a :class:`ModelArch` from a HF config dict (text sub-config is unwrapped)."""
+    if str(cfg.get("architecture", "")).lower() == "fimodra":
+        return arch_from_fimodra_config(cfg)
     archs = cfg.get("architectures") or ["LlamaForCausalLM"]
     architecture = archs[0]
     text = cfg.get("text_config") or cfg

@@ -130,7 +130,8 @@ class MLAAttention(nn.Module):
         out_lat = torch.empty(nh, T, self.kv_lora, dtype=x.dtype, device=x.device)
         rc = lib.fi_mla_decode(_p(q_cat), _p(cache), _p(out_lat), out_lat.stride(0), out_lat.stride(1),
                                _p(batch.block_tables), _p(row_lens), _p(seq_of_row), _p(ws_o), _p(ws_ml), rows, nh,
-                               batch.block_tables.shape[1], bs, splits, self.sm_scale, dt, _stream())
+                               self.kv_lora + self.rope, self.kv_lora, batch.block_tables.shape[1], bs, splits, 0, None,
+                               self.sm_scale, dt, _stream())
         _lib.check(rc, "fi_mla_decode")
         _count(3 if splits > 1 else 2)
         o = torch.bmm(out_lat, w[:, nope:, :].transpose(1, 2))                      # [nh, T, vd]

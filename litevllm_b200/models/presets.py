@@ -127,6 +127,24 @@ PRESETS["tiny-qwen2vl-test"] = dict(PRESETS["tiny-llama-test"], architectures=["
                                     rope_scaling={"type": "mrope", "mrope_section": [16, 8, 8]})
 
 
+def fimodra_config(width: int, vocab: int, ff: int, pattern: str, heads: int, dim: int, rot_dim: int, vdim: int,
+                   kv_rank: int, window: int, lin_heads: int, lin_dim: int, lin_vdim: int, groups: int = 4,
+                   rot_base: float = 10000.0) -> dict:
+    """Fimodra configuration from a layer pattern: "a" latent attention, "h" HGRN2, upper case without a feed-forward."""
+    attn = {"dim": dim, "heads": heads, "kv_rank": kv_rank, "mask": {"size": window},
+            "rot": {"base": rot_base, "dims": rot_dim}, "rot_dim": rot_dim, "scale": (dim + rot_dim) ** -0.5, "vdim": vdim}
+    lin = {"dim": lin_dim, "heads": lin_heads, "vdim": lin_vdim}
+    layers = [{"type": "latent_attention" if c in "aA" else "hgrn2", "mixer": copy.deepcopy(attn if c in "aA" else lin),
+               "mlp": {"kind": "dense", "ff": ff} if c.islower() else None} for c in pattern]
+    return {"architecture": "Fimodra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6, "groups": groups},
+            "layers": layers}
+
+
+PRESETS["tiny-fimodra-test"] = fimodra_config(256, 512, 192, "ahHaA", 3, 24, 8, 40, 80, 20, 5, 32, 24)
+# layers of the width and head geometry of a 1B-class decoder
+PRESETS["fimodra-1b"] = fimodra_config(2048, 32000, 5632, "aaha" * 5, 16, 96, 32, 128, 512, 1024, 16, 128, 128, groups=2)
+
+
 def get_preset(name: str) -> dict:
     key = name.lower()
     if key not in PRESETS:

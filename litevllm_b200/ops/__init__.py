@@ -15,7 +15,7 @@ import torch
 
 from . import _lib, reference
 
-_ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "gelu": 2}
+_ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "gelu": 2, "relu": 3}
 _DT = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
 
 _status_words: dict[int, torch.Tensor] = {}
@@ -140,6 +140,19 @@ def _rms_scaled(x, eps):
     return (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps)).to(x.dtype)
 
 
+def _needs_plain_product(x, w) -> bool:
+    """The TMA operand loads want rows of whole 16-byte groups on 16-byte addresses."""
+    return (x.shape[1] % 8 != 0 or x.stride(0) % 8 != 0 or w.stride(0) % 8 != 0
+            or x.data_ptr() % 16 != 0 or w.data_ptr() % 16 != 0)
+
+
+def _plain_product(x, w) -> torch.Tensor:
+    """``x @ w.T`` in true 32-bit arithmetic (vendor product, no reduced-precision matrix mode)."""
+    if torch.backends.cuda.matmul.allow_tf32:
+        torch.backends.cuda.matmul.allow_tf32 = False
+    return x.float() @ w.float().t()
+
+
 def linear(x, w, bias=None, residual=None, act=None, out=None, out_dtype=None, splits=0, bn=0, rms_eps=0.0,
            static_weight=True):
     """``act(x @ w.T) + bias + residual``.  x: [T, K], w: [N, K] (same 16-bit dtype).  With
@@ -165,15 +178,13 @@ def linear(x, w, bias=None, residual=None, act=None, out=None, out_dtype=None, s
     if T == 0:
         return out
     assert x.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
-    if out.stride(0) % 8 != 0 or K % 8 != 0 or out.data_ptr() % 16 != 0:
-        # shapes the tensor-core kernel does not take (a caller-provided narrow output, odd K): plain matmul
-        y = x.float() @ w.float().t()
-        if rms_eps > 0:
-            y = _rms_scaled(x, rms_eps).float() @ w.float().t()
-        if bias is not None:
-            y = y + bias.float()
+    if x.dtype == torch.float32 or _needs_plain_product(x, w) or out.stride(0) % 8 != 0 or out.data_ptr() % 16 != 0:
+        # 32-bit models, and shapes the tensor-core kernel does not take (a caller-provided narrow output, odd K)
+        y = _plain_product(x if rms_eps <= 0 else _rms_scaled(x, rms_eps), w)
         if act:
             y = reference.apply_act(y, act)
+        if bias is not None:
+            y = y + bias.float()
         if residual is not None:
             y = y + residual.float()
         out.copy_(y)
@@ -194,11 +205,13 @@ def linear(x, w, bias=None, residual=None, act=None, out=None, out_dtype=None, s
         _lib.check(rc, "fi_dense_gemm_rmsnorm")
         _count()
         return out
-    if _PERSISTENT_PLAIN and T >= _PERSISTENT_MIN_T and splits == 0 and bn == 0 and out.dtype == x.dtype and N % 8 == 0:
+    wide_out = out.dtype == torch.float32
+    if _PERSISTENT_PLAIN and T >= _PERSISTENT_MIN_T and splits == 0 and bn == 0 and N % 8 == 0 \
+            and (not wide_out or residual is None):
         # prefill-sized: persistent CTAs with two TMEM accumulators (epilogue overlaps the next main loop)
         rc = _lib.kernels().fi_dense_gemm_persistent(
             _p(x), _p(w), _p(out), _p(bias), _p(residual), T, N, K, x.stride(0), w.stride(0), out.stride(0),
-            _ACT[act], 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
+            _ACT[act], 0, 1 if wide_out else 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
         _lib.check(rc, "fi_dense_gemm_persistent")
         _count()
         return out
@@ -244,13 +257,13 @@ def linear_rope_cache(x, w, bias, positions, cos_sin, slot_mapping, k_cache, v_c
     return out
 
 
-def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0):
-    """``act(x @ Wg.T) * (x @ Wu.T)`` with ``w_gate_up = [Wg; Wu]`` of shape [2*I, K] -> [T, I]
-    (``rms_eps > 0``: rows of ``x`` RMS-normalised inside the kernel)."""
+def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0, bias=None):
+    """``act(x @ Wg.T + bg) * (x @ Wu.T + bu)`` with ``w_gate_up = [Wg; Wu]`` of shape [2*I, K] and the optional
+    ``bias = [bg; bu]`` -> [T, I] (``rms_eps > 0``: rows of ``x`` RMS-normalised inside the kernel)."""
     if not x.is_cuda:
         if rms_eps > 0:
             x = _rms_scaled(x, rms_eps)
-        y = reference.gated_linear(x, w_gate_up, act)
+        y = reference.gated_linear(x, w_gate_up, act, bias=bias)
         if out is not None:
             out.copy_(y)
             return out
@@ -258,24 +271,30 @@ def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0
     T, K = x.shape
     inter = w_gate_up.shape[0] // 2
     if out is None:
-        out = torch.empty(T, inter, dtype=x.dtype, device=x.device)
+        out = torch.empty(T, (inter + 7) // 8 * 8, dtype=x.dtype, device=x.device)[:, :inter]
     if T == 0:
+        return out
+    if x.dtype == torch.float32 or _needs_plain_product(x, w_gate_up) or out.stride(0) % 8 != 0 or out.data_ptr() % 16 != 0:
+        y = _plain_product(x if rms_eps <= 0 else _rms_scaled(x, rms_eps), w_gate_up)
+        if bias is not None:
+            y = y + bias.float()
+        out.copy_(reference.apply_act(y[:, :inter], act) * y[:, inter:])
         return out
     if rms_eps <= 0 and _PERSISTENT_GEMM and T >= _PERSISTENT_MIN_T and splits == 0 and bn == 0 and inter % 8 == 0:
         rc = _lib.kernels().fi_dense_gemm_persistent(
-            _p(x), _p(w_gate_up), _p(out), None, None, T, inter, K, x.stride(0), w_gate_up.stride(0), out.stride(0),
-            _ACT[act], inter, _DT[x.dtype], _p(status_word(x.device)), _stream())
+            _p(x), _p(w_gate_up), _p(out), _p(bias), None, T, inter, K, x.stride(0), w_gate_up.stride(0), out.stride(0),
+            _ACT[act], inter, 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
         _lib.check(rc, "fi_dense_gemm_persistent(gated)")
         _count()
         return out
     if rms_eps > 0:
         rc = _lib.kernels().fi_dense_gemm_rmsnorm(
-            _p(x), _p(w_gate_up), _p(out), None, None, T, inter, K, x.stride(0), w_gate_up.stride(0),
+            _p(x), _p(w_gate_up), _p(out), _p(bias), None, T, inter, K, x.stride(0), w_gate_up.stride(0),
             out.stride(0), _ACT[act], inter, 0, _DT[x.dtype], splits, bn, float(rms_eps),
             _p(status_word(x.device)), _stream())
     else:
         rc = _lib.kernels().fi_dense_gemm(
-            _p(x), _p(w_gate_up), _p(out), None, None, T, inter, K, x.stride(0), w_gate_up.stride(0),
+            _p(x), _p(w_gate_up), _p(out), _p(bias), None, T, inter, K, x.stride(0), w_gate_up.stride(0),
             out.stride(0), _ACT[act], inter, 0, _DT[x.dtype], splits, bn,
             _p(status_word(x.device)), _stream())
     _lib.check(rc, "fi_dense_gemm(gated)")
@@ -533,11 +552,16 @@ def paged_metadata_snapshot(q, k_cache, block_tables, seq_lens, cu_q=None, scope
 
 
 def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv,
-                            hd, sm_scale, window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None):
-    """Varlen causal attention of new tokens against the paged cache (which already holds them)."""
+                            hd, sm_scale, window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, sinks=None,
+                            v_dim=None):
+    """Varlen causal attention of new tokens against the paged cache (which already holds them).  ``sinks`` (fp32
+    [nh]): a number per head whose exponential joins the softmax denominator.  ``v_dim``: only the leading ``v_dim``
+    channels of a head's output exist (rows of nh * v_dim)."""
+    od = hd if v_dim is None else int(v_dim)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_prefill", block_tables, seq_lens, k_cache, cu_q)
     if not q.is_cuda:
+        assert sinks is None and od == hd, "the CPU form of sinks and narrow outputs lives in ops.latent_attn"
         y = reference.paged_attention(q, k_cache, v_cache, block_tables, seq_lens, cu_q, nh, nkv, hd,
                                       sm_scale, window, softcap, k_scale, v_scale)
         if out is not None:
@@ -547,13 +571,14 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
     T = q.shape[0]
     B = seq_lens.shape[0]
     if out is None:
-        out = torch.empty(T, nh * hd, dtype=q.dtype, device=q.device)
+        out = torch.empty(T, nh * od, dtype=q.dtype, device=q.device)
     elif not out.is_contiguous():
         tmp = paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv, hd,
-                                      sm_scale, window, softcap, k_scale, v_scale, None)
+                                      sm_scale, window, softcap, k_scale, v_scale, None, sinks, v_dim)
         out.copy_(tmp)
         return out
     mode = reference.kv_mode(k_cache)
+    assert mode < 2 or (sinks is None and od == hd), "row-scaled caches take no sinks and no narrow outputs"
     if mode >= 2:
         rc = _lib.kernels().fi_paged_prefill_rowscaled(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(k_cache.fi_scales), _p(v_cache.fi_scales), _p(out),
@@ -568,7 +593,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         rc = _lib.kernels().fi_paged_prefill_tc(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens), _p(cu_q), B, T,
             int(max_q_len), nh, nkv, hd, k_cache.shape[0], block_tables.shape[1], k_cache.shape[2], int(window or 0),
-            sm_scale, float(softcap or 0.0), _DT[q.dtype], _p(status_word(q.device)), _stream())
+            sm_scale, float(softcap or 0.0), _p(sinks), od, _DT[q.dtype], _p(status_word(q.device)), _stream())
         if rc != -12:       # -12: outside what the tensor-core kernel covers, take the general one
             _lib.check(rc, "fi_paged_prefill_tc")
             _count()
@@ -577,7 +602,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
         _p(cu_q), B, int(max_q_len), nh, nkv, hd, block_tables.shape[1], k_cache.shape[2],
         int(window or 0), sm_scale, float(softcap or 0.0),
-        1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, _DT[q.dtype], _stream())
+        1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, _p(sinks), od, _DT[q.dtype], _stream())
     _lib.check(rc, "fi_paged_prefill")
     _count()
     return out

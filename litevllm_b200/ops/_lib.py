@@ -71,9 +71,20 @@ def declare(lib, name: str, codes: str, restype=ctypes.c_int):
     return fn
 
 
+_kernel_path = _C_DIR / "libfi_kernels.so"
+
+
+def use_kernel_library(path) -> None:
+    """Bind another kernel library (a family's own set) before the first kernel call of the process."""
+    global _kernel_path
+    if kernels.cache_info().currsize:
+        raise RuntimeError("the kernel library is already loaded")
+    _kernel_path = Path(path)
+
+
 @lru_cache(maxsize=None)
 def kernels():
-    path = _C_DIR / "libfi_kernels.so"
+    path = _kernel_path
     if not path.exists():
         raise NativeLibraryMissing(
             f"{path} not found: run `python -m litevllm_b200._C.build` (or __graft_entry__.build())")

@@ -129,3 +129,89 @@ def conv1d_step(x: torch.Tensor, pool: torch.Tensor, slots: torch.Tensor, w: tor
     _lib.check(rc, "fi_conv1d_step")
     _count()
     return y
+
+
+# ---------------------------------------------------------------------------- HGRN2
+def _hgrn2_gates(q, f, f_bias, lower):
+    """fp32 activated query, write strength 1 - forget gate: [n, H * d] each."""
+    z = f.float() + f_bias
+    return F.silu(q.float()), (1.0 - lower) * torch.sigmoid(-z)
+
+
+def _hgrn2_tokens(q, k, v, S):
+    """q, k: fp32 [L, H, d] (activated query, write strength), v: fp32 [L, H, dv], S: fp32 [H, d, dv], updated in
+    place.  Returns o fp32 [L, H, dv]."""
+    o = torch.empty(q.shape[0], v.shape[1], v.shape[2], dtype=torch.float32, device=q.device)
+    for t in range(q.shape[0]):
+        S.mul_((1.0 - k[t])[:, :, None]).add_(k[t][:, :, None] * v[t][:, None, :])
+        o[t] = torch.einsum("hkv,hk->hv", S, q[t])
+    return o
+
+
+def hgrn2_scan(q, f, v, f_bias, lower, pool, slots, cu_q, seq_lens, H: int, d: int, dv: int):
+    """Portions of sequences: ``f_t = l + (1 - l) sigmoid(z_t + b)``, ``S = diag(f) S + (1 - f) v^T``, ``o = S^T silu(q)``.
+
+    q, f [T, H * d] and v [T, H * dv]: projection outputs (any row pitch; q and v share a dtype).  f_bias, lower: fp32
+    [H * d].  pool: fp32 [num_slots, H, d, dv], updated in place; slots, seq_lens: int32 [B]; cu_q: int32 [B + 1].  A
+    portion as long as its sequence starts from a zero state.  Returns o fp32 [T, H, dv]."""
+    T, B = q.shape[0], slots.shape[0]
+    o = torch.empty(T, H, dv, dtype=torch.float32, device=q.device)
+    if not q.is_cuda:
+        qa, ka = _hgrn2_gates(q, f, f_bias, lower)
+        cu, lens = cu_q.tolist(), seq_lens.tolist()
+        for b, s in enumerate(slots.tolist()):
+            lo, hi = cu[b], cu[b + 1]
+            if hi <= lo:
+                continue
+            S = pool[s]
+            if lens[b] == hi - lo:
+                S.zero_()
+            o[lo:hi] = _hgrn2_tokens(qa[lo:hi].view(-1, H, d), ka[lo:hi].view(-1, H, d),
+                                     v[lo:hi].float().reshape(-1, H, dv), S)
+        return o
+    assert q.dtype == v.dtype and q.stride(1) == f.stride(1) == v.stride(1) == 1
+    assert pool.dtype == torch.float32 and pool.is_contiguous() and slots.dtype == torch.int32 == cu_q.dtype
+    rc = _lib.kernels().fi_hgrn2_scan(_p(q), q.stride(0), _p(f), f.stride(0), _p(v), v.stride(0), _p(f_bias), _p(lower),
+                                      _p(pool), _p(slots), _p(cu_q), _p(seq_lens), _p(o), B, H, d, dv, pool.shape[0],
+                                      _DT[q.dtype], _DT[f.dtype], _stream())
+    _lib.check(rc, "fi_hgrn2_scan")
+    _count()
+    return o
+
+
+def head_norm(o, w, eps: float, out_dtype):
+    """RMS norm of every head's row: o fp32 [T, H, dv], w fp32 [dv] -> [T, H * dv]."""
+    T, H, dv = o.shape
+    if not o.is_cuda:
+        y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w
+        return y.reshape(T, H * dv).to(out_dtype)
+    out = torch.empty(T, H * dv, dtype=out_dtype, device=o.device)
+    rc = _lib.kernels().fi_head_norm(_p(o), _p(w), _p(out), T * H, dv, eps, _DT[out_dtype], _stream())
+    _lib.check(rc, "fi_head_norm")
+    _count()
+    return out
+
+
+def hgrn2_step(q, f, v, f_bias, lower, pool, slots, seq_lens, norm_w, eps: float, H: int, d: int, dv: int, out_dtype):
+    """One token per sequence, head norm included: same operands as :func:`hgrn2_scan`.  Rows with ``seq_lens`` <= 0
+    are padding (zero output, no state touched).  Returns [B, H * dv]."""
+    B = slots.shape[0]
+    if not q.is_cuda:
+        qa, ka = _hgrn2_gates(q, f, f_bias, lower)
+        o = torch.zeros(B, H, dv, dtype=torch.float32)
+        for b, (s, n) in enumerate(zip(slots.tolist(), seq_lens.tolist())):
+            if n <= 0 or s < 0:
+                continue
+            if n == 1:
+                pool[s].zero_()
+            o[b] = _hgrn2_tokens(qa[b:b + 1].view(1, H, d), ka[b:b + 1].view(1, H, d), v[b:b + 1].float().reshape(1, H, dv),
+                                 pool[s])[0]
+        return head_norm(o, norm_w, eps, out_dtype)
+    assert q.dtype == v.dtype and pool.dtype == torch.float32 and pool.is_contiguous()
+    out = torch.empty(B, H * dv, dtype=out_dtype, device=q.device)
+    rc = _lib.kernels().fi_hgrn2_step(_p(q), q.stride(0), _p(f), f.stride(0), _p(v), v.stride(0), _p(f_bias), _p(lower),
+                                      _p(pool), _p(slots), _p(seq_lens), _p(norm_w), eps, _p(out), B, H, d, dv,
+                                      pool.shape[0], _DT[q.dtype], _DT[f.dtype], _DT[out_dtype], _stream())
+    _lib.check(rc, "fi_hgrn2_step")
+    _count()
+    return out

@@ -23,6 +23,8 @@ def apply_act(x: torch.Tensor, act: str | None) -> torch.Tensor:
         return F.silu(x)
     if act in ("gelu_tanh", "gelu_pytorch_tanh", "gelu"):
         return F.gelu(x, approximate="tanh")
+    if act == "relu":
+        return F.relu(x)
     raise ValueError(f"unknown activation {act}")
 
 
@@ -37,9 +39,11 @@ def linear(x, w, bias=None, residual=None, act=None, out_dtype=None):
     return y.to(out_dtype or x.dtype)
 
 
-def gated_linear(x, w_gate_up, act="silu", out_dtype=None):
+def gated_linear(x, w_gate_up, act="silu", out_dtype=None, bias=None):
     inter = w_gate_up.shape[0] // 2
     y = x.float() @ w_gate_up.float().t()
+    if bias is not None:
+        y = y + bias.float()
     return (apply_act(y[:, :inter], act) * y[:, inter:]).to(out_dtype or x.dtype)
 
 

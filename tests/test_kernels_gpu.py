@@ -771,7 +771,8 @@ def test_mla_absorbed_decode_kernel(nh, splits):
     ws_ml = torch.empty(rows * nh * splits * 2, dtype=torch.float32, device=dev) if splits > 1 else None
     scale = 192 ** -0.5
     rc = _lib.kernels().fi_mla_decode(_p(q), _p(cache), _p(out), out.stride(0), out.stride(1), _p(bt), _p(row_lens),
-                                      _p(sor), _p(ws_o), _p(ws_ml), rows, nh, max_blocks, bs, splits, scale, 0, _stream())
+                                      _p(sor), _p(ws_o), _p(ws_ml), rows, nh, KD, VD, max_blocks, bs, splits, 0, None, scale, 0,
+                                      _stream())
     assert rc == 0
     torch.cuda.synchronize()
     flat = cache.view(nb * bs, KD).float()
