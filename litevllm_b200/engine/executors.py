@@ -140,6 +140,11 @@ class DecodeExecutor:
         full_ctx = self.builder.kv.blocks_per_seq * self.builder.kv.block_size
         saved = batch.max_kv_len
         batch.max_kv_len = full_ctx
+        # the warm-up passes run the step for real: cache rows are rewritten with the same values, but recurrent
+        # states would advance, so the batch's slots are put back afterwards
+        states = [s for s in getattr(self.kv_cache, "states", ()) if s is not None]
+        slots = self.builder._decode_buffers(batch.num_seqs)["meta"][3].long()
+        saved_states = [s.index_select(0, slots) for s in states]
         # warm up outside capture (lazy allocations, scratch growth, kernel attribute setup)
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
@@ -149,6 +154,8 @@ class DecodeExecutor:
                 self._step_body(batch, greedy_only)
                 batch.input_ids.copy_(ids_saved)      # the body leaves the greedy tokens in the id buffer
         torch.cuda.current_stream().wait_stream(side)
+        for s, old in zip(states, saved_states):
+            s.index_copy_(0, slots, old)
         torch.cuda.synchronize()
         graph = torch.cuda.CUDAGraph()
         n0 = ops.launch_count()

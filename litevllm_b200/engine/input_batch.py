@@ -84,10 +84,20 @@ class InputBatchBuilder:
         self._h_meta = torch.zeros(2 * cap + 4 * (max_active + 1), dtype=torch.int32, pin_memory=pin)
         self._d_ids = torch.zeros(cap, dtype=torch.int64, device=device)
         self._d_meta = torch.zeros_like(self._h_meta, device=device)
+        self._prefill_upload = None      # event behind the last upload from the prefill staging buffers
         # persistent decode inputs per bucket (CUDA-graph inputs): [ids int64 | pos, slots, seq_lens, slot_ids]
         self._dec: dict[int, dict] = {}
 
     # ------------------------------------------------------------------ helpers
+    def _uploaded(self):
+        """Event behind the copies just enqueued: the pinned buffers may be refilled once it has passed (a caller
+        that reads nothing back can be several steps ahead of the device)."""
+        if self.device.type != "cuda":
+            return None
+        ev = torch.cuda.Event()
+        ev.record()
+        return ev
+
     def _slots_for(self, blocks: list[int], start: int, n: int) -> np.ndarray:
         pos = np.arange(start, start + n, dtype=np.int64)
         blk = np.asarray(blocks, dtype=np.int64)[pos // self.bs]
@@ -106,6 +116,8 @@ class InputBatchBuilder:
         T = sum(it.chunk_len for it in items)
         if T > self._cap:
             raise ValueError(f"prefill step of {T} tokens exceeds the staging capacity {self._cap}")
+        if self._prefill_upload is not None:
+            self._prefill_upload.synchronize()
         ids = self._h_ids.numpy()
         meta = self._h_meta.numpy()
         pos_h, slot_h = meta[:T], meta[T:2 * T]
@@ -131,6 +143,7 @@ class InputBatchBuilder:
         n_meta = base + 3 * B + 1
         self._d_ids[:T].copy_(self._h_ids[:T], non_blocking=True)
         self._d_meta[:n_meta].copy_(self._h_meta[:n_meta], non_blocking=True)
+        self._prefill_upload = self._uploaded()
         dm = self._d_meta
         cu = dm[base:base + B + 1]
         slot_ids = dm[base + 2 * B + 1:base + 3 * B + 1]
@@ -165,6 +178,8 @@ class InputBatchBuilder:
         n = len(reqs)
         bucket = self.bucket_for(n)
         d = self._decode_buffers(bucket)
+        if d.get("uploaded") is not None:
+            d["uploaded"].synchronize()
         hm = d["h_meta"].numpy()
         hi = d["h_ids"].numpy()
         hm[0, n:] = 0
@@ -188,6 +203,7 @@ class InputBatchBuilder:
         else:
             d["ids"][:n].copy_(device_tokens[:n], non_blocking=True)
         d["meta"].copy_(d["h_meta"], non_blocking=True)
+        d["uploaded"] = self._uploaded()
         self.kv.flush()
         torch.index_select(self.kv.block_tables, 0, d["meta"][3].long(), out=d["block_tables"])
         return ForwardBatch(
