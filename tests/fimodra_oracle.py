@@ -135,3 +135,91 @@ def forward(cfg, w, tokens, collect=None):
         if collect is not None:
             collect.append(x)
     return grouped_rms_norm(x, w["final.norm"], eps, groups) @ w["head"].t()
+
+
+# ------------------------------------------------------------------ small random models
+def layer(kind, mlp=None, **mixer):
+    if kind == "latent_attention":
+        mixer = dict(mixer)
+        mixer["mask"] = {"size": mixer.pop("window")}
+        mixer["rot"] = {"base": mixer.pop("base", 10000.0), "dims": mixer["rot_dim"]}
+        mixer.setdefault("scale", (mixer["dim"] + mixer["rot_dim"]) ** -0.5)
+    return {"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": mlp} if mlp else None}
+
+
+def config(width, vocab, groups, layers, eps=1e-6):
+    return {"architecture": "Fimodra", "width": width, "vocab": vocab, "norm": {"eps": eps, "groups": groups}, "layers": layers}
+
+
+def weights(cfg, seed=0, sharp=2.0):
+    """bf16-representable fp32 weights.  ``sharp`` widens the attention scores so that single keys matter."""
+    g = torch.Generator().manual_seed(seed)
+    W, w = cfg["width"], {}
+
+    def put(name, *shape, std=1.0, base=0.0):
+        w[name] = (base + std * torch.randn(*shape, generator=g)).bfloat16().float()
+
+    def lin(name, out_f, in_f, gain=1.0):
+        put(name, out_f, in_f, std=gain * in_f ** -0.5)
+
+    put("embed", cfg["vocab"], W)
+    for i, l in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        H = m["heads"]
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if l["mlp"] else ()):
+            put(p + n, W, std=0.2, base=1.0)
+        if l["type"] == "latent_attention":
+            lin(p + "mix.q", H * (m["dim"] + m["rot_dim"]), W, sharp)
+            lin(p + "mix.dkv", m["kv_rank"] + m["rot_dim"], W)
+            put(p + "mix.dkv.norm", m["kv_rank"], std=0.2, base=1.0)
+            lin(p + "mix.uk", H * m["dim"], m["kv_rank"])
+            lin(p + "mix.uv", H * m["vdim"], m["kv_rank"])
+            put(p + "mix.sink", H, std=1.0, base=1.0)
+            lin(p + "mix.o", W, H * m["vdim"])
+        else:
+            lin(p + "mix.q", H * m["dim"], W)
+            lin(p + "mix.f", H * m["dim"], W)
+            put(p + "mix.f.b", H * m["dim"], std=3.0, base=2.0)
+            w[p + "mix.lower"] = (torch.rand(H * m["dim"], generator=g) * 0.9 * (torch.rand(H * m["dim"], generator=g) > 0.3)).bfloat16().float()
+            lin(p + "mix.v", H * m["vdim"], W)
+            put(p + "mix.norm", m["vdim"], std=0.2, base=1.0)
+            lin(p + "mix.o", W, H * m["vdim"])
+        if l["mlp"]:
+            ff = l["mlp"]["ff"]
+            for n, o, k in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+                lin(p + "mlp." + n, o, k)
+                put(p + "mlp." + n + ".b", o, std=0.3)
+        put(p + "dwa", i + 2, std=0.5)
+        w[p + "dwa"][-1] += 1.0
+        w[p + "dwa"] = w[p + "dwa"].bfloat16().float()
+    put("final.norm", W, std=0.2, base=1.0)
+    lin("head", cfg["vocab"], W)
+    return w
+
+
+def save(folder, cfg, w):
+    import json
+
+    from safetensors.torch import save_file
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(cfg))
+    save_file({k: v.bfloat16().contiguous() for k, v in w.items()}, str(folder / "model.safetensors"))
+    return str(folder)
+
+
+def greedy(cfg, w, prompt, n):
+    """Greedy continuation from scratch, and the smallest margin between the best two logits on the way."""
+    ids, margin = list(prompt), math.inf
+    for _ in range(n):
+        top = torch.topk(forward(cfg, w, ids)[-1], 2)
+        margin = min(margin, float(top.values[0] - top.values[1]))
+        ids.append(int(top.indices[0]))
+    return ids[len(prompt):], margin
+
+
+def error(got, want):
+    """Root mean square over the vocabulary of the difference (mean taken off), relative to the logits' spread."""
+    d = got.double().cpu() - want.double()
+    d = d - d.mean(-1, keepdim=True)
+    s = want.double() - want.double().mean(-1, keepdim=True)
+    return float((d.pow(2).mean(-1).sqrt() / s.pow(2).mean().sqrt()).max())
