@@ -217,9 +217,19 @@ def greedy(cfg, w, prompt, n):
     return ids[len(prompt):], margin
 
 
-def error(got, want):
-    """Root mean square over the vocabulary of the difference (mean taken off), relative to the logits' spread."""
+def errors(got, want):
+    """Per position: root mean square over the vocabulary of the difference (mean taken off), relative to the spread of
+    the logits."""
     d = got.double().cpu() - want.double()
     d = d - d.mean(-1, keepdim=True)
     s = want.double() - want.double().mean(-1, keepdim=True)
-    return float((d.pow(2).mean(-1).sqrt() / s.pow(2).mean().sqrt()).max())
+    return d.pow(2).mean(-1).sqrt() / s.pow(2).mean().sqrt()
+
+
+def fits(got, want, dtype):
+    """32-bit runs agree everywhere; 16-bit ones up to rounding, which a norm over a few small channels can enlarge at
+    a position here and there."""
+    e = errors(got, want)
+    if dtype == "float32":
+        return float(e.max()) < 2e-4
+    return float(torch.quantile(e, 0.95)) < 0.08 and float(e.max()) < 0.4
