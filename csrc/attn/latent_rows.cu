@@ -39,8 +39,34 @@ struct PrepareParams {
   void* q_out;              // [T, nh, q_pitch]
   long ldq, ldkv;
   int T, nh, dim, rot, rdims, rank, q_pitch, nope_off, rot_off, zero_from, max_pos;
+  int pairs, vec;           // alignment of all rows and parts: whole pairs, whole 16-byte groups
   float eps;
 };
+
+// Values are handled in pairs: a pair of 16-bit values is one 32-bit access, and a rotation turns exactly one pair.
+template <typename T> struct Pair;
+template <> struct Pair<float> { typedef float2 type; };
+template <> struct Pair<__nv_bfloat16> { typedef __nv_bfloat162 type; };
+template <> struct Pair<__half> { typedef __half2 type; };
+template <typename T> __device__ __forceinline__ float2 load_pair(const T* p, bool whole) {
+  float2 r;
+  if (whole) {
+    const typename Pair<T>::type v = *reinterpret_cast<const typename Pair<T>::type*>(p);
+    r.x = to_f(v.x); r.y = to_f(v.y);
+  } else {
+    r.x = to_f(p[0]); r.y = to_f(p[1]);
+  }
+  return r;
+}
+template <typename T> __device__ __forceinline__ void store_pair(T* p, float a, float b, bool whole) {
+  if (whole) {
+    typename Pair<T>::type v;
+    v.x = from_f<T>(a); v.y = from_f<T>(b);
+    *reinterpret_cast<typename Pair<T>::type*>(p) = v;
+  } else {
+    p[0] = from_f<T>(a); p[1] = from_f<T>(b);
+  }
+}
 
 // Block: (token, share of the heads).  The first block of a token also writes its cache row.
 template <typename T>
@@ -54,10 +80,31 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(const PrepareParams
   const float* cs = p.cos_sin + static_cast<long>(pos) * p.rdims;
   const int half = p.rdims / 2;
   const T* q = reinterpret_cast<const T*>(p.q) + t * p.ldq;
+  const bool even = p.pairs != 0;                  // every row and every part of it starts on a whole pair
+  // pair i of a rotary part of `n` channels (the last one may be half a pair, which never turns)
+  auto turn = [&](const T* src, T* dst, int i, int n) {
+    if (2 * i + 1 < n) {
+      float2 v = load_pair(src + 2 * i, even);
+      if (i < half) {
+        const float c = cs[i], s = cs[half + i];
+        v = make_float2(v.x * c - v.y * s, v.y * c + v.x * s);
+      }
+      store_pair(dst + 2 * i, v.x, v.y, even);
+    } else {
+      dst[2 * i] = src[2 * i];
+    }
+  };
   if (blockIdx.y == 0) {
     const T* row = reinterpret_cast<const T*>(p.dkv) + t * p.ldkv;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < p.rank; i += 128) { const float f = to_f(row[i]); ss += f * f; }
+    if (even) {
+      for (int i = threadIdx.x; i < p.rank / 2; i += 128) {
+        const float2 f = load_pair(row + 2 * i, true);
+        ss += f.x * f.x + f.y * f.y;
+      }
+    } else {
+      for (int i = threadIdx.x; i < p.rank; i += 128) { const float f = to_f(row[i]); ss += f * f; }
+    }
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
@@ -65,33 +112,30 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(const PrepareParams
     const int slot = p.slot_mapping[t];
     if (slot >= 0) {
       T* dst = reinterpret_cast<T*>(p.cache) + static_cast<long>(slot) * (p.rank + p.rot);
-      for (int i = threadIdx.x; i < p.rank; i += 128) dst[i] = from_f<T>(to_f(row[i]) * inv * p.norm_w[i]);
-      for (int i = threadIdx.x; i < p.rot; i += 128) {
-        float v = to_f(row[p.rank + i]);
-        if (i < 2 * half) {
-          const float other = to_f(row[p.rank + (i ^ 1)]);
-          const float c = cs[i >> 1], s = cs[half + (i >> 1)];
-          v = (i & 1) ? v * c + other * s : v * c - other * s;
+      if (even) {
+        for (int i = threadIdx.x; i < p.rank / 2; i += 128) {
+          const float2 f = load_pair(row + 2 * i, true);
+          store_pair(dst + 2 * i, f.x * inv * p.norm_w[2 * i], f.y * inv * p.norm_w[2 * i + 1], true);
         }
-        dst[p.rank + i] = from_f<T>(v);
+      } else {
+        for (int i = threadIdx.x; i < p.rank; i += 128) dst[i] = from_f<T>(to_f(row[i]) * inv * p.norm_w[i]);
       }
+      for (int i = threadIdx.x; i < (p.rot + 1) / 2; i += 128) turn(row + p.rank, dst + p.rank, i, p.rot);
     }
   }
   const int hd = p.dim + p.rot;
+  constexpr int V = 16 / sizeof(T);
   for (int h = blockIdx.y * 4 + warp; h < p.nh; h += 4 * gridDim.y) {
     const T* src = q + static_cast<long>(h) * hd;
     T* dst = reinterpret_cast<T*>(p.q_out) + (static_cast<long>(t) * p.nh + h) * p.q_pitch;
-    for (int i = lane; i < p.rot; i += 32) {
-      float v = to_f(src[p.dim + i]);
-      if (i < 2 * half) {
-        const float other = to_f(src[p.dim + (i ^ 1)]);
-        const float c = cs[i >> 1], s = cs[half + (i >> 1)];
-        v = (i & 1) ? v * c + other * s : v * c - other * s;
-      }
-      dst[p.rot_off + i] = from_f<T>(v);
-    }
+    for (int i = lane; i < (p.rot + 1) / 2; i += 32) turn(src + p.dim, dst + p.rot_off, i, p.rot);
     if (p.nope_off >= 0) {
-      for (int i = lane; i < p.dim; i += 32) dst[p.nope_off + i] = src[i];
+      if (p.vec) {
+        for (int i = lane; i < p.dim / V; i += 32)
+          reinterpret_cast<uint4*>(dst + p.nope_off)[i] = reinterpret_cast<const uint4*>(src)[i];
+      } else {
+        for (int i = lane; i < p.dim; i += 32) dst[p.nope_off + i] = src[i];
+      }
       for (int i = p.zero_from + lane; i < p.q_pitch; i += 32) dst[i] = from_f<T>(0.f);
     }
   }
@@ -291,6 +335,12 @@ extern "C" int fi_latent_prepare(const void* q, long ldq, const void* dkv, long 
   p.cache = cache; p.q_out = q_out; p.ldq = ldq; p.ldkv = ldkv; p.T = T; p.nh = nh; p.dim = dim; p.rot = rot;
   p.rdims = rdims; p.rank = rank; p.q_pitch = q_pitch; p.nope_off = nope_off; p.rot_off = rot_off;
   p.zero_from = zero_from; p.max_pos = max_pos; p.eps = eps;
+  const int esz = dtype == 2 ? 4 : 2, v = 16 / esz;
+  const uintptr_t at = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(dkv) | reinterpret_cast<uintptr_t>(cache) |
+                       reinterpret_cast<uintptr_t>(q_out);
+  p.pairs = ((ldq | ldkv | dim | rot | rank | q_pitch | rot_off) & 1) == 0 && (at & (2 * esz - 1)) == 0;
+  p.vec = nope_off >= 0 && ldq % v == 0 && (dim + rot) % v == 0 && dim % v == 0 && q_pitch % v == 0 && nope_off % v == 0 &&
+          ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(q_out)) & 15) == 0;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid(T, T >= 256 ? 1 : (nh + 3) / 4);
 #define FI_CALL(TT) return static_cast<int>(fi::launch_kernel(latent_prepare_kernel<TT>, grid, dim3(128), 0, s, 0, p))

@@ -165,14 +165,19 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   const T* cache = reinterpret_cast<const T*>(p.cache);
 
   for (int c = c_begin; c < c_end; ++c) {
-    // ---- stage 64 cache rows (rows past the visible length are zero)
-    for (int i = threadIdx.x; i < CH * (kd / 8); i += 128) {
-      const int row = i / (kd / 8), ch = i % (kd / 8);
-      const int tok = c * CH + row;
-      const bool valid = tok < len;
-      const int blk = valid ? bt[tok / p.block_size] : 0;
-      const long src = (static_cast<long>(blk) * p.block_size + (valid ? tok % p.block_size : 0)) * kd + ch * 8;
-      cp_async16(sK + row_off<KDT>(row, ch, pitch), cache + src, valid);
+    // ---- stage 64 cache rows (rows past the visible length are zero): a warp takes 16 rows, its lanes look the
+    // 16 cache rows up once and then copy row by row
+    {
+      const int tok = c * CH + warp * 16 + (lane & 15);
+      int src_row = -1;
+      if (tok < len) src_row = bt[tok / p.block_size] * p.block_size + tok % p.block_size;
+#pragma unroll 4
+      for (int rr = 0; rr < 16; ++rr) {
+        const int row = warp * 16 + rr;
+        const int sr = __shfl_sync(0xffffffffu, src_row, rr);
+        const T* src = cache + static_cast<long>(sr < 0 ? 0 : sr) * kd;
+        for (int ch = lane; ch < kd / 8; ch += 32) cp_async16(sK + row_off<KDT>(row, ch, pitch), src + ch * 8, sr >= 0);
+      }
     }
     cp_async_commit();
     cp_async_wait_all();

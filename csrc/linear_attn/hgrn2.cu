@@ -72,25 +72,58 @@ struct Hgrn2Params {
   const float* norm_w;    // step: [dv]
   void* out;              // step: [B, H * dv]
   long ldq, ldf, ldv;
+  int vec4;               // rows of q, f and v start on whole groups of four values
   int H, d, dv, qv_type, f_type, out_type, num_slots;
   float eps;
 };
 
 constexpr int kWarps = 8;
 
-// R rows per lane (16 R >= d), C columns per lane (a warp: 2 C columns, a block: 16 C).
-template <int R, int C>
+// Four consecutive raw values of the projections; they stay raw until they are activated, so that the loads of a stage
+// are all in flight at once.
+template <typename T> struct Raw4;
+template <> struct Raw4<float> { float4 r; };
+template <> struct Raw4<uint16_t> { uint2 r; };
+template <typename T>
+__device__ __forceinline__ Raw4<T> load4(const T* p, int n, int vec4) {      // n valid values (n >= 4: whole group)
+  Raw4<T> v;
+  if (vec4 && n >= 4) {
+    v.r = *reinterpret_cast<const decltype(v.r)*>(p);
+  } else {
+    alignas(16) T e[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) e[i] = i < n ? p[i] : T(0);
+    v.r = *reinterpret_cast<const decltype(v.r)*>(e);
+  }
+  return v;
+}
+__device__ __forceinline__ void expand4(const Raw4<float>& v, int, float* o) {
+  o[0] = v.r.x; o[1] = v.r.y; o[2] = v.r.z; o[3] = v.r.w;
+}
+__device__ __forceinline__ void expand4(const Raw4<uint16_t>& v, int type, float* o) {
+  const uint32_t w[2] = {v.r.x, v.r.y};
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const float2 h = __half22float2(*reinterpret_cast<const __half2*>(&w[i]));
+    o[2 * i] = type == kBf16 ? __uint_as_float(w[i] << 16) : h.x;
+    o[2 * i + 1] = type == kBf16 ? __uint_as_float(w[i] & 0xffff0000u) : h.y;
+  }
+}
+
+// R rows per lane (16 R >= d), C columns per lane (a warp: 2 C columns, a block: 16 C); T: storage of q and v.
+template <int R, int C, typename T>
 __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Params p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   constexpr int kTok = R <= 8 ? 16 : (R <= 16 ? 8 : 4);     // tokens staged at a time
   constexpr int D = 16 * R;                 // padded rows: q = k = 0 there, the state stays 0
   constexpr int COLS = kWarps * 2 * C;
-  constexpr int NQ = (kTok * D + 255) / 256;
-  constexpr int NVAL = (kTok * COLS + 255) / 256;
+  constexpr int NQ = (kTok * D / 4 + 255) / 256;             // groups of four values per thread
+  constexpr int NVAL = (kTok * COLS / 4 + 255) / 256;
   __shared__ __align__(16) float sq[2][kTok][D];
   __shared__ __align__(16) float sk[2][kTok][D];
   __shared__ __align__(16) float sv[2][kTok][COLS];
+  __shared__ float open_gate[D], gate_bias[D];
   const int slices = (p.dv + COLS - 1) / COLS;
   const int head = blockIdx.x / slices, slice = blockIdx.x % slices;
   const int b = blockIdx.y;
@@ -120,48 +153,64 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
     }
   }
 
-  float rq[NQ], rf[NQ], rv[NVAL];           // raw values of the next kTok tokens
+  Raw4<T> rq[NQ], rv[NVAL];                 // raw values of the next kTok tokens
+  Raw4<float> rf[NQ];
+  const T* gq = reinterpret_cast<const T*>(p.q) + head * p.d;
+  const T* gv = reinterpret_cast<const T*>(p.v) + head * p.dv + slice * COLS;
+  const float* gf = reinterpret_cast<const float*>(p.f) + head * p.d;
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
-      const int e = i * 256 + threadIdx.x, tok = e / D, ch = e % D;
-      rq[i] = 0.f; rf[i] = 0.f;
-      if (tok < kTok && t0 + tok < n && ch < p.d) {
-        const long t = t_begin + t0 + tok;
-        rq[i] = ld(p.q, t * p.ldq + head * p.d + ch, p.qv_type);
-        rf[i] = ld(p.f, t * p.ldf + head * p.d + ch, p.f_type);
-      }
+      const int e = (i * 256 + threadIdx.x) * 4, tok = e / D, ch = e % D;
+      const int left = (tok < kTok && t0 + tok < n) ? p.d - ch : 0;
+      const long t = t_begin + t0 + tok;
+      rq[i] = load4(gq + t * p.ldq + ch, left, p.vec4);
+      rf[i] = load4(gf + t * p.ldf + ch, left, p.vec4);
     }
 #pragma unroll
     for (int i = 0; i < NVAL; ++i) {
-      const int e = i * 256 + threadIdx.x, tok = e / COLS, c = e % COLS;
-      rv[i] = 0.f;
-      if (tok < kTok && t0 + tok < n && slice * COLS + c < p.dv)
-        rv[i] = ld(p.v, static_cast<long>(t_begin + t0 + tok) * p.ldv + head * p.dv + slice * COLS + c, p.qv_type);
+      const int e = (i * 256 + threadIdx.x) * 4, tok = e / COLS, c = e % COLS;
+      const int left = (tok < kTok && t0 + tok < n) ? p.dv - slice * COLS - c : 0;
+      rv[i] = load4(gv + static_cast<long>(t_begin + t0 + tok) * p.ldv + c, left, p.vec4);
     }
   };
   auto stage = [&](int buf) {
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
-      const int e = i * 256 + threadIdx.x, tok = e / D, ch = e % D;
+      const int e = (i * 256 + threadIdx.x) * 4, tok = e / D, ch = e % D;
       if (tok < kTok) {
-        float qa = 0.f, ka = 0.f;
-        if (ch < p.d) {
-          qa = rq[i] * sigmoidf(rq[i]);
-          ka = (1.f - p.lower[head * p.d + ch]) * sigmoidf(-(rf[i] + p.f_bias[head * p.d + ch]));
+        float zq[4], zf[4], qa[4], ka[4];
+        expand4(rq[i], p.qv_type, zq);
+        expand4(rf[i], kFp32, zf);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          qa[j] = 0.f; ka[j] = 0.f;
+          if (ch + j < p.d) {
+            qa[j] = zq[j] * sigmoidf(zq[j]);
+            ka[j] = open_gate[ch + j] * sigmoidf(-(zf[j] + gate_bias[ch + j]));
+          }
         }
-        sq[buf][tok][ch] = qa;
-        sk[buf][tok][ch] = ka;
+        *reinterpret_cast<float4*>(&sq[buf][tok][ch]) = make_float4(qa[0], qa[1], qa[2], qa[3]);
+        *reinterpret_cast<float4*>(&sk[buf][tok][ch]) = make_float4(ka[0], ka[1], ka[2], ka[3]);
       }
     }
 #pragma unroll
     for (int i = 0; i < NVAL; ++i) {
-      const int e = i * 256 + threadIdx.x, tok = e / COLS, c = e % COLS;
-      if (tok < kTok) sv[buf][tok][c] = rv[i];
+      const int e = (i * 256 + threadIdx.x) * 4, tok = e / COLS, c = e % COLS;
+      if (tok < kTok) {
+        float v4[4];
+        expand4(rv[i], p.qv_type, v4);
+        *reinterpret_cast<float4*>(&sv[buf][tok][c]) = make_float4(v4[0], v4[1], v4[2], v4[3]);
+      }
     }
   };
 
+  for (int c = threadIdx.x; c < D; c += 256) {
+    open_gate[c] = c < p.d ? 1.f - p.lower[head * p.d + c] : 0.f;
+    gate_bias[c] = c < p.d ? p.f_bias[head * p.d + c] : 0.f;
+  }
   fetch(0);
+  __syncthreads();
   stage(0);
   __syncthreads();
   const f2 one2 = pack2(1.f, 1.f), neg2 = pack2(-1.f, -1.f);
@@ -298,25 +347,39 @@ __global__ void __launch_bounds__(256) hgrn2_step_kernel(const Hgrn2Params p) {
       v[e] = ld(p.v, b * p.ldv + head * p.dv + cx * VEC + e, p.qv_type);
       o[e] = 0.f;
     }
-#pragma unroll 8
-    for (int r = ry; r < p.d; r += ry_n) {
-      float* row = S + static_cast<long>(r) * p.dv + cx * VEC;
-      float s[VEC];
-      if constexpr (VEC == 4) {
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (!fresh) x = *reinterpret_cast<const float4*>(row);
-        s[0] = x.x; s[1] = x.y; s[2] = x.z; s[3] = x.w;
-      } else {
-        s[0] = fresh ? 0.f : row[0];
-      }
-      const float k = sk[r], q = sq[r], f = 1.f - k;
+    constexpr int U = 8;                  // rows whose loads are in flight together
+    for (int r0 = ry; r0 < p.d; r0 += U * ry_n) {
+      float s[U][VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        s[e] = fmaf(f, s[e], k * v[e]);
-        o[e] = fmaf(q, s[e], o[e]);
+      for (int u = 0; u < U; ++u) {
+        const int r = r0 + u * ry_n;
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s[u][e] = 0.f;
+        if (!fresh && r < p.d) {
+          const float* row = S + static_cast<long>(r) * p.dv + cx * VEC;
+          if constexpr (VEC == 4) {
+            const float4 x = *reinterpret_cast<const float4*>(row);
+            s[u][0] = x.x; s[u][1] = x.y; s[u][2] = x.z; s[u][3] = x.w;
+          } else {
+            s[u][0] = row[0];
+          }
+        }
       }
-      if constexpr (VEC == 4) *reinterpret_cast<float4*>(row) = make_float4(s[0], s[1], s[2], s[3]);
-      else row[0] = s[0];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int r = r0 + u * ry_n;
+        if (r < p.d) {
+          float* row = S + static_cast<long>(r) * p.dv + cx * VEC;
+          const float k = sk[r], q = sq[r], f = 1.f - k;
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) {
+            s[u][e] = fmaf(f, s[u][e], k * v[e]);
+            o[e] = fmaf(q, s[u][e], o[e]);
+          }
+          if constexpr (VEC == 4) *reinterpret_cast<float4*>(row) = make_float4(s[u][0], s[u][1], s[u][2], s[u][3]);
+          else row[0] = s[u][0];
+        }
+      }
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) so[ry * p.dv + cx * VEC + e] = o[e];
@@ -368,7 +431,7 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
         if (type == kFp32) {
           *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + row * dv + c) = make_float4(y[0], y[1], y[2], y[3]);
         } else {
-          uint16_t h[4];
+          alignas(8) uint16_t h[4];
           for (int e = 0; e < 4; ++e)
             h[e] = type == kBf16 ? __bfloat16_as_ushort(__float2bfloat16_rn(y[e])) : __half_as_ushort(__float2half_rn(y[e]));
           *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(out) + row * dv + c) = *reinterpret_cast<uint2*>(h);
@@ -386,8 +449,9 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
 template <int R, int C>
 int launch_scan(const Hgrn2Params& p, int B, cudaStream_t s) {
   constexpr int COLS = kWarps * 2 * C;
-  const int slices = (p.dv + COLS - 1) / COLS;
-  return static_cast<int>(fi::launch_kernel(hgrn2_scan_kernel<R, C>, dim3(p.H * slices, B), dim3(kWarps * 32), 0, s, 0, p));
+  const dim3 grid(p.H * ((p.dv + COLS - 1) / COLS), B), block(kWarps * 32);
+  if (p.qv_type == kFp32) return static_cast<int>(fi::launch_kernel(hgrn2_scan_kernel<R, C, float>, grid, block, 0, s, 0, p));
+  return static_cast<int>(fi::launch_kernel(hgrn2_scan_kernel<R, C, uint16_t>, grid, block, 0, s, 0, p));
 }
 
 template <int R>
@@ -403,7 +467,7 @@ int pick_cols(const Hgrn2Params& p, int B, cudaStream_t s) {
 
 }  // namespace
 
-// Portions of sequences.  q, v: type qv_type (0 bf16, 1 fp16, 2 fp32), f: type f_type, rows of pitch ldq / ldf / ldv;
+// Portions of sequences.  q, v: type qv_type (0 bf16, 1 fp16, 2 fp32), f: fp32 (f_type 2), rows of pitch ldq / ldf / ldv;
 // f_bias, lower: fp32 [H * d]; pool: fp32 [num_slots, H, d, dv]; slots, seq_lens: int32 [B]; cu_q: int32 [B + 1];
 // o: fp32 [T, H, dv].
 extern "C" int fi_hgrn2_scan(const void* q, long ldq, const void* f, long ldf, const void* v, long ldv,
@@ -411,11 +475,14 @@ extern "C" int fi_hgrn2_scan(const void* q, long ldq, const void* f, long ldf, c
                              const int* seq_lens, float* o, int B, int H, int d, int dv, int num_slots, int qv_type,
                              int f_type, void* stream) {
   if (B <= 0) return 0;
-  if (H <= 0 || d <= 0 || dv <= 0 || B > 65535 || qv_type < 0 || qv_type > 2 || f_type < 0 || f_type > 2) return -10;
+  if (H <= 0 || d <= 0 || dv <= 0 || B > 65535 || qv_type < 0 || qv_type > 2 || f_type != kFp32) return -10;
   Hgrn2Params p = {};
   p.q = q; p.f = f; p.v = v; p.ldq = ldq; p.ldf = ldf; p.ldv = ldv; p.f_bias = f_bias; p.lower = lower; p.pool = pool;
   p.slots = slots; p.cu_q = cu_q; p.seq_lens = seq_lens; p.o = o; p.H = H; p.d = d; p.dv = dv; p.num_slots = num_slots;
-  p.qv_type = qv_type; p.f_type = f_type;
+  p.qv_type = qv_type;
+  const uintptr_t mask = qv_type == kFp32 ? 15 : 7;
+  p.vec4 = d % 4 == 0 && dv % 4 == 0 && ldq % 4 == 0 && ldf % 4 == 0 && ldv % 4 == 0 &&
+           ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(v)) & mask) == 0 && (reinterpret_cast<uintptr_t>(f) & 15) == 0;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (d <= 64) return pick_cols<4>(p, B, s);
   if (d <= 128) return pick_cols<8>(p, B, s);

@@ -40,9 +40,11 @@ struct StreamParams {
   float eps;
 };
 
-template <int VEC>
+// 16-bit or 32-bit storage is a compile-time choice (H16): a branch around every load would keep the loads of a row
+// from being issued together.  bf16 / fp16 is a select on the loaded bits.
+template <int VEC, bool H16>
 __device__ __forceinline__ void load_any(const void* p, long i, int type, float* v) {
-  if (type == kFp32) {
+  if constexpr (!H16) {
     if constexpr (VEC == 4) {
       const float4 f = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p) + i);
       v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
@@ -51,7 +53,7 @@ __device__ __forceinline__ void load_any(const void* p, long i, int type, float*
     }
     return;
   }
-  uint16_t raw[VEC];
+  alignas(8) uint16_t raw[VEC];
   if constexpr (VEC == 4) {
     *reinterpret_cast<uint2*>(raw) = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(p) + i);
   } else {
@@ -63,16 +65,16 @@ __device__ __forceinline__ void load_any(const void* p, long i, int type, float*
                          : __half2float(__ushort_as_half(raw[e]));
 }
 
-template <int VEC>
+template <int VEC, bool H16>
 __device__ __forceinline__ void store_any(void* p, long i, int type, const float* v) {
-  if (type == kFp32) {
+  if constexpr (!H16) {
     if constexpr (VEC == 4)
       *reinterpret_cast<float4*>(reinterpret_cast<float*>(p) + i) = make_float4(v[0], v[1], v[2], v[3]);
     else
       reinterpret_cast<float*>(p)[i] = v[0];
     return;
   }
-  uint16_t raw[VEC];
+  alignas(8) uint16_t raw[VEC];
 #pragma unroll
   for (int e = 0; e < VEC; ++e)
     raw[e] = type == kBf16 ? __bfloat16_as_ushort(__float2bfloat16_rn(v[e])) : __half_as_ushort(__float2half_rn(v[e]));
@@ -98,7 +100,7 @@ __device__ __forceinline__ float row_sum(float v, float* red) {
   return v;
 }
 
-template <int MODE, int TPR, int VEC, int NV>
+template <int MODE, int TPR, int VEC, int NV, bool H16>
 __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -119,7 +121,7 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
-      if (c < p.group) load_any<VEC>(p.table, id * p.W + c0 + c, p.h_type, v + i * VEC);
+      if (c < p.group) load_any<VEC, H16>(p.table, id * p.W + c0 + c, p.h_type, v + i * VEC);
       else
 #pragma unroll
         for (int e = 0; e < VEC; ++e) v[i * VEC + e] = 0.f;
@@ -131,22 +133,22 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
       if (c < p.group) {
-        load_any<VEC>(p.y, t * p.ldy + c0 + c, p.y_type, v + i * VEC);
-        load_any<VEC>(p.x, t * p.W + c0 + c, kFp32, xv + i * VEC);
+        load_any<VEC, H16>(p.y, t * p.ldy + c0 + c, p.y_type, v + i * VEC);
+        load_any<VEC, false>(p.x, t * p.W + c0 + c, kFp32, xv + i * VEC);
       } else {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) { v[i * VEC + e] = 0.f; xv[i * VEC + e] = 0.f; }
       }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) ss += v[i * VEC + e] * v[i * VEC + e];
     }
+#pragma unroll
+    for (int i = 0; i < NV * VEC; ++i) ss += v[i] * v[i];
     const float inv = 1.f / sqrtf(row_sum<TPR>(ss, red) * inv_n + p.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
       if (c < p.group) {
         float w[VEC];
-        load_any<VEC>(p.w_post, c0 + c, kFp32, w);
+        load_any<VEC, false>(p.w_post, c0 + c, kFp32, w);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(v[i * VEC + e] * inv, w[e], xv[i * VEC + e]);
       }
@@ -157,7 +159,7 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
       for (int i = 0; i < NV; ++i) {
         const int c = (i * TPR + tid) * VEC;
         if (c < p.group && p.sel == nullptr)
-          store_any<VEC>(p.hist, p.n * p.hist_stride + t * p.W + c0 + c, kFp32, v + i * VEC);
+          store_any<VEC, false>(p.hist, p.n * p.hist_stride + t * p.W + c0 + c, kFp32, v + i * VEC);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) v[i * VEC + e] *= an;
       }
@@ -170,7 +172,7 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
           const int c = (i * TPR + tid) * VEC;
           if (c < p.group) {
             float o[VEC];
-            load_any<VEC>(hrow + j * p.hist_stride, c, kFp32, o);
+            load_any<VEC, false>(hrow + j * p.hist_stride, c, kFp32, o);
 #pragma unroll
             for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(a, o[e], v[i * VEC + e]);
           }
@@ -183,7 +185,7 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
-      if (c < p.group) store_any<VEC>(p.x_out, t * p.W + c0 + c, kFp32, v + i * VEC);
+      if (c < p.group) store_any<VEC, false>(p.x_out, t * p.W + c0 + c, kFp32, v + i * VEC);
     }
   }
   if (p.w_pre != nullptr) {
@@ -201,10 +203,10 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
       const int c = (i * TPR + tid) * VEC;
       if (c < p.group) {
         float w[VEC], o[VEC];
-        load_any<VEC>(p.w_pre, c0 + c, kFp32, w);
+        load_any<VEC, false>(p.w_pre, c0 + c, kFp32, w);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) o[e] = v[i * VEC + e] * inv * w[e];
-        store_any<VEC>(p.h, static_cast<long>(r) * p.ldh + c0 + c, p.h_type, o);
+        store_any<VEC, H16>(p.h, static_cast<long>(r) * p.ldh + c0 + c, p.h_type, o);
       }
     }
   }
@@ -215,8 +217,10 @@ int launch(const StreamParams& p, cudaStream_t s) {
   const long rows = static_cast<long>(p.rows) * p.groups;
   const long grid = (rows + 256 / TPR - 1) / (256 / TPR);
   if (grid > 2147483647l) return -10;
-  return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV>, dim3(static_cast<unsigned>(grid)),
-                                            dim3(256), 0, s, 0, p));
+  const dim3 g(static_cast<unsigned>(grid));
+  if (p.h_type == kFp32)
+    return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV, false>, g, dim3(256), 0, s, 0, p));
+  return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV, true>, g, dim3(256), 0, s, 0, p));
 }
 
 template <int MODE>
@@ -259,12 +263,12 @@ extern "C" int fi_stream_start(const long long* ids, const void* table, int voca
   return dispatch<kStart>(p, vec4, reinterpret_cast<cudaStream_t>(stream));
 }
 
-// x_out = x + norm(y) * w_post; h = norm(x_out) * w_pre (w_pre null: no h).  x_out may be x.
+// x_out = x + norm(y) * w_post; h = norm(x_out) * w_pre (w_pre null: no h).  x_out may be x.  y and h share a type.
 extern "C" int fi_stream_step(const void* y, long ldy, int y_type, const float* x, const float* w_post,
                               const float* w_pre, float* x_out, void* h, long ldh, int h_type, int T, int W, int groups,
                               float eps, void* stream) {
   if (T <= 0) return 0;
-  if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || y_type < 0 || y_type > 2) return -10;
+  if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || y_type != h_type) return -10;
   StreamParams p = {};
   p.y = y; p.ldy = ldy; p.y_type = y_type; p.x = x; p.w_post = w_post; p.w_pre = w_pre; p.x_out = x_out; p.h = h;
   p.ldh = ldh; p.h_type = h_type; p.rows = T; p.W = W; p.group = W / groups; p.groups = groups; p.eps = eps;
@@ -281,7 +285,7 @@ extern "C" int fi_stream_average(const void* y, long ldy, int y_type, const floa
                                  float* x_out, void* h, long ldh, int h_type, const long long* sel, int rows, int W,
                                  int groups, float eps, void* stream) {
   if (rows <= 0) return 0;
-  if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || y_type < 0 || y_type > 2 || n < 1) return -10;
+  if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || y_type != h_type || n < 1) return -10;
   if (sel != nullptr && x_out != nullptr) return -10;
   StreamParams p = {};
   p.y = y; p.ldy = ldy; p.y_type = y_type; p.x = x; p.w_post = w_post; p.w_pre = w_pre; p.hist = hist;

@@ -171,6 +171,7 @@ def hgrn2_scan(q, f, v, f_bias, lower, pool, slots, cu_q, seq_lens, H: int, d: i
         return o
     assert q.dtype == v.dtype and q.stride(1) == f.stride(1) == v.stride(1) == 1
     assert pool.dtype == torch.float32 and pool.is_contiguous() and slots.dtype == torch.int32 == cu_q.dtype
+    assert f.dtype == torch.float32, "the forget gate's projection stays 32-bit"
     rc = _lib.kernels().fi_hgrn2_scan(_p(q), q.stride(0), _p(f), f.stride(0), _p(v), v.stride(0), _p(f_bias), _p(lower),
                                       _p(pool), _p(slots), _p(cu_q), _p(seq_lens), _p(o), B, H, d, dv, pool.shape[0],
                                       _DT[q.dtype], _DT[f.dtype], _stream())
