@@ -174,7 +174,8 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
       rv[i] = load4(gv + static_cast<long>(t_begin + t0 + tok) * p.ldv + c, left, p.vec4);
     }
   };
-  auto stage = [&](int buf) {
+  // tokens past the end are staged with q = k = 0: they leave the state as it is
+  auto stage = [&](int buf, int t0) {
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
       const int e = (i * 256 + threadIdx.x) * 4, tok = e / D, ch = e % D;
@@ -185,7 +186,7 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           qa[j] = 0.f; ka[j] = 0.f;
-          if (ch + j < p.d) {
+          if (ch + j < p.d && t0 + tok < n) {
             qa[j] = zq[j] * sigmoidf(zq[j]);
             ka[j] = open_gate[ch + j] * sigmoidf(-(zf[j] + gate_bias[ch + j]));
           }
@@ -211,7 +212,7 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
   }
   fetch(0);
   __syncthreads();
-  stage(0);
+  stage(0, 0);
   __syncthreads();
   const f2 one2 = pack2(1.f, 1.f), neg2 = pack2(-1.f, -1.f);
   for (int t0 = 0, it = 0; t0 < n; t0 += kTok, ++it) {
@@ -219,35 +220,32 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
     const bool more = t0 + kTok < n;
     if (more) fetch(t0 + kTok);
     const int here = min(kTok, n - t0);
-    for (int tq = 0; tq < here; tq += 4) {
+    auto four_tokens = [&](int tq) {
       float part[4 * C];                    // partial outputs [token][column] of this lane's rows
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
         f2 acc[C], vv[C];
         const int tok = tq + u;
 #pragma unroll
-        for (int c = 0; c < C; ++c) acc[c] = pack2(0.f, 0.f);
-        if (tok < here) {                   // uniform: a token past the end must not decay the state
+        for (int c = 0; c < C; ++c) {
+          acc[c] = pack2(0.f, 0.f);
+          const float x = sv[buf][tok][(warp * 2 + cg) * C + c];
+          vv[c] = pack2(x, x);
+        }
 #pragma unroll
-          for (int c = 0; c < C; ++c) {
-            const float x = sv[buf][tok][(warp * 2 + cg) * C + c];
-            vv[c] = pack2(x, x);
-          }
+        for (int i4 = 0; i4 < R / 4; ++i4) {
+          const float4 q4 = *reinterpret_cast<const float4*>(&sq[buf][tok][i4 * 64 + rg * 4]);
+          const float4 k4 = *reinterpret_cast<const float4*>(&sk[buf][tok][i4 * 64 + rg * 4]);
+          const f2 qp[2] = {pack2(q4.x, q4.y), pack2(q4.z, q4.w)};
+          const f2 kp[2] = {pack2(k4.x, k4.y), pack2(k4.z, k4.w)};
 #pragma unroll
-          for (int i4 = 0; i4 < R / 4; ++i4) {
-            const float4 q4 = *reinterpret_cast<const float4*>(&sq[buf][tok][i4 * 64 + rg * 4]);
-            const float4 k4 = *reinterpret_cast<const float4*>(&sk[buf][tok][i4 * 64 + rg * 4]);
-            const f2 qp[2] = {pack2(q4.x, q4.y), pack2(q4.z, q4.w)};
-            const f2 kp[2] = {pack2(k4.x, k4.y), pack2(k4.z, k4.w)};
+          for (int j = 0; j < 2; ++j) {
+            const f2 fp = fma2(kp[j], neg2, one2);
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-              const f2 fp = fma2(kp[j], neg2, one2);
-#pragma unroll
-              for (int c = 0; c < C; ++c) {
-                const f2 s = fma2(fp, S[i4 * 2 + j][c], mul2(kp[j], vv[c]));
-                S[i4 * 2 + j][c] = s;
-                acc[c] = fma2(qp[j], s, acc[c]);
-              }
+            for (int c = 0; c < C; ++c) {
+              const f2 s = fma2(fp, S[i4 * 2 + j][c], mul2(kp[j], vv[c]));
+              S[i4 * 2 + j][c] = s;
+              acc[c] = fma2(qp[j], s, acc[c]);
             }
           }
         }
@@ -292,8 +290,14 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
             p.o[(static_cast<long>(t_begin + t0 + tq + u) * p.H + head) * p.dv + col0 + c] = part[i];
         }
       }
+    };
+    if (here == kTok) {                     // full stage: straight-line code, the sums of one group of four tokens
+#pragma unroll                              // overlap the products of the next
+      for (int tq = 0; tq < kTok; tq += 4) four_tokens(tq);
+    } else {
+      for (int tq = 0; tq < here; tq += 4) four_tokens(tq);
     }
-    if (more) stage(buf ^ 1);
+    if (more) stage(buf ^ 1, t0 + kTok);
     __syncthreads();
   }
 
@@ -459,7 +463,7 @@ int pick_cols(const Hgrn2Params& p, int B, cudaStream_t s) {
   // wide tiles spend the fewest instructions per element, narrow ones fill the device when there are few sequences
   const long ctas4 = static_cast<long>(B) * p.H * ((p.dv + 63) / 64);
   if constexpr (R <= 8) {
-    if (ctas4 >= 296) return launch_scan<R, 4>(p, B, s);
+    if (ctas4 >= 192) return launch_scan<R, 4>(p, B, s);
   }
   if (ctas4 >= 120) return launch_scan<R, 2>(p, B, s);
   return launch_scan<R, 1>(p, B, s);

@@ -237,7 +237,6 @@ int dispatch(const StreamParams& p, bool vec4, cudaStream_t s) {
   if (!few || g <= 256) {
     if (g <= 256) return launch<MODE, 32, 4, 2>(p, s);
     if (g <= 512) return launch<MODE, 32, 4, 4>(p, s);
-    if (g <= 1024) return launch<MODE, 32, 4, 8>(p, s);
   }
   if (g <= 1024) return launch<MODE, 256, 4, 1>(p, s);
   if (g <= 4096) return launch<MODE, 256, 4, 4>(p, s);
