@@ -62,6 +62,10 @@ def parse_args():
                     help="no further extra configuration is started once this much time went into them")
     ap.add_argument("--no-check-tokens", dest="check_tokens", action="store_false",
                     help="multi-GPU runs: skip the one-GPU reference pass that the first tokens are compared with")
+    ap.add_argument("--fimodra", action="store_true",
+                    help="instead of the headline workload: kernels and prefill / decode throughput of the Fimodra design at a "
+                         "few layer sizes beside the closest models (one GPU, random weights); one JSON line")
+    ap.add_argument("--fimodra-sizes", type=int, nargs="*", default=None, help="widths for --fimodra (default: all)")
     return ap.parse_args()
 
 
@@ -569,8 +573,24 @@ def run_reference(args) -> dict:
     return run_reference_bench(args, METRIC, BASELINE_TPS)
 
 
+def run_fimodra(args) -> dict:
+    import torch
+
+    from benchmarks import fimodra_shapes
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = fimodra_shapes.run(args.fimodra_sizes or sorted(fimodra_shapes.SIZES))
+    sampler.stop()
+    res["clocks"] = sampler.summary(min_power_w=250.0)
+    return res
+
+
 def main():
     args = parse_args()
+    if args.fimodra:
+        print(json.dumps(run_fimodra(args)), flush=True)
+        return
     res = run_reference(args) if args.impl == "reference" else run_ours(args)
     if res:
         print(json.dumps(res), flush=True)
