@@ -2,7 +2,7 @@
 //
 // Same operand roles as dense_gemm.cu (weight rows on the UMMA M side, tokens on N, both K-major
 // with the 128-byte swizzle, TMA -> shared memory -> tcgen05.mma -> TMEM), but every CTA walks a list
-// of output tiles and keeps TWO accumulators in tensor memory: while the four epilogue warps drain
+// of output tiles and keeps TWO accumulators in tensor memory: while the epilogue warps drain
 // accumulator b (tcgen05.ld -> bias / residual / gated activation -> global), the MMA warp is
 // already filling accumulator b^1 with the next tile and the TMA warp is several k-blocks ahead of
 // it.  With tiles of only 32 k-blocks (K = 2048) the epilogue is a third of a tile's time, which the
@@ -11,7 +11,8 @@
 //   C[T, N] = act(X[T, K] W[N, K]^T) + bias + residual           (dual_rows == 0)
 //   C[T, I] = act(X Wg^T + bg) * (X Wu^T + bu)   with W = [Wg; Wu], bias = [bg; bu]   (dual_rows == I)
 //
-// Warp roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer and TMEM owner, warps 2..5 epilogue.
+// Warp roles (320 threads): warp 0 TMA producer, warp 1 MMA issuer and TMEM owner, warps 2..9 epilogue (two per TMEM
+// quarter, each draining half of the tile's tokens: with short K the epilogue is the longer half of a tile's time).
 // Barriers: full/empty per pipeline stage (running across tiles), acc_full/acc_empty per accumulator.
 // Tile order: consecutive CTAs take different weight tiles of the same 128 tokens, so the token tile
 // is shared through L2 and the weights (a few MB per layer) stay L2-resident across token tiles.
@@ -35,7 +36,8 @@ namespace {
 constexpr int BM = 128;   // weight rows per tile (UMMA M)
 constexpr int BN = 128;   // tokens per tile (UMMA N)
 constexpr int BK = 64;    // k-block: 64 16-bit values = one 128-byte swizzled row
-constexpr int kThreads = 192;
+constexpr int kEpiWarps = 8;
+constexpr int kThreads = 64 + 32 * kEpiWarps;
 
 struct PParams {
   void* C;
@@ -85,13 +87,13 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
   uint64_t* acc_empty = acc_full + 2;         // [2] epilogue -> MMA
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
   volatile int* aborted = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* stage = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(tmem_slot) + 16);   // [4 warps][16 tokens][32 rows]
+  float* stage = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(tmem_slot) + 16);   // [epilogue warps][16 tokens][32 rows]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_launch_dependents();
   if (threadIdx.x == 0) {
     for (int s = 0; s < STAGES; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
-    for (int b = 0; b < 2; ++b) { mbar_init(&acc_full[b], 1); mbar_init(&acc_empty[b], 4); }
+    for (int b = 0; b < 2; ++b) { mbar_init(&acc_full[b], 1); mbar_init(&acc_empty[b], kEpiWarps); }
     *aborted = 0;
     mbar_fence_init();
   }
@@ -178,7 +180,8 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
       }
     }
   } else {
-    // ------------------------------------------------------------ epilogue warps 2..5
+    // ------------------------------------------------------------ epilogue warps
+    const int c_begin = ((warp - 2) >> 2) * (BN / 2), c_end = c_begin + BN / 2;   // this warp's half of the tokens
     const int q = warp & 3;                     // TMEM lane quarter this warp may read
     const int n_local = q * 32 + lane;          // weight row inside the tile
     int local = 0;
@@ -220,15 +223,15 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
           for (int rep = 0; rep < 2; ++rep) {
             const int t = t0 + c0 + vj + rep * 8;
             dst[rep] = make_uint4(0, 0, 0, 0);
-            if (p.residual != nullptr && nv_ok && c0 < BN && t < p.T)
+            if (p.residual != nullptr && nv_ok && c0 < c_end && t < p.T)
               dst[rep] = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.residual) +
                                                          static_cast<size_t>(t) * p.ldc + nv);
           }
         };
         uint4 res_cur[2], res_next[2];
-        load_res(0, res_cur);
+        load_res(c_begin, res_cur);
 #pragma unroll 1
-        for (int c0 = 0; c0 < BN; c0 += 16) {
+        for (int c0 = c_begin; c0 < c_end; c0 += 16) {
           uint32_t r[16], u[16];
           tmem_ld_x16(taddr + hh * BN + c0, r);
           if (DUAL && gated) tmem_ld_x16(taddr + BN + c0, u);
@@ -298,7 +301,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
 template <int STAGES, bool DUAL>
 int launch(const CUtensorMap& tw, const CUtensorMap& tx, const PParams& p, cudaStream_t stream) {
   auto kern = dense_gemm_persistent_kernel<STAGES, DUAL>;
-  constexpr int smem = STAGES * (BM * 128 * (DUAL ? 2 : 1) + BN * 128) + (2 * STAGES + 4) * 8 + 16 + 4 * 16 * 32 * 4 + 1024;
+  constexpr int smem = STAGES * (BM * 128 * (DUAL ? 2 : 1) + BN * 128) + (2 * STAGES + 4) * 8 + 16 + kEpiWarps * 16 * 32 * 4 + 1024;
   {
     cudaError_t e = fi::ensure_dynamic_smem(kern, smem);
     if (e != cudaSuccess) return static_cast<int>(e);
