@@ -40,6 +40,7 @@ struct PrepareParams {
   long ldq, ldkv;
   int T, nh, dim, rot, rdims, rank, q_pitch, nope_off, rot_off, zero_from, max_pos;
   int pairs, vec;           // alignment of all rows and parts: whole pairs, whole 16-byte groups
+  int chunks;               // > 0: 16-byte groups written per head (all parts aligned)
   float eps;
 };
 
@@ -125,6 +126,36 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(const PrepareParams
   }
   const int hd = p.dim + p.rot;
   constexpr int V = 16 / sizeof(T);
+  if (p.chunks > 0) {
+    // everything starts on 16-byte groups: a thread takes whole groups of all heads (copied, turned or cleared);
+    // `chunks` groups per head are written, starting at group 0 of the query or at its rotary part
+    const int total = p.nh * p.chunks, step = 128 * gridDim.y;
+    const int first = p.nope_off >= 0 ? 0 : p.dim;
+#pragma unroll 2
+    for (int i = blockIdx.y * 128 + threadIdx.x; i < total; i += step) {
+      const int h = i / p.chunks, c = first + (i % p.chunks) * V;
+      T* dst = reinterpret_cast<T*>(p.q_out) + (static_cast<long>(t) * p.nh + h) * p.q_pitch +
+               (c >= p.dim ? c - p.dim + p.rot_off : c + p.nope_off);
+      uint4 raw = make_uint4(0, 0, 0, 0);
+      if (c < hd) raw = *reinterpret_cast<const uint4*>(q + static_cast<long>(h) * hd + c);
+      if (c >= p.dim && c < hd) {
+        alignas(16) typename Pair<T>::type v[V / 2];
+        *reinterpret_cast<uint4*>(v) = raw;
+#pragma unroll
+        for (int e = 0; e < V / 2; ++e) {
+          const int pr = (c - p.dim) / 2 + e;
+          if (pr < half) {
+            const float x = to_f(v[e].x), y = to_f(v[e].y), cc = cs[pr], ss = cs[half + pr];
+            v[e].x = from_f<T>(x * cc - y * ss);
+            v[e].y = from_f<T>(y * cc + x * ss);
+          }
+        }
+        raw = *reinterpret_cast<const uint4*>(v);
+      }
+      *reinterpret_cast<uint4*>(dst) = raw;
+    }
+    return;
+  }
   for (int h = blockIdx.y * 4 + warp; h < p.nh; h += 4 * gridDim.y) {
     const T* src = q + static_cast<long>(h) * hd;
     T* dst = reinterpret_cast<T*>(p.q_out) + (static_cast<long>(t) * p.nh + h) * p.q_pitch;
@@ -185,25 +216,32 @@ __global__ void __launch_bounds__(256) latent_pool_kernel(const T* __restrict__ 
   const T* vrow = krow + static_cast<long>(nh) * dim;
   const T* rrow = cache + static_cast<long>(ok ? slot : 0) * (rank + rot) + rank;
   const bool vec = ((dim | rot | vdim | rank) & 7) == 0 && (ldkv & 7) == 0;
+  if (vec) {
+    // hd / 8 groups of K and as many of V per head, spread over the block
+    const int per = hd / 4, total = nh * per;
+    const long row0 = (static_cast<long>(r / BS) * nh * BS + r % BS) * hd;
+#pragma unroll 4
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < total; i += 256 * gridDim.y) {
+      const int h = i / per, c8 = i % per;
+      const bool is_v = c8 >= hd / 8;
+      const int c = (is_v ? c8 - hd / 8 : c8) * 8;
+      const T* src = nullptr;
+      if (ok) {
+        if (is_v) src = c < vdim ? vrow + static_cast<long>(h) * vdim + c : nullptr;
+        else src = c < dim ? krow + static_cast<long>(h) * dim + c : (c < dim + rot ? rrow + c - dim : nullptr);
+      }
+      uint4 v = make_uint4(0, 0, 0, 0);
+      if (src != nullptr) v = *reinterpret_cast<const uint4*>(src);
+      *reinterpret_cast<uint4*>((is_v ? v_pool : k_pool) + row0 + static_cast<long>(h) * BS * hd + c) = v;
+    }
+    return;
+  }
   for (int h = blockIdx.y * 8 + warp; h < nh; h += 8 * gridDim.y) {
     const long dst = ((static_cast<long>(r / BS) * nh + h) * BS + r % BS) * hd;
     for (int c8 = lane; c8 < hd / 4; c8 += 32) {        // hd / 8 chunks of K, then of V
       const bool is_v = c8 >= hd / 8;
       const int c = (is_v ? c8 - hd / 8 : c8) * 8;
       T* out = (is_v ? v_pool : k_pool) + dst + c;
-      if (vec) {
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (ok) {
-          if (is_v) {
-            if (c < vdim) v = *reinterpret_cast<const uint4*>(vrow + static_cast<long>(h) * vdim + c);
-          } else if (c < dim) {
-            v = *reinterpret_cast<const uint4*>(krow + static_cast<long>(h) * dim + c);
-          } else if (c < dim + rot) {
-            v = *reinterpret_cast<const uint4*>(rrow + c - dim);
-          }
-        }
-        *reinterpret_cast<uint4*>(out) = v;
-      } else {
         for (int e = 0; e < 8; ++e) {
           T v = from_f<T>(0.f);
           if (ok) {
@@ -217,7 +255,6 @@ __global__ void __launch_bounds__(256) latent_pool_kernel(const T* __restrict__ 
           }
           out[e] = v;
         }
-      }
     }
   }
 }
@@ -341,6 +378,11 @@ extern "C" int fi_latent_prepare(const void* q, long ldq, const void* dkv, long 
   p.pairs = ((ldq | ldkv | dim | rot | rank | q_pitch | rot_off) & 1) == 0 && (at & (2 * esz - 1)) == 0;
   p.vec = nope_off >= 0 && ldq % v == 0 && (dim + rot) % v == 0 && dim % v == 0 && q_pitch % v == 0 && nope_off % v == 0 &&
           ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(q_out)) & 15) == 0;
+  const bool groups = ((dim | rot | q_pitch | rot_off) % v) == 0 && ldq % v == 0 &&
+                      ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(q_out)) & 15) == 0;
+  if (groups && nope_off < 0) p.chunks = rot / v;
+  // parts in the order [other dimensions | rotary part | cleared]
+  if (groups && nope_off == 0 && rot_off == dim && zero_from == dim + rot) p.chunks = q_pitch / v;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid(T, T >= 256 ? 1 : (nh + 3) / 4);
 #define FI_CALL(TT) return static_cast<int>(fi::launch_kernel(latent_prepare_kernel<TT>, grid, dim3(128), 0, s, 0, p))
