@@ -189,10 +189,11 @@ def kernel_rows(width: int, iters: int = 10) -> list[dict]:
     table = i32([[1 + b * (ctx // 16) + j for j in range(ctx // 16)] for b in range(B)])
     qc, q5, ln = rnd(B, H, kd), rnd(B, H, 576), i32([ctx] * B)
     seen = min(window, ctx)
+    short = i32([seen] * B)            # the like kernel has no window: a context of as many tokens
     case(f"latent attention rows, decode batch {B}, window {window}",
          lambda: la.attend_rows(qc, cache, table, ln, None, rank, 0.1, window, sinks, ctx), B * seen * kd * 2, 2.0 * B * seen * H * (kd + rank),
-         like=(f"DeepSeek MLA decode, context {ctx}", lambda: la.attend_rows(q5, cache576, table, ln, None, 512, 0.1, 0, None, ctx),
-               B * ctx * 576 * 2, 2.0 * B * ctx * H * (576 + 512), tensor))
+         like=(f"DeepSeek MLA decode, context {seen}", lambda: la.attend_rows(q5, cache576, table, short, None, 512, 0.1, 0, None, seen),
+               B * seen * 576 * 2, 2.0 * B * seen * H * (576 + 512), tensor))
     return rows
 
 

@@ -19,13 +19,15 @@
 //                       the scores (36 k-steps of mma.sync m16n8k16, each warp 16 of the 64 tokens) and,
 //                       through ldmatrix.trans, as V for the output (each warp 128 of the 512 latent
 //                       channels over all 64 tokens; P goes through shared memory once per chunk).
-//   mla_merge_kernel    combines the split partials.
+//                       Up to 8 splits form a thread-block cluster and merge through distributed shared memory.
+//   mla_merge_kernel    combines the split partials when there are more splits.
 //   mla_ctx_to_pool_kernel  prefill: up-projected context rows -> padded per-head K/V rows of a temporary pool
 // A "row" is a (sequence, query token): decode batches have one row per sequence; rows may also carry their
 // own visible length and point at their sequence's block table (seq_of_row), the flattening the reference
 // uses for its prefill (vllm/engine/lite_engine.py:53-104).  The model itself prefills in the per-head form
 // on a temporary pool (many query rows per sequence amortise a K/V tile there).
 // The reference keeps per-head K/V for this model family; the absorbed form follows the DeepSeek-V2 paper.
+#include <cooperative_groups.h>
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
@@ -115,6 +117,7 @@ struct MlaParams {
   float sm_scale;
   const float* sinks;         // [nh] or null
   int window;                 // > 0: only the last `window` rows of the visible ones count
+  int cluster;                // 1: the split CTAs are one cluster and merge in the kernel
   int kd, vd, pitch;          // run-time geometry: row width, latent width, shared-memory pitch (elements)
 };
 
@@ -145,17 +148,14 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
   const int c_begin = c_first + split * per, c_end = min(c_first + n_chunks, c_begin + per);
 
   if constexpr (KDT == 0) {             // columns between the row width and the pitch are read as zero
-    for (int i = threadIdx.x; i < (CH + 16) * pitch / 8; i += 128)
-      *reinterpret_cast<uint4*>(sK + i * 8) = make_uint4(0, 0, 0, 0);
-    __syncthreads();
+    const int pad = (pitch - kd) / 8;
+    for (int i = threadIdx.x; i < (CH + 16) * pad; i += 128)
+      *reinterpret_cast<uint4*>(sK + (i / pad) * pitch + kd + (i % pad) * 8) = make_uint4(0, 0, 0, 0);
   }
-  for (int i = threadIdx.x; i < 16 * (kd / 8); i += 128) {
-    const int row = i / (kd / 8), c = i % (kd / 8);
-    uint4 v = make_uint4(0, 0, 0, 0);
-    if (row < heads_here)
-      v = *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.q_cat) +
-                                          (static_cast<long>(r) * p.nh + head0 + row) * kd + c * 8);
-    *reinterpret_cast<uint4*>(sQ + row_off<KDT>(row, c, pitch)) = v;
+  for (int row = warp * 4; row < warp * 4 + 4; ++row) {      // the queries arrive with the first chunk
+    const bool have = row < heads_here;
+    const T* src = reinterpret_cast<const T*>(p.q_cat) + (static_cast<long>(r) * p.nh + head0 + (have ? row : 0)) * kd;
+    for (int ch = lane; ch < kd / 8; ch += 32) cp_async16(sQ + row_off<KDT>(row, ch, pitch), src + ch * 8, have);
   }
   float o[VB * 2][4];                   // 16 rows x this warp's quarter of the latent channels
 #pragma unroll
@@ -257,6 +257,7 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
     }
     __syncthreads();        // the next chunk overwrites sK, sP and sMax
   }
+  cp_async_wait_all();      // a split without chunks still has its queries in flight
   // ---- denominators: quad sums, then the four warps' shares
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
@@ -269,6 +270,53 @@ __global__ void __launch_bounds__(128) mla_decode_kernel(const MlaParams p) {
 #pragma unroll
   for (int w = 0; w < 4; ++w) { lt0 += sMax[w * 16 + (lane >> 2)]; lt1 += sMax[w * 16 + (lane >> 2) + 8]; }
   const int r0 = lane >> 2, r1 = r0 + 8;
+  if (p.cluster) {
+    namespace cg = cooperative_groups;
+    cg::cluster_group cluster = cg::this_cluster();
+    float* so = reinterpret_cast<float*>(sK);               // [16][VB * 64] sums of this split (the tile is done with)
+    float* sml = reinterpret_cast<float*>(sQ);              // [16][2] maximum, denominator
+    constexpr int OW = VB * 64;
+#pragma unroll
+    for (int i = 0; i < VB * 2; ++i) {
+      const int d = warp * (VB * 16) + i * 8 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(so + r0 * OW + d) = make_float2(o[i][0], o[i][1]);
+      *reinterpret_cast<float2*>(so + r1 * OW + d) = make_float2(o[i][2], o[i][3]);
+    }
+    if (warp == 0 && (lane & 3) == 0) {
+      sml[2 * r0] = m0; sml[2 * r0 + 1] = lt0;
+      sml[2 * r1] = m1; sml[2 * r1 + 1] = lt1;
+    }
+    cluster.sync();
+    T* out = reinterpret_cast<T*>(p.out);
+    for (int row = split; row < heads_here; row += p.splits) {
+      float m = -CUDART_INF_F, l = 0.f, w[8];
+#pragma unroll
+      for (int s = 0; s < 8; ++s) w[s] = s < p.splits ? cluster.map_shared_rank(sml, s)[2 * row] : -CUDART_INF_F;
+#pragma unroll
+      for (int s = 0; s < 8; ++s) m = fmaxf(m, w[s]);
+#pragma unroll
+      for (int s = 0; s < 8; ++s) {
+        w[s] = w[s] == -CUDART_INF_F ? 0.f : exp2f(w[s] - m);
+        if (s < p.splits) l += w[s] * cluster.map_shared_rank(sml, s)[2 * row + 1];
+      }
+      if (p.sinks != nullptr && m != -CUDART_INF_F) l += exp2f(p.sinks[head0 + row] * kLog2e - m);
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+      for (int d = threadIdx.x * 2; d < vd; d += 256) {
+        float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int s = 0; s < 8; ++s)
+          if (s < p.splits) {
+            const float2 v = *reinterpret_cast<const float2*>(cluster.map_shared_rank(so, s) + row * OW + d);
+            acc.x = fmaf(w[s], v.x, acc.x);
+            acc.y = fmaf(w[s], v.y, acc.y);
+          }
+        *reinterpret_cast<uint32_t*>(out + (head0 + row) * p.out_head_stride + r * p.out_row_stride + d) =
+            Mma<T>::pack(acc.x * inv, acc.y * inv);
+      }
+    }
+    cluster.sync();          // nobody leaves while its tile is being read
+    return;
+  }
   if (p.splits == 1) {
     if (p.sinks != nullptr) {             // scores are in units of log2: so is the sink
       if (r0 < heads_here && m0 != -CUDART_INF_F) lt0 += exp2f(p.sinks[head0 + r0] * kLog2e - m0);
@@ -478,6 +526,10 @@ int launch_decode(const MlaParams& p, int rows, cudaStream_t s) {
   auto kern = mla_decode_kernel<T, KDT, VB>;
   cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
   if (ce != cudaSuccess) return static_cast<int>(ce);
+  if (p.cluster) {
+    ce = fi::launch_kernel_cluster(kern, dim3(p.splits, (p.nh + 15) / 16, rows), dim3(128), smem, s, dim3(p.splits, 1, 1), p);
+    return static_cast<int>(ce != cudaSuccess ? ce : cudaGetLastError());
+  }
   fi::launch_kernel(kern, dim3(p.splits, (p.nh + 15) / 16, rows), dim3(128), smem, s, 0, p);
   if (p.splits > 1) fi::launch_kernel(mla_merge_kernel<T>, dim3(p.nh, rows), dim3(128), 0, s, 0, p);
   return static_cast<int>(cudaGetLastError());
@@ -495,14 +547,15 @@ int dispatch_decode(const MlaParams& p, int rows, cudaStream_t s) {
 }  // namespace
 
 // Attention of flattened rows over the shared cache rows [latent (vd) | rotary key] of kd values.
-// ws_o: rows * nh * splits * vd floats, ws_ml: rows * nh * splits * 2 floats (splits > 1 only).  window <= 0: none;
+// Up to 8 splits without ws_o / ws_ml merge inside a cluster; otherwise ws_o: rows * nh * splits * vd floats, ws_ml:
+// rows * nh * splits * 2 floats.  window <= 0: none;
 // sinks: fp32 [nh] or null.  Returns -12 for a geometry the kernel does not cover (the caller takes the general one).
 extern "C" int fi_mla_decode(const void* q_cat, const void* cache, void* out, long out_head_stride,
                              long out_row_stride, const int* block_tables, const int* row_lens, const int* seq_of_row,
                              float* ws_o, float* ws_ml, int rows, int nh, int kd, int vd, int max_blocks, int block_size,
                              int splits, int window, const float* sinks, float sm_scale, int dtype, void* stream) {
   if (rows <= 0 || nh <= 0) return 0;
-  if (splits < 1 || block_size <= 0 || (splits > 1 && (ws_o == nullptr || ws_ml == nullptr)) || vd > kd) return -10;
+  if (splits < 1 || block_size <= 0 || (splits > 8 && (ws_o == nullptr || ws_ml == nullptr)) || vd > kd) return -10;
   if (kd % 8 != 0 || vd % 2 != 0 || vd <= 0 || vd > 512 || kd > 640 || rows > 65535) return -12;
   if ((reinterpret_cast<uintptr_t>(q_cat) | reinterpret_cast<uintptr_t>(cache)) & 15) return -10;
   if (out_head_stride % 2 != 0 || out_row_stride % 2 != 0) return -12;
@@ -511,6 +564,7 @@ extern "C" int fi_mla_decode(const void* q_cat, const void* cache, void* out, lo
   p.block_tables = block_tables; p.row_lens = row_lens; p.seq_of_row = seq_of_row; p.ws_o = ws_o; p.ws_ml = ws_ml;
   p.nh = nh; p.max_blocks = max_blocks; p.block_size = block_size; p.splits = splits; p.sm_scale = sm_scale;
   p.window = window; p.sinks = sinks; p.kd = kd; p.vd = vd;
+  p.cluster = splits > 1 && (ws_o == nullptr || ws_ml == nullptr);
   const int vcols = vd <= 64 ? 64 : vd <= 128 ? 128 : vd <= 256 ? 256 : 512;
   const int kcols = (kd + 15) / 16 * 16;
   p.pitch = (kcols > vcols ? kcols : vcols) + 8;

@@ -97,9 +97,10 @@ def attend_rows(q_cat, cache, block_tables, row_lens, seq_of_row, rank: int, sca
         seen = min(int(max_len), window + 63) if window else int(max_len)
         chunks = max(1, (seen + 63) // 64)
         ctas = max(1, R * ((nh + 15) // 16))
-        splits = int(max(1, min((2 * 148 + ctas - 1) // ctas, chunks, 16)))
+        # up to 8 splits merge inside a thread-block cluster; long contexts of few rows take more, merged by a kernel
+        splits = int(max(1, min(2 * 148 // ctas, chunks, 16 if chunks > 64 else 8)))
         ws_o = ws_ml = None
-        if splits > 1:
+        if splits > 8:
             n_o = R * nh * splits * rank
             ws = scratch("mla_ws", (n_o + R * nh * splits * 2) * 4, dev).view(torch.float32)
             ws_o, ws_ml = ws[:n_o], ws[n_o:]
@@ -107,7 +108,7 @@ def attend_rows(q_cat, cache, block_tables, row_lens, seq_of_row, rank: int, sca
                                _p(seq_of_row), _p(ws_o), _p(ws_ml), R, nh, kd, rank, block_tables.shape[1], bs, splits,
                                int(window), _p(sinks), scale, dt, _stream())
         _lib.check(rc, "fi_mla_decode")
-        _count(2 if splits > 1 else 1)
+        _count(2 if splits > 8 else 1)
         return out
     rc = lib.fi_latent_rows(_p(q_cat), _p(cache), _p(out), out.stride(0), out.stride(1), _p(block_tables), _p(row_lens),
                             _p(seq_of_row), R, nh, kd, rank, block_tables.shape[1], bs, cache.shape[0] * bs, int(window),

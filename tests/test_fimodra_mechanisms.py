@@ -376,3 +376,23 @@ def test_scan_of_16_bit_projections(H, d, dv):
     want, S = O.outer_product_recurrence(qa, fa, va, torch.zeros(H, d, dv))
     close(o, want, 2e-5)
     close(pool[1], S, 2e-5)
+
+
+@gpu
+@pytest.mark.parametrize("n, window", [(600, 0), (4300, 0), (4300, 70), (9000, 4200)])
+def test_few_rows_over_long_contexts(n, window):
+    """One row split over many blocks, merged inside a cluster or by the merge kernel; far keys stand out."""
+    nh, rank, rot = 3, 128, 16
+    kd = rank + rot
+    rows = rnd(n, kd, seed=1, std=0.3).bfloat16()
+    pages = Paged([n], kd, 16, torch.bfloat16, "cuda")
+    pages.fill(0, rows)
+    first = max(0, n - window) if window else 0
+    q = rnd(1, nh, kd, seed=2, std=0.3).bfloat16()
+    q[0, 0] += 2 * rows[first]
+    q[0, 1] += 2 * rows[max(0, first - 1)]
+    sink = torch.tensor([1.0, 0.0, 3.0])
+    got = la.attend_rows(q.cuda(), pages.cache, pages.table.cuda(), torch.tensor([n], dtype=torch.int32, device="cuda"), None, rank, 0.4,
+                         window, sink.cuda(), n)[:, 0]
+    k = rows.float()[:, None].expand(n, nh, kd)
+    close(got.float(), O.sink_attention(q.float(), k, k[..., :rank], 0.4, window, sink)[0], 1.5e-2)
