@@ -2,7 +2,7 @@
 the models the framework served before (DeepSeek-style latent attention, the gated delta rule, RMSNorm) and beside a
 Qwen3.5-style hybrid decoder of equal width, depth, feed-forward and vocabulary.  Random weights, one GPU.
 
-    python benchmarks/fimodra_shapes.py [--kernels] [--models] [--sizes 1024 2048 4096] [--json out.json]
+    python benchmarks/fimodra_shapes.py [--kernels] [--models] [--sizes 1024 2048 4096] [--only TEXT] [--json out.json]
 
 A kernel's roofline time is the larger of its algorithmic bytes over the measured copy bandwidth and its FLOPs over the
 measured product rate (MEASURED_PEAKS.json); "x roofline" is the measured time over that.  Caches are flushed between
@@ -56,7 +56,7 @@ class Timer:
         return statistics.median(out)
 
 
-def kernel_rows(width: int, iters: int = 10) -> list[dict]:
+def kernel_rows(width: int, iters: int = 10, only: str = "") -> list[dict]:
     import torch
 
     from litevllm_b200 import ops
@@ -80,10 +80,12 @@ def kernel_rows(width: int, iters: int = 10) -> list[dict]:
     rows = []
 
     def case(name, fn, nbytes, flops=0.0, peak=tensor, like=None):
+        if only not in name:
+            return
         us = time_us(fn)
         roof = max(nbytes / (hbm * 1e3), flops / (peak * 1e6))
         r = {"width": width, "kernel": name, "us": round(us, 1), "roofline_us": round(roof, 1), "x_roofline": round(us / roof, 2)}
-        if like is not None:
+        if like is not None and not only:
             lname, lfn, lbytes, lflops, lpeak = like
             lus = time_us(lfn)
             lroof = max(lbytes / (hbm * 1e3), lflops / (lpeak * 1e6))
@@ -273,13 +275,13 @@ def model_rows(width: int, layers: int = 8, batch: int = 32, prompt: int = 1024,
     return rows
 
 
-def run(sizes, kernels: bool = True, models: bool = True) -> dict:
+def run(sizes, kernels: bool = True, models: bool = True, only: str = "") -> dict:
     import torch
     torch.cuda.set_device(0)
     out = {"metric": "Fimodra kernels and throughput beside the closest models", "peaks": _peaks(), "tokens": TOKENS}
     if kernels:
         with torch.inference_mode():
-            out["kernels"] = [r for w in sizes for r in kernel_rows(w)]
+            out["kernels"] = [r for w in sizes for r in kernel_rows(w, only=only)]
     if models:
         out["models"] = [r for w in sizes for r in model_rows(w)]
     return out
@@ -290,10 +292,11 @@ def main() -> None:
     ap.add_argument("--kernels", action="store_true")
     ap.add_argument("--models", action="store_true")
     ap.add_argument("--sizes", type=int, nargs="*", default=sorted(SIZES))
+    ap.add_argument("--only", default="", help="kernel cases whose name contains this (without the like kernels)")
     ap.add_argument("--json", default=None)
     a = ap.parse_args()
     both = a.kernels == a.models
-    res = run(a.sizes, a.kernels or both, a.models or both)
+    res = run(a.sizes, a.kernels or both, a.models or both, a.only)
     for r in res.get("kernels", []):
         print(f"{r['width']:5d} {r['kernel']:58s} {r['us']:9.1f} us  {r['x_roofline']:7.2f} x roofline"
               + (f"   | {r['like']:38s} {r['like_us']:9.1f} us {r['like_x_roofline']:7.2f} x" if "like" in r else ""))

@@ -318,7 +318,7 @@ __global__ void __launch_bounds__(kWarps * 32) hgrn2_scan_kernel(const Hgrn2Para
 
 // One token per sequence.  Block: one (head, sequence); thread: VEC columns of every RY-th row.
 template <int VEC>
-__global__ void __launch_bounds__(256) hgrn2_step_kernel(const Hgrn2Params p) {
+__global__ void __launch_bounds__(256, 3) hgrn2_step_kernel(const Hgrn2Params p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   extern __shared__ float smem[];
