@@ -90,7 +90,8 @@ def build_vllm_config(model: str, **kwargs: Any) -> VllmConfig:
         synthetic = True
     arch = arch_from_hf_config(hf_cfg)
 
-    dtype = resolve_dtype(kwargs.get("dtype") or hf_cfg.get("torch_dtype") or hf_cfg.get("dtype") or "bfloat16")
+    asked = kwargs.get("dtype")
+    dtype = resolve_dtype((None if asked == "auto" else asked) or hf_cfg.get("torch_dtype") or hf_cfg.get("dtype") or "bfloat16")
     max_len = int(kwargs.get("max_model_len") or min(arch.max_position, 4096))
     seqs = int(kwargs.get("max_num_seqs") or kwargs.get("concurrent_reqs") or 8)
     batched = int(kwargs.get("max_num_batched_tokens") or max(8192, seqs * min(max_len, 1024)))
