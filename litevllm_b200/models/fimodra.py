@@ -64,6 +64,21 @@ class FimodraLayer(nn.Module):
             self.mlp = DenseMLP(W, spec["mlp"]["ff"], dtype, arch.act)
             self.norm2, self.norm2b = _fp32(W), _fp32(W)
         self.depth_weights = nn.Parameter(torch.zeros(i + 2, dtype=torch.float32), requires_grad=False)
+        self.index, self.eps, self.groups = i, eps, int(arch.extra["norm_groups"])
+
+    def forward(self, h, src, x, hist, batch, kv_caches, next_norm, sel=None):
+        """h: this layer's normalised input; src: the stream before it (fp32); x: buffer that receives what the layer
+        hands on; hist: results X_0 .. X_i, X_(i+1) is added.  Returns the next sublayer's input (rows ``sel`` only)."""
+        i = self.index
+        with stage("layer.mixer"):
+            y = self.mixer(h, batch, kv_caches[i][0] if self.kind == "latent_attention" else kv_caches.states[i])
+        post = self.norm1b
+        if self.mlp is not None:
+            with stage("layer.mlp"):
+                h = stream.step(y, src, post, self.norm2, self.eps, self.groups, x, h.dtype)
+                y = self.mlp(h)
+            src, post = x, self.norm2b
+        return stream.average(y, src, post, next_norm, self.eps, self.groups, hist, i + 1, self.depth_weights, x, h.dtype, sel)
 
 
 class FimodraForCausalLM(nn.Module):
@@ -102,19 +117,8 @@ class FimodraForCausalLM(nn.Module):
         for i, layer in enumerate(self.layers):
             last = i + 1 == L
             nxt = self.final_norm if last else self.layers[i + 1].norm1
-            with stage("layer.mixer"):
-                if layer.kind == "latent_attention":
-                    y = layer.mixer(h, batch, kv_caches[i][0])
-                else:
-                    y = layer.mixer(h, batch, kv_caches.states[i])
-            post = layer.norm1b
-            if layer.mlp is not None:
-                with stage("layer.mlp"):
-                    h = stream.step(y, src, post, layer.norm2, self.eps, self.groups, x, self.dtype)
-                    y = layer.mlp(h)
-                src, post = x, layer.norm2b
             sel = batch.logits_indices if last and collect is None else None
-            h = stream.average(y, src, post, nxt, self.eps, self.groups, hist, i + 1, layer.depth_weights, x, self.dtype, sel)
+            h = layer(h, src, x, hist, batch, kv_caches, nxt, sel)
             src = x
             if collect is not None:
                 collect.append(x.clone())
