@@ -4,7 +4,7 @@
 
 Steps arrive on standard input, one JSON object a line::
 
-    {"step": 0, "entries": [{"id": "a", "tokens": [5, 17, 3], "want": [0, 2]}], "end": []}
+    {"step": 7, "entries": [{"id": "q1", "tokens": [12, 9], "want": [1]}, {"id": "q2", "tokens": [4], "want": []}], "end": ["q1"]}
 
 All entries of a step run as one batch of the engine, portions of prompts beside single tokens, through the executors,
 the paged cache and the state slots that generation uses; nothing is sampled.  A step that wants logits leaves
