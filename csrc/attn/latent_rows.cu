@@ -7,7 +7,8 @@
 //   latent_pool_kernel      up-projected keys and values + the cached rotary keys -> padded per-head K / V tiles of a
 //                           temporary pool that the prefill attention kernels read
 //   latent_rows_kernel      a warp per (row, head): scores against the cache rows, softmax with window and sink, sum of
-//                           latents.  Runs 32-bit models and geometries outside the tensor-core kernels.
+//                           latents (or of the rows of a value cache, with grouped heads and an output gate).  Runs
+//                           32-bit models and geometries outside the tensor-core kernels.
 // Rotation pairs are neighbours: channels (2i, 2i + 1) turn by the angle of frequency i; cos_sin rows are
 // [cos(dims / 2) | sin(dims / 2)].  Positions, angles, norms, scores and weights are 32-bit.
 #include <cuda_bf16.h>
@@ -261,7 +262,11 @@ __global__ void __launch_bounds__(256) latent_pool_kernel(const T* __restrict__ 
 
 struct RowsParams {
   const void* q_cat;        // [rows, nh, kd]
-  const void* cache;        // rows of kd values; the first vd are the value
+  const void* cache;        // [blocks, nkv, block size] rows of kd values
+  const void* v_cache;      // the same with rows of vd values; null: the first vd values of a cache row are the value
+  const void* gate;         // [rows, >= nh * vd] of pitch gate_stride or null: out *= sigmoid(gate)
+  long gate_stride;
+  int nkv;
   void* out;                // element (row r, head h, d) at out + h * out_head_stride + r * out_row_stride + d
   long out_head_stride, out_row_stride;
   const int* block_tables;
@@ -289,6 +294,8 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
   const int lo = p.window > 0 ? max(0, len - p.window) : 0;
   const int* bt = p.block_tables + static_cast<long>(p.seq_of_row ? p.seq_of_row[r] : r) * p.max_blocks;
   const T* cache = reinterpret_cast<const T*>(p.cache);
+  const T* values = reinterpret_cast<const T*>(p.v_cache != nullptr ? p.v_cache : p.cache);
+  const int vpitch = p.v_cache != nullptr ? p.vd : p.kd, kvh = h / (p.nh / p.nkv);
   float o[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) o[i] = 0.f;
@@ -298,9 +305,10 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
     long src = 0;
     float s = -CUDART_INF_F;
     if (tok < len) {
-      src = (static_cast<long>(bt[tok / p.block_size]) * p.block_size + tok % p.block_size);
-      src = (src < 0 || src >= p.num_rows ? 0 : src) * p.kd;
-      const T* row = cache + src;
+      long blk = bt[tok / p.block_size];
+      blk = blk < 0 || (blk + 1) * p.block_size > p.num_rows ? 0 : blk;
+      src = (blk * p.nkv + kvh) * p.block_size + tok % p.block_size;
+      const T* row = cache + src * p.kd;
       float a0 = 0.f, a1 = 0.f;
       int i = 0;
       for (; i + 1 < p.kd; i += 2) { a0 = fmaf(q[i], to_f(row[i]), a0); a1 = fmaf(q[i + 1], to_f(row[i + 1]), a1); }
@@ -321,7 +329,7 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
     const int n = min(32, len - k0);
     for (int j = 0; j < n; ++j) {
       const float pj = __shfl_sync(0xffffffffu, pv, j);
-      const T* row = cache + __shfl_sync(0xffffffffu, src, j);
+      const T* row = values + __shfl_sync(0xffffffffu, src, j) * vpitch;
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (i * 32 + lane < p.vd) o[i] = fmaf(pj, to_f(row[i * 32 + lane]), o[i]);
@@ -332,7 +340,12 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
   T* out = reinterpret_cast<T*>(p.out) + h * p.out_head_stride + r * p.out_row_stride;
 #pragma unroll
   for (int i = 0; i < NV; ++i)
-    if (i * 32 + lane < p.vd) out[i * 32 + lane] = from_f<T>(o[i] * inv);
+    if (i * 32 + lane < p.vd) {
+      float v = o[i] * inv;
+      if (p.gate != nullptr)
+        v /= 1.f + __expf(-to_f(reinterpret_cast<const T*>(p.gate)[r * p.gate_stride + h * p.vd + i * 32 + lane]));
+      out[i * 32 + lane] = from_f<T>(v);
+    }
 }
 
 template <typename T>
@@ -439,7 +452,31 @@ extern "C" int fi_latent_rows(const void* q_cat, const void* cache, void* out, l
   p.q_cat = q_cat; p.cache = cache; p.out = out; p.out_head_stride = out_head_stride; p.out_row_stride = out_row_stride;
   p.block_tables = block_tables; p.row_lens = row_lens; p.seq_of_row = seq_of_row; p.sinks = sinks; p.rows = rows;
   p.nh = nh; p.kd = kd; p.vd = vd; p.max_blocks = max_blocks; p.block_size = block_size; p.num_rows = num_rows;
-  p.window = window; p.sm_scale = sm_scale;
+  p.window = window; p.sm_scale = sm_scale; p.nkv = 1;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define FI_CALL(TT) return launch_rows<TT>(p, s)
+  FI_BY_TYPE(dtype, FI_CALL)
+#undef FI_CALL
+  return 0;
+}
+
+// The same over separate key and value caches [blocks, nkv, block_size, kd | vd] (query head h reads key / value head
+// h / (nh / nkv)): q [rows, nh, kd], out [rows, nh * vd]; row r sees the first row_lens[r] tokens (the last `window` of
+// them) of sequence seq_of_row[r] (null: sequence r); gate: rows of pitch gate_stride in the type of out, or null.
+extern "C" int fi_attn_rows(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_tables,
+                            const int* row_lens, const int* seq_of_row, int rows, int nh, int nkv, int kd, int vd,
+                            int max_blocks, int block_size, int num_blocks, int window, const float* sinks,
+                            const void* gate, long gate_stride, float sm_scale, int dtype, void* stream) {
+  if (rows <= 0 || nh <= 0) return 0;
+  if (kd <= 0 || vd <= 0 || vd > 1024 || kd > 2048 || block_size <= 0 || max_blocks <= 0 || num_blocks <= 0 || nkv <= 0 ||
+      nh % nkv != 0 || v_cache == nullptr)
+    return -10;
+  RowsParams p = {};
+  p.q_cat = q; p.cache = k_cache; p.v_cache = v_cache; p.out = out; p.out_head_stride = vd;
+  p.out_row_stride = static_cast<long>(nh) * vd; p.block_tables = block_tables; p.row_lens = row_lens;
+  p.seq_of_row = seq_of_row; p.sinks = sinks; p.rows = rows; p.nh = nh; p.nkv = nkv; p.kd = kd; p.vd = vd;
+  p.max_blocks = max_blocks; p.block_size = block_size; p.num_rows = num_blocks * block_size; p.window = window;
+  p.sm_scale = sm_scale; p.gate = gate; p.gate_stride = gate_stride;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_CALL(TT) return launch_rows<TT>(p, s)
   FI_BY_TYPE(dtype, FI_CALL)

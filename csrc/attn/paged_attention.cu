@@ -114,11 +114,28 @@ struct AttnParams {
   // partials through distributed shared memory at this byte offset of the dynamic shared memory
   // ([16][HD] sums + [16][2] max/denominator per CTA): no global scratch, no tickets, no second launch
   int cluster_off;
-  // prefill: fp32 [nh] or null, one extra exp(sink) per head in the softmax denominator; channels of a head
-  // that are stored (0 = HD)
+  // fp32 [nh] or null, one extra exp(sink) per head in the softmax denominator; channels of a head that are stored
+  // (0 = HD; rows of nh * out_dim); output gate: row t at gate + t * gate_stride (same type as out, channels as in
+  // out) or null, out is multiplied by sigmoid(gate)
   const float* sinks;
   int out_dim;
+  const void* gate;
+  long gate_stride;
 };
+
+// Scatter of one finished channel: sum of exponentials l, reference m, accumulated value acc.
+template <typename T, int HD>
+__device__ __forceinline__ void store_decoded(const AttnParams& p, int b, int head, int d, float acc, float l, float m) {
+  const int od = p.out_dim > 0 ? p.out_dim : HD;
+  if (d >= od) return;
+  if (p.sinks != nullptr && m != -CUDART_INF_F) l += exp2f((p.sinks[head] - m) * kLog2e);
+  float v = l > 0.f ? acc / l * (p.kv_fp8 == 1 ? p.v_scale : 1.f) : 0.f;
+  if (p.gate != nullptr) {
+    const float g = static_cast<float>(reinterpret_cast<const T*>(p.gate)[b * p.gate_stride + head * od + d]);
+    v /= 1.f + __expf(-g);
+  }
+  reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * od + d] = MmaT<T>::from_f(v);
+}
 
 // Load `rows` KV tokens starting at token tok0 of sequence b / kv head kvh into a swizzled tile.
 // Tokens outside [lo, hi) are zero-filled.
@@ -357,8 +374,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
     }
     const int head = head0 + r;
     if (p.splits == 1) {
-      const float v = l > 0.f ? acc / l * (p.kv_fp8 == 1 ? p.v_scale : 1.f) : 0.f;
-      reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * HD + d] = MmaT<T>::from_f(v);
+      store_decoded<T, HD>(p, b, head, d, acc, l, m);
     } else {
       const long base = (static_cast<long>(b) * p.nh + head) * p.splits + split;
       p.ws_o[base * HD + d] = acc;
@@ -585,8 +601,7 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
     }
     const int head = head0 + r;
     if (p.splits == 1) {
-      const float v = l > 0.f ? acc / l * (fp8 ? p.v_scale : 1.f) : 0.f;
-      reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * HD + d] = MmaT<T>::from_f(v);
+      store_decoded<T, HD>(p, b, head, d, acc, l, m);
     } else if (p.cluster_off > 0) {
       float* cO = reinterpret_cast<float*>(smem_raw + p.cluster_off);
       cO[i] = acc;
@@ -627,8 +642,7 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
           l += f * peer[16 * HD + r * 2 + 1];
         }
       }
-      const float v = l > 0.f ? acc / l * (fp8 ? p.v_scale : 1.f) : 0.f;
-      reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head0) * HD + i] = MmaT<T>::from_f(v);
+      store_decoded<T, HD>(p, b, head0 + r, i % HD, acc, l, m);
     }
     cluster.sync();
   } else if (p.splits > 1 && p.merge_tickets != nullptr) {
@@ -658,8 +672,7 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
           acc += f * __ldcg(p.ws_o + (base + sidx) * HD + d);
           l += f * __ldcg(p.ws_ml + (base + sidx) * 2 + 1);
         }
-        const float v = l > 0.f ? acc / l * (fp8 ? p.v_scale : 1.f) : 0.f;
-        reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head0 + r) * HD + d] = MmaT<T>::from_f(v);
+        store_decoded<T, HD>(p, b, head0 + r, d, acc, l, m);
       }
     }
   }
@@ -681,8 +694,7 @@ __global__ void decode_merge_kernel(const AttnParams p) {
       acc += f * p.ws_o[(base + s) * HD + d];
       l += f * p.ws_ml[(base + s) * 2 + 1];
     }
-    const float v = l > 0.f ? acc / l * (p.kv_fp8 == 1 ? p.v_scale : 1.f) : 0.f;
-    reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * HD + d] = MmaT<T>::from_f(v);
+    store_decoded<T, HD>(p, b, head, d, acc, l, m);
   }
 }
 
@@ -844,13 +856,17 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   for (int i = 0; i < HD / 8; ++i) {
     const int d = i * 8 + (lane & 3) * 2;
     if (d >= od) break;
-    if (row0 < q_len) {
-      const long off = (static_cast<long>(q_begin + row0) * p.nh + head) * od + d;
-      *reinterpret_cast<uint32_t*>(out + off) = MmaT<T>::pack(o[i][0] * i0, o[i][1] * i0);
-    }
-    if (row0 + 8 < q_len) {
-      const long off = (static_cast<long>(q_begin + row0 + 8) * p.nh + head) * od + d;
-      *reinterpret_cast<uint32_t*>(out + off) = MmaT<T>::pack(o[i][2] * i1, o[i][3] * i1);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int row = row0 + 8 * h;
+      if (row >= q_len) continue;
+      float a = o[i][2 * h] * (h ? i1 : i0), bb = o[i][2 * h + 1] * (h ? i1 : i0);
+      if (p.gate != nullptr) {
+        const T* g = reinterpret_cast<const T*>(p.gate) + (q_begin + row) * p.gate_stride + head * od + d;
+        a /= 1.f + __expf(-static_cast<float>(g[0]));
+        bb /= 1.f + __expf(-static_cast<float>(g[1]));
+      }
+      *reinterpret_cast<uint32_t*>(out + (static_cast<long>(q_begin + row) * p.nh + head) * od + d) = MmaT<T>::pack(a, bb);
     }
   }
 }
@@ -908,13 +924,16 @@ int launch_prefill(const AttnParams& p, int B, int max_q_len, cudaStream_t s) {
 
 }  // namespace
 
-// Decode scratch: ws_o needs B*nh*splits*hd floats, ws_ml B*nh*splits*2 floats (splits > 1 only).
+// Decode scratch: ws_o needs B*nh*splits*hd floats, ws_ml B*nh*splits*2 floats (splits > 1 only).  sinks: fp32 [nh] or
+// null; out_dim: stored channels per head (0 = hd), out rows are nh * out_dim wide; gate: rows of pitch gate_stride in
+// the type of out, or null.
 extern "C" int fi_paged_decode(const void* q, long q_stride, const void* k_cache,
                                const void* v_cache, void* out, const int* block_tables,
                                const int* seq_lens, float* ws_o, float* ws_ml, int B, int nh,
                                int nkv, int hd, int max_blocks, int block_size, int window,
                                float sm_scale, float softcap, int kv_fp8, float k_scale,
-                               float v_scale, int splits, int dtype, void* stream) {
+                               float v_scale, int splits, const float* sinks, int out_dim, const void* gate,
+                               long gate_stride, int dtype, void* stream) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || splits < 1) return -10;
   AttnParams p = {};
@@ -923,6 +942,8 @@ extern "C" int fi_paged_decode(const void* q, long q_stride, const void* k_cache
   p.ws_ml = ws_ml; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = k_scale;
   p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = splits;
+  if (out_dim < 0 || out_dim > hd) return -10;
+  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -946,7 +967,8 @@ extern "C" int fi_paged_decode_merged(const void* q, long q_stride, const void* 
                                const int* seq_lens, float* ws_o, float* ws_ml, unsigned int* tickets, int B, int nh,
                                int nkv, int hd, int max_blocks, int block_size, int window,
                                float sm_scale, float softcap, int kv_fp8, float k_scale,
-                               float v_scale, int splits, int dtype, void* stream) {
+                               float v_scale, int splits, const float* sinks, int out_dim, const void* gate,
+                               long gate_stride, int dtype, void* stream) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || splits < 1) return -10;
   AttnParams p = {};
@@ -955,6 +977,8 @@ extern "C" int fi_paged_decode_merged(const void* q, long q_stride, const void* 
   p.ws_ml = ws_ml; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = k_scale;
   p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = splits; p.merge_tickets = tickets;
+  if (out_dim < 0 || out_dim > hd) return -10;
+  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -1039,7 +1063,8 @@ extern "C" int fi_paged_decode_cluster(const void* q, long q_stride, const void*
                                const int* seq_lens, int B, int nh,
                                int nkv, int hd, int max_blocks, int block_size, int window,
                                float sm_scale, float softcap, int kv_fp8, float k_scale,
-                               float v_scale, int splits, int dtype, void* stream) {
+                               float v_scale, int splits, const float* sinks, int out_dim, const void* gate,
+                               long gate_stride, int dtype, void* stream) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || splits < 1 || splits > 8 || block_size % 16 != 0) return -10;
   AttnParams p = {};
@@ -1048,6 +1073,8 @@ extern "C" int fi_paged_decode_cluster(const void* q, long q_stride, const void*
   p.ws_ml = nullptr; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = k_scale;
   p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = splits; p.cluster_off = 1;
+  if (out_dim < 0 || out_dim > hd) return -10;
+  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -1068,7 +1095,8 @@ extern "C" int fi_paged_prefill(const void* q, long q_stride, const void* k_cach
                                 const int* seq_lens, const int* cu_q, int B, int max_q_len, int nh,
                                 int nkv, int hd, int max_blocks, int block_size, int window,
                                 float sm_scale, float softcap, int kv_fp8, float k_scale,
-                                float v_scale, const float* sinks, int out_dim, int dtype, void* stream) {
+                                float v_scale, const float* sinks, int out_dim, const void* gate, long gate_stride,
+                                int dtype, void* stream) {
   if (B <= 0 || max_q_len <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0) return -10;
   AttnParams p = {};
@@ -1077,7 +1105,7 @@ extern "C" int fi_paged_prefill(const void* q, long q_stride, const void* k_cach
   p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window; p.sm_scale = sm_scale;
   p.softcap = softcap; p.k_scale = k_scale; p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = 1;
   if (out_dim < 0 || out_dim > hd || out_dim % 2 != 0) return -10;
-  p.sinks = sinks; p.out_dim = out_dim;
+  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == 0) {
     if (hd == 64) return launch_prefill<__nv_bfloat16, 64, 64>(p, B, max_q_len, s);
@@ -1128,7 +1156,7 @@ extern "C" int fi_paged_decode_noalloc(const void* q, long q_stride, const void*
   if (splits == 1)   // one split writes straight to `out`: no partials, so no scratch and no size limit
     return fi_paged_decode(q, q_stride, k_cache, v_cache, out, block_tables, seq_lens, nullptr, nullptr, B,
                            nh, nkv, hd, max_blocks, block_size, window, sm_scale, softcap, kv_fp8,
-                           k_scale, v_scale, 1, dtype, stream);
+                           k_scale, v_scale, 1, nullptr, 0, nullptr, 0, dtype, stream);
   const size_t n_o = static_cast<size_t>(B) * nh * splits * hd;
   const size_t n_ml = static_cast<size_t>(B) * nh * splits * 2;
   if (n_o + n_ml > kNoAllocScratchFloats) {
@@ -1155,5 +1183,5 @@ extern "C" int fi_paged_decode_noalloc(const void* q, long q_stride, const void*
   float* ws_ml = ws_o + n_o;
   return fi_paged_decode(q, q_stride, k_cache, v_cache, out, block_tables, seq_lens, ws_o, ws_ml, B,
                          nh, nkv, hd, max_blocks, block_size, window, sm_scale, softcap, kv_fp8,
-                         k_scale, v_scale, splits, dtype, stream);
+                         k_scale, v_scale, splits, nullptr, 0, nullptr, 0, dtype, stream);
 }

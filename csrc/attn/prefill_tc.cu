@@ -36,6 +36,8 @@ struct TcParams {
   void* out;                 // [T, nh * out_dim]
   const float* sinks;        // [nh] or null: one extra exp(sink) per head in the softmax denominator
   int out_dim;               // output channels per head that are stored (<= HD)
+  const void* gate;          // row t at gate + t * gate_stride, channels as in out, or null: out *= sigmoid(gate)
+  long gate_stride;
   const int* block_tables;   // [B, max_blocks]
   const int* seq_lens;       // [B]
   const int* cu_q;           // [B + 1]
@@ -399,11 +401,30 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 #pragma unroll
         for (int c = 0; c < HH / 8; ++c) {
           if (half * HH + c * 8 >= p.out_dim) break;
+          float y[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) y[e] = o[c * 8 + e] * inv;
+          if (p.gate != nullptr) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.gate) +
+                                                              (q_begin + qt0 + row) * p.gate_stride + head * p.out_dim +
+                                                              half * HH + c * 8);
+            const uint32_t gw[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              float g0 = __uint_as_float(gw[e] << 16), g1 = __uint_as_float(gw[e] & 0xffff0000u);
+              if (p.is_fp16) {
+                const float2 h = __half22float2(*reinterpret_cast<const __half2*>(&gw[e]));
+                g0 = h.x; g1 = h.y;
+              }
+              y[2 * e] /= 1.f + __expf(-g0);
+              y[2 * e + 1] /= 1.f + __expf(-g1);
+            }
+          }
           uint4 v;
-          v.x = pack2(o[c * 8 + 0] * inv, o[c * 8 + 1] * inv, p.is_fp16);
-          v.y = pack2(o[c * 8 + 2] * inv, o[c * 8 + 3] * inv, p.is_fp16);
-          v.z = pack2(o[c * 8 + 4] * inv, o[c * 8 + 5] * inv, p.is_fp16);
-          v.w = pack2(o[c * 8 + 6] * inv, o[c * 8 + 7] * inv, p.is_fp16);
+          v.x = pack2(y[0], y[1], p.is_fp16);
+          v.y = pack2(y[2], y[3], p.is_fp16);
+          v.z = pack2(y[4], y[5], p.is_fp16);
+          v.w = pack2(y[6], y[7], p.is_fp16);
           *reinterpret_cast<uint4*>(dst + c * 8) = v;
         }
       }
@@ -450,12 +471,13 @@ extern "C" int fi_paged_prefill_tc_set_trace(void* trace) {
 // the general kernel), other negative values for malformed arguments.
 //   q: token t, head h at q + (t * q_stride + h * hd) elements, T_total rows; caches [num_blocks, nkv,
 //   block_size, hd]; out [T_total, nh * out_dim] (out_dim <= hd, a multiple of 8: the leading channels of each
-//   head); sinks: fp32 [nh] or null.
+//   head); sinks: fp32 [nh] or null; gate: rows of pitch gate_stride in the type of out, or null.
 extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_cache, const void* v_cache, void* out,
                                    const int* block_tables, const int* seq_lens, const int* cu_q, int B,
                                    int T_total, int max_q_len, int nh, int nkv, int hd, long num_blocks,
                                    int max_blocks, int block_size, int window, float sm_scale, float softcap,
-                                   const float* sinks, int out_dim, int dtype, int* status, void* stream) {
+                                   const float* sinks, int out_dim, const void* gate, long gate_stride, int dtype,
+                                   int* status, void* stream) {
   if (B <= 0 || max_q_len <= 0 || T_total <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || out_dim <= 0 || out_dim > hd) return -10;
   if (out_dim % 8 != 0) return -12;
@@ -464,6 +486,7 @@ extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_c
   if ((reinterpret_cast<uintptr_t>(q) & 15) != 0 || (q_stride * 2) % 16 != 0 ||
       (reinterpret_cast<uintptr_t>(out) & 15) != 0)
     return -12;
+  if (gate != nullptr && ((reinterpret_cast<uintptr_t>(gate) & 15) != 0 || gate_stride % 8 != 0)) return -12;
   CUtensorMap qm, km, vm;
   const uint64_t kv_rows = static_cast<uint64_t>(num_blocks) * nkv * block_size;
   if (fi::make_tmap_2d_16bit_sw128(&qm, q, T_total, static_cast<uint64_t>(nh) * hd, q_stride, kTile) != 0 ||
@@ -472,7 +495,7 @@ extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_c
     return -12;
   TcParams p = {};
   p.out = out; p.block_tables = block_tables; p.seq_lens = seq_lens; p.cu_q = cu_q; p.status = status;
-  p.trace = g_tc_trace; p.sinks = sinks; p.out_dim = out_dim;
+  p.trace = g_tc_trace; p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
   p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window;
   p.sm_scale = sm_scale; p.softcap = softcap; p.is_fp16 = dtype == 1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);

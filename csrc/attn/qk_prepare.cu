@@ -1,0 +1,159 @@
+// Queries, keys and values of one step from a merged projection [q (H * dim) | k (G * dim) | ..]:
+//
+//   q' = R(pos) rmsnorm(q) over all H * dim channels,   k' = R(pos) rmsnorm(k) over all G * dim channels,   v = k
+//
+// Keys and values go to their paged caches, queries to rows the attention kernels read; heads are padded with zeros
+// from dim to the kernels' head size.  The rotation turns channels i and i + dims / 2 of a head (i < dims / 2) by the
+// angle of frequency i; cos_sin rows are [cos (dims / 2) | sin (dims / 2)]; channels from dims on pass.  Norms and angles
+// are 32-bit.  One block per token: the sums of squares, then a second walk over the row (cached in L1) in whole
+// 16-byte groups where the sizes allow it.
+#include <cuda_bf16.h>
+#include <cuda_fp16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "../common/launch.cuh"
+
+namespace {
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f(__half v) { return __half2float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+template <> __device__ __forceinline__ __half from_f<__half>(float v) { return __float2half_rn(v); }
+
+struct QkParams {
+  const void* proj;         // [T, ld]
+  const float* wq;          // [H * dim]
+  const float* wk;          // [G * dim]
+  const int* positions;     // [T]
+  const float* cos_sin;     // [max_pos, dims]
+  const int* slot_mapping;  // [T], < 0: no cache row
+  void* q_out;              // [T, H, hd]
+  void* k_cache;            // [blocks, G, block_size, hd]
+  void* v_cache;
+  long ld;
+  int H, G, dim, hd, dims, block_size, max_pos, vec;
+  float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  constexpr int V = 16 / sizeof(T);
+  __shared__ float red[2][8];
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const T* row = reinterpret_cast<const T*>(p.proj) + t * p.ld;
+  const int nq = p.H * p.dim, nk = p.G * p.dim;
+  float sq = 0.f, sk = 0.f;
+  if (p.vec) {
+    for (int i = tid; i < (nq + nk) / V; i += 256) {
+      alignas(16) T x[V];
+      *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(row + i * V);
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < V; ++e) { const float f = to_f(x[e]); s = fmaf(f, f, s); }
+      if (i * V < nq) sq += s; else sk += s;
+    }
+  } else {
+    for (int i = tid; i < nq + nk; i += 256) {
+      const float f = to_f(row[i]);
+      if (i < nq) sq = fmaf(f, f, sq); else sk = fmaf(f, f, sk);
+    }
+  }
+  for (int m = 16; m > 0; m >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, m);
+    sk += __shfl_xor_sync(0xffffffffu, sk, m);
+  }
+  if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) { sq += red[0][w]; sk += red[1][w]; }
+  const float iq = 1.f / sqrtf(sq / static_cast<float>(nq) + p.eps), ik = 1.f / sqrtf(sk / static_cast<float>(nk) + p.eps);
+  const int pos = min(max(p.positions[t], 0), p.max_pos - 1);
+  const float* cs = p.cos_sin + static_cast<long>(pos) * p.dims;
+  const int half = p.dims / 2;
+  const int slot = p.slot_mapping[t];
+  const int heads = slot >= 0 ? p.H + p.G : p.H;
+  const long blk = slot >= 0 ? slot / p.block_size : 0, off = slot >= 0 ? slot % p.block_size : 0;
+  const int per = p.vec ? p.hd / V : p.hd;                 // groups (or channels) per padded head
+  for (int i = tid; i < heads * per; i += 256) {
+    const int h = i / per;
+    const bool is_k = h >= p.H;
+    const T* src = row + h * p.dim;                        // heads of k follow those of q
+    const float* w = is_k ? p.wk + (h - p.H) * p.dim : p.wq + h * p.dim;
+    const float inv = is_k ? ik : iq;
+    T* dst = is_k ? reinterpret_cast<T*>(p.k_cache) + ((blk * p.G + h - p.H) * p.block_size + off) * p.hd
+                  : reinterpret_cast<T*>(p.q_out) + (static_cast<long>(t) * p.H + h) * p.hd;
+    T* vdst = is_k ? reinterpret_cast<T*>(p.v_cache) + ((blk * p.G + h - p.H) * p.block_size + off) * p.hd : nullptr;
+    if (p.vec) {
+      const int c = (i % per) * V;
+      alignas(16) T x[V], y[V], o[V];
+      *reinterpret_cast<uint4*>(x) = make_uint4(0, 0, 0, 0);
+      *reinterpret_cast<uint4*>(o) = make_uint4(0, 0, 0, 0);
+      if (c < p.dim) {
+        *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(src + c);
+        const bool turns = c < p.dims, first = c < half;
+        const int other = first ? c + half : c - half;
+        if (turns) *reinterpret_cast<uint4*>(y) = *reinterpret_cast<const uint4*>(src + other);
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          float a = to_f(x[e]) * inv * w[c + e];
+          if (turns) {
+            const float bb = to_f(y[e]) * inv * w[other + e];
+            const int f = first ? c + e : other + e;
+            a = first ? a * cs[f] - bb * cs[half + f] : a * cs[f] + bb * cs[half + f];
+          }
+          o[e] = from_f<T>(a);
+        }
+      }
+      *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(o);
+      if (is_k) *reinterpret_cast<uint4*>(vdst + c) = *reinterpret_cast<const uint4*>(x);
+    } else {
+      const int c = i % per;
+      T x = from_f<T>(0.f);
+      float a = 0.f;
+      if (c < p.dim) {
+        x = src[c];
+        a = to_f(x) * inv * w[c];
+        if (c < p.dims) {
+          const bool first = c < half;
+          const int other = first ? c + half : c - half, f = first ? c : other;
+          const float bb = to_f(src[other]) * inv * w[other];
+          a = first ? a * cs[f] - bb * cs[half + f] : a * cs[f] + bb * cs[half + f];
+        }
+      }
+      dst[c] = from_f<T>(a);
+      if (is_k) vdst[c] = x;
+    }
+  }
+}
+
+}  // namespace
+
+// dtype: 0 bf16, 1 fp16, 2 fp32 (projection, queries, caches).  Slots >= 0 must lie inside the caches.
+extern "C" int fi_qk_prepare(const void* proj, long ld, const float* wq, const float* wk, float eps, const int* positions,
+                             const float* cos_sin, int max_pos, const int* slot_mapping, void* q_out, void* k_cache,
+                             void* v_cache, int T, int H, int G, int dim, int hd, int dims, int block_size, int dtype,
+                             void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || dim <= 0 || hd < dim || dims < 0 || dims > dim || dims % 2 != 0 || block_size <= 0 || max_pos <= 0)
+    return -10;
+  QkParams p = {};
+  p.proj = proj; p.wq = wq; p.wk = wk; p.positions = positions; p.cos_sin = cos_sin; p.slot_mapping = slot_mapping;
+  p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache; p.ld = ld; p.H = H; p.G = G; p.dim = dim; p.hd = hd;
+  p.dims = dims; p.block_size = block_size; p.max_pos = max_pos; p.eps = eps;
+  const int v = dtype == 2 ? 4 : 8;
+  const uintptr_t at = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out) |
+                       reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
+  p.vec = dim % v == 0 && hd % v == 0 && (dims / 2) % v == 0 && ld % v == 0 && (at & 15) == 0;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (dtype == 0) return static_cast<int>(fi::launch_kernel(qk_prepare_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, s, 0, p));
+  if (dtype == 1) return static_cast<int>(fi::launch_kernel(qk_prepare_kernel<__half>, dim3(T), dim3(256), 0, s, 0, p));
+  if (dtype == 2) return static_cast<int>(fi::launch_kernel(qk_prepare_kernel<float>, dim3(T), dim3(256), 0, s, 0, p));
+  return -11;
+}

@@ -61,7 +61,15 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
     ag_copier<BN>(p);
     return;
   }
-  const int t0 = token_tile_index<BN>(p, static_cast<int>(blockIdx.y) - p.copy_rows) * BN;
+  // grouped mode: the tile table comes from the kernels in front, so nothing may be fetched before they are done
+  const bool grouped = p.tile_expert != nullptr;
+  if (grouped) {
+    pdl_wait();
+    if (static_cast<int>(blockIdx.y) >= *p.n_tiles) return;   // uniform for the whole cluster
+  }
+  const int t0 = grouped ? p.tile_row0[blockIdx.y] : token_tile_index<BN>(p, static_cast<int>(blockIdx.y) - p.copy_rows) * BN;
+  const int t_end = grouped ? t0 + p.tile_rows[blockIdx.y] : p.T;
+  const int w_row = n0 + (grouped ? p.tile_expert[blockIdx.y] * p.expert_rows : 0);
   const int S = p.splits;
   const int rank = (S > 1) ? static_cast<int>(blockIdx.z) : 0;
 
@@ -111,8 +119,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
       for (int it = 0; it < n_pre; ++it) {
         uint8_t* a = stage_base + it * STAGE_BYTES;
         mbar_expect_tx(&full_bar[it], STAGE_BYTES);
-        tma_load_2d(a, &tmap_w, &full_bar[it], (kb_begin + it) * BK, n0);
-        if (DUAL) tma_load_2d(a + A_BYTES, &tmap_w, &full_bar[it], (kb_begin + it) * BK, p.dual_rows + n0);
+        tma_load_2d(a, &tmap_w, &full_bar[it], (kb_begin + it) * BK, w_row);
+        if (DUAL) tma_load_2d(a + A_BYTES, &tmap_w, &full_bar[it], (kb_begin + it) * BK, p.dual_rows + w_row);
       }
       pdl_wait();
       if (!ag_handshake(p, x_map, epoch_now) ||
@@ -135,8 +143,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
         }
         uint8_t* a = stage_base + s * STAGE_BYTES;
         mbar_expect_tx(&full_bar[s], STAGE_BYTES);
-        tma_load_2d(a, &tmap_w, &full_bar[s], kb * BK, n0);
-        if (DUAL) tma_load_2d(a + A_BYTES, &tmap_w, &full_bar[s], kb * BK, p.dual_rows + n0);
+        tma_load_2d(a, &tmap_w, &full_bar[s], kb * BK, w_row);
+        if (DUAL) tma_load_2d(a + A_BYTES, &tmap_w, &full_bar[s], kb * BK, p.dual_rows + w_row);
         tma_load_2d(a + A_BYTES * (DUAL ? 2 : 1), tmap_x_ptr, &full_bar[s], kb * BK, x_row);
       }
     }
@@ -234,7 +242,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w,
   // ---------------------------------------------------------------- epilogue (epilogue.cuh)
   if (warp >= 2) epilogue_tmem_to_smem<BN, DUAL>(p, accum_bar, tmem_base, stage_f32, aborted, warp, lane, row_ss, n0);
   __syncthreads();
-  epilogue_reduce_store<BN, DUAL>(p, stage_f32, aborted, n0, t0, epoch_now, p.T, row_ss);
+  epilogue_reduce_store<BN, DUAL>(p, stage_f32, aborted, n0, t0, epoch_now, t_end, row_ss);
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
@@ -307,7 +315,7 @@ int launch(const CUtensorMap& tw, const TokenMaps& tx, GemmParams p, cudaStream_
   if (p.x_full != nullptr) {   // staged all-gather: about 64 copier CTAs in the first rows of the grid
     p.copy_rows = (64 + nx * p.splits - 1) / (nx * p.splits);   // (x 192 threads x 8 loads of 16 bytes in flight)
   }
-  return static_cast<int>(launch_kernel(kern, dim3(nx, (p.T + BN - 1) / BN + p.copy_rows, p.splits),
+  return static_cast<int>(launch_kernel(kern, dim3(nx, p.grid_tiles > 0 ? p.grid_tiles : (p.T + BN - 1) / BN + p.copy_rows, p.splits),
                                         dim3(kThreads), smem, stream, p.splits, tw, tx, p));
 }
 
@@ -345,13 +353,14 @@ static int fi_dense_gemm_impl(const void* X, const void* W, void* C, const void*
                              int act, int dual_rows, int out_fp32, int dtype, int splits, int bn,
                              int* status, void* stream,
                              const FiComm* comm, float rms_eps = 0.f, int w_dynamic = 0,
-                             const FiRope* rope = nullptr) {
+                             const FiRope* rope = nullptr, const FiGrouped* grp = nullptr) {
   if (T <= 0 || N <= 0 || K <= 0) return 0;
   if (rms_eps > 0.f && (K % BK) != 0) return -21;   // the sum of squares reads whole 64-wide K blocks
   if ((K % 8) != 0 || (ldc % 8) != 0 || (reinterpret_cast<uintptr_t>(C) & 15) != 0) return -10;
   if (dual_rows > 0 && N != dual_rows) return -11;
   if (bn == 0) bn = fi_dense_gemm_pick_bn(T);
-  const int w_rows = dual_rows > 0 ? 2 * dual_rows : N;
+  const uint64_t w_rows = grp != nullptr ? static_cast<uint64_t>(grp->num_experts) * grp->expert_rows
+                                         : static_cast<uint64_t>(dual_rows > 0 ? 2 * dual_rows : N);
   CUtensorMap tw;
   TokenMaps tx;
   int r = make_tmap_2d_16bit_sw128(&tw, W, w_rows, K, ldw, BM);
@@ -387,6 +396,10 @@ static int fi_dense_gemm_impl(const void* X, const void* W, void* C, const void*
   p.dual_rows = dual_rows; p.act = act; p.out_fp32 = out_fp32; p.is_fp16 = dtype == 1;
   p.splits = splits; p.status = status;
   p.tile_expert = nullptr; p.tile_row0 = nullptr; p.tile_rows = nullptr; p.n_tiles = nullptr; p.expert_rows = 0; p.grid_tiles = 0;
+  if (grp != nullptr) {
+    p.tile_expert = grp->tile_expert; p.tile_row0 = grp->tile_row0; p.tile_rows = grp->tile_rows;
+    p.n_tiles = grp->n_tiles; p.expert_rows = grp->expert_rows; p.grid_tiles = grp->max_tiles;
+  }
   p.comm_mode = 0; p.world = 1; p.rank = 0; p.rows_per_rank = 0; p.xfer_16bit = 0; p.comm_phases = 0; p.trace = g_plain_trace;
   p.rms_eps = rms_eps; p.w_dynamic = w_dynamic;
   p.x_full = nullptr; p.ag_flags = nullptr; p.copy_rows = 0;
@@ -476,6 +489,17 @@ extern "C" int fi_dense_gemm_dynw(const void* X, const void* W, void* C, const v
                              int act, int dual_rows, int out_fp32, int dtype, int splits, int bn,
                              int* status, void* stream) {
   return fi_dense_gemm_impl(X, W, C, bias, residual, T, N, K, ldx, ldw, ldc, act, dual_rows, out_fp32, dtype, splits, bn, status, stream, nullptr, 0.f, 1);
+}
+
+// Mixture-of-experts form: rows of X [n_rows, K], sorted by expert, meet the weights of their expert.  g: tile table for
+// tiles of `bn` rows (16, 32, 64 or 128), W [experts * g->expert_rows, K]; gated mode as above with an expert's rows
+// stored [gate; up].
+extern "C" int fi_dense_gemm_grouped(const void* X, const void* W, void* C, int n_rows, int N, int K, int ldx, int ldc,
+                             int act, int dual_rows, int dtype, int bn, const FiGrouped* g, int* status, void* stream) {
+  if (g == nullptr || bn <= 0 || g->max_tiles > 65535) return -25;
+  if (g->max_tiles <= 0) return 0;
+  return fi_dense_gemm_impl(X, W, C, nullptr, nullptr, n_rows, N, K, ldx, K, ldc, act, dual_rows, 0, dtype, 1, bn, status,
+                            stream, nullptr, 0.f, 0, nullptr, g);
 }
 
 // Same GEMM with a fused collective and/or an all-gathered token operand (see comm_desc.h).

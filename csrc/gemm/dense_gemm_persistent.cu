@@ -16,6 +16,8 @@
 // Barriers: full/empty per pipeline stage (running across tiles), acc_full/acc_empty per accumulator.
 // Tile order: consecutive CTAs take different weight tiles of the same 128 tokens, so the token tile
 // is shared through L2 and the weights (a few MB per layer) stay L2-resident across token tiles.
+// Grouped mode (mixture of experts): token tiles come from a table built on the device (expert, first row, rows) over
+// activations sorted by expert, and a tile's weights are those of its expert.
 // Every wait is bounded; a timeout records a status code and the kernel winds down normally.
 // The reference runs these products through torch.nn.functional.linear (vllm/model_executor/layers/
 // lite_linear.py:46-62).
@@ -28,6 +30,7 @@
 #include "../common/launch.cuh"
 #include "../common/ptx.cuh"
 #include "../common/tensormap.h"
+#include "comm_desc.h"
 
 using namespace fi;
 
@@ -49,6 +52,12 @@ struct PParams {
   int rows_per_tile;   // output rows (of N) one tile covers: 128 (gated or single) or 256
   int n_tiles_n, n_tiles;
   int* status;
+  // grouped mode (tile_expert != null): n_tiles is the grid's upper bound, the true number of token tiles is *tiles
+  const int* tile_expert;
+  const int* tile_row0;
+  const int* tile_rows;
+  const int* tiles;
+  int expert_rows;     // weight rows per expert
 };
 
 __device__ __forceinline__ float act_f(float g, int act) {
@@ -107,6 +116,8 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
   const uint32_t tmem_base = *tmem_slot;
   pdl_wait();
   const int kb_total = (p.K + BK - 1) / BK;
+  const bool grouped = p.tile_expert != nullptr;
+  const int n_tiles = grouped ? *p.tiles * p.n_tiles_n : p.n_tiles;
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer
@@ -114,9 +125,10 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
       tma_prefetch_desc(&tmap_w);
       tma_prefetch_desc(&tmap_x);
       long it = 0;
-      for (int tile = blockIdx.x; tile < p.n_tiles && !*aborted; tile += gridDim.x) {
-        const int n0 = (tile % p.n_tiles_n) * p.rows_per_tile;
-        const int t0 = (tile / p.n_tiles_n) * BN;
+      for (int tile = blockIdx.x; tile < n_tiles && !*aborted; tile += gridDim.x) {
+        const int tt = tile / p.n_tiles_n;
+        const int n0 = (tile % p.n_tiles_n) * p.rows_per_tile + (grouped ? p.tile_expert[tt] * p.expert_rows : 0);
+        const int t0 = grouped ? p.tile_row0[tt] : tt * BN;
         for (int kb = 0; kb < kb_total; ++kb, ++it) {
           const int s = static_cast<int>(it % STAGES);
           const uint32_t ph = static_cast<uint32_t>(it / STAGES) & 1u;
@@ -139,7 +151,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
       const uint32_t idesc = umma_idesc_f16(p.is_fp16 ? 0 : 1, BM, BN);
       long it = 0;
       int local = 0;
-      for (int tile = blockIdx.x; tile < p.n_tiles && !*aborted; tile += gridDim.x, ++local) {
+      for (int tile = blockIdx.x; tile < n_tiles && !*aborted; tile += gridDim.x, ++local) {
         const int b = local & 1;
         const uint32_t use = static_cast<uint32_t>(local >> 1);
         if (!mbar_wait(&acc_empty[b], (use & 1u) ^ 1u)) {     // epilogue has drained this accumulator
@@ -185,7 +197,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
     const int q = warp & 3;                     // TMEM lane quarter this warp may read
     const int n_local = q * 32 + lane;          // weight row inside the tile
     int local = 0;
-    for (int tile = blockIdx.x; tile < p.n_tiles; tile += gridDim.x, ++local) {
+    for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++local) {
       const int b = local & 1;
       const uint32_t use = static_cast<uint32_t>(local >> 1);
       if (*aborted || !mbar_wait(&acc_full[b], use & 1u)) {
@@ -194,7 +206,8 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
       }
       tc_fence_after();
       const int n0 = (tile % p.n_tiles_n) * p.rows_per_tile;
-      const int t0 = (tile / p.n_tiles_n) * BN;
+      const int t0 = grouped ? p.tile_row0[tile / p.n_tiles_n] : (tile / p.n_tiles_n) * BN;
+      const int t_end = grouped ? t0 + p.tile_rows[tile / p.n_tiles_n] : p.T;
       const bool gated = p.dual_rows > 0;
       const uint32_t taddr = tmem_base + (static_cast<uint32_t>(q * 32) << 16) + static_cast<uint32_t>(b * ACC_COLS);
       // Each thread owns one weight row of the accumulator (a TMEM lane) but the output is
@@ -223,7 +236,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
           for (int rep = 0; rep < 2; ++rep) {
             const int t = t0 + c0 + vj + rep * 8;
             dst[rep] = make_uint4(0, 0, 0, 0);
-            if (p.residual != nullptr && nv_ok && c0 < c_end && t < p.T)
+            if (p.residual != nullptr && nv_ok && c0 < c_end && t < t_end)
               dst[rep] = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.residual) +
                                                          static_cast<size_t>(t) * p.ldc + nv);
           }
@@ -249,7 +262,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
           for (int rep = 0; rep < 2; ++rep) {
             const int j = vj + rep * 8;
             const int t = t0 + c0 + j;
-            if (nv_ok && t < p.T) {
+            if (nv_ok && t < t_end) {
               const float4 a0 = *reinterpret_cast<const float4*>(patch + j * 32 + vc * 8);
               const float4 a1 = *reinterpret_cast<const float4*>(patch + j * 32 + vc * 8 + 4);
               float v[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
@@ -338,7 +351,7 @@ extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, c
   if (r != 0) return r * 100 - 1;
   r = make_tmap_2d_16bit_sw128(&tx, X, T, K, ldx, BN);
   if (r != 0) return r * 100 - 2;
-  PParams p;
+  PParams p = {};
   p.C = C; p.bias = bias; p.residual = residual;
   p.T = T; p.N = N; p.K = K; p.ldc = ldc;
   p.dual_rows = dual_rows; p.act = act; p.is_fp16 = dtype == 1; p.out_fp32 = out_fp32;
@@ -350,6 +363,34 @@ extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, c
   p.n_tiles_n = (N + p.rows_per_tile - 1) / p.rows_per_tile;
   p.n_tiles = p.n_tiles_n * ((T + BN - 1) / BN);
   p.status = status;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (dual_rows > 0 || wide) return launch<4, true>(tw, tx, p, s);
+  return launch<6, false>(tw, tx, p, s);
+}
+
+// Grouped form over activations sorted by expert: rows of X [n_rows, K] (pitch ldx) belong to the experts of g's tile
+// table (built for tiles of 128 rows), W [experts * g->expert_rows, K]; C [n_rows, ldc] in X's type.  Gated mode
+// (dual_rows > 0): an expert's rows are [gate; up] and N == dual_rows.
+extern "C" int fi_dense_gemm_persistent_grouped(const void* X, const void* W, void* C, int n_rows, int N, int K, int ldx,
+                                                int ldc, int act, int dual_rows, int dtype, const FiGrouped* g, int* status,
+                                                void* stream) {
+  if (n_rows <= 0 || N <= 0 || K <= 0 || g->max_tiles <= 0) return 0;
+  if ((K % 8) != 0 || (ldx % 8) != 0 || (N % 8) != 0 || (ldc % 8) != 0 || (reinterpret_cast<uintptr_t>(C) & 15) != 0) return -10;
+  if (dual_rows > 0 && N != dual_rows) return -11;
+  CUtensorMap tw, tx;
+  int r = make_tmap_2d_16bit_sw128(&tw, W, static_cast<uint64_t>(g->num_experts) * g->expert_rows, K, K, BM);
+  if (r != 0) return r * 100 - 1;
+  r = make_tmap_2d_16bit_sw128(&tx, X, n_rows, K, ldx, BN);
+  if (r != 0) return r * 100 - 2;
+  PParams p = {};
+  p.C = C; p.T = n_rows; p.N = N; p.K = K; p.ldc = ldc; p.dual_rows = dual_rows; p.act = act; p.is_fp16 = dtype == 1;
+  const bool wide = dual_rows == 0 && N > BM;
+  p.second_off = dual_rows > 0 ? dual_rows : BM;
+  p.rows_per_tile = wide ? 2 * BM : BM;
+  p.n_tiles_n = (N + p.rows_per_tile - 1) / p.rows_per_tile;
+  p.n_tiles = p.n_tiles_n * g->max_tiles;
+  p.tile_expert = g->tile_expert; p.tile_row0 = g->tile_row0; p.tile_rows = g->tile_rows; p.tiles = g->n_tiles;
+  p.expert_rows = g->expert_rows; p.status = status;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dual_rows > 0 || wide) return launch<4, true>(tw, tx, p, s);
   return launch<6, false>(tw, tx, p, s);

@@ -1,0 +1,799 @@
+// Gated delta rule with one decay per head and key channel.  Per head, with state S [d, dv] (32-bit, one slot per
+// sequence), after a short causal convolution and SiLU on q, k and v:
+//
+//   q^ = q / |q| * d^-1/2,   k^ = k / |k|,   g = exp(-exp(A) softplus(z + bias)),   beta = sigmoid(b)
+//   S <- diag(g) S;   u = beta (v - S^T k^);   S <- S + k^ u^T;   o = S^T q^
+//
+// q and k may have fewer heads than v (head h reads q / k head h / (H / G)).  All arithmetic is 32-bit.
+//
+// Portions of prompts run in chunks of 16 tokens.  With E_i the product of the decays from the chunk's start through
+// token i (per channel), a chunk's writes are u_i = beta_i (v_i - S_0^T (E_i k_i) - sum_{j<i} a_ij u_j) with
+// a_ij = sum_c k_i k_j E_i / E_j, so they solve a unit lower-triangular system:  U = U0 - W S_0.
+//
+//   delta_chunk_kernel   everything that does not depend on the state, for all chunks in parallel: convolutions, unit
+//                        vectors, decays, a_ij and p_ij = sum_c q_i k_j E_i / E_j, the solved U0 and W.  Ratios
+//                        E_i / E_j are running products of decays from j to i: at most one, and nothing is divided.
+//   delta_scan_kernel    chunk after chunk: X = [W; E q] S (a reduction over d), U = U0 - X_W, o = X_q + P U,
+//                        S <- E_16 S + sum_j (E_16 / E_j) k_j u_j^T.  Columns of S never interact: a warp owns a few of
+//                        them with its share of S in registers (16 lanes split the rows), one block-wide meeting per
+//                        chunk hands over the operands, which arrive by bulk copies.
+//   delta_step_kernel    one token per sequence (decode): convolution, unit vectors, decays, state, per-head norm and
+//                        output gate in one pass that reads and writes the state once.
+//
+// The last taps - 1 convolution inputs of a sequence live in a ring of `taps` rows per slot: position p in row p % taps.
+// A step writes its own row and reads the others, so blocks that share q / k channels never race.
+// A sequence whose first position is 0 starts from a zero state and zero inputs whatever its slot holds.
+#include <cuda_bf16.h>
+#include <cuda_fp16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+#include "../common/launch.cuh"
+#include "../common/ptx.cuh"
+
+namespace {
+
+constexpr int kTok = 16;              // tokens per chunk
+constexpr float kUnitEps = 1e-6f;
+
+typedef unsigned long long f2;      // two packed floats
+__device__ __forceinline__ f2 pack2(float a, float b) {
+  f2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f2 v, float& a, float& b) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+}
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) {
+  f2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) {
+  f2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+__device__ __forceinline__ float to_f(float v) { return v; }
+__device__ __forceinline__ float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_f(__half v) { return __half2float(v); }
+__device__ __forceinline__ void st_any(void* p, long i, int type, float v) {
+  if (type == 2) reinterpret_cast<float*>(p)[i] = v;
+  else if (type == 0) reinterpret_cast<__nv_bfloat16*>(p)[i] = __float2bfloat16_rn(v);
+  else reinterpret_cast<__half*>(p)[i] = __float2half_rn(v);
+}
+__device__ __forceinline__ float ld_any(const void* p, long i, int type) {
+  if (type == 2) return reinterpret_cast<const float*>(p)[i];
+  if (type == 0) return __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(p)[i]);
+  return __half2float(reinterpret_cast<const __half*>(p)[i]);
+}
+__device__ __forceinline__ float sigmoidf(float z) { return 1.f / (1.f + __expf(-z)); }
+// log(1 + e^z) without overflow; the small branch keeps the relative precision of tiny results
+__device__ __forceinline__ float softplusf(float z) {
+  const float e = __expf(-fabsf(z));
+  return fmaxf(z, 0.f) + (e < 1e-3f ? e - 0.5f * e * e : log1pf(e));
+}
+// e^x for x <= 0.  Slow decays multiply over thousands of tokens, so close to one the error has to stay at rounding:
+// the power series there, the special-function unit further out (what it loses is forgotten within a few tokens).
+__device__ __forceinline__ float decay_exp(float x) {
+  float s = 1.f / 40320.f;
+  s = fmaf(s, x, 1.f / 5040.f);
+  s = fmaf(s, x, 1.f / 720.f);
+  s = fmaf(s, x, 1.f / 120.f);
+  s = fmaf(s, x, 1.f / 24.f);
+  s = fmaf(s, x, 1.f / 6.f);
+  s = fmaf(s, x, 0.5f);
+  s = fmaf(s, x, 1.f);
+  return x > -0.3f ? fmaf(s, x, 1.f) : __expf(x);
+}
+
+struct DeltaParams {
+  const void* qkv;        // [T, ld]: q (G * d) | k (G * d) | v (H * dv)
+  const float* z;         // [T, ldz]: decay projection (H * d)
+  const float* b;         // [T, ldb]: write strength projection (H)
+  const float* conv;      // [C, taps], last column = current token
+  const float* rate;      // [H]: exp(A)
+  const float* bias;      // [H * d]
+  float* pool;            // [slots, H, d, dv]
+  float* ring;            // [slots, taps, C]
+  const int* slots;       // [B]
+  const int* cu_q;        // [B + 1] (portions)
+  const int* seq_lens;    // [B] length after this step
+  const int* chunk_base;  // [B + 1] chunks before each sequence (portions)
+  float* work;            // [chunks, H, work_stride]
+  float* o;               // portions: [T, H, dv]
+  const float* norm_w;    // step: [dv]
+  const void* gate;       // step: [B, ldg] (H * dv) or null
+  void* out;              // step: [B, H * dv]
+  long ld, ldz, ldb, ldg, work_stride;
+  int B, H, G, d, dv, dp, dvp, C, taps, num_slots, n_chunks, gate_type, out_type;
+  float eps, q_scale;
+};
+
+// work block of a (chunk, head), in floats: W [16][dp] | E q [16][dp] | (E_16 / E) k [16][dp] | E_16 [dp] | P [16][16] |
+// U0 [dvp / 16][16 tokens][16 columns]
+__host__ __device__ inline long work_floats(int dp, int dvp) { return 49l * dp + 256 + 16l * dvp; }
+
+template <typename T>
+__global__ void __launch_bounds__(256, 2) delta_chunk_kernel(const DeltaParams p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  extern __shared__ __align__(128) float smem[];
+  const int chunk = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
+  int lo = 0, hi = p.B - 1;            // the sequence this chunk belongs to
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (p.chunk_base[mid] <= chunk) lo = mid; else hi = mid - 1;
+  }
+  const int b = lo;
+  const int t0 = (chunk - p.chunk_base[b]) * kTok;
+  const int t_begin = p.cu_q[b], n = p.cu_q[b + 1] - t_begin;
+  const int valid = min(kTok, n - t0);
+  const int slot = p.slots[b];
+  if (valid <= 0 || slot < 0 || slot >= p.num_slots) return;
+  const int pos0 = p.seq_lens[b] - n;  // position of the portion's first token
+  const int d = p.d, dv = p.dv, dp = p.dp, taps = p.taps, hist = taps - 1;
+  const int width = 2 * d + dv;
+  const int kvh = head / (p.H / p.G);
+  float* xs = smem;                                        // [16 + hist][width] convolution inputs
+  float* sq = xs + max((kTok + hist) * width, kTok * d);   // [16][d]
+  float* sk = sq + kTok * d;                               // [16][d]
+  float* sg = sk + kTok * d;                               // [16][d]
+  float* sv = sg + kTok * d;                               // [16][dv]
+  float* sA = sv + kTok * dv;                              // [16][16]
+  float* sP = sA + 256;                                    // [16][16]
+  float* sb = sP + 256;                                    // [16]
+  float* skd = xs;                                         // [16][d] E k, once the inputs are used up
+  float* work = p.work + (static_cast<long>(chunk) * p.H + head) * p.work_stride;
+
+  const T* qkv = reinterpret_cast<const T*>(p.qkv);
+  const int cq = kvh * d, ck = p.G * d + kvh * d, cv = 2 * p.G * d + head * dv;
+  const float* ring = p.ring + static_cast<long>(slot) * taps * p.C;
+  for (int c = tid; c < width; c += 256) {
+    const int ch = c < d ? cq + c : (c < 2 * d ? ck + c - d : cv + c - 2 * d);
+#pragma unroll 4
+    for (int r = 0; r < kTok + hist; ++r) {
+      const int s = t0 + r - hist;     // token of the portion; negative: before it
+      float x = 0.f;
+      if (s >= 0) {
+        if (r - hist < valid) x = to_f(qkv[(t_begin + s) * p.ld + ch]);
+      } else if (pos0 + s >= 0) {
+        x = ring[((pos0 + s) % taps) * p.C + ch];
+      }
+      xs[r * width + c] = x;
+    }
+  }
+  {
+    const float rate = p.rate[head];
+    for (int c = tid; c < d; c += 256) {
+      const float bias = p.bias[head * d + c];
+      const float* z = p.z + head * d + c;
+#pragma unroll 4
+      for (int t = 0; t < kTok; ++t)
+        sg[t * d + c] = t < valid ? decay_exp(-rate * softplusf(z[(t_begin + t0 + t) * p.ldz] + bias)) : 1.f;
+    }
+  }
+  if (tid < kTok) sb[tid] = tid < valid ? sigmoidf(p.b[(t_begin + t0 + tid) * p.ldb + head]) : 0.f;
+  __syncthreads();
+  for (int c = tid; c < width; c += 256) {
+    const int ch = c < d ? cq + c : (c < 2 * d ? ck + c - d : cv + c - 2 * d);
+    float y[kTok];
+#pragma unroll
+    for (int t = 0; t < kTok; ++t) y[t] = 0.f;
+    for (int j = 0; j < taps; ++j) {
+      const float w = p.conv[static_cast<long>(ch) * taps + j];
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) y[t] = fmaf(w, xs[(t + j) * width + c], y[t]);
+    }
+    float* dst = c < d ? sq + c : (c < 2 * d ? sk + c - d : sv + c - 2 * d);
+    const int pitch = c < 2 * d ? d : dv;
+#pragma unroll
+    for (int t = 0; t < kTok; ++t) dst[t * pitch] = t < valid ? y[t] * sigmoidf(y[t]) : 0.f;
+  }
+  __syncthreads();
+  const int warp = tid >> 5, lane = tid & 31;
+  for (int r = warp; r < 2 * kTok; r += 8) {               // unit vectors: rows of q, then of k
+    float* row = r < kTok ? sq + r * d : sk + (r - kTok) * d;
+    float ss = 0.f;
+    for (int c = lane; c < d; c += 32) ss += row[c] * row[c];
+    for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+    const float f = (r < kTok ? p.q_scale : 1.f) / sqrtf(ss + kUnitEps);
+    for (int c = lane; c < d; c += 32) row[c] *= f;
+  }
+  __syncthreads();
+  float* gq = work + 16l * dp;
+  float* gk = work + 32l * dp;
+  for (int c = tid; c < dp; c += 256) {
+    float e = 1.f;
+    if (c < d) {
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) {
+        e *= sg[t * d + c];
+        gq[t * dp + c] = sq[t * d + c] * e;
+        skd[t * d + c] = sk[t * d + c] * e;
+      }
+      work[48l * dp + c] = e;
+      float r = 1.f;
+#pragma unroll
+      for (int t = kTok - 1; t >= 0; --t) {
+        gk[t * dp + c] = sk[t * d + c] * r;
+        r *= sg[t * d + c];
+      }
+    } else {
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) { gq[t * dp + c] = 0.f; gk[t * dp + c] = 0.f; work[t * dp + c] = 0.f; }
+      work[48l * dp + c] = 0.f;
+    }
+  }
+  // a_ij (lanes 0-15 end with rows i) and p_ij (lanes 16-31) of two columns j per warp
+  for (int side = 0; side < 2; ++side) {
+    const int j = side == 0 ? warp : kTok - 1 - warp;
+    float v[32];
+#pragma unroll
+    for (int i = 0; i < 32; ++i) v[i] = 0.f;
+    for (int c = lane; c < d; c += 32) {
+      float w = sk[j * d + c];
+#pragma unroll
+      for (int i = 0; i < kTok; ++i) {
+        if (i > j) {
+          w *= sg[i * d + c];
+          v[i] = fmaf(sk[i * d + c], w, v[i]);
+        }
+        if (i >= j) v[16 + i] = fmaf(sq[i * d + c], w, v[16 + i]);
+      }
+    }
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) {
+      const bool up = (lane & m) != 0;
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        if (i < m) {
+          const float send = up ? v[i] : v[i + m];
+          const float keep = up ? v[i + m] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+        }
+      }
+    }
+    if (lane < 16) sA[lane * 16 + j] = v[0];
+    else sP[(lane - 16) * 16 + j] = v[0];
+  }
+  __syncthreads();
+  work[49l * dp + tid] = sP[tid];
+  for (int c = tid; c < d + dv; c += 256) {                // solve for one column of W or U0
+    const float* src = c < d ? skd + c : sv + c - d;
+    const int pitch = c < d ? d : dv;
+    float x[kTok];
+#pragma unroll
+    for (int i = 0; i < kTok; ++i) {
+      asm volatile("" ::: "memory");                       // keeps the 120 coefficients from being loaded all at once
+      float r = src[i * pitch];
+#pragma unroll
+      for (int j = 0; j < i; ++j) r = fmaf(-sA[i * 16 + j], x[j], r);
+      x[i] = sb[i] * r;
+    }
+    if (c < d) {
+#pragma unroll
+      for (int i = 0; i < kTok; ++i) work[i * dp + c] = x[i];
+    } else {
+      const int cc = c - d;
+      float* u0 = work + 49l * dp + 256 + (cc >> 4) * 256 + (cc & 15);
+#pragma unroll
+      for (int i = 0; i < kTok; ++i) u0[i * 16] = x[i];
+    }
+  }
+  for (int i = tid; i < (p.dvp - dv) * 16; i += 256) {
+    const int cc = dv + i / 16;
+    work[49l * dp + 256 + (cc >> 4) * 256 + (i & 15) * 16 + (cc & 15)] = 0.f;
+  }
+}
+
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(fi::smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(fi::smem_u32(bar))
+               : "memory");
+}
+
+constexpr int kWarps = 8;
+
+// R rows per lane (dp == 16 R), C columns per lane (a warp: 2 C columns, a block: 16 C).
+template <int R, int C, int STAGES>
+__global__ void __launch_bounds__(kWarps * 32) delta_scan_kernel(const DeltaParams p, int* status) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  constexpr int DP = 16 * R;
+  constexpr int COLS = kWarps * 2 * C;
+  constexpr int kOper = 49 * DP + 256;                     // floats of a stage before U0
+  constexpr int kStage = kOper + COLS * 16;
+  constexpr int TG = 16 / C;                               // tokens whose partial sums are reduced together
+  extern __shared__ __align__(128) float smem[];
+  float* sx_all = smem + STAGES * kStage;                  // [warps][2][16][2 C]
+  __shared__ uint64_t full[STAGES];
+  const int slices = p.dvp / COLS;
+  const int head = blockIdx.x / slices, slice = blockIdx.x % slices, b = blockIdx.y;
+  const int t_begin = p.cu_q[b], n = p.cu_q[b + 1] - t_begin;
+  const int slot = p.slots[b];
+  if (n <= 0 || slot < 0 || slot >= p.num_slots) return;
+  const int first = p.chunk_base[b], chunks = (n + kTok - 1) / kTok;
+  const int seq_len = p.seq_lens[b];
+  const bool fresh = seq_len == n;                         // the portion starts at position 0
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int rg = lane & 15, cg = lane >> 4;
+  const int wcol = warp * 2 * C;                           // first column of the warp inside the block's slice
+  const int col0 = slice * COLS + wcol + cg * C;           // first of this lane's columns
+  float* S0 = p.pool + (static_cast<long>(slot) * p.H + head) * p.d * p.dv;
+  float* sx = sx_all + warp * 2 * 16 * 2 * C;
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < STAGES; ++s) fi::mbar_init(&full[s], 1);
+    fi::mbar_fence_init();
+  }
+  __syncthreads();
+  auto request = [&](int i) {                              // one thread
+    const int s = i % STAGES;
+    const float* w = p.work + (static_cast<long>(first + i) * p.H + head) * p.work_stride;
+    fi::mbar_expect_tx(&full[s], kStage * 4);
+    bulk_load(smem + s * kStage, w, kOper * 4, &full[s]);
+    bulk_load(smem + s * kStage + kOper, w + kOper + slice * COLS * 16, COLS * 64, &full[s]);
+  };
+  int issued = 0;
+  if (threadIdx.x == 0)
+    for (; issued < min(STAGES, chunks); ++issued) request(issued);
+
+  // the sequence's convolution inputs that the next portion needs
+  {
+    const int keep = min(n, p.taps - 1);
+    const long per = static_cast<long>(p.C);
+    for (long i = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; i < keep * per; i += static_cast<long>(gridDim.x) * 256) {
+      const int back = static_cast<int>(i / per) + 1, ch = static_cast<int>(i % per);
+      p.ring[(static_cast<long>(slot) * p.taps + (seq_len - back) % p.taps) * p.C + ch] =
+          ld_any(p.qkv, (t_begin + n - back) * p.ld + ch, p.out_type);
+    }
+  }
+
+  // rows of this lane: 64 i4 + 4 rg + e, pairs (e = 0, 1) and (2, 3)
+  f2 S[R / 2][C];
+#pragma unroll
+  for (int i = 0; i < R / 2; ++i) {
+    const int row = (i >> 1) * 64 + rg * 4 + (i & 1) * 2;
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      float a = 0.f, bb = 0.f;
+      if (!fresh && col0 + c < p.dv) {
+        if (row < p.d) a = S0[static_cast<long>(row) * p.dv + col0 + c];
+        if (row + 1 < p.d) bb = S0[static_cast<long>(row + 1) * p.dv + col0 + c];
+      }
+      S[i][c] = pack2(a, bb);
+    }
+  }
+  bool ok = true;
+  int waited = chunks;
+  for (int i = 0; i < chunks; ++i) {
+    const int s = i % STAGES;
+    if (!fi::mbar_wait(&full[s], (i / STAGES) & 1)) {
+      fi::set_status(status, fi::kStatusTimeoutFull);
+      ok = false;
+    }
+    if (__syncthreads_or(ok ? 0 : 1)) { ok = false; waited = i; break; }
+    const float* st = smem + s * kStage;
+    const float* u0 = st + kOper;
+    // X = [W; E q] S
+#pragma unroll
+    for (int part = 0; part < 2; ++part) {
+#pragma unroll 1
+      for (int tq = 0; tq < 16; tq += TG) {
+        float v[16];                                       // [token][column]
+        const float* a = st + (part * 16 + tq) * DP + rg * 4;
+#pragma unroll
+        for (int u = 0; u < TG; ++u) {
+          f2 acc[C];
+#pragma unroll
+          for (int c = 0; c < C; ++c) acc[c] = pack2(0.f, 0.f);
+#pragma unroll
+          for (int i4 = 0; i4 < R / 4; ++i4) {
+            const float4 a4 = *reinterpret_cast<const float4*>(a + u * DP + i4 * 64);
+            const f2 a01 = pack2(a4.x, a4.y), a23 = pack2(a4.z, a4.w);
+#pragma unroll
+            for (int c = 0; c < C; ++c) acc[c] = fma2(a23, S[i4 * 2 + 1][c], fma2(a01, S[i4 * 2][c], acc[c]));
+          }
+#pragma unroll
+          for (int c = 0; c < C; ++c) {
+            float x, y;
+            unpack2(acc[c], x, y);
+            v[u * C + c] = x + y;
+          }
+        }
+#pragma unroll
+        for (int m = 8; m > 0; m >>= 1) {                  // row lane rg ends with the sum of value rg
+          const bool up = (rg & m) != 0;
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            if (e < m) {
+              const float send = up ? v[e] : v[e + m];
+              const float keep = up ? v[e + m] : v[e];
+              v[e] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+            }
+          }
+        }
+        sx[(part * 16 + tq + rg / C) * 2 * C + cg * C + rg % C] = v[0];
+      }
+    }
+    __syncwarp();
+    // U = U0 - X_W, in place
+#pragma unroll
+    for (int m = 0; m < C; ++m) {
+      const int e = m * 32 + lane, t = e / (2 * C), c = e % (2 * C), wc = wcol + c;
+      sx[e] = u0[(wc >> 4) * 256 + t * 16 + (wc & 15)] - sx[e];
+    }
+    __syncwarp();
+    // S <- E_16 S + sum_j (E_16 / E_j) k_j u_j^T
+#pragma unroll
+    for (int i4 = 0; i4 < R / 4; ++i4) {
+      const float4 e4 = *reinterpret_cast<const float4*>(st + 48 * DP + i4 * 64 + rg * 4);
+      const f2 e01 = pack2(e4.x, e4.y), e23 = pack2(e4.z, e4.w);
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        S[i4 * 2][c] = mul2(e01, S[i4 * 2][c]);
+        S[i4 * 2 + 1][c] = mul2(e23, S[i4 * 2 + 1][c]);
+      }
+    }
+#pragma unroll 4
+    for (int j = 0; j < 16; ++j) {
+      f2 uu[C];
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const float x = sx[j * 2 * C + cg * C + c];
+        uu[c] = pack2(x, x);
+      }
+#pragma unroll
+      for (int i4 = 0; i4 < R / 4; ++i4) {
+        const float4 k4 = *reinterpret_cast<const float4*>(st + (32 + j) * DP + i4 * 64 + rg * 4);
+        const f2 k01 = pack2(k4.x, k4.y), k23 = pack2(k4.z, k4.w);
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          S[i4 * 2][c] = fma2(k01, uu[c], S[i4 * 2][c]);
+          S[i4 * 2 + 1][c] = fma2(k23, uu[c], S[i4 * 2 + 1][c]);
+        }
+      }
+    }
+    // o = X_q + P U
+    const float* P = st + 49 * DP;
+#pragma unroll
+    for (int m = 0; m < C; ++m) {
+      const int e = m * 32 + lane, t = e / (2 * C), c = e % (2 * C);
+      float o = sx[16 * 2 * C + e];
+#pragma unroll
+      for (int j4 = 0; j4 < 4; ++j4) {
+        const float4 p4 = *reinterpret_cast<const float4*>(P + t * 16 + j4 * 4);
+        o = fmaf(p4.x, sx[(j4 * 4) * 2 * C + c], o);
+        o = fmaf(p4.y, sx[(j4 * 4 + 1) * 2 * C + c], o);
+        o = fmaf(p4.z, sx[(j4 * 4 + 2) * 2 * C + c], o);
+        o = fmaf(p4.w, sx[(j4 * 4 + 3) * 2 * C + c], o);
+      }
+      const int tok = i * kTok + t, col = slice * COLS + wcol + c;
+      if (tok < n && col < p.dv) p.o[(static_cast<long>(t_begin + tok) * p.H + head) * p.dv + col] = o;
+    }
+    __syncthreads();                                       // the stage is free, and so are the warps' own patches
+    if (threadIdx.x == 0 && issued < chunks) request(issued++);
+  }
+  if (!ok) {                                               // uniform: leave once the copies in flight have landed
+    if (threadIdx.x == 0)
+      for (int i = waited; i < issued; ++i) fi::mbar_wait(&full[i % STAGES], (i / STAGES) & 1);
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < R / 2; ++i) {
+    const int row = (i >> 1) * 64 + rg * 4 + (i & 1) * 2;
+#pragma unroll
+    for (int c = 0; c < C; ++c) {
+      float a, bb;
+      unpack2(S[i][c], a, bb);
+      if (col0 + c < p.dv) {
+        if (row < p.d) S0[static_cast<long>(row) * p.dv + col0 + c] = a;
+        if (row + 1 < p.d) S0[static_cast<long>(row + 1) * p.dv + col0 + c] = bb;
+      }
+    }
+  }
+}
+
+// One token per sequence.  Block: one (head, sequence); thread: VEC columns of every RY-th row.  KEEP > 0: rows per
+// thread whose values stay in registers between the two passes over the state (d <= KEEP * RY); 0: read twice.
+template <int VEC, int KEEP, typename T>
+__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaParams p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  extern __shared__ __align__(128) float smem[];
+  __shared__ float red[2][8];
+  const int head = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  const int len = p.seq_lens[b], slot = p.slots[b];
+  const int d = p.d, dv = p.dv, taps = p.taps;
+  const long orow = static_cast<long>(b) * p.H * dv + static_cast<long>(head) * dv;
+  if (len <= 0 || slot < 0 || slot >= p.num_slots) {       // padded row of a decode bucket
+    for (int j = tid; j < dv; j += 256) st_any(p.out, orow + j, p.out_type, 0.f);
+    return;
+  }
+  const int nx = (dv + VEC - 1) / VEC;                     // threads across the columns (<= 256)
+  const int ry_n = 256 / nx;
+  const int cx = tid % nx, ry = tid / nx;
+  const bool fresh = len == 1;
+  float* S = p.pool + (static_cast<long>(slot) * p.H + head) * d * dv;
+  auto fetch = [&](int r, float* s) {
+    const float* row = S + static_cast<long>(r) * dv + cx * VEC;
+    if constexpr (VEC == 4) {
+      const float4 x = *reinterpret_cast<const float4*>(row);
+      s[0] = x.x; s[1] = x.y; s[2] = x.z; s[3] = x.w;
+    } else {
+      s[0] = row[0];
+    }
+  };
+  float keep[KEEP > 0 ? KEEP : 1][VEC];
+  if constexpr (KEEP > 0) {                                // in flight while the operands are prepared
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int r = ry + i * ry_n;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) keep[i][e] = 0.f;
+      if (!fresh && ry < ry_n && r < d) fetch(r, keep[i]);
+    }
+  }
+  float* sq = smem;                 // [d]
+  float* sk = sq + d;               // [d]
+  float* sg = sk + d;               // [d]
+  float* sv = sg + d;               // [dv]
+  float* so = sv + dv;              // [ry][dv] partial sums
+  const int pos = len - 1, group = p.H / p.G, kvh = head / group;
+  const int cq = kvh * d, ck = p.G * d + kvh * d, cv = 2 * p.G * d + head * dv;
+  float* ring = p.ring + static_cast<long>(slot) * taps * p.C;
+  const T* x = reinterpret_cast<const T*>(p.qkv) + b * p.ld;
+  float ssq = 0.f, ssk = 0.f;
+  for (int c = tid; c < 2 * d + dv; c += 256) {
+    const int ch = c < d ? cq + c : (c < 2 * d ? ck + c - d : cv + c - 2 * d);
+    const float* w = p.conv + static_cast<long>(ch) * taps;
+    const float now = to_f(x[ch]);
+    float y = w[taps - 1] * now;
+    for (int j = 1; j < taps; ++j)
+      if (pos - j >= 0) y = fmaf(w[taps - 1 - j], ring[((pos - j) % taps) * p.C + ch], y);
+    if (c >= 2 * d || head % group == 0) ring[(pos % taps) * p.C + ch] = now;
+    y *= sigmoidf(y);
+    if (c < d) { sq[c] = y; ssq += y * y; }
+    else if (c < 2 * d) { sk[c - d] = y; ssk += y * y; }
+    else sv[c - 2 * d] = y;
+  }
+  const float rate = p.rate[head];
+  for (int c = tid; c < d; c += 256) sg[c] = decay_exp(-rate * softplusf(p.z[b * p.ldz + head * d + c] + p.bias[head * d + c]));
+  const float beta = sigmoidf(p.b[b * p.ldb + head]);
+  for (int m = 16; m > 0; m >>= 1) {
+    ssq += __shfl_xor_sync(0xffffffffu, ssq, m);
+    ssk += __shfl_xor_sync(0xffffffffu, ssk, m);
+  }
+  if ((tid & 31) == 0) { red[0][tid >> 5] = ssq; red[1][tid >> 5] = ssk; }
+  __syncthreads();
+  ssq = ssk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) { ssq += red[0][w]; ssk += red[1][w]; }
+  const float fq = p.q_scale / sqrtf(ssq + kUnitEps), fk = 1.f / sqrtf(ssk + kUnitEps);
+  // first pass: S^T k of the decayed state
+  float acc[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+  if (ry < ry_n) {
+    if constexpr (KEEP > 0) {
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        const int r = ry + i * ry_n;
+        if (r < d) {
+          const float g = sg[r], k = sk[r];
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) { keep[i][e] *= g; acc[e] = fmaf(k, keep[i][e], acc[e]); }
+        }
+      }
+    } else if (!fresh) {
+#pragma unroll 4
+      for (int r = ry; r < d; r += ry_n) {
+        float s[VEC];
+        fetch(r, s);
+        const float gk = sg[r] * sk[r];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) acc[e] = fmaf(gk, s[e], acc[e]);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e)
+      if (cx * VEC + e < dv) so[ry * dv + cx * VEC + e] = acc[e];
+  }
+  __syncthreads();
+  float u[VEC], o[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) { u[e] = 0.f; o[e] = 0.f; }
+  if (ry < ry_n) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      const int c = cx * VEC + e;
+      float a = 0.f;
+      for (int r = 0; r < ry_n; ++r) a += so[r * dv + c];
+      u[e] = beta * (sv[c] - fk * a);
+    }
+  }
+  __syncthreads();
+  // second pass: the write, the read-out and the new state
+  if (ry < ry_n) {
+    auto finish = [&](int r, float* s) {
+      const float k = fk * sk[r], q = sq[r];
+      float* row = S + static_cast<long>(r) * dv + cx * VEC;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        s[e] = fmaf(k, u[e], s[e]);
+        o[e] = fmaf(q, s[e], o[e]);
+      }
+      if constexpr (VEC == 4) *reinterpret_cast<float4*>(row) = make_float4(s[0], s[1], s[2], s[3]);
+      else row[0] = s[0];
+    };
+    if constexpr (KEEP > 0) {
+#pragma unroll
+      for (int i = 0; i < KEEP; ++i) {
+        const int r = ry + i * ry_n;
+        if (r < d) finish(r, keep[i]);
+      }
+    } else {
+#pragma unroll 4
+      for (int r = ry; r < d; r += ry_n) {
+        float s[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s[e] = 0.f;
+        if (!fresh) fetch(r, s);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s[e] *= sg[r];
+        finish(r, s);
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) so[ry * dv + cx * VEC + e] = o[e];
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int j = tid; j < dv; j += 256) {
+    float a = 0.f;
+    for (int r = 0; r < ry_n; ++r) a += so[r * dv + j];
+    a *= fq;
+    so[j] = a;                      // row 0 of its own column: nobody else reads it any more
+    ss += a * a;
+  }
+  for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+  if ((tid & 31) == 0) red[0][tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) tot += red[0][w];
+  const float inv = 1.f / sqrtf(tot / static_cast<float>(dv) + p.eps);
+  for (int j = tid; j < dv; j += 256) {
+    float y = so[j] * inv * p.norm_w[j];
+    if (p.gate != nullptr) y *= sigmoidf(ld_any(p.gate, b * p.ldg + head * dv + j, p.gate_type));
+    st_any(p.out, orow + j, p.out_type, y);
+  }
+}
+
+int check(const DeltaParams& p, int type) {
+  if (p.B <= 0 || p.H <= 0 || p.G <= 0 || p.H % p.G != 0 || p.d <= 0 || p.dv <= 0 || p.taps < 1 || p.taps > 16 ||
+      p.B > 65535 || p.H > 65535 || type < 0 || type > 2 || p.num_slots <= 0)
+    return -10;
+  return 0;
+}
+
+template <int R, int C>
+int launch_scan(const DeltaParams& p, int* status, cudaStream_t s) {
+  constexpr int COLS = kWarps * 2 * C, STAGES = R <= 8 ? 3 : 2;
+  constexpr int smem = (STAGES * (49 * 16 * R + 256 + COLS * 16) + kWarps * 2 * 16 * 2 * C) * 4;
+  auto kern = delta_scan_kernel<R, C, STAGES>;
+  cudaError_t e = fi::ensure_dynamic_smem(kern, smem);
+  if (e != cudaSuccess) return static_cast<int>(e);
+  return static_cast<int>(fi::launch_kernel(kern, dim3(p.H * (p.dvp / COLS), p.B), dim3(kWarps * 32), smem, s, 0, p, status));
+}
+
+template <int R>
+int pick_cols(const DeltaParams& p, int* status, cudaStream_t s) {
+  // wide tiles spend the fewest instructions per element, narrow ones fill the device when there are few sequences
+  const long ctas = static_cast<long>(p.B) * p.H * (p.dvp / 64);
+  if constexpr (R <= 8) {
+    if (ctas >= 192) return launch_scan<R, 4>(p, status, s);
+  }
+  if constexpr (R <= 16) {
+    if (ctas >= 120) return launch_scan<R, 2>(p, status, s);
+  }
+  return launch_scan<R, 1>(p, status, s);
+}
+
+}  // namespace
+
+// Floats of the work buffer per (chunk of 16 tokens, head), or -1 for sizes outside the kernels.
+extern "C" long fi_delta_work_floats(int d, int dv) {
+  if (d <= 0 || dv <= 0 || d > 512) return -1;
+  const int dp = d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : 512;
+  return work_floats(dp, (dv + 63) / 64 * 64);
+}
+
+// Portions of sequences.  qkv: type (0 bf16, 1 fp16, 2 fp32) rows of pitch ld, q (G * d) | k (G * d) | v (H * dv); z, b:
+// fp32 rows; conv: fp32 [C, taps]; rate, bias: fp32 [H], [H * d]; pool: fp32 [num_slots, H, d, dv]; ring: fp32
+// [num_slots, taps, C]; slots, seq_lens: int32 [B]; cu_q, chunk_base: int32 [B + 1] (chunk_base: running count of
+// ceil(portion / 16), n_chunks in total); work: n_chunks * H * fi_delta_work_floats(d, dv) floats, 16-byte aligned;
+// o: fp32 [T, H, dv].
+extern "C" int fi_delta_portions(const void* qkv, long ld, const float* z, long ldz, const float* b, long ldb,
+                                 const float* conv, const float* rate, const float* bias, float* pool, float* ring,
+                                 const int* slots, const int* cu_q, const int* seq_lens, const int* chunk_base,
+                                 int n_chunks, float* work, float* o, int B, int H, int G, int d, int dv, int taps,
+                                 int num_slots, int type, int* status, void* stream) {
+  if (B <= 0 || n_chunks <= 0) return 0;
+  DeltaParams p = {};
+  p.qkv = qkv; p.ld = ld; p.z = z; p.ldz = ldz; p.b = b; p.ldb = ldb; p.conv = conv; p.rate = rate; p.bias = bias;
+  p.pool = pool; p.ring = ring; p.slots = slots; p.cu_q = cu_q; p.seq_lens = seq_lens; p.chunk_base = chunk_base;
+  p.n_chunks = n_chunks; p.work = work; p.o = o; p.B = B; p.H = H; p.G = G; p.d = d; p.dv = dv; p.taps = taps;
+  p.num_slots = num_slots; p.C = 2 * G * d + H * dv; p.q_scale = 1.f / sqrtf(static_cast<float>(d)); p.out_type = type;
+  const int bad = check(p, type);
+  if (bad != 0) return bad;
+  if (d > 512 || (reinterpret_cast<uintptr_t>(work) & 15) != 0) return -11;
+  p.dp = d <= 64 ? 64 : d <= 128 ? 128 : d <= 256 ? 256 : 512;
+  p.dvp = (dv + 63) / 64 * 64;
+  p.work_stride = work_floats(p.dp, p.dvp);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  const long xs = static_cast<long>(kTok + taps - 1) * (2 * d + dv), kd = static_cast<long>(kTok) * d;
+  const long floats = (xs > kd ? xs : kd) + 3 * kd + static_cast<long>(kTok) * dv + 528;
+  if (floats * 4 > 227 * 1024) return -11;
+  const int smem = static_cast<int>(floats * 4);
+  cudaError_t e = cudaSuccess;
+#define FI_CHUNK(TT)                                                                                            \
+  {                                                                                                             \
+    e = fi::ensure_dynamic_smem(delta_chunk_kernel<TT>, smem);                                                  \
+    if (e == cudaSuccess) e = fi::launch_kernel(delta_chunk_kernel<TT>, dim3(n_chunks, H), dim3(256), smem, s, 0, p); \
+  }
+  if (type == 0) FI_CHUNK(__nv_bfloat16)
+  else if (type == 1) FI_CHUNK(__half)
+  else FI_CHUNK(float)
+#undef FI_CHUNK
+  if (e != cudaSuccess) return static_cast<int>(e);
+  if (p.dp == 64) return pick_cols<4>(p, status, s);
+  if (p.dp == 128) return pick_cols<8>(p, status, s);
+  if (p.dp == 256) return pick_cols<16>(p, status, s);
+  return pick_cols<32>(p, status, s);
+}
+
+// One token per sequence with head norm and output gate.  Operands as above; norm_w: fp32 [dv]; gate: rows of pitch ldg
+// of gate_type, or null; out: [B, H * dv] of out_type.  Rows with seq_lens <= 0 are padding: zero output, no state or
+// ring row touched.
+extern "C" int fi_delta_step(const void* qkv, long ld, const float* z, long ldz, const float* b, long ldb,
+                             const float* conv, const float* rate, const float* bias, float* pool, float* ring,
+                             const int* slots, const int* seq_lens, const float* norm_w, float eps, const void* gate,
+                             long ldg, int gate_type, void* out, int B, int H, int G, int d, int dv, int taps,
+                             int num_slots, int type, int out_type, void* stream) {
+  if (B <= 0) return 0;
+  DeltaParams p = {};
+  p.qkv = qkv; p.ld = ld; p.z = z; p.ldz = ldz; p.b = b; p.ldb = ldb; p.conv = conv; p.rate = rate; p.bias = bias;
+  p.pool = pool; p.ring = ring; p.slots = slots; p.seq_lens = seq_lens; p.norm_w = norm_w; p.eps = eps; p.gate = gate;
+  p.ldg = ldg; p.gate_type = gate_type; p.out = out; p.B = B; p.H = H; p.G = G; p.d = d; p.dv = dv; p.taps = taps;
+  p.num_slots = num_slots; p.C = 2 * G * d + H * dv; p.q_scale = 1.f / sqrtf(static_cast<float>(d)); p.out_type = out_type;
+  const int bad = check(p, type);
+  if (bad != 0) return bad;
+  if (gate_type < 0 || gate_type > 2 || out_type < 0 || out_type > 2) return -10;
+  const bool vec4 = dv % 4 == 0 && (reinterpret_cast<uintptr_t>(pool) & 15) == 0;
+  const int nx = vec4 ? dv / 4 : dv;
+  if (nx > 256) return -11;
+  const int ry = 256 / nx;
+  const long floats = 3l * d + dv + static_cast<long>(ry) * dv;
+  if (floats * 4 > 48 * 1024) return -11;
+  const int smem = static_cast<int>(floats * 4);
+  const int rows = (d + ry - 1) / ry;                      // per thread
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define FI_STEP(V, K, TT) return static_cast<int>(fi::launch_kernel(delta_step_kernel<V, K, TT>, dim3(H, B), dim3(256), smem, s, 0, p))
+#define FI_STEP_T(V, K)                     \
+  {                                         \
+    if (type == 0) FI_STEP(V, K, __nv_bfloat16); \
+    if (type == 1) FI_STEP(V, K, __half);   \
+    FI_STEP(V, K, float);                   \
+  }
+  if (!vec4) FI_STEP_T(1, 0)
+  if (rows <= 4) FI_STEP_T(4, 4)
+  if (rows <= 8) FI_STEP_T(4, 8)
+  if (rows <= 16) FI_STEP_T(4, 16)
+  FI_STEP_T(4, 0)
+#undef FI_STEP_T
+#undef FI_STEP
+}

@@ -13,7 +13,7 @@
 //                       (fma.rn.f32x2).
 //   hgrn2_step_kernel   one token per sequence (decode): reads and writes the state once, 16 bytes per thread and
 //                       access, and finishes with the per-head RMS norm.
-//   head_norm_kernel    RMS norm of each head's output row (after the scan).
+//   head_norm_kernel    RMS norm of each head's output row (after the scan), optionally times sigmoid of a gate.
 // A sequence whose first position is 0 starts from a zero state whatever its slot holds.
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
@@ -406,8 +406,10 @@ __global__ void __launch_bounds__(256, 3) hgrn2_step_kernel(const Hgrn2Params p)
   for (int j = threadIdx.x; j < p.dv; j += blockDim.x) st(p.out, orow + j, p.out_type, so[j] * inv * p.norm_w[j]);
 }
 
-// RMS norm of rows of length dv (fp32 in), one warp per row.
+// RMS norm of rows of length dv (fp32 in), one warp per row; with `gate` (row of token t at t * ldg, H heads of dv) the
+// result is multiplied by sigmoid(gate).
 __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                                        const void* __restrict__ gate, long ldg, int gate_type, int H,
                                                         void* __restrict__ out, long rows, int dv, float eps, int type) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -415,9 +417,21 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
   if (row >= rows) return;
   const int lane = threadIdx.x & 31;
   const float* src = x + row * dv;
+  const long grow = gate != nullptr ? (row / H) * ldg + (row % H) * dv : 0;
   float ss = 0.f;
-  if ((dv & 3) == 0 && dv <= 512) {
+  if ((dv & 3) == 0 && dv <= 512 && ((grow | ldg) & 3) == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0) {
     float4 v[4];
+    float gt[4][4];                         // raw gates, in flight together with the row
+    if (gate != nullptr) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        if (c < dv) {
+          if (gate_type == kFp32) expand4(load4(reinterpret_cast<const float*>(gate) + grow + c, 4, 1), kFp32, gt[i]);
+          else expand4(load4(reinterpret_cast<const uint16_t*>(gate) + grow + c, 4, 1), gate_type, gt[i]);
+        }
+      }
+    }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int c = (i * 32 + lane) * 4;
@@ -431,7 +445,10 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
       const int c = (i * 32 + lane) * 4;
       if (c < dv) {
         const float4 g = *reinterpret_cast<const float4*>(w + c);
-        const float y[4] = {v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w};
+        float y[4] = {v[i].x * inv * g.x, v[i].y * inv * g.y, v[i].z * inv * g.z, v[i].w * inv * g.w};
+        if (gate != nullptr)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) y[e] *= sigmoidf(gt[i][e]);
         if (type == kFp32) {
           *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + row * dv + c) = make_float4(y[0], y[1], y[2], y[3]);
         } else {
@@ -447,7 +464,11 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
   for (int c = lane; c < dv; c += 32) ss += src[c] * src[c];
   for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
   const float inv = 1.f / sqrtf(ss / static_cast<float>(dv) + eps);
-  for (int c = lane; c < dv; c += 32) st(out, row * dv + c, type, src[c] * inv * w[c]);
+  for (int c = lane; c < dv; c += 32) {
+    float y = src[c] * inv * w[c];
+    if (gate != nullptr) y *= sigmoidf(ld(gate, grow + c, gate_type));
+    st(out, row * dv + c, type, y);
+  }
 }
 
 template <int R, int C>
@@ -495,15 +516,17 @@ extern "C" int fi_hgrn2_scan(const void* q, long ldq, const void* f, long ldf, c
   return -11;
 }
 
-// RMS norm of every head's row: x fp32 [rows, dv] -> out [rows, dv] (type 0 bf16, 1 fp16, 2 fp32), w fp32 [dv].
-extern "C" int fi_head_norm(const float* x, const float* w, void* out, long rows, int dv, float eps, int type,
-                            void* stream) {
+// RMS norm of every head's row: x fp32 [rows, dv] -> out [rows, dv] (type 0 bf16, 1 fp16, 2 fp32), w fp32 [dv].  gate
+// (or null): rows [rows / H, >= H * dv] of pitch ldg and gate_type; out is multiplied by sigmoid(gate).
+extern "C" int fi_head_norm(const float* x, const float* w, const void* gate, long ldg, int gate_type, int H, void* out,
+                            long rows, int dv, float eps, int type, void* stream) {
   if (rows <= 0) return 0;
-  if (dv <= 0 || type < 0 || type > 2 || (reinterpret_cast<uintptr_t>(x) & 15) != 0 ||
+  if (dv <= 0 || H <= 0 || type < 0 || type > 2 || gate_type < 0 || gate_type > 2 || (reinterpret_cast<uintptr_t>(x) & 15) != 0 ||
       (reinterpret_cast<uintptr_t>(w) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 7) != 0)
     return -10;
   return static_cast<int>(fi::launch_kernel(head_norm_kernel, dim3(static_cast<unsigned>((rows + 7) / 8)), dim3(256), 0,
-                                            reinterpret_cast<cudaStream_t>(stream), 0, x, w, out, rows, dv, eps, type));
+                                            reinterpret_cast<cudaStream_t>(stream), 0, x, w, gate, ldg, gate_type, H, out, rows, dv, eps,
+                                            type));
 }
 
 // One token per sequence, norm included.  Same operands as fi_hgrn2_scan; norm_w: fp32 [dv]; out: [B, H * dv] of type

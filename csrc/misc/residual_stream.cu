@@ -1,8 +1,9 @@
-// Residual-stream kernels for decoders whose sublayers are normalised on both sides and whose layers read a
-// weighted average of everything before them.  The stream and every norm are 32-bit; the sublayers' inputs and
-// outputs may be 16-bit.
+// Residual-stream kernels: decoders whose sublayers are normalised on both sides and whose layers read a weighted
+// average of everything before them, and decoders whose sublayers read one norm side by side.  The stream and every
+// norm are 32-bit; the sublayers' inputs and outputs may be 16-bit.
 //
-//   start    v = table[token]                                          X_0 = v
+//   start    v = table[token] * scale                                  X_0 = v
+//   add      v = x + y + sum_k w_k e_(slot k)                          x   = v     (y: mixer, e: routed experts' rows)
 //   step     v = x + norm(y) * w_post                                  x   = v
 //   average  X_n = x + norm(y) * w_post;  v = sum_{j<=n} a_j X_j        x   = v
 //   each:    h = norm(v) * w_pre          (what the next sublayer reads)
@@ -20,7 +21,7 @@
 
 namespace {
 
-enum Mode : int { kStart = 0, kStep = 1, kAverage = 2 };
+enum Mode : int { kStart = 0, kStep = 1, kAverage = 2, kAdd = 3 };
 enum DType : int { kBf16 = 0, kFp16 = 1, kFp32 = 2 };
 
 struct StreamParams {
@@ -35,7 +36,12 @@ struct StreamParams {
   float* x_out;          // [*, W] or null
   void* h;               // [*, ldh] (type h_type)
   const long long* sel;  // optional: output row r comes from token sel[r]; x_out is not written then
-  long ldy, ldh, hist_stride;
+  const void* routed;    // kAdd: expert outputs (type y_type), rows of pitch ldr, or null
+  const int* slot_of;    // kAdd: [*, top] row of each (token, choice), < 0: none; null: row = token * top + choice
+  const float* route_w;  // kAdd: [*, top]
+  long ldy, ldh, hist_stride, ldr;
+  float scale;           // kStart
+  int top;
   int rows, W, group, groups, n, y_type, h_type, vocab;
   float eps;
 };
@@ -125,7 +131,42 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
       else
 #pragma unroll
         for (int e = 0; e < VEC; ++e) v[i * VEC + e] = 0.f;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[i * VEC + e] *= p.scale;
     }
+  } else if constexpr (MODE == kAdd) {
+    float yv[NV * VEC];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * TPR + tid) * VEC;
+      if (c < p.group) {
+        load_any<VEC, H16>(p.y, t * p.ldy + c0 + c, p.y_type, yv + i * VEC);
+        load_any<VEC, false>(p.x, t * p.W + c0 + c, kFp32, v + i * VEC);
+      } else {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { v[i * VEC + e] = 0.f; yv[i * VEC + e] = 0.f; }
+      }
+    }
+    if (p.routed != nullptr) {
+#pragma unroll 4
+      for (int k = 0; k < p.top; ++k) {
+        const long at = t * p.top + k;
+        const long slot = p.slot_of != nullptr ? p.slot_of[at] : at;
+        const float w = slot >= 0 ? p.route_w[at] : 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = (i * TPR + tid) * VEC;
+          if (c < p.group && slot >= 0) {
+            float e4[VEC];
+            load_any<VEC, H16>(p.routed, slot * p.ldr + c0 + c, p.y_type, e4);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) yv[i * VEC + e] = fmaf(w, e4[e], yv[i * VEC + e]);
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV * VEC; ++i) v[i] += yv[i];
   } else {
     float xv[NV * VEC];
     float ss = 0.f;
@@ -248,14 +289,15 @@ bool aligned(const void* p, unsigned a) { return (reinterpret_cast<uintptr_t>(p)
 
 }  // namespace
 
-// X_0 = table[ids] (32-bit) into `hist` slot 0, h = norm(X_0) * w_pre.  h_type (0 bf16, 1 fp16, 2 fp32) is also the
+// X_0 = table[ids] * scale (32-bit) into x0, h = norm(X_0) * w_pre.  h_type (0 bf16, 1 fp16, 2 fp32) is also the
 // table's type.  Token ids outside the table read row 0.
-extern "C" int fi_stream_start(const long long* ids, const void* table, int vocab, const float* w_pre, float* x0,
-                               void* h, long ldh, int T, int W, int groups, float eps, int h_type, void* stream) {
+extern "C" int fi_stream_start(const long long* ids, const void* table, int vocab, float scale, const float* w_pre,
+                               float* x0, void* h, long ldh, int T, int W, int groups, float eps, int h_type,
+                               void* stream) {
   if (T <= 0) return 0;
   if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || vocab <= 0) return -10;
   StreamParams p = {};
-  p.ids = ids; p.table = table; p.vocab = vocab; p.w_pre = w_pre; p.x_out = x0; p.h = h; p.ldh = ldh; p.rows = T; p.W = W;
+  p.ids = ids; p.table = table; p.vocab = vocab; p.scale = scale; p.w_pre = w_pre; p.x_out = x0; p.h = h; p.ldh = ldh; p.rows = T; p.W = W;
   p.group = W / groups; p.groups = groups; p.eps = eps; p.h_type = h_type; p.y_type = h_type;
   const bool vec4 = p.group % 4 == 0 && ldh % 4 == 0 && aligned(table, 16) && aligned(x0, 16) && aligned(h, 16) &&
                     aligned(w_pre, 16);
@@ -294,4 +336,23 @@ extern "C" int fi_stream_average(const void* y, long ldy, int y_type, const floa
                     aligned(x, 16) && aligned(x_out, 16) && aligned(h, 16) && aligned(hist, 16) && aligned(w_post, 16) &&
                     aligned(w_pre, 16);
   return dispatch<kAverage>(p, vec4, reinterpret_cast<cudaStream_t>(stream));
+}
+
+// v = x + y + sum_k route_w[t, k] routed[slot_of[t, k]]; x_out = v (may be x, or null), h = norm(v) * w_pre.  y, routed
+// and h share a type.  routed null: no experts.  sel (optional, int64 [rows]): only these tokens are wanted; row r of h
+// belongs to token sel[r] and x_out must be null.
+extern "C" int fi_stream_add(const void* y, long ldy, int y_type, const float* x, const void* routed, long ldr,
+                             const int* slot_of, const float* route_w, int top, const float* w_pre, float* x_out, void* h,
+                             long ldh, int h_type, const long long* sel, int rows, int W, int groups, float eps,
+                             void* stream) {
+  if (rows <= 0) return 0;
+  if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || y_type != h_type || top < 0) return -10;
+  if ((sel != nullptr && x_out != nullptr) || (routed != nullptr && (route_w == nullptr || top <= 0))) return -10;
+  StreamParams p = {};
+  p.y = y; p.ldy = ldy; p.y_type = y_type; p.x = x; p.routed = routed; p.ldr = ldr; p.slot_of = slot_of; p.route_w = route_w;
+  p.top = top; p.w_pre = w_pre; p.x_out = x_out; p.h = h; p.ldh = ldh; p.h_type = h_type; p.sel = sel; p.rows = rows;
+  p.W = W; p.group = W / groups; p.groups = groups; p.eps = eps;
+  const bool vec4 = p.group % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0 && ldr % 4 == 0 && aligned(y, 16) && aligned(x, 16) &&
+                    aligned(x_out, 16) && aligned(h, 16) && aligned(routed, 16) && aligned(w_pre, 16);
+  return dispatch<kAdd>(p, vec4, reinterpret_cast<cudaStream_t>(stream));
 }

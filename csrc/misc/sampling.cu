@@ -203,3 +203,44 @@ extern "C" int fi_sample(const float* logits, long ld, int rows, int V, const fl
                     V, temperature, top_k, top_p, min_p, uniform, out);
   return static_cast<int>(cudaGetLastError());
 }
+
+namespace {
+
+// x <- cap * tanh(x / cap) over rows of pitch ld.  tanh(y) = 1 - 2 / (1 + e^(2 y)) keeps the absolute error at 32-bit
+// rounding of the cap, which the special-function unit's own tanh does not.
+__global__ void __launch_bounds__(256) soft_cap_kernel(float* __restrict__ x, long ld, int n, float cap, int vec) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  float* row = x + blockIdx.y * ld;
+  const float k = 2.f / cap;
+  const int step = gridDim.x * 256, first = blockIdx.x * 256 + threadIdx.x;
+  if (vec) {
+    for (int i = first; i < n / 4; i += step) {
+      float4 v = reinterpret_cast<float4*>(row)[i];
+      v.x = cap - 2.f * cap / (1.f + __expf(k * v.x));
+      v.y = cap - 2.f * cap / (1.f + __expf(k * v.y));
+      v.z = cap - 2.f * cap / (1.f + __expf(k * v.z));
+      v.w = cap - 2.f * cap / (1.f + __expf(k * v.w));
+      reinterpret_cast<float4*>(row)[i] = v;
+    }
+    return;
+  }
+  for (int i = first; i < n; i += step) row[i] = cap - 2.f * cap / (1.f + __expf(k * row[i]));
+}
+
+}  // namespace
+
+// In place on fp32 rows [rows, n] of pitch ld.
+extern "C" int fi_soft_cap(float* x, long ld, int rows, int n, float cap, void* stream) {
+  if (rows <= 0 || n <= 0) return 0;
+  if (!(cap > 0.f)) return -10;
+  const int vec = n % 4 == 0 && ld % 4 == 0 && (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+  for (int r = 0; r < rows; r += 65535) {                  // rows on the second grid axis
+    const int here = rows - r < 65535 ? rows - r : 65535;
+    const int want = (n / (vec ? 4 : 1) + 255) / 256;
+    const cudaError_t e = fi::launch_kernel(soft_cap_kernel, dim3(want > 0 ? want : 1, here), dim3(256), 0,
+                                            reinterpret_cast<cudaStream_t>(stream), 0, x + r * ld, ld, n, cap, vec);
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  return 0;
+}

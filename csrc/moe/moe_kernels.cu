@@ -8,12 +8,15 @@
 //                      scores x routed scaling (DeepSeek-V3 style),
 //                    2 sqrt(softplus) scores with bias (DeepSeek-V4-Flash: deepseek_v4_flash/
 //                      gpu_layers.py:323-352).
+//                    Optionally the experts form equal groups of neighbours and only the best groups (by the sum
+//                    of their two largest selection scores) can be chosen.
 //   fi_moe_align   : counting sort of the (token, k) routes by expert restricted to the experts this
 //                    rank owns; emits sorted route ids, the inverse map, per-expert offsets and the
 //                    tile table (expert, first row, rows) consumed by fi_awq_gemm_grouped.
 //   fi_moe_gather  : x_sorted[slot] = x[route / k]
 //   fi_moe_combine : out[t] = sum_k w[t,k] * y_sorted[slot(t,k)]  (+ optional residual), fp32 sums in
 //                    a fixed order, so the result does not depend on the order of the sort.
+//   fi_moe_expert_rows : expert products on the general cores in 32-bit arithmetic (32-bit models, odd sizes)
 // The reference routes with torch.topk/softmax and runs experts in Python loops or M<=16 Triton
 // kernels (vllm/kernels/triton/gemma4_moe_int4.py); nothing there sorts tokens by expert on device.
 #include <cuda_bf16.h>
@@ -32,14 +35,14 @@ constexpr int kMaxExpertsPerLane = 16;   // experts <= 512
 
 __global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                  const float* __restrict__ expert_scale, int* __restrict__ topk_ids,
-                                 float* __restrict__ topk_w, int T, int E, int K, int mode,
-                                 int renorm, float routed_scale) {
+                                 float* __restrict__ topk_w, long ld, int T, int E, int K, int mode,
+                                 int renorm, float routed_scale, int groups, int keep_groups) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
-  const float* row = logits + static_cast<long>(t) * E;
+  const float* row = logits + t * ld;
   float score[kMaxExpertsPerLane];   // value used for the weight
   float sel[kMaxExpertsPerLane];     // value used for the selection
   const int per = (E + 31) / 32;
@@ -73,6 +76,52 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
       }
     }
   }
+  if (keep_groups < groups) {
+    // score of group g ends in lane g % 32; ties go to the lower group
+    const int size = E / groups;
+    float gscore[kMaxExpertsPerLane];
+    const int gper = (groups + 31) / 32;
+    for (int i = 0; i < gper; ++i) gscore[i] = -CUDART_INF_F;
+    for (int g = 0; g < groups; ++g) {
+      float m1 = -CUDART_INF_F, m2 = -CUDART_INF_F;          // the two largest of this lane's experts in the group
+      for (int i = 0; i < per; ++i) {
+        const int e = i * 32 + lane;
+        if (e >= g * size && e < (g + 1) * size) {
+          m2 = fmaxf(m2, fminf(m1, sel[i]));
+          m1 = fmaxf(m1, sel[i]);
+        }
+      }
+      for (int o = 16; o > 0; o >>= 1) {
+        const float o1 = __shfl_xor_sync(0xffffffffu, m1, o), o2 = __shfl_xor_sync(0xffffffffu, m2, o);
+        m2 = fmaxf(fmaxf(m2, o2), fminf(m1, o1));
+        m1 = fmaxf(m1, o1);
+      }
+      if ((g & 31) == lane) gscore[g >> 5] = size > 1 ? m1 + m2 : m1;
+    }
+    unsigned kept[kMaxExpertsPerLane];                       // bit g & 31 of word g >> 5: the group may be chosen
+    for (int i = 0; i < gper; ++i) kept[i] = 0u;
+    for (int k = 0; k < keep_groups; ++k) {
+      float best = -CUDART_INF_F;
+      int bi = 0x7fffffff;
+      for (int i = 0; i < gper; ++i) {
+        const int g = i * 32 + lane;
+        if (g < groups && !((kept[i] >> (g & 31)) & 1u) && (gscore[i] > best || (gscore[i] == best && g < bi))) {
+          best = gscore[i];
+          bi = g;
+        }
+      }
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
+      }
+      if (bi < groups) kept[bi >> 5] |= 1u << (bi & 31);
+    }
+    for (int i = 0; i < per; ++i) {
+      const int e = i * 32 + lane, g = e / size;
+      if (e < E && !((kept[g >> 5] >> (g & 31)) & 1u)) sel[i] = -CUDART_INF_F;
+    }
+  }
   float wsum = 0.f;
   float my_w = 0.f;
   int my_id = 0;
@@ -88,6 +137,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
     }
+    if (bi >= E) bi = 0;                                     // no comparable score left (a router output that is no number)
     // owner lane reads the weight score and retires the expert
     float w = 0.f;
     if ((bi & 31) == lane) {
@@ -330,6 +380,86 @@ __global__ void moe_combine_allreduce_kernel(const T* __restrict__ y_sorted, con
   }
 }
 
+// Expert products on the general cores: 32 rows x 64 outputs per block, 32-bit arithmetic.
+//   gather: out[row] = act(Wg x) * (Wu x) with x = X[sorted_route[row] / top] and weights [Wg (N rows); Wu (N rows)]
+//   else:   out[row] = W x with x = X[row]
+struct ExpertRows {
+  const void* x;            // rows of pitch ldx
+  const void* w;            // [experts, gather ? 2 N : N, K]
+  void* out;                // rows of pitch ldo
+  const int* sorted_route;
+  const int* tile_expert;
+  const int* tile_row0;
+  const int* tile_rows;     // at most 32
+  const int* n_tiles;
+  long ldx, ldo;
+  int N, K, top, gather;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) moe_expert_rows_kernel(const ExpertRows p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  constexpr int RB = 32, NB = 64, KB = 32;
+  const int tile = blockIdx.y;
+  if (tile >= *p.n_tiles) return;
+  const int e = p.tile_expert[tile], row0 = p.tile_row0[tile], rows = min(p.tile_rows[tile], RB);
+  const int n0 = blockIdx.x * NB;
+  __shared__ float sx[KB][RB + 1], swg[KB][NB + 1], swu[KB][NB + 1];
+  __shared__ long src[RB];
+  const int tid = threadIdx.x;
+  if (tid < RB) src[tid] = tid < rows ? static_cast<long>(p.gather ? p.sorted_route[row0 + tid] / p.top : row0 + tid) * p.ldx : -1;
+  __syncthreads();
+  const T* x = reinterpret_cast<const T*>(p.x);
+  const T* wg = reinterpret_cast<const T*>(p.w) + static_cast<long>(e) * (p.gather ? 2 : 1) * p.N * p.K;
+  const T* wu = wg + static_cast<long>(p.N) * p.K;
+  const int tr = tid >> 4, tn = tid & 15;           // rows tr, tr + 16; outputs tn + 16 i
+  float ag[2][4] = {}, au[2][4] = {};
+  for (int k0 = 0; k0 < p.K; k0 += KB) {
+    for (int i = tid; i < RB * KB; i += 256) {
+      const int r = i / KB, k = i % KB;
+      sx[k][r] = (src[r] >= 0 && k0 + k < p.K) ? static_cast<float>(x[src[r] + k0 + k]) : 0.f;
+    }
+    for (int i = tid; i < NB * KB; i += 256) {
+      const int n = i / KB, k = i % KB;
+      const bool in = n0 + n < p.N && k0 + k < p.K;
+      const long at = static_cast<long>(n0 + n) * p.K + k0 + k;
+      swg[k][n] = in ? static_cast<float>(wg[at]) : 0.f;
+      if (p.gather) swu[k][n] = in ? static_cast<float>(wu[at]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int k = 0; k < KB; ++k) {
+      const float x0 = sx[k][tr], x1 = sx[k][tr + 16];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float g = swg[k][tn + 16 * i];
+        ag[0][i] = fmaf(x0, g, ag[0][i]);
+        ag[1][i] = fmaf(x1, g, ag[1][i]);
+        if (p.gather) {
+          const float u = swu[k][tn + 16 * i];
+          au[0][i] = fmaf(x0, u, au[0][i]);
+          au[1][i] = fmaf(x1, u, au[1][i]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int r = tr + 16 * h;
+    if (r >= rows) continue;
+    T* out = reinterpret_cast<T*>(p.out) + (row0 + r) * p.ldo;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int n = n0 + tn + 16 * i;
+      if (n >= p.N) continue;
+      const float g = ag[h][i];
+      out[n] = static_cast<T>(p.gather ? g / (1.f + __expf(-g)) * au[h][i] : g);
+    }
+  }
+}
+
 }  // namespace
 
 #define FI_STREAM(s) reinterpret_cast<cudaStream_t>(s)
@@ -358,12 +488,14 @@ extern "C" int fi_moe_combine_allreduce(const void* y_sorted, const int* slot_of
 }
 
 extern "C" int fi_moe_route(const float* logits, const float* bias, const float* expert_scale,
-                            int* topk_ids, float* topk_w, int T, int E, int K, int mode, int renorm,
-                            float routed_scale, void* stream) {
+                            long ld, int* topk_ids, float* topk_w, int T, int E, int K, int mode, int renorm,
+                            float routed_scale, int groups, int keep_groups, void* stream) {
   if (T <= 0) return 0;
-  if (E > 32 * kMaxExpertsPerLane || K > 32 || K > E) return -10;
+  if (E > 32 * kMaxExpertsPerLane || K > 32 || K > E || groups < 1 || E % groups != 0 || keep_groups < 1 ||
+      keep_groups > groups || K > keep_groups * (E / groups) || ld < E)
+    return -10;
   fi::launch_kernel(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, FI_STREAM(stream), 0, logits, bias,
-                    expert_scale, topk_ids, topk_w, T, E, K, mode, renorm, routed_scale);
+                    expert_scale, topk_ids, topk_w, ld, T, E, K, mode, renorm, routed_scale, groups, keep_groups);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -406,4 +538,22 @@ extern "C" int fi_moe_combine(const void* y_sorted, const int* slot_of, const fl
     fi::launch_kernel(moe_combine_kernel<__half>, dim3(T, T < 128 ? (H / 8 + 127) / 128 : 1), dim3(128), 0, FI_STREAM(stream), 0,
                       (const __half*)y_sorted, slot_of, topk_w, (const __half*)residual, (__half*)out, K, H);
   return static_cast<int>(cudaGetLastError());
+}
+
+// Expert products without tensor cores (dtype 0 bf16, 1 fp16, 2 fp32; any sizes), over the tile table of fi_moe_align
+// (built with bn <= 32).  gather != 0: out[row] = silu(Wg x) * (Wu x) with x = X[sorted_route[row] / top], weights
+// [experts, 2 N, K]; gather == 0: out[row] = W X[row], weights [experts, N, K].
+extern "C" int fi_moe_expert_rows(const void* x, long ldx, const void* w, void* out, long ldo, const int* sorted_route,
+                                  const int* tile_expert, const int* tile_row0, const int* tile_rows, const int* n_tiles,
+                                  int max_tiles, int N, int K, int top, int gather, int dtype, void* stream) {
+  if (max_tiles <= 0) return 0;
+  if (N <= 0 || K <= 0 || top <= 0 || max_tiles > 65535 || (gather && sorted_route == nullptr)) return -10;
+  ExpertRows p = {};
+  p.x = x; p.w = w; p.out = out; p.ldx = ldx; p.ldo = ldo; p.sorted_route = sorted_route; p.tile_expert = tile_expert;
+  p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.n_tiles = n_tiles; p.N = N; p.K = K; p.top = top; p.gather = gather;
+  const dim3 grid((N + 63) / 64, max_tiles);
+  if (dtype == 0) return static_cast<int>(fi::launch_kernel(moe_expert_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, FI_STREAM(stream), 0, p));
+  if (dtype == 1) return static_cast<int>(fi::launch_kernel(moe_expert_rows_kernel<__half>, grid, dim3(256), 0, FI_STREAM(stream), 0, p));
+  if (dtype == 2) return static_cast<int>(fi::launch_kernel(moe_expert_rows_kernel<float>, grid, dim3(256), 0, FI_STREAM(stream), 0, p));
+  return -11;
 }

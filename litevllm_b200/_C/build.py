@@ -71,6 +71,10 @@ KERNEL_SETS = {
     "fimodra": ["attn/latent_rows.cu", "attn/mla_decode.cu", "attn/paged_attention.cu", "attn/prefill_tc.cu",
                 "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "linear_attn/hgrn2.cu",
                 "misc/norm_rope_misc.cu", "misc/residual_stream.cu", "misc/sampling.cu"],
+    "pofadra": ["attn/latent_rows.cu", "attn/paged_attention.cu", "attn/prefill_tc.cu", "attn/qk_prepare.cu",
+                "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "linear_attn/channel_delta.cu",
+                "linear_attn/hgrn2.cu", "misc/norm_rope_misc.cu", "misc/residual_stream.cu", "misc/sampling.cu",
+                "moe/moe_kernels.cu"],
 }
 
 

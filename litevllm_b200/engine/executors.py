@@ -142,7 +142,7 @@ class DecodeExecutor:
         batch.max_kv_len = full_ctx
         # the warm-up passes run the step for real: cache rows are rewritten with the same values, but recurrent
         # states would advance, so the batch's slots are put back afterwards
-        states = [s for s in getattr(self.kv_cache, "states", ()) if s is not None]
+        states = self.kv_cache.slot_tensors() if hasattr(self.kv_cache, "slot_tensors") else []
         slots = self.builder._decode_buffers(batch.num_seqs)["meta"][3].long()
         saved_states = [s.index_select(0, slots) for s in states]
         # warm up outside capture (lazy allocations, scratch growth, kernel attribute setup)

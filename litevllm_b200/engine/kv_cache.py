@@ -24,6 +24,7 @@ class KVLayerSpec:
     head_dim: int
     v_head_dim: int | None = None     # MLA-style caches may use another width for V (0 = no V)
     state_shape: tuple | None = None  # recurrent layers: shape of the fp32 state a request slot owns
+    ring_shape: tuple | None = None   # short convolutions: fp32 rows of recent inputs a request slot owns
 
     @property
     def v_dim(self) -> int:
@@ -31,7 +32,7 @@ class KVLayerSpec:
 
     @property
     def state_bytes(self) -> int:
-        return 4 * math.prod(self.state_shape) if self.state_shape else 0
+        return 4 * sum(math.prod(s) for s in (self.state_shape, self.ring_shape) if s)
 
 
 def kv_torch_dtype(kv_cache_dtype: str, model_dtype: torch.dtype) -> torch.dtype:
@@ -65,8 +66,9 @@ class FlatKVCache:
     def __init__(self, specs: list[KVLayerSpec], num_blocks: int, block_size: int,
                  dtype: torch.dtype, device: torch.device, fmt: int = 0, num_slots: int = 0):
         """``num_slots``: request slots of the engine; recurrent layers (``state_shape``) get one fp32 state per slot
-        in ``states[layer]``.  A slot's state is not cleared when it changes hands: a sequence that starts at
-        position 0 starts from a zero state."""
+        in ``states[layer]``, layers with short convolutions (``ring_shape``) their recent inputs in ``rings[layer]``.
+        A slot's state is not cleared when it changes hands: a sequence that starts at position 0 starts from a zero
+        state and zero inputs."""
         self.specs, self.num_blocks, self.block_size = specs, num_blocks, block_size
         self.dtype, self.device, self.fmt = dtype, device, fmt
         e = dtype_nbytes(dtype)
@@ -96,11 +98,16 @@ class FlatKVCache:
                     self.scale_bytes += t.fi_scales.numel() * 4
             self.layers.append((k, v))
         self.total_bytes += self.scale_bytes
-        self.states: list[torch.Tensor | None] = [
-            torch.zeros(num_slots, *s.state_shape, dtype=torch.float32, device=device) if s.state_shape else None
-            for s in specs]
-        self.state_bytes = sum(t.numel() * 4 for t in self.states if t is not None)
+        def per_slot(shape):
+            return torch.zeros(num_slots, *shape, dtype=torch.float32, device=device) if shape else None
+        self.states: list[torch.Tensor | None] = [per_slot(s.state_shape) for s in specs]
+        self.rings: list[torch.Tensor | None] = [per_slot(s.ring_shape) for s in specs]
+        self.state_bytes = sum(t.numel() * 4 for t in self.slot_tensors())
         self.total_bytes += self.state_bytes
+
+    def slot_tensors(self) -> list[torch.Tensor]:
+        """Everything indexed by request slot that a step advances."""
+        return [t for t in (*self.states, *self.rings) if t is not None]
 
     def __getitem__(self, i: int):
         return self.layers[i]

@@ -22,12 +22,18 @@ from pathlib import Path
 MAX_LIVE = 4
 
 
-def _ensure_kernels() -> None:
+def _ensure_kernels(model: str) -> None:
+    """Build what the model's family needs, unless the full library is there."""
     from .._C import build
     if build.full_library_is_current():
         return
+    from ..models.arch import arch_from_hf_config
     from ..ops import _lib
-    _lib.use_kernel_library(build.build_set("fimodra", verbose=False))
+    family = arch_from_hf_config(json.loads((Path(model) / "config.json").read_text())).family
+    if family in build.KERNEL_SETS:
+        _lib.use_kernel_library(build.build_set(family, verbose=False))
+    else:
+        build.build_all(verbose=False)
 
 
 def make_engine(model: str, dtype: str, max_tokens: int, device: str = "auto"):
@@ -65,7 +71,7 @@ def main(argv=None) -> int:
     if not torch.cuda.is_available():
         print("trace_run needs a CUDA device", file=sys.stderr)
         return 2
-    _ensure_kernels()
+    _ensure_kernels(args.model)
     from .. import ops
     engine = make_engine(args.model, args.dtype, args.max_tokens)
     out = Path(args.out)

@@ -264,3 +264,49 @@ def iter_fimodra_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, de
         yield p + "dwa", a
     yield vec("final.norm", W, 1.0, 0.1)
     yield lin("head", V, W)
+
+
+def iter_pofadra_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, device="cpu") -> Iterator[tuple[str, torch.Tensor]]:
+    """Linear weights ~ N(0, 1 / fan-in); norms near one; decays between a few and thousands of tokens; corrections that
+    move the choice of experts.  The rank of the low-rank projections is the head size of the key channels."""
+    W, V = arch.hidden_size, arch.vocab_size
+
+    def lin(name, out_f, in_f):
+        return name, normal(name, (out_f, in_f), seed, in_f ** -0.5, dtype, device)
+
+    def vec(name, n, base=0.0, std=1.0):
+        return name, base + normal(name, (n,) if isinstance(n, int) else n, seed, std, torch.float32, device)
+
+    yield "embed", normal("embed", (V, W), seed, 1.0 / arch.embed_scale, dtype, device)
+    for i, l in enumerate(arch.extra["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        yield vec(p + "norm1", W, 1.0, 0.1)
+        yield lin(p + "mix.q", (G if l["type"] == "channel_delta" else H) * d, W)
+        yield lin(p + "mix.k", G * d, W)
+        if l["type"] == "attention":
+            yield vec(p + "mix.q.norm", H * d, 1.0, 0.1)
+            yield vec(p + "mix.k.norm", G * d, 1.0, 0.1)
+            yield lin(p + "mix.g", H * d, W)
+        else:
+            yield lin(p + "mix.v", H * dv, W)
+            for n, rows in (("q", G * d), ("k", G * d), ("v", H * dv)):
+                yield vec(p + f"mix.{n}.conv", (rows, m["conv"]), 0.0, 0.5)
+            yield lin(p + "mix.b", H, W)
+            yield vec(p + "mix.A_log", H, -1.0, 1.0)
+            yield vec(p + "mix.norm", dv, 1.0, 0.1)
+            yield lin(p + "mix.a1", d, W)
+            yield lin(p + "mix.a2", H * d, d)
+            yield vec(p + "mix.dt_bias", H * d, -3.0, 1.5)
+            yield lin(p + "mix.g1", d, W)
+            yield lin(p + "mix.g2", H * dv, d)
+        yield lin(p + "mix.o", W, H * dv)
+        if l.get("mlp"):
+            ff, E = l["mlp"]["expert"]["ff"], l["mlp"]["router"]["experts"]
+            for e in range(E):
+                for n, o, k in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+                    yield lin(p + f"mlp.e{e}.{n}", o, k)
+            yield lin(p + "mlp.router", E, W)
+            yield vec(p + "mlp.correction", E, 0.0, 0.1)
+    yield vec("final.norm", W, 1.0, 0.1)
+    yield lin("head", V, W)

@@ -84,13 +84,18 @@ def load_mapped(param_map: dict, weights: Iterable[tuple[str, torch.Tensor]], st
 
 
 def load_exact(dest: dict, weights: Iterable[tuple[str, torch.Tensor]]) -> set[str]:
-    """Fill destinations by full checkpoint name: a parameter, or ``(LiteLinear, piece, "weight" | "bias")``.  Shapes
-    must match; a tensor without a destination and a destination without a tensor are both errors."""
+    """Fill destinations by full checkpoint name: a parameter (or a view of one), ``(LiteLinear, piece, "weight" |
+    "bias")``, or a function that takes the tensor (sizes only the checkpoint knows).  Shapes must match; a tensor
+    without a destination and a destination without a tensor are both errors."""
     seen: set[str] = set()
     for name, tensor in weights:
         d = dest.get(name)
         if d is None:
             raise KeyError(f"no destination for checkpoint tensor {name!r}")
+        if callable(d) and not isinstance(d, torch.Tensor):
+            d(tensor)
+            seen.add(name)
+            continue
         if isinstance(d, tuple):
             lin, piece, which = d
             want = (lin.out_splits[piece], lin.full_in) if which == "weight" else (lin.out_splits[piece],)

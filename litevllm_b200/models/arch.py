@@ -41,7 +41,7 @@ class MLASpec:
 
 @dataclass
 class ModelArch:
-    family: str                      # llama | qwen2 | qwen3_5 | gemma4 | deepseek_mla | qwen2_vl | fimodra
+    family: str                      # llama | qwen2 | qwen3_5 | gemma4 | deepseek_mla | qwen2_vl | fimodra | pofadra
     architecture: str
     hidden_size: int
     num_layers: int
@@ -162,8 +162,56 @@ def arch_from_fimodra_config(cfg: dict) -> ModelArch:
     return arch
 
 
+def arch_from_pofadra_config(cfg: dict) -> ModelArch:
+    """Pofadra configurations list their layers one by one (mixer type and sizes, routed experts or null)."""
+    layers = cfg["layers"]
+    if not layers:
+        raise ValueError("the configuration lists no layers")
+    for i, l in enumerate(layers):
+        m, where = l["mixer"], f"layers[{i}]"
+        if l["type"] == "attention":
+            _sizes(m, ("heads", "kv_heads", "dim", "vdim"), where)
+            if m["vdim"] != m["dim"]:
+                raise ValueError(f"{where}: keys are the values, so 'vdim' must equal 'dim'")
+            dims = m["rot"]["dims"]
+            if dims % 2 or dims > m["dim"] or dims < 0:
+                raise ValueError(f"{where}: cannot rotate {dims} of {m['dim']} dimensions")
+            _sizes(m["mask"], ("size",), where)
+        elif l["type"] == "channel_delta":
+            _sizes(m, ("heads", "kv_heads", "dim", "vdim", "conv"), where)
+        else:
+            raise ValueError(f"{where}: unknown mixer {l['type']!r}")
+        if m["heads"] % m["kv_heads"]:
+            raise ValueError(f"{where}: {m['heads']} heads do not share {m['kv_heads']} key heads evenly")
+        if l.get("mlp"):
+            if l["mlp"].get("kind") != "moe":
+                raise ValueError(f"{where}: unknown feed-forward {l['mlp'].get('kind')!r}")
+            r = l["mlp"]["router"]
+            _sizes(l["mlp"]["expert"], ("ff",), where)
+            _sizes(r, ("experts", "top"), where)
+            g = r.get("groups") or {"count": 1, "keep": 1}
+            _sizes(g, ("count", "keep"), where)
+            if r["experts"] % g["count"] or g["keep"] > g["count"] or r["top"] > g["keep"] * (r["experts"] // g["count"]):
+                raise ValueError(f"{where}: cannot choose {r['top']} of {r['experts']} experts from {g['keep']} of {g['count']} groups")
+    moes = [l["mlp"] for l in layers if l.get("mlp")]
+    attn = [l["mixer"] for l in layers if l["type"] == "attention"]
+    arch = ModelArch(
+        family="pofadra", architecture="Pofadra", hidden_size=int(cfg["width"]), num_layers=len(layers),
+        num_heads=max(l["mixer"]["heads"] for l in layers), num_kv_heads=max((m["kv_heads"] for m in attn), default=1),
+        head_dim=max(l["mixer"]["dim"] for l in layers), intermediate_size=max((m["expert"]["ff"] for m in moes), default=0),
+        vocab_size=int(cfg["vocab"]), rms_eps=float(cfg["norm"]["eps"]), act="silu",
+        embed_scale=float((cfg.get("embedding") or {}).get("scale", 1.0)), final_softcap=float(cfg.get("logit_softcap") or 0.0),
+        max_position=int(cfg.get("max_position_embeddings", 1 << 20)), eos_token_ids=_eos_list(cfg),
+        bos_token_id=cfg.get("bos_token_id"))
+    arch.layer_types = ["linear" if l["type"] == "channel_delta" else "sliding" for l in layers]
+    arch.extra.update(layers=layers)
+    return arch
+
+
 def arch_from_hf_config(cfg: dict) -> ModelArch:
     """Build a :class:`ModelArch` from a HF config dict (text sub-config is unwrapped)."""
+    if str(cfg.get("architecture", "")).lower() == "pofadra":
+        return arch_from_pofadra_config(cfg)
     if str(cfg.get("architecture", "")).lower() == "fimodra":
         return arch_from_fimodra_config(cfg)
     archs = cfg.get("architectures") or ["LlamaForCausalLM"]

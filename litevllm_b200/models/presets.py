@@ -145,6 +145,27 @@ PRESETS["tiny-fimodra-test"] = fimodra_config(256, 512, 192, "ahHaA", 3, 24, 8, 
 PRESETS["fimodra-1b"] = fimodra_config(2048, 32000, 5632, "aaha" * 5, 16, 96, 32, 128, 512, 1024, 16, 128, 128, groups=2)
 
 
+def pofadra_config(width: int, vocab: int, pattern: str, attn: tuple, delta: tuple, moe: tuple, rot_base: float = 10000.0,
+                   softcap: float = 30.0, embed_scale: float = 1.0) -> dict:
+    """Pofadra configuration from a layer pattern: "a" attention, "d" delta rule, upper case without a feed-forward.
+    ``attn``: heads, kv heads, dim, rotated dims, window; ``delta``: heads, kv heads, dim, vdim, taps; ``moe``: experts,
+    top, groups, kept groups, ff."""
+    a = dict(zip(("heads", "kv_heads", "dim"), attn[:3]), vdim=attn[2], rot={"base": rot_base, "dims": attn[3]},
+             mask={"size": attn[4]}, scale=attn[2] ** -0.5)
+    d = dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), delta))
+    ff = {"kind": "moe", "expert": {"ff": moe[4]}, "router": {"experts": moe[0], "top": moe[1], "scale": 1.0,
+                                                               "groups": {"count": moe[2], "keep": moe[3]}}}
+    layers = [{"type": "attention" if c in "aA" else "channel_delta", "mixer": copy.deepcopy(a if c in "aA" else d),
+               "mlp": copy.deepcopy(ff) if c.islower() else None} for c in pattern]
+    return {"architecture": "Pofadra", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "layers": layers,
+            "embedding": {"scale": embed_scale}, "logit_softcap": softcap}
+
+
+PRESETS["tiny-pofadra-test"] = pofadra_config(160, 384, "ddaDA", (6, 2, 40, 24, 24), (4, 2, 24, 40, 3), (12, 2, 3, 2, 72))
+# layers of the width and head geometry of a 1B-class decoder
+PRESETS["pofadra-1b"] = pofadra_config(2048, 32000, "ddad" * 3, (16, 4, 128, 64, 1024), (16, 16, 128, 128, 4), (32, 4, 4, 2, 768))
+
+
 def get_preset(name: str) -> dict:
     key = name.lower()
     if key not in PRESETS:

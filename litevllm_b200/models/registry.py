@@ -22,12 +22,13 @@ _MODELS = {
     "DeepseekV2ForCausalLM": ("deepseek_mla", "DeepseekMLAForCausalLM"),
     "DeepseekV4FlashForCausalLM": ("deepseek_v4_flash", "DeepseekV4FlashForCausalLM"),
     "Fimodra": ("fimodra", "FimodraForCausalLM"),
+    "Pofadra": ("pofadra", "PofadraForCausalLM"),
 }
 _FAMILY_DEFAULT = {
     "llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen3_5": "Qwen3_5ForCausalLM",
     "qwen2_vl": "Qwen2VLForConditionalGeneration", "gemma4": "Gemma4ForCausalLM",
     "deepseek_mla": "DeepseekV3ForCausalLM", "deepseek_v4_flash": "DeepseekV4FlashForCausalLM",
-    "fimodra": "Fimodra",
+    "fimodra": "Fimodra", "pofadra": "Pofadra",
 }
 
 

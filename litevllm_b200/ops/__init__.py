@@ -433,12 +433,17 @@ def pick_decode_splits(B: int, nkv: int, max_kv_len: int, sm_count: int = 148) -
 
 def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv, hd, sm_scale,
                            window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, splits=0,
-                           max_kv_len=None, cu_q=None):
-    """One query token per sequence.  q: [B, >= nh*hd] with row stride q.stride(0)."""
+                           max_kv_len=None, cu_q=None, sinks=None, v_dim=None, gate=None):
+    """One query token per sequence.  q: [B, >= nh*hd] with row stride q.stride(0).  ``sinks`` (fp32 [nh]): a number per
+    head whose exponential joins the softmax denominator.  ``v_dim``: only the leading channels of a head's output
+    exist.  ``gate`` [B, nh * v_dim] (any row pitch, the type of the output): the output is multiplied by its sigmoid."""
     B = seq_lens.shape[0]
+    od = hd if v_dim is None else int(v_dim)
+    extra = (_p(sinks), od, _p(gate), gate.stride(0) if gate is not None else 0)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_decode", block_tables, seq_lens, k_cache)
     if not q.is_cuda:
+        assert sinks is None and gate is None and od == hd, "the CPU form of sinks, gates and narrow outputs is ops.qk_attn"
         cu = torch.arange(B + 1, dtype=torch.int32)
         y = reference.paged_attention(q, k_cache, v_cache, block_tables, seq_lens, cu, nh, nkv, hd,
                                       sm_scale, window, softcap, k_scale, v_scale)
@@ -447,11 +452,11 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
             return out
         return y
     if out is None:
-        out = torch.empty(B, nh * hd, dtype=q.dtype, device=q.device)
+        out = torch.empty(B, nh * od, dtype=q.dtype, device=q.device)
     elif not out.is_contiguous():
-        # the kernels write rows of nh * hd values back to back
+        # the kernels write rows of nh * od values back to back
         tmp = paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv, hd, sm_scale, window,
-                                     softcap, k_scale, v_scale, None, splits, max_kv_len, cu_q)
+                                     softcap, k_scale, v_scale, None, splits, max_kv_len, cu_q, sinks, v_dim, gate)
         out.copy_(tmp)
         return out
     if splits <= 0:
@@ -460,6 +465,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
         eff = min(max_kv_len, window) if window and window > 0 else max_kv_len
         splits = pick_decode_splits(B, nkv, eff)
     mode = reference.kv_mode(k_cache)
+    assert mode < 2 or (sinks is None and gate is None and od == hd), "row-scaled caches take no sinks, gates or narrow outputs"
     if mode >= 2:
         ws_o = ws_ml = None
         if splits > 1:
@@ -477,7 +483,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
         rc = _lib.kernels().fi_paged_decode_cluster(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens), B, nh, nkv, hd,
             block_tables.shape[1], k_cache.shape[2], int(window or 0), sm_scale, float(softcap or 0.0),
-            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, _DT[q.dtype], _stream())
+            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, *extra, _DT[q.dtype], _stream())
         _lib.check(rc, "fi_paged_decode_cluster")
         _count()
         return out
@@ -499,7 +505,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
             _p(ws_o), _p(ws_ml), _p(_merge_tickets(q.device)), B, nh, nkv, hd, block_tables.shape[1],
             k_cache.shape[2], int(window or 0), sm_scale, float(softcap or 0.0),
-            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, _DT[q.dtype], _stream())
+            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, *extra, _DT[q.dtype], _stream())
         _lib.check(rc, "fi_paged_decode_merged")
         _count()
         return out
@@ -507,7 +513,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
         _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
         _p(ws_o), _p(ws_ml), B, nh, nkv, hd, block_tables.shape[1], k_cache.shape[2], int(window or 0),
         sm_scale, float(softcap or 0.0), 1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale,
-        v_scale, splits, _DT[q.dtype], _stream())
+        v_scale, splits, *extra, _DT[q.dtype], _stream())
     _lib.check(rc, "fi_paged_decode")
     _count(2 if splits > 1 else 1)
     return out
@@ -553,15 +559,17 @@ def paged_metadata_snapshot(q, k_cache, block_tables, seq_lens, cu_q=None, scope
 
 def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv,
                             hd, sm_scale, window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, sinks=None,
-                            v_dim=None):
+                            v_dim=None, gate=None):
     """Varlen causal attention of new tokens against the paged cache (which already holds them).  ``sinks`` (fp32
     [nh]): a number per head whose exponential joins the softmax denominator.  ``v_dim``: only the leading ``v_dim``
-    channels of a head's output exist (rows of nh * v_dim)."""
+    channels of a head's output exist (rows of nh * v_dim).  ``gate`` [T, nh * v_dim] (any row pitch, the type of the
+    output): the output is multiplied by its sigmoid."""
     od = hd if v_dim is None else int(v_dim)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_prefill", block_tables, seq_lens, k_cache, cu_q)
     if not q.is_cuda:
-        assert sinks is None and od == hd, "the CPU form of sinks and narrow outputs lives in ops.latent_attn"
+        assert sinks is None and gate is None and od == hd, \
+            "the CPU forms of sinks, gates and narrow outputs live in ops.latent_attn and ops.qk_attn"
         y = reference.paged_attention(q, k_cache, v_cache, block_tables, seq_lens, cu_q, nh, nkv, hd,
                                       sm_scale, window, softcap, k_scale, v_scale)
         if out is not None:
@@ -578,7 +586,8 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         out.copy_(tmp)
         return out
     mode = reference.kv_mode(k_cache)
-    assert mode < 2 or (sinks is None and od == hd), "row-scaled caches take no sinks and no narrow outputs"
+    assert mode < 2 or (sinks is None and gate is None and od == hd), "row-scaled caches take no sinks, gates or narrow outputs"
+    gate_args = (_p(gate), gate.stride(0) if gate is not None else 0)
     if mode >= 2:
         rc = _lib.kernels().fi_paged_prefill_rowscaled(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(k_cache.fi_scales), _p(v_cache.fi_scales), _p(out),
@@ -593,7 +602,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         rc = _lib.kernels().fi_paged_prefill_tc(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens), _p(cu_q), B, T,
             int(max_q_len), nh, nkv, hd, k_cache.shape[0], block_tables.shape[1], k_cache.shape[2], int(window or 0),
-            sm_scale, float(softcap or 0.0), _p(sinks), od, _DT[q.dtype], _p(status_word(q.device)), _stream())
+            sm_scale, float(softcap or 0.0), _p(sinks), od, *gate_args, _DT[q.dtype], _p(status_word(q.device)), _stream())
         if rc != -12:       # -12: outside what the tensor-core kernel covers, take the general one
             _lib.check(rc, "fi_paged_prefill_tc")
             _count()
@@ -602,7 +611,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
         _p(cu_q), B, int(max_q_len), nh, nkv, hd, block_tables.shape[1], k_cache.shape[2],
         int(window or 0), sm_scale, float(softcap or 0.0),
-        1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, _p(sinks), od, _DT[q.dtype], _stream())
+        1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, _p(sinks), od, *gate_args, _DT[q.dtype], _stream())
     _lib.check(rc, "fi_paged_prefill")
     _count()
     return out
@@ -654,6 +663,17 @@ def activation(x, act="silu", out=None):
     _lib.check(rc, "fi_act")
     _count()
     return out
+
+
+def soft_cap(x, cap: float):
+    """``x <- cap * tanh(x / cap)`` in place on fp32 rows."""
+    if not x.is_cuda:
+        return x.div_(cap).tanh_().mul_(cap)
+    assert x.dtype == torch.float32 and x.stride(1) == 1 and cap > 0
+    rc = _lib.kernels().fi_soft_cap(_p(x), x.stride(0), x.shape[0], x.shape[1], float(cap), _stream())
+    _lib.check(rc, "fi_soft_cap")
+    _count()
+    return x
 
 
 def slot_mapping(positions, token_seq, block_tables, block_size, out=None):

@@ -12,6 +12,9 @@ Per value head, with state ``S [dk, dv]``, decay ``a_t = exp(g_t)`` and write st
 * :func:`gated_delta_step` / :func:`conv1d_step` - one decode step for a batch of sequences on state
   pools indexed by slot (CUDA kernels in csrc/linear_attn/gated_delta.cu; PyTorch on the CPU).
 
+* :func:`delta_portions` / :func:`delta_step` - the rule with one decay per key channel, its short convolutions, unit
+  vectors, head norm and gate included (csrc/linear_attn/channel_delta.cu; PyTorch on the CPU).
+
 Reference: vllm/model_executor/models/qwen3_5.py:127-200 (chunk-64 rule), :203-260 (recurrent rule).
 """
 from __future__ import annotations
@@ -19,7 +22,7 @@ from __future__ import annotations
 import torch
 import torch.nn.functional as F
 
-from . import _DT, _count, _lib, _p, _stream
+from . import _DT, _count, _lib, _p, _stream, scratch, status_word
 
 
 def gated_delta_recurrent(q, k, v, g, beta, S0=None):
@@ -180,14 +183,18 @@ def hgrn2_scan(q, f, v, f_bias, lower, pool, slots, cu_q, seq_lens, H: int, d: i
     return o
 
 
-def head_norm(o, w, eps: float, out_dtype):
-    """RMS norm of every head's row: o fp32 [T, H, dv], w fp32 [dv] -> [T, H * dv]."""
+def head_norm(o, w, eps: float, out_dtype, gate=None):
+    """RMS norm of every head's row: o fp32 [T, H, dv], w fp32 [dv] -> [T, H * dv], times ``sigmoid(gate)`` if there is a
+    gate [T, H * dv] (any row pitch and type)."""
     T, H, dv = o.shape
     if not o.is_cuda:
-        y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w
-        return y.reshape(T, H * dv).to(out_dtype)
+        y = (o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w).reshape(T, H * dv)
+        return (y if gate is None else y * torch.sigmoid(gate.float())).to(out_dtype)
     out = torch.empty(T, H * dv, dtype=out_dtype, device=o.device)
-    rc = _lib.kernels().fi_head_norm(_p(o), _p(w), _p(out), T * H, dv, eps, _DT[out_dtype], _stream())
+    assert gate is None or gate.stride(1) == 1
+    rc = _lib.kernels().fi_head_norm(_p(o), _p(w), _p(gate), gate.stride(0) if gate is not None else 0,
+                                     _DT[gate.dtype] if gate is not None else 0, H, _p(out), T * H, dv, eps,
+                                     _DT[out_dtype], _stream())
     _lib.check(rc, "fi_head_norm")
     _count()
     return out
@@ -214,5 +221,118 @@ def hgrn2_step(q, f, v, f_bias, lower, pool, slots, seq_lens, norm_w, eps: float
                                       _p(pool), _p(slots), _p(seq_lens), _p(norm_w), eps, _p(out), B, H, d, dv,
                                       pool.shape[0], _DT[q.dtype], _DT[f.dtype], _DT[out_dtype], _stream())
     _lib.check(rc, "fi_hgrn2_step")
+    _count()
+    return out
+
+
+# ---------------------------------------------------------------------------- delta rule with channel decays
+DELTA_CHUNK = 16
+
+
+class DeltaSpec:
+    """Sizes and small weights of one layer: ``H`` value heads, ``G`` query / key heads, ``d`` and ``dv`` channels, the
+    convolution ``conv`` fp32 [2 G d + H dv, taps], ``rate`` fp32 [H] (exp of the stored logarithm) and ``bias`` fp32
+    [H * d] of the decays."""
+
+    def __init__(self, H: int, G: int, d: int, dv: int, conv, rate, bias):
+        self.H, self.G, self.d, self.dv, self.conv, self.rate, self.bias = H, G, d, dv, conv, rate, bias
+        self.taps = conv.shape[1]
+        self.channels = 2 * G * d + H * dv
+
+
+def _delta_operands(x, z, b, m: DeltaSpec):
+    """x fp32 [taps - 1 + L, C] (with the inputs before the portion) -> q, k [L, H, d], v [L, H, dv], g [L, H, d],
+    beta [L, H]."""
+    L, G, H, d = z.shape[0], m.G, m.H, m.d
+    y = F.silu((x.unfold(0, m.taps, 1) * m.conv).sum(-1))
+    q, k = y[:, :G * d].view(L, G, d), y[:, G * d:2 * G * d].view(L, G, d)
+    q = q / torch.sqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6) * d ** -0.5
+    k = k / torch.sqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+    g = torch.exp(-m.rate[:, None] * F.softplus(z.float() + m.bias).view(L, H, d))
+    return (q.repeat_interleave(H // G, 1), k.repeat_interleave(H // G, 1), y[:, 2 * G * d:].view(L, H, m.dv), g,
+            torch.sigmoid(b.float()))
+
+
+def _delta_sequence(x, z, b, m: DeltaSpec, S, ring, pos0: int):
+    """One portion on the CPU; ``S`` and ``ring`` are updated in place.  Returns fp32 [L, H, dv]."""
+    L, taps = x.shape[0], m.taps
+    before = [ring[p % taps] if p >= 0 else torch.zeros(m.channels) for p in range(pos0 - taps + 1, pos0)]
+    q, k, v, g, beta = _delta_operands(torch.cat([torch.stack(before), x.float()] if before else [x.float()]), z, b, m)
+    o = torch.empty(L, m.H, m.dv)
+    for t in range(L):
+        S.mul_(g[t][:, :, None])
+        u = beta[t][:, None] * (v[t] - torch.einsum("hkv,hk->hv", S, k[t]))
+        S.add_(k[t][:, :, None] * u[:, None, :])
+        o[t] = torch.einsum("hkv,hk->hv", S, q[t])
+    for p in range(max(pos0, pos0 + L - taps + 1), pos0 + L):
+        ring[p % taps].copy_(x[p - pos0])
+    return o
+
+
+def delta_chunks(cu_q):
+    """Running count (int32 [B + 1]) of the chunks of each portion."""
+    n = (cu_q[1:] - cu_q[:-1] + DELTA_CHUNK - 1) // DELTA_CHUNK
+    return F.pad(torch.cumsum(n, 0), (1, 0)).to(torch.int32)
+
+
+def delta_portions(x, z, b, m: DeltaSpec, pool, ring, slots, cu_q, seq_lens, chunk_base, n_chunks: int):
+    """Portions of sequences.  x [T, C] (q | k | v projections), z [T, H * d] fp32 (decays), b [T, H] fp32 (write
+    strengths), rows of any pitch.  pool fp32 [num_slots, H, d, dv] and ring fp32 [num_slots, taps, C], updated in place;
+    slots, seq_lens: int32 [B]; cu_q: int32 [B + 1]; ``chunk_base`` of :func:`delta_chunks`, ``n_chunks`` its last entry.
+    A portion as long as its sequence starts from a zero state.  Returns o fp32 [T, H, dv]."""
+    T, B = x.shape[0], slots.shape[0]
+    if not x.is_cuda:
+        o = torch.empty(T, m.H, m.dv, dtype=torch.float32)
+        cu, lens = cu_q.tolist(), seq_lens.tolist()
+        for i, s in enumerate(slots.tolist()):
+            lo, hi = cu[i], cu[i + 1]
+            if hi <= lo:
+                continue
+            if lens[i] == hi - lo:
+                pool[s].zero_()
+            o[lo:hi] = _delta_sequence(x[lo:hi], z[lo:hi], b[lo:hi], m, pool[s], ring[s], lens[i] - (hi - lo))
+        return o
+    lib = _lib.kernels()
+    per = lib.fi_delta_work_floats(m.d, m.dv)
+    if per < 0:
+        raise ValueError(f"no kernel for {m.d} key channels and {m.dv} value channels per head")
+    assert x.stride(1) == z.stride(1) == b.stride(1) == 1 and z.dtype == b.dtype == torch.float32
+    assert pool.dtype == ring.dtype == torch.float32 and pool.is_contiguous() and ring.is_contiguous()
+    assert slots.dtype == cu_q.dtype == seq_lens.dtype == chunk_base.dtype == torch.int32
+    work = scratch("delta_work", n_chunks * m.H * per * 4, x.device)
+    o = torch.empty(T, m.H, m.dv, dtype=torch.float32, device=x.device)
+    rc = lib.fi_delta_portions(_p(x), x.stride(0), _p(z), z.stride(0), _p(b), b.stride(0), _p(m.conv), _p(m.rate), _p(m.bias),
+                               _p(pool), _p(ring), _p(slots), _p(cu_q), _p(seq_lens), _p(chunk_base), n_chunks, _p(work),
+                               _p(o), B, m.H, m.G, m.d, m.dv, m.taps, pool.shape[0], _DT[x.dtype], _p(status_word(x.device)),
+                               _stream())
+    _lib.check(rc, "fi_delta_portions")
+    _count(2)
+    return o
+
+
+def delta_step(x, z, b, m: DeltaSpec, pool, ring, slots, seq_lens, norm_w, eps: float, gate, out_dtype):
+    """One token per sequence with head norm and output gate: operands as in :func:`delta_portions`, ``norm_w`` fp32
+    [dv], ``gate`` [B, H * dv] or None.  Rows with ``seq_lens`` <= 0 are padding (zero output, no state touched).
+    Returns [B, H * dv]."""
+    B = slots.shape[0]
+    if not x.is_cuda:
+        o = torch.zeros(B, m.H, m.dv, dtype=torch.float32)
+        for i, (s, n) in enumerate(zip(slots.tolist(), seq_lens.tolist())):
+            if n <= 0 or s < 0:
+                continue
+            if n == 1:
+                pool[s].zero_()
+            o[i] = _delta_sequence(x[i:i + 1], z[i:i + 1], b[i:i + 1], m, pool[s], ring[s], n - 1)[0]
+        return head_norm(o, norm_w, eps, out_dtype, gate)
+    assert x.stride(1) == z.stride(1) == b.stride(1) == 1 and z.dtype == b.dtype == torch.float32
+    assert pool.dtype == ring.dtype == torch.float32 and pool.is_contiguous() and ring.is_contiguous()
+    assert gate is None or gate.stride(1) == 1
+    out = torch.empty(B, m.H * m.dv, dtype=out_dtype, device=x.device)
+    rc = _lib.kernels().fi_delta_step(
+        _p(x), x.stride(0), _p(z), z.stride(0), _p(b), b.stride(0), _p(m.conv), _p(m.rate), _p(m.bias), _p(pool), _p(ring),
+        _p(slots), _p(seq_lens), _p(norm_w), eps, _p(gate), gate.stride(0) if gate is not None else 0,
+        _DT[gate.dtype] if gate is not None else 0, _p(out), B, m.H, m.G, m.d, m.dv, m.taps, pool.shape[0], _DT[x.dtype],
+        _DT[out_dtype], _stream())
+    _lib.check(rc, "fi_delta_step")
     _count()
     return out

@@ -1,6 +1,8 @@
-"""32-bit residual stream with norms before and after each sublayer and a weighted average over depth.
+"""32-bit residual stream with norms before and after each sublayer and a weighted average over depth, or with one norm
+that sublayers read side by side.
 
-    start    X_0 = table[ids]
+    start    X_0 = table[ids] * scale
+    add      x = x + y + sum_k w_k e_k        (y: mixer, e: outputs of the chosen experts)
     step     x = x + norm(y) * w_post
     average  X_n = x + norm(y) * w_post;  x = sum_{j <= n} a_j X_j
     each returns h = norm(x) * w_pre, the input of the next sublayer
@@ -30,18 +32,18 @@ def _padded_rows(rows: int, width: int, dtype, device):
     return buf[:, :width] if w8 != width else buf
 
 
-def start(ids, table, w_pre, eps: float, groups: int, x0):
+def start(ids, table, w_pre, eps: float, groups: int, x0, scale: float = 1.0):
     """``x0`` (fp32 [T, W]) receives the embedding output; returns h in the table's dtype."""
     T, W = x0.shape
     if not table.is_cuda:
-        x0.copy_(table.index_select(0, ids.long()))
+        x0.copy_(table.index_select(0, ids.long()).float() * scale)
         return grouped_rmsnorm(x0, w_pre, eps, groups, table.dtype)
     if _ops._BOUNDS_CHECK:
         _check_index("residual_stream.start.ids", ids, 0, table.shape[0], "rows of the embedding table")
     assert ids.dtype == torch.int64 and x0.dtype == torch.float32 and x0.is_contiguous() and table.is_contiguous()
     h = _padded_rows(T, W, table.dtype, table.device)
-    rc = _lib.kernels().fi_stream_start(_p(ids), _p(table), table.shape[0], _p(w_pre), _p(x0), _p(h), h.stride(0), T, W,
-                                        groups, eps, _DT[table.dtype], _stream())
+    rc = _lib.kernels().fi_stream_start(_p(ids), _p(table), table.shape[0], float(scale), _p(w_pre), _p(x0), _p(h), h.stride(0),
+                                        T, W, groups, eps, _DT[table.dtype], _stream())
     _lib.check(rc, "fi_stream_start")
     _count()
     return h
@@ -89,5 +91,39 @@ def average(y, x, w_post, w_pre, eps: float, groups: int, hist, n: int, avg, x_o
                                           h.stride(0) if h is not None else W, _DT[h_dtype], _p(sel), rows, W, groups,
                                           eps, _stream())
     _lib.check(rc, "fi_stream_average")
+    _count()
+    return h
+
+
+def add(y, x, routed, w_pre, eps: float, groups: int, x_out, h_dtype, sel=None):
+    """``x_out = x + y + routed`` (``x_out`` may alias ``x``); returns ``norm(x_out) * w_pre`` (None without ``w_pre``).
+    ``routed`` (:class:`ops.moe.RoutedRows` or None): weighted sum of expert outputs.  ``sel`` (int64 token rows): only
+    these rows are wanted; h has one row per entry and ``x_out`` is not written."""
+    T, W = x.shape
+    if not x.is_cuda:
+        v = x + y.float()
+        if routed is not None:
+            v = v + routed.combined()
+        if sel is not None:
+            v = v.index_select(0, sel)
+        elif x_out is not None:
+            x_out.copy_(v)
+        return None if w_pre is None else grouped_rmsnorm(v, w_pre, eps, groups, h_dtype)
+    assert x.is_contiguous() and x.dtype == torch.float32 and y.stride(1) == 1
+    rows = T if sel is None else sel.shape[0]
+    if sel is not None:
+        x_out = None
+        assert sel.dtype == torch.int64
+        if _ops._BOUNDS_CHECK:
+            _check_index("residual_stream.add.sel", sel, 0, T, "token rows of the step")
+    h = None if w_pre is None else _padded_rows(rows, W, h_dtype, x.device)
+    r = routed
+    if r is not None:
+        assert r.rows.dtype == y.dtype and r.rows.stride(1) == 1 and r.weights.is_contiguous()
+    rc = _lib.kernels().fi_stream_add(
+        _p(y), y.stride(0), _DT[y.dtype], _p(x), _p(r.rows) if r else None, r.rows.stride(0) if r else 0,
+        _p(r.slot_of) if r else None, _p(r.weights) if r else None, r.weights.shape[1] if r else 0, _p(w_pre), _p(x_out),
+        _p(h), h.stride(0) if h is not None else W, _DT[h_dtype], _p(sel), rows, W, groups, eps, _stream())
+    _lib.check(rc, "fi_stream_add")
     _count()
     return h
