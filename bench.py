@@ -66,6 +66,8 @@ def parse_args():
                     help="instead of the headline workload: kernels and prefill / decode throughput of the Fimodra design at a "
                          "few layer sizes beside the closest models (one GPU, random weights); one JSON line")
     ap.add_argument("--fimodra-sizes", type=int, nargs="*", default=None, help="widths for --fimodra (default: all)")
+    ap.add_argument("--pofadra", action="store_true", help="the same for the Pofadra design")
+    ap.add_argument("--pofadra-sizes", type=int, nargs="*", default=None, help="widths for --pofadra (default: all)")
     return ap.parse_args()
 
 
@@ -573,14 +575,12 @@ def run_reference(args) -> dict:
     return run_reference_bench(args, METRIC, BASELINE_TPS)
 
 
-def run_fimodra(args) -> dict:
+def run_shapes(shapes, sizes) -> dict:
     import torch
-
-    from benchmarks import fimodra_shapes
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    res = fimodra_shapes.run(args.fimodra_sizes or sorted(fimodra_shapes.SIZES))
+    res = shapes.run(sizes or sorted(shapes.SIZES))
     sampler.stop()
     res["clocks"] = sampler.summary(min_power_w=250.0)
     return res
@@ -589,7 +589,12 @@ def run_fimodra(args) -> dict:
 def main():
     args = parse_args()
     if args.fimodra:
-        print(json.dumps(run_fimodra(args)), flush=True)
+        from benchmarks import fimodra_shapes
+        print(json.dumps(run_shapes(fimodra_shapes, args.fimodra_sizes)), flush=True)
+        return
+    if args.pofadra:
+        from benchmarks import pofadra_shapes
+        print(json.dumps(run_shapes(pofadra_shapes, args.pofadra_sizes)), flush=True)
         return
     res = run_reference(args) if args.impl == "reference" else run_ours(args)
     if res:

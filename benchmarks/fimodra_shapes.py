@@ -213,66 +213,66 @@ def _configs(width: int, layers: int) -> dict:
     return {"fimodra": ours, "qwen3.5-style hybrid": qwen}
 
 
-def model_rows(width: int, layers: int = 8, batch: int = 32, prompt: int = 1024, steps: int = 64) -> list[dict]:
+def throughput_row(width: int, name: str, cfg: dict, layers: int = 8, batch: int = 32, prompt: int = 1024, steps: int = 64) -> dict:
     """Prefill tokens/s of ``8 x prompt`` token steps and decode tokens/s at ``batch`` through the engine."""
     import torch
 
     from litevllm_b200 import LLM, SamplingParams
     from litevllm_b200.models.presets import PRESETS
-    rows = []
-    for name, cfg in _configs(width, layers).items():
-        PRESETS["shape-comparison"] = cfg
-        llm = LLM("synthetic:shape-comparison", dtype="bfloat16", max_num_seqs=batch, max_model_len=prompt + steps + 64,
-                  max_num_batched_tokens=8192, fastinference_config={"profile": "throughput", "tuning_keyvals": {
-                      "FASTINFERENCE_KV_MAX_ACTIVE_REQUESTS": str(batch), "FASTINFERENCE_LITE_PREFILL_MICROBATCH": "8",
-                      "FASTINFERENCE_GPU_GREEDY_SAMPLING": "0"}})
-        eng = llm.engine
-        g = torch.Generator().manual_seed(1)
-        ids = torch.randint(0, 32000, (batch, prompt), generator=g).tolist()
-        times = []
-        for rep in range(3):
-            done = batch
-            sp = SamplingParams(temperature=0.0, max_tokens=1, ignore_eos=True)
-            for i in range(batch):
-                eng.add_request(f"p{rep}-{i}", ids[i], sp)
-            torch.cuda.synchronize()
-            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            a.record()
-            while eng.has_unfinished_requests():
-                eng.step()
-            b.record()
-            torch.cuda.synchronize()
-            times.append(a.elapsed_time(b))
-            assert done == batch
-        prefill = batch * prompt / (min(times[1:]) / 1e3)
-        sp = SamplingParams(temperature=0.0, max_tokens=steps + 32, ignore_eos=True)
+    PRESETS["shape-comparison"] = cfg
+    llm = LLM("synthetic:shape-comparison", dtype="bfloat16", max_num_seqs=batch, max_model_len=prompt + steps + 64,
+              max_num_batched_tokens=8192, fastinference_config={"profile": "throughput", "tuning_keyvals": {
+                  "FASTINFERENCE_KV_MAX_ACTIVE_REQUESTS": str(batch), "FASTINFERENCE_LITE_PREFILL_MICROBATCH": "8",
+                  "FASTINFERENCE_GPU_GREEDY_SAMPLING": "0"}})
+    eng = llm.engine
+    g = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, 32000, (batch, prompt), generator=g).tolist()
+    times = []
+    for rep in range(3):
+        sp = SamplingParams(temperature=0.0, max_tokens=1, ignore_eos=True)
         for i in range(batch):
-            eng.add_request(f"d-{i}", ids[i], sp)
-        while any(st.is_prefill for st in eng.scheduler.requests.values()):
-            eng.step()
-        for _ in range(8):
-            eng.step()
+            eng.add_request(f"p{rep}-{i}", ids[i], sp)
         torch.cuda.synchronize()
         a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        n = 0
         a.record()
-        for _ in range(steps):
-            n += len(eng.step())
-        b.record()
-        torch.cuda.synchronize()
-        ms = a.elapsed_time(b)
-        rows.append({"width": width, "layers": layers, "model": name, "prefill_tok_s": round(prefill), "decode_tok_s": round(n / (ms / 1e3)),
-                     "decode_ms_per_step": round(ms / steps, 3), "batch": batch, "prompt": prompt,
-                     "params_m": round(sum(p.numel() for p in eng.model.parameters()) / 1e6),
-                     "kernels_per_decode_step": eng.decode_executor.launches_per_graph.get(eng.builder.bucket_for(batch))})
         while eng.has_unfinished_requests():
             eng.step()
-        llm.shutdown()
-        del llm, eng
-        PRESETS.pop("shape-comparison")
-        gc.collect()
-        torch.cuda.empty_cache()
-    return rows
+        b.record()
+        torch.cuda.synchronize()
+        times.append(a.elapsed_time(b))
+    prefill = batch * prompt / (min(times[1:]) / 1e3)
+    sp = SamplingParams(temperature=0.0, max_tokens=steps + 32, ignore_eos=True)
+    for i in range(batch):
+        eng.add_request(f"d-{i}", ids[i], sp)
+    while any(st.is_prefill for st in eng.scheduler.requests.values()):
+        eng.step()
+    for _ in range(8):
+        eng.step()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    n = 0
+    a.record()
+    for _ in range(steps):
+        n += len(eng.step())
+    b.record()
+    torch.cuda.synchronize()
+    ms = a.elapsed_time(b)
+    row = {"width": width, "layers": layers, "model": name, "prefill_tok_s": round(prefill), "decode_tok_s": round(n / (ms / 1e3)),
+           "decode_ms_per_step": round(ms / steps, 3), "batch": batch, "prompt": prompt,
+           "params_m": round(sum(p.numel() for p in eng.model.parameters()) / 1e6),
+           "kernels_per_decode_step": eng.decode_executor.launches_per_graph.get(eng.builder.bucket_for(batch))}
+    while eng.has_unfinished_requests():
+        eng.step()
+    llm.shutdown()
+    del llm, eng
+    PRESETS.pop("shape-comparison")
+    gc.collect()
+    torch.cuda.empty_cache()
+    return row
+
+
+def model_rows(width: int, layers: int = 8) -> list[dict]:
+    return [throughput_row(width, name, cfg, layers) for name, cfg in _configs(width, layers).items()]
 
 
 def run(sizes, kernels: bool = True, models: bool = True, only: str = "") -> dict:
