@@ -8,15 +8,17 @@
 //
 // Portions of prompts run in chunks of 16 tokens.  With E_i the product of the decays from the chunk's start through
 // token i (per channel), a chunk's writes are u_i = beta_i (v_i - S_0^T (E_i k_i) - sum_{j<i} a_ij u_j) with
-// a_ij = sum_c k_i k_j E_i / E_j, so they solve a unit lower-triangular system:  U = U0 - W S_0.
+// a_ij = sum_c k_i k_j E_i / E_j, so they solve a unit lower-triangular system, U = U0 - W S_0, and its outputs are
+// o = (E q) S_0 + P U = (E q - P W) S_0 + P U0 with p_ij = sum_c q_i k_j E_i / E_j (j <= i).
 //
 //   delta_chunk_kernel   everything that does not depend on the state, for all chunks in parallel: convolutions, unit
-//                        vectors, decays, a_ij and p_ij = sum_c q_i k_j E_i / E_j, the solved U0 and W.  Ratios
-//                        E_i / E_j are running products of decays from j to i: at most one, and nothing is divided.
-//   delta_scan_kernel    chunk after chunk: X = [W; E q] S (a reduction over d), U = U0 - X_W, o = X_q + P U,
-//                        S <- E_16 S + sum_j (E_16 / E_j) k_j u_j^T.  Columns of S never interact: a warp owns a few of
-//                        them with its share of S in registers (16 lanes split the rows), one block-wide meeting per
-//                        chunk hands over the operands, which arrive by bulk copies.
+//                        vectors, decays, a_ij and p_ij, the solved W and U0, Q = E q - P W and P U0.  Ratios E_i / E_j
+//                        are running products of decays from j to i: at most one, and nothing is divided.
+//   delta_scan_kernel    chunk after chunk: [U; o] = [U0; P U0] + [-W; Q] S, S <- E_16 S + sum_j (E_16 / E_j) k_j u_j^T.
+//                        A block owns some columns of S, each warp (or half of one) a range of its rows, and each lane
+//                        one or two columns of those in registers, so the operand rows are read as broadcasts and a
+//                        product needs no exchange between lanes; the row ranges' partial sums meet in shared memory,
+//                        first those of U, then those of o.  Operands arrive by bulk copies.
 //   delta_step_kernel    one token per sequence (decode): convolution, unit vectors, decays, state, per-head norm and
 //                        output gate in one pass that reads and writes the state once.
 //
@@ -70,10 +72,20 @@ __device__ __forceinline__ float ld_any(const void* p, long i, int type) {
   return __half2float(reinterpret_cast<const __half*>(p)[i]);
 }
 __device__ __forceinline__ float sigmoidf(float z) { return 1.f / (1.f + __expf(-z)); }
-// log(1 + e^z) without overflow; the small branch keeps the relative precision of tiny results
+// log(1 + e^z) = max(z, 0) + log(1 + e), e = e^-|z|, by log(1 + e) = 2 artanh(e / (2 + e)): a power series of s <= 1/3
+// that keeps the relative precision of tiny results
 __device__ __forceinline__ float softplusf(float z) {
   const float e = __expf(-fabsf(z));
-  return fmaxf(z, 0.f) + (e < 1e-3f ? e - 0.5f * e * e : log1pf(e));
+  const float s = __fdividef(e, 2.f + e), s2 = s * s;
+  float a = 1.f / 15.f;
+  a = fmaf(a, s2, 1.f / 13.f);
+  a = fmaf(a, s2, 1.f / 11.f);
+  a = fmaf(a, s2, 1.f / 9.f);
+  a = fmaf(a, s2, 1.f / 7.f);
+  a = fmaf(a, s2, 1.f / 5.f);
+  a = fmaf(a, s2, 1.f / 3.f);
+  a = fmaf(a, s2, 1.f);
+  return fmaf(2.f * s, a, fmaxf(z, 0.f));
 }
 // e^x for x <= 0.  Slow decays multiply over thousands of tokens, so close to one the error has to stay at rounding:
 // the power series there, the special-function unit further out (what it loses is forgotten within a few tokens).
@@ -108,16 +120,17 @@ struct DeltaParams {
   const void* gate;       // step: [B, ldg] (H * dv) or null
   void* out;              // step: [B, H * dv]
   long ld, ldz, ldb, ldg, work_stride;
-  int B, H, G, d, dv, dp, dvp, C, taps, num_slots, n_chunks, gate_type, out_type;
+  int B, H, G, d, dv, dp, dvp, C, taps, num_slots, n_chunks, gate_type, out_type, vec_o;
   float eps, q_scale;
 };
 
-// work block of a (chunk, head), in floats: W [16][dp] | E q [16][dp] | (E_16 / E) k [16][dp] | E_16 [dp] | P [16][16] |
-// U0 [dvp / 16][16 tokens][16 columns]
-__host__ __device__ inline long work_floats(int dp, int dvp) { return 49l * dp + 256 + 16l * dvp; }
+// work block of a (chunk, head), in floats: -W [16][dp] | Q [16][dp] | (E_16 / E) k [16][dp] | E_16 [dp] |
+// groups of 16 columns [dvp / 16] of U0 [16 tokens][16] | P U0 [16 tokens][16]
+__host__ __device__ inline long work_floats(int dp, int dvp) { return 49l * dp + 32l * dvp; }
 
-template <typename T>
-__global__ void __launch_bounds__(256, 2) delta_chunk_kernel(const DeltaParams p) {
+// TAPS: convolution length known at compile time (0: any).
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256, 3) delta_chunk_kernel(const DeltaParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   extern __shared__ __align__(128) float smem[];
@@ -134,114 +147,159 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_kernel(const DeltaParams p
   const int slot = p.slots[b];
   if (valid <= 0 || slot < 0 || slot >= p.num_slots) return;
   const int pos0 = p.seq_lens[b] - n;  // position of the portion's first token
-  const int d = p.d, dv = p.dv, dp = p.dp, taps = p.taps, hist = taps - 1;
+  const int d = p.d, dv = p.dv, dp = p.dp, taps = TAPS > 0 ? TAPS : p.taps, hist = taps - 1;
+  const int sp = (d + 3) & ~3;         // pitch of the key-channel rows
   const int width = 2 * d + dv;
   const int kvh = head / (p.H / p.G);
-  float* xs = smem;                                        // [16 + hist][width] convolution inputs
-  float* sq = xs + max((kTok + hist) * width, kTok * d);   // [16][d]
-  float* sk = sq + kTok * d;                               // [16][d]
-  float* sg = sk + kTok * d;                               // [16][d]
-  float* sv = sg + kTok * d;                               // [16][dv]
-  float* sA = sv + kTok * dv;                              // [16][16]
-  float* sP = sA + 256;                                    // [16][16]
-  float* sb = sP + 256;                                    // [16]
-  float* skd = xs;                                         // [16][d] E k, once the inputs are used up
+  float* sq = smem;                    // [16][sp] activated q (not yet unit vectors)
+  float* sk = sq + kTok * sp;          // [16][sp]
+  float* sg = sk + kTok * sp;          // [16][sp] decays
+  float* skd = sg + kTok * sp;         // [16][sp] E k
+  float* sqd = skd + kTok * sp;        // [16][sp] E q
+  float* sA = sqd + kTok * sp;         // [16][16]
+  float* sP = sA + 256;                // [16][16]
+  float* sb = sP + 256;                // [16]
+  float* sf = sb + 16;                 // [32] factors that make q (and its scale) and k unit vectors
+  float* sv = sf + 32;                 // [16][dv]
   float* work = p.work + (static_cast<long>(chunk) * p.H + head) * p.work_stride;
 
-  const T* qkv = reinterpret_cast<const T*>(p.qkv);
-  const int cq = kvh * d, ck = p.G * d + kvh * d, cv = 2 * p.G * d + head * dv;
+  // ---- convolutions, activations and decays: an item is one channel over the chunk's tokens
+  const T* qkv = reinterpret_cast<const T*>(p.qkv) + (t_begin + t0) * p.ld;
   const float* ring = p.ring + static_cast<long>(slot) * taps * p.C;
-  for (int c = tid; c < width; c += 256) {
-    const int ch = c < d ? cq + c : (c < 2 * d ? ck + c - d : cv + c - 2 * d);
-#pragma unroll 4
-    for (int r = 0; r < kTok + hist; ++r) {
-      const int s = t0 + r - hist;     // token of the portion; negative: before it
-      float x = 0.f;
-      if (s >= 0) {
-        if (r - hist < valid) x = to_f(qkv[(t_begin + s) * p.ld + ch]);
-      } else if (pos0 + s >= 0) {
-        x = ring[((pos0 + s) % taps) * p.C + ch];
+  const float rate = p.rate[head];
+  for (int c = tid; c < width + d; c += 256) {
+    if (c < width) {
+      const int ch = c < d ? kvh * d + c : (c < 2 * d ? p.G * d + kvh * d + c - d : 2 * p.G * d + head * dv + c - 2 * d);
+      auto input = [&](int r) -> float {         // token t0 + r of the portion (r may be negative)
+        if (r >= 0) {
+          const float x = to_f(qkv[min(r, valid - 1) * p.ld + ch]);
+          return r < valid ? x : 0.f;
+        }
+        if (t0 > 0) return to_f(qkv[r * p.ld + ch]);      // (chunks are longer than the convolution)
+        const int pos = pos0 + r;
+        return pos >= 0 ? ring[(pos % taps) * p.C + ch] : 0.f;
+      };
+      float y[kTok];
+      if constexpr (TAPS > 0) {
+        float x[kTok + TAPS - 1], w[TAPS];
+#pragma unroll
+        for (int r = 0; r < kTok + TAPS - 1; ++r) x[r] = input(r - (TAPS - 1));
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = p.conv[static_cast<long>(ch) * TAPS + j];
+#pragma unroll
+        for (int t = 0; t < kTok; ++t) {
+          y[t] = w[0] * x[t];
+#pragma unroll
+          for (int j = 1; j < TAPS; ++j) y[t] = fmaf(w[j], x[t + j], y[t]);
+        }
+      } else {
+#pragma unroll
+        for (int t = 0; t < kTok; ++t) y[t] = 0.f;
+        for (int j = 0; j < taps; ++j) {
+          const float w = p.conv[static_cast<long>(ch) * taps + j];
+#pragma unroll
+          for (int t = 0; t < kTok; ++t) y[t] = fmaf(w, input(t + j - hist), y[t]);
+        }
       }
-      xs[r * width + c] = x;
+      float* dst = c < d ? sq + c : (c < 2 * d ? sk + c - d : sv + c - 2 * d);
+      const int pitch = c < 2 * d ? sp : dv;
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) dst[t * pitch] = t < valid ? y[t] * sigmoidf(y[t]) : 0.f;
+    } else {
+      const int cg = c - width;
+      const float bias = p.bias[head * d + cg];
+      const float* z = p.z + (t_begin + t0) * p.ldz + head * d + cg;
+      float zz[kTok];
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) zz[t] = z[min(t, valid - 1) * p.ldz];
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) sg[t * sp + cg] = t < valid ? decay_exp(-rate * softplusf(zz[t] + bias)) : 1.f;
     }
   }
-  {
-    const float rate = p.rate[head];
-    for (int c = tid; c < d; c += 256) {
-      const float bias = p.bias[head * d + c];
-      const float* z = p.z + head * d + c;
-#pragma unroll 4
-      for (int t = 0; t < kTok; ++t)
-        sg[t * d + c] = t < valid ? decay_exp(-rate * softplusf(z[(t_begin + t0 + t) * p.ldz] + bias)) : 1.f;
-    }
+  for (int i = tid; i < kTok * (sp - d); i += 256) {       // channels that only fill up the last group of four
+    const int at = (i / (sp - d)) * sp + d + i % (sp - d);
+    sq[at] = 0.f; sk[at] = 0.f; sg[at] = 0.f;
   }
   if (tid < kTok) sb[tid] = tid < valid ? sigmoidf(p.b[(t_begin + t0 + tid) * p.ldb + head]) : 0.f;
   __syncthreads();
-  for (int c = tid; c < width; c += 256) {
-    const int ch = c < d ? cq + c : (c < 2 * d ? ck + c - d : cv + c - 2 * d);
-    float y[kTok];
-#pragma unroll
-    for (int t = 0; t < kTok; ++t) y[t] = 0.f;
-    for (int j = 0; j < taps; ++j) {
-      const float w = p.conv[static_cast<long>(ch) * taps + j];
-#pragma unroll
-      for (int t = 0; t < kTok; ++t) y[t] = fmaf(w, xs[(t + j) * width + c], y[t]);
-    }
-    float* dst = c < d ? sq + c : (c < 2 * d ? sk + c - d : sv + c - 2 * d);
-    const int pitch = c < 2 * d ? d : dv;
-#pragma unroll
-    for (int t = 0; t < kTok; ++t) dst[t * pitch] = t < valid ? y[t] * sigmoidf(y[t]) : 0.f;
-  }
-  __syncthreads();
   const int warp = tid >> 5, lane = tid & 31;
-  for (int r = warp; r < 2 * kTok; r += 8) {               // unit vectors: rows of q, then of k
-    float* row = r < kTok ? sq + r * d : sk + (r - kTok) * d;
-    float ss = 0.f;
-    for (int c = lane; c < d; c += 32) ss += row[c] * row[c];
-    for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
-    const float f = (r < kTok ? p.q_scale : 1.f) / sqrtf(ss + kUnitEps);
-    for (int c = lane; c < d; c += 32) row[c] *= f;
+  {
+    float ss[4];                                           // rows warp, warp + 8 of q, then of k
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float* row = (i < 2 ? sq : sk) + (warp + 8 * (i & 1)) * sp;
+      ss[i] = 0.f;
+      for (int c = lane * 4; c < sp; c += 128) {
+        const float4 v = *reinterpret_cast<const float4*>(row + c);
+        ss[i] += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+      }
+    }
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], m);
+    if (lane < 4) {
+      const float t = lane == 0 ? ss[0] : lane == 1 ? ss[1] : lane == 2 ? ss[2] : ss[3];
+      sf[(lane >> 1) * 16 + warp + 8 * (lane & 1)] = (lane < 2 ? p.q_scale : 1.f) / sqrtf(t + kUnitEps);
+    }
   }
   __syncthreads();
-  float* gq = work + 16l * dp;
-  float* gk = work + 32l * dp;
-  for (int c = tid; c < dp; c += 256) {
-    float e = 1.f;
-    if (c < d) {
+  // ---- running products of decays, forward (E q, E k, E_16) and backward (E_16 / E k)
+  for (int it = tid; it < 2 * dp; it += 256) {
+    const bool back = it >= dp;
+    const int c = back ? it - dp : it;
+    if (c >= d) {                                          // rows of S that only fill up the lanes' groups
+      float* out = work + (back ? 32l : 0l) * dp + c;
 #pragma unroll
       for (int t = 0; t < kTok; ++t) {
-        e *= sg[t * d + c];
-        gq[t * dp + c] = sq[t * d + c] * e;
-        skd[t * d + c] = sk[t * d + c] * e;
+        out[t * dp] = 0.f;
+        if (!back) out[(16 + t) * dp] = 0.f;
+      }
+      if (!back) work[48l * dp + c] = 0.f;
+    } else if (!back) {
+      float e = 1.f;
+#pragma unroll
+      for (int t = 0; t < kTok; ++t) {
+        e *= sg[t * sp + c];
+        sqd[t * sp + c] = sq[t * sp + c] * e * sf[t];
+        skd[t * sp + c] = sk[t * sp + c] * e * sf[16 + t];
       }
       work[48l * dp + c] = e;
+    } else {
       float r = 1.f;
+      float* out = work + 32l * dp + c;
 #pragma unroll
       for (int t = kTok - 1; t >= 0; --t) {
-        gk[t * dp + c] = sk[t * d + c] * r;
-        r *= sg[t * d + c];
+        out[t * dp] = sk[t * sp + c] * r * sf[16 + t];
+        r *= sg[t * sp + c];
       }
-    } else {
-#pragma unroll
-      for (int t = 0; t < kTok; ++t) { gq[t * dp + c] = 0.f; gk[t * dp + c] = 0.f; work[t * dp + c] = 0.f; }
-      work[48l * dp + c] = 0.f;
     }
   }
-  // a_ij (lanes 0-15 end with rows i) and p_ij (lanes 16-31) of two columns j per warp
+  // ---- a_ij (lanes 0-15 end with rows i) and p_ij (lanes 16-31) of two columns j per warp
+#pragma unroll 1
   for (int side = 0; side < 2; ++side) {
     const int j = side == 0 ? warp : kTok - 1 - warp;
     float v[32];
 #pragma unroll
     for (int i = 0; i < 32; ++i) v[i] = 0.f;
-    for (int c = lane; c < d; c += 32) {
-      float w = sk[j * d + c];
+    for (int c = lane * 4; c < sp; c += 128) {
+      const float4 k4 = *reinterpret_cast<const float4*>(sk + j * sp + c);
+      f2 w0 = pack2(k4.x, k4.y), w1 = pack2(k4.z, k4.w);
 #pragma unroll
       for (int i = 0; i < kTok; ++i) {
+        if (i < j) continue;
+        float x, y;
         if (i > j) {
-          w *= sg[i * d + c];
-          v[i] = fmaf(sk[i * d + c], w, v[i]);
+          const float4 g4 = *reinterpret_cast<const float4*>(sg + i * sp + c);
+          const float4 a4 = *reinterpret_cast<const float4*>(sk + i * sp + c);
+          w0 = mul2(w0, pack2(g4.x, g4.y));
+          w1 = mul2(w1, pack2(g4.z, g4.w));
+          unpack2(fma2(pack2(a4.x, a4.y), w0, mul2(pack2(a4.z, a4.w), w1)), x, y);
+          v[i] += x + y;
         }
-        if (i >= j) v[16 + i] = fmaf(sq[i * d + c], w, v[16 + i]);
+        const float4 q4 = *reinterpret_cast<const float4*>(sq + i * sp + c);
+        unpack2(fma2(pack2(q4.x, q4.y), w0, mul2(pack2(q4.z, q4.w), w1)), x, y);
+        v[16 + i] += x + y;
       }
     }
 #pragma unroll
@@ -256,36 +314,52 @@ __global__ void __launch_bounds__(256, 2) delta_chunk_kernel(const DeltaParams p
         }
       }
     }
-    if (lane < 16) sA[lane * 16 + j] = v[0];
-    else sP[(lane - 16) * 16 + j] = v[0];
+    const int i = lane & 15;
+    const float scaled = v[0] * sf[16 + j] * sf[(lane < 16 ? 16 : 0) + i];
+    if (lane < 16) sA[i * 16 + j] = scaled;
+    else sP[i * 16 + j] = scaled;
   }
   __syncthreads();
-  work[49l * dp + tid] = sP[tid];
-  for (int c = tid; c < d + dv; c += 256) {                // solve for one column of W or U0
+  // ---- solve for one column of W or U0 per thread
+  for (int c = tid; c < d + dv; c += 256) {
     const float* src = c < d ? skd + c : sv + c - d;
-    const int pitch = c < d ? d : dv;
+    const int pitch = c < d ? sp : dv;
     float x[kTok];
 #pragma unroll
     for (int i = 0; i < kTok; ++i) {
-      asm volatile("" ::: "memory");                       // keeps the 120 coefficients from being loaded all at once
+      asm volatile("" ::: "memory");                       // keeps the coefficients from being loaded all at once
       float r = src[i * pitch];
 #pragma unroll
-      for (int j = 0; j < i; ++j) r = fmaf(-sA[i * 16 + j], x[j], r);
+      for (int j4 = 0; j4 < (i + 3) / 4; ++j4) {           // coefficients from i on are zero
+        const float4 a4 = *reinterpret_cast<const float4*>(sA + i * 16 + j4 * 4);
+        r = fmaf(-a4.x, x[j4 * 4], r);
+        if (j4 * 4 + 1 < i) r = fmaf(-a4.y, x[j4 * 4 + 1], r);
+        if (j4 * 4 + 2 < i) r = fmaf(-a4.z, x[j4 * 4 + 2], r);
+        if (j4 * 4 + 3 < i) r = fmaf(-a4.w, x[j4 * 4 + 3], r);
+      }
       x[i] = sb[i] * r;
     }
-    if (c < d) {
+    float* out = c < d ? work + c : work + 49l * dp + ((c - d) >> 4) * 512 + ((c - d) & 15);
+    const int step = c < d ? dp : 16;
 #pragma unroll
-      for (int i = 0; i < kTok; ++i) work[i * dp + c] = x[i];
-    } else {
-      const int cc = c - d;
-      float* u0 = work + 49l * dp + 256 + (cc >> 4) * 256 + (cc & 15);
+    for (int i = 0; i < kTok; ++i) {                       // P W or P U0
+      asm volatile("" ::: "memory");
+      float r = 0.f;
 #pragma unroll
-      for (int i = 0; i < kTok; ++i) u0[i * 16] = x[i];
+      for (int j4 = 0; j4 <= i / 4; ++j4) {
+        const float4 p4 = *reinterpret_cast<const float4*>(sP + i * 16 + j4 * 4);
+        r = fmaf(p4.x, x[j4 * 4], r);
+        if (j4 * 4 + 1 <= i) r = fmaf(p4.y, x[j4 * 4 + 1], r);
+        if (j4 * 4 + 2 <= i) r = fmaf(p4.z, x[j4 * 4 + 2], r);
+        if (j4 * 4 + 3 <= i) r = fmaf(p4.w, x[j4 * 4 + 3], r);
+      }
+      out[i * step] = c < d ? -x[i] : x[i];
+      out[(16 + i) * step] = c < d ? sqd[i * sp + c] - r : r;
     }
   }
-  for (int i = tid; i < (p.dvp - dv) * 16; i += 256) {
-    const int cc = dv + i / 16;
-    work[49l * dp + 256 + (cc >> 4) * 256 + (i & 15) * 16 + (cc & 15)] = 0.f;
+  for (int i = tid; i < (p.dvp - dv) * 32; i += 256) {
+    const int cc = dv + i / 32;
+    work[49l * dp + (cc >> 4) * 512 + (i & 31) * 16 + (cc & 15)] = 0.f;
   }
 }
 
@@ -295,20 +369,20 @@ __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t b
                : "memory");
 }
 
-constexpr int kWarps = 8;
-
-// R rows per lane (dp == 16 R), C columns per lane (a warp: 2 C columns, a block: 16 C).
-template <int R, int C, int STAGES>
-__global__ void __launch_bounds__(kWarps * 32) delta_scan_kernel(const DeltaParams p, int* status) {
+// WARPS x LR row ranges of RPL rows (dp == WARPS LR RPL); a lane owns CPL columns of its range, a block 32 / LR * CPL.
+template <int RPL, int LR, int CPL, int WARPS, int STAGES>
+__global__ void __launch_bounds__(WARPS * 32) delta_scan_kernel(const DeltaParams p, int* status) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
-  constexpr int DP = 16 * R;
-  constexpr int COLS = kWarps * 2 * C;
-  constexpr int kOper = 49 * DP + 256;                     // floats of a stage before U0
-  constexpr int kStage = kOper + COLS * 16;
-  constexpr int TG = 16 / C;                               // tokens whose partial sums are reduced together
+  constexpr int THREADS = WARPS * 32;
+  constexpr int PARTS = WARPS * LR, DP = PARTS * RPL;
+  constexpr int COLS = 32 / LR * CPL;
+  constexpr int kBase = 49 * DP;                           // stage offset of U0 | P U0
+  constexpr int kStage = kBase + 32 * COLS;
+  constexpr int NP = RPL / 2;                              // pairs of rows per lane
   extern __shared__ __align__(128) float smem[];
-  float* sx_all = smem + STAGES * kStage;                  // [warps][2][16][2 C]
+  float* part = smem + STAGES * kStage;                    // [PARTS][16][COLS] partial products of U, then of o
+  float* su = part + PARTS * 16 * COLS;                    // [16][COLS] U
   __shared__ uint64_t full[STAGES];
   const int slices = p.dvp / COLS;
   const int head = blockIdx.x / slices, slice = blockIdx.x % slices, b = blockIdx.y;
@@ -318,14 +392,13 @@ __global__ void __launch_bounds__(kWarps * 32) delta_scan_kernel(const DeltaPara
   const int first = p.chunk_base[b], chunks = (n + kTok - 1) / kTok;
   const int seq_len = p.seq_lens[b];
   const bool fresh = seq_len == n;                         // the portion starts at position 0
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int rg = lane & 15, cg = lane >> 4;
-  const int wcol = warp * 2 * C;                           // first column of the warp inside the block's slice
-  const int col0 = slice * COLS + wcol + cg * C;           // first of this lane's columns
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int range = warp * LR + lane / (32 / LR);          // this lane's rows: [range * RPL, ..)
+  const int lcol = lane % (32 / LR) * CPL;                 // first of this lane's columns inside the block
+  const int col0 = slice * COLS + lcol;
   float* S0 = p.pool + (static_cast<long>(slot) * p.H + head) * p.d * p.dv;
-  float* sx = sx_all + warp * 2 * 16 * 2 * C;
 
-  if (threadIdx.x == 0) {
+  if (tid == 0) {
     for (int s = 0; s < STAGES; ++s) fi::mbar_init(&full[s], 1);
     fi::mbar_fence_init();
   }
@@ -334,31 +407,30 @@ __global__ void __launch_bounds__(kWarps * 32) delta_scan_kernel(const DeltaPara
     const int s = i % STAGES;
     const float* w = p.work + (static_cast<long>(first + i) * p.H + head) * p.work_stride;
     fi::mbar_expect_tx(&full[s], kStage * 4);
-    bulk_load(smem + s * kStage, w, kOper * 4, &full[s]);
-    bulk_load(smem + s * kStage + kOper, w + kOper + slice * COLS * 16, COLS * 64, &full[s]);
+    bulk_load(smem + s * kStage, w, kBase * 4, &full[s]);
+    bulk_load(smem + s * kStage + kBase, w + kBase + slice * COLS * 32, COLS * 128, &full[s]);
   };
   int issued = 0;
-  if (threadIdx.x == 0)
+  if (tid == 0)
     for (; issued < min(STAGES, chunks); ++issued) request(issued);
 
   // the sequence's convolution inputs that the next portion needs
   {
     const int keep = min(n, p.taps - 1);
     const long per = static_cast<long>(p.C);
-    for (long i = static_cast<long>(blockIdx.x) * 256 + threadIdx.x; i < keep * per; i += static_cast<long>(gridDim.x) * 256) {
+    for (long i = static_cast<long>(blockIdx.x) * THREADS + tid; i < keep * per; i += static_cast<long>(gridDim.x) * THREADS) {
       const int back = static_cast<int>(i / per) + 1, ch = static_cast<int>(i % per);
       p.ring[(static_cast<long>(slot) * p.taps + (seq_len - back) % p.taps) * p.C + ch] =
           ld_any(p.qkv, (t_begin + n - back) * p.ld + ch, p.out_type);
     }
   }
 
-  // rows of this lane: 64 i4 + 4 rg + e, pairs (e = 0, 1) and (2, 3)
-  f2 S[R / 2][C];
+  f2 S[NP][CPL];
 #pragma unroll
-  for (int i = 0; i < R / 2; ++i) {
-    const int row = (i >> 1) * 64 + rg * 4 + (i & 1) * 2;
+  for (int i = 0; i < NP; ++i) {
+    const int row = range * RPL + 2 * i;
 #pragma unroll
-    for (int c = 0; c < C; ++c) {
+    for (int c = 0; c < CPL; ++c) {
       float a = 0.f, bb = 0.f;
       if (!fresh && col0 + c < p.dv) {
         if (row < p.d) a = S0[static_cast<long>(row) * p.dv + col0 + c];
@@ -367,6 +439,45 @@ __global__ void __launch_bounds__(kWarps * 32) delta_scan_kernel(const DeltaPara
       S[i][c] = pack2(a, bb);
     }
   }
+  // partial products of 16 operand rows with this lane's part of S
+  auto products = [&](const float* a) {
+    float* out = part + range * 16 * COLS + lcol;
+#pragma unroll 4
+    for (int row = 0; row < 16; ++row) {
+      f2 acc[CPL][2];
+#pragma unroll
+      for (int q = 0; q < NP; q += 2) {
+        const float4 v = *reinterpret_cast<const float4*>(a + row * DP + q * 2);
+        const f2 v0 = pack2(v.x, v.y), v1 = pack2(v.z, v.w);
+#pragma unroll
+        for (int c = 0; c < CPL; ++c) {
+          acc[c][0] = q == 0 ? mul2(v0, S[0][c]) : fma2(v0, S[q][c], acc[c][0]);
+          acc[c][1] = q == 0 ? mul2(v1, S[1][c]) : fma2(v1, S[q + 1][c], acc[c][1]);
+        }
+      }
+      float y[CPL];
+#pragma unroll
+      for (int c = 0; c < CPL; ++c) {
+        float x0, x1, x2, x3;
+        unpack2(acc[c][0], x0, x1);
+        unpack2(acc[c][1], x2, x3);
+        y[c] = (x0 + x1) + (x2 + x3);
+      }
+      if constexpr (CPL == 2) *reinterpret_cast<float2*>(out + row * COLS) = make_float2(y[0], y[CPL - 1]);
+      else out[row * COLS] = y[0];
+    }
+  };
+  // four columns of one row: the start value plus the row ranges' partial products
+  auto gather = [&](const float* base, int row, int c4) {
+    float4 y = *reinterpret_cast<const float4*>(base + (c4 >> 2) * 512 + row * 16 + (c4 & 3) * 4);
+#pragma unroll
+    for (int r = 0; r < PARTS; ++r) {
+      const float4 x = *reinterpret_cast<const float4*>(part + (r * 16 + row) * COLS + c4 * 4);
+      y.x += x.x; y.y += x.y; y.z += x.z; y.w += x.w;
+    }
+    return y;
+  };
+  constexpr int kGroups = COLS / 4;                        // groups of four columns per row
   bool ok = true;
   int waited = chunks;
   for (int i = 0; i < chunks; ++i) {
@@ -375,118 +486,77 @@ __global__ void __launch_bounds__(kWarps * 32) delta_scan_kernel(const DeltaPara
       fi::set_status(status, fi::kStatusTimeoutFull);
       ok = false;
     }
+    // the meeting also frees the stage and the partial sums of the chunk before (and tells everybody about a wait that
+    // ran out)
     if (__syncthreads_or(ok ? 0 : 1)) { ok = false; waited = i; break; }
+    if (STAGES > 1 && i > 0 && tid == 0 && issued < chunks) request(issued++);
     const float* st = smem + s * kStage;
-    const float* u0 = st + kOper;
-    // X = [W; E q] S
-#pragma unroll
-    for (int part = 0; part < 2; ++part) {
-#pragma unroll 1
-      for (int tq = 0; tq < 16; tq += TG) {
-        float v[16];                                       // [token][column]
-        const float* a = st + (part * 16 + tq) * DP + rg * 4;
-#pragma unroll
-        for (int u = 0; u < TG; ++u) {
-          f2 acc[C];
-#pragma unroll
-          for (int c = 0; c < C; ++c) acc[c] = pack2(0.f, 0.f);
-#pragma unroll
-          for (int i4 = 0; i4 < R / 4; ++i4) {
-            const float4 a4 = *reinterpret_cast<const float4*>(a + u * DP + i4 * 64);
-            const f2 a01 = pack2(a4.x, a4.y), a23 = pack2(a4.z, a4.w);
-#pragma unroll
-            for (int c = 0; c < C; ++c) acc[c] = fma2(a23, S[i4 * 2 + 1][c], fma2(a01, S[i4 * 2][c], acc[c]));
-          }
-#pragma unroll
-          for (int c = 0; c < C; ++c) {
-            float x, y;
-            unpack2(acc[c], x, y);
-            v[u * C + c] = x + y;
-          }
-        }
-#pragma unroll
-        for (int m = 8; m > 0; m >>= 1) {                  // row lane rg ends with the sum of value rg
-          const bool up = (rg & m) != 0;
-#pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            if (e < m) {
-              const float send = up ? v[e] : v[e + m];
-              const float keep = up ? v[e + m] : v[e];
-              v[e] = keep + __shfl_xor_sync(0xffffffffu, send, m);
-            }
-          }
-        }
-        sx[(part * 16 + tq + rg / C) * 2 * C + cg * C + rg % C] = v[0];
-      }
-    }
-    __syncwarp();
-    // U = U0 - X_W, in place
-#pragma unroll
-    for (int m = 0; m < C; ++m) {
-      const int e = m * 32 + lane, t = e / (2 * C), c = e % (2 * C), wc = wcol + c;
-      sx[e] = u0[(wc >> 4) * 256 + t * 16 + (wc & 15)] - sx[e];
-    }
-    __syncwarp();
+    const float* base = st + kBase;
+    products(st + range * RPL);                            // -W S
+    __syncthreads();
+    for (int g = tid; g < 16 * kGroups; g += THREADS)
+      *reinterpret_cast<float4*>(su + g * 4) = gather(base, g / kGroups, g % kGroups);
+    __syncthreads();
+    products(st + 16 * DP + range * RPL);                  // Q S
     // S <- E_16 S + sum_j (E_16 / E_j) k_j u_j^T
 #pragma unroll
-    for (int i4 = 0; i4 < R / 4; ++i4) {
-      const float4 e4 = *reinterpret_cast<const float4*>(st + 48 * DP + i4 * 64 + rg * 4);
-      const f2 e01 = pack2(e4.x, e4.y), e23 = pack2(e4.z, e4.w);
+    for (int q = 0; q < NP; q += 2) {
+      const float4 v = *reinterpret_cast<const float4*>(st + 48 * DP + range * RPL + q * 2);
+      const f2 v0 = pack2(v.x, v.y), v1 = pack2(v.z, v.w);
 #pragma unroll
-      for (int c = 0; c < C; ++c) {
-        S[i4 * 2][c] = mul2(e01, S[i4 * 2][c]);
-        S[i4 * 2 + 1][c] = mul2(e23, S[i4 * 2 + 1][c]);
+      for (int c = 0; c < CPL; ++c) {
+        S[q][c] = mul2(v0, S[q][c]);
+        S[q + 1][c] = mul2(v1, S[q + 1][c]);
       }
     }
 #pragma unroll 4
     for (int j = 0; j < 16; ++j) {
-      f2 uu[C];
+      f2 uu[CPL];
 #pragma unroll
-      for (int c = 0; c < C; ++c) {
-        const float x = sx[j * 2 * C + cg * C + c];
+      for (int c = 0; c < CPL; ++c) {
+        const float x = su[j * COLS + lcol + c];
         uu[c] = pack2(x, x);
       }
+      const float* k = st + (32 + j) * DP + range * RPL;
 #pragma unroll
-      for (int i4 = 0; i4 < R / 4; ++i4) {
-        const float4 k4 = *reinterpret_cast<const float4*>(st + (32 + j) * DP + i4 * 64 + rg * 4);
-        const f2 k01 = pack2(k4.x, k4.y), k23 = pack2(k4.z, k4.w);
+      for (int q = 0; q < NP; q += 2) {
+        const float4 v = *reinterpret_cast<const float4*>(k + q * 2);
+        const f2 v0 = pack2(v.x, v.y), v1 = pack2(v.z, v.w);
 #pragma unroll
-        for (int c = 0; c < C; ++c) {
-          S[i4 * 2][c] = fma2(k01, uu[c], S[i4 * 2][c]);
-          S[i4 * 2 + 1][c] = fma2(k23, uu[c], S[i4 * 2 + 1][c]);
+        for (int c = 0; c < CPL; ++c) {
+          S[q][c] = fma2(v0, uu[c], S[q][c]);
+          S[q + 1][c] = fma2(v1, uu[c], S[q + 1][c]);
         }
       }
     }
-    // o = X_q + P U
-    const float* P = st + 49 * DP;
-#pragma unroll
-    for (int m = 0; m < C; ++m) {
-      const int e = m * 32 + lane, t = e / (2 * C), c = e % (2 * C);
-      float o = sx[16 * 2 * C + e];
-#pragma unroll
-      for (int j4 = 0; j4 < 4; ++j4) {
-        const float4 p4 = *reinterpret_cast<const float4*>(P + t * 16 + j4 * 4);
-        o = fmaf(p4.x, sx[(j4 * 4) * 2 * C + c], o);
-        o = fmaf(p4.y, sx[(j4 * 4 + 1) * 2 * C + c], o);
-        o = fmaf(p4.z, sx[(j4 * 4 + 2) * 2 * C + c], o);
-        o = fmaf(p4.w, sx[(j4 * 4 + 3) * 2 * C + c], o);
+    __syncthreads();
+    for (int g = tid; g < 16 * kGroups; g += THREADS) {
+      const int row = g / kGroups, c4 = g % kGroups, tok = i * kTok + row, col = slice * COLS + c4 * 4;
+      if (tok >= n || col >= p.dv) continue;
+      const float4 y = gather(base + 256, row, c4);
+      float* dst = p.o + (static_cast<long>(t_begin + tok) * p.H + head) * p.dv + col;
+      if (p.vec_o) {
+        *reinterpret_cast<float4*>(dst) = y;
+      } else {
+        const float o[4] = {y.x, y.y, y.z, y.w};
+        for (int c = 0; c < 4 && col + c < p.dv; ++c) dst[c] = o[c];
       }
-      const int tok = i * kTok + t, col = slice * COLS + wcol + c;
-      if (tok < n && col < p.dv) p.o[(static_cast<long>(t_begin + tok) * p.H + head) * p.dv + col] = o;
     }
-    __syncthreads();                                       // the stage is free, and so are the warps' own patches
-    if (threadIdx.x == 0 && issued < chunks) request(issued++);
+    if constexpr (STAGES == 1) {                           // the only stage has to be read to the end first
+      __syncthreads();
+      if (tid == 0 && issued < chunks) request(issued++);
+    }
   }
   if (!ok) {                                               // uniform: leave once the copies in flight have landed
-    if (threadIdx.x == 0)
+    if (tid == 0)
       for (int i = waited; i < issued; ++i) fi::mbar_wait(&full[i % STAGES], (i / STAGES) & 1);
     return;
   }
 #pragma unroll
-  for (int i = 0; i < R / 2; ++i) {
-    const int row = (i >> 1) * 64 + rg * 4 + (i & 1) * 2;
+  for (int i = 0; i < NP; ++i) {
+    const int row = range * RPL + 2 * i;
 #pragma unroll
-    for (int c = 0; c < C; ++c) {
+    for (int c = 0; c < CPL; ++c) {
       float a, bb;
       unpack2(S[i][c], a, bb);
       if (col0 + c < p.dv) {
@@ -680,27 +750,38 @@ int check(const DeltaParams& p, int type) {
   return 0;
 }
 
-template <int R, int C>
+template <int DP, int LR, int CPL>
 int launch_scan(const DeltaParams& p, int* status, cudaStream_t s) {
-  constexpr int COLS = kWarps * 2 * C, STAGES = R <= 8 ? 3 : 2;
-  constexpr int smem = (STAGES * (49 * 16 * R + 256 + COLS * 16) + kWarps * 2 * 16 * 2 * C) * 4;
-  auto kern = delta_scan_kernel<R, C, STAGES>;
+  constexpr int WARPS = DP <= 256 ? 8 : 16, RPL = DP / (WARPS * LR), COLS = 32 / LR * CPL;
+  constexpr int STAGES = DP <= 256 ? 2 : 1;
+  constexpr int smem = (STAGES * (49 * DP + 32 * COLS) + WARPS * LR * 16 * COLS + 16 * COLS) * 4;
+  auto kern = delta_scan_kernel<RPL, LR, CPL, WARPS, STAGES>;
   cudaError_t e = fi::ensure_dynamic_smem(kern, smem);
   if (e != cudaSuccess) return static_cast<int>(e);
-  return static_cast<int>(fi::launch_kernel(kern, dim3(p.H * (p.dvp / COLS), p.B), dim3(kWarps * 32), smem, s, 0, p, status));
+  return static_cast<int>(fi::launch_kernel(kern, dim3(p.H * (p.dvp / COLS), p.B), dim3(WARPS * 32), smem, s, 0, p, status));
 }
 
-template <int R>
+template <int DP>
 int pick_cols(const DeltaParams& p, int* status, cudaStream_t s) {
-  // wide tiles spend the fewest instructions per element, narrow ones fill the device when there are few sequences
+  // wide tiles read every operand row the fewest times, narrow ones fill the device when there are few sequences
   const long ctas = static_cast<long>(p.B) * p.H * (p.dvp / 64);
-  if constexpr (R <= 8) {
-    if (ctas >= 192) return launch_scan<R, 4>(p, status, s);
+  if constexpr (DP <= 256) {
+    if (ctas >= 120) return launch_scan<DP, 1, 2>(p, status, s);
+    if (ctas >= 60) return launch_scan<DP, 1, 1>(p, status, s);
   }
-  if constexpr (R <= 16) {
-    if (ctas >= 120) return launch_scan<R, 2>(p, status, s);
-  }
-  return launch_scan<R, 1>(p, status, s);
+  return launch_scan<DP, 2, 1>(p, status, s);
+}
+
+template <typename T>
+cudaError_t launch_chunks(const DeltaParams& p, int smem, cudaStream_t s) {
+  auto go = [&](auto kern) {
+    const cudaError_t e = fi::ensure_dynamic_smem(kern, smem);
+    return e != cudaSuccess ? e : fi::launch_kernel(kern, dim3(p.n_chunks, p.H), dim3(256), smem, s, 0, p);
+  };
+  if (p.taps == 4) return go(delta_chunk_kernel<T, 4>);
+  if (p.taps == 3) return go(delta_chunk_kernel<T, 3>);
+  if (p.taps == 2) return go(delta_chunk_kernel<T, 2>);
+  return go(delta_chunk_kernel<T, 0>);
 }
 
 }  // namespace
@@ -735,25 +816,18 @@ extern "C" int fi_delta_portions(const void* qkv, long ld, const float* z, long 
   p.dvp = (dv + 63) / 64 * 64;
   p.work_stride = work_floats(p.dp, p.dvp);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  const long xs = static_cast<long>(kTok + taps - 1) * (2 * d + dv), kd = static_cast<long>(kTok) * d;
-  const long floats = (xs > kd ? xs : kd) + 3 * kd + static_cast<long>(kTok) * dv + 528;
+  p.vec_o = dv % 4 == 0 && (reinterpret_cast<uintptr_t>(o) & 15) == 0;
+  const long floats = static_cast<long>(kTok) * (5 * ((d + 3) & ~3) + dv) + 560;
   if (floats * 4 > 227 * 1024) return -11;
   const int smem = static_cast<int>(floats * 4);
-  cudaError_t e = cudaSuccess;
-#define FI_CHUNK(TT)                                                                                            \
-  {                                                                                                             \
-    e = fi::ensure_dynamic_smem(delta_chunk_kernel<TT>, smem);                                                  \
-    if (e == cudaSuccess) e = fi::launch_kernel(delta_chunk_kernel<TT>, dim3(n_chunks, H), dim3(256), smem, s, 0, p); \
-  }
-  if (type == 0) FI_CHUNK(__nv_bfloat16)
-  else if (type == 1) FI_CHUNK(__half)
-  else FI_CHUNK(float)
-#undef FI_CHUNK
+  const cudaError_t e = type == 0   ? launch_chunks<__nv_bfloat16>(p, smem, s)
+                        : type == 1 ? launch_chunks<__half>(p, smem, s)
+                                    : launch_chunks<float>(p, smem, s);
   if (e != cudaSuccess) return static_cast<int>(e);
-  if (p.dp == 64) return pick_cols<4>(p, status, s);
-  if (p.dp == 128) return pick_cols<8>(p, status, s);
-  if (p.dp == 256) return pick_cols<16>(p, status, s);
-  return pick_cols<32>(p, status, s);
+  if (p.dp == 64) return pick_cols<64>(p, status, s);
+  if (p.dp == 128) return pick_cols<128>(p, status, s);
+  if (p.dp == 256) return pick_cols<256>(p, status, s);
+  return pick_cols<512>(p, status, s);
 }
 
 // One token per sequence with head norm and output gate.  Operands as above; norm_w: fp32 [dv]; gate: rows of pitch ldg
