@@ -131,7 +131,7 @@ __host__ __device__ inline long work_floats(int dp, int dvp) { return 49l * dp +
 // TAPS: convolution length known at compile time (0: any).
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256, 3) delta_chunk_kernel(const DeltaParams p) {
-  fi::pdl_launch_dependents();
+  // no early launch of the scan: its few long-lived blocks would pile up on the multiprocessors that drain first
   fi::pdl_wait();
   extern __shared__ __align__(128) float smem[];
   const int chunk = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;

@@ -161,7 +161,7 @@ def pofadra_config(width: int, vocab: int, pattern: str, attn: tuple, delta: tup
             "embedding": {"scale": embed_scale}, "logit_softcap": softcap}
 
 
-PRESETS["tiny-pofadra-test"] = pofadra_config(160, 384, "ddaDA", (6, 2, 40, 24, 24), (4, 2, 24, 40, 3), (12, 2, 3, 2, 72))
+PRESETS["tiny-pofadra-test"] = pofadra_config(160, 512, "ddaDA", (6, 2, 40, 24, 24), (4, 2, 24, 40, 3), (12, 2, 3, 2, 72))
 # layers of the width and head geometry of a 1B-class decoder
 PRESETS["pofadra-1b"] = pofadra_config(2048, 32000, "ddad" * 3, (16, 4, 128, 64, 1024), (16, 16, 128, 128, 4), (32, 4, 4, 2, 768))
 

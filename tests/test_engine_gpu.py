@@ -98,7 +98,10 @@ def _prefill_logits(llm, prompts):
 @pytest.mark.parametrize("preset,min_cos", [("tiny-gemma4-moe-test", 0.96), ("tiny-llama-awq-test", 0.99),
                                              ("tiny-llama-ct-test", 0.99), ("tiny-deepseek-test", 0.97),
                                              ("tiny-qwen35-test", 0.97), ("tiny-qwen35-moe-test", 0.95), ("tiny-qwen2vl-test", 0.99), ("tiny-qwen3-test", 0.99),
-                                             ("tiny-fimodra-test", 0.99)])
+                                             ("tiny-fimodra-test", 0.99),
+                                             # (rounding the weights to 16 bits flips a near tie of a router in the
+                                             # first prompt's last token: 0.909 in exact arithmetic)
+                                             ("tiny-pofadra-test", 0.89)])
 def test_quantised_models_match_cpu_oracle(preset, min_cos):
     """int4 weights (+ fp8 KV, MoE routing for Gemma4): GPU kernels vs the CPU fp32 path on the same
     synthetic checkpoint."""
