@@ -331,6 +331,17 @@ int dispatch(int bn, const CUtensorMap& tw, const TokenMaps& tx, const GemmParam
   }
 }
 
+// Grouped products have many short tiles: shallower rings let several CTAs share an SM, so that one streams weights
+// while another sets up or stores.
+template <bool DUAL>
+int dispatch_grouped(int bn, const CUtensorMap& tw, const TokenMaps& tx, const GemmParams& p, cudaStream_t s) {
+  switch (bn) {
+    case 16: return launch<16, DUAL ? 3 : 4, DUAL>(tw, tx, p, s);
+    case 32: return launch<32, DUAL ? 3 : 4, DUAL>(tw, tx, p, s);
+    default: return launch<64, DUAL ? 3 : 4, DUAL>(tw, tx, p, s);
+  }
+}
+
 }  // namespace
 
 // Token-tile choice: the smallest tile that covers T up to 128; 128 for everything larger (two CTAs
@@ -441,6 +452,7 @@ static int fi_dense_gemm_impl(const void* X, const void* W, void* C, const void*
     if (comm->xfer_16bit == kXferTwoShot && (comm->mode != kCommAllReduce || out_fp32 || (ldc % 4) != 0)) return -24;
   }
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (grp != nullptr) return dual_rows > 0 ? dispatch_grouped<true>(bn, tw, tx, p, s) : dispatch_grouped<false>(bn, tw, tx, p, s);
   if (dual_rows > 0) return dispatch<true>(bn, tw, tx, p, s);
   return dispatch<false>(bn, tw, tx, p, s);
 }
@@ -492,11 +504,11 @@ extern "C" int fi_dense_gemm_dynw(const void* X, const void* W, void* C, const v
 }
 
 // Mixture-of-experts form: rows of X [n_rows, K], sorted by expert, meet the weights of their expert.  g: tile table for
-// tiles of `bn` rows (16, 32, 64 or 128), W [experts * g->expert_rows, K]; gated mode as above with an expert's rows
+// tiles of `bn` rows (16, 32 or 64), W [experts * g->expert_rows, K]; gated mode as above with an expert's rows
 // stored [gate; up].
 extern "C" int fi_dense_gemm_grouped(const void* X, const void* W, void* C, int n_rows, int N, int K, int ldx, int ldc,
                              int act, int dual_rows, int dtype, int bn, const FiGrouped* g, int* status, void* stream) {
-  if (g == nullptr || bn <= 0 || g->max_tiles > 65535) return -25;
+  if (g == nullptr || (bn != 16 && bn != 32 && bn != 64) || g->max_tiles > 65535) return -25;
   if (g->max_tiles <= 0) return 0;
   return fi_dense_gemm_impl(X, W, C, nullptr, nullptr, n_rows, N, K, ldx, K, ldc, act, dual_rows, 0, dtype, 1, bn, status,
                             stream, nullptr, 0.f, 0, nullptr, g);
