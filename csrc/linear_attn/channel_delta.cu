@@ -567,9 +567,9 @@ __global__ void __launch_bounds__(WARPS * 32) delta_scan_kernel(const DeltaParam
   }
 }
 
-// One token per sequence.  Block: one (head, sequence); thread: VEC columns of every RY-th row.  KEEP > 0: rows per
-// thread whose values stay in registers between the two passes over the state (d <= KEEP * RY); 0: read twice.
-template <int VEC, int KEEP, typename T>
+// One token per sequence.  Block: one (head, sequence); thread: VEC columns of every RY-th row.  STAGED: the state waits in
+// shared memory between the two passes over it (every thread copies, and reads back, its own part); else it is read twice.
+template <int VEC, bool STAGED, typename T>
 __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -588,8 +588,16 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaParams p) {
   const int cx = tid % nx, ry = tid / nx;
   const bool fresh = len == 1;
   float* S = p.pool + (static_cast<long>(slot) * p.H + head) * d * dv;
+  const float* old = STAGED ? smem : S;
+  if constexpr (STAGED) {                                  // in flight while the operands are prepared
+    if (!fresh && ry < ry_n)
+      for (int r = ry; r < d; r += ry_n)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(fi::smem_u32(smem + r * dv + cx * VEC)),
+                     "l"(S + static_cast<long>(r) * dv + cx * VEC)
+                     : "memory");
+  }
   auto fetch = [&](int r, float* s) {
-    const float* row = S + static_cast<long>(r) * dv + cx * VEC;
+    const float* row = old + static_cast<long>(r) * dv + cx * VEC;
     if constexpr (VEC == 4) {
       const float4 x = *reinterpret_cast<const float4*>(row);
       s[0] = x.x; s[1] = x.y; s[2] = x.z; s[3] = x.w;
@@ -597,17 +605,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaParams p) {
       s[0] = row[0];
     }
   };
-  float keep[KEEP > 0 ? KEEP : 1][VEC];
-  if constexpr (KEEP > 0) {                                // in flight while the operands are prepared
-#pragma unroll
-    for (int i = 0; i < KEEP; ++i) {
-      const int r = ry + i * ry_n;
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) keep[i][e] = 0.f;
-      if (!fresh && ry < ry_n && r < d) fetch(r, keep[i]);
-    }
-  }
-  float* sq = smem;                 // [d]
+  float* sq = smem + (STAGED ? static_cast<long>(d) * dv : 0);   // [d]
   float* sk = sq + d;               // [d]
   float* sg = sk + d;               // [d]
   float* sv = sg + d;               // [dv]
@@ -648,17 +646,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaParams p) {
 #pragma unroll
   for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
   if (ry < ry_n) {
-    if constexpr (KEEP > 0) {
-#pragma unroll
-      for (int i = 0; i < KEEP; ++i) {
-        const int r = ry + i * ry_n;
-        if (r < d) {
-          const float g = sg[r], k = sk[r];
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) { keep[i][e] *= g; acc[e] = fmaf(k, keep[i][e], acc[e]); }
-        }
-      }
-    } else if (!fresh) {
+    if (!fresh) {
+      if constexpr (STAGED) asm volatile("cp.async.wait_all;" ::: "memory");
 #pragma unroll 4
       for (int r = ry; r < d; r += ry_n) {
         float s[VEC];
@@ -688,34 +677,21 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaParams p) {
   __syncthreads();
   // second pass: the write, the read-out and the new state
   if (ry < ry_n) {
-    auto finish = [&](int r, float* s) {
-      const float k = fk * sk[r], q = sq[r];
+#pragma unroll 4
+    for (int r = ry; r < d; r += ry_n) {
+      float s[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s[e] = 0.f;
+      if (!fresh) fetch(r, s);
+      const float k = fk * sk[r], q = sq[r], g = sg[r];
       float* row = S + static_cast<long>(r) * dv + cx * VEC;
 #pragma unroll
       for (int e = 0; e < VEC; ++e) {
-        s[e] = fmaf(k, u[e], s[e]);
+        s[e] = fmaf(k, u[e], g * s[e]);
         o[e] = fmaf(q, s[e], o[e]);
       }
       if constexpr (VEC == 4) *reinterpret_cast<float4*>(row) = make_float4(s[0], s[1], s[2], s[3]);
       else row[0] = s[0];
-    };
-    if constexpr (KEEP > 0) {
-#pragma unroll
-      for (int i = 0; i < KEEP; ++i) {
-        const int r = ry + i * ry_n;
-        if (r < d) finish(r, keep[i]);
-      }
-    } else {
-#pragma unroll 4
-      for (int r = ry; r < d; r += ry_n) {
-        float s[VEC];
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) s[e] = 0.f;
-        if (!fresh) fetch(r, s);
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) s[e] *= sg[r];
-        finish(r, s);
-      }
     }
 #pragma unroll
     for (int e = 0; e < VEC; ++e) so[ry * dv + cx * VEC + e] = o[e];
@@ -851,23 +827,26 @@ extern "C" int fi_delta_step(const void* qkv, long ld, const float* z, long ldz,
   const int nx = vec4 ? dv / 4 : dv;
   if (nx > 256) return -11;
   const int ry = 256 / nx;
-  const long floats = 3l * d + dv + static_cast<long>(ry) * dv;
-  if (floats * 4 > 48 * 1024) return -11;
-  const int smem = static_cast<int>(floats * 4);
-  const int rows = (d + ry - 1) / ry;                      // per thread
+  const long small = (3l * d + dv + static_cast<long>(ry) * dv) * 4, tile = static_cast<long>(d) * dv * 4;
+  if (small > 100 * 1024) return -11;
+  const bool staged = vec4 && small + tile <= 200 * 1024;
+  const int smem = static_cast<int>(staged ? small + tile : small);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-#define FI_STEP(V, K, TT) return static_cast<int>(fi::launch_kernel(delta_step_kernel<V, K, TT>, dim3(H, B), dim3(256), smem, s, 0, p))
-#define FI_STEP_T(V, K)                     \
-  {                                         \
-    if (type == 0) FI_STEP(V, K, __nv_bfloat16); \
-    if (type == 1) FI_STEP(V, K, __half);   \
-    FI_STEP(V, K, float);                   \
+#define FI_STEP(V, K, TT)                                                                                    \
+  {                                                                                                          \
+    const cudaError_t e = fi::ensure_dynamic_smem(delta_step_kernel<V, K, TT>, smem);                        \
+    if (e != cudaSuccess) return static_cast<int>(e);                                                        \
+    return static_cast<int>(fi::launch_kernel(delta_step_kernel<V, K, TT>, dim3(H, B), dim3(256), smem, s, 0, p)); \
   }
-  if (!vec4) FI_STEP_T(1, 0)
-  if (rows <= 4) FI_STEP_T(4, 4)
-  if (rows <= 8) FI_STEP_T(4, 8)
-  if (rows <= 16) FI_STEP_T(4, 16)
-  FI_STEP_T(4, 0)
+#define FI_STEP_T(V, K)                          \
+  {                                              \
+    if (type == 0) FI_STEP(V, K, __nv_bfloat16)  \
+    if (type == 1) FI_STEP(V, K, __half)         \
+    FI_STEP(V, K, float)                         \
+  }
+  if (!vec4) FI_STEP_T(1, false)
+  if (!staged) FI_STEP_T(4, false)
+  FI_STEP_T(4, true)
 #undef FI_STEP_T
 #undef FI_STEP
 }
