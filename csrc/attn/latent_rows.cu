@@ -18,6 +18,7 @@
 #include <stdint.h>
 
 #include "../common/launch.cuh"
+#include "attn_extra.h"
 
 namespace {
 
@@ -261,33 +262,32 @@ __global__ void __launch_bounds__(256) latent_pool_kernel(const T* __restrict__ 
 }
 
 struct RowsParams {
-  const void* q_cat;        // [rows, nh, kd]
+  const void* q_cat;        // [rows, nh, kd / maps]
   const void* cache;        // [blocks, nkv, block size] rows of kd values
   const void* v_cache;      // the same with rows of vd values; null: the first vd values of a cache row are the value
-  const void* gate;         // [rows, >= nh * vd] of pitch gate_stride or null: out *= sigmoid(gate)
-  long gate_stride;
   int nkv;
-  void* out;                // element (row r, head h, d) at out + h * out_head_stride + r * out_row_stride + d
+  void* out;                // element (row r, output head h, d) at out + h * out_head_stride + r * out_row_stride + d
   long out_head_stride, out_row_stride;
   const int* block_tables;
   const int* row_lens;
   const int* seq_of_row;    // or null
-  const float* sinks;       // or null
   int rows, nh, kd, vd, max_blocks, block_size, window, num_rows;
   float sm_scale;
+  FiAttnExtra x;            // sinks, output gate, two maps per head (the key row of a head is [map 1 | map 2])
 };
 
-template <typename T, int NV>
+template <typename T, int NV, int MAPS>
 __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   extern __shared__ float smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long item = static_cast<long>(blockIdx.x) * 4 + warp;
-  if (item >= static_cast<long>(p.rows) * p.nh) return;
-  const int r = static_cast<int>(item / p.nh), h = static_cast<int>(item % p.nh);
+  const int heads = p.nh / MAPS, qd = p.kd / MAPS;
+  if (item >= static_cast<long>(p.rows) * heads) return;
+  const int r = static_cast<int>(item / heads), h = static_cast<int>(item % heads);
   float* q = smem + warp * p.kd;
-  const T* qs = reinterpret_cast<const T*>(p.q_cat) + item * p.kd;
+  const T* qs = reinterpret_cast<const T*>(p.q_cat) + item * p.kd;      // a head's maps follow one another
   for (int i = lane; i < p.kd; i += 32) q[i] = to_f(qs[i]) * p.sm_scale;
   __syncwarp();
   const int len = min(p.row_lens[r], p.max_blocks * p.block_size);
@@ -295,65 +295,92 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
   const int* bt = p.block_tables + static_cast<long>(p.seq_of_row ? p.seq_of_row[r] : r) * p.max_blocks;
   const T* cache = reinterpret_cast<const T*>(p.cache);
   const T* values = reinterpret_cast<const T*>(p.v_cache != nullptr ? p.v_cache : p.cache);
-  const int vpitch = p.v_cache != nullptr ? p.vd : p.kd, kvh = h / (p.nh / p.nkv);
+  const int vpitch = p.v_cache != nullptr ? p.vd : p.kd, kvh = h / (heads / p.nkv);
+  float first[MAPS == 2 ? NV : 1];       // the first map's output
   float o[NV];
+  for (int map = 0; map < MAPS; ++map) {
 #pragma unroll
-  for (int i = 0; i < NV; ++i) o[i] = 0.f;
-  float m = -CUDART_INF_F, l = 0.f;
-  for (int k0 = lo; k0 < len; k0 += 32) {
-    const int tok = k0 + lane;
-    long src = 0;
-    float s = -CUDART_INF_F;
-    if (tok < len) {
-      long blk = bt[tok / p.block_size];
-      blk = blk < 0 || (blk + 1) * p.block_size > p.num_rows ? 0 : blk;
-      src = (blk * p.nkv + kvh) * p.block_size + tok % p.block_size;
-      const T* row = cache + src * p.kd;
-      float a0 = 0.f, a1 = 0.f;
-      int i = 0;
-      for (; i + 1 < p.kd; i += 2) { a0 = fmaf(q[i], to_f(row[i]), a0); a1 = fmaf(q[i + 1], to_f(row[i + 1]), a1); }
-      if (i < p.kd) a0 = fmaf(q[i], to_f(row[i]), a0);
-      s = a0 + a1;
+    for (int i = 0; i < NV; ++i) o[i] = 0.f;
+    float m = -CUDART_INF_F, l = 0.f;
+    for (int k0 = lo; k0 < len; k0 += 32) {
+      const int tok = k0 + lane;
+      long src = 0;
+      float s = -CUDART_INF_F;
+      if (tok < len) {
+        long blk = bt[tok / p.block_size];
+        blk = blk < 0 || (blk + 1) * p.block_size > p.num_rows ? 0 : blk;
+        src = (blk * p.nkv + kvh) * p.block_size + tok % p.block_size;
+        const T* row = cache + src * p.kd + map * qd;
+        const float* qm = q + map * qd;
+        float a0 = 0.f, a1 = 0.f;
+        int i = 0;
+        for (; i + 1 < qd; i += 2) { a0 = fmaf(qm[i], to_f(row[i]), a0); a1 = fmaf(qm[i + 1], to_f(row[i + 1]), a1); }
+        if (i < qd) a0 = fmaf(qm[i], to_f(row[i]), a0);
+        s = a0 + a1;
+      }
+      float mx = s;
+      for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+      const float nm = fmaxf(m, mx);            // at least one key of the chunk is visible
+      const float alpha = __expf(m - nm);
+      const float pv = __expf(s - nm);
+      float rs = pv;
+      for (int x = 16; x > 0; x >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, x);
+      l = l * alpha + rs;
+      m = nm;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) o[i] *= alpha;
+      const int n = min(32, len - k0);
+      for (int j = 0; j < n; ++j) {
+        const float pj = __shfl_sync(0xffffffffu, pv, j);
+        const T* row = values + __shfl_sync(0xffffffffu, src, j) * vpitch;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (i * 32 + lane < p.vd) o[i] = fmaf(pj, to_f(row[i * 32 + lane]), o[i]);
+      }
     }
-    float mx = s;
-    for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-    const float nm = fmaxf(m, mx);            // at least one key of the chunk is visible
-    const float alpha = __expf(m - nm);
-    const float pv = __expf(s - nm);
-    float rs = pv;
-    for (int x = 16; x > 0; x >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, x);
-    l = l * alpha + rs;
-    m = nm;
+    if (p.x.sinks != nullptr && m != -CUDART_INF_F) l += __expf(p.x.sinks[h * MAPS + map] - m);
+    const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i) o[i] *= alpha;
-    const int n = min(32, len - k0);
-    for (int j = 0; j < n; ++j) {
-      const float pj = __shfl_sync(0xffffffffu, pv, j);
-      const T* row = values + __shfl_sync(0xffffffffu, src, j) * vpitch;
-#pragma unroll
-      for (int i = 0; i < NV; ++i)
-        if (i * 32 + lane < p.vd) o[i] = fmaf(pj, to_f(row[i * 32 + lane]), o[i]);
+    for (int i = 0; i < NV; ++i) {
+      o[i] *= inv;
+      if constexpr (MAPS == 2) {
+        if (map == 0) first[i] = o[i];
+      }
     }
   }
-  if (p.sinks != nullptr && m != -CUDART_INF_F) l += __expf(p.sinks[h] - m);
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  if constexpr (MAPS == 2) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      o[i] = first[i] - p.x.lambda * o[i];       // channels from vd on are zero
+      ss = fmaf(o[i], o[i], ss);
+    }
+    for (int x = 16; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float f = p.x.out_scale / sqrtf(ss / static_cast<float>(p.vd) + p.x.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) o[i] *= f;
+  }
   T* out = reinterpret_cast<T*>(p.out) + h * p.out_head_stride + r * p.out_row_stride;
 #pragma unroll
   for (int i = 0; i < NV; ++i)
     if (i * 32 + lane < p.vd) {
-      float v = o[i] * inv;
-      if (p.gate != nullptr)
-        v /= 1.f + __expf(-to_f(reinterpret_cast<const T*>(p.gate)[r * p.gate_stride + h * p.vd + i * 32 + lane]));
+      float v = o[i];
+      if (p.x.gate != nullptr) {
+        const long at = r * p.x.gate_stride + (p.x.gate_per_head ? h : h * p.vd + i * 32 + lane);
+        v /= 1.f + __expf(-to_f(reinterpret_cast<const T*>(p.x.gate)[at]));
+      }
       out[i * 32 + lane] = from_f<T>(v);
     }
 }
 
 template <typename T>
 int launch_rows(const RowsParams& p, cudaStream_t s) {
-  const long items = static_cast<long>(p.rows) * p.nh;
+  const long items = static_cast<long>(p.rows) * (p.nh / p.x.maps);
   const dim3 grid(static_cast<unsigned>((items + 3) / 4));
   const int smem = 4 * p.kd * 4;
-#define FI_ROWS(N) return static_cast<int>(fi::launch_kernel(latent_rows_kernel<T, N>, grid, dim3(128), smem, s, 0, p))
+#define FI_ROWS(N)                                                                                                         \
+  return static_cast<int>(p.x.maps == 2 ? fi::launch_kernel(latent_rows_kernel<T, N, 2>, grid, dim3(128), smem, s, 0, p)   \
+                                        : fi::launch_kernel(latent_rows_kernel<T, N, 1>, grid, dim3(128), smem, s, 0, p))
   if (p.vd <= 64) FI_ROWS(2);
   if (p.vd <= 128) FI_ROWS(4);
   if (p.vd <= 256) FI_ROWS(8);
@@ -450,9 +477,9 @@ extern "C" int fi_latent_rows(const void* q_cat, const void* cache, void* out, l
     return -10;
   RowsParams p = {};
   p.q_cat = q_cat; p.cache = cache; p.out = out; p.out_head_stride = out_head_stride; p.out_row_stride = out_row_stride;
-  p.block_tables = block_tables; p.row_lens = row_lens; p.seq_of_row = seq_of_row; p.sinks = sinks; p.rows = rows;
+  p.block_tables = block_tables; p.row_lens = row_lens; p.seq_of_row = seq_of_row; p.rows = rows;
   p.nh = nh; p.kd = kd; p.vd = vd; p.max_blocks = max_blocks; p.block_size = block_size; p.num_rows = num_rows;
-  p.window = window; p.sm_scale = sm_scale; p.nkv = 1;
+  p.window = window; p.sm_scale = sm_scale; p.nkv = 1; p.x.maps = 1; p.x.sinks = sinks;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_CALL(TT) return launch_rows<TT>(p, s)
   FI_BY_TYPE(dtype, FI_CALL)
@@ -462,21 +489,23 @@ extern "C" int fi_latent_rows(const void* q_cat, const void* cache, void* out, l
 
 // The same over separate key and value caches [blocks, nkv, block_size, kd | vd] (query head h reads key / value head
 // h / (nh / nkv)): q [rows, nh, kd], out [rows, nh * vd]; row r sees the first row_lens[r] tokens (the last `window` of
-// them) of sequence seq_of_row[r] (null: sequence r); gate: rows of pitch gate_stride in the type of out, or null.
+// them) of sequence seq_of_row[r] (null: sequence r).  extra: see attn_extra.h, or null.  Two maps per head: q [rows, nh,
+// kd / 2] with query heads 2 j and 2 j + 1 for output head j, key rows [map 1 | map 2], out [rows, nh / 2 * vd].
 extern "C" int fi_attn_rows(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_tables,
                             const int* row_lens, const int* seq_of_row, int rows, int nh, int nkv, int kd, int vd,
-                            int max_blocks, int block_size, int num_blocks, int window, const float* sinks,
-                            const void* gate, long gate_stride, float sm_scale, int dtype, void* stream) {
+                            int max_blocks, int block_size, int num_blocks, int window, const FiAttnExtra* extra,
+                            float sm_scale, int dtype, void* stream) {
   if (rows <= 0 || nh <= 0) return 0;
   if (kd <= 0 || vd <= 0 || vd > 1024 || kd > 2048 || block_size <= 0 || max_blocks <= 0 || num_blocks <= 0 || nkv <= 0 ||
       nh % nkv != 0 || v_cache == nullptr)
     return -10;
   RowsParams p = {};
+  if (!fi::take_extra(p, extra, vd, nh, nkv) || p.x.out_dim != vd || kd % p.x.maps != 0) return -10;
   p.q_cat = q; p.cache = k_cache; p.v_cache = v_cache; p.out = out; p.out_head_stride = vd;
-  p.out_row_stride = static_cast<long>(nh) * vd; p.block_tables = block_tables; p.row_lens = row_lens;
-  p.seq_of_row = seq_of_row; p.sinks = sinks; p.rows = rows; p.nh = nh; p.nkv = nkv; p.kd = kd; p.vd = vd;
+  p.out_row_stride = static_cast<long>(nh / p.x.maps) * vd; p.block_tables = block_tables; p.row_lens = row_lens;
+  p.seq_of_row = seq_of_row; p.rows = rows; p.nh = nh; p.nkv = nkv; p.kd = kd; p.vd = vd;
   p.max_blocks = max_blocks; p.block_size = block_size; p.num_rows = num_blocks * block_size; p.window = window;
-  p.sm_scale = sm_scale; p.gate = gate; p.gate_stride = gate_stride;
+  p.sm_scale = sm_scale;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_CALL(TT) return launch_rows<TT>(p, s)
   FI_BY_TYPE(dtype, FI_CALL)

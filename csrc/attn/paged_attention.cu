@@ -17,6 +17,7 @@
 #include <cuda_runtime.h>
 
 #include "../common/launch.cuh"
+#include "attn_extra.h"
 #include "paged_attention_noalloc.h"
 #include <atomic>
 #include <cooperative_groups.h>
@@ -92,7 +93,7 @@ struct AttnParams {
   long q_stride;
   const void* k_cache;
   const void* v_cache;
-  void* out;            // [T, nh * HD]
+  void* out;            // [T, nh * out_dim] (two maps: [T, nh / 2 * out_dim])
   const int* block_tables;  // [B, max_blocks]
   const int* seq_lens;      // [B] KV length including this step's tokens
   const int* cu_q;          // [B + 1] query token offsets (prefill); null for decode
@@ -114,27 +115,53 @@ struct AttnParams {
   // partials through distributed shared memory at this byte offset of the dynamic shared memory
   // ([16][HD] sums + [16][2] max/denominator per CTA): no global scratch, no tickets, no second launch
   int cluster_off;
-  // fp32 [nh] or null, one extra exp(sink) per head in the softmax denominator; channels of a head that are stored
-  // (0 = HD; rows of nh * out_dim); output gate: row t at gate + t * gate_stride (same type as out, channels as in
-  // out) or null, out is multiplied by sigmoid(gate)
-  const float* sinks;
-  int out_dim;
-  const void* gate;
-  long gate_stride;
+  FiAttnExtra x;        // sinks, output gate, stored channels, two maps per head
 };
 
 // Scatter of one finished channel: sum of exponentials l, reference m, accumulated value acc.
 template <typename T, int HD>
 __device__ __forceinline__ void store_decoded(const AttnParams& p, int b, int head, int d, float acc, float l, float m) {
-  const int od = p.out_dim > 0 ? p.out_dim : HD;
+  const int od = p.x.out_dim;
   if (d >= od) return;
-  if (p.sinks != nullptr && m != -CUDART_INF_F) l += exp2f((p.sinks[head] - m) * kLog2e);
+  if (p.x.sinks != nullptr && m != -CUDART_INF_F) l += exp2f((p.x.sinks[head] - m) * kLog2e);
   float v = l > 0.f ? acc / l * (p.kv_fp8 == 1 ? p.v_scale : 1.f) : 0.f;
-  if (p.gate != nullptr) {
-    const float g = static_cast<float>(reinterpret_cast<const T*>(p.gate)[b * p.gate_stride + head * od + d]);
-    v /= 1.f + __expf(-g);
+  if (p.x.gate != nullptr) {
+    const long at = b * p.x.gate_stride + (p.x.gate_per_head ? head : head * od + d);
+    v /= 1.f + __expf(-static_cast<float>(reinterpret_cast<const T*>(p.x.gate)[at]));
   }
   reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * od + d] = MmaT<T>::from_f(v);
+}
+
+// Two maps per head: one warp finishes query heads head and head + 1 (rows r and r + 1 of its tile).  get(row, channel,
+// acc, l, m) gives the accumulated value of a channel, the sum of exponentials and their reference.
+template <typename T, int HD, typename F>
+__device__ __forceinline__ void store_map_pair(const AttnParams& p, int b, int head, int r, F get) {
+  const int lane = threadIdx.x & 31, od = p.x.out_dim;
+  const float vs = p.kv_fp8 == 1 ? p.v_scale : 1.f;
+  float v[HD / 32], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < HD / 32; ++i) {
+    const int d = i * 32 + lane;
+    v[i] = 0.f;
+    if (d < od) {
+      float a[2];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        float acc, l, m;
+        get(r + k, d, acc, l, m);
+        if (p.x.sinks != nullptr && m != -CUDART_INF_F) l += exp2f((p.x.sinks[head + k] - m) * kLog2e);
+        a[k] = l > 0.f ? acc / l * vs : 0.f;
+      }
+      v[i] = a[0] - p.x.lambda * a[1];
+      ss = fmaf(v[i], v[i], ss);
+    }
+  }
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float f = p.x.out_scale / sqrtf(ss / static_cast<float>(od) + p.x.eps);
+  T* out = reinterpret_cast<T*>(p.out) + (static_cast<long>(b) * (p.nh / 2) + head / 2) * od;
+#pragma unroll
+  for (int i = 0; i < HD / 32; ++i)
+    if (i * 32 + lane < od) out[i * 32 + lane] = MmaT<T>::from_f(v[i] * f);
 }
 
 // Load `rows` KV tokens starting at token tok0 of sequence b / kv head kvh into a swizzled tile.
@@ -359,12 +386,12 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
-    const int r = i / HD, d = i % HD;
-    float m = -CUDART_INF_F;
+  auto merged = [&](int r, int d, float& acc, float& l, float& m) {     // the four warps' shares of one channel
+    m = -CUDART_INF_F;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, mML[(w * 16 + r) * 2]);
-    float acc = 0.f, l = 0.f;
+    acc = 0.f;
+    l = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float mw = mML[(w * 16 + r) * 2];
@@ -372,6 +399,15 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
       acc += f * mO[(w * 16 + r) * HD + d];
       l += f * mML[(w * 16 + r) * 2 + 1];
     }
+  };
+  if (p.splits == 1 && p.x.maps == 2) {
+    for (int r = 2 * warp; r < heads_here; r += 8) store_map_pair<T, HD>(p, b, head0 + r, r, merged);
+    return;
+  }
+  for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
+    const int r = i / HD, d = i % HD;
+    float acc, l, m;
+    merged(r, d, acc, l, m);
     const int head = head0 + r;
     if (p.splits == 1) {
       store_decoded<T, HD>(p, b, head, d, acc, l, m);
@@ -586,12 +622,12 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
-    const int r = i / HD, d = i % HD;
-    float m = -CUDART_INF_F;
+  auto merged = [&](int r, int d, float& acc, float& l, float& m) {     // the four warps' shares of one channel
+    m = -CUDART_INF_F;
 #pragma unroll
     for (int w = 0; w < 4; ++w) m = fmaxf(m, mML[(w * 16 + r) * 2]);
-    float acc = 0.f, l = 0.f;
+    acc = 0.f;
+    l = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float mw = mML[(w * 16 + r) * 2];
@@ -599,6 +635,15 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
       acc += f * mO[(w * 16 + r) * HD + d];
       l += f * mML[(w * 16 + r) * 2 + 1];
     }
+  };
+  if (p.splits == 1 && p.x.maps == 2) {
+    for (int r = 2 * warp; r < heads_here; r += 8) store_map_pair<T, HD>(p, b, head0 + r, r, merged);
+    return;
+  }
+  for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
+    const int r = i / HD, d = i % HD;
+    float acc, l, m;
+    merged(r, d, acc, l, m);
     const int head = head0 + r;
     if (p.splits == 1) {
       store_decoded<T, HD>(p, b, head, d, acc, l, m);
@@ -619,12 +664,9 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
     cg::cluster_group cluster = cg::this_cluster();
     cluster.sync();
     float* cO = reinterpret_cast<float*>(smem_raw + p.cluster_off);
-    const int E = heads_here * HD;
-    const int per = (E + p.splits - 1) / p.splits;
-    const int i_end = min(E, (split + 1) * per);
-    for (int i = split * per + threadIdx.x; i < i_end; i += 128) {
-      const int r = i / HD;
-      float ms[8], m = -CUDART_INF_F;
+    auto gathered = [&](int r, int d, float& acc, float& l, float& m) {
+      float ms[8];
+      m = -CUDART_INF_F;
 #pragma unroll
       for (int sidx = 0; sidx < 8; ++sidx) {
         if (sidx < p.splits) {
@@ -632,17 +674,30 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
           m = fmaxf(m, ms[sidx]);
         }
       }
-      float acc = 0.f, l = 0.f;
+      acc = 0.f;
+      l = 0.f;
 #pragma unroll
       for (int sidx = 0; sidx < 8; ++sidx) {
         if (sidx < p.splits) {
           const float* peer = cluster.map_shared_rank(cO, sidx);
           const float f = ms[sidx] == -CUDART_INF_F ? 0.f : exp2f((ms[sidx] - m) * kLog2e);
-          acc += f * peer[i];
+          acc += f * peer[r * HD + d];
           l += f * peer[16 * HD + r * 2 + 1];
         }
       }
-      store_decoded<T, HD>(p, b, head0 + r, i % HD, acc, l, m);
+    };
+    if (p.x.maps == 2) {
+      for (int r = 2 * (split * 4 + warp); r < heads_here; r += 8 * p.splits)
+        store_map_pair<T, HD>(p, b, head0 + r, r, gathered);
+    } else {
+      const int E = heads_here * HD;
+      const int per = (E + p.splits - 1) / p.splits;
+      const int i_end = min(E, (split + 1) * per);
+      for (int i = split * per + threadIdx.x; i < i_end; i += 128) {
+        float acc, l, m;
+        gathered(i / HD, i % HD, acc, l, m);
+        store_decoded<T, HD>(p, b, head0 + i / HD, i % HD, acc, l, m);
+      }
     }
     cluster.sync();
   } else if (p.splits > 1 && p.merge_tickets != nullptr) {
@@ -660,19 +715,27 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
     __syncthreads();
     if (is_last) {
       __threadfence();
-      for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
-        const int r = i / HD, d = i % HD;
+      auto gathered = [&](int r, int d, float& acc, float& l, float& m) {
         const long base = (static_cast<long>(b) * p.nh + head0 + r) * p.splits;
-        float m = -CUDART_INF_F;
+        m = -CUDART_INF_F;
         for (int sidx = 0; sidx < p.splits; ++sidx) m = fmaxf(m, __ldcg(p.ws_ml + (base + sidx) * 2));
-        float acc = 0.f, l = 0.f;
+        acc = 0.f;
+        l = 0.f;
         for (int sidx = 0; sidx < p.splits; ++sidx) {
           const float ms = __ldcg(p.ws_ml + (base + sidx) * 2);
           const float f = ms == -CUDART_INF_F ? 0.f : exp2f((ms - m) * kLog2e);
           acc += f * __ldcg(p.ws_o + (base + sidx) * HD + d);
           l += f * __ldcg(p.ws_ml + (base + sidx) * 2 + 1);
         }
-        store_decoded<T, HD>(p, b, head0 + r, d, acc, l, m);
+      };
+      if (p.x.maps == 2) {
+        for (int r = 2 * warp; r < heads_here; r += 8) store_map_pair<T, HD>(p, b, head0 + r, r, gathered);
+        return;
+      }
+      for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
+        float acc, l, m;
+        gathered(i / HD, i % HD, acc, l, m);
+        store_decoded<T, HD>(p, b, head0 + i / HD, i % HD, acc, l, m);
       }
     }
   }
@@ -682,26 +745,36 @@ template <typename T, int HD>
 __global__ void decode_merge_kernel(const AttnParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
-  const int b = blockIdx.y, head = blockIdx.x;
-  const long base = (static_cast<long>(b) * p.nh + head) * p.splits;
-  float m = -CUDART_INF_F;
-  for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.ws_ml[(base + s) * 2]);
-  for (int d = threadIdx.x; d < HD; d += blockDim.x) {
-    float acc = 0.f, l = 0.f;
+  const int b = blockIdx.y, head = blockIdx.x * p.x.maps;
+  auto gathered = [&](int r, int d, float& acc, float& l, float& m) {
+    const long base = (static_cast<long>(b) * p.nh + head + r) * p.splits;
+    m = -CUDART_INF_F;
+    for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.ws_ml[(base + s) * 2]);
+    acc = 0.f;
+    l = 0.f;
     for (int s = 0; s < p.splits; ++s) {
       const float ms = p.ws_ml[(base + s) * 2];
       const float f = ms == -CUDART_INF_F ? 0.f : exp2f((ms - m) * kLog2e);
       acc += f * p.ws_o[(base + s) * HD + d];
       l += f * p.ws_ml[(base + s) * 2 + 1];
     }
+  };
+  if (p.x.maps == 2) {
+    if (threadIdx.x < 32) store_map_pair<T, HD>(p, b, head, 0, gathered);
+    return;
+  }
+  for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+    float acc, l, m;
+    gathered(0, d, acc, l, m);
     store_decoded<T, HD>(p, b, head, d, acc, l, m);
   }
 }
 
 // ------------------------------------------------------------------------------ prefill
-// grid (q_tiles, nh, B); 128 threads; each warp owns 16 consecutive query tokens of the 64-token
-// tile; KV streamed in CH-token chunks shared by the four warps.
-template <typename T, int HD, int CH>
+// grid (q_tiles, nh / MAPS, B); 128 threads; each warp owns 16 consecutive rows of the 64-row tile (a
+// row is a query token, or one of the MAPS = 2 maps of a token, side by side); KV streamed in CH-token
+// chunks shared by the four warps.
+template <typename T, int HD, int CH, int MAPS>
 __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -709,9 +782,10 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   T* sQ = reinterpret_cast<T*>(smem_raw);   // [64][HD]
   T* sK = sQ + 64 * HD;                     // [2][CH][HD]
   T* sV = sK + 2 * CH * HD;                 // [2][CH][HD]
-  const int b = blockIdx.z, head = blockIdx.y;
+  constexpr int kTokens = 64 / MAPS;
+  const int b = blockIdx.z, head = blockIdx.y * MAPS;
   const int q_begin = p.cu_q[b], q_len = p.cu_q[b + 1] - q_begin;
-  const int qt0 = blockIdx.x * 64;
+  const int qt0 = blockIdx.x * kTokens;
   if (qt0 >= q_len) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int kvh = head / (p.nh / p.nkv);
@@ -722,20 +796,20 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   for (int i = threadIdx.x; i < 64 * (HD / 8); i += 128) {
     const int r = i / (HD / 8), c = i % (HD / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (qt0 + r < q_len)
+    if (qt0 + r / MAPS < q_len)
       v = *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.q) +
-                                          static_cast<long>(q_begin + qt0 + r) * p.q_stride +
-                                          static_cast<long>(head) * HD + c * 8);
+                                          static_cast<long>(q_begin + qt0 + r / MAPS) * p.q_stride +
+                                          static_cast<long>(head + r % MAPS) * HD + c * 8);
     *reinterpret_cast<uint4*>(sQ + tile_off<HD>(r, c)) = v;
   }
-  const int last_pos = pos0 + min(q_len, qt0 + 64) - 1;  // last query position of this tile
+  const int last_pos = pos0 + min(q_len, qt0 + kTokens) - 1;  // last query position of this tile
   const int first_pos = pos0 + qt0;
   const int lo_tile = p.window > 0 ? max(0, first_pos - p.window + 1) : 0;
   const int c_begin = lo_tile / CH;
   const int c_end = last_pos / CH + 1;
   const float scale = p.sm_scale * (p.kv_fp8 == 1 ? p.k_scale : 1.f);
-  const int row0 = qt0 + warp * 16 + (lane >> 2);  // query index (within the sequence's new tokens)
-  const int posr0 = pos0 + row0, posr1 = posr0 + 8;
+  const int row0 = qt0 + (warp * 16 + (lane >> 2)) / MAPS;  // query index (within the sequence's new tokens)
+  const int posr0 = pos0 + row0, posr1 = posr0 + 8 / MAPS;
 
   float o[HD / 8][4];
 #pragma unroll
@@ -843,15 +917,46 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   cp_async_wait<0>();
   l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
-  if (p.sinks != nullptr) {
-    const float sink = p.sinks[head];
+  if (p.x.sinks != nullptr) {
+    const float sink = p.x.sinks[head + (MAPS == 2 ? (lane >> 2) & 1 : 0)];
     if (m0 != -CUDART_INF_F) l0 += exp2f((sink - m0) * kLog2e);
     if (m1 != -CUDART_INF_F) l1 += exp2f((sink - m1) * kLog2e);
   }
   const float vs = p.kv_fp8 == 1 ? p.v_scale : 1.f;
   const float i0 = l0 > 0.f ? vs / l0 : 0.f, i1 = l1 > 0.f ? vs / l1 : 0.f;
   T* out = reinterpret_cast<T*>(p.out);
-  const int od = p.out_dim > 0 ? p.out_dim : HD;
+  const int od = p.x.out_dim;
+  if constexpr (MAPS == 2) {
+    // lanes 4 apart hold the two maps of a token; both form the difference, each stores one of its two tokens
+    const bool second = (lane >> 2) & 1;
+    float ss[2] = {0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < HD / 8; ++i) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float mine = o[i][e] * (e < 2 ? i0 : i1), other = __shfl_xor_sync(0xffffffffu, mine, 4);
+        const float v = second ? other - p.x.lambda * mine : mine - p.x.lambda * other;
+        o[i][e] = v;
+        ss[e >> 1] = fmaf(v, v, ss[e >> 1]);      // channels from out_dim on are zero in the cache
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      ss[h] += __shfl_xor_sync(0xffffffffu, ss[h], 1);
+      ss[h] += __shfl_xor_sync(0xffffffffu, ss[h], 2);
+    }
+    const float f = p.x.out_scale / sqrtf((second ? ss[1] : ss[0]) / static_cast<float>(od) + p.x.eps);
+    const int row = row0 + (second ? 4 : 0);
+    if (row >= q_len) return;
+#pragma unroll
+    for (int i = 0; i < HD / 8; ++i) {
+      const int d = i * 8 + (lane & 3) * 2;
+      if (d >= od) break;
+      *reinterpret_cast<uint32_t*>(out + (static_cast<long>(q_begin + row) * (p.nh / 2) + head / 2) * od + d) =
+          MmaT<T>::pack((second ? o[i][2] : o[i][0]) * f, (second ? o[i][3] : o[i][1]) * f);
+    }
+    return;
+  }
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) {
     const int d = i * 8 + (lane & 3) * 2;
@@ -861,10 +966,11 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
       const int row = row0 + 8 * h;
       if (row >= q_len) continue;
       float a = o[i][2 * h] * (h ? i1 : i0), bb = o[i][2 * h + 1] * (h ? i1 : i0);
-      if (p.gate != nullptr) {
-        const T* g = reinterpret_cast<const T*>(p.gate) + (q_begin + row) * p.gate_stride + head * od + d;
+      if (p.x.gate != nullptr) {
+        const T* g = reinterpret_cast<const T*>(p.x.gate) + (q_begin + row) * p.x.gate_stride +
+                     (p.x.gate_per_head ? head : head * od + d);
         a /= 1.f + __expf(-static_cast<float>(g[0]));
-        bb /= 1.f + __expf(-static_cast<float>(g[1]));
+        bb /= 1.f + __expf(-static_cast<float>(g[p.x.gate_per_head ? 0 : 1]));
       }
       *reinterpret_cast<uint32_t*>(out + (static_cast<long>(q_begin + row) * p.nh + head) * od + d) = MmaT<T>::pack(a, bb);
     }
@@ -908,32 +1014,32 @@ int launch_decode(const AttnParams& p, int B, cudaStream_t s) {
   const bool merged_in_kernel = (p.merge_tickets != nullptr || (p.cluster_off != 0 && p.splits <= 8)) &&
                                 p.block_size % 16 == 0 && p.kv_fp8 <= 1;
   if (p.splits > 1 && !merged_in_kernel)
-    fi::launch_kernel(decode_merge_kernel<T, HD>, dim3(p.nh, B), dim3(HD >= 128 ? 128 : 64), 0, s, 0, p);
+    fi::launch_kernel(decode_merge_kernel<T, HD>, dim3(p.nh / p.x.maps, B), dim3(HD >= 128 ? 128 : 64), 0, s, 0, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T, int HD, int CH>
 int launch_prefill(const AttnParams& p, int B, int max_q_len, cudaStream_t s) {
   const int smem = (64 * HD + 4 * CH * HD) * 2;
-  auto kern = paged_prefill_kernel<T, HD, CH>;
+  auto kern = p.x.maps == 2 ? paged_prefill_kernel<T, HD, CH, 2> : paged_prefill_kernel<T, HD, CH, 1>;
   cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
   if (ce != cudaSuccess) return static_cast<int>(ce);
-  fi::launch_kernel(kern, dim3((max_q_len + 63) / 64, p.nh, B), dim3(128), smem, s, 0, p);
+  const int tokens = 64 / p.x.maps;
+  fi::launch_kernel(kern, dim3((max_q_len + tokens - 1) / tokens, p.nh / p.x.maps, B), dim3(128), smem, s, 0, p);
   return static_cast<int>(cudaGetLastError());
 }
 
 }  // namespace
 
-// Decode scratch: ws_o needs B*nh*splits*hd floats, ws_ml B*nh*splits*2 floats (splits > 1 only).  sinks: fp32 [nh] or
-// null; out_dim: stored channels per head (0 = hd), out rows are nh * out_dim wide; gate: rows of pitch gate_stride in
-// the type of out, or null.
+// Decode scratch: ws_o needs B*nh*splits*hd floats, ws_ml B*nh*splits*2 floats (splits > 1 only).  extra: see
+// attn_extra.h, or null.
 extern "C" int fi_paged_decode(const void* q, long q_stride, const void* k_cache,
                                const void* v_cache, void* out, const int* block_tables,
                                const int* seq_lens, float* ws_o, float* ws_ml, int B, int nh,
                                int nkv, int hd, int max_blocks, int block_size, int window,
                                float sm_scale, float softcap, int kv_fp8, float k_scale,
-                               float v_scale, int splits, const float* sinks, int out_dim, const void* gate,
-                               long gate_stride, int dtype, void* stream) {
+                               float v_scale, int splits, const FiAttnExtra* extra, int dtype,
+                               void* stream) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || splits < 1) return -10;
   AttnParams p = {};
@@ -942,8 +1048,7 @@ extern "C" int fi_paged_decode(const void* q, long q_stride, const void* k_cache
   p.ws_ml = ws_ml; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = k_scale;
   p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = splits;
-  if (out_dim < 0 || out_dim > hd) return -10;
-  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
+  if (!fi::take_extra(p, extra, hd, nh, nkv)) return -10;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -967,8 +1072,8 @@ extern "C" int fi_paged_decode_merged(const void* q, long q_stride, const void* 
                                const int* seq_lens, float* ws_o, float* ws_ml, unsigned int* tickets, int B, int nh,
                                int nkv, int hd, int max_blocks, int block_size, int window,
                                float sm_scale, float softcap, int kv_fp8, float k_scale,
-                               float v_scale, int splits, const float* sinks, int out_dim, const void* gate,
-                               long gate_stride, int dtype, void* stream) {
+                               float v_scale, int splits, const FiAttnExtra* extra, int dtype,
+                               void* stream) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || splits < 1) return -10;
   AttnParams p = {};
@@ -977,8 +1082,7 @@ extern "C" int fi_paged_decode_merged(const void* q, long q_stride, const void* 
   p.ws_ml = ws_ml; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = k_scale;
   p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = splits; p.merge_tickets = tickets;
-  if (out_dim < 0 || out_dim > hd) return -10;
-  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
+  if (!fi::take_extra(p, extra, hd, nh, nkv)) return -10;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -1013,6 +1117,7 @@ extern "C" int fi_paged_decode_rowscaled(const void* q, long q_stride, const voi
   p.ws_ml = ws_ml; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = 1.f;
   p.v_scale = 1.f; p.kv_fp8 = kv_mode; p.splits = splits; p.k_scales = k_scales; p.v_scales = v_scales;
+  fi::take_extra(p, nullptr, hd, nh, nkv);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -1042,6 +1147,7 @@ extern "C" int fi_paged_prefill_rowscaled(const void* q, long q_stride, const vo
   p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window; p.sm_scale = sm_scale;
   p.softcap = softcap; p.k_scale = 1.f; p.v_scale = 1.f; p.kv_fp8 = kv_mode; p.splits = 1;
   p.k_scales = k_scales; p.v_scales = v_scales;
+  fi::take_extra(p, nullptr, hd, nh, nkv);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == 0) {
     if (hd == 64) return launch_prefill<__nv_bfloat16, 64, 64>(p, B, max_q_len, s);
@@ -1063,8 +1169,8 @@ extern "C" int fi_paged_decode_cluster(const void* q, long q_stride, const void*
                                const int* seq_lens, int B, int nh,
                                int nkv, int hd, int max_blocks, int block_size, int window,
                                float sm_scale, float softcap, int kv_fp8, float k_scale,
-                               float v_scale, int splits, const float* sinks, int out_dim, const void* gate,
-                               long gate_stride, int dtype, void* stream) {
+                               float v_scale, int splits, const FiAttnExtra* extra, int dtype,
+                               void* stream) {
   if (B <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || splits < 1 || splits > 8 || block_size % 16 != 0) return -10;
   AttnParams p = {};
@@ -1073,8 +1179,7 @@ extern "C" int fi_paged_decode_cluster(const void* q, long q_stride, const void*
   p.ws_ml = nullptr; p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv;
   p.window = window; p.sm_scale = sm_scale; p.softcap = softcap; p.k_scale = k_scale;
   p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = splits; p.cluster_off = 1;
-  if (out_dim < 0 || out_dim > hd) return -10;
-  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
+  if (!fi::take_extra(p, extra, hd, nh, nkv)) return -10;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_DEC(TT, HD) return launch_decode<TT, HD>(p, B, s)
   if (dtype == 0) {
@@ -1095,8 +1200,7 @@ extern "C" int fi_paged_prefill(const void* q, long q_stride, const void* k_cach
                                 const int* seq_lens, const int* cu_q, int B, int max_q_len, int nh,
                                 int nkv, int hd, int max_blocks, int block_size, int window,
                                 float sm_scale, float softcap, int kv_fp8, float k_scale,
-                                float v_scale, const float* sinks, int out_dim, const void* gate, long gate_stride,
-                                int dtype, void* stream) {
+                                float v_scale, const FiAttnExtra* extra, int dtype, void* stream) {
   if (B <= 0 || max_q_len <= 0) return 0;
   if (nkv <= 0 || nh <= 0 || nh % nkv != 0) return -10;
   AttnParams p = {};
@@ -1104,8 +1208,7 @@ extern "C" int fi_paged_prefill(const void* q, long q_stride, const void* k_cach
   p.block_tables = block_tables; p.seq_lens = seq_lens; p.cu_q = cu_q; p.max_blocks = max_blocks;
   p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window; p.sm_scale = sm_scale;
   p.softcap = softcap; p.k_scale = k_scale; p.v_scale = v_scale; p.kv_fp8 = kv_fp8; p.splits = 1;
-  if (out_dim < 0 || out_dim > hd || out_dim % 2 != 0) return -10;
-  p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
+  if (!fi::take_extra(p, extra, hd, nh, nkv) || p.x.out_dim % 2 != 0) return -10;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == 0) {
     if (hd == 64) return launch_prefill<__nv_bfloat16, 64, 64>(p, B, max_q_len, s);
@@ -1156,7 +1259,7 @@ extern "C" int fi_paged_decode_noalloc(const void* q, long q_stride, const void*
   if (splits == 1)   // one split writes straight to `out`: no partials, so no scratch and no size limit
     return fi_paged_decode(q, q_stride, k_cache, v_cache, out, block_tables, seq_lens, nullptr, nullptr, B,
                            nh, nkv, hd, max_blocks, block_size, window, sm_scale, softcap, kv_fp8,
-                           k_scale, v_scale, 1, nullptr, 0, nullptr, 0, dtype, stream);
+                           k_scale, v_scale, 1, nullptr, dtype, stream);
   const size_t n_o = static_cast<size_t>(B) * nh * splits * hd;
   const size_t n_ml = static_cast<size_t>(B) * nh * splits * 2;
   if (n_o + n_ml > kNoAllocScratchFloats) {
@@ -1183,5 +1286,5 @@ extern "C" int fi_paged_decode_noalloc(const void* q, long q_stride, const void*
   float* ws_ml = ws_o + n_o;
   return fi_paged_decode(q, q_stride, k_cache, v_cache, out, block_tables, seq_lens, ws_o, ws_ml, B,
                          nh, nkv, hd, max_blocks, block_size, window, sm_scale, softcap, kv_fp8,
-                         k_scale, v_scale, splits, nullptr, 0, nullptr, 0, dtype, stream);
+                         k_scale, v_scale, splits, nullptr, dtype, stream);
 }

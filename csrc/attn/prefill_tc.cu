@@ -17,6 +17,10 @@
 //            then fold PV of the previous tile into the row's fp32 output registers
 //            (o = o * alpha + PV) so TMEM never has to be rescaled
 //
+// With two maps per head (MAPS = 2) the 128 rows are 64 tokens times the two maps of one head, side by side: query rows
+// [q1 | 0] and [0 | q2] against key rows [k1 | k2] share every K and V tile, and the epilogue takes the difference of
+// neighbouring rows, its norm over the head's channels and the scale before it stores.
+//
 // Masks (causal edge, sliding window, end of sequence) are applied only in tiles that touch an edge.
 // Every wait is bounded; a wait that runs out sets the status word and the CTA leaves through the
 // common teardown (TMEM freed).
@@ -28,16 +32,14 @@
 #include "../common/launch.cuh"
 #include "../common/ptx.cuh"
 #include "../common/tensormap.h"
+#include "attn_extra.h"
 
 namespace {
 using namespace fi;
 
 struct TcParams {
-  void* out;                 // [T, nh * out_dim]
-  const float* sinks;        // [nh] or null: one extra exp(sink) per head in the softmax denominator
-  int out_dim;               // output channels per head that are stored (<= HD)
-  const void* gate;          // row t at gate + t * gate_stride, channels as in out, or null: out *= sigmoid(gate)
-  long gate_stride;
+  void* out;                 // [T, nh / MAPS * out_dim]
+  FiAttnExtra x;             // sinks, output gate, stored channels, two maps per head
   const int* block_tables;   // [B, max_blocks]
   const int* seq_lens;       // [B]
   const int* cu_q;           // [B + 1]
@@ -77,7 +79,7 @@ __device__ __forceinline__ uint32_t pack2(float a, float b, int is_fp16) {
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-template <int HD, int STAGES>
+template <int HD, int STAGES, int MAPS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                   const __grid_constant__ CUtensorMap v_map, const TcParams p) {
@@ -97,16 +99,17 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   pdl_wait();
   // a kernel of this stream already reported a failed wait: do not add seconds of waiting per CTA
   if (p.status != nullptr && *reinterpret_cast<volatile int*>(p.status) != 0) return;
-  const int b = blockIdx.z, head = blockIdx.y;
+  constexpr int kTokens = kTile / MAPS;                       // query tokens per CTA
+  const int b = blockIdx.z, head = blockIdx.y * MAPS;
   const int q_begin = p.cu_q[b];
   const int q_len = p.cu_q[b + 1] - q_begin;
   // the tiles with the longest KV range are scheduled first
-  const int qt0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * kTile;
+  const int qt0 = (static_cast<int>(gridDim.x) - 1 - static_cast<int>(blockIdx.x)) * kTokens;
   if (qt0 >= q_len) return;
   const int seq_len = p.seq_lens[b];
   const int pos0 = seq_len - q_len;
-  const int rows = min(kTile, q_len - qt0);
-  const int first_pos = pos0 + qt0, last_pos = first_pos + rows - 1;
+  const int tokens = min(kTokens, q_len - qt0), rows = tokens * MAPS;
+  const int first_pos = pos0 + qt0, last_pos = first_pos + tokens - 1;
   const int kv_lo = p.window > 0 ? max(0, first_pos - p.window + 1) : 0;
   const int tile_begin = kv_lo / kTile;
   const int n_tiles = last_pos / kTile + 1 - tile_begin;
@@ -179,8 +182,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       tma_prefetch_desc(&q_map);
       mbar_expect_tx(q_full, L::kQ);
 #pragma unroll
-      for (int a = 0; a < kAtoms; ++a)
-        tma_load_2d(sQ + a * kAtomBytes, &q_map, q_full, head * HD + a * 64, q_begin + qt0);
+      for (int a = 0; a < kAtoms; ++a) {
+        if constexpr (MAPS == 2) tma_load_3d(sQ + a * kAtomBytes, &q_map, q_full, a * 64, head, q_begin + qt0);
+        else tma_load_2d(sQ + a * kAtomBytes, &q_map, q_full, head * HD + a * 64, q_begin + qt0);
+      }
     }
     if (lane < 2 * n_boxes) {
       const bool is_v = lane >= n_boxes;
@@ -286,7 +291,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const int half = (warp - 2) >> 2;                // 0: keys 0-63 / channels 0-HH-1, 1: the other halves
     const int row = quad * 32 + lane;
     const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
-    const int qpos = first_pos + row;
+    const int qpos = first_pos + row / MAPS;
     const float sl2 = p.sm_scale * kLog2e;
     const bool capped = p.softcap > 0.f;
     const float cap_in = capped ? p.sm_scale / p.softcap : 0.f, cap_out = p.softcap * kLog2e;
@@ -393,20 +398,62 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       half_sum[half * 128 + row] = l;
       ok = pair_sync();
       l += half_sum[(half ^ 1) * 128 + row];
-      if (p.sinks != nullptr) l += fast_exp2(fmaf(p.sinks[head], kLog2e, -m));   // every row sees at least its own key
+      if (p.x.sinks != nullptr)       // every row sees at least its own key
+        l += fast_exp2(fmaf(p.x.sinks[head + (MAPS == 2 ? row & 1 : 0)], kLog2e, -m));
+    }
+    if constexpr (MAPS == 2) {
+      // rows 2 i and 2 i + 1 are the maps of one token; both lanes form the difference and each stores half of it
+      ok = __all_sync(0xffffffffu, ok);
+      if (ok) {
+        const float inv = l > 0.f ? 1.f / l : 0.f, lam = p.x.lambda;
+        const bool second = row & 1;
+        float ss = 0.f;
+#pragma unroll
+        for (int d = 0; d < HH; ++d) {
+          const float mine = o[d] * inv, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+          o[d] = second ? other - lam * mine : mine - lam * other;
+          ss = fmaf(o[d], o[d], ss);                           // channels from out_dim on are zero in the cache
+        }
+        float* half_sq = half_max + ((n_tiles + 1) & 1) * 2 * 128;   // read for the last time before the meeting above
+        half_sq[half * 128 + row] = ss;
+        ok = pair_sync();
+        ss += half_sq[(half ^ 1) * 128 + row];
+        if (ok && row < rows) {
+          const float f = p.x.out_scale / sqrtf(ss / static_cast<float>(p.x.out_dim) + p.x.eps);
+          uint16_t* dst = reinterpret_cast<uint16_t*>(p.out) +
+                          (static_cast<long>(q_begin + qt0 + row / 2) * (p.nh / 2) + head / 2) * p.x.out_dim + half * HH;
+#pragma unroll
+          for (int c = 0; c < HH / 8; ++c) {
+            if (half * HH + c * 8 >= p.x.out_dim) break;
+            if ((c & 1) != static_cast<int>(second)) continue;
+            uint4 v;
+            v.x = pack2(o[c * 8] * f, o[c * 8 + 1] * f, p.is_fp16);
+            v.y = pack2(o[c * 8 + 2] * f, o[c * 8 + 3] * f, p.is_fp16);
+            v.z = pack2(o[c * 8 + 4] * f, o[c * 8 + 5] * f, p.is_fp16);
+            v.w = pack2(o[c * 8 + 6] * f, o[c * 8 + 7] * f, p.is_fp16);
+            *reinterpret_cast<uint4*>(dst + c * 8) = v;
+          }
+        }
+      }
+    } else {
       if (row < rows && ok) {
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        if (p.x.gate != nullptr && p.x.gate_per_head) {
+          const uint16_t raw = reinterpret_cast<const uint16_t*>(p.x.gate)[(q_begin + qt0 + row) * p.x.gate_stride + head];
+          const float g = p.is_fp16 ? __half2float(__ushort_as_half(raw)) : __uint_as_float(static_cast<uint32_t>(raw) << 16);
+          inv /= 1.f + __expf(-g);
+        }
         uint16_t* dst = reinterpret_cast<uint16_t*>(p.out) +
-                        (static_cast<long>(q_begin + qt0 + row) * p.nh + head) * p.out_dim + half * HH;
+                        (static_cast<long>(q_begin + qt0 + row) * p.nh + head) * p.x.out_dim + half * HH;
 #pragma unroll
         for (int c = 0; c < HH / 8; ++c) {
-          if (half * HH + c * 8 >= p.out_dim) break;
+          if (half * HH + c * 8 >= p.x.out_dim) break;
           float y[8];
 #pragma unroll
           for (int e = 0; e < 8; ++e) y[e] = o[c * 8 + e] * inv;
-          if (p.gate != nullptr) {
-            const uint4 raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.gate) +
-                                                              (q_begin + qt0 + row) * p.gate_stride + head * p.out_dim +
+          if (p.x.gate != nullptr && !p.x.gate_per_head) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.x.gate) +
+                                                              (q_begin + qt0 + row) * p.x.gate_stride + head * p.x.out_dim +
                                                               half * HH + c * 8);
             const uint32_t gw[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
@@ -443,14 +490,14 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   }
 }
 
-template <int HD, int STAGES>
+template <int HD, int STAGES, int MAPS>
 int launch_tc(const CUtensorMap& qm, const CUtensorMap& km, const CUtensorMap& vm, const TcParams& p, int B,
               int max_q_len, cudaStream_t s) {
-  auto kern = prefill_tc_kernel<HD, STAGES>;
+  auto kern = prefill_tc_kernel<HD, STAGES, MAPS>;
   constexpr int smem = TcSmem<HD, STAGES>::kBytes;
   cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
   if (ce != cudaSuccess) return static_cast<int>(ce);
-  ce = fi::launch_kernel(kern, dim3((max_q_len + kTile - 1) / kTile, p.nh, B), dim3(kTcThreads), smem, s, 0, qm, km,
+  ce = fi::launch_kernel(kern, dim3((max_q_len + kTile / MAPS - 1) / (kTile / MAPS), p.nh / MAPS, B), dim3(kTcThreads), smem, s, 0, qm, km,
                          vm, p);
   return static_cast<int>(ce != cudaSuccess ? ce : cudaGetLastError());
 }
@@ -471,34 +518,39 @@ extern "C" int fi_paged_prefill_tc_set_trace(void* trace) {
 // the general kernel), other negative values for malformed arguments.
 //   q: token t, head h at q + (t * q_stride + h * hd) elements, T_total rows; caches [num_blocks, nkv,
 //   block_size, hd]; out [T_total, nh * out_dim] (out_dim <= hd, a multiple of 8: the leading channels of each
-//   head); sinks: fp32 [nh] or null; gate: rows of pitch gate_stride in the type of out, or null.
+//   head); extra: see attn_extra.h, or null (two maps: query rows [q1 | 0] and [0 | q2], out [T_total, nh / 2 * out_dim]).
 extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_cache, const void* v_cache, void* out,
                                    const int* block_tables, const int* seq_lens, const int* cu_q, int B,
                                    int T_total, int max_q_len, int nh, int nkv, int hd, long num_blocks,
                                    int max_blocks, int block_size, int window, float sm_scale, float softcap,
-                                   const float* sinks, int out_dim, const void* gate, long gate_stride, int dtype,
-                                   int* status, void* stream) {
+                                   const FiAttnExtra* extra, int dtype, int* status, void* stream) {
   if (B <= 0 || max_q_len <= 0 || T_total <= 0) return 0;
-  if (nkv <= 0 || nh <= 0 || nh % nkv != 0 || out_dim <= 0 || out_dim > hd) return -10;
-  if (out_dim % 8 != 0) return -12;
+  if (nkv <= 0 || nh <= 0 || nh % nkv != 0) return -10;
+  TcParams p = {};
+  if (!fi::take_extra(p, extra, hd, nh, nkv)) return -10;
+  if (p.x.out_dim % 8 != 0) return -12;
   if ((hd != 64 && hd != 128) || (dtype != 0 && dtype != 1)) return -12;
   if (block_size != 16 && block_size != 32 && block_size != 64 && block_size % 128 != 0) return -12;
   if ((reinterpret_cast<uintptr_t>(q) & 15) != 0 || (q_stride * 2) % 16 != 0 ||
       (reinterpret_cast<uintptr_t>(out) & 15) != 0)
     return -12;
-  if (gate != nullptr && ((reinterpret_cast<uintptr_t>(gate) & 15) != 0 || gate_stride % 8 != 0)) return -12;
+  if (p.x.gate != nullptr && !p.x.gate_per_head &&
+      ((reinterpret_cast<uintptr_t>(p.x.gate) & 15) != 0 || p.x.gate_stride % 8 != 0))
+    return -12;
+  const bool pairs = p.x.maps == 2;
   CUtensorMap qm, km, vm;
   const uint64_t kv_rows = static_cast<uint64_t>(num_blocks) * nkv * block_size;
-  if (fi::make_tmap_2d_16bit_sw128(&qm, q, T_total, static_cast<uint64_t>(nh) * hd, q_stride, kTile) != 0 ||
+  if ((pairs ? fi::make_tmap_3d_16bit_sw128(&qm, q, T_total, nh, hd, q_stride, hd, kTile / 2, 2)
+             : fi::make_tmap_2d_16bit_sw128(&qm, q, T_total, static_cast<uint64_t>(nh) * hd, q_stride, kTile)) != 0 ||
       fi::make_tmap_2d_16bit_sw128(&km, k_cache, kv_rows, hd, hd, block_size < kTile ? block_size : kTile) != 0 ||
       fi::make_tmap_2d_16bit_sw128(&vm, v_cache, kv_rows, hd, hd, block_size < kTile ? block_size : kTile) != 0)
     return -12;
-  TcParams p = {};
   p.out = out; p.block_tables = block_tables; p.seq_lens = seq_lens; p.cu_q = cu_q; p.status = status;
-  p.trace = g_tc_trace; p.sinks = sinks; p.out_dim = out_dim; p.gate = gate; p.gate_stride = gate_stride;
+  p.trace = g_tc_trace;
   p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window;
   p.sm_scale = sm_scale; p.softcap = softcap; p.is_fp16 = dtype == 1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (hd == 64) return launch_tc<64, 6>(qm, km, vm, p, B, max_q_len, s);
-  return launch_tc<128, 3>(qm, km, vm, p, B, max_q_len, s);
+  if (hd == 64)
+    return pairs ? launch_tc<64, 6, 2>(qm, km, vm, p, B, max_q_len, s) : launch_tc<64, 6, 1>(qm, km, vm, p, B, max_q_len, s);
+  return pairs ? launch_tc<128, 3, 2>(qm, km, vm, p, B, max_q_len, s) : launch_tc<128, 3, 1>(qm, km, vm, p, B, max_q_len, s);
 }

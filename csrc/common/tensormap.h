@@ -46,4 +46,21 @@ inline int make_tmap_2d_16bit_sw128(CUtensorMap* out, const void* base, uint64_t
   return r == CUDA_SUCCESS ? 0 : -3;
 }
 
+// The same over rows that are split into equal parts: element (row, part, col) at row * ld + part * part_ld + col.
+// Box = [box_rows, box_parts, 64 columns]; in shared memory the parts of a row follow one another.
+inline int make_tmap_3d_16bit_sw128(CUtensorMap* out, const void* base, uint64_t rows, uint64_t parts, uint64_t cols,
+                                    uint64_t ld, uint64_t part_ld, uint32_t box_rows, uint32_t box_parts) {
+  EncodeTiledFn enc = get_encode_tiled();
+  if (enc == nullptr) return -1;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) != 0 || ((ld * 2) & 15) != 0 || ((part_ld * 2) & 15) != 0) return -2;
+  cuuint64_t dims[3] = {cols, parts, rows};
+  cuuint64_t strides[2] = {part_ld * 2, ld * 2};
+  cuuint32_t box[3] = {64, box_parts, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  CUresult r = enc(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims,
+                   strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                   CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -3;
+}
+
 }  // namespace fi

@@ -593,7 +593,7 @@ static int fi_awq_gemm_impl(const void* X, const void* qw, const void* scales, c
   GemmParams p;
   p.C = C; p.bias = bias; p.residual = residual;
   p.T = T; p.N = N; p.K = K; p.ldc = ldc;
-  p.dual_rows = dual_rows; p.act = act; p.out_fp32 = out_fp32; p.is_fp16 = dtype == 1;
+  p.dual_rows = dual_rows; p.act = act; p.act_limit = 0.f; p.out_fp32 = out_fp32; p.is_fp16 = dtype == 1;
   p.splits = splits; p.status = status;
   p.scales = scales; p.zeros = reinterpret_cast<const uint8_t*>(zeros); p.group = group;
   p.n_rows_total = w_rows;

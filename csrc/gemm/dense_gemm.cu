@@ -364,11 +364,12 @@ static int fi_dense_gemm_impl(const void* X, const void* W, void* C, const void*
                              int act, int dual_rows, int out_fp32, int dtype, int splits, int bn,
                              int* status, void* stream,
                              const FiComm* comm, float rms_eps = 0.f, int w_dynamic = 0,
-                             const FiRope* rope = nullptr, const FiGrouped* grp = nullptr) {
+                             const FiRope* rope = nullptr, const FiGrouped* grp = nullptr, float act_limit = 0.f) {
   if (T <= 0 || N <= 0 || K <= 0) return 0;
   if (rms_eps > 0.f && (K % BK) != 0) return -21;   // the sum of squares reads whole 64-wide K blocks
   if ((K % 8) != 0 || (ldc % 8) != 0 || (reinterpret_cast<uintptr_t>(C) & 15) != 0) return -10;
   if (dual_rows > 0 && N != dual_rows) return -11;
+  if (act == kActClippedSwiglu && (dual_rows <= 0 || !(act_limit > 0.f))) return -12;
   if (bn == 0) bn = fi_dense_gemm_pick_bn(T);
   const uint64_t w_rows = grp != nullptr ? static_cast<uint64_t>(grp->num_experts) * grp->expert_rows
                                          : static_cast<uint64_t>(dual_rows > 0 ? 2 * dual_rows : N);
@@ -404,7 +405,7 @@ static int fi_dense_gemm_impl(const void* X, const void* W, void* C, const void*
   GemmParams p;
   p.C = C; p.bias = bias; p.residual = residual;
   p.T = T; p.N = N; p.K = K; p.ldc = ldc;
-  p.dual_rows = dual_rows; p.act = act; p.out_fp32 = out_fp32; p.is_fp16 = dtype == 1;
+  p.dual_rows = dual_rows; p.act = act; p.act_limit = act_limit; p.out_fp32 = out_fp32; p.is_fp16 = dtype == 1;
   p.splits = splits; p.status = status;
   p.tile_expert = nullptr; p.tile_row0 = nullptr; p.tile_rows = nullptr; p.n_tiles = nullptr; p.expert_rows = 0; p.grid_tiles = 0;
   if (grp != nullptr) {
@@ -464,11 +465,12 @@ extern "C" int fi_dense_gemm_set_trace(void* trace) {
   return 0;
 }
 
+// act 4 (gated mode only): the clipped form of apply_gated with act_limit.
 extern "C" int fi_dense_gemm(const void* X, const void* W, void* C, const void* bias,
                              const void* residual, int T, int N, int K, int ldx, int ldw, int ldc,
-                             int act, int dual_rows, int out_fp32, int dtype, int splits, int bn,
+                             int act, float act_limit, int dual_rows, int out_fp32, int dtype, int splits, int bn,
                              int* status, void* stream) {
-  return fi_dense_gemm_impl(X, W, C, bias, residual, T, N, K, ldx, ldw, ldc, act, dual_rows, out_fp32, dtype, splits, bn, status, stream, nullptr);
+  return fi_dense_gemm_impl(X, W, C, bias, residual, T, N, K, ldx, ldw, ldc, act, dual_rows, out_fp32, dtype, splits, bn, status, stream, nullptr, 0.f, 0, nullptr, nullptr, act_limit);
 }
 
 // RMSNorm fused in front of the GEMM: C = (X W'^T) * rsqrt(mean_k(X^2) + eps), W' = W * diag(norm weight)
@@ -498,20 +500,20 @@ extern "C" int fi_dense_gemm_rope(const void* X, const void* W, void* C, const v
 // programmatic-launch wait.  fi_dense_gemm itself assumes weights that never change.
 extern "C" int fi_dense_gemm_dynw(const void* X, const void* W, void* C, const void* bias,
                              const void* residual, int T, int N, int K, int ldx, int ldw, int ldc,
-                             int act, int dual_rows, int out_fp32, int dtype, int splits, int bn,
+                             int act, float act_limit, int dual_rows, int out_fp32, int dtype, int splits, int bn,
                              int* status, void* stream) {
-  return fi_dense_gemm_impl(X, W, C, bias, residual, T, N, K, ldx, ldw, ldc, act, dual_rows, out_fp32, dtype, splits, bn, status, stream, nullptr, 0.f, 1);
+  return fi_dense_gemm_impl(X, W, C, bias, residual, T, N, K, ldx, ldw, ldc, act, dual_rows, out_fp32, dtype, splits, bn, status, stream, nullptr, 0.f, 1, nullptr, nullptr, act_limit);
 }
 
 // Mixture-of-experts form: rows of X [n_rows, K], sorted by expert, meet the weights of their expert.  g: tile table for
 // tiles of `bn` rows (16, 32 or 64), W [experts * g->expert_rows, K]; gated mode as above with an expert's rows
 // stored [gate; up].
 extern "C" int fi_dense_gemm_grouped(const void* X, const void* W, void* C, int n_rows, int N, int K, int ldx, int ldc,
-                             int act, int dual_rows, int dtype, int bn, const FiGrouped* g, int* status, void* stream) {
+                             int act, float act_limit, int dual_rows, int dtype, int bn, const FiGrouped* g, int* status, void* stream) {
   if (g == nullptr || (bn != 16 && bn != 32 && bn != 64) || g->max_tiles > 65535) return -25;
   if (g->max_tiles <= 0) return 0;
   return fi_dense_gemm_impl(X, W, C, nullptr, nullptr, n_rows, N, K, ldx, K, ldc, act, dual_rows, 0, dtype, 1, bn, status,
-                            stream, nullptr, 0.f, 0, nullptr, g);
+                            stream, nullptr, 0.f, 0, nullptr, g, act_limit);
 }
 
 // Same GEMM with a fused collective and/or an all-gathered token operand (see comm_desc.h).

@@ -48,6 +48,7 @@ struct PParams {
   const void* residual;
   int T, N, K, ldc;
   int dual_rows, act, is_fp16, out_fp32;
+  float act_limit;     // act 4
   int second_off;   // weight rows between the two A tiles of a CTA: dual_rows (gated) or 128 (plain, 256-row tile)
   int rows_per_tile;   // output rows (of N) one tile covers: 128 (gated or single) or 256
   int n_tiles_n, n_tiles;
@@ -68,6 +69,15 @@ __device__ __forceinline__ float act_f(float g, int act) {
   }
   if (act == 3) return fmaxf(g, 0.f);
   return g;
+}
+// Gated form of one channel: act(g) * u; 4: bounds on both halves (g from above only), g sigmoid(1.702 g) * (u + 1).
+__device__ __forceinline__ float gated_f(float g, float u, int act, float limit) {
+  if (act == 4) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+  }
+  return act_f(g, act) * u;
 }
 __device__ __forceinline__ float ld16(const void* p, size_t i, int is_fp16) {
   if (is_fp16) return __half2float(reinterpret_cast<const __half*>(p)[i]);
@@ -253,7 +263,7 @@ dense_gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmap_w, const _
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             float v = __uint_as_float(r[j]);
-            if (DUAL && gated) v = act_f(v + bias_g, p.act) * (__uint_as_float(u[j]) + bias_u);
+            if (DUAL && gated) v = gated_f(v + bias_g, __uint_as_float(u[j]) + bias_u, p.act, p.act_limit);
             else v = act_f(v, p.act);
             patch[j * 32 + lane] = v;
           }
@@ -337,13 +347,14 @@ int launch(const CUtensorMap& tw, const CUtensorMap& tx, const PParams& p, cudaS
 // rows], bias (if any) [gate bias; up bias] and N must equal dual_rows.  Nothing is
 // allocated; returns 0, a negative argument error or a positive CUDA error code.
 extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, const void* bias, const void* residual,
-                                        int T, int N, int K, int ldx, int ldw, int ldc, int act, int dual_rows,
-                                        int out_fp32, int dtype, int* status, void* stream) {
+                                        int T, int N, int K, int ldx, int ldw, int ldc, int act, float act_limit,
+                                        int dual_rows, int out_fp32, int dtype, int* status, void* stream) {
   if (T <= 0 || N <= 0 || K <= 0) return 0;
   if ((K % 8) != 0 || (ldx % 8) != 0 || (ldw % 8) != 0 || (N % 8) != 0 || (ldc % 8) != 0 ||
       (reinterpret_cast<uintptr_t>(C) & 15) != 0 || (residual != nullptr && (reinterpret_cast<uintptr_t>(residual) & 15) != 0))
     return -10;
   if (dual_rows > 0 && N != dual_rows) return -11;
+  if (act == 4 && (dual_rows <= 0 || !(act_limit > 0.f))) return -12;
   if (out_fp32 && residual != nullptr) return -13;
   const int w_rows = dual_rows > 0 ? 2 * dual_rows : N;
   CUtensorMap tw, tx;
@@ -354,7 +365,7 @@ extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, c
   PParams p = {};
   p.C = C; p.bias = bias; p.residual = residual;
   p.T = T; p.N = N; p.K = K; p.ldc = ldc;
-  p.dual_rows = dual_rows; p.act = act; p.is_fp16 = dtype == 1; p.out_fp32 = out_fp32;
+  p.dual_rows = dual_rows; p.act = act; p.act_limit = act_limit; p.is_fp16 = dtype == 1; p.out_fp32 = out_fp32;
   // plain products use a 256-row tile (two A tiles per stage against one token tile), which halves the
   // L2 -> shared-memory traffic per FLOP; 128 x 128 tiles were L2-bandwidth-bound at ~55 % of peak
   const bool wide = dual_rows == 0 && N > BM;
@@ -372,18 +383,19 @@ extern "C" int fi_dense_gemm_persistent(const void* X, const void* W, void* C, c
 // table (built for tiles of 128 rows), W [experts * g->expert_rows, K]; C [n_rows, ldc] in X's type.  Gated mode
 // (dual_rows > 0): an expert's rows are [gate; up] and N == dual_rows.
 extern "C" int fi_dense_gemm_persistent_grouped(const void* X, const void* W, void* C, int n_rows, int N, int K, int ldx,
-                                                int ldc, int act, int dual_rows, int dtype, const FiGrouped* g, int* status,
-                                                void* stream) {
+                                                int ldc, int act, float act_limit, int dual_rows, int dtype, const FiGrouped* g,
+                                                int* status, void* stream) {
   if (n_rows <= 0 || N <= 0 || K <= 0 || g->max_tiles <= 0) return 0;
   if ((K % 8) != 0 || (ldx % 8) != 0 || (N % 8) != 0 || (ldc % 8) != 0 || (reinterpret_cast<uintptr_t>(C) & 15) != 0) return -10;
   if (dual_rows > 0 && N != dual_rows) return -11;
+  if (act == 4 && (dual_rows <= 0 || !(act_limit > 0.f))) return -12;
   CUtensorMap tw, tx;
   int r = make_tmap_2d_16bit_sw128(&tw, W, static_cast<uint64_t>(g->num_experts) * g->expert_rows, K, K, BM);
   if (r != 0) return r * 100 - 1;
   r = make_tmap_2d_16bit_sw128(&tx, X, n_rows, K, ldx, BN);
   if (r != 0) return r * 100 - 2;
   PParams p = {};
-  p.C = C; p.T = n_rows; p.N = N; p.K = K; p.ldc = ldc; p.dual_rows = dual_rows; p.act = act; p.is_fp16 = dtype == 1;
+  p.C = C; p.T = n_rows; p.N = N; p.K = K; p.ldc = ldc; p.dual_rows = dual_rows; p.act = act; p.act_limit = act_limit; p.is_fp16 = dtype == 1;
   const bool wide = dual_rows == 0 && N > BM;
   p.second_off = dual_rows > 0 ? dual_rows : BM;
   p.rows_per_tile = wide ? 2 * BM : BM;

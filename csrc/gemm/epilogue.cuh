@@ -34,7 +34,7 @@ constexpr int kXferTwoShot = 3;      // all-reduce in two hops: partials go to t
 constexpr int kPhasePush = 1, kPhaseReduce = 2, kPhaseCollect = 4;
 constexpr int kMaxCommTiles = 8192; // tiles per call that the flag area can describe
 
-enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2, kActRelu = 3 };
+enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2, kActRelu = 3, kActClippedSwiglu = 4 };
 enum CommMode : int { kCommNone = 0, kCommAllReduce = 1, kCommReduceScatter = 2 };
 
 struct GemmParams {
@@ -45,6 +45,7 @@ struct GemmParams {
   int ldc;
   int dual_rows;  // > 0: gated mode, W = [2 * dual_rows, K]; N == dual_rows
   int act;
+  float act_limit;   // kActClippedSwiglu
   int out_fp32;
   int is_fp16;
   int splits;
@@ -113,6 +114,17 @@ __device__ __forceinline__ float apply_act(float g, int act) {
   }
   if (act == kActRelu) return fmaxf(g, 0.f);
   return g;
+}
+
+// Gated form of one channel: act(g) * u, or with bounds on both halves (g from above only)
+// g sigmoid(1.702 g) * (u + 1).
+__device__ __forceinline__ float apply_gated(float g, float u, int act, float limit) {
+  if (act == kActClippedSwiglu) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
+  }
+  return apply_act(g, act) * u;
 }
 
 __device__ __forceinline__ float ld16_as_float(const void* p, size_t i, int is_fp16) {
@@ -398,7 +410,7 @@ __device__ __forceinline__ void epilogue_tmem_to_smem(const GemmParams& p, uint6
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             stage_f32[(c0 + j) * BM + n_local] =
-                apply_act(__uint_as_float(r[j]) + bias_g, p.act) * (__uint_as_float(u[j]) + bias_u);
+                apply_gated(__uint_as_float(r[j]) + bias_g, __uint_as_float(u[j]) + bias_u, p.act, p.act_limit);
         } else {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -483,7 +495,7 @@ __device__ __forceinline__ void epilogue_reduce_store(const GemmParams& p, float
             bg = ld16_as_float(p.bias, n + j, p.is_fp16);
             bu = ld16_as_float(p.bias, p.dual_rows + n + j, p.is_fp16);
           }
-          g[j] = apply_act(g[j] + bg, p.act) * (u[j] + bu);
+          g[j] = apply_gated(g[j] + bg, u[j] + bu, p.act, p.act_limit);
         }
       } else if (!DUAL && p.act != kActNone && !comm) {
 #pragma unroll

@@ -1,12 +1,13 @@
 // Residual-stream kernels: decoders whose sublayers are normalised on both sides and whose layers read a weighted
-// average of everything before them, and decoders whose sublayers read one norm side by side.  The stream and every
-// norm are 32-bit; the sublayers' inputs and outputs may be 16-bit.
+// average of everything before them, decoders whose sublayers read one norm side by side, and decoders that normalise
+// only what a sublayer returns.  The stream and every norm are 32-bit; the sublayers' inputs and outputs may be 16-bit.
 //
 //   start    v = table[token] * scale                                  X_0 = v
 //   add      v = x + y + sum_k w_k e_(slot k)                          x   = v     (y: mixer, e: routed experts' rows)
 //   step     v = x + norm(y) * w_post                                  x   = v
+//   post     v = x + norm(y + sum_k w_k e_k) * w_post                  x   = v     (e_k: routed experts' rows, or x)
 //   average  X_n = x + norm(y) * w_post;  v = sum_{j<=n} a_j X_j        x   = v
-//   each:    h = norm(v) * w_pre          (what the next sublayer reads)
+//   each:    h = norm(v) * w_pre          (what the next sublayer reads; start, post: v itself without w_pre)
 //
 // The norm is an RMS norm over equal consecutive parts ("groups") of the vector, so a group of one token needs
 // nothing from any other group: the unit of work is a (token, group) row.  Steps with many tokens give a row to a
@@ -21,11 +22,11 @@
 
 namespace {
 
-enum Mode : int { kStart = 0, kStep = 1, kAverage = 2, kAdd = 3 };
+enum Mode : int { kStart = 0, kStep = 1, kAverage = 2, kAdd = 3, kPost = 4 };
 enum DType : int { kBf16 = 0, kFp16 = 1, kFp32 = 2 };
 
 struct StreamParams {
-  const void* y;         // [*, ldy] sublayer output (type y_type)
+  const void* y;         // [*, ldy] sublayer output (type y_type); kPost: null = zeros
   const float* x;        // [*, W] stream before the sublayer
   const void* table;     // kStart: [V, W] embedding (type h_type)
   const long long* ids;  // kStart: token per row
@@ -36,12 +37,12 @@ struct StreamParams {
   float* x_out;          // [*, W] or null
   void* h;               // [*, ldh] (type h_type)
   const long long* sel;  // optional: output row r comes from token sel[r]; x_out is not written then
-  const void* routed;    // kAdd: expert outputs (type y_type), rows of pitch ldr, or null
-  const int* slot_of;    // kAdd: [*, top] row of each (token, choice), < 0: none; null: row = token * top + choice
-  const float* route_w;  // kAdd: [*, top]
+  const void* routed;    // kAdd, kPost: expert outputs (type y_type), rows of pitch ldr, or null
+  const int* slot_of;    // kAdd, kPost: [*, top] row of each (token, choice), < 0: none; null: row = token * top + choice
+  const float* route_w;  // kAdd, kPost: [*, top]
   long ldy, ldh, hist_stride, ldr;
   float scale;           // kStart
-  int top;
+  int top, pass_through; // pass_through: a choice without a row stands for x itself (kPost)
   int rows, W, group, groups, n, y_type, h_type, vocab;
   float eps;
 };
@@ -174,11 +175,42 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
       if (c < p.group) {
-        load_any<VEC, H16>(p.y, t * p.ldy + c0 + c, p.y_type, v + i * VEC);
+        if (MODE != kPost || p.y != nullptr) {
+          load_any<VEC, H16>(p.y, t * p.ldy + c0 + c, p.y_type, v + i * VEC);
+        } else {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[i * VEC + e] = 0.f;
+        }
         load_any<VEC, false>(p.x, t * p.W + c0 + c, kFp32, xv + i * VEC);
       } else {
 #pragma unroll
         for (int e = 0; e < VEC; ++e) { v[i * VEC + e] = 0.f; xv[i * VEC + e] = 0.f; }
+      }
+    }
+    if constexpr (MODE == kPost) {
+      float through = 0.f;                 // weight of x itself
+      if (p.routed != nullptr) {
+#pragma unroll 4
+        for (int k = 0; k < p.top; ++k) {
+          const long at = t * p.top + k;
+          const long slot = p.slot_of != nullptr ? p.slot_of[at] : at;
+          const float w = p.route_w[at];
+          if (slot < 0) through += w;
+#pragma unroll
+          for (int i = 0; i < NV; ++i) {
+            const int c = (i * TPR + tid) * VEC;
+            if (c < p.group && slot >= 0) {
+              float e4[VEC];
+              load_any<VEC, H16>(p.routed, slot * p.ldr + c0 + c, p.y_type, e4);
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(w, e4[e], v[i * VEC + e]);
+            }
+          }
+        }
+      }
+      if (p.pass_through) {
+#pragma unroll
+        for (int i = 0; i < NV * VEC; ++i) v[i] = fmaf(through, xv[i], v[i]);
       }
     }
 #pragma unroll
@@ -250,6 +282,12 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
         store_any<VEC, H16>(p.h, static_cast<long>(r) * p.ldh + c0 + c, p.h_type, o);
       }
     }
+  } else if ((MODE == kStart || MODE == kPost) && p.h != nullptr) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * TPR + tid) * VEC;
+      if (c < p.group) store_any<VEC, H16>(p.h, static_cast<long>(r) * p.ldh + c0 + c, p.h_type, v + i * VEC);
+    }
   }
 }
 
@@ -289,7 +327,7 @@ bool aligned(const void* p, unsigned a) { return (reinterpret_cast<uintptr_t>(p)
 
 }  // namespace
 
-// X_0 = table[ids] * scale (32-bit) into x0, h = norm(X_0) * w_pre.  h_type (0 bf16, 1 fp16, 2 fp32) is also the
+// X_0 = table[ids] * scale (32-bit) into x0, h = norm(X_0) * w_pre (w_pre null: h = X_0; h null: none).  h_type (0 bf16, 1 fp16, 2 fp32) is also the
 // table's type.  Token ids outside the table read row 0.
 extern "C" int fi_stream_start(const long long* ids, const void* table, int vocab, float scale, const float* w_pre,
                                float* x0, void* h, long ldh, int T, int W, int groups, float eps, int h_type,
@@ -355,4 +393,24 @@ extern "C" int fi_stream_add(const void* y, long ldy, int y_type, const float* x
   const bool vec4 = p.group % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0 && ldr % 4 == 0 && aligned(y, 16) && aligned(x, 16) &&
                     aligned(x_out, 16) && aligned(h, 16) && aligned(routed, 16) && aligned(w_pre, 16);
   return dispatch<kAdd>(p, vec4, reinterpret_cast<cudaStream_t>(stream));
+}
+
+// v = x + norm(y + sum_k route_w[t, k] routed[slot_of[t, k]]) * w_post; x_out = v (may be x, or null); h = norm(v) *
+// w_pre, or v itself without w_pre (h null: none).  y (null: zeros), routed and h share a type; routed null: no experts.
+// pass_through: a choice whose slot is negative stands for x itself, otherwise it adds nothing.  sel as in fi_stream_add.
+extern "C" int fi_stream_post(const void* y, long ldy, int y_type, const float* x, const void* routed, long ldr,
+                              const int* slot_of, const float* route_w, int top, int pass_through, const float* w_post,
+                              const float* w_pre, float* x_out, void* h, long ldh, int h_type, const long long* sel, int rows,
+                              int W, int groups, float eps, void* stream) {
+  if (rows <= 0) return 0;
+  if (W <= 0 || groups <= 0 || W % groups != 0 || h_type < 0 || h_type > 2 || y_type != h_type || top < 0) return -10;
+  if ((sel != nullptr && x_out != nullptr) || (routed != nullptr && (route_w == nullptr || top <= 0))) return -10;
+  if (w_post == nullptr || (y == nullptr && routed == nullptr) || (w_pre != nullptr && h == nullptr)) return -10;
+  StreamParams p = {};
+  p.y = y; p.ldy = ldy; p.y_type = y_type; p.x = x; p.routed = routed; p.ldr = ldr; p.slot_of = slot_of; p.route_w = route_w;
+  p.top = top; p.pass_through = pass_through; p.w_post = w_post; p.w_pre = w_pre; p.x_out = x_out; p.h = h; p.ldh = ldh;
+  p.h_type = h_type; p.sel = sel; p.rows = rows; p.W = W; p.group = W / groups; p.groups = groups; p.eps = eps;
+  const bool vec4 = p.group % 4 == 0 && ldh % 4 == 0 && ldy % 4 == 0 && ldr % 4 == 0 && aligned(y, 16) && aligned(x, 16) &&
+                    aligned(x_out, 16) && aligned(h, 16) && aligned(routed, 16) && aligned(w_post, 16) && aligned(w_pre, 16);
+  return dispatch<kPost>(p, vec4, reinterpret_cast<cudaStream_t>(stream));
 }

@@ -3,13 +3,14 @@
 //
 //   fi_moe_route   : scores -> top-k experts and weights per token, three scoring rules:
 //                    0 softmax over all experts, top-k, renormalise (Gemma4: vllm/model_executor/
-//                      models/gemma4/moe.py:98-125, optional per-expert scale),
+//                      models/gemma4/moe.py:98-125, optional per-expert scale); selection by score +
+//                      correction bias where there is one,
 //                    1 sigmoid scores, selection by score + correction bias, weights = normalised
 //                      scores x routed scaling (DeepSeek-V3 style),
 //                    2 sqrt(softplus) scores with bias (DeepSeek-V4-Flash: deepseek_v4_flash/
 //                      gpu_layers.py:323-352).
-//                    Optionally the experts form equal groups of neighbours and only the best groups (by the sum
-//                    of their two largest selection scores) can be chosen.
+//                    Optionally the experts form equal groups of neighbours and only the best groups (by their
+//                    largest selection score, or the sum of their two largest) can be chosen.
 //   fi_moe_align   : counting sort of the (token, k) routes by expert restricted to the experts this
 //                    rank owns; emits sorted route ids, the inverse map, per-expert offsets and the
 //                    tile table (expert, first row, rows) consumed by fi_awq_gemm_grouped.
@@ -36,7 +37,7 @@ constexpr int kMaxExpertsPerLane = 16;   // experts <= 512
 __global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                  const float* __restrict__ expert_scale, int* __restrict__ topk_ids,
                                  float* __restrict__ topk_w, long ld, int T, int E, int K, int mode,
-                                 int renorm, float routed_scale, int groups, int keep_groups) {
+                                 int renorm, float routed_scale, int groups, int keep_groups, int group_best) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -62,7 +63,11 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
       sum += score[i];
     }
     for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    for (int i = 0; i < per; ++i) { score[i] /= sum; sel[i] = (i * 32 + lane) < E ? score[i] : -CUDART_INF_F; }
+    for (int i = 0; i < per; ++i) {
+      const int e = i * 32 + lane;
+      score[i] /= sum;
+      sel[i] = e < E ? score[i] + (bias ? bias[e] : 0.f) : -CUDART_INF_F;
+    }
   } else {
     for (int i = 0; i < per; ++i) {
       const int e = i * 32 + lane;
@@ -91,12 +96,16 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
           m1 = fmaxf(m1, sel[i]);
         }
       }
-      for (int o = 16; o > 0; o >>= 1) {
-        const float o1 = __shfl_xor_sync(0xffffffffu, m1, o), o2 = __shfl_xor_sync(0xffffffffu, m2, o);
-        m2 = fmaxf(fmaxf(m2, o2), fminf(m1, o1));
-        m1 = fmaxf(m1, o1);
+      if (group_best < 2) {
+        for (int o = 16; o > 0; o >>= 1) m1 = fmaxf(m1, __shfl_xor_sync(0xffffffffu, m1, o));
+      } else {
+        for (int o = 16; o > 0; o >>= 1) {
+          const float o1 = __shfl_xor_sync(0xffffffffu, m1, o), o2 = __shfl_xor_sync(0xffffffffu, m2, o);
+          m2 = fmaxf(fmaxf(m2, o2), fminf(m1, o1));
+          m1 = fmaxf(m1, o1);
+        }
       }
-      if ((g & 31) == lane) gscore[g >> 5] = size > 1 ? m1 + m2 : m1;
+      if ((g & 31) == lane) gscore[g >> 5] = group_best >= 2 && size > 1 ? m1 + m2 : m1;
     }
     unsigned kept[kMaxExpertsPerLane];                       // bit g & 31 of word g >> 5: the group may be chosen
     for (int i = 0; i < gper; ++i) kept[i] = 0u;
@@ -381,7 +390,7 @@ __global__ void moe_combine_allreduce_kernel(const T* __restrict__ y_sorted, con
 }
 
 // Expert products on the general cores: 32 rows x 64 outputs per block, 32-bit arithmetic.
-//   gather: out[row] = act(Wg x) * (Wu x) with x = X[sorted_route[row] / top] and weights [Wg (N rows); Wu (N rows)]
+//   gather: out[row] = act(Wg x) * (Wu x), or its clipped form (act 4), with x = X[sorted_route[row] / top] and weights [Wg (N rows); Wu (N rows)]
 //   else:   out[row] = W x with x = X[row]
 struct ExpertRows {
   const void* x;            // rows of pitch ldx
@@ -393,7 +402,8 @@ struct ExpertRows {
   const int* tile_rows;     // at most 32
   const int* n_tiles;
   long ldx, ldo;
-  int N, K, top, gather;
+  int N, K, top, gather, act;
+  float limit;
 };
 
 template <typename T>
@@ -454,8 +464,14 @@ __global__ void __launch_bounds__(256) moe_expert_rows_kernel(const ExpertRows p
     for (int i = 0; i < 4; ++i) {
       const int n = n0 + tn + 16 * i;
       if (n >= p.N) continue;
-      const float g = ag[h][i];
-      out[n] = static_cast<T>(p.gather ? g / (1.f + __expf(-g)) * au[h][i] : g);
+      float v = ag[h][i];
+      if (p.gather && p.act == 4) {
+        const float g = fminf(v, p.limit);
+        v = g / (1.f + __expf(-1.702f * g)) * (fminf(fmaxf(au[h][i], -p.limit), p.limit) + 1.f);
+      } else if (p.gather) {
+        v = v / (1.f + __expf(-v)) * au[h][i];
+      }
+      out[n] = static_cast<T>(v);
     }
   }
 }
@@ -489,13 +505,14 @@ extern "C" int fi_moe_combine_allreduce(const void* y_sorted, const int* slot_of
 
 extern "C" int fi_moe_route(const float* logits, const float* bias, const float* expert_scale,
                             long ld, int* topk_ids, float* topk_w, int T, int E, int K, int mode, int renorm,
-                            float routed_scale, int groups, int keep_groups, void* stream) {
+                            float routed_scale, int groups, int keep_groups, int group_best, void* stream) {
   if (T <= 0) return 0;
   if (E > 32 * kMaxExpertsPerLane || K > 32 || K > E || groups < 1 || E % groups != 0 || keep_groups < 1 ||
-      keep_groups > groups || K > keep_groups * (E / groups) || ld < E)
+      keep_groups > groups || K > keep_groups * (E / groups) || ld < E || group_best < 1 || group_best > 2)
     return -10;
   fi::launch_kernel(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, FI_STREAM(stream), 0, logits, bias,
-                    expert_scale, topk_ids, topk_w, ld, T, E, K, mode, renorm, routed_scale, groups, keep_groups);
+                    expert_scale, topk_ids, topk_w, ld, T, E, K, mode, renorm, routed_scale, groups, keep_groups,
+                    group_best);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -541,16 +558,20 @@ extern "C" int fi_moe_combine(const void* y_sorted, const int* slot_of, const fl
 }
 
 // Expert products without tensor cores (dtype 0 bf16, 1 fp16, 2 fp32; any sizes), over the tile table of fi_moe_align
-// (built with bn <= 32).  gather != 0: out[row] = silu(Wg x) * (Wu x) with x = X[sorted_route[row] / top], weights
+// (built with bn <= 32).  gather != 0: out[row] = silu(Wg x) * (Wu x) (act 1) or, with g = min(Wg x, limit) and
+// u = Wu x bounded by limit on both sides, g sigmoid(1.702 g) (u + 1) (act 4), for x = X[sorted_route[row] / top], weights
 // [experts, 2 N, K]; gather == 0: out[row] = W X[row], weights [experts, N, K].
 extern "C" int fi_moe_expert_rows(const void* x, long ldx, const void* w, void* out, long ldo, const int* sorted_route,
                                   const int* tile_expert, const int* tile_row0, const int* tile_rows, const int* n_tiles,
-                                  int max_tiles, int N, int K, int top, int gather, int dtype, void* stream) {
+                                  int max_tiles, int N, int K, int top, int gather, int act, float limit, int dtype,
+                                  void* stream) {
   if (max_tiles <= 0) return 0;
+  if (gather && act != 1 && act != 4) return -11;
   if (N <= 0 || K <= 0 || top <= 0 || max_tiles > 65535 || (gather && sorted_route == nullptr)) return -10;
   ExpertRows p = {};
   p.x = x; p.w = w; p.out = out; p.ldx = ldx; p.ldo = ldo; p.sorted_route = sorted_route; p.tile_expert = tile_expert;
   p.tile_row0 = tile_row0; p.tile_rows = tile_rows; p.n_tiles = n_tiles; p.N = N; p.K = K; p.top = top; p.gather = gather;
+  p.act = act; p.limit = limit;
   const dim3 grid((N + 63) / 64, max_tiles);
   if (dtype == 0) return static_cast<int>(fi::launch_kernel(moe_expert_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, FI_STREAM(stream), 0, p));
   if (dtype == 1) return static_cast<int>(fi::launch_kernel(moe_expert_rows_kernel<__half>, grid, dim3(256), 0, FI_STREAM(stream), 0, p));

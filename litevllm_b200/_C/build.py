@@ -75,6 +75,9 @@ KERNEL_SETS = {
                 "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "linear_attn/channel_delta.cu",
                 "linear_attn/hgrn2.cu", "misc/norm_rope_misc.cu", "misc/residual_stream.cu", "misc/sampling.cu",
                 "moe/moe_kernels.cu"],
+    "luzerax": ["attn/head_prepare.cu", "attn/latent_rows.cu", "attn/paged_attention.cu", "attn/prefill_tc.cu",
+                "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "misc/norm_rope_misc.cu", "misc/residual_stream.cu",
+                "misc/sampling.cu", "moe/moe_kernels.cu"],
 }
 
 

@@ -1,12 +1,13 @@
-"""Routed experts without biases, each ``W_down (act(W_gate x) * (W_up x))``.  The router's logits come from outside (they
+"""Routed experts without biases, each ``W_down (act(W_gate x) * (W_up x))`` (``act`` may be the clipped form of
+``ops.gated_linear``).  The router's logits come from outside (they
 may share a product with other small 32-bit projections) and the weighted sum over the chosen experts is left to the
 caller's residual add.
 
     s = score(z);  chosen: the ``top`` largest s + correction among the best groups;  weight = s * scale (optionally
     divided by the sum over the chosen)
 
-``groups`` equal groups of neighbouring experts are ranked by the sum of their two largest s + correction; only experts of
-the best ``keep`` can be chosen.
+``groups`` equal groups of neighbouring experts are ranked by the sum of their ``group_best`` largest s + correction; only
+experts of the best ``keep`` can be chosen.  The last ``identity`` router outputs stand for experts that return their input.
 """
 from __future__ import annotations
 
@@ -18,13 +19,15 @@ from ...ops import moe
 
 class RoutedExperts(nn.Module):
     def __init__(self, hidden: int, inter: int, experts: int, top: int, dtype, act: str = "silu", score: str = "sigmoid",
-                 groups: int = 1, keep: int = 1, scale: float = 1.0, renormalize: bool = False):
+                 groups: int = 1, keep: int = 1, scale: float = 1.0, renormalize: bool = False, group_best: int = 2,
+                 identity: int = 0, act_limit: float = 0.0):
         super().__init__()
         self.E, self.top, self.act, self.score, self.inter = experts, top, act, score, inter
         self.groups, self.keep, self.scale, self.renormalize = groups, keep, float(scale), renormalize
+        self.group_best, self.act_limit, self.outputs = group_best, float(act_limit), experts + identity
         self.w_gate_up = nn.Parameter(torch.empty(experts, 2 * inter, hidden, dtype=dtype), requires_grad=False)
         self.w_down = nn.Parameter(torch.empty(experts, hidden, inter, dtype=dtype), requires_grad=False)
-        self.correction = nn.Parameter(torch.zeros(experts, dtype=torch.float32), requires_grad=False)
+        self.correction = nn.Parameter(torch.zeros(self.outputs, dtype=torch.float32), requires_grad=False)
 
     def destinations(self, prefix: str) -> dict:
         """Checkpoint name -> where its values go."""
@@ -37,7 +40,8 @@ class RoutedExperts(nn.Module):
         return d
 
     def forward(self, x, logits) -> moe.RoutedRows:
-        """x [T, hidden], logits fp32 [T, experts]."""
+        """x [T, hidden], logits fp32 [T, experts + identity]."""
         ids, w = moe.route(logits, self.top, mode=self.score, bias=self.correction, renormalize=self.renormalize,
-                           routed_scale=self.scale, groups=self.groups, keep_groups=self.keep)
-        return moe.expert_rows(x, self.w_gate_up, self.w_down, ids, w, self.act)
+                           routed_scale=self.scale, groups=self.groups, keep_groups=self.keep,
+                           group_best=self.group_best)
+        return moe.expert_rows(x, self.w_gate_up, self.w_down, ids, w, self.act, self.act_limit, self.outputs > self.E)

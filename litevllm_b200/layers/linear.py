@@ -19,13 +19,14 @@ class LiteLinear(nn.Module):
     def __init__(self, in_features: int, out_features: int, bias: bool = False,
                  dtype: torch.dtype = torch.bfloat16, shard: str | None = None,
                  quant_config=None, prefix: str = "", gated_act: str | None = None,
-                 out_splits: list[int] | None = None):
+                 out_splits: list[int] | None = None, act_limit: float = 0.0):
         super().__init__()
         tp = pstate.tp_size() if shard else 1
         self.shard = shard
         self.tp = tp
         self.prefix = prefix
         self.gated_act = gated_act          # set: weight is [gate; up] and forward returns act(g)*u
+        self.act_limit = float(act_limit)   # bounds of the "clipped_swiglu" form
         self.full_in, self.full_out = in_features, out_features
         self.out_splits = out_splits or [out_features]   # logical pieces of a merged weight
         self.in_features = in_features // tp if shard == "row" else in_features
@@ -64,7 +65,7 @@ class LiteLinear(nn.Module):
                                            use_bias=use_bias)
         if self.gated_act is not None:
             return ops.gated_linear(x, self.weight, self.gated_act, out=out, rms_eps=norm_eps,
-                                    bias=self.bias if use_bias else None)
+                                    bias=self.bias if use_bias else None, act_limit=self.act_limit)
         return ops.linear(x, self.weight, self.bias if use_bias else None, residual, out=out,
                           out_dtype=out_dtype, rms_eps=norm_eps)
 

@@ -310,3 +310,50 @@ def iter_pofadra_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, de
             yield vec(p + "mlp.correction", E, 0.0, 0.1)
     yield vec("final.norm", W, 1.0, 0.1)
     yield lin("head", V, W)
+
+
+def iter_luzerax_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, device="cpu") -> Iterator[tuple[str, torch.Tensor]]:
+    """Linear weights ~ N(0, 1 / fan-in); norms and scales near one; corrections that move the choice of experts."""
+    W, V = arch.hidden_size, arch.vocab_size
+
+    def lin(name, out_f, in_f):
+        return name, normal(name, (out_f, in_f), seed, in_f ** -0.5, dtype, device)
+
+    def vec(name, n, base=0.0, std=1.0):
+        return name, base + normal(name, (n,), seed, std, torch.float32, device)
+
+    def gated(p, ff):
+        for n, o, k in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+            yield lin(p + n, o, k)
+
+    yield "embed", normal("embed", (V, W), seed, 1.0, dtype, device)
+    for i, l in enumerate(arch.extra["layers"]):
+        p, m, mlp = f"l{i}.", l["mixer"], l.get("mlp")
+        H, G, d, dv, maps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], 2 if l["type"] == "attention" else 1
+        for n in ("norm1", "ls1") + (("norm2", "ls2") if mlp else ()):
+            yield vec(p + n, W, 1.0, 0.1)
+        yield lin(p + "mix.q", H * maps * d, W)
+        yield lin(p + "mix.k", G * maps * d, W)
+        yield lin(p + "mix.v", G * dv, W)
+        yield lin(p + "mix.o", W, H * dv)
+        if maps == 2:
+            for n in ("q.norm", "k.norm"):
+                yield vec(p + "mix." + n, d, 1.0, 0.1)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                yield vec(p + "mix." + n, d, 0.0, 0.3 * d ** -0.25)
+        else:
+            yield lin(p + "mix.g", H, W)
+        if not mlp:
+            continue
+        if mlp["kind"] == "dense":
+            yield from gated(p + "mlp.", mlp["ff"])
+            continue
+        r = mlp["router"]
+        for e in range(r["experts"]):
+            yield from gated(p + f"mlp.e{e}.", mlp["expert"]["ff"])
+        yield lin(p + "mlp.router", r["experts"] + r.get("identity", 0), W)
+        yield vec(p + "mlp.correction", r["experts"] + r.get("identity", 0), 0.0, 0.02)
+        if mlp.get("shared"):
+            yield from gated(p + "mlp.shared.", mlp["shared"]["ff"])
+    yield vec("final.norm", W, 1.0, 0.1)
+    yield lin("head", V, W)

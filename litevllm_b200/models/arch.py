@@ -208,8 +208,68 @@ def arch_from_pofadra_config(cfg: dict) -> ModelArch:
     return arch
 
 
+def arch_from_luzerax_config(cfg: dict) -> ModelArch:
+    """Luzerax configurations list their layers one by one (mixer type and sizes; dense, routed or no feed-forward)."""
+    layers = cfg["layers"]
+    if not layers:
+        raise ValueError("the configuration lists no layers")
+
+    def positive(entry: dict, name: str, where: str) -> None:
+        if not isinstance(entry.get(name), (int, float)) or not entry[name] > 0:
+            raise ValueError(f"{where}: {name!r} must be a positive number, got {entry.get(name)!r}")
+
+    for i, l in enumerate(layers):
+        m, where = l["mixer"], f"layers[{i}]"
+        if l["type"] not in ("attention", "attention_2"):
+            raise ValueError(f"{where}: unknown mixer {l['type']!r}")
+        _sizes(m, ("heads", "kv_heads", "dim", "vdim"), where)
+        positive(m, "scale", where)
+        if m["heads"] % m["kv_heads"]:
+            raise ValueError(f"{where}: {m['heads']} heads do not share {m['kv_heads']} key heads evenly")
+        if l["type"] == "attention":
+            if not isinstance(m.get("diff"), (int, float)):
+                raise ValueError(f"{where}: 'diff' must be a number, got {m.get('diff')!r}")
+            if m.get("q_temp"):
+                positive(m["q_temp"], "every", where)
+        else:
+            dims = m["rot"]["dims"]
+            if dims % 2 or dims > m["dim"] or dims < 0:
+                raise ValueError(f"{where}: cannot rotate {dims} of {m['dim']} dimensions")
+        mlp = l.get("mlp")
+        if not mlp:
+            continue
+        if mlp.get("kind") == "dense":
+            _sizes(mlp, ("ff",), where)
+        elif mlp.get("kind") == "moe":
+            r = mlp["router"]
+            for part in (mlp["expert"], *([mlp["shared"]] if mlp.get("shared") else [])):
+                _sizes(part, ("ff",), where)
+                positive(part, "limit", where)
+            _sizes(r, ("experts", "top"), where)
+            g, n = r.get("groups") or {"count": 1, "keep": 1}, r["experts"] + r.get("identity", 0)
+            _sizes(g, ("count", "keep"), where)
+            if n % g["count"] or g["keep"] > g["count"] or r["top"] > g["keep"] * (n // g["count"]):
+                raise ValueError(f"{where}: cannot choose {r['top']} of {n} router outputs from {g['keep']} of {g['count']} groups")
+        else:
+            raise ValueError(f"{where}: unknown feed-forward {mlp.get('kind')!r}")
+    mixers, mlps = [l["mixer"] for l in layers], [l["mlp"] for l in layers if l.get("mlp")]
+    arch = ModelArch(
+        family="luzerax", architecture="Luzerax", hidden_size=int(cfg["width"]), num_layers=len(layers),
+        num_heads=max(m["heads"] for m in mixers), num_kv_heads=max(m["kv_heads"] for m in mixers),
+        head_dim=max(m["dim"] for m in mixers),
+        intermediate_size=max((m["ff"] if m["kind"] == "dense" else m["expert"]["ff"] for m in mlps), default=0),
+        vocab_size=int(cfg["vocab"]), rms_eps=float(cfg["norm"]["eps"]), act="silu",
+        max_position=int(cfg.get("max_position_embeddings", 1 << 20)), eos_token_ids=_eos_list(cfg),
+        bos_token_id=cfg.get("bos_token_id"))
+    arch.layer_types = ["full"] * len(layers)
+    arch.extra.update(layers=layers)
+    return arch
+
+
 def arch_from_hf_config(cfg: dict) -> ModelArch:
     """Build a :class:`ModelArch` from a HF config dict (text sub-config is unwrapped)."""
+    if str(cfg.get("architecture", "")).lower() == "luzerax":
+        return arch_from_luzerax_config(cfg)
     if str(cfg.get("architecture", "")).lower() == "pofadra":
         return arch_from_pofadra_config(cfg)
     if str(cfg.get("architecture", "")).lower() == "fimodra":

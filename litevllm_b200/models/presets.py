@@ -166,6 +166,31 @@ PRESETS["tiny-pofadra-test"] = pofadra_config(160, 512, "ddaDA", (6, 2, 40, 24, 
 PRESETS["pofadra-1b"] = pofadra_config(2048, 32000, "ddad" * 3, (16, 4, 128, 64, 1024), (16, 16, 128, 128, 4), (32, 4, 4, 2, 768))
 
 
+def luzerax_config(width: int, vocab: int, pattern: str, diff: tuple, gated: tuple, ff: int, moe: tuple, rot_base: float = 1e5,
+                   temp: tuple = (0.4, 4096), diff_init: float = 0.4, eps: float = 1e-6) -> dict:
+    """Luzerax configuration from a layer pattern: per layer a mixer ("d" differential, "g" gated) and a feed-forward ("f"
+    dense, "m" routed, "-" none).  ``diff``: heads, kv heads, dim of a map, vdim; ``gated``: heads, kv heads, dim, vdim,
+    rotated dims; ``moe``: experts, pass-through outputs, top, groups, kept groups, ff, ff of the shared expert; ``temp``:
+    coefficient and span of the queries' factor."""
+    d = dict(zip(("heads", "kv_heads", "dim", "vdim"), diff), scale=diff[2] ** -0.5, diff=diff_init,
+             q_temp=dict(zip(("coef", "every"), temp)))
+    g = dict(zip(("heads", "kv_heads", "dim", "vdim"), gated[:4]), scale=gated[2] ** -0.5 * 8,
+             rot={"base": rot_base, "dims": gated[4]})
+    routed = {"kind": "moe", "expert": {"ff": moe[5], "limit": 7.0}, "shared": {"ff": moe[6], "limit": 5.0},
+              "router": {"experts": moe[0], "identity": moe[1], "top": moe[2], "groups": {"count": moe[3], "keep": moe[4]}}}
+    mlps = {"f": {"kind": "dense", "ff": ff}, "m": routed, "-": None}
+    layers = [{"type": "attention" if pattern[i] == "d" else "attention_2", "mixer": copy.deepcopy(d if pattern[i] == "d" else g),
+               "mlp": copy.deepcopy(mlps[pattern[i + 1]])} for i in range(0, len(pattern), 2)]
+    return {"architecture": "Luzerax", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers}
+
+
+PRESETS["tiny-luzerax-test"] = luzerax_config(160, 512, "dfgmd-gf", (6, 2, 24, 40), (4, 2, 40, 24, 16), 176, (9, 3, 3, 4, 2, 48, 80),
+                                              temp=(0.7, 20))
+# layers of the width and head geometry of a 1B-class decoder
+PRESETS["luzerax-1b"] = luzerax_config(2048, 32000, "df" + "gmdmgm" * 3, (16, 4, 64, 128), (16, 4, 128, 128, 64), 5632,
+                                       (32, 8, 4, 4, 2, 768, 1536))
+
+
 def get_preset(name: str) -> dict:
     key = name.lower()
     if key not in PRESETS:

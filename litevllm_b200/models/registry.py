@@ -23,12 +23,13 @@ _MODELS = {
     "DeepseekV4FlashForCausalLM": ("deepseek_v4_flash", "DeepseekV4FlashForCausalLM"),
     "Fimodra": ("fimodra", "FimodraForCausalLM"),
     "Pofadra": ("pofadra", "PofadraForCausalLM"),
+    "Luzerax": ("luzerax", "LuzeraxForCausalLM"),
 }
 _FAMILY_DEFAULT = {
     "llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen3_5": "Qwen3_5ForCausalLM",
     "qwen2_vl": "Qwen2VLForConditionalGeneration", "gemma4": "Gemma4ForCausalLM",
     "deepseek_mla": "DeepseekV3ForCausalLM", "deepseek_v4_flash": "DeepseekV4FlashForCausalLM",
-    "fimodra": "Fimodra", "pofadra": "Pofadra",
+    "fimodra": "Fimodra", "pofadra": "Pofadra", "luzerax": "Luzerax",
 }
 
 

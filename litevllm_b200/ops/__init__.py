@@ -15,7 +15,7 @@ import torch
 
 from . import _lib, reference
 
-_ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "gelu": 2, "relu": 3}
+_ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "gelu": 2, "relu": 3, "clipped_swiglu": 4}
 _DT = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
 
 _status_words: dict[int, torch.Tensor] = {}
@@ -211,13 +211,13 @@ def linear(x, w, bias=None, residual=None, act=None, out=None, out_dtype=None, s
         # prefill-sized: persistent CTAs with two TMEM accumulators (epilogue overlaps the next main loop)
         rc = _lib.kernels().fi_dense_gemm_persistent(
             _p(x), _p(w), _p(out), _p(bias), _p(residual), T, N, K, x.stride(0), w.stride(0), out.stride(0),
-            _ACT[act], 0, 1 if wide_out else 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
+            _ACT[act], 0.0, 0, 1 if wide_out else 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
         _lib.check(rc, "fi_dense_gemm_persistent")
         _count()
         return out
     fn = _lib.kernels().fi_dense_gemm if static_weight else _lib.kernels().fi_dense_gemm_dynw
     rc = fn(_p(x), _p(w), _p(out), _p(bias), _p(residual), T, N, K, x.stride(0), w.stride(0),
-            out.stride(0), _ACT[act], 0, 1 if out.dtype == torch.float32 else 0, _DT[x.dtype], splits,
+            out.stride(0), _ACT[act], 0.0, 0, 1 if out.dtype == torch.float32 else 0, _DT[x.dtype], splits,
             bn, _p(status_word(x.device)), _stream())
     _lib.check(rc, "fi_dense_gemm")
     _count()
@@ -257,13 +257,14 @@ def linear_rope_cache(x, w, bias, positions, cos_sin, slot_mapping, k_cache, v_c
     return out
 
 
-def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0, bias=None):
+def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0, bias=None, act_limit=0.0):
     """``act(x @ Wg.T + bg) * (x @ Wu.T + bu)`` with ``w_gate_up = [Wg; Wu]`` of shape [2*I, K] and the optional
-    ``bias = [bg; bu]`` -> [T, I] (``rms_eps > 0``: rows of ``x`` RMS-normalised inside the kernel)."""
+    ``bias = [bg; bu]`` -> [T, I] (``rms_eps > 0``: rows of ``x`` RMS-normalised inside the kernel).  ``act =
+    "clipped_swiglu"``: ``g sigmoid(1.702 g) * (u + 1)`` with g bounded from above and u on both sides by ``act_limit``."""
     if not x.is_cuda:
         if rms_eps > 0:
             x = _rms_scaled(x, rms_eps)
-        y = reference.gated_linear(x, w_gate_up, act, bias=bias)
+        y = reference.gated_linear(x, w_gate_up, act, bias=bias, limit=act_limit)
         if out is not None:
             out.copy_(y)
             return out
@@ -278,16 +279,17 @@ def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0
         y = _plain_product(x if rms_eps <= 0 else _rms_scaled(x, rms_eps), w_gate_up)
         if bias is not None:
             y = y + bias.float()
-        out.copy_(reference.apply_act(y[:, :inter], act) * y[:, inter:])
+        out.copy_(reference.apply_gated(y[:, :inter], y[:, inter:], act, act_limit))
         return out
     if rms_eps <= 0 and _PERSISTENT_GEMM and T >= _PERSISTENT_MIN_T and splits == 0 and bn == 0 and inter % 8 == 0:
         rc = _lib.kernels().fi_dense_gemm_persistent(
             _p(x), _p(w_gate_up), _p(out), _p(bias), None, T, inter, K, x.stride(0), w_gate_up.stride(0), out.stride(0),
-            _ACT[act], inter, 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
+            _ACT[act], act_limit, inter, 0, _DT[x.dtype], _p(status_word(x.device)), _stream())
         _lib.check(rc, "fi_dense_gemm_persistent(gated)")
         _count()
         return out
     if rms_eps > 0:
+        assert act != "clipped_swiglu", "the fused input norm has no bounded activation"
         rc = _lib.kernels().fi_dense_gemm_rmsnorm(
             _p(x), _p(w_gate_up), _p(out), _p(bias), None, T, inter, K, x.stride(0), w_gate_up.stride(0),
             out.stride(0), _ACT[act], inter, 0, _DT[x.dtype], splits, bn, float(rms_eps),
@@ -295,7 +297,7 @@ def gated_linear(x, w_gate_up, act="silu", out=None, splits=0, bn=0, rms_eps=0.0
     else:
         rc = _lib.kernels().fi_dense_gemm(
             _p(x), _p(w_gate_up), _p(out), _p(bias), None, T, inter, K, x.stride(0), w_gate_up.stride(0),
-            out.stride(0), _ACT[act], inter, 0, _DT[x.dtype], splits, bn,
+            out.stride(0), _ACT[act], act_limit, inter, 0, _DT[x.dtype], splits, bn,
             _p(status_word(x.device)), _stream())
     _lib.check(rc, "fi_dense_gemm(gated)")
     _count()
@@ -431,19 +433,44 @@ def pick_decode_splits(B: int, nkv: int, max_kv_len: int, sm_count: int = 148) -
     return int(max(1, min(want, chunks, 32)))
 
 
+class FiAttnExtra(ctypes.Structure):
+    """csrc/attn/attn_extra.h"""
+    _fields_ = [("sinks", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_long), ("out_dim", ctypes.c_int),
+                ("gate_per_head", ctypes.c_int), ("maps", ctypes.c_int), ("lam", ctypes.c_float), ("out_scale", ctypes.c_float),
+                ("eps", ctypes.c_float)]
+
+
+def attn_extra(nh: int, od: int, sinks=None, gate=None, diff=None):
+    """Argument of the attention kernels: sinks, an output gate (one value per channel or per head), and ``diff =
+    (lambda, scale, eps)`` for two maps per head."""
+    if gate is not None:
+        if diff is not None:
+            raise ValueError("attention with two maps per head takes no output gate")
+        if gate.shape[1] not in (nh, nh * od) or gate.stride(1) != 1:
+            raise ValueError(f"a gate of shape {tuple(gate.shape)} fits neither {nh} heads nor their {od} channels")
+    lam, scale, eps = diff if diff is not None else (0.0, 1.0, 0.0)
+    return ctypes.byref(FiAttnExtra(_p(sinks), _p(gate), gate.stride(0) if gate is not None else 0, od,
+                                    1 if gate is not None and gate.shape[1] == nh else 0, 1 if diff is None else 2,
+                                    float(lam), float(scale), float(eps)))
+
+
 def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv, hd, sm_scale,
                            window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, splits=0,
-                           max_kv_len=None, cu_q=None, sinks=None, v_dim=None, gate=None):
+                           max_kv_len=None, cu_q=None, sinks=None, v_dim=None, gate=None, diff=None):
     """One query token per sequence.  q: [B, >= nh*hd] with row stride q.stride(0).  ``sinks`` (fp32 [nh]): a number per
     head whose exponential joins the softmax denominator.  ``v_dim``: only the leading channels of a head's output
-    exist.  ``gate`` [B, nh * v_dim] (any row pitch, the type of the output): the output is multiplied by its sigmoid."""
+    exist.  ``gate`` [B, nh * v_dim or nh] (any row pitch, the type of the output): the output is multiplied by its
+    sigmoid.  ``diff = (lambda, scale, eps)``: query heads 2 j and 2 j + 1 (rows [q1 | 0] and [0 | q2] against keys
+    [k1 | k2]) are the two maps of output head j, ``rms(a1 - lambda a2) * scale``; the output has nh / 2 heads."""
     B = seq_lens.shape[0]
     od = hd if v_dim is None else int(v_dim)
-    extra = (_p(sinks), od, _p(gate), gate.stride(0) if gate is not None else 0)
+    heads_out = nh if diff is None else nh // 2
+    plain = sinks is None and gate is None and od == hd and diff is None
+    extra = attn_extra(nh, od, sinks, gate, diff)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_decode", block_tables, seq_lens, k_cache)
     if not q.is_cuda:
-        assert sinks is None and gate is None and od == hd, "the CPU form of sinks, gates and narrow outputs is ops.qk_attn"
+        assert plain, "the CPU form of sinks, gates, narrow outputs and two maps is ops.qk_attn"
         cu = torch.arange(B + 1, dtype=torch.int32)
         y = reference.paged_attention(q, k_cache, v_cache, block_tables, seq_lens, cu, nh, nkv, hd,
                                       sm_scale, window, softcap, k_scale, v_scale)
@@ -452,11 +479,11 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
             return out
         return y
     if out is None:
-        out = torch.empty(B, nh * od, dtype=q.dtype, device=q.device)
+        out = torch.empty(B, heads_out * od, dtype=q.dtype, device=q.device)
     elif not out.is_contiguous():
         # the kernels write rows of nh * od values back to back
         tmp = paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv, hd, sm_scale, window,
-                                     softcap, k_scale, v_scale, None, splits, max_kv_len, cu_q, sinks, v_dim, gate)
+                                     softcap, k_scale, v_scale, None, splits, max_kv_len, cu_q, sinks, v_dim, gate, diff)
         out.copy_(tmp)
         return out
     if splits <= 0:
@@ -465,7 +492,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
         eff = min(max_kv_len, window) if window and window > 0 else max_kv_len
         splits = pick_decode_splits(B, nkv, eff)
     mode = reference.kv_mode(k_cache)
-    assert mode < 2 or (sinks is None and gate is None and od == hd), "row-scaled caches take no sinks, gates or narrow outputs"
+    assert mode < 2 or plain, "row-scaled caches take no sinks, gates, narrow outputs or two maps"
     if mode >= 2:
         ws_o = ws_ml = None
         if splits > 1:
@@ -483,7 +510,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
         rc = _lib.kernels().fi_paged_decode_cluster(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens), B, nh, nkv, hd,
             block_tables.shape[1], k_cache.shape[2], int(window or 0), sm_scale, float(softcap or 0.0),
-            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, *extra, _DT[q.dtype], _stream())
+            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, extra, _DT[q.dtype], _stream())
         _lib.check(rc, "fi_paged_decode_cluster")
         _count()
         return out
@@ -505,7 +532,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
             _p(ws_o), _p(ws_ml), _p(_merge_tickets(q.device)), B, nh, nkv, hd, block_tables.shape[1],
             k_cache.shape[2], int(window or 0), sm_scale, float(softcap or 0.0),
-            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, *extra, _DT[q.dtype], _stream())
+            1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, splits, extra, _DT[q.dtype], _stream())
         _lib.check(rc, "fi_paged_decode_merged")
         _count()
         return out
@@ -513,7 +540,7 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
         _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
         _p(ws_o), _p(ws_ml), B, nh, nkv, hd, block_tables.shape[1], k_cache.shape[2], int(window or 0),
         sm_scale, float(softcap or 0.0), 1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale,
-        v_scale, splits, *extra, _DT[q.dtype], _stream())
+        v_scale, splits, extra, _DT[q.dtype], _stream())
     _lib.check(rc, "fi_paged_decode")
     _count(2 if splits > 1 else 1)
     return out
@@ -559,17 +586,16 @@ def paged_metadata_snapshot(q, k_cache, block_tables, seq_lens, cu_q=None, scope
 
 def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv,
                             hd, sm_scale, window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, sinks=None,
-                            v_dim=None, gate=None):
-    """Varlen causal attention of new tokens against the paged cache (which already holds them).  ``sinks`` (fp32
-    [nh]): a number per head whose exponential joins the softmax denominator.  ``v_dim``: only the leading ``v_dim``
-    channels of a head's output exist (rows of nh * v_dim).  ``gate`` [T, nh * v_dim] (any row pitch, the type of the
-    output): the output is multiplied by its sigmoid."""
+                            v_dim=None, gate=None, diff=None):
+    """Varlen causal attention of new tokens against the paged cache (which already holds them).  ``sinks``, ``v_dim``,
+    ``gate`` and ``diff`` as in :func:`paged_attention_decode`."""
     od = hd if v_dim is None else int(v_dim)
+    plain = sinks is None and gate is None and od == hd and diff is None
+    extra = attn_extra(nh, od, sinks, gate, diff)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_prefill", block_tables, seq_lens, k_cache, cu_q)
     if not q.is_cuda:
-        assert sinks is None and gate is None and od == hd, \
-            "the CPU forms of sinks, gates and narrow outputs live in ops.latent_attn and ops.qk_attn"
+        assert plain, "the CPU forms of sinks, gates, narrow outputs and two maps live in ops.latent_attn and ops.qk_attn"
         y = reference.paged_attention(q, k_cache, v_cache, block_tables, seq_lens, cu_q, nh, nkv, hd,
                                       sm_scale, window, softcap, k_scale, v_scale)
         if out is not None:
@@ -579,15 +605,14 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
     T = q.shape[0]
     B = seq_lens.shape[0]
     if out is None:
-        out = torch.empty(T, nh * od, dtype=q.dtype, device=q.device)
+        out = torch.empty(T, (nh if diff is None else nh // 2) * od, dtype=q.dtype, device=q.device)
     elif not out.is_contiguous():
         tmp = paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv, hd,
-                                      sm_scale, window, softcap, k_scale, v_scale, None, sinks, v_dim)
+                                      sm_scale, window, softcap, k_scale, v_scale, None, sinks, v_dim, gate, diff)
         out.copy_(tmp)
         return out
     mode = reference.kv_mode(k_cache)
-    assert mode < 2 or (sinks is None and gate is None and od == hd), "row-scaled caches take no sinks, gates or narrow outputs"
-    gate_args = (_p(gate), gate.stride(0) if gate is not None else 0)
+    assert mode < 2 or plain, "row-scaled caches take no sinks, gates, narrow outputs or two maps"
     if mode >= 2:
         rc = _lib.kernels().fi_paged_prefill_rowscaled(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(k_cache.fi_scales), _p(v_cache.fi_scales), _p(out),
@@ -602,7 +627,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         rc = _lib.kernels().fi_paged_prefill_tc(
             _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens), _p(cu_q), B, T,
             int(max_q_len), nh, nkv, hd, k_cache.shape[0], block_tables.shape[1], k_cache.shape[2], int(window or 0),
-            sm_scale, float(softcap or 0.0), _p(sinks), od, *gate_args, _DT[q.dtype], _p(status_word(q.device)), _stream())
+            sm_scale, float(softcap or 0.0), extra, _DT[q.dtype], _p(status_word(q.device)), _stream())
         if rc != -12:       # -12: outside what the tensor-core kernel covers, take the general one
             _lib.check(rc, "fi_paged_prefill_tc")
             _count()
@@ -611,7 +636,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(seq_lens),
         _p(cu_q), B, int(max_q_len), nh, nkv, hd, block_tables.shape[1], k_cache.shape[2],
         int(window or 0), sm_scale, float(softcap or 0.0),
-        1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, _p(sinks), od, *gate_args, _DT[q.dtype], _stream())
+        1 if k_cache.dtype == torch.float8_e4m3fn else 0, k_scale, v_scale, extra, _DT[q.dtype], _stream())
     _lib.check(rc, "fi_paged_prefill")
     _count()
     return out

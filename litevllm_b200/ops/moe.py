@@ -30,22 +30,22 @@ class FiGrouped(ctypes.Structure):
 
 def route(logits: torch.Tensor, top_k: int, mode: str = "softmax", bias: torch.Tensor | None = None,
           expert_scale: torch.Tensor | None = None, renormalize: bool = True, routed_scale: float = 1.0,
-          groups: int = 1, keep_groups: int = 1):
-    """logits [T, E] float32 (any row pitch) -> (ids int32 [T, k], weights float32 [T, k]).  With ``keep_groups <
-    groups`` the experts form ``groups`` equal groups of neighbours, and only the ``keep_groups`` with the largest sums of
-    their two best selection scores can be chosen."""
+          groups: int = 1, keep_groups: int = 1, group_best: int = 2):
+    """logits [T, E] float32 (any row pitch) -> (ids int32 [T, k], weights float32 [T, k]).  Selection is by score +
+    ``bias``, weights come from the scores.  With ``keep_groups < groups`` the experts form ``groups`` equal groups of
+    neighbours, and only the ``keep_groups`` with the largest sums of their ``group_best`` (1 or 2) best selection scores
+    can be chosen."""
     T, E = logits.shape
     if not logits.is_cuda:
         lf = logits.float()
         if mode == "softmax":
             score = torch.softmax(lf, dim=-1)
-            sel = score
         else:
             score = torch.sigmoid(lf) if mode == "sigmoid" else torch.sqrt(torch.nn.functional.softplus(lf))
-            sel = score + (bias.float() if bias is not None else 0.0)
+        sel = score + (bias.float() if bias is not None else 0.0)
         if keep_groups < groups:
             per = sel.view(T, groups, -1)
-            gs = torch.topk(per, min(2, per.shape[-1]), dim=-1).values.sum(-1)
+            gs = torch.topk(per, min(group_best, per.shape[-1]), dim=-1).values.sum(-1)
             drop = torch.ones_like(gs, dtype=torch.bool).scatter_(1, torch.topk(gs, keep_groups, dim=-1).indices, False)
             sel = per.masked_fill(drop[..., None], float("-inf")).view(T, E)
         ids = torch.topk(sel, top_k, dim=-1).indices
@@ -61,7 +61,7 @@ def route(logits: torch.Tensor, top_k: int, mode: str = "softmax", bias: torch.T
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     rc = _lib.kernels().fi_moe_route(_p(logits), _p(bias), _p(expert_scale), logits.stride(0), _p(ids), _p(w), T, E, top_k,
                                      ROUTER_MODES[mode], 1 if renormalize else 0, float(routed_scale), groups, keep_groups,
-                                     _stream())
+                                     group_best, _stream())
     _lib.check(rc, "fi_moe_route")
     _count()
     return ids, w
@@ -70,16 +70,22 @@ def route(logits: torch.Tensor, top_k: int, mode: str = "softmax", bias: torch.T
 @dataclass
 class RoutedRows:
     """Outputs of the chosen experts before their weighted sum: choice k of token t is row ``slot_of[t, k]`` of ``rows``
-    (row t * K + k without a map), its weight ``weights[t, k]``."""
+    (row t * K + k without a map), its weight ``weights[t, k]``.  A choice whose slot is negative has no row: it adds nothing,
+    or with ``pass_through`` the experts' input itself."""
     rows: torch.Tensor               # [T * K, H]
     weights: torch.Tensor            # fp32 [T, K]
     slot_of: torch.Tensor | None = None
+    pass_through: bool = False
 
-    def combined(self) -> torch.Tensor:
-        """fp32 [T, H]; PyTorch form (the kernels fold the sum into the residual add)."""
+    def combined(self, x: torch.Tensor | None = None) -> torch.Tensor:
+        """fp32 [T, H]; PyTorch form (the kernels fold the sum into the residual add).  ``x``: the experts' input."""
         T, K = self.weights.shape
-        r = self.rows if self.slot_of is None else self.rows.index_select(0, self.slot_of.reshape(-1).long())
-        return (r.float().view(T, K, -1) * self.weights[..., None]).sum(1)
+        if self.slot_of is None:
+            return (self.rows.float().view(T, K, -1) * self.weights[..., None]).sum(1)
+        none = (self.slot_of < 0)[..., None]
+        r = self.rows.index_select(0, self.slot_of.clamp(min=0).reshape(-1).long()).float().view(T, K, -1)
+        r = torch.where(none, x.float()[:, None] if self.pass_through else torch.zeros_like(r), r)
+        return (r * self.weights[..., None]).sum(1)
 
 
 def _tile_table(ids, n: int, E: int, bn: int, dev, scratch_name: str):
@@ -98,26 +104,28 @@ def _tile_table(ids, n: int, E: int, bn: int, dev, scratch_name: str):
 
 
 def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
-                weights: torch.Tensor, act: str = "silu") -> RoutedRows:
+                weights: torch.Tensor, act: str = "silu", act_limit: float = 0.0, pass_through: bool = False) -> RoutedRows:
     """Unquantised experts: x [T, H], ``w_gate_up`` [E, 2 I, H] (gate | up), ``w_down`` [E, H, I], ids / weights of
-    :func:`route`.  No host synchronisation.  16-bit weights whose rows are whole 16-byte groups run grouped tcgen05
+    :func:`route`; ids from E on have no row (``pass_through``: they stand for x itself).  ``act`` and ``act_limit`` as in
+    :func:`ops.gated_linear`.  No host synchronisation.  16-bit weights whose rows are whole 16-byte groups run grouped tcgen05
     products (persistent tiles when an expert sees many rows), everything else the general 32-bit kernel."""
     T, H = x.shape
     E, two_i, _ = w_gate_up.shape
     inter, K = two_i // 2, ids.shape[1]
     if not x.is_cuda:
-        rows = torch.empty(T * K, H, dtype=x.dtype)
+        rows = torch.zeros(T * K, H, dtype=x.dtype)
         flat = ids.reshape(-1).long()
-        for e in flat.unique().tolist():
+        for e in flat[flat < E].unique().tolist():
             at = torch.nonzero(flat == e).view(-1)
             h = x[at // K].float() @ w_gate_up[e].float().t()
-            a = (reference.apply_act(h[:, :inter], act) * h[:, inter:]).to(x.dtype)
+            a = reference.apply_gated(h[:, :inter], h[:, inter:], act, act_limit).to(x.dtype)
             rows[at] = (a.float() @ w_down[e].float().t()).to(x.dtype)
-        return RoutedRows(rows, weights)
+        slots = torch.where(flat < E, torch.arange(T * K), -1).view(T, K).to(torch.int32)
+        return RoutedRows(rows, weights, slots, pass_through)
     n, dev, lib, st, dt = T * K, x.device, _lib.kernels(), _stream(), _DT[x.dtype]
     rows = torch.empty(n, (H + 7) // 8 * 8, dtype=x.dtype, device=dev)[:, :H]
     if n == 0:
-        return RoutedRows(rows, weights)
+        return RoutedRows(rows, weights, None, pass_through)
     mean = (n + E - 1) // E
     tensor = x.dtype != torch.float32 and H % 8 == 0 and inter % 8 == 0 and x.stride(0) % 8 == 0
     persistent = tensor and mean >= 64
@@ -127,17 +135,17 @@ def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     slot_of = slots.view(T, K)
     acts = torch.empty(n, inter, dtype=x.dtype, device=dev)
     if not tensor:
-        if act != "silu":
-            raise ValueError("the general expert kernel computes silu gates")
+        if act not in ("silu", "clipped_swiglu"):
+            raise ValueError("the general expert kernel computes silu gates, plain or clipped")
         w1, w2 = w_gate_up.contiguous(), w_down.contiguous()
         rc = lib.fi_moe_expert_rows(_p(x), x.stride(0), _p(w1), _p(acts), inter, _p(order), _p(t_e), _p(t_r0), _p(t_n),
-                                    _p(n_tiles), bound, inter, H, K, 1, dt, st)
+                                    _p(n_tiles), bound, inter, H, K, 1, _ACT[act], act_limit, dt, st)
         _lib.check(rc, "fi_moe_expert_rows(gate_up)")
         rc = lib.fi_moe_expert_rows(_p(acts), inter, _p(w2), _p(rows), rows.stride(0), None, _p(t_e), _p(t_r0), _p(t_n),
-                                    _p(n_tiles), bound, H, inter, K, 0, dt, st)
+                                    _p(n_tiles), bound, H, inter, K, 0, 0, 0.0, dt, st)
         _lib.check(rc, "fi_moe_expert_rows(down)")
         _count(2)
-        return RoutedRows(rows, weights, slot_of)
+        return RoutedRows(rows, weights, slot_of, pass_through)
     x_sorted = torch.empty(n, H, dtype=x.dtype, device=dev)
     xc = x if x.is_contiguous() else x.contiguous()
     rc = lib.fi_moe_gather(_p(xc), _p(order), _p(offsets), E, n, K, H, _p(x_sorted), dt, st)
@@ -147,20 +155,20 @@ def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     sw = _p(status_word(dev))
     if persistent:
         rc = lib.fi_dense_gemm_persistent_grouped(_p(x_sorted), _p(w_gate_up), _p(acts), n, inter, H, H, inter, _ACT[act],
-                                                  inter, dt, ctypes.byref(g1), sw, st)
+                                                  act_limit, inter, dt, ctypes.byref(g1), sw, st)
         _lib.check(rc, "fi_dense_gemm_persistent_grouped(gate_up)")
-        rc = lib.fi_dense_gemm_persistent_grouped(_p(acts), _p(w_down), _p(rows), n, H, inter, inter, rows.stride(0), 0, 0, dt,
+        rc = lib.fi_dense_gemm_persistent_grouped(_p(acts), _p(w_down), _p(rows), n, H, inter, inter, rows.stride(0), 0, 0.0, 0, dt,
                                                   ctypes.byref(g2), sw, st)
         _lib.check(rc, "fi_dense_gemm_persistent_grouped(down)")
     else:
-        rc = lib.fi_dense_gemm_grouped(_p(x_sorted), _p(w_gate_up), _p(acts), n, inter, H, H, inter, _ACT[act], inter, dt, bn,
+        rc = lib.fi_dense_gemm_grouped(_p(x_sorted), _p(w_gate_up), _p(acts), n, inter, H, H, inter, _ACT[act], act_limit, inter, dt, bn,
                                        ctypes.byref(g1), sw, st)
         _lib.check(rc, "fi_dense_gemm_grouped(gate_up)")
-        rc = lib.fi_dense_gemm_grouped(_p(acts), _p(w_down), _p(rows), n, H, inter, inter, rows.stride(0), 0, 0, dt, bn,
+        rc = lib.fi_dense_gemm_grouped(_p(acts), _p(w_down), _p(rows), n, H, inter, inter, rows.stride(0), 0, 0.0, 0, dt, bn,
                                        ctypes.byref(g2), sw, st)
         _lib.check(rc, "fi_dense_gemm_grouped(down)")
     _count(3)
-    return RoutedRows(rows, weights, slot_of)
+    return RoutedRows(rows, weights, slot_of, pass_through)
 
 
 def _reference_experts(x, w_gate_up: Int4Weight, w_down: Int4Weight, ids, weights, num_experts, e_lo, e_hi, act):

@@ -28,6 +28,14 @@ def apply_act(x: torch.Tensor, act: str | None) -> torch.Tensor:
     raise ValueError(f"unknown activation {act}")
 
 
+def apply_gated(g: torch.Tensor, u: torch.Tensor, act: str, limit: float = 0.0) -> torch.Tensor:
+    """``act(g) * u``, or the form with bounds on both halves (g from above only)."""
+    if act == "clipped_swiglu":
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return g * torch.sigmoid(1.702 * g) * (u + 1.0)
+    return apply_act(g, act) * u
+
+
 def linear(x, w, bias=None, residual=None, act=None, out_dtype=None):
     y = x.float() @ w.float().t()
     if act:
@@ -39,12 +47,12 @@ def linear(x, w, bias=None, residual=None, act=None, out_dtype=None):
     return y.to(out_dtype or x.dtype)
 
 
-def gated_linear(x, w_gate_up, act="silu", out_dtype=None, bias=None):
+def gated_linear(x, w_gate_up, act="silu", out_dtype=None, bias=None, limit=0.0):
     inter = w_gate_up.shape[0] // 2
     y = x.float() @ w_gate_up.float().t()
     if bias is not None:
         y = y + bias.float()
-    return (apply_act(y[:, :inter], act) * y[:, inter:]).to(out_dtype or x.dtype)
+    return apply_gated(y[:, :inter], y[:, inter:], act, limit).to(out_dtype or x.dtype)
 
 
 def rmsnorm(x, w, eps, residual=None, w_mode=0, out_scale=1.0):
