@@ -68,6 +68,8 @@ def parse_args():
     ap.add_argument("--fimodra-sizes", type=int, nargs="*", default=None, help="widths for --fimodra (default: all)")
     ap.add_argument("--pofadra", action="store_true", help="the same for the Pofadra design")
     ap.add_argument("--pofadra-sizes", type=int, nargs="*", default=None, help="widths for --pofadra (default: all)")
+    ap.add_argument("--luzerax", action="store_true", help="the same for the Luzerax design")
+    ap.add_argument("--luzerax-sizes", type=int, nargs="*", default=None, help="widths for --luzerax (default: all)")
     return ap.parse_args()
 
 
@@ -595,6 +597,10 @@ def main():
     if args.pofadra:
         from benchmarks import pofadra_shapes
         print(json.dumps(run_shapes(pofadra_shapes, args.pofadra_sizes)), flush=True)
+        return
+    if args.luzerax:
+        from benchmarks import luzerax_shapes
+        print(json.dumps(run_shapes(luzerax_shapes, args.luzerax_sizes)), flush=True)
         return
     res = run_reference(args) if args.impl == "reference" else run_ours(args)
     if res:

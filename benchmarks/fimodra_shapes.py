@@ -223,7 +223,7 @@ def throughput_row(width: int, name: str, cfg: dict, layers: int = 8, batch: int
     llm = LLM("synthetic:shape-comparison", dtype="bfloat16", max_num_seqs=batch, max_model_len=prompt + steps + 64,
               max_num_batched_tokens=8192, fastinference_config={"profile": "throughput", "tuning_keyvals": {
                   "FASTINFERENCE_KV_MAX_ACTIVE_REQUESTS": str(batch), "FASTINFERENCE_LITE_PREFILL_MICROBATCH": "8",
-                  "FASTINFERENCE_GPU_GREEDY_SAMPLING": "0"}})
+                  "FASTINFERENCE_GPU_GREEDY_SAMPLING": "0", "FASTINFERENCE_PREFIX_CACHE_MAX_ENTRIES": "0"}})
     eng = llm.engine
     g = torch.Generator().manual_seed(1)
     ids = torch.randint(0, 32000, (batch, prompt), generator=g).tolist()

@@ -88,15 +88,12 @@ class LiteGpuBackend:
             self.observer.on_prefix_cache_event("store", n)
 
     # ------------------------------------------------------------------ steps
-    def run_prefills(self, plan: StepPlan) -> list:
-        if not plan.prefills:
-            return []
-        states = self.scheduler.requests
-        outs = self.drain_pipeline()
-        # exact prefix hits sample their first token from the cached logits without a forward pass
+    def _serve_exact_hits(self, prefills: list, outs: list) -> list:
+        """Exact prefix hits sample their first token from the cached logits without a forward pass; returns the items
+        that need one."""
         items = []
-        for it in plan.prefills:
-            st = states[it.request_id]
+        for it in prefills:
+            st = self.scheduler.requests[it.request_id]
             if st.cached_first_logits is not None and st.seq_len >= st.prompt_len:
                 tok = self.sampling.sample_batch_tokens(st.cached_first_logits[None].float(), [st])[0]
                 st.cached_first_logits = None
@@ -104,6 +101,14 @@ class LiteGpuBackend:
                 outs.append(self._process_completion(st, tok))
             else:
                 items.append(it)
+        return items
+
+    def run_prefills(self, plan: StepPlan) -> list:
+        if not plan.prefills:
+            return []
+        states = self.scheduler.requests
+        outs = self.drain_pipeline()
+        items = self._serve_exact_hits(plan.prefills, outs)
         if not items:
             return outs
         if self.mixed_batches:
@@ -139,7 +144,8 @@ class LiteGpuBackend:
         """One forward pass for the step's portions of prompts and its decoding requests."""
         states = self.scheduler.requests
         outs = self.drain_pipeline()
-        items = sorted((it for it in plan.prefills if it.chunk_len > 0), key=lambda it: -it.chunk_len)
+        items = sorted((it for it in self._serve_exact_hits(plan.prefills, outs) if it.chunk_len > 0),
+                       key=lambda it: -it.chunk_len)
         reqs = [states[r] for r in plan.decodes if r in states and not states[r].finished]
         n_prompt = len(items)
         for st in reqs:
@@ -158,6 +164,8 @@ class LiteGpuBackend:
             st.seq_len = it.end
             if st.is_prefill and st.seq_len < st.prompt_len:
                 continue
+            if st.is_prefill:
+                self._maybe_store_prefix(st, res.logits[row])
             st.is_prefill = False
             done_reqs.append(st)
             done_rows.append(row)

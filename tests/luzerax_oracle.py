@@ -157,3 +157,119 @@ def forward(cfg, w, tokens, collect=None, margins=None):
         if collect is not None:
             collect.append(x)
     return rms_norm(x, w["final.norm"], eps) @ w["head"].t()
+
+
+# ------------------------------------------------------------------ small random models
+def diff(heads, kv_heads, dim, vdim, mlp=None, init=0.35, temp=(0.6, 9), scale=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "diff": init, "scale": dim ** -0.5 if scale is None else scale}
+    if temp:
+        m["q_temp"] = {"coef": temp[0], "every": temp[1]}
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def gated(heads, kv_heads, dim, vdim, mlp=None, dims=None, base=10000.0, scale=4.0):
+    return {"type": "attention_2", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale * dim ** -0.5,
+                      "rot": {"base": base, "dims": dim if dims is None else dims}}}
+
+
+def plain(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts, identity, top, ff, count=1, keep=1, limit=1.2, shared=(24, 0.9)):
+    r = {"experts": experts, "identity": identity, "top": top, "groups": {"count": count, "keep": keep}}
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": r}
+    if shared:
+        mlp["shared"] = dict(zip(("ff", "limit"), shared))
+    return mlp
+
+
+def config(width, vocab, layers, eps=1e-6):
+    return {"architecture": "Luzerax", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers}
+
+
+def weights(cfg, seed=0, sharp=2.0):
+    """bf16-representable fp32 weights.  ``sharp`` widens attention scores so that single keys matter; clipping bounds are
+    often reached; corrections are as large as the scores they compete with, partly negative sums."""
+    g = torch.Generator().manual_seed(seed)
+    W, w = cfg["width"], {}
+
+    def put(name, *shape, std=1.0, base=0.0):
+        w[name] = (base + std * torch.randn(*shape, generator=g)).bfloat16().float()
+
+    def lin(name, out_f, in_f, gain=1.0):
+        put(name, out_f, in_f, std=gain * in_f ** -0.5)
+
+    def ff(p, inter):
+        for n, o, k in (("gate", inter, W), ("up", inter, W), ("down", W, inter)):
+            lin(p + n, o, k)
+
+    put("embed", cfg["vocab"], W)
+    for i, l in enumerate(cfg["layers"]):
+        p, m, mlp = f"l{i}.", l["mixer"], l["mlp"]
+        H, G, d, dv, maps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], 2 if l["type"] == "attention" else 1
+        for n in ("norm1", "ls1") + (("norm2", "ls2") if mlp else ()):
+            put(p + n, W, std=0.25, base=0.9)
+        lin(p + "mix.q", H * maps * d, W)
+        lin(p + "mix.k", G * maps * d, W)
+        lin(p + "mix.v", G * dv, W)
+        lin(p + "mix.o", W, H * dv)
+        if maps == 2:
+            put(p + "mix.q.norm", d, std=0.4, base=sharp)
+            put(p + "mix.k.norm", d, std=0.3, base=1.0)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                put(p + "mix." + n, d, std=0.6 * d ** -0.25)
+        else:
+            lin(p + "mix.g", H, W, 2.0)
+        if mlp and mlp["kind"] == "dense":
+            ff(p + "mlp.", mlp["ff"])
+        elif mlp:
+            r = mlp["router"]
+            for e in range(r["experts"]):
+                ff(f"{p}mlp.e{e}.", mlp["expert"]["ff"])
+            lin(p + "mlp.router", r["experts"] + r["identity"], W, 0.7)
+            put(p + "mlp.correction", r["experts"] + r["identity"], std=0.15, base=-0.2)
+            if mlp.get("shared"):
+                ff(p + "mlp.shared.", mlp["shared"]["ff"])
+    put("final.norm", W, std=0.2, base=1.0)
+    lin("head", cfg["vocab"], W, 2.0)
+    return w
+
+
+def save(folder, cfg, w):
+    from safetensors.torch import save_file
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(cfg))
+    save_file({k: v.bfloat16().contiguous() for k, v in w.items()}, str(folder / "model.safetensors"))
+    return str(folder)
+
+
+def greedy(cfg, w, prompt, n):
+    """Greedy continuation from scratch, and the smallest margin between the best two logits on the way."""
+    ids, margin = list(prompt), math.inf
+    for _ in range(n):
+        top = torch.topk(forward(cfg, w, ids)[-1], 2)
+        margin = min(margin, float(top.values[0] - top.values[1]))
+        ids.append(int(top.indices[0]))
+    return ids[len(prompt):], margin
+
+
+def errors(got, want):
+    """Per position: root mean square over the vocabulary of the difference (mean taken off), relative to the spread of
+    the logits."""
+    d = got.double().cpu() - want.double()
+    d = d - d.mean(-1, keepdim=True)
+    s = want.double() - want.double().mean(-1, keepdim=True)
+    return d.pow(2).mean(-1).sqrt() / s.pow(2).mean().sqrt()
+
+
+def fits(got, want, dtype, margins=None):
+    """32-bit runs agree everywhere; 16-bit ones up to rounding.  Positions where a router all but tied may go either way
+    in 16 bits and are left out (a position that such a token feeds moves a little)."""
+    e = errors(got, want)
+    if dtype == "float32":
+        return float(e.max()) < 1e-4
+    if margins is not None:
+        e = e[torch.tensor([m > 0.01 for m in margins])]
+    return e.numel() == 0 or (float(torch.quantile(e, 0.9)) < 0.08 and float(e.max()) < 0.3)
