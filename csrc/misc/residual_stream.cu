@@ -11,7 +11,7 @@
 //
 // The norm is an RMS norm over equal consecutive parts ("groups") of the vector, so a group of one token needs
 // nothing from any other group: the unit of work is a (token, group) row.  Steps with many tokens give a row to a
-// warp, steps with few tokens (decode) to a block, whose threads then fetch the whole history at once.
+// warp, steps with few tokens (decode) and long rows to a block, whose threads then fetch the whole history at once.
 // Rows keep their values in registers between the two norms: one read of y and x, one write of x and h.
 #include <cuda_bf16.h>
 #include <cuda_fp16.h>
@@ -107,14 +107,17 @@ __device__ __forceinline__ float row_sum(float v, float* red) {
   return v;
 }
 
+// Threads of a block whose rows take tpr threads each.
+constexpr int block_threads(int tpr) { return tpr > 256 ? tpr : 256; }
+
 template <int MODE, int TPR, int VEC, int NV, bool H16>
-__global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
+__global__ void __launch_bounds__(block_threads(TPR)) stream_kernel(const StreamParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
-  __shared__ float red[8];
-  constexpr int kRowsPerBlock = 256 / TPR;
-  const int row = blockIdx.x * kRowsPerBlock + (TPR == 256 ? 0 : static_cast<int>(threadIdx.x) / TPR);
-  const int tid = TPR == 256 ? threadIdx.x : threadIdx.x % TPR;
+  __shared__ float red[16];
+  constexpr int kRowsPerBlock = block_threads(TPR) / TPR;
+  const int row = blockIdx.x * kRowsPerBlock + (kRowsPerBlock == 1 ? 0 : static_cast<int>(threadIdx.x) / TPR);
+  const int tid = kRowsPerBlock == 1 ? threadIdx.x : threadIdx.x % TPR;
   if (row >= p.rows * p.groups) return;    // uniform over the threads of a row
   const int r = row / p.groups, g = row % p.groups;
   const long t = p.sel != nullptr ? static_cast<long>(p.sel[r]) : r;
@@ -215,15 +218,32 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
     }
 #pragma unroll
     for (int i = 0; i < NV * VEC; ++i) ss += v[i] * v[i];
+    if constexpr (MODE == kPost) {         // the weight is applied ahead of the reduction: less to do behind it
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * TPR + tid) * VEC;
+        if (c < p.group) {
+          float w[VEC];
+          load_any<VEC, false>(p.w_post, c0 + c, kFp32, w);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[i * VEC + e] *= w[e];
+        }
+      }
+    }
     const float inv = 1.f / sqrtf(row_sum<TPR>(ss, red) * inv_n + p.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
       if (c < p.group) {
-        float w[VEC];
-        load_any<VEC, false>(p.w_post, c0 + c, kFp32, w);
+        if constexpr (MODE == kPost) {
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(v[i * VEC + e] * inv, w[e], xv[i * VEC + e]);
+          for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(v[i * VEC + e], inv, xv[i * VEC + e]);
+        } else {
+          float w[VEC];
+          load_any<VEC, false>(p.w_post, c0 + c, kFp32, w);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(v[i * VEC + e] * inv, w[e], xv[i * VEC + e]);
+        }
       }
     }
     if constexpr (MODE == kAverage) {
@@ -294,12 +314,13 @@ __global__ void __launch_bounds__(256) stream_kernel(const StreamParams p) {
 template <int MODE, int TPR, int VEC, int NV>
 int launch(const StreamParams& p, cudaStream_t s) {
   const long rows = static_cast<long>(p.rows) * p.groups;
-  const long grid = (rows + 256 / TPR - 1) / (256 / TPR);
+  constexpr int threads = block_threads(TPR), per = threads / TPR;
+  const long grid = (rows + per - 1) / per;
   if (grid > 2147483647l) return -10;
   const dim3 g(static_cast<unsigned>(grid));
   if (p.h_type == kFp32)
-    return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV, false>, g, dim3(256), 0, s, 0, p));
-  return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV, true>, g, dim3(256), 0, s, 0, p));
+    return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV, false>, g, dim3(threads), 0, s, 0, p));
+  return static_cast<int>(fi::launch_kernel(stream_kernel<MODE, TPR, VEC, NV, true>, g, dim3(threads), 0, s, 0, p));
 }
 
 template <int MODE>
@@ -318,8 +339,14 @@ int dispatch(const StreamParams& p, bool vec4, cudaStream_t s) {
     if (g <= 512) return launch<MODE, 32, 4, 4>(p, s);
   }
   if (g <= 1024) return launch<MODE, 256, 4, 1>(p, s);
-  if (g <= 4096) return launch<MODE, 256, 4, 4>(p, s);
-  if (g <= 8192) return launch<MODE, 256, 4, 8>(p, s);
+  if (g <= 2048) return launch<MODE, 256, 4, 2>(p, s);
+  if constexpr (MODE == kPost) {      // everything it stores lies behind the reduction: more warps hide that
+    if (g <= 4096) return launch<MODE, 512, 4, 2>(p, s);
+    if (g <= 8192) return launch<MODE, 512, 4, 4>(p, s);
+  } else {
+    if (g <= 4096) return launch<MODE, 256, 4, 4>(p, s);
+    if (g <= 8192) return launch<MODE, 256, 4, 8>(p, s);
+  }
   return -11;
 }
 

@@ -34,126 +34,151 @@ namespace {
 
 constexpr int kMaxExpertsPerLane = 16;   // experts <= 512
 
+// Order-preserving map of scores to unsigned numbers above 0; what is no number (and whatever is out of the race) is 0.
+__device__ __forceinline__ unsigned score_key(float v) {
+  const unsigned u = __float_as_uint(v);
+  if ((u & 0x7fffffffu) > 0x7f800000u) return 0u;
+  return u ^ ((u >> 31) ? 0xffffffffu : 0x80000000u);
+}
+__device__ __forceinline__ float key_score(unsigned k) {
+  return __uint_as_float(k ^ ((k >> 31) ? 0x80000000u : 0xffffffffu));
+}
+
+// One warp per token; lane l owns experts l, l + 32, ... (PER of them, in registers).
+template <int PER>
 __global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
                                  const float* __restrict__ expert_scale, int* __restrict__ topk_ids,
                                  float* __restrict__ topk_w, long ld, int T, int E, int K, int mode,
                                  int renorm, float routed_scale, int groups, int keep_groups, int group_best) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
+  constexpr unsigned kAll = 0xffffffffu;
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (t >= T) return;
   const float* row = logits + t * ld;
-  float score[kMaxExpertsPerLane];   // value used for the weight
-  float sel[kMaxExpertsPerLane];     // value used for the selection
-  const int per = (E + 31) / 32;
+  float score[PER];     // value used for the weight
+  unsigned key[PER];    // value used for the selection
   float mx = -CUDART_INF_F;
-  for (int i = 0; i < per; ++i) {
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
-    const float v = e < E ? row[e] : -CUDART_INF_F;
-    score[i] = v;
-    mx = fmaxf(mx, v);
+    score[i] = e < E ? row[e] : -CUDART_INF_F;
+    mx = fmaxf(mx, score[i]);
   }
-  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   if (mode == 0) {
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(kAll, mx, o));
     float sum = 0.f;
-    for (int i = 0; i < per; ++i) {
-      const int e = i * 32 + lane;
-      score[i] = e < E ? __expf(score[i] - mx) : 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      score[i] = i * 32 + lane < E ? __expf(score[i] - mx) : 0.f;
       sum += score[i];
     }
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    for (int i = 0; i < per; ++i) {
-      const int e = i * 32 + lane;
-      score[i] /= sum;
-      sel[i] = e < E ? score[i] + (bias ? bias[e] : 0.f) : -CUDART_INF_F;
-    }
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(kAll, sum, o);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) score[i] /= sum;
   } else {
-    for (int i = 0; i < per; ++i) {
-      const int e = i * 32 + lane;
-      if (e < E) {
-        const float x = score[i];
-        score[i] = mode == 1 ? 1.f / (1.f + __expf(-x)) : sqrtf(x > 20.f ? x : log1pf(__expf(x)));
-        sel[i] = score[i] + (bias ? bias[e] : 0.f);
-      } else {
-        score[i] = 0.f;
-        sel[i] = -CUDART_INF_F;
-      }
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const float x = score[i];
+      score[i] = mode == 1 ? 1.f / (1.f + __expf(-x)) : sqrtf(x > 20.f ? x : log1pf(__expf(x)));
     }
   }
+#pragma unroll
+  for (int i = 0; i < PER; ++i) {
+    const int e = i * 32 + lane;
+    key[i] = e < E ? score_key(score[i] + (bias ? bias[e] : 0.f)) : 0u;
+  }
+  // the largest key among this warp's entries that `open` lets through and the lowest expert that has it
+  auto best_of = [&](auto open, int& expert) -> unsigned {
+    unsigned b = 0u;
+    int at = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (key[i] > b && open(i)) { b = key[i]; at = i * 32 + lane; }
+    const unsigned top = __reduce_max_sync(kAll, b);
+    expert = static_cast<int>(__reduce_min_sync(kAll, b == top ? static_cast<unsigned>(at) : 0x7fffffffu));
+    return top;
+  };
   if (keep_groups < groups) {
-    // score of group g ends in lane g % 32; ties go to the lower group
+    // kept groups are bits in registers: bit g & 31 of word g >> 5; ties go to the lower group
     const int size = E / groups;
-    float gscore[kMaxExpertsPerLane];
-    const int gper = (groups + 31) / 32;
-    for (int i = 0; i < gper; ++i) gscore[i] = -CUDART_INF_F;
-    for (int g = 0; g < groups; ++g) {
-      float m1 = -CUDART_INF_F, m2 = -CUDART_INF_F;          // the two largest of this lane's experts in the group
-      for (int i = 0; i < per; ++i) {
-        const int e = i * 32 + lane;
-        if (e >= g * size && e < (g + 1) * size) {
-          m2 = fmaxf(m2, fminf(m1, sel[i]));
-          m1 = fmaxf(m1, sel[i]);
-        }
+    unsigned kept[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) kept[i] = 0u;
+    auto is_kept = [&](int g) {
+      bool in = false;
+#pragma unroll
+      for (int w = 0; w < PER; ++w) in |= w == (g >> 5) && ((kept[w] >> (g & 31)) & 1u);
+      return in;
+    };
+    auto keep = [&](int g) {
+#pragma unroll
+      for (int w = 0; w < PER; ++w)
+        if (w == (g >> 5)) kept[w] |= 1u << (g & 31);
+    };
+    int group[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) group[i] = (i * 32 + lane) / size;
+    if (group_best < 2) {
+      // the best group left is the one of the best expert left
+      for (int k = 0; k < keep_groups; ++k) {
+        int e;
+        if (best_of([&](int i) { return !is_kept(group[i]); }, e) != 0u) keep(e / size);
       }
-      if (group_best < 2) {
-        for (int o = 16; o > 0; o >>= 1) m1 = fmaxf(m1, __shfl_xor_sync(0xffffffffu, m1, o));
-      } else {
+    } else {
+      float gscore[PER];                                       // score of group g ends in lane g % 32
+#pragma unroll
+      for (int i = 0; i < PER; ++i) gscore[i] = -CUDART_INF_F;
+      for (int g = 0; g < groups; ++g) {
+        float m1 = -CUDART_INF_F, m2 = -CUDART_INF_F;          // the two largest of this lane's experts in the group
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+          if (group[i] == g && key[i] != 0u) {
+            const float v = key_score(key[i]);
+            m2 = fmaxf(m2, fminf(m1, v));
+            m1 = fmaxf(m1, v);
+          }
+        }
         for (int o = 16; o > 0; o >>= 1) {
-          const float o1 = __shfl_xor_sync(0xffffffffu, m1, o), o2 = __shfl_xor_sync(0xffffffffu, m2, o);
+          const float o1 = __shfl_xor_sync(kAll, m1, o), o2 = __shfl_xor_sync(kAll, m2, o);
           m2 = fmaxf(fmaxf(m2, o2), fminf(m1, o1));
           m1 = fmaxf(m1, o1);
         }
+#pragma unroll
+        for (int w = 0; w < PER; ++w)
+          if (g == w * 32 + lane) gscore[w] = size > 1 ? m1 + m2 : m1;
       }
-      if ((g & 31) == lane) gscore[g >> 5] = group_best >= 2 && size > 1 ? m1 + m2 : m1;
-    }
-    unsigned kept[kMaxExpertsPerLane];                       // bit g & 31 of word g >> 5: the group may be chosen
-    for (int i = 0; i < gper; ++i) kept[i] = 0u;
-    for (int k = 0; k < keep_groups; ++k) {
-      float best = -CUDART_INF_F;
-      int bi = 0x7fffffff;
-      for (int i = 0; i < gper; ++i) {
-        const int g = i * 32 + lane;
-        if (g < groups && !((kept[i] >> (g & 31)) & 1u) && (gscore[i] > best || (gscore[i] == best && g < bi))) {
-          best = gscore[i];
-          bi = g;
+      for (int k = 0; k < keep_groups; ++k) {
+        unsigned b = 0u;
+        int at = 0x7fffffff;
+#pragma unroll
+        for (int w = 0; w < PER; ++w) {
+          const int g = w * 32 + lane;
+          const unsigned v = g < groups && !((kept[w] >> lane) & 1u) ? score_key(gscore[w]) : 0u;
+          if (v > b) { b = v; at = g; }
         }
+        const unsigned top = __reduce_max_sync(kAll, b);
+        const int g = static_cast<int>(__reduce_min_sync(kAll, b == top ? static_cast<unsigned>(at) : 0x7fffffffu));
+        if (top != 0u) keep(g);
       }
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-        if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
-      }
-      if (bi < groups) kept[bi >> 5] |= 1u << (bi & 31);
     }
-    for (int i = 0; i < per; ++i) {
-      const int e = i * 32 + lane, g = e / size;
-      if (e < E && !((kept[g >> 5] >> (g & 31)) & 1u)) sel[i] = -CUDART_INF_F;
-    }
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (!is_kept(group[i])) key[i] = 0u;
   }
   float wsum = 0.f;
   float my_w = 0.f;
   int my_id = 0;
   for (int k = 0; k < K; ++k) {
-    float best = -CUDART_INF_F;
-    int bi = 0x7fffffff;
-    for (int i = 0; i < per; ++i) {
-      const int e = i * 32 + lane;
-      if (sel[i] > best || (sel[i] == best && e < bi)) { best = sel[i]; bi = e; }
-    }
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
-    }
-    if (bi >= E) bi = 0;                                     // no comparable score left (a router output that is no number)
-    // owner lane reads the weight score and retires the expert
+    int bi;
+    if (best_of([](int) { return true; }, bi) == 0u) bi = 0;  // no comparable score left (a router output that is no number)
+    // the owner lane reads the weight score and retires the expert
     float w = 0.f;
-    if ((bi & 31) == lane) {
-      w = score[bi >> 5];
-      sel[bi >> 5] = -CUDART_INF_F;
-    }
-    w = __shfl_sync(0xffffffffu, w, bi & 31);
+#pragma unroll
+    for (int i = 0; i < PER; ++i)
+      if (i * 32 + lane == bi) { w = score[i]; key[i] = 0u; }
+    w = __shfl_sync(kAll, w, bi & 31);
     wsum += w;
     if (lane == k) { my_w = w; my_id = bi; }
   }
@@ -510,7 +535,9 @@ extern "C" int fi_moe_route(const float* logits, const float* bias, const float*
   if (E > 32 * kMaxExpertsPerLane || K > 32 || K > E || groups < 1 || E % groups != 0 || keep_groups < 1 ||
       keep_groups > groups || K > keep_groups * (E / groups) || ld < E || group_best < 1 || group_best > 2)
     return -10;
-  fi::launch_kernel(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, FI_STREAM(stream), 0, logits, bias,
+  auto kern = E <= 32 ? moe_route_kernel<1> : E <= 64 ? moe_route_kernel<2> : E <= 128 ? moe_route_kernel<4>
+              : E <= 256 ? moe_route_kernel<8> : moe_route_kernel<kMaxExpertsPerLane>;
+  fi::launch_kernel(kern, dim3((T + 3) / 4), dim3(128), 0, FI_STREAM(stream), 0, logits, bias,
                     expert_scale, topk_ids, topk_w, ld, T, E, K, mode, renorm, routed_scale, groups, keep_groups,
                     group_best);
   return static_cast<int>(cudaGetLastError());

@@ -189,7 +189,7 @@ def config(width, vocab, layers, eps=1e-6):
     return {"architecture": "Luzerax", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers}
 
 
-def weights(cfg, seed=0, sharp=2.0):
+def weights(cfg, seed=0, sharp=1.5):
     """bf16-representable fp32 weights.  ``sharp`` widens attention scores so that single keys matter; clipping bounds are
     often reached; corrections are as large as the scores they compete with, partly negative sums."""
     g = torch.Generator().manual_seed(seed)
@@ -265,11 +265,12 @@ def errors(got, want):
 
 
 def fits(got, want, dtype, margins=None):
-    """32-bit runs agree everywhere; 16-bit ones up to rounding.  Positions where a router all but tied may go either way
-    in 16 bits and are left out (a position that such a token feeds moves a little)."""
+    """32-bit runs agree everywhere, 16-bit ones up to rounding.  Without routers that is a tight bound.  Where a router all
+    but tied a 16-bit run may go either way: those positions are left out, and positions that such a token feeds move too."""
     e = errors(got, want)
     if dtype == "float32":
         return float(e.max()) < 1e-4
-    if margins is not None:
-        e = e[torch.tensor([m > 0.01 for m in margins])]
-    return e.numel() == 0 or (float(torch.quantile(e, 0.9)) < 0.08 and float(e.max()) < 0.3)
+    if margins is None or min(margins) == math.inf:
+        return float(torch.quantile(e, 0.9)) < 0.05 and float(e.max()) < 0.15
+    e = e[torch.tensor([m > 0.02 for m in margins])]
+    return e.numel() == 0 or (float(torch.quantile(e, 0.9)) < 0.12 and float(e.max()) < 0.6)
