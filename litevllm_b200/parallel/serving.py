@@ -55,7 +55,12 @@ class ServingCoordinator:
         self._new.append((st.request_id, list(st.prompt_token_ids), sampling_params_to_wire(st.sampling_params)))
 
     def record_abort(self, request_id: str) -> None:
-        self._aborts.append(request_id)
+        # a request that was never published is simply forgotten (workers apply aborts before admissions)
+        left = [r for r in self._new if r[0] != request_id]
+        if len(left) < len(self._new):
+            self._new = left
+        else:
+            self._aborts.append(request_id)
 
     def before_step(self, engine) -> bool:
         """Publish what changed and whether a step follows; returns that decision."""
@@ -75,7 +80,9 @@ class ServingCoordinator:
     def shutdown(self) -> None:
         if not self.closed:
             self.closed = True
-            self.channel.publish(ControlMessage(seq=0, step=False, shutdown=True))
+            # aborts since the last step travel with the last message: workers end with nothing running either
+            self.channel.publish(ControlMessage(seq=0, aborts=self._aborts, step=False, shutdown=True))
+            self._new, self._aborts = [], []
 
 
 def worker_serve_loop(engine, channel: ControlChannel, on_step=None) -> int:

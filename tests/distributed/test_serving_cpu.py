@@ -151,3 +151,23 @@ def test_mirrored_worker_follows_a_storm_of_clients():
     assert len(finished_all) >= 8 and all(rid in r0["tokens"] for rid in finished_all)
     for r in (r0, r1):
         assert r["running"] == 0 and r["free"] == r["total"] - 1
+
+
+def test_aborts_without_a_step_behind_them_still_reach_the_workers():
+    """A request that comes and goes between two steps is never published; an abort after the last step travels with the
+    shutdown message."""
+    from types import SimpleNamespace
+
+    from litevllm_b200 import SamplingParams
+    from litevllm_b200.parallel.serving import ServingCoordinator
+    sent = []
+    c = ServingCoordinator(SimpleNamespace(publish=sent.append))
+    busy = SimpleNamespace(has_unfinished_requests=lambda: True)
+    req = lambda rid: SimpleNamespace(request_id=rid, prompt_token_ids=[1], sampling_params=SamplingParams())
+    c.record_request(req("a"))
+    c.record_request(req("b"))
+    c.record_abort("a")
+    assert c.before_step(busy) and [r[0] for r in sent[0].new_requests] == ["b"] and sent[0].aborts == []
+    c.record_abort("b")
+    c.shutdown()
+    assert sent[1].shutdown and sent[1].aborts == ["b"] and not sent[1].step
