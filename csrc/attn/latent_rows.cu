@@ -276,7 +276,7 @@ struct RowsParams {
   FiAttnExtra x;            // sinks, output gate, two maps per head (the key row of a head is [map 1 | map 2])
 };
 
-template <typename T, int NV, int MAPS>
+template <typename T, int NV, int MAPS, bool SIG>
 __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -291,7 +291,7 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
   for (int i = lane; i < p.kd; i += 32) q[i] = to_f(qs[i]) * p.sm_scale;
   __syncwarp();
   const int len = min(p.row_lens[r], p.max_blocks * p.block_size);
-  const int lo = p.window > 0 ? max(0, len - p.window) : 0;
+  const int lo = SIG ? fi::first_key(p, max(0, len - 1)) : (p.window > 0 ? max(0, len - p.window) : 0);
   const int* bt = p.block_tables + static_cast<long>(p.seq_of_row ? p.seq_of_row[r] : r) * p.max_blocks;
   const T* cache = reinterpret_cast<const T*>(p.cache);
   const T* values = reinterpret_cast<const T*>(p.v_cache != nullptr ? p.v_cache : p.cache);
@@ -318,17 +318,22 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
         if (i < qd) a0 = fmaf(qm[i], to_f(row[i]), a0);
         s = a0 + a1;
       }
-      float mx = s;
-      for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-      const float nm = fmaxf(m, mx);            // at least one key of the chunk is visible
-      const float alpha = __expf(m - nm);
-      const float pv = __expf(s - nm);
-      float rs = pv;
-      for (int x = 16; x > 0; x >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, x);
-      l = l * alpha + rs;
-      m = nm;
+      float pv;
+      if constexpr (SIG) {
+        pv = tok < len ? 1.f / (1.f + __expf(-(s + p.x.bias[h]))) : 0.f;
+      } else {
+        float mx = s;
+        for (int x = 16; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+        const float nm = fmaxf(m, mx);            // at least one key of the chunk is visible
+        const float alpha = __expf(m - nm);
+        pv = __expf(s - nm);
+        float rs = pv;
+        for (int x = 16; x > 0; x >>= 1) rs += __shfl_xor_sync(0xffffffffu, rs, x);
+        l = l * alpha + rs;
+        m = nm;
 #pragma unroll
-      for (int i = 0; i < NV; ++i) o[i] *= alpha;
+        for (int i = 0; i < NV; ++i) o[i] *= alpha;
+      }
       const int n = min(32, len - k0);
       for (int j = 0; j < n; ++j) {
         const float pj = __shfl_sync(0xffffffffu, pv, j);
@@ -339,7 +344,7 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
       }
     }
     if (p.x.sinks != nullptr && m != -CUDART_INF_F) l += __expf(p.x.sinks[h * MAPS + map] - m);
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    const float inv = SIG ? 1.f : (l > 0.f ? 1.f / l : 0.f);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       o[i] *= inv;
@@ -361,6 +366,20 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const RowsParams p) {
     for (int i = 0; i < NV; ++i) o[i] *= f;
   }
   T* out = reinterpret_cast<T*>(p.out) + h * p.out_head_stride + r * p.out_row_stride;
+  if constexpr (SIG) {
+    if (p.x.turn != nullptr) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {           // neighbouring lanes hold the two channels of a pair
+        const float other = __shfl_xor_sync(0xffffffffu, o[i], 1);
+        const int d = i * 32 + lane;
+        if (d < p.vd) {
+          float u = lane & 1 ? other : o[i], v = lane & 1 ? o[i] : other;
+          fi::turn_back(p, len - 1, d >> 1, u, v);
+          o[i] = lane & 1 ? v : u;
+        }
+      }
+    }
+  }
 #pragma unroll
   for (int i = 0; i < NV; ++i)
     if (i * 32 + lane < p.vd) {
@@ -379,8 +398,9 @@ int launch_rows(const RowsParams& p, cudaStream_t s) {
   const dim3 grid(static_cast<unsigned>((items + 3) / 4));
   const int smem = 4 * p.kd * 4;
 #define FI_ROWS(N)                                                                                                         \
-  return static_cast<int>(p.x.maps == 2 ? fi::launch_kernel(latent_rows_kernel<T, N, 2>, grid, dim3(128), smem, s, 0, p)   \
-                                        : fi::launch_kernel(latent_rows_kernel<T, N, 1>, grid, dim3(128), smem, s, 0, p))
+  return static_cast<int>(p.x.bias != nullptr ? fi::launch_kernel(latent_rows_kernel<T, N, 1, true>, grid, dim3(128), smem, s, 0, p) \
+                          : p.x.maps == 2 ? fi::launch_kernel(latent_rows_kernel<T, N, 2, false>, grid, dim3(128), smem, s, 0, p)    \
+                                          : fi::launch_kernel(latent_rows_kernel<T, N, 1, false>, grid, dim3(128), smem, s, 0, p))
   if (p.vd <= 64) FI_ROWS(2);
   if (p.vd <= 128) FI_ROWS(4);
   if (p.vd <= 256) FI_ROWS(8);

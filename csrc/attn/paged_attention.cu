@@ -132,6 +132,28 @@ __device__ __forceinline__ void store_decoded(const AttnParams& p, int b, int he
   reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * od + d] = MmaT<T>::from_f(v);
 }
 
+// One channel of a finished row; get(row, channel, acc, l, m) gives its accumulated value, the sum of exponentials and their
+// reference.  SIG (weights without a softmax): the value stands as it is, and turns with its neighbour.
+template <typename T, int HD, bool SIG, typename F>
+__device__ __forceinline__ void finish_channel(const AttnParams& p, int b, int head, int r, int d, F get) {
+  float acc, l, m;
+  get(r, d, acc, l, m);
+  if constexpr (!SIG) {
+    store_decoded<T, HD>(p, b, head, d, acc, l, m);
+  } else {
+    if (d >= p.x.out_dim) return;
+    if (p.x.turn != nullptr) {
+      float other;
+      get(r, d ^ 1, other, l, m);
+      float u = d & 1 ? other : acc, v = d & 1 ? acc : other;
+      fi::turn_back(p, p.seq_lens[b] - 1, d >> 1, u, v);
+      acc = d & 1 ? v : u;
+    }
+    reinterpret_cast<T*>(p.out)[(static_cast<long>(b) * p.nh + head) * p.x.out_dim + d] =
+        MmaT<T>::from_f(acc * (p.kv_fp8 == 1 ? p.v_scale : 1.f));
+  }
+}
+
 // Two maps per head: one warp finishes query heads head and head + 1 (rows r and r + 1 of its tile).  get(row, channel,
 // acc, l, m) gives the accumulated value of a channel, the sum of exponentials and their reference.
 template <typename T, int HD, typename F>
@@ -246,7 +268,7 @@ __device__ __forceinline__ float softcap_f(float s, float cap) {
 // ------------------------------------------------------------------------------ decode
 // grid (splits, nkv * head_groups, B); 128 threads.  Rows of the 16-row tile = query heads of one
 // KV head (up to 16 per group).  Each warp owns 16 of the 64 tokens of a chunk.
-template <typename T, int HD>
+template <typename T, int HD, bool SIG>
 __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -266,7 +288,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
   const int head0 = kvh * G + grp * 16;
   const int seq_len = p.seq_lens[b];
   const int* bt = p.block_tables + static_cast<long>(b) * p.max_blocks;
-  const int lo = p.window > 0 ? max(0, seq_len - p.window) : 0;
+  const int lo = SIG ? fi::first_key(p, max(0, seq_len - 1)) : (p.window > 0 ? max(0, seq_len - p.window) : 0);
   const int first_chunk = lo / CH;
   const int n_chunks = (seq_len + CH - 1) / CH - first_chunk;
   const int per = (n_chunks + p.splits - 1) / p.splits;
@@ -288,6 +310,9 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
   for (int i = 0; i < HD / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
   const float scale = p.sm_scale * (p.kv_fp8 == 1 ? p.k_scale : 1.f);
+  [[maybe_unused]] const float bias0 = SIG && (lane >> 2) < heads_here ? p.x.bias[head0 + (lane >> 2)] : 0.f;
+  [[maybe_unused]] const float bias1 = SIG && (lane >> 2) + 8 < heads_here ? p.x.bias[head0 + (lane >> 2) + 8] : 0.f;
+  if constexpr (SIG) m0 = m1 = 0.f;        // shares of several warps or splits simply add up
 
   if (c_begin < c_end) {
     load_kv_tile<T, HD, CH, 128>(sK, p.k_cache, bt, p.block_size, p.nkv, kvh, c_begin * CH, lo, seq_len, p.kv_fp8, p.k_scales);
@@ -318,39 +343,51 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
         MmaT<T>::mma(s[0], a, kb);
         MmaT<T>::mma(s[1], a, kb + 2);
       }
-      float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
+      if constexpr (SIG) {
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
+        for (int j = 0; j < 2; ++j) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int tok = tok_base + j * 8 + (lane & 3) * 2 + (e & 1);
-          float v = softcap_f(s[j][e] * scale, p.softcap);
-          if (tok >= seq_len || tok < lo) v = -CUDART_INF_F;
-          s[j][e] = v;
-          if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+          for (int e = 0; e < 4; ++e) {
+            const int tok = tok_base + j * 8 + (lane & 3) * 2 + (e & 1);
+            const float w = fi::sigmoid_weight(fmaf(s[j][e], scale, e < 2 ? bias0 : bias1));
+            s[j][e] = tok >= seq_len || tok < lo ? 0.f : w;
+          }
         }
-      }
-      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-      const float nm0 = fmaxf(m0, mx0), nm1 = fmaxf(m1, mx1);
-      const float a0 = nm0 == -CUDART_INF_F ? 1.f : exp2f((m0 - nm0) * kLog2e);
-      const float a1 = nm1 == -CUDART_INF_F ? 1.f : exp2f((m1 - nm1) * kLog2e);
-      float rs0 = 0.f, rs1 = 0.f;
+      } else {
+        float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
+        for (int j = 0; j < 2; ++j) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float nm = e < 2 ? nm0 : nm1;
-          const float pv = nm == -CUDART_INF_F ? 0.f : exp2f((s[j][e] - nm) * kLog2e);
-          s[j][e] = pv;
-          if (e < 2) rs0 += pv; else rs1 += pv;
+          for (int e = 0; e < 4; ++e) {
+            const int tok = tok_base + j * 8 + (lane & 3) * 2 + (e & 1);
+            float v = softcap_f(s[j][e] * scale, p.softcap);
+            if (tok >= seq_len || tok < lo) v = -CUDART_INF_F;
+            s[j][e] = v;
+            if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+          }
         }
-      }
-      l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
+        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+        const float nm0 = fmaxf(m0, mx0), nm1 = fmaxf(m1, mx1);
+        const float a0 = nm0 == -CUDART_INF_F ? 1.f : exp2f((m0 - nm0) * kLog2e);
+        const float a1 = nm1 == -CUDART_INF_F ? 1.f : exp2f((m1 - nm1) * kLog2e);
+        float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-      for (int i = 0; i < HD / 8; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+        for (int j = 0; j < 2; ++j) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float nm = e < 2 ? nm0 : nm1;
+            const float pv = nm == -CUDART_INF_F ? 0.f : exp2f((s[j][e] - nm) * kLog2e);
+            s[j][e] = pv;
+            if (e < 2) rs0 += pv; else rs1 += pv;
+          }
+        }
+        l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
+#pragma unroll
+        for (int i = 0; i < HD / 8; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+      }
       uint32_t pa[4] = {MmaT<T>::pack(s[0][0], s[0][1]), MmaT<T>::pack(s[0][2], s[0][3]),
                         MmaT<T>::pack(s[1][0], s[1][1]), MmaT<T>::pack(s[1][2], s[1][3])};
 #pragma unroll
@@ -406,16 +443,16 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
   }
   for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
     const int r = i / HD, d = i % HD;
-    float acc, l, m;
-    merged(r, d, acc, l, m);
     const int head = head0 + r;
     if (p.splits == 1) {
-      store_decoded<T, HD>(p, b, head, d, acc, l, m);
-    } else {
-      const long base = (static_cast<long>(b) * p.nh + head) * p.splits + split;
-      p.ws_o[base * HD + d] = acc;
-      if (d == 0) { p.ws_ml[base * 2] = m; p.ws_ml[base * 2 + 1] = l; }
+      finish_channel<T, HD, SIG>(p, b, head, r, d, merged);
+      continue;
     }
+    float acc, l, m;
+    merged(r, d, acc, l, m);
+    const long base = (static_cast<long>(b) * p.nh + head) * p.splits + split;
+    p.ws_o[base * HD + d] = acc;
+    if (d == 0) { p.ws_ml[base * 2] = m; p.ws_ml[base * 2 + 1] = l; }
   }
 }
 
@@ -424,7 +461,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const AttnParams p) {
 // multi-stage cp.async pipeline over 16-token groups (one KV block slice each), so the main loop has
 // no CTA-wide barrier and each SM keeps tens of KB of KV reads in flight.  Block-table entries are
 // fetched 32 groups at a time into registers and handed out by shuffle.  Needs block_size % 16 == 0.
-template <typename T, int HD, int NST>
+template <typename T, int HD, int NST, bool SIG>
 __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -452,7 +489,7 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
   const int head0 = kvh * G + grp * 16;
   const int seq_len = p.seq_lens[b];
   const int* bt = p.block_tables + static_cast<long>(b) * p.max_blocks;
-  const int lo = p.window > 0 ? max(0, seq_len - p.window) : 0;
+  const int lo = SIG ? fi::first_key(p, max(0, seq_len - 1)) : (p.window > 0 ? max(0, seq_len - p.window) : 0);
   // 16-token groups of this CTA: [g_begin, g_end), dealt round-robin to the four warps
   const int first_g = lo / 16;
   const int n_groups = (seq_len + 15) / 16 - first_g;
@@ -476,6 +513,9 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
   for (int i = 0; i < HD / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m0 = -CUDART_INF_F, m1 = -CUDART_INF_F, l0 = 0.f, l1 = 0.f;
   const float scale = p.sm_scale * (fp8 ? p.k_scale : 1.f);
+  [[maybe_unused]] const float bias0 = SIG && (lane >> 2) < heads_here ? p.x.bias[head0 + (lane >> 2)] : 0.f;
+  [[maybe_unused]] const float bias1 = SIG && (lane >> 2) + 8 < heads_here ? p.x.bias[head0 + (lane >> 2) + 8] : 0.f;
+  if constexpr (SIG) m0 = m1 = 0.f;        // shares of several warps or splits simply add up
   const int bpb = p.block_size / 16;                 // 16-token groups per KV block
 
   int bt_reg = 0;
@@ -557,40 +597,52 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
       MmaT<T>::mma(s[0], a, kb);
       MmaT<T>::mma(s[1], a, kb + 2);
     }
-    float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
+    if constexpr (SIG) {
 #pragma unroll
-    for (int j = 0; j < 2; ++j) {
+      for (int j = 0; j < 2; ++j) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int tok = tok_base + j * 8 + (lane & 3) * 2 + (e & 1);
-        float v = softcap_f(s[j][e] * scale, p.softcap);
-        if (tok >= seq_len || tok < lo) v = -CUDART_INF_F;
-        s[j][e] = v;
-        if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+        for (int e = 0; e < 4; ++e) {
+          const int tok = tok_base + j * 8 + (lane & 3) * 2 + (e & 1);
+          const float w = fi::sigmoid_weight(fmaf(s[j][e], scale, e < 2 ? bias0 : bias1));
+          s[j][e] = tok >= seq_len || tok < lo ? 0.f : w;
+        }
       }
-    }
-    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-    const float nm0 = fmaxf(m0, mx0), nm1 = fmaxf(m1, mx1);
-    const float a0 = nm0 == -CUDART_INF_F ? 1.f : exp2f((m0 - nm0) * kLog2e);
-    const float a1 = nm1 == -CUDART_INF_F ? 1.f : exp2f((m1 - nm1) * kLog2e);
-    float rs0 = 0.f, rs1 = 0.f;
+    } else {
+      float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
 #pragma unroll
-    for (int j = 0; j < 2; ++j) {
+      for (int j = 0; j < 2; ++j) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float nm = e < 2 ? nm0 : nm1;
-        // tokens past seq_len inside a valid block hold stale cache data: their weight is exactly 0
-        const float pv = nm == -CUDART_INF_F ? 0.f : exp2f((s[j][e] - nm) * kLog2e);
-        s[j][e] = pv;
-        if (e < 2) rs0 += pv; else rs1 += pv;
+        for (int e = 0; e < 4; ++e) {
+          const int tok = tok_base + j * 8 + (lane & 3) * 2 + (e & 1);
+          float v = softcap_f(s[j][e] * scale, p.softcap);
+          if (tok >= seq_len || tok < lo) v = -CUDART_INF_F;
+          s[j][e] = v;
+          if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+        }
       }
-    }
-    l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+      const float nm0 = fmaxf(m0, mx0), nm1 = fmaxf(m1, mx1);
+      const float a0 = nm0 == -CUDART_INF_F ? 1.f : exp2f((m0 - nm0) * kLog2e);
+      const float a1 = nm1 == -CUDART_INF_F ? 1.f : exp2f((m1 - nm1) * kLog2e);
+      float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+      for (int j = 0; j < 2; ++j) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float nm = e < 2 ? nm0 : nm1;
+          // tokens past seq_len inside a valid block hold stale cache data: their weight is exactly 0
+          const float pv = nm == -CUDART_INF_F ? 0.f : exp2f((s[j][e] - nm) * kLog2e);
+          s[j][e] = pv;
+          if (e < 2) rs0 += pv; else rs1 += pv;
+        }
+      }
+      l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
+#pragma unroll
+      for (int i = 0; i < HD / 8; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+    }
     uint32_t pa[4] = {MmaT<T>::pack(s[0][0], s[0][1]), MmaT<T>::pack(s[0][2], s[0][3]),
                       MmaT<T>::pack(s[1][0], s[1][1]), MmaT<T>::pack(s[1][2], s[1][3])};
 #pragma unroll
@@ -642,12 +694,14 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
   }
   for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
     const int r = i / HD, d = i % HD;
-    float acc, l, m;
-    merged(r, d, acc, l, m);
     const int head = head0 + r;
     if (p.splits == 1) {
-      store_decoded<T, HD>(p, b, head, d, acc, l, m);
-    } else if (p.cluster_off > 0) {
+      finish_channel<T, HD, SIG>(p, b, head, r, d, merged);
+      continue;
+    }
+    float acc, l, m;
+    merged(r, d, acc, l, m);
+    if (p.cluster_off > 0) {
       float* cO = reinterpret_cast<float*>(smem_raw + p.cluster_off);
       cO[i] = acc;
       if (d == 0) { cO[16 * HD + r * 2] = m; cO[16 * HD + r * 2 + 1] = l; }
@@ -694,9 +748,7 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
       const int per = (E + p.splits - 1) / p.splits;
       const int i_end = min(E, (split + 1) * per);
       for (int i = split * per + threadIdx.x; i < i_end; i += 128) {
-        float acc, l, m;
-        gathered(i / HD, i % HD, acc, l, m);
-        store_decoded<T, HD>(p, b, head0 + i / HD, i % HD, acc, l, m);
+        finish_channel<T, HD, SIG>(p, b, head0 + i / HD, i / HD, i % HD, gathered);
       }
     }
     cluster.sync();
@@ -733,15 +785,13 @@ __global__ void __launch_bounds__(128) paged_decode_v2_kernel(const AttnParams p
         return;
       }
       for (int i = threadIdx.x; i < heads_here * HD; i += 128) {
-        float acc, l, m;
-        gathered(i / HD, i % HD, acc, l, m);
-        store_decoded<T, HD>(p, b, head0 + i / HD, i % HD, acc, l, m);
+        finish_channel<T, HD, SIG>(p, b, head0 + i / HD, i / HD, i % HD, gathered);
       }
     }
   }
 }
 
-template <typename T, int HD>
+template <typename T, int HD, bool SIG>
 __global__ void decode_merge_kernel(const AttnParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -764,9 +814,7 @@ __global__ void decode_merge_kernel(const AttnParams p) {
     return;
   }
   for (int d = threadIdx.x; d < HD; d += blockDim.x) {
-    float acc, l, m;
-    gathered(0, d, acc, l, m);
-    store_decoded<T, HD>(p, b, head, d, acc, l, m);
+    finish_channel<T, HD, SIG>(p, b, head, 0, d, gathered);
   }
 }
 
@@ -774,7 +822,7 @@ __global__ void decode_merge_kernel(const AttnParams p) {
 // grid (q_tiles, nh / MAPS, B); 128 threads; each warp owns 16 consecutive rows of the 64-row tile (a
 // row is a query token, or one of the MAPS = 2 maps of a token, side by side); KV streamed in CH-token
 // chunks shared by the four warps.
-template <typename T, int HD, int CH, int MAPS>
+template <typename T, int HD, int CH, int MAPS, bool SIG>
 __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -804,12 +852,14 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   }
   const int last_pos = pos0 + min(q_len, qt0 + kTokens) - 1;  // last query position of this tile
   const int first_pos = pos0 + qt0;
-  const int lo_tile = p.window > 0 ? max(0, first_pos - p.window + 1) : 0;
+  const int lo_tile = SIG ? fi::first_key(p, first_pos) : (p.window > 0 ? max(0, first_pos - p.window + 1) : 0);
   const int c_begin = lo_tile / CH;
   const int c_end = last_pos / CH + 1;
   const float scale = p.sm_scale * (p.kv_fp8 == 1 ? p.k_scale : 1.f);
   const int row0 = qt0 + (warp * 16 + (lane >> 2)) / MAPS;  // query index (within the sequence's new tokens)
   const int posr0 = pos0 + row0, posr1 = posr0 + 8 / MAPS;
+  [[maybe_unused]] const int lor0 = SIG ? fi::first_key(p, posr0) : 0, lor1 = SIG ? fi::first_key(p, posr1) : 0;
+  [[maybe_unused]] const float bias = SIG ? p.x.bias[head] : 0.f;
 
   float o[HD / 8][4];
 #pragma unroll
@@ -849,57 +899,69 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
         MmaT<T>::mma(s[2 * jp + 1], qa[ks], kb + 2);
       }
     }
-    float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
-    // chunks that lie entirely below every query row of this warp (and inside the window and the
-    // sequence) need no per-element mask
-    const bool interior = (c + 1) * CH - 1 <= posr0 && (c + 1) * CH <= seq_len &&
-                          (p.window <= 0 || c * CH > posr1 - p.window);
-    if (interior) {
-#pragma unroll
-      for (int j = 0; j < CH / 8; ++j) {
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float v = softcap_f(s[j][e] * scale, p.softcap);
-          s[j][e] = v;
-          if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
-        }
-      }
-    } else {
+    if constexpr (SIG) {
 #pragma unroll
       for (int j = 0; j < CH / 8; ++j) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int tok = c * CH + j * 8 + (lane & 3) * 2 + (e & 1);
-          const int pr = e < 2 ? posr0 : posr1;
-          float v = softcap_f(s[j][e] * scale, p.softcap);
-          const bool masked = tok > pr || tok >= seq_len || (p.window > 0 && tok <= pr - p.window);
-          if (masked) v = -CUDART_INF_F;
-          s[j][e] = v;
-          if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+          const float w = fi::sigmoid_weight(fmaf(s[j][e], scale, bias));
+          s[j][e] = tok > (e < 2 ? posr0 : posr1) || tok >= seq_len || tok < (e < 2 ? lor0 : lor1) ? 0.f : w;
         }
       }
-    }
-    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
-    mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
-    mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-    const float nm0 = fmaxf(m0, mx0), nm1 = fmaxf(m1, mx1);
-    const float a0 = nm0 == -CUDART_INF_F ? 1.f : exp2f((m0 - nm0) * kLog2e);
-    const float a1 = nm1 == -CUDART_INF_F ? 1.f : exp2f((m1 - nm1) * kLog2e);
-    float rs0 = 0.f, rs1 = 0.f;
+    } else {
+      float mx0 = -CUDART_INF_F, mx1 = -CUDART_INF_F;
+      // chunks that lie entirely below every query row of this warp (and inside the window and the
+      // sequence) need no per-element mask
+      const bool interior = (c + 1) * CH - 1 <= posr0 && (c + 1) * CH <= seq_len &&
+                            (p.window <= 0 || c * CH > posr1 - p.window);
+      if (interior) {
 #pragma unroll
-    for (int j = 0; j < CH / 8; ++j) {
+        for (int j = 0; j < CH / 8; ++j) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float nm = e < 2 ? nm0 : nm1;
-        const float pv = nm == -CUDART_INF_F ? 0.f : exp2f((s[j][e] - nm) * kLog2e);
-        s[j][e] = pv;
-        if (e < 2) rs0 += pv; else rs1 += pv;
+          for (int e = 0; e < 4; ++e) {
+            const float v = softcap_f(s[j][e] * scale, p.softcap);
+            s[j][e] = v;
+            if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < CH / 8; ++j) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int tok = c * CH + j * 8 + (lane & 3) * 2 + (e & 1);
+            const int pr = e < 2 ? posr0 : posr1;
+            float v = softcap_f(s[j][e] * scale, p.softcap);
+            const bool masked = tok > pr || tok >= seq_len || (p.window > 0 && tok <= pr - p.window);
+            if (masked) v = -CUDART_INF_F;
+            s[j][e] = v;
+            if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
+          }
+        }
       }
-    }
-    l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1));
+      mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1));
+      mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+      const float nm0 = fmaxf(m0, mx0), nm1 = fmaxf(m1, mx1);
+      const float a0 = nm0 == -CUDART_INF_F ? 1.f : exp2f((m0 - nm0) * kLog2e);
+      const float a1 = nm1 == -CUDART_INF_F ? 1.f : exp2f((m1 - nm1) * kLog2e);
+      float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-    for (int i = 0; i < HD / 8; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+      for (int j = 0; j < CH / 8; ++j) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float nm = e < 2 ? nm0 : nm1;
+          const float pv = nm == -CUDART_INF_F ? 0.f : exp2f((s[j][e] - nm) * kLog2e);
+          s[j][e] = pv;
+          if (e < 2) rs0 += pv; else rs1 += pv;
+        }
+      }
+      l0 = l0 * a0 + rs0; l1 = l1 * a1 + rs1; m0 = nm0; m1 = nm1;
+#pragma unroll
+      for (int i = 0; i < HD / 8; ++i) { o[i][0] *= a0; o[i][1] *= a0; o[i][2] *= a1; o[i][3] *= a1; }
+    }
 #pragma unroll
     for (int kt = 0; kt < CH / 16; ++kt) {
       uint32_t pa[4] = {MmaT<T>::pack(s[2 * kt][0], s[2 * kt][1]), MmaT<T>::pack(s[2 * kt][2], s[2 * kt][3]),
@@ -923,7 +985,7 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
     if (m1 != -CUDART_INF_F) l1 += exp2f((sink - m1) * kLog2e);
   }
   const float vs = p.kv_fp8 == 1 ? p.v_scale : 1.f;
-  const float i0 = l0 > 0.f ? vs / l0 : 0.f, i1 = l1 > 0.f ? vs / l1 : 0.f;
+  const float i0 = SIG ? vs : (l0 > 0.f ? vs / l0 : 0.f), i1 = SIG ? vs : (l1 > 0.f ? vs / l1 : 0.f);
   T* out = reinterpret_cast<T*>(p.out);
   const int od = p.x.out_dim;
   if constexpr (MAPS == 2) {
@@ -966,6 +1028,9 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
       const int row = row0 + 8 * h;
       if (row >= q_len) continue;
       float a = o[i][2 * h] * (h ? i1 : i0), bb = o[i][2 * h + 1] * (h ? i1 : i0);
+      if constexpr (SIG) {
+        if (p.x.turn != nullptr) fi::turn_back(p, h ? posr1 : posr0, d >> 1, a, bb);
+      }
       if (p.x.gate != nullptr) {
         const T* g = reinterpret_cast<const T*>(p.x.gate) + (q_begin + row) * p.x.gate_stride +
                      (p.x.gate_per_head ? head : head * od + d);
@@ -977,8 +1042,8 @@ __global__ void __launch_bounds__(128) paged_prefill_kernel(const AttnParams p) 
   }
 }
 
-template <typename T, int HD>
-int launch_decode(const AttnParams& p, int B, cudaStream_t s) {
+template <typename T, int HD, bool SIG>
+int launch_decode_as(const AttnParams& p, int B, cudaStream_t s) {
   const int G = p.nh / p.nkv;
   const int groups = (G + 15) / 16;
   if (p.block_size % 16 == 0 && p.kv_fp8 <= 1) {
@@ -994,7 +1059,7 @@ int launch_decode(const AttnParams& p, int B, cudaStream_t s) {
       pc.cluster_off = (smem + 127) & ~127;
       smem = pc.cluster_off + (16 * HD + 32) * 4;
     }
-    auto kern = paged_decode_v2_kernel<T, HD, NST>;
+    auto kern = paged_decode_v2_kernel<T, HD, NST, SIG>;
     cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
     if (ce != cudaSuccess) return static_cast<int>(ce);
     if (pc.cluster_off > 0) {
@@ -1006,7 +1071,7 @@ int launch_decode(const AttnParams& p, int B, cudaStream_t s) {
     const int kv_bytes = (16 * HD + 4 * 64 * HD) * 2;
     const int merge_bytes = (4 * 16 * HD + 4 * 16 * 2) * 4 + 16 * HD * 2;
     const int smem = kv_bytes > merge_bytes ? kv_bytes : merge_bytes;
-    auto kern = paged_decode_kernel<T, HD>;
+    auto kern = paged_decode_kernel<T, HD, SIG>;
     cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
     if (ce != cudaSuccess) return static_cast<int>(ce);
     fi::launch_kernel(kern, dim3(p.splits, p.nkv * groups, B), dim3(128), smem, s, 0, p);
@@ -1014,14 +1079,21 @@ int launch_decode(const AttnParams& p, int B, cudaStream_t s) {
   const bool merged_in_kernel = (p.merge_tickets != nullptr || (p.cluster_off != 0 && p.splits <= 8)) &&
                                 p.block_size % 16 == 0 && p.kv_fp8 <= 1;
   if (p.splits > 1 && !merged_in_kernel)
-    fi::launch_kernel(decode_merge_kernel<T, HD>, dim3(p.nh / p.x.maps, B), dim3(HD >= 128 ? 128 : 64), 0, s, 0, p);
+    fi::launch_kernel(decode_merge_kernel<T, HD, SIG>, dim3(p.nh / p.x.maps, B), dim3(HD >= 128 ? 128 : 64), 0, s, 0, p);
   return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T, int HD>
+int launch_decode(const AttnParams& p, int B, cudaStream_t s) {
+  return p.x.bias != nullptr ? launch_decode_as<T, HD, true>(p, B, s) : launch_decode_as<T, HD, false>(p, B, s);
 }
 
 template <typename T, int HD, int CH>
 int launch_prefill(const AttnParams& p, int B, int max_q_len, cudaStream_t s) {
   const int smem = (64 * HD + 4 * CH * HD) * 2;
-  auto kern = p.x.maps == 2 ? paged_prefill_kernel<T, HD, CH, 2> : paged_prefill_kernel<T, HD, CH, 1>;
+  auto kern = p.x.bias != nullptr ? paged_prefill_kernel<T, HD, CH, 1, true>
+              : p.x.maps == 2   ? paged_prefill_kernel<T, HD, CH, 2, false>
+                                : paged_prefill_kernel<T, HD, CH, 1, false>;
   cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
   if (ce != cudaSuccess) return static_cast<int>(ce);
   const int tokens = 64 / p.x.maps;

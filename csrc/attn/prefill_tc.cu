@@ -21,6 +21,9 @@
 // [q1 | 0] and [0 | q2] against key rows [k1 | k2] share every K and V tile, and the epilogue takes the difference of
 // neighbouring rows, its norm over the head's channels and the scale before it stores.
 //
+// Weights without a softmax (SIG): P = sigmoid(score + bias), the products of all tiles add up in one TMEM buffer, rows see
+// keys from the start of their chunk on, and pairs of output channels may turn by the row's position when they are stored.
+//
 // Masks (causal edge, sliding window, end of sequence) are applied only in tiles that touch an edge.
 // Every wait is bounded; a wait that runs out sets the status word and the CTA leaves through the
 // common teardown (TMEM freed).
@@ -79,7 +82,7 @@ __device__ __forceinline__ uint32_t pack2(float a, float b, int is_fp16) {
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-template <int HD, int STAGES, int MAPS>
+template <int HD, int STAGES, int MAPS, bool SIG>
 __global__ void __launch_bounds__(kTcThreads, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                   const __grid_constant__ CUtensorMap v_map, const TcParams p) {
@@ -110,7 +113,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   const int pos0 = seq_len - q_len;
   const int tokens = min(kTokens, q_len - qt0), rows = tokens * MAPS;
   const int first_pos = pos0 + qt0, last_pos = first_pos + tokens - 1;
-  const int kv_lo = p.window > 0 ? max(0, first_pos - p.window + 1) : 0;
+  const int kv_lo = SIG ? fi::first_key(p, first_pos) : (p.window > 0 ? max(0, first_pos - p.window + 1) : 0);
   const int tile_begin = kv_lo / kTile;
   const int n_tiles = last_pos / kTile + 1 - tile_begin;
   const int kvh = head / (p.nh / p.nkv);
@@ -273,10 +276,15 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           const uint32_t tp = tmem_base + (j & 1) * kTile + k * 8;
           // V: 16 keys = 16 rows of 128 bytes; the second 64 channels follow one 128-row block later
           const uint64_t dv = umma_desc_sw128_mnmajor(smem_u32(sV + st * L::kKV + k * 2048), kAtomBytes);
-          umma_f16_a_tmem(tmem_base + kPvCol + (j & 1) * HD, tp, dv, idesc_pv, k != 0 ? 1u : 0u);
+          if constexpr (SIG) umma_f16_a_tmem(tmem_base + kPvCol, tp, dv, idesc_pv, (k | j) != 0 ? 1u : 0u);
+          else umma_f16_a_tmem(tmem_base + kPvCol + (j & 1) * HD, tp, dv, idesc_pv, k != 0 ? 1u : 0u);
         }
         umma_commit(&v_empty[st]);
-        umma_commit(&pv_full[j & 1]);
+        if constexpr (SIG) {
+          if (j + 1 == n_tiles) umma_commit(&pv_full[0]);
+        } else {
+          umma_commit(&pv_full[j & 1]);
+        }
         if (j < 16) mark(p.trace, 131 + j * 4);
       }
       if (!ok) {
@@ -293,6 +301,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
     const int qpos = first_pos + row / MAPS;
     const float sl2 = p.sm_scale * kLog2e;
+    [[maybe_unused]] const int row_lo = SIG ? fi::first_key(p, qpos) : 0;                    // first key of this row
+    [[maybe_unused]] const int edge_lo = SIG ? fi::first_key(p, last_pos) : 0;               // and of the last one
+    [[maybe_unused]] const float nb = SIG ? -p.x.bias[head] * kLog2e : 0.f;
     const bool capped = p.softcap > 0.f;
     const float cap_in = capped ? p.sm_scale / p.softcap : 0.f, cap_out = p.softcap * kLog2e;
     float o[HH];
@@ -334,54 +345,78 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       if (j < 16) mark(tr, j * 8 + 1);
 
       const int k0 = (tile_begin + j) * kTile + half * 64;   // first key of this thread's 64
-      // keys of this half-tile the row may see: [vis_lo, vis_hi); only tiles on an edge look at them
-      const bool edge = (k0 + 63 > first_pos) || (p.window > 0 && k0 <= last_pos - p.window);
-      if (capped) {
-#pragma unroll
-        for (int e = 0; e < 64; ++e) sr[e] = __float_as_uint(fast_tanh(__uint_as_float(sr[e]) * cap_in));
-      }
-      if (edge) {
-        const int vis_hi = qpos - k0 + 1;
-        const int vis_lo = p.window > 0 ? qpos - p.window + 1 - k0 : 0;
+      float alpha = 1.f;
+      if constexpr (SIG) {
+        // weights 1 / (1 + e^-s), two at a time with one reciprocal; exponents are held where the product of two sums
+        // stays finite (a weight that small is zero beside any other)
 #pragma unroll
         for (int e = 0; e < 64; ++e)
-          if (e < vis_lo || e >= vis_hi) sr[e] = 0xff800000u;   // -inf: probability 0
-      }
-      float mt4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
+          sr[e] = __float_as_uint(1.f + fast_exp2(fminf(fmaf(__uint_as_float(sr[e]), -sl2, nb), 60.f)));
 #pragma unroll
-      for (int e = 0; e < 64; ++e) mt4[e & 3] = fmaxf(mt4[e & 3], __uint_as_float(sr[e]));
-      float mt = fmaxf(fmaxf(mt4[0], mt4[1]), fmaxf(mt4[2], mt4[3])) * to_log2;   // the factor is positive
-      half_max[(sb * 2 + half) * 128 + row] = mt;
-      if (j < 16) mark(tr, j * 8 + 2);
-      // after this meeting both halves hold their scores in registers: the buffer may take P
-      if (!pair_sync()) { ok = false; break; }
-      if (j < 16) mark(tr, j * 8 + 3);
-      mt = fmaxf(mt, half_max[(sb * 2 + (half ^ 1)) * 128 + row]);
-      const float m_new = fmaxf(m, mt);
-      const float m_use = m_new == -CUDART_INF_F ? 0.f : m_new;
-      const float alpha = fast_exp2(m - m_use);
+        for (int e = 0; e < 64; e += 2) {
+          const float a = __uint_as_float(sr[e]), c = __uint_as_float(sr[e + 1]), inv = __fdividef(1.f, a * c);
+          sr[e] = __float_as_uint(inv * c);
+          sr[e + 1] = __float_as_uint(inv * a);
+        }
+        if ((k0 + 63 > first_pos) || k0 < edge_lo) {
+          const int vis_hi = qpos - k0 + 1, vis_lo = row_lo - k0;
+#pragma unroll
+          for (int e = 0; e < 64; ++e)
+            if (e < vis_lo || e >= vis_hi) sr[e] = 0u;
+        }
+#pragma unroll
+        for (int e = 0; e < 64; e += 2) sr[e >> 1] = pack2(__uint_as_float(sr[e]), __uint_as_float(sr[e + 1]), p.is_fp16);
+        if (!pair_sync()) { ok = false; break; }     // both halves hold their scores in registers: the buffer may take P
+      } else {
+        // keys of this half-tile the row may see: [vis_lo, vis_hi); only tiles on an edge look at them
+        const bool edge = (k0 + 63 > first_pos) || (p.window > 0 && k0 <= last_pos - p.window);
+        if (capped) {
+#pragma unroll
+          for (int e = 0; e < 64; ++e) sr[e] = __float_as_uint(fast_tanh(__uint_as_float(sr[e]) * cap_in));
+        }
+        if (edge) {
+          const int vis_hi = qpos - k0 + 1;
+          const int vis_lo = p.window > 0 ? qpos - p.window + 1 - k0 : 0;
+#pragma unroll
+          for (int e = 0; e < 64; ++e)
+            if (e < vis_lo || e >= vis_hi) sr[e] = 0xff800000u;   // -inf: probability 0
+        }
+        float mt4[4] = {-CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F, -CUDART_INF_F};
+#pragma unroll
+        for (int e = 0; e < 64; ++e) mt4[e & 3] = fmaxf(mt4[e & 3], __uint_as_float(sr[e]));
+        float mt = fmaxf(fmaxf(mt4[0], mt4[1]), fmaxf(mt4[2], mt4[3])) * to_log2;   // the factor is positive
+        half_max[(sb * 2 + half) * 128 + row] = mt;
+        if (j < 16) mark(tr, j * 8 + 2);
+        // after this meeting both halves hold their scores in registers: the buffer may take P
+        if (!pair_sync()) { ok = false; break; }
+        if (j < 16) mark(tr, j * 8 + 3);
+        mt = fmaxf(mt, half_max[(sb * 2 + (half ^ 1)) * 128 + row]);
+        const float m_new = fmaxf(m, mt);
+        const float m_use = m_new == -CUDART_INF_F ? 0.f : m_new;
+        alpha = fast_exp2(m - m_use);
 
-      // probabilities, packed in place (two per register) and written over the first 64 columns of the
-      // S buffer: the A operand of P V, read from tensor memory
-      float rs0 = 0.f, rs1 = 0.f;
+        // probabilities, packed in place (two per register) and written over the first 64 columns of the
+        // S buffer: the A operand of P V, read from tensor memory
+        float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-      for (int e = 0; e < 64; e += 2) {
-        const float p0 = fast_exp2(fmaf(__uint_as_float(sr[e]), to_log2, -m_use));
-        const float p1 = fast_exp2(fmaf(__uint_as_float(sr[e + 1]), to_log2, -m_use));
-        rs0 += p0;
-        rs1 += p1;
-        sr[e >> 1] = pack2(p0, p1, p.is_fp16);
+        for (int e = 0; e < 64; e += 2) {
+          const float p0 = fast_exp2(fmaf(__uint_as_float(sr[e]), to_log2, -m_use));
+          const float p1 = fast_exp2(fmaf(__uint_as_float(sr[e + 1]), to_log2, -m_use));
+          rs0 += p0;
+          rs1 += p1;
+          sr[e >> 1] = pack2(p0, p1, p.is_fp16);
+        }
+        l = l * alpha + (rs0 + rs1);                   // this half's share of the denominator
+        m = m_new;
       }
-      l = l * alpha + (rs0 + rs1);                   // this half's share of the denominator
-      m = m_new;
       if (j < 16) mark(tr, j * 8 + 4);
       tmem_st_x32(t_lane + sb * kTile + half * 32, sr);
       tmem_st_wait();
       tc_fence_before();
       mbar_arrive(&p_full[sb]);
       if (j < 16) mark(tr, j * 8 + 5);
-      // fold the previous tile's product while the tensor core works on this one
-      if (j > 0) {
+      // fold the previous tile's product while the tensor core works on this one (SIG: products add up in tensor memory)
+      if (!SIG && j > 0) {
         if (!mbar_wait(&pv_full[(j - 1) & 1], ((j - 1) >> 1) & 1)) { ok = false; break; }
         if (j < 16) mark(tr, j * 8 + 6);
         tc_fence_after();
@@ -391,8 +426,17 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       if (j < 16) mark(tr, j * 8 + 7);
       alpha_prev = alpha;
     }
-    if (ok) ok = mbar_wait(&pv_full[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1);
-    if (ok) {
+    if constexpr (SIG) {
+      ok = ok && mbar_wait(&pv_full[0], 0);
+      if (ok) {
+        tc_fence_after();
+        fold_pv(0, 0.f);
+        l = 1.f;
+      }
+    } else if (ok) {
+      ok = mbar_wait(&pv_full[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1);
+    }
+    if (!SIG && ok) {
       tc_fence_after();
       fold_pv((n_tiles - 1) & 1, alpha_prev);
       half_sum[half * 128 + row] = l;
@@ -451,6 +495,11 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           float y[8];
 #pragma unroll
           for (int e = 0; e < 8; ++e) y[e] = o[c * 8 + e] * inv;
+          if constexpr (SIG) {
+            if (p.x.turn != nullptr)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) fi::turn_back(p, qpos, (half * HH + c * 8) / 2 + e, y[2 * e], y[2 * e + 1]);
+          }
           if (p.x.gate != nullptr && !p.x.gate_per_head) {
             const uint4 raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.x.gate) +
                                                               (q_begin + qt0 + row) * p.x.gate_stride + head * p.x.out_dim +
@@ -490,10 +539,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   }
 }
 
-template <int HD, int STAGES, int MAPS>
+template <int HD, int STAGES, int MAPS, bool SIG = false>
 int launch_tc(const CUtensorMap& qm, const CUtensorMap& km, const CUtensorMap& vm, const TcParams& p, int B,
               int max_q_len, cudaStream_t s) {
-  auto kern = prefill_tc_kernel<HD, STAGES, MAPS>;
+  auto kern = prefill_tc_kernel<HD, STAGES, MAPS, SIG>;
   constexpr int smem = TcSmem<HD, STAGES>::kBytes;
   cudaError_t ce = fi::ensure_dynamic_smem(kern, smem);
   if (ce != cudaSuccess) return static_cast<int>(ce);
@@ -550,6 +599,8 @@ extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_c
   p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window;
   p.sm_scale = sm_scale; p.softcap = softcap; p.is_fp16 = dtype == 1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (p.x.bias != nullptr)
+    return hd == 64 ? launch_tc<64, 6, 1, true>(qm, km, vm, p, B, max_q_len, s) : launch_tc<128, 3, 1, true>(qm, km, vm, p, B, max_q_len, s);
   if (hd == 64)
     return pairs ? launch_tc<64, 6, 2>(qm, km, vm, p, B, max_q_len, s) : launch_tc<64, 6, 1>(qm, km, vm, p, B, max_q_len, s);
   return pairs ? launch_tc<128, 3, 2>(qm, km, vm, p, B, max_q_len, s) : launch_tc<128, 3, 1>(qm, km, vm, p, B, max_q_len, s);

@@ -1,6 +1,8 @@
 // Queries, keys and values of one step from a merged projection [q (H * dim) | k (G * dim) | ..]:
 //
-//   q' = R(pos) rmsnorm(q) over all H * dim channels,   k' = R(pos) rmsnorm(k) over all G * dim channels,   v = k
+//   q' = R(pos) rmsnorm(q) over all H * dim channels,   k' = R(pos) rmsnorm(k) over all G * dim channels,
+//   v = k, or a projection of its own [.. | v (G * vdim)] whose channels 2 i and 2 i + 1 may turn by angle i of a second
+//   table (over all vdim channels)
 //
 // Keys and values go to their paged caches, queries to rows the attention kernels read; heads are padded with zeros
 // from dim to the kernels' head size.  The rotation turns channels i and i + dims / 2 of a head (i < dims / 2) by the
@@ -37,6 +39,8 @@ struct QkParams {
   long ld;
   int H, G, dim, hd, dims, block_size, max_pos, vec;
   float eps;
+  int v_off, vdim, vp;      // v_off > 0: values start there; vp: row pitch of the value cache
+  const float* v_cs;        // [max_pos, vdim] or null
 };
 
 template <typename T>
@@ -89,7 +93,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
     const float inv = is_k ? ik : iq;
     T* dst = is_k ? reinterpret_cast<T*>(p.k_cache) + ((blk * p.G + h - p.H) * p.block_size + off) * p.hd
                   : reinterpret_cast<T*>(p.q_out) + (static_cast<long>(t) * p.H + h) * p.hd;
-    T* vdst = is_k ? reinterpret_cast<T*>(p.v_cache) + ((blk * p.G + h - p.H) * p.block_size + off) * p.hd : nullptr;
+    T* vdst = is_k && p.v_off == 0 ? reinterpret_cast<T*>(p.v_cache) + ((blk * p.G + h - p.H) * p.block_size + off) * p.hd : nullptr;
     if (p.vec) {
       const int c = (i % per) * V;
       alignas(16) T x[V], y[V], o[V];
@@ -112,7 +116,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
         }
       }
       *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(o);
-      if (is_k) *reinterpret_cast<uint4*>(vdst + c) = *reinterpret_cast<const uint4*>(x);
+      if (vdst != nullptr) *reinterpret_cast<uint4*>(vdst + c) = *reinterpret_cast<const uint4*>(x);
     } else {
       const int c = i % per;
       T x = from_f<T>(0.f);
@@ -128,29 +132,71 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
         }
       }
       dst[c] = from_f<T>(a);
-      if (is_k) vdst[c] = x;
+      if (vdst != nullptr) vdst[c] = x;
+    }
+  }
+  if (p.v_off == 0 || slot < 0) return;
+  const float* vcs = p.v_cs != nullptr ? p.v_cs + static_cast<long>(pos) * p.vdim : nullptr;
+  T* v0 = reinterpret_cast<T*>(p.v_cache);
+  if (p.vec) {
+    const int vper = p.vp / V;
+    for (int i = tid; i < p.G * vper; i += 256) {
+      const int g = i / vper, c = (i % vper) * V;
+      alignas(16) T x[V];
+      *reinterpret_cast<uint4*>(x) = make_uint4(0, 0, 0, 0);
+      if (c < p.vdim) {
+        *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(row + p.v_off + g * p.vdim + c);
+        if (vcs != nullptr) {
+#pragma unroll
+          for (int e = 0; e < V; e += 2) {
+            const float a = to_f(x[e]), bb = to_f(x[e + 1]), cc = vcs[(c + e) / 2], ss = vcs[(p.vdim + c + e) / 2];
+            x[e] = from_f<T>(a * cc - bb * ss);
+            x[e + 1] = from_f<T>(bb * cc + a * ss);
+          }
+        }
+      }
+      *reinterpret_cast<uint4*>(v0 + ((blk * p.G + g) * p.block_size + off) * p.vp + c) = *reinterpret_cast<const uint4*>(x);
+    }
+  } else {
+    for (int i = tid; i < p.G * p.vp; i += 256) {
+      const int g = i / p.vp, c = i % p.vp;
+      float a = 0.f;
+      if (c < p.vdim) {
+        const T* src = row + p.v_off + g * p.vdim;
+        a = to_f(src[c]);
+        if (vcs != nullptr) {
+          const float bb = to_f(src[c ^ 1]), cc = vcs[c / 2], ss = vcs[p.vdim / 2 + c / 2];
+          a = c & 1 ? a * cc + bb * ss : a * cc - bb * ss;
+        }
+      }
+      v0[((blk * p.G + g) * p.block_size + off) * p.vp + c] = from_f<T>(a);
     }
   }
 }
 
 }  // namespace
 
-// dtype: 0 bf16, 1 fp16, 2 fp32 (projection, queries, caches).  Slots >= 0 must lie inside the caches.
+// dtype: 0 bf16, 1 fp16, 2 fp32 (projection, queries, caches).  Slots >= 0 must lie inside the caches.  v_off 0: the value is
+// the key's projection (vdim, vp and v_cs unused); otherwise values are G heads of vdim channels from column v_off on, in
+// cache rows of vp channels, turned by v_cs [max_pos, vdim] unless that is null.
 extern "C" int fi_qk_prepare(const void* proj, long ld, const float* wq, const float* wk, float eps, const int* positions,
                              const float* cos_sin, int max_pos, const int* slot_mapping, void* q_out, void* k_cache,
-                             void* v_cache, int T, int H, int G, int dim, int hd, int dims, int block_size, int dtype,
-                             void* stream) {
+                             void* v_cache, int T, int H, int G, int dim, int hd, int dims, int block_size, int v_off, int vdim,
+                             int vp, const float* v_cs, int dtype, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || dim <= 0 || hd < dim || dims < 0 || dims > dim || dims % 2 != 0 || block_size <= 0 || max_pos <= 0)
     return -10;
+  if (v_off != 0 && (v_off < (H + G) * dim || vdim <= 0 || vp < vdim || (v_cs != nullptr && vdim % 2 != 0))) return -10;
   QkParams p = {};
+  p.v_off = v_off; p.vdim = vdim; p.vp = vp; p.v_cs = v_cs;
   p.proj = proj; p.wq = wq; p.wk = wk; p.positions = positions; p.cos_sin = cos_sin; p.slot_mapping = slot_mapping;
   p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache; p.ld = ld; p.H = H; p.G = G; p.dim = dim; p.hd = hd;
   p.dims = dims; p.block_size = block_size; p.max_pos = max_pos; p.eps = eps;
   const int v = dtype == 2 ? 4 : 8;
   const uintptr_t at = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out) |
                        reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
-  p.vec = dim % v == 0 && hd % v == 0 && (dims / 2) % v == 0 && ld % v == 0 && (at & 15) == 0;
+  p.vec = dim % v == 0 && hd % v == 0 && (dims / 2) % v == 0 && ld % v == 0 && (at & 15) == 0 &&
+          (v_off == 0 || (v_off % v == 0 && vdim % v == 0 && vp % v == 0));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == 0) return static_cast<int>(fi::launch_kernel(qk_prepare_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, s, 0, p));
   if (dtype == 1) return static_cast<int>(fi::launch_kernel(qk_prepare_kernel<__half>, dim3(T), dim3(256), 0, s, 0, p));

@@ -68,6 +68,8 @@ __device__ __forceinline__ float act_f(float g, int act) {
     return g / (1.f + __expf(-2.f * inner));
   }
   if (act == 3) return fmaxf(g, 0.f);
+  if (act == 5) { g = fmaxf(g, 0.f); return g * g; }
+  if (act == 6) return 1.f - 2.f / (1.f + __expf(2.f * g));
   return g;
 }
 // Gated form of one channel: act(g) * u; 4: bounds on both halves (g from above only), g sigmoid(1.702 g) * (u + 1).

@@ -34,7 +34,7 @@ constexpr int kXferTwoShot = 3;      // all-reduce in two hops: partials go to t
 constexpr int kPhasePush = 1, kPhaseReduce = 2, kPhaseCollect = 4;
 constexpr int kMaxCommTiles = 8192; // tiles per call that the flag area can describe
 
-enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2, kActRelu = 3, kActClippedSwiglu = 4 };
+enum Act : int { kActNone = 0, kActSilu = 1, kActGeluTanh = 2, kActRelu = 3, kActClippedSwiglu = 4, kActRelu2 = 5, kActTanh = 6 };
 enum CommMode : int { kCommNone = 0, kCommAllReduce = 1, kCommReduceScatter = 2 };
 
 struct GemmParams {
@@ -113,6 +113,8 @@ __device__ __forceinline__ float apply_act(float g, int act) {
     return g / (1.f + __expf(-2.f * inner));
   }
   if (act == kActRelu) return fmaxf(g, 0.f);
+  if (act == kActRelu2) { g = fmaxf(g, 0.f); return g * g; }
+  if (act == kActTanh) return 1.f - 2.f / (1.f + __expf(2.f * g));
   return g;
 }
 

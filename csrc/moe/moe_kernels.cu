@@ -254,6 +254,19 @@ __global__ void moe_align_kernel(const int* __restrict__ topk_ids, int n_routes,
   }
 }
 
+// Experts that a table assigns to token ids, all with the same weight.
+__global__ void __launch_bounds__(256) moe_lookup_kernel(const int* __restrict__ table, const long long* __restrict__ ids, int vocab,
+                                                         int n, int top, float weight, int* __restrict__ topk_ids,
+                                                         float* __restrict__ topk_w) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i >= n) return;
+  const long long id = ids[i / top];
+  topk_ids[i] = table[(id < 0 || id >= vocab ? 0 : id) * top + i % top];     // padded rows of a decode bucket carry stale ids
+  topk_w[i] = weight;
+}
+
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ sorted_route,
                                   const int* __restrict__ expert_offsets, int EL, int K, int H,
@@ -541,6 +554,15 @@ extern "C" int fi_moe_route(const float* logits, const float* bias, const float*
                     expert_scale, topk_ids, topk_w, ld, T, E, K, mode, renorm, routed_scale, groups, keep_groups,
                     group_best);
   return static_cast<int>(cudaGetLastError());
+}
+
+// topk_ids, topk_w [T, top] = table [vocab, top] rows of the token ids, each choice with `weight`.
+extern "C" int fi_moe_lookup(const int* table, const long long* ids, int vocab, int T, int top, float weight, int* topk_ids,
+                             float* topk_w, void* stream) {
+  if (T <= 0) return 0;
+  if (vocab <= 0 || top <= 0 || static_cast<long>(T) * top > 2147483647l) return -10;
+  return static_cast<int>(fi::launch_kernel(moe_lookup_kernel, dim3((T * top + 255) / 256), dim3(256), 0, FI_STREAM(stream), 0, table,
+                                            ids, vocab, T * top, top, weight, topk_ids, topk_w));
 }
 
 extern "C" int fi_moe_align(const int* topk_ids, int n_routes, int e_lo, int e_hi, int bn,

@@ -78,6 +78,9 @@ KERNEL_SETS = {
     "luzerax": ["attn/head_prepare.cu", "attn/latent_rows.cu", "attn/paged_attention.cu", "attn/prefill_tc.cu",
                 "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "misc/norm_rope_misc.cu", "misc/residual_stream.cu",
                 "misc/sampling.cu", "moe/moe_kernels.cu"],
+    "divadra": ["attn/latent_rows.cu", "attn/paged_attention.cu", "attn/prefill_tc.cu", "attn/qk_prepare.cu",
+                "gemm/dense_gemm.cu", "gemm/dense_gemm_persistent.cu", "linear_attn/decay_scan.cu", "misc/norm_rope_misc.cu",
+                "misc/sampling.cu", "misc/shift_stream.cu", "moe/moe_kernels.cu"],
 }
 
 

@@ -25,6 +25,8 @@ class KVLayerSpec:
     v_head_dim: int | None = None     # MLA-style caches may use another width for V (0 = no V)
     state_shape: tuple | None = None  # recurrent layers: shape of the fp32 state a request slot owns
     ring_shape: tuple | None = None   # short convolutions: fp32 rows of recent inputs a request slot owns
+    input_shape: tuple | None = None  # the same for a convolution in front of the layer's sublayers
+    last_token: bool = False          # the model reads a sequence's previous token (one number per request slot)
 
     @property
     def v_dim(self) -> int:
@@ -32,7 +34,7 @@ class KVLayerSpec:
 
     @property
     def state_bytes(self) -> int:
-        return 4 * sum(math.prod(s) for s in (self.state_shape, self.ring_shape) if s)
+        return 4 * (sum(math.prod(s) for s in (self.state_shape, self.ring_shape, self.input_shape) if s) + int(self.last_token))
 
 
 def kv_torch_dtype(kv_cache_dtype: str, model_dtype: torch.dtype) -> torch.dtype:
@@ -66,7 +68,8 @@ class FlatKVCache:
     def __init__(self, specs: list[KVLayerSpec], num_blocks: int, block_size: int,
                  dtype: torch.dtype, device: torch.device, fmt: int = 0, num_slots: int = 0):
         """``num_slots``: request slots of the engine; recurrent layers (``state_shape``) get one fp32 state per slot
-        in ``states[layer]``, layers with short convolutions (``ring_shape``) their recent inputs in ``rings[layer]``.
+        in ``states[layer]``, layers with short convolutions (``ring_shape``, ``input_shape``) their recent inputs in
+        ``rings[layer]`` and ``inputs[layer]``; ``last_tokens`` (int32) holds a token per slot if a layer asks for it.
         A slot's state is not cleared when it changes hands: a sequence that starts at position 0 starts from a zero
         state and zero inputs."""
         self.specs, self.num_blocks, self.block_size = specs, num_blocks, block_size
@@ -102,12 +105,14 @@ class FlatKVCache:
             return torch.zeros(num_slots, *shape, dtype=torch.float32, device=device) if shape else None
         self.states: list[torch.Tensor | None] = [per_slot(s.state_shape) for s in specs]
         self.rings: list[torch.Tensor | None] = [per_slot(s.ring_shape) for s in specs]
+        self.inputs: list[torch.Tensor | None] = [per_slot(s.input_shape) for s in specs]
+        self.last_tokens = torch.zeros(num_slots, dtype=torch.int32, device=device) if any(s.last_token for s in specs) else None
         self.state_bytes = sum(t.numel() * 4 for t in self.slot_tensors())
         self.total_bytes += self.state_bytes
 
     def slot_tensors(self) -> list[torch.Tensor]:
         """Everything indexed by request slot that a step advances."""
-        return [t for t in (*self.states, *self.rings) if t is not None]
+        return [t for t in (*self.states, *self.rings, *self.inputs, self.last_tokens) if t is not None]
 
     def __getitem__(self, i: int):
         return self.layers[i]

@@ -45,3 +45,35 @@ class RoutedExperts(nn.Module):
                            routed_scale=self.scale, groups=self.groups, keep_groups=self.keep,
                            group_best=self.group_best)
         return moe.expert_rows(x, self.w_gate_up, self.w_down, ids, w, self.act, self.act_limit, self.outputs > self.E)
+
+
+class AssignedExperts(nn.Module):
+    """The same experts without a router: a table gives every token id its ``top`` experts, each of weight 1 / top."""
+
+    def __init__(self, hidden: int, inter: int, experts: int, top: int, vocab: int, dtype, act: str = "silu"):
+        super().__init__()
+        self.E, self.top, self.act, self.inter = experts, top, act, inter
+        self.w_gate_up = nn.Parameter(torch.empty(experts, 2 * inter, hidden, dtype=dtype), requires_grad=False)
+        self.w_down = nn.Parameter(torch.empty(experts, hidden, inter, dtype=dtype), requires_grad=False)
+        self.table = nn.Parameter(torch.zeros(vocab, top, dtype=torch.int32), requires_grad=False)
+
+    def _take_table(self, tensor: torch.Tensor) -> None:
+        if tuple(tensor.shape) != tuple(self.table.shape):
+            raise ValueError(f"expert table has shape {tuple(tensor.shape)}, the configuration asks for {tuple(self.table.shape)}")
+        if tensor.is_floating_point() or int(tensor.min()) < 0 or int(tensor.max()) >= self.E:
+            raise ValueError(f"expert tables hold integers below {self.E}")
+        self.table.data.copy_(tensor.to(torch.int32))
+
+    def destinations(self, prefix: str) -> dict:
+        """Checkpoint name -> where its values go."""
+        d = {prefix + "table": self._take_table}
+        for e in range(self.E):
+            d[f"{prefix}e{e}.gate"] = self.w_gate_up[e, :self.inter]
+            d[f"{prefix}e{e}.up"] = self.w_gate_up[e, self.inter:]
+            d[f"{prefix}e{e}.down"] = self.w_down[e]
+        return d
+
+    def forward(self, x, token_ids) -> moe.RoutedRows:
+        """x [T, hidden], token_ids int64 [T]."""
+        ids, w = moe.lookup(self.table, token_ids, 1.0 / self.top)
+        return moe.expert_rows(x, self.w_gate_up, self.w_down, ids, w, self.act)

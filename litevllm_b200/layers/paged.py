@@ -18,7 +18,7 @@ def tensor_head_size(dtype, *widths: int) -> int:
     return next(hd for hd in (64, 128, 256) if max(widths) <= hd)
 
 
-def _portions(q, k_cache, v_cache, batch, nh, nkv, hd, scale, window, sinks, v_dim, gate, diff):
+def _portions(q, k_cache, v_cache, batch, nh, nkv, hd, scale, window, sinks, v_dim, gate, diff, sigmoid):
     """Varlen portions on the tensor-core kernels; long ones (at the front of the step) and short ones apart."""
     n = 0
     for m in batch.q_lens_cpu:
@@ -38,24 +38,26 @@ def _portions(q, k_cache, v_cache, batch, nh, nkv, hd, scale, window, sinks, v_d
                 cu = batch.extras["short_cu"] = (batch.cu_q[lo:hi + 1] - t).contiguous()
         ops.paged_attention_prefill(q[a:e].view(e - a, -1), k_cache, v_cache, batch.block_tables[lo:hi], batch.seq_lens[lo:hi],
                                     cu, max(batch.q_lens_cpu[lo:hi]), nh, nkv, hd, scale, window, out=out[a:e], sinks=sinks,
-                                    v_dim=v_dim, gate=None if gate is None else gate[a:e], diff=diff)
+                                    v_dim=v_dim, gate=None if gate is None else gate[a:e], diff=diff, sigmoid=sigmoid)
     return out
 
 
-def attend(q, kv, batch, nkv: int, scale: float, window: int, v_dim: int, tensor: bool, sinks=None, gate=None, diff=None):
+def attend(q, kv, batch, nkv: int, scale: float, window: int, v_dim: int, tensor: bool, sinks=None, gate=None, diff=None,
+           sigmoid=None):
     """q [T, query heads, row] of :mod:`ops.qk_attn`; kv: the layer's key and value pages; ``tensor``: rows are padded for
-    the tensor-core kernels.  Returns [T, heads * v_dim]; ``sinks``, ``gate``, ``diff`` as in ``ops.paged_attention_decode``."""
+    the tensor-core kernels.  Returns [T, heads * v_dim]; ``sinks``, ``gate``, ``diff``, ``sigmoid`` as in ``ops.paged_attention_decode``."""
     k_cache, v_cache = kv
     T, nh, hd = q.shape
     if q.is_cuda and tensor:
         if batch.is_decode:
-            tables, lens = batch.attention_tables(window)
+            tables, lens = batch.attention_tables(window or (sigmoid.chunk if sigmoid is not None else 0))
             return ops.paged_attention_decode(q.view(T, -1), k_cache, v_cache, tables, lens, nh, nkv, hd, scale, window,
-                                              max_kv_len=batch.max_kv_len, sinks=sinks, v_dim=v_dim, gate=gate, diff=diff)
-        return _portions(q, k_cache, v_cache, batch, nh, nkv, hd, scale, window, sinks, v_dim, gate, diff)
+                                              max_kv_len=batch.max_kv_len, sinks=sinks, v_dim=v_dim, gate=gate, diff=diff,
+                                              sigmoid=sigmoid)
+        return _portions(q, k_cache, v_cache, batch, nh, nkv, hd, scale, window, sinks, v_dim, gate, diff, sigmoid)
     tables, lens, seq = batch.block_tables, batch.seq_lens, None
     if batch.is_decode:
-        tables, lens = batch.attention_tables(window)
+        tables, lens = batch.attention_tables(window or (sigmoid.chunk if sigmoid is not None else 0))
     else:
         rows = batch.extras.get("token_rows")
         if rows is None:
@@ -63,4 +65,4 @@ def attend(q, kv, batch, nkv: int, scale: float, window: int, v_dim: int, tensor
             seq = torch.searchsorted(batch.cu_q[1:].contiguous(), tok, right=True).to(torch.int32)
             rows = batch.extras["token_rows"] = ((batch.positions + 1).to(torch.int32), seq)
         lens, seq = rows
-    return qk_attn.attend_rows(q, k_cache, v_cache, tables, lens, seq, scale, window, sinks, gate, v_dim, diff)
+    return qk_attn.attend_rows(q, k_cache, v_cache, tables, lens, seq, scale, window, sinks, gate, v_dim, diff, sigmoid)

@@ -65,6 +65,8 @@ def synthetic_weights(vllm_config, device) -> Iterator[tuple[str, torch.Tensor]]
         return synth.iter_pofadra_weights(mc.arch, mc.seed, mc.dtype, gen_dev)
     if fam == "luzerax":
         return synth.iter_luzerax_weights(mc.arch, mc.seed, mc.dtype, gen_dev)
+    if fam == "divadra":
+        return synth.iter_divadra_weights(mc.arch, mc.seed, mc.dtype, gen_dev)
     if fam == "deepseek_v4_flash":
         return iter(())             # the model draws its own seeded weights when no tensor arrives
     raise ValueError(f"no synthetic weight stream for family {fam}")

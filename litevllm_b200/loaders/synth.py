@@ -357,3 +357,67 @@ def iter_luzerax_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, de
             yield from gated(p + "mlp.shared.", mlp["shared"]["ff"])
     yield vec("final.norm", W, 1.0, 0.1)
     yield lin("head", V, W)
+
+
+def iter_divadra_weights(arch: ModelArch, seed: int = 0, dtype=torch.float32, device="cpu") -> Iterator[tuple[str, torch.Tensor]]:
+    """Linear weights ~ N(0, 1 / fan-in); norms near one; decays between a few and thousands of tokens; small attention
+    weights (a negative bias).  The rank of the decay's projection is the head size."""
+    W, V, taps = arch.hidden_size, arch.vocab_size, arch.extra["canon_taps"]
+
+    def lin(name, out_f, in_f):
+        return name, normal(name, (out_f, in_f), seed, in_f ** -0.5, dtype, device)
+
+    def vec(name, n, base=0.0, std=1.0):
+        return name, base + normal(name, (n,) if isinstance(n, int) else n, seed, std, torch.float32, device)
+
+    yield "embed", normal("embed", (V, W), seed, 1.0, dtype, device)
+    yield "bigram", normal("bigram", (arch.extra["bigram"]["buckets"] + 1, W), seed, 0.5, dtype, device)
+    yield vec("embed.norm", W, 1.0, 0.1)
+    for i, l in enumerate(arch.extra["layers"]):
+        p, m, x, mlp = f"l{i}.", l["mixer"], f"l{i}.mix.", l.get("mlp")
+        for n in "12" if mlp else "1":
+            yield vec(p + "norm" + n, W, 1.0, 0.1)
+            yield vec(p + "canon" + n, (W, taps), 0.0, 0.3)
+        if l["type"] == "mamba2":
+            H, dv = m["heads"], m["vdim"]
+            C = H * dv + 2 * m["groups"] * m["state"]
+            yield lin(x + "in", H * dv + C + H, W)
+            yield vec(x + "conv", (C, m["conv"]), 0.0, 0.5)
+            yield vec(x + "conv.b", C, 0.0, 0.1)
+            yield vec(x + "dt_bias", H, -1.0, 1.0)
+            yield vec(x + "A_log", H, -1.0, 1.0)
+            yield vec(x + "D", H, 1.0, 0.2)
+            yield vec(x + "norm", H * dv, 1.0, 0.1)
+            yield lin(x + "o", W, H * dv)
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, dv, n = a["heads"], a["kv_heads"], a["dim"], a["vdim"], r["heads"] * r["dim"]
+            for c, rows in (("q", H * d), ("k", G * d), ("v", G * dv)):
+                yield lin(x + "left." + c, rows, W)
+            yield vec(x + "left.q.norm", H * d, 1.0, 0.1)
+            yield vec(x + "left.k.norm", G * d, 1.0, 0.1)
+            yield vec(x + "left.pb", H, -2.0, 0.5)
+            yield lin(x + "left.o", W, H * dv)
+            for c in "rkvgw":
+                yield vec(x + "right.mu." + c, W, 0.5, 0.2)
+            for c in "rkvg":
+                yield lin(x + "right." + c, n, W)
+            yield lin(x + "right.w1", r["dim"], W)
+            yield lin(x + "right.w2", n, r["dim"])
+            yield vec(x + "right.w0", n, -3.0, 1.5)
+            yield vec(x + "right.u", (r["heads"], r["dim"]), 0.0, 0.5)
+            yield vec(x + "right.norm", n, 1.0, 0.1)
+            yield lin(x + "right.o", W, n)
+            yield vec(x + "left.out", W, 1.0, 0.1)
+            yield vec(x + "right.out", W, 1.0, 0.1)
+        if mlp and mlp["kind"] == "dense":
+            yield lin(p + "mlp.up", mlp["ff"], W)
+            yield lin(p + "mlp.down", W, mlp["ff"])
+        elif mlp:
+            E, top, ff = mlp["router"]["experts"], mlp["router"]["top"], mlp["expert"]["ff"]
+            for e in range(E):
+                for n, o, k in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+                    yield lin(p + f"mlp.e{e}.{n}", o, k)
+            yield p + "mlp.table", normal(p + "mlp.table", (V, E), seed, 1.0, torch.float32, device).topk(top, -1).indices.to(torch.int32)
+    yield vec("final.norm", W, 1.0, 0.1)
+    yield lin("head", V, W)

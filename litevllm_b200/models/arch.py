@@ -266,8 +266,78 @@ def arch_from_luzerax_config(cfg: dict) -> ModelArch:
     return arch
 
 
+def arch_from_divadra_config(cfg: dict) -> ModelArch:
+    """Divadra configurations list their layers one by one (mixer type and sizes; dense, assigned or no feed-forward)."""
+    layers, taps, bigram = cfg["layers"], cfg["canon"].get("taps"), cfg["embedding"]["bigram"]
+    if not layers:
+        raise ValueError("the configuration lists no layers")
+    _sizes(cfg["canon"], ("taps",), "canon")
+    _sizes(bigram, ("buckets",), "embedding.bigram")
+    for n in ("mul_prev", "mul_cur"):
+        if not isinstance(bigram.get(n), int):
+            raise ValueError(f"embedding.bigram: {n!r} must be an integer, got {bigram.get(n)!r}")
+
+    def short(n: int, where: str) -> None:
+        if n > 16:
+            raise ValueError(f"{where}: convolutions of at most 16 taps, got {n}")
+
+    short(taps, "canon")
+    for i, l in enumerate(layers):
+        m, where = l["mixer"], f"layers[{i}]"
+        if l["type"] == "mamba2":
+            _sizes(m, ("heads", "vdim", "state", "groups", "norm_groups", "conv"), where)
+            short(m["conv"], where)
+            if m["heads"] % m["groups"]:
+                raise ValueError(f"{where}: {m['heads']} heads do not share {m['groups']} groups evenly")
+            if m["heads"] * m["vdim"] % m["norm_groups"]:
+                raise ValueError(f"{where}: {m['heads'] * m['vdim']} channels do not make {m['norm_groups']} equal norm parts")
+        elif l["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            _sizes(a, ("heads", "kv_heads", "dim", "vdim"), where)
+            _sizes(a["mask"], ("size",), where)
+            _sizes(r, ("heads", "dim"), where)
+            if not isinstance(a.get("scale"), (int, float)):
+                raise ValueError(f"{where}: 'scale' must be a number, got {a.get('scale')!r}")
+            if a["heads"] % a["kv_heads"]:
+                raise ValueError(f"{where}: {a['heads']} heads do not share {a['kv_heads']} key heads evenly")
+            dims = a["rot"]["dims"]
+            if dims % 2 or dims > a["dim"] or dims < 0:
+                raise ValueError(f"{where}: cannot rotate {dims} of {a['dim']} dimensions")
+            if a["vdim"] % 2:
+                raise ValueError(f"{where}: cannot rotate values of {a['vdim']} dimensions")
+        else:
+            raise ValueError(f"{where}: unknown mixer {l['type']!r}")
+        mlp = l.get("mlp")
+        if not mlp:
+            continue
+        if mlp.get("kind") == "dense":
+            _sizes(mlp, ("ff",), where)
+        elif mlp.get("kind") == "moe":
+            _sizes(mlp["expert"], ("ff",), where)
+            _sizes(mlp["router"], ("experts", "top"), where)
+            if mlp["router"]["top"] > mlp["router"]["experts"]:
+                raise ValueError(f"{where}: cannot choose {mlp['router']['top']} of {mlp['router']['experts']} experts")
+        else:
+            raise ValueError(f"{where}: unknown feed-forward {mlp.get('kind')!r}")
+    attn = [l["mixer"]["left"] for l in layers if l["type"] == "parallel"]
+    mlps = [l["mlp"] for l in layers if l.get("mlp")]
+    arch = ModelArch(
+        family="divadra", architecture="Divadra", hidden_size=int(cfg["width"]), num_layers=len(layers),
+        num_heads=max((a["heads"] for a in attn), default=1), num_kv_heads=max((a["kv_heads"] for a in attn), default=1),
+        head_dim=max((a["dim"] for a in attn), default=64),
+        intermediate_size=max((m["ff"] if m["kind"] == "dense" else m["expert"]["ff"] for m in mlps), default=0),
+        vocab_size=int(cfg["vocab"]), rms_eps=float(cfg["norm"]["eps"]), act="relu2",
+        max_position=int(cfg.get("max_position_embeddings", 1 << 20)), eos_token_ids=_eos_list(cfg),
+        bos_token_id=cfg.get("bos_token_id"))
+    arch.layer_types = ["linear" if l["type"] == "mamba2" else "sliding" for l in layers]
+    arch.extra.update(layers=layers, canon_taps=taps, bigram=bigram)
+    return arch
+
+
 def arch_from_hf_config(cfg: dict) -> ModelArch:
     """Build a :class:`ModelArch` from a HF config dict (text sub-config is unwrapped)."""
+    if str(cfg.get("architecture", "")).lower() == "divadra":
+        return arch_from_divadra_config(cfg)
     if str(cfg.get("architecture", "")).lower() == "luzerax":
         return arch_from_luzerax_config(cfg)
     if str(cfg.get("architecture", "")).lower() == "pofadra":

@@ -191,6 +191,30 @@ PRESETS["luzerax-1b"] = luzerax_config(2048, 32000, "df" + "gmdmgm" * 3, (16, 4,
                                        (32, 8, 4, 4, 2, 768, 1536))
 
 
+def divadra_config(width: int, vocab: int, pattern: str, mamba: tuple, left: tuple, right: tuple, ff: int, moe: tuple,
+                   bigram: tuple = (4093, 31, 7), taps: int = 4, rot_base: float = 1e4, eps: float = 1e-6) -> dict:
+    """Divadra configuration from a layer pattern: per layer a mixer ("s" state space, "p" parallel) and a feed-forward ("f"
+    dense, "m" assigned experts, "-" none).  ``mamba``: heads, vdim, state, groups, norm groups, taps; ``left``: heads, kv
+    heads, dim, vdim, rotated dims, chunk; ``right``: heads, dim; ``moe``: experts, top, ff; ``bigram``: buckets, multipliers."""
+    s = dict(zip(("heads", "vdim", "state", "groups", "norm_groups", "conv"), mamba))
+    p = {"left": dict(zip(("heads", "kv_heads", "dim", "vdim"), left[:4]), scale=left[2] ** -0.5, mask={"size": left[5]},
+                      rot={"base": rot_base, "dims": left[4]}),
+         "right": dict(zip(("heads", "dim"), right))}
+    mlps = {"f": {"kind": "dense", "ff": ff}, "-": None,
+            "m": {"kind": "moe", "expert": {"ff": moe[2]}, "router": {"experts": moe[0], "top": moe[1]}}}
+    layers = [{"type": "mamba2" if pattern[i] == "s" else "parallel", "mixer": copy.deepcopy(s if pattern[i] == "s" else p),
+               "mlp": copy.deepcopy(mlps[pattern[i + 1]])} for i in range(0, len(pattern), 2)]
+    return {"architecture": "Divadra", "width": width, "vocab": vocab, "norm": {"eps": eps}, "canon": {"taps": taps},
+            "embedding": {"bigram": dict(zip(("buckets", "mul_prev", "mul_cur"), bigram))}, "layers": layers}
+
+
+PRESETS["tiny-divadra-test"] = divadra_config(160, 512, "sfpmp-pf", (4, 40, 24, 2, 5, 3), (6, 2, 40, 24, 16, 20), (4, 40), 176, (9, 3, 48),
+                                              bigram=(251, 31, 7), taps=3)
+# layers of the width and head geometry of a 1B-class decoder
+PRESETS["divadra-1b"] = divadra_config(2048, 32000, "sf" + "pmpfpm" * 3, (32, 128, 128, 4, 4, 4), (16, 4, 128, 128, 128, 1024), (32, 64), 5632,
+                                       (32, 4, 768))
+
+
 def get_preset(name: str) -> dict:
     key = name.lower()
     if key not in PRESETS:

@@ -24,12 +24,13 @@ _MODELS = {
     "Fimodra": ("fimodra", "FimodraForCausalLM"),
     "Pofadra": ("pofadra", "PofadraForCausalLM"),
     "Luzerax": ("luzerax", "LuzeraxForCausalLM"),
+    "Divadra": ("divadra", "DivadraForCausalLM"),
 }
 _FAMILY_DEFAULT = {
     "llama": "LlamaForCausalLM", "qwen2": "Qwen2ForCausalLM", "qwen3_5": "Qwen3_5ForCausalLM",
     "qwen2_vl": "Qwen2VLForConditionalGeneration", "gemma4": "Gemma4ForCausalLM",
     "deepseek_mla": "DeepseekV3ForCausalLM", "deepseek_v4_flash": "DeepseekV4FlashForCausalLM",
-    "fimodra": "Fimodra", "pofadra": "Pofadra", "luzerax": "Luzerax",
+    "fimodra": "Fimodra", "pofadra": "Pofadra", "luzerax": "Luzerax", "divadra": "Divadra",
 }
 
 

@@ -10,12 +10,13 @@ import math
 
 import ctypes
 import os
+from dataclasses import dataclass
 
 import torch
 
 from . import _lib, reference
 
-_ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "gelu": 2, "relu": 3, "clipped_swiglu": 4}
+_ACT = {None: 0, "none": 0, "silu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "gelu": 2, "relu": 3, "clipped_swiglu": 4, "relu2": 5, "tanh": 6}
 _DT = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
 
 _status_words: dict[int, torch.Tensor] = {}
@@ -437,12 +438,31 @@ class FiAttnExtra(ctypes.Structure):
     """csrc/attn/attn_extra.h"""
     _fields_ = [("sinks", ctypes.c_void_p), ("gate", ctypes.c_void_p), ("gate_stride", ctypes.c_long), ("out_dim", ctypes.c_int),
                 ("gate_per_head", ctypes.c_int), ("maps", ctypes.c_int), ("lam", ctypes.c_float), ("out_scale", ctypes.c_float),
-                ("eps", ctypes.c_float)]
+                ("eps", ctypes.c_float), ("bias", ctypes.c_void_p), ("turn", ctypes.c_void_p), ("turn_rows", ctypes.c_int),
+                ("chunk", ctypes.c_int)]
 
 
-def attn_extra(nh: int, od: int, sinks=None, gate=None, diff=None):
-    """Argument of the attention kernels: sinks, an output gate (one value per channel or per head), and ``diff =
-    (lambda, scale, eps)`` for two maps per head."""
+@dataclass(frozen=True)
+class SigmoidWeights:
+    """Attention without a softmax: a key's weight is sigmoid(score + bias of the head).  ``chunk`` > 0: a position sees
+    keys from the start of its chunk of that many positions on.  ``turn`` fp32 [positions, channels] = [cos | sin]:
+    channels 2 i and 2 i + 1 of the output turn back by angle i of the query's position."""
+    bias: torch.Tensor
+    chunk: int = 0
+    turn: torch.Tensor | None = None
+
+
+def attn_extra(nh: int, od: int, sinks=None, gate=None, diff=None, sigmoid: SigmoidWeights | None = None):
+    """Argument of the attention kernels: sinks, an output gate (one value per channel or per head), ``diff =
+    (lambda, scale, eps)`` for two maps per head, or ``sigmoid`` weights."""
+    if sigmoid is not None:
+        if sinks is not None or gate is not None or diff is not None:
+            raise ValueError("attention without a softmax takes no sinks, gates or two maps")
+        t = sigmoid.turn
+        if t is not None and t.shape[1] != od:
+            raise ValueError(f"outputs of {od} channels do not turn by a table of {t.shape[1]}")
+        return ctypes.byref(FiAttnExtra(None, None, 0, od, 0, 1, 0.0, 1.0, 0.0, _p(sigmoid.bias), _p(t),
+                                        0 if t is None else t.shape[0], int(sigmoid.chunk)))
     if gate is not None:
         if diff is not None:
             raise ValueError("attention with two maps per head takes no output gate")
@@ -456,17 +476,18 @@ def attn_extra(nh: int, od: int, sinks=None, gate=None, diff=None):
 
 def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv, hd, sm_scale,
                            window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, splits=0,
-                           max_kv_len=None, cu_q=None, sinks=None, v_dim=None, gate=None, diff=None):
+                           max_kv_len=None, cu_q=None, sinks=None, v_dim=None, gate=None, diff=None, sigmoid=None):
     """One query token per sequence.  q: [B, >= nh*hd] with row stride q.stride(0).  ``sinks`` (fp32 [nh]): a number per
     head whose exponential joins the softmax denominator.  ``v_dim``: only the leading channels of a head's output
     exist.  ``gate`` [B, nh * v_dim or nh] (any row pitch, the type of the output): the output is multiplied by its
     sigmoid.  ``diff = (lambda, scale, eps)``: query heads 2 j and 2 j + 1 (rows [q1 | 0] and [0 | q2] against keys
-    [k1 | k2]) are the two maps of output head j, ``rms(a1 - lambda a2) * scale``; the output has nh / 2 heads."""
+    [k1 | k2]) are the two maps of output head j, ``rms(a1 - lambda a2) * scale``; the output has nh / 2 heads.
+    ``sigmoid`` (:class:`SigmoidWeights`): no softmax."""
     B = seq_lens.shape[0]
     od = hd if v_dim is None else int(v_dim)
     heads_out = nh if diff is None else nh // 2
-    plain = sinks is None and gate is None and od == hd and diff is None
-    extra = attn_extra(nh, od, sinks, gate, diff)
+    plain = sinks is None and gate is None and od == hd and diff is None and sigmoid is None
+    extra = attn_extra(nh, od, sinks, gate, diff, sigmoid)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_decode", block_tables, seq_lens, k_cache)
     if not q.is_cuda:
@@ -483,13 +504,15 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv,
     elif not out.is_contiguous():
         # the kernels write rows of nh * od values back to back
         tmp = paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, nh, nkv, hd, sm_scale, window,
-                                     softcap, k_scale, v_scale, None, splits, max_kv_len, cu_q, sinks, v_dim, gate, diff)
+                                     softcap, k_scale, v_scale, None, splits, max_kv_len, cu_q, sinks, v_dim, gate, diff, sigmoid)
         out.copy_(tmp)
         return out
     if splits <= 0:
         if max_kv_len is None:
             max_kv_len = block_tables.shape[1] * k_cache.shape[2]
         eff = min(max_kv_len, window) if window and window > 0 else max_kv_len
+        if sigmoid is not None and sigmoid.chunk > 0:
+            eff = min(eff, sigmoid.chunk)
         splits = pick_decode_splits(B, nkv, eff)
     mode = reference.kv_mode(k_cache)
     assert mode < 2 or plain, "row-scaled caches take no sinks, gates, narrow outputs or two maps"
@@ -586,12 +609,12 @@ def paged_metadata_snapshot(q, k_cache, block_tables, seq_lens, cu_q=None, scope
 
 def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv,
                             hd, sm_scale, window=0, softcap=0.0, k_scale=1.0, v_scale=1.0, out=None, sinks=None,
-                            v_dim=None, gate=None, diff=None):
+                            v_dim=None, gate=None, diff=None, sigmoid=None):
     """Varlen causal attention of new tokens against the paged cache (which already holds them).  ``sinks``, ``v_dim``,
-    ``gate`` and ``diff`` as in :func:`paged_attention_decode`."""
+    ``gate``, ``diff`` and ``sigmoid`` as in :func:`paged_attention_decode`."""
     od = hd if v_dim is None else int(v_dim)
-    plain = sinks is None and gate is None and od == hd and diff is None
-    extra = attn_extra(nh, od, sinks, gate, diff)
+    plain = sinks is None and gate is None and od == hd and diff is None and sigmoid is None
+    extra = attn_extra(nh, od, sinks, gate, diff, sigmoid)
     if _BOUNDS_CHECK:
         _check_paged("paged_attention_prefill", block_tables, seq_lens, k_cache, cu_q)
     if not q.is_cuda:
@@ -608,7 +631,7 @@ def paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, m
         out = torch.empty(T, (nh if diff is None else nh // 2) * od, dtype=q.dtype, device=q.device)
     elif not out.is_contiguous():
         tmp = paged_attention_prefill(q, k_cache, v_cache, block_tables, seq_lens, cu_q, max_q_len, nh, nkv, hd,
-                                      sm_scale, window, softcap, k_scale, v_scale, None, sinks, v_dim, gate, diff)
+                                      sm_scale, window, softcap, k_scale, v_scale, None, sinks, v_dim, gate, diff, sigmoid)
         out.copy_(tmp)
         return out
     mode = reference.kv_mode(k_cache)

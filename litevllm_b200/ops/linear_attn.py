@@ -12,6 +12,8 @@ Per value head, with state ``S [dk, dv]``, decay ``a_t = exp(g_t)`` and write st
 * :func:`gated_delta_step` / :func:`conv1d_step` - one decode step for a batch of sequences on state
   pools indexed by slot (CUDA kernels in csrc/linear_attn/gated_delta.cu; PyTorch on the CPU).
 
+* :func:`time_mix` and :func:`ssd` - linear attention with channel decays and a bonus for the current token, or with scalar
+  decays, a skip and a short convolution in front (csrc/linear_attn/decay_scan.cu; PyTorch on the CPU).
 * :func:`delta_portions` / :func:`delta_step` - the rule with one decay per key channel, its short convolutions, unit
   vectors, head norm and gate included (csrc/linear_attn/channel_delta.cu; PyTorch on the CPU).
 
@@ -336,3 +338,152 @@ def delta_step(x, z, b, m: DeltaSpec, pool, ring, slots, seq_lens, norm_w, eps: 
     _lib.check(rc, "fi_delta_step")
     _count()
     return out
+
+
+# ---------------------------------------------------------------------------- decays with a bonus or a skip
+def time_mix_tokens(r, k, v, w, u, S):
+    """CPU form: r, k, w [L, H, d], v [L, H, dv], u [H, d]; ``S`` [H, d, dv] is updated in place."""
+    o = torch.empty(v.shape)
+    for t in range(r.shape[0]):
+        kv = k[t][:, :, None] * v[t][:, None, :]
+        o[t] = torch.einsum("hkv,hk->hv", S + u[:, :, None] * kv, r[t])
+        S.mul_(w[t][:, :, None]).add_(kv)
+    return o
+
+
+def ssd_tokens(x, b, c, dt, rate, skip, S):
+    """CPU form: x [L, H, dv], b, c [L, H, d], dt [L, H], rate, skip [H]; ``S`` [H, d, dv] is updated in place."""
+    o = torch.empty(x.shape)
+    for t in range(x.shape[0]):
+        S.mul_(torch.exp(-rate * dt[t])[:, None, None]).add_((dt[t][:, None] * b[t])[:, :, None] * x[t][:, None, :])
+        o[t] = torch.einsum("hkv,hk->hv", S, c[t]) + skip[:, None] * x[t]
+    return o
+
+
+def part_norm(o, w, parts: int, eps: float, out_dtype, gate=None, gate_first: bool = False):
+    """RMS norm over ``parts`` equal parts of each row of o fp32 [T, n], times ``w`` fp32 [n]; ``silu(gate)`` (any row pitch
+    and type) multiplies before the norm (``gate_first``) or after it."""
+    T, n = o.shape
+    if not o.is_cuda:
+        g = None if gate is None else F.silu(gate.float())
+        y = o * g if gate_first else o
+        y = y.view(T, parts, -1)
+        y = (y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)).view(T, n) * w
+        return (y if g is None or gate_first else y * g).to(out_dtype)
+    assert o.is_contiguous() and o.dtype == torch.float32 and (gate is None or gate.stride(1) == 1)
+    out = torch.empty(T, n, dtype=out_dtype, device=o.device)
+    rc = _lib.kernels().fi_part_norm(_p(o), _p(gate), gate.stride(0) if gate is not None else 0,
+                                     _DT[gate.dtype] if gate is not None else 0, int(gate_first), _p(w), parts, _p(out), T,
+                                     n // parts, eps, _DT[out_dtype], _stream())
+    _lib.check(rc, "fi_part_norm")
+    _count()
+    return out
+
+
+def _check_pool(pool, batch) -> None:
+    assert pool.dtype == torch.float32 and pool.is_contiguous() and batch.extras["slot_ids"].dtype == batch.seq_lens.dtype == torch.int32
+
+
+def _scan(kind: int, q, k, v, z, zb, u, rate, pool, batch, G: int):
+    T, (slots, H, d, dv) = v.shape[0], pool.shape
+    o = torch.empty(T, H * dv, dtype=torch.float32, device=v.device)
+    assert q.dtype == k.dtype == v.dtype and z.dtype == torch.float32 and q.stride(1) == k.stride(1) == v.stride(1) == z.stride(1) == 1
+    _check_pool(pool, batch)
+    rc = _lib.kernels().fi_decay_scan(kind, _p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), z.stride(0), _p(zb),
+                                      _p(u), _p(rate), _p(pool), _p(batch.extras["slot_ids"]), _p(batch.cu_q), _p(batch.seq_lens),
+                                      _p(o), batch.seq_lens.shape[0], H, G, d, dv, slots, _DT[v.dtype], _stream())
+    _lib.check(rc, "fi_decay_scan")
+    _count()
+    return o
+
+
+def time_mix(r, k, v, gate, z, w0, u, pool, batch, norm_w, eps: float, out_dtype):
+    """Time mixing of a step: ``o_t = (S + diag(u) k_t v_t^T)^T r_t``, ``S = diag(exp(-exp(z_t + w0))) S + k_t v_t^T``, then per
+    head norm, ``norm_w`` and ``silu(gate)``.
+
+    r, k, v, gate [T, H * d] (any row pitch, one type), z fp32 [T, H * d], w0 [H * d], u [H, d], norm_w [H * d] fp32; pool fp32
+    [slots, H, d, d], updated in place.  A sequence whose first position is 0 starts from zero.  Returns [T, H * d]."""
+    slots_n, H, d, dv = pool.shape
+    T = r.shape[0]
+    if not r.is_cuda:
+        from .shift_stream import sequences
+        o = torch.zeros(T, H * dv)
+        for slot, lo, hi, pos0 in sequences(batch):
+            if pos0 == 0:
+                pool[slot].zero_()
+            w = torch.exp(-torch.exp(z[lo:hi].float() + w0))
+            h = [t.float().reshape(hi - lo, H, -1) for t in (r[lo:hi], k[lo:hi], v[lo:hi], w)]
+            o[lo:hi] = time_mix_tokens(*h, u, pool[slot]).view(hi - lo, -1)
+        return part_norm(o, norm_w, H, eps, out_dtype, gate)
+    if not batch.is_decode:
+        return part_norm(_scan(0, r, k, v, z, w0, u, None, pool, batch, H), norm_w, H, eps, out_dtype, gate)
+    assert r.dtype == k.dtype == v.dtype == gate.dtype and z.dtype == torch.float32
+    assert r.stride(1) == k.stride(1) == v.stride(1) == gate.stride(1) == z.stride(1) == 1
+    _check_pool(pool, batch)
+    out = torch.empty(T, H * dv, dtype=out_dtype, device=r.device)
+    rc = _lib.kernels().fi_decay_step(_p(r), r.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), z.stride(0), _p(w0), _p(u),
+                                      _p(gate), gate.stride(0), _p(norm_w), eps, _p(pool), _p(batch.extras["slot_ids"]),
+                                      _p(batch.seq_lens), _p(out), T, H, d, dv, slots_n, _DT[r.dtype], _DT[out_dtype], _stream())
+    _lib.check(rc, "fi_decay_step")
+    _count()
+    return out
+
+
+def conv_silu(x, w, bias, ring, batch, out_dtype):
+    """silu(causal convolution + bias) of a step's portions: x [T, C] (any row pitch), w fp32 [taps, C] (last row: the present
+    token), ring fp32 [slots, taps, C], updated in place.  Returns [T, C]."""
+    T, C = x.shape
+    taps = w.shape[0]
+    if not x.is_cuda:
+        from .shift_stream import ring_before, ring_store, sequences
+        y = torch.zeros(T, C)
+        for slot, lo, hi, pos0 in sequences(batch):
+            seq = torch.cat([ring_before(ring[slot], pos0, taps - 1), x[lo:hi].float()])
+            y[lo:hi] = F.silu((seq.unfold(0, taps, 1) * w.t()).sum(-1) + bias)
+            ring_store(ring[slot], pos0, x[lo:hi].float())
+        return y.to(out_dtype)
+    from .shift_stream import tiles
+    base, n_tiles, tile = tiles(batch, taps)
+    assert x.stride(1) == 1 and ring.is_contiguous() and w.is_contiguous() and ring.dtype == w.dtype == bias.dtype == torch.float32
+    y = torch.empty(T, C, dtype=out_dtype, device=x.device)
+    rc = _lib.kernels().fi_conv_silu(_p(x), x.stride(0), _p(w), _p(bias), taps, _p(ring), _p(y), _p(batch.extras["slot_ids"]),
+                                     _p(batch.cu_q), _p(batch.seq_lens), _p(base), n_tiles, tile, batch.seq_lens.shape[0], C,
+                                     ring.shape[0], _DT[x.dtype], _DT[out_dtype], _stream())
+    _lib.check(rc, "fi_conv_silu")
+    _count()
+    return y
+
+
+def ssd(xbc, z, dt, dt_bias, rate, skip, conv, conv_b, pool, ring, G: int, batch, norm_w, parts: int, eps: float, out_dtype):
+    """State-space step: x | B | C = silu(conv(xbc) + conv_b); dt = softplus(dt + dt_bias); ``S = exp(-rate dt) S + dt B x^T``,
+    ``y = S^T C + skip x``; then ``norm(y silu(z))`` over ``parts`` equal parts, times ``norm_w``.
+
+    xbc [T, H dv + 2 G d] (x, B and C of G groups; any row pitch), z [T, H dv], dt fp32 [T, H]; conv fp32 [taps, channels]; pool
+    fp32 [slots, H, d, dv] and ring fp32 [slots, taps, channels], updated in place.  Returns [T, H dv]."""
+    slots_n, H, d, dv = pool.shape
+    T, inner = xbc.shape[0], H * dv
+    if not xbc.is_cuda:
+        from .shift_stream import sequences
+        u = conv_silu(xbc, conv, conv_b, ring, batch, torch.float32)
+        o = torch.zeros(T, inner)
+        for slot, lo, hi, pos0 in sequences(batch):
+            if pos0 == 0:
+                pool[slot].zero_()
+            L = hi - lo
+            b, c = (u[lo:hi, at:at + G * d].reshape(L, G, d).repeat_interleave(H // G, 1) for at in (inner, inner + G * d))
+            o[lo:hi] = ssd_tokens(u[lo:hi, :inner].reshape(L, H, dv), b, c, F.softplus(dt[lo:hi].float() + dt_bias), rate, skip,
+                                  pool[slot]).view(L, inner)
+        return part_norm(o, norm_w, parts, eps, out_dtype, z, True)
+    if batch.is_decode:
+        _check_pool(pool, batch)
+        assert xbc.stride(1) == dt.stride(1) == 1 and dt.dtype == torch.float32 and ring.is_contiguous()
+        o = torch.empty(T, inner, dtype=torch.float32, device=xbc.device)
+        rc = _lib.kernels().fi_decay_step_conv(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(rate), _p(skip), _p(conv),
+                                               _p(conv_b), conv.shape[0], _p(ring), _p(pool), _p(batch.extras["slot_ids"]),
+                                               _p(batch.seq_lens), _p(o), T, H, G, d, dv, slots_n, _DT[xbc.dtype], _stream())
+        _lib.check(rc, "fi_decay_step_conv")
+        _count()
+    else:
+        u = conv_silu(xbc, conv, conv_b, ring, batch, out_dtype)
+        o = _scan(1, u[:, inner + G * d:], u[:, inner:inner + G * d], u[:, :inner], dt, dt_bias, skip, rate, pool, batch, G)
+    return part_norm(o, norm_w, parts, eps, out_dtype, z, True)

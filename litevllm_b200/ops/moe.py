@@ -67,6 +67,21 @@ def route(logits: torch.Tensor, top_k: int, mode: str = "softmax", bias: torch.T
     return ids, w
 
 
+def lookup(table: torch.Tensor, token_ids: torch.Tensor, weight: float):
+    """Experts that a table int32 [vocab, k] assigns to token ids (int64 [T]), each with ``weight``: (ids int32 [T, k],
+    weights float32 [T, k])."""
+    T, (V, K) = token_ids.shape[0], table.shape
+    if not table.is_cuda:
+        return table.index_select(0, token_ids), torch.full((T, K), float(weight))
+    ids = torch.empty(T, K, dtype=torch.int32, device=table.device)
+    w = torch.empty(T, K, dtype=torch.float32, device=table.device)
+    assert table.dtype == torch.int32 and table.is_contiguous() and token_ids.dtype == torch.int64 and token_ids.is_contiguous()
+    rc = _lib.kernels().fi_moe_lookup(_p(table), _p(token_ids), V, T, K, float(weight), _p(ids), _p(w), _stream())
+    _lib.check(rc, "fi_moe_lookup")
+    _count()
+    return ids, w
+
+
 @dataclass
 class RoutedRows:
     """Outputs of the chosen experts before their weighted sum: choice k of token t is row ``slot_of[t, k]`` of ``rows``
@@ -86,6 +101,40 @@ class RoutedRows:
         r = self.rows.index_select(0, self.slot_of.clamp(min=0).reshape(-1).long()).float().view(T, K, -1)
         r = torch.where(none, x.float()[:, None] if self.pass_through else torch.zeros_like(r), r)
         return (r * self.weights[..., None]).sum(1)
+
+
+_stack_tiles: dict[tuple, torch.Tensor] = {}
+
+
+def _stacked_tile_table(E: int, T: int, bn: int, device) -> torch.Tensor:
+    """int32 [3, n]: matrix, first row and rows of each tile of ``bn`` rows of E stacked matrices of T rows.  Tables stay
+    alive: captured steps hold their addresses."""
+    key = (E, T, bn, str(device))
+    if key not in _stack_tiles:
+        rows = [(e, e * T + t, min(bn, T - t)) for e in range(E) for t in range(0, T, bn)]
+        with torch.inference_mode(False):
+            _stack_tiles[key] = torch.tensor(rows + [(len(rows),) * 3], dtype=torch.int32, device="cpu").t().contiguous().to(device)
+    return _stack_tiles[key]
+
+
+def stacked_linear(x: torch.Tensor, w: torch.Tensor):
+    """x [E, T, K] (rows of one pitch, matrices back to back), w [E, N, K] -> E matrices [T, N].  Small steps run one grouped product."""
+    from .. import ops
+    E, T, K = x.shape
+    N = w.shape[1]
+    if not x.is_cuda or x.dtype == torch.float32 or T >= ops._PERSISTENT_MIN_T or K % 8 or N % 8 or x.stride(1) % 8 \
+            or x.stride(0) != T * x.stride(1) or x.data_ptr() % 16 or not w.is_contiguous():
+        return [ops.linear(x[e], w[e]) for e in range(E)]
+    out = torch.empty(E, T, N, dtype=x.dtype, device=x.device)
+    bn = 16 if T <= 16 else 32 if T <= 32 else 64
+    t = _stacked_tile_table(E, T, bn, x.device)
+    n = t.shape[1] - 1
+    g = FiGrouped(t[0].data_ptr(), t[1].data_ptr(), t[2].data_ptr(), t[0, n:].data_ptr(), n, E, N, 0)
+    rc = _lib.kernels().fi_dense_gemm_grouped(_p(x), _p(w), _p(out), E * T, N, K, x.stride(1), N, 0, 0.0, 0, _DT[x.dtype], bn,
+                                              ctypes.byref(g), _p(status_word(x.device)), _stream())
+    _lib.check(rc, "fi_dense_gemm_grouped")
+    _count()
+    return out
 
 
 def _tile_table(ids, n: int, E: int, bn: int, dev, scratch_name: str):

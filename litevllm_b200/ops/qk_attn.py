@@ -32,9 +32,12 @@ def _normed(x, w, eps: float):
     return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w
 
 
-def prepare(proj, wq, wk, eps: float, positions, cos_sin, slot_mapping, k_cache, v_cache, H: int, G: int, dim: int):
+def prepare(proj, wq, wk, eps: float, positions, cos_sin, slot_mapping, k_cache, v_cache, H: int, G: int, dim: int,
+            vdim: int = 0, v_cos_sin=None):
     """proj [T, >= (H + G) * dim] (q | k); caches [blocks, G, block size, hd] with hd >= dim (the rest is cleared); slots
-    < 0 write no cache row.  Returns queries [T, H, hd] in the type of ``proj``."""
+    < 0 write no cache row.  ``vdim`` > 0: values have a projection of their own, proj [.. | v (G * vdim)], whose channels
+    2 i and 2 i + 1 turn by angle i of ``v_cos_sin`` [positions, vdim] (None: as they are); otherwise the value is the key
+    before norm and rotation.  Returns queries [T, H, hd] in the type of ``proj``."""
     T, hd, bs = proj.shape[0], k_cache.shape[3], k_cache.shape[2]
     q_out = torch.empty(T, H, hd, dtype=proj.dtype, device=proj.device)
     if not proj.is_cuda:
@@ -46,11 +49,17 @@ def prepare(proj, wq, wk, eps: float, positions, cos_sin, slot_mapping, k_cache,
         q_out.zero_()
         q_out[..., :dim] = _rotate_halves(q, cs[..., :half], cs[..., half:]).to(proj.dtype)
         k = _rotate_halves(k, cs[..., :half], cs[..., half:])
+        v = raw.view(T, G, dim)
+        if vdim:
+            v = proj[:, (H + G) * dim:(H + G) * dim + G * vdim].float().reshape(T, G, vdim)
+            if v_cos_sin is not None:
+                vcs = v_cos_sin[positions.long()][:, None]
+                v = _turn(v, vcs[..., :vdim // 2], vcs[..., vdim // 2:], vdim, True)
         at = torch.nonzero(slot_mapping >= 0).view(-1)
         slot = slot_mapping[at].long()
-        for cache, rows in ((k_cache, k), (v_cache, raw.view(T, G, dim))):
-            full = torch.zeros(at.shape[0], G, hd, dtype=cache.dtype)
-            full[..., :dim] = rows[at].to(cache.dtype)
+        for cache, rows in ((k_cache, k), (v_cache, v)):
+            full = torch.zeros(at.shape[0], G, cache.shape[3], dtype=cache.dtype)
+            full[..., :rows.shape[-1]] = rows[at].to(cache.dtype)
             cache[slot // bs, :, slot % bs] = full
         return q_out
     if _ops._BOUNDS_CHECK:
@@ -59,9 +68,11 @@ def prepare(proj, wq, wk, eps: float, positions, cos_sin, slot_mapping, k_cache,
         _ops._check_index("qk_attn.prepare.positions", positions, 0, cos_sin.shape[0], "rows of the cos/sin table")
     assert proj.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous()
     assert k_cache.dtype == v_cache.dtype == proj.dtype and positions.dtype == slot_mapping.dtype == torch.int32
+    assert v_cos_sin is None or v_cos_sin.shape == (cos_sin.shape[0], vdim)
     rc = _lib.kernels().fi_qk_prepare(_p(proj), proj.stride(0), _p(wq), _p(wk), eps, _p(positions), _p(cos_sin),
                                       cos_sin.shape[0], _p(slot_mapping), _p(q_out), _p(k_cache), _p(v_cache), T, H, G, dim,
-                                      hd, cos_sin.shape[1], bs, _DT[proj.dtype], _stream())
+                                      hd, cos_sin.shape[1], bs, (H + G) * dim if vdim else 0, vdim, v_cache.shape[3],
+                                      _p(v_cos_sin), _DT[proj.dtype], _stream())
     _lib.check(rc, "fi_qk_prepare")
     _count()
     return q_out
@@ -154,11 +165,12 @@ def prepare_heads(proj, wq, wk, spec: HeadSpec, positions, cos_sin, factor, slot
 
 
 def attend_rows(q, k_cache, v_cache, block_tables, row_lens, seq_of_row, scale: float, window: int, sinks, gate, dim: int,
-                diff=None):
+                diff=None, sigmoid=None):
     """q [R, H, hd]; row r sees the first ``row_lens[r]`` tokens (the last ``window`` of them) of sequence
     ``seq_of_row[r]`` (None: sequence r).  Returns [R, H * dim], gated by ``sigmoid(gate)`` (a value per channel or per
     head).  ``diff = (lambda, scale, eps)``: query heads 2 j and 2 j + 1 meet the two halves of the key rows and are the
-    maps of output head j, ``rms(a1 - lambda a2) * scale``; returns [R, H / 2 * dim]."""
+    maps of output head j, ``rms(a1 - lambda a2) * scale``; returns [R, H / 2 * dim].  ``sigmoid``
+    (:class:`ops.SigmoidWeights`): no softmax."""
     R, H, hd = q.shape
     G, bs = k_cache.shape[1], k_cache.shape[2]
     if not q.is_cuda:
@@ -176,11 +188,21 @@ def attend_rows(q, k_cache, v_cache, block_tables, row_lens, seq_of_row, scale: 
             if n <= 0:
                 continue
             b = r if seq_of_row is None else int(seq_of_row[r])
-            pos = torch.arange(max(0, n - window) if window else 0, n)
+            first = max(0, n - window) if window else 0
+            if sigmoid is not None and sigmoid.chunk:
+                first = (n - 1) // sigmoid.chunk * sigmoid.chunk
+            pos = torch.arange(first, n)
             blk = block_tables[b].long()[pos // bs]
             k = k_cache[blk, :, pos % bs].float().repeat_interleave(H // G, 1)              # [n, H, hd]
             v = v_cache[blk, :, pos % bs].float().repeat_interleave(H // G, 1)
             s = torch.einsum("hd,nhd->hn", q[r].float(), k) * scale
+            if sigmoid is not None:
+                o = torch.einsum("hn,nhd->hd", torch.sigmoid(s + sigmoid.bias[:, None]), v)[:, :dim]
+                if sigmoid.turn is not None:
+                    cs = sigmoid.turn[n - 1]
+                    o = _turn(o[None], cs[:dim // 2], -cs[dim // 2:], dim, True)[0]
+                out[r] = o.to(out.dtype)
+                continue
             if sinks is not None:
                 s = torch.cat([s, sinks[:, None]], dim=1)
             a = torch.softmax(s, dim=-1)[:, :k.shape[0]]
@@ -199,7 +221,7 @@ def attend_rows(q, k_cache, v_cache, block_tables, row_lens, seq_of_row, scale: 
     out = torch.empty(R, H // maps * dim, dtype=q.dtype, device=q.device)
     rc = _lib.kernels().fi_attn_rows(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(block_tables), _p(row_lens), _p(seq_of_row),
                                      R, H, G, hd * maps, dim, block_tables.shape[1], bs, k_cache.shape[0], int(window),
-                                     _ops.attn_extra(H, dim, sinks, gate, diff), scale, _DT[q.dtype], _stream())
+                                     _ops.attn_extra(H, dim, sinks, gate, diff, sigmoid), scale, _DT[q.dtype], _stream())
     _lib.check(rc, "fi_attn_rows")
     _count()
     return out

@@ -25,6 +25,10 @@ def apply_act(x: torch.Tensor, act: str | None) -> torch.Tensor:
         return F.gelu(x, approximate="tanh")
     if act == "relu":
         return F.relu(x)
+    if act == "relu2":
+        return F.relu(x).square()
+    if act == "tanh":
+        return torch.tanh(x)
     raise ValueError(f"unknown activation {act}")
 
 
