@@ -70,6 +70,8 @@ def parse_args():
     ap.add_argument("--pofadra-sizes", type=int, nargs="*", default=None, help="widths for --pofadra (default: all)")
     ap.add_argument("--luzerax", action="store_true", help="the same for the Luzerax design")
     ap.add_argument("--luzerax-sizes", type=int, nargs="*", default=None, help="widths for --luzerax (default: all)")
+    ap.add_argument("--divadra", action="store_true", help="the same for the Divadra design")
+    ap.add_argument("--divadra-sizes", type=int, nargs="*", default=None, help="widths for --divadra (default: all)")
     return ap.parse_args()
 
 
@@ -601,6 +603,10 @@ def main():
     if args.luzerax:
         from benchmarks import luzerax_shapes
         print(json.dumps(run_shapes(luzerax_shapes, args.luzerax_sizes)), flush=True)
+        return
+    if args.divadra:
+        from benchmarks import divadra_shapes
+        print(json.dumps(run_shapes(divadra_shapes, args.divadra_sizes)), flush=True)
         return
     res = run_reference(args) if args.impl == "reference" else run_ours(args)
     if res:
