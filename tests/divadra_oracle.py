@@ -259,10 +259,12 @@ def weights(cfg, seed=0, sharp=2.0):
                 put(x + "right.mu." + c, W, std=0.3, base=0.5)
             for c in "rkvg":
                 lin(x + "right." + c, n, W)
+            # a first token's output is its bonus, sum(r u k), times v, and a norm follows: keep that sum away from zero
+            w[x + "right.k"] = (0.8 * w[x + "right.r"] + 0.6 * w[x + "right.k"]).bfloat16().float()
             lin(x + "right.w1", l["rank"], W)
             lin(x + "right.w2", n, l["rank"])
             put(x + "right.w0", n, std=2.0, base=-2.5)
-            put(x + "right.u", r["heads"], r["dim"], std=0.7)
+            put(x + "right.u", r["heads"], r["dim"], std=0.4, base=0.8)
             put(x + "right.norm", n, std=0.2, base=1.0)
             lin(x + "right.o", W, n)
             for c in ("left.out", "right.out"):

@@ -102,7 +102,7 @@ def _prefill_logits(llm, prompts):
                                              # (rounding the weights to 16 bits flips a near tie of a router in the
                                              # first prompt's last token: 0.909 in exact arithmetic)
                                              ("tiny-pofadra-test", 0.89),
-                                             ("tiny-luzerax-test", 0.98)])
+                                             ("tiny-luzerax-test", 0.98), ("tiny-divadra-test", 0.99)])
 def test_quantised_models_match_cpu_oracle(preset, min_cos):
     """int4 weights (+ fp8 KV, MoE routing for Gemma4): GPU kernels vs the CPU fp32 path on the same
     synthetic checkpoint."""

@@ -332,7 +332,7 @@ def test_http_structured_outputs_choice_errors_and_limits():
 @pytest.mark.parametrize("preset,seed", [("tiny-llama-test", 1), ("tiny-llama-test", 2), ("tiny-llama-test", 3),
                                          ("tiny-qwen35-test", 4), ("tiny-qwen35-moe-test", 5), ("tiny-gemma4-moe-test", 6),
                                          ("tiny-deepseek-test", 7), ("tiny-deepseek-v4-flash-test", 8), ("tiny-fimodra-test", 9),
-                                         ("tiny-pofadra-test", 10), ("tiny-luzerax-test", 11)])
+                                         ("tiny-pofadra-test", 10), ("tiny-luzerax-test", 11), ("tiny-divadra-test", 12)])
 def test_random_arrivals_and_aborts_keep_every_invariant(preset, seed):
     """A seeded storm on a small engine: requests of random length arrive while others decode, some are aborted
     at random moments, prefill runs in small chunks.  Every surviving request generates exactly what it generates
