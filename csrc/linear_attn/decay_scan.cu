@@ -357,6 +357,26 @@ __global__ void __launch_bounds__(256, 3) decay_step_kernel(const ScanParams p) 
   const bool fresh = len == 1;
   float* S = p.pool + (static_cast<long>(slot) * p.H + head) * d * dv;
   const int per = p.H / p.G, group = head / per;
+  constexpr int U = 8;                  // rows whose loads are in flight together; the first ones while the operands are prepared
+  float s[U][VEC];
+  auto fetch = [&](int r0) {
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+      const int r = r0 + i * ry_n;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) s[i][e] = 0.f;
+      if (!fresh && r < d) {
+        const float* row = S + static_cast<long>(r) * dv + cx * VEC;
+        if constexpr (VEC == 4) {
+          const float4 x = *reinterpret_cast<const float4*>(row);
+          s[i][0] = x.x; s[i][1] = x.y; s[i][2] = x.z; s[i][3] = x.w;
+        } else {
+          s[i][0] = row[0];
+        }
+      }
+    }
+  };
+  if (ry < ry_n) fetch(ry);
   float decay = 1.f, g = 0.f;       // kScalar: decay and skip; kChannel: g is the bonus
   if constexpr (KIND == kChannel) {
     for (int c = tid; c < d; c += 256) {
@@ -398,24 +418,8 @@ __global__ void __launch_bounds__(256, 3) decay_step_kernel(const ScanParams p) 
       v[e] = sv[cx * VEC + e];
       o[e] = 0.f;
     }
-    constexpr int U = 8;                  // rows whose loads are in flight together
     for (int r0 = ry; r0 < d; r0 += U * ry_n) {
-      float s[U][VEC];
-#pragma unroll
-      for (int i = 0; i < U; ++i) {
-        const int r = r0 + i * ry_n;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) s[i][e] = 0.f;
-        if (!fresh && r < d) {
-          const float* row = S + static_cast<long>(r) * dv + cx * VEC;
-          if constexpr (VEC == 4) {
-            const float4 x = *reinterpret_cast<const float4*>(row);
-            s[i][0] = x.x; s[i][1] = x.y; s[i][2] = x.z; s[i][3] = x.w;
-          } else {
-            s[i][0] = row[0];
-          }
-        }
-      }
+      if (r0 != ry) fetch(r0);
 #pragma unroll
       for (int i = 0; i < U; ++i) {
         const int r = r0 + i * ry_n;
@@ -513,18 +517,14 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvParams p) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) a[j][e] = win[j][e] = 0.f;
     if (tap >= 0) {
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) a[j][e] = p.w[static_cast<long>(tap) * p.C + c + e];
+      load_x<VEC>(p.w + static_cast<long>(tap) * p.C + c, kFp32, a[j]);
       if (j + 1 < KT) {
         if (i >= 0) load_x<VEC>(x + i * p.ld, p.type, win[j]);
-        else if (pos0 + i >= 0)
-#pragma unroll
-          for (int e = 0; e < VEC; ++e) win[j][e] = ring[static_cast<long>((pos0 + i) % taps) * p.C + e];
+        else if (pos0 + i >= 0) load_x<VEC>(ring + static_cast<long>((pos0 + i) % taps) * p.C, kFp32, win[j]);
       }
     }
   }
-#pragma unroll
-  for (int e = 0; e < VEC; ++e) bias[e] = p.bias[c + e];
+  load_x<VEC>(p.bias + c, kFp32, bias);
   const int i_end = min(n, i0 + p.tile);
   for (int i = i0; i < i_end; i += 4) {
     float xn[4][VEC];
@@ -588,15 +588,17 @@ struct NormParams {
   float eps;
 };
 
-// A row of n values per TPR threads, NV groups of four each (NV = 0: any n, one value at a time, read twice).
+// A row of n values per TPR threads (16, 32 or 256), NV groups of four each (NV = 0: any n, one value at a time, read twice).
 template <int TPR, int NV>
 __global__ void __launch_bounds__(256) part_norm_kernel(const NormParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   __shared__ float red[8];
   constexpr int per = 256 / TPR;
-  const long row = static_cast<long>(blockIdx.x) * per + (per == 1 ? 0 : static_cast<int>(threadIdx.x) / TPR);
-  if (row >= p.rows) return;
+  long row = static_cast<long>(blockIdx.x) * per + (per == 1 ? 0 : static_cast<int>(threadIdx.x) / TPR);
+  if (TPR >= 32 && row >= p.rows) return;
+  const bool live = row < p.rows;          // half warps leave together
+  if (!live) row = p.rows - 1;
   const int tid = per == 1 ? threadIdx.x : threadIdx.x % TPR;
   const long t = row / p.parts;
   const int part = static_cast<int>(row % p.parts), n = p.n;
@@ -605,7 +607,8 @@ __global__ void __launch_bounds__(256) part_norm_kernel(const NormParams p) {
   const long grow = t * p.ldg + static_cast<long>(part) * n;
   float ss = 0.f;
   auto total = [&]() {
-    for (int m = 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
+#pragma unroll
+    for (int m = TPR < 32 ? TPR / 2 : 16; m > 0; m >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, m);
     if constexpr (TPR > 32) {
       if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
       __syncthreads();
@@ -643,7 +646,7 @@ __global__ void __launch_bounds__(256) part_norm_kernel(const NormParams p) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * 4;
-      if (c >= n) continue;
+      if (c >= n || !live) continue;
       const float4 f = *reinterpret_cast<const float4*>(w + c);
       float y[4] = {v[i][0] * inv * f.x, v[i][1] * inv * f.y, v[i][2] * inv * f.z, v[i][3] * inv * f.w};
       if (!p.gate_first)
@@ -787,7 +790,8 @@ extern "C" int fi_conv_silu(const void* x, long ld, const float* w, const float*
   p.x = x; p.ld = ld; p.w = w; p.bias = bias; p.taps = taps; p.ring = ring; p.out = out; p.slots = slots; p.cu_q = cu_q;
   p.seq_lens = seq_lens; p.tile_base = tile_base; p.tile = tile; p.B = B; p.C = C; p.num_slots = num_slots; p.type = type;
   p.out_type = out_type;
-  const bool vec4 = C % 4 == 0 && ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  const bool vec4 = C % 4 == 0 && ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(w) |
+                                                   reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(ring)) & 15) == 0;
   const dim3 g(n_tiles, (C + (vec4 ? 512 : 128) - 1) / (vec4 ? 512 : 128));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define FI_CONV(KT)                                                                                                   \
@@ -822,6 +826,7 @@ extern "C" int fi_part_norm(const float* x, const void* gate, long ldg, int gate
     if (n <= 256) FI_NORM(32, 0);
     FI_NORM(256, 0);
   }
+  if (n <= 64) FI_NORM(16, 1);
   if (n <= 128) FI_NORM(32, 1);
   if (n <= 256) FI_NORM(32, 2);
   if (n <= 512) FI_NORM(32, 4);

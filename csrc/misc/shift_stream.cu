@@ -138,7 +138,8 @@ __device__ __forceinline__ int find_seq(const int* base, int B, int at) {
 
 constexpr int block_threads(int tpr) { return tpr > 256 ? tpr : 256; }
 
-template <int TPR, int VEC, int NV, bool H16>
+// TOKEN: one token per sequence, what the next layer reads included; otherwise rows of portions or of the end of the model.
+template <int TPR, int VEC, int NV, bool H16, bool TOKEN>
 __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const ShiftParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -150,10 +151,9 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
   const long t = p.sel != nullptr ? static_cast<long>(p.sel[r]) : r;
   const int W = p.W;
   const float inv_n = 1.f / static_cast<float>(W);
-  const bool token = p.out_kind == kToken;
   int len = 0, slot = 0;
   const int n_out = 1 + (p.a2 != nullptr) + (p.mu != nullptr ? kBlends : 0);
-  if (token) {
+  if constexpr (TOKEN) {
     len = p.seq_lens[r];
     slot = p.slots[r];
     if (len <= 0 || slot < 0 || slot >= p.num_slots) {       // padded row of a decode bucket
@@ -168,47 +168,12 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
     }
   }
 
-  // what the ring contributes does not wait for this token: partial h1 and h2, and the previous token's h1
-  float s1[N], s2[N], before[N];
-  const int pos = len - 1, R = p.taps + 1;
-  float* ring = p.ring + static_cast<long>(slot) * R * W;
-  if (token) {
-#pragma unroll
-    for (int i = 0; i < N; ++i) s1[i] = s2[i] = before[i] = 0.f;
-    for (int j = 1; j <= p.taps; ++j) {    // j tokens back
-      if (pos - j < 0) break;
-      const float* row = ring + static_cast<long>((pos - j) % R) * W;
-#pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int c = (i * TPR + tid) * VEC;
-        if (c < W) {
-          float v[VEC], a[VEC];
-          load_f<VEC>(row, c, v);
-          if (p.mu != nullptr) {
-            load_f<VEC>(p.a1, static_cast<long>(p.taps - j) * W + c, a);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) before[i * VEC + e] = fmaf(a[e], v[e], before[i * VEC + e]);
-          }
-          if (j < p.taps) {
-            load_f<VEC>(p.a1, static_cast<long>(p.taps - 1 - j) * W + c, a);
-#pragma unroll
-            for (int e = 0; e < VEC; ++e) s1[i * VEC + e] = fmaf(a[e], v[e], s1[i * VEC + e]);
-            if (p.a2 != nullptr) {
-              load_f<VEC>(p.a2, static_cast<long>(p.taps - 1 - j) * W + c, a);
-#pragma unroll
-              for (int e = 0; e < VEC; ++e) s2[i * VEC + e] = fmaf(a[e], v[e], s2[i * VEC + e]);
-            }
-          }
-        }
-      }
-    }
-  }
-
-  float v[N];
+  // everything that is read is requested ahead of the first reduction
+  float v[N], y[N], z[N];
   if (p.mode == kStart) {
     long long id = p.ids[t], prev = -1;
-    if (token) {
-      if (pos > 0) prev = p.last_token[slot];
+    if constexpr (TOKEN) {
+      if (len > 1) prev = p.last_token[slot];
     } else {
       const int b = find_seq(p.cu_q, p.B, static_cast<int>(t));
       const int idx = static_cast<int>(t) - p.cu_q[b], n = p.cu_q[b + 1] - p.cu_q[b], s = p.slots[b];
@@ -226,18 +191,17 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
-      float q[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[i * VEC + e] = q[e] = 0.f;
+      for (int e = 0; e < VEC; ++e) v[i * VEC + e] = y[i * VEC + e] = 0.f;
       if (c < W) {
         load_h<VEC, H16>(p.table, id * W + c, p.h_type, v + i * VEC);
-        load_h<VEC, H16>(p.pairs, pr * W + c, p.h_type, q);
+        load_h<VEC, H16>(p.pairs, pr * W + c, p.h_type, y + i * VEC);
       }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) { v[i * VEC + e] += q[e]; ss = fmaf(v[i * VEC + e], v[i * VEC + e], ss); }
     }
+#pragma unroll
+    for (int i = 0; i < N; ++i) { v[i] += y[i]; ss = fmaf(v[i], v[i], ss); }
     row_sums<TPR>(ss, none, red);
-    if (token) {
+    if constexpr (TOKEN) {
       __syncwarp();
       if (tid == 0) p.last_token[slot] = static_cast<int>(now);     // every thread of the row has read it
     }
@@ -253,45 +217,17 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
       }
     }
   } else {
-    float y[N];
+    const bool pair = p.mode == kPair;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[i * VEC + e] = y[i * VEC + e] = 0.f;
+      for (int e = 0; e < VEC; ++e) v[i * VEC + e] = y[i * VEC + e] = z[i * VEC + e] = 0.f;
       if (c < W) {
         load_f<VEC>(p.x, t * W + c, v + i * VEC);
         load_h<VEC, H16>(p.y, t * p.ldy + c, p.h_type, y + i * VEC);
+        if (pair) load_h<VEC, H16>(p.y2, t * p.ldy2 + c, p.h_type, z + i * VEC);
       }
-    }
-    if (p.mode == kPair) {
-      float z[N], sy = 0.f, sz = 0.f;
-#pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int c = (i * TPR + tid) * VEC;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) z[i * VEC + e] = 0.f;
-        if (c < W) load_h<VEC, H16>(p.y2, t * p.ldy2 + c, p.h_type, z + i * VEC);
-      }
-#pragma unroll
-      for (int i = 0; i < N; ++i) { sy = fmaf(y[i], y[i], sy); sz = fmaf(z[i], z[i], sz); }
-      row_sums<TPR>(sy, sz, red);
-      const float iy = 1.f / sqrtf(sy * inv_n + p.eps), iz = 1.f / sqrtf(sz * inv_n + p.eps);
-#pragma unroll
-      for (int i = 0; i < NV; ++i) {
-        const int c = (i * TPR + tid) * VEC;
-        if (c < W) {
-          float wy[VEC], wz[VEC];
-          load_f<VEC>(p.w_y, c, wy);
-          load_f<VEC>(p.w_y2, c, wz);
-#pragma unroll
-          for (int e = 0; e < VEC; ++e)
-            v[i * VEC + e] += fmaf(y[i * VEC + e] * iy, wy[e], z[i * VEC + e] * iz * wz[e]);
-        }
-      }
-    } else {
-#pragma unroll
-      for (int i = 0; i < N; ++i) v[i] += y[i];
     }
     if (p.f != nullptr) {
 #pragma unroll
@@ -306,9 +242,6 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
       }
     }
     if (p.routed != nullptr) {
-      float g[N];
-#pragma unroll
-      for (int i = 0; i < N; ++i) g[i] = 0.f;
 #pragma unroll 4
       for (int k = 0; k < p.top; ++k) {
         const long at = t * p.top + k;
@@ -321,13 +254,71 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
             float q[VEC];
             load_h<VEC, H16>(p.routed, s * p.ldr + c, p.h_type, q);
 #pragma unroll
-            for (int e = 0; e < VEC; ++e) g[i * VEC + e] = fmaf(w, q[e], g[i * VEC + e]);
+            for (int e = 0; e < VEC; ++e) v[i * VEC + e] = fmaf(w, q[e], v[i * VEC + e]);
           }
         }
       }
-#pragma unroll
-      for (int i = 0; i < N; ++i) v[i] += g[i];
     }
+    if (pair) {
+      float sy = 0.f, sz = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) { sy = fmaf(y[i], y[i], sy); sz = fmaf(z[i], z[i], sz); }
+      row_sums<TPR>(sy, sz, red);
+      const float iy = 1.f / sqrtf(sy * inv_n + p.eps), iz = 1.f / sqrtf(sz * inv_n + p.eps);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * TPR + tid) * VEC;
+        if (c < W) {
+          float wy[VEC], wz[VEC];
+          load_f<VEC>(p.w_y, c, wy);
+          load_f<VEC>(p.w_y2, c, wz);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) v[i * VEC + e] += fmaf(y[i * VEC + e] * iy, wy[e], z[i * VEC + e] * iz * wz[e]);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < N; ++i) v[i] += y[i];
+    }
+  }
+
+  // what the ring contributes does not wait for this token's norm: partial h1 and h2, and the previous token's h1
+  [[maybe_unused]] float s1[TOKEN ? N : 1], s2[TOKEN ? N : 1], before[TOKEN ? N : 1];
+  [[maybe_unused]] const int pos = len - 1, R = p.taps + 1;
+  [[maybe_unused]] float* ring = TOKEN ? p.ring + static_cast<long>(slot) * R * W : nullptr;
+  if constexpr (TOKEN) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) s1[i] = s2[i] = before[i] = 0.f;
+    auto back = [&](int j) {               // j tokens back
+      if (j > p.taps || pos - j < 0) return;
+      const float* row = ring + static_cast<long>((pos - j) % R) * W;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (i * TPR + tid) * VEC;
+        if (c < W) {
+          float u[VEC], a[VEC];
+          load_f<VEC>(row, c, u);
+          if (p.mu != nullptr) {
+            load_f<VEC>(p.a1, static_cast<long>(p.taps - j) * W + c, a);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) before[i * VEC + e] = fmaf(a[e], u[e], before[i * VEC + e]);
+          }
+          if (j < p.taps) {
+            load_f<VEC>(p.a1, static_cast<long>(p.taps - 1 - j) * W + c, a);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) s1[i * VEC + e] = fmaf(a[e], u[e], s1[i * VEC + e]);
+            if (p.a2 != nullptr) {
+              load_f<VEC>(p.a2, static_cast<long>(p.taps - 1 - j) * W + c, a);
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) s2[i * VEC + e] = fmaf(a[e], u[e], s2[i * VEC + e]);
+            }
+          }
+        }
+      }
+    };
+#pragma unroll
+    for (int j = 1; j <= 4; ++j) back(j);
+    for (int j = 5; j <= p.taps; ++j) back(j);
   }
 
   float ss = 0.f, none = 0.f;
@@ -342,11 +333,11 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
   }
   row_sums<TPR>(ss, none, red);
   const float inv = 1.f / sqrtf(ss * inv_n + p.eps);
-  if (p.out_kind == kInv) {
-    if (tid == 0) p.inv[t] = inv;
-    return;
-  }
-  if (p.out_kind == kNorm) {
+  if constexpr (!TOKEN) {
+    if (p.out_kind == kInv) {
+      if (tid == 0) p.inv[t] = inv;
+      return;
+    }
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (i * TPR + tid) * VEC;
@@ -358,39 +349,39 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
         store_h<VEC, H16>(p.out, r * p.ldo + c, p.h_type, w);
       }
     }
-    return;
-  }
-  float* mine = ring + static_cast<long>(pos % R) * W;
+  } else {
+    float* mine = ring + static_cast<long>(pos % R) * W;
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int c = (i * TPR + tid) * VEC;
-    if (c >= W) continue;
-    float a[VEC], h[VEC], n[VEC];
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * TPR + tid) * VEC;
+      if (c >= W) continue;
+      float a[VEC], h[VEC], n[VEC];
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) n[e] = v[i * VEC + e] * inv;
-    store_h<VEC, false>(mine, c, kFp32, n);
-    load_f<VEC>(p.a1, static_cast<long>(p.taps - 1) * W + c, a);
+      for (int e = 0; e < VEC; ++e) n[e] = v[i * VEC + e] * inv;
+      store_h<VEC, false>(mine, c, kFp32, n);
+      load_f<VEC>(p.a1, static_cast<long>(p.taps - 1) * W + c, a);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) h[e] = fmaf(a[e], n[e], s1[i * VEC + e]);
-    long at = static_cast<long>(r) * p.ldo + c;
-    store_h<VEC, H16>(p.out, at, p.h_type, h);
-    if (p.a2 != nullptr) {
-      float g[VEC];
-      load_f<VEC>(p.a2, static_cast<long>(p.taps - 1) * W + c, a);
+      for (int e = 0; e < VEC; ++e) h[e] = fmaf(a[e], n[e], s1[i * VEC + e]);
+      long at = static_cast<long>(r) * p.ldo + c;
+      store_h<VEC, H16>(p.out, at, p.h_type, h);
+      if (p.a2 != nullptr) {
+        float g[VEC];
+        load_f<VEC>(p.a2, static_cast<long>(p.taps - 1) * W + c, a);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) g[e] = fmaf(a[e], n[e], s2[i * VEC + e]);
-      at += p.out_stride;
-      store_h<VEC, H16>(p.out, at, p.h_type, g);
-    }
-    if (p.mu != nullptr) {
-#pragma unroll
-      for (int k = 0; k < kBlends; ++k) {
-        float m[VEC];
-        load_f<VEC>(p.mu, static_cast<long>(k) * W + c, m);
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) m[e] = fmaf(before[i * VEC + e] - h[e], m[e], h[e]);
+        for (int e = 0; e < VEC; ++e) g[e] = fmaf(a[e], n[e], s2[i * VEC + e]);
         at += p.out_stride;
-        store_h<VEC, H16>(p.out, at, p.h_type, m);
+        store_h<VEC, H16>(p.out, at, p.h_type, g);
+      }
+      if (p.mu != nullptr) {
+#pragma unroll
+        for (int k = 0; k < kBlends; ++k) {
+          float m[VEC];
+          load_f<VEC>(p.mu, static_cast<long>(k) * W + c, m);
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) m[e] = fmaf(before[i * VEC + e] - h[e], m[e], h[e]);
+          at += p.out_stride;
+          store_h<VEC, H16>(p.out, at, p.h_type, m);
+        }
       }
     }
   }
@@ -502,8 +493,9 @@ template <int TPR, int VEC, int NV>
 int launch_rows(const ShiftParams& p, cudaStream_t s) {
   constexpr int threads = block_threads(TPR), per = threads / TPR;
   const dim3 g(static_cast<unsigned>((p.rows + per - 1) / per));
-  if (p.h_type == kFp32) return static_cast<int>(fi::launch_kernel(shift_rows_kernel<TPR, VEC, NV, false>, g, dim3(threads), 0, s, 0, p));
-  return static_cast<int>(fi::launch_kernel(shift_rows_kernel<TPR, VEC, NV, true>, g, dim3(threads), 0, s, 0, p));
+  auto kern = p.out_kind == kToken ? (p.h_type == kFp32 ? shift_rows_kernel<TPR, VEC, NV, false, true> : shift_rows_kernel<TPR, VEC, NV, true, true>)
+                                   : (p.h_type == kFp32 ? shift_rows_kernel<TPR, VEC, NV, false, false> : shift_rows_kernel<TPR, VEC, NV, true, false>);
+  return static_cast<int>(fi::launch_kernel(kern, g, dim3(threads), 0, s, 0, p));
 }
 
 template <int KT>
@@ -537,7 +529,7 @@ int dispatch_rows(const ShiftParams& p, cudaStream_t s) {
     if (W <= 512) return launch_rows<32, 4, 4>(p, s);
   }
   if (W <= 1024) return launch_rows<256, 4, 1>(p, s);
-  if (W <= 2048) return launch_rows<512, 4, 1>(p, s);
+  if (W <= 2048) return few ? launch_rows<512, 4, 1>(p, s) : launch_rows<256, 4, 2>(p, s);
   if (W <= 4096) return launch_rows<512, 4, 2>(p, s);
   if (W <= 8192) return launch_rows<512, 4, 4>(p, s);
   return -11;

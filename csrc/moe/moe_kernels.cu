@@ -267,6 +267,21 @@ __global__ void __launch_bounds__(256) moe_lookup_kernel(const int* __restrict__
   topk_w[i] = weight;
 }
 
+// Tile table of E stacked matrices of T rows each.
+__global__ void __launch_bounds__(256) stack_tiles_kernel(int E, int T, int bn, int per, int* __restrict__ tile_expert,
+                                                          int* __restrict__ tile_row0, int* __restrict__ tile_rows,
+                                                          int* __restrict__ n_tiles) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i == 0) *n_tiles = E * per;
+  if (i >= E * per) return;
+  const int e = i / per, r = (i % per) * bn;
+  tile_expert[i] = e;
+  tile_row0[i] = e * T + r;
+  tile_rows[i] = min(bn, T - r);
+}
+
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ sorted_route,
                                   const int* __restrict__ expert_offsets, int EL, int K, int H,
@@ -563,6 +578,15 @@ extern "C" int fi_moe_lookup(const int* table, const long long* ids, int vocab, 
   if (vocab <= 0 || top <= 0 || static_cast<long>(T) * top > 2147483647l) return -10;
   return static_cast<int>(fi::launch_kernel(moe_lookup_kernel, dim3((T * top + 255) / 256), dim3(256), 0, FI_STREAM(stream), 0, table,
                                             ids, vocab, T * top, top, weight, topk_ids, topk_w));
+}
+
+// Tile table (as of fi_moe_align) of E stacked matrices of T rows: E * ceil(T / bn) tiles.
+extern "C" int fi_stack_tiles(int E, int T, int bn, int* tile_expert, int* tile_row0, int* tile_rows, int* n_tiles, void* stream) {
+  if (E <= 0 || T <= 0) return 0;
+  if (bn <= 0) return -10;
+  const int per = (T + bn - 1) / bn;
+  return static_cast<int>(fi::launch_kernel(stack_tiles_kernel, dim3((E * per + 255) / 256), dim3(256), 0, FI_STREAM(stream), 0, E, T, bn,
+                                            per, tile_expert, tile_row0, tile_rows, n_tiles));
 }
 
 extern "C" int fi_moe_align(const int* topk_ids, int n_routes, int e_lo, int e_hi, int bn,

@@ -7,7 +7,7 @@ and the decay each read their own blend of the present and the previous input:
     y = W_o [rms(o_h) norm_h gate_h]
 
 The state S [heads, dim, dim] is 32-bit and lives in a per-layer pool of the cache manager with one slot per request.  The
-four square projections run as one grouped product (steps of many tokens: one by one).  Portions of prompts run one scan
+four square projections run as one grouped product.  Portions of prompts run one scan
 kernel for the whole step, decode one step kernel that includes norm and gate.
 """
 from __future__ import annotations

@@ -443,7 +443,7 @@ def conv_silu(x, w, bias, ring, batch, out_dtype):
             ring_store(ring[slot], pos0, x[lo:hi].float())
         return y.to(out_dtype)
     from .shift_stream import tiles
-    base, n_tiles, tile = tiles(batch, taps)
+    base, n_tiles, tile = tiles(batch, taps, C)
     assert x.stride(1) == 1 and ring.is_contiguous() and w.is_contiguous() and ring.dtype == w.dtype == bias.dtype == torch.float32
     y = torch.empty(T, C, dtype=out_dtype, device=x.device)
     rc = _lib.kernels().fi_conv_silu(_p(x), x.stride(0), _p(w), _p(bias), taps, _p(ring), _p(y), _p(batch.extras["slot_ids"]),

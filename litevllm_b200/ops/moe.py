@@ -103,36 +103,50 @@ class RoutedRows:
         return (r * self.weights[..., None]).sum(1)
 
 
-_stack_tiles: dict[tuple, torch.Tensor] = {}
+_stack_tables: dict[tuple, torch.Tensor] = {}
 
 
-def _stacked_tile_table(E: int, T: int, bn: int, device) -> torch.Tensor:
-    """int32 [3, n]: matrix, first row and rows of each tile of ``bn`` rows of E stacked matrices of T rows.  Tables stay
-    alive: captured steps hold their addresses."""
+def _stacked_tile_table(E: int, T: int, bn: int, device) -> tuple[torch.Tensor, int]:
+    """(int32 table, number of tiles n): matrix [n], first row [n] and rows [n] of each tile of ``bn`` rows of E stacked matrices
+    of T rows, then n itself.  The few tables of small steps are kept (captured steps hold their addresses), others are
+    written by a kernel."""
+    n = E * -(-T // bn)
     key = (E, T, bn, str(device))
-    if key not in _stack_tiles:
-        rows = [(e, e * T + t, min(bn, T - t)) for e in range(E) for t in range(0, T, bn)]
-        with torch.inference_mode(False):
-            _stack_tiles[key] = torch.tensor(rows + [(len(rows),) * 3], dtype=torch.int32, device="cpu").t().contiguous().to(device)
-    return _stack_tiles[key]
+    t = _stack_tables.get(key)
+    if t is None:
+        if T <= 64:
+            with torch.inference_mode(False):
+                t = _stack_tables[key] = torch.empty(3 * n + 1, dtype=torch.int32, device=device)
+        else:
+            t = scratch("stack_tiles", (3 * n + 1) * 4, device).view(torch.int32)[:3 * n + 1]
+        at = t.data_ptr()
+        rc = _lib.kernels().fi_stack_tiles(E, T, bn, at, at + 4 * n, at + 8 * n, at + 12 * n, _stream())
+        _lib.check(rc, "fi_stack_tiles")
+        _count()
+    return t, n
 
 
 def stacked_linear(x: torch.Tensor, w: torch.Tensor):
-    """x [E, T, K] (rows of one pitch, matrices back to back), w [E, N, K] -> E matrices [T, N].  Small steps run one grouped product."""
+    """x [E, T, K] (rows of one pitch, matrices back to back), w [E, N, K] -> E matrices [T, N], by one grouped product."""
     from .. import ops
     E, T, K = x.shape
     N = w.shape[1]
-    if not x.is_cuda or x.dtype == torch.float32 or T >= ops._PERSISTENT_MIN_T or K % 8 or N % 8 or x.stride(1) % 8 \
+    if not x.is_cuda or x.dtype == torch.float32 or K % 8 or N % 8 or x.stride(1) % 8 \
             or x.stride(0) != T * x.stride(1) or x.data_ptr() % 16 or not w.is_contiguous():
         return [ops.linear(x[e], w[e]) for e in range(E)]
     out = torch.empty(E, T, N, dtype=x.dtype, device=x.device)
-    bn = 16 if T <= 16 else 32 if T <= 32 else 64
-    t = _stacked_tile_table(E, T, bn, x.device)
-    n = t.shape[1] - 1
-    g = FiGrouped(t[0].data_ptr(), t[1].data_ptr(), t[2].data_ptr(), t[0, n:].data_ptr(), n, E, N, 0)
-    rc = _lib.kernels().fi_dense_gemm_grouped(_p(x), _p(w), _p(out), E * T, N, K, x.stride(1), N, 0, 0.0, 0, _DT[x.dtype], bn,
-                                              ctypes.byref(g), _p(status_word(x.device)), _stream())
-    _lib.check(rc, "fi_dense_gemm_grouped")
+    many = T >= ops._PERSISTENT_MIN_T
+    bn = 128 if many else 16 if T <= 16 else 32 if T <= 32 else 64
+    t, n = _stacked_tile_table(E, T, bn, x.device)
+    at = t.data_ptr()
+    g = FiGrouped(at, at + 4 * n, at + 8 * n, at + 12 * n, n, E, N, 0)
+    if many:
+        rc = _lib.kernels().fi_dense_gemm_persistent_grouped(_p(x), _p(w), _p(out), E * T, N, K, x.stride(1), N, 0, 0.0, 0, _DT[x.dtype],
+                                                             ctypes.byref(g), _p(status_word(x.device)), _stream())
+    else:
+        rc = _lib.kernels().fi_dense_gemm_grouped(_p(x), _p(w), _p(out), E * T, N, K, x.stride(1), N, 0, 0.0, 0, _DT[x.dtype], bn,
+                                                  ctypes.byref(g), _p(status_word(x.device)), _stream())
+    _lib.check(rc, "stacked_linear")
     _count()
     return out
 

@@ -79,9 +79,11 @@ class Paired:
     routed: object = None
 
 
-def tiles(batch, taps: int):
-    """(running count of tiles per portion int32 [B + 1], their number, tokens per tile) of the convolution kernels."""
-    t = 16 if taps > 8 or sum(batch.q_lens_cpu) >= 4096 else 8
+def tiles(batch, taps: int, width: int):
+    """(running count of tiles per portion int32 [B + 1], their number, tokens per tile) of the convolution kernels on rows of
+    ``width`` channels: long tiles where they still fill the device."""
+    T, blocks = sum(batch.q_lens_cpu), -(-width // 512)
+    t = next((n for n in (64, 32, 16) if T // n * blocks >= 888), 8 if taps <= 8 else 16)
     key = f"tiles{t}"
     if key not in batch.extras:
         n = (batch.cu_q[1:] - batch.cu_q[:-1] + t - 1) // t
@@ -191,7 +193,7 @@ def layer_inputs(src, x, spec: ShiftSpec, ring, batch, eps: float, h_dtype):
     _lib.check(rc, "fi_shift_rows")
     _count()
     if not decode:
-        base, n_tiles, tile = tiles(batch, spec.taps)
+        base, n_tiles, tile = tiles(batch, spec.taps, W)
         first = isinstance(src, Embedded)
         rc = lib.fi_shift_conv(_p(x), _p(inv), _p(spec.a1), _p(spec.a2), _p(spec.mu), spec.taps, _p(ring), _p(buf), w8, T * w8,
                                _p(src.ids) if first else None, _p(src.last_token) if first else None, _p(slots),
