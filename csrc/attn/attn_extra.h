@@ -53,6 +53,19 @@ __device__ __forceinline__ void turn_back(const P& p, int pos, int i, float& u, 
   u = a * c + v * s;
   v = v * c - a * s;
 }
+// The same for pairs i .. i + 3 (channels y[0] .. y[7]); i is a multiple of four, and so is out_dim / 2.
+template <typename P>
+__device__ __forceinline__ void turn_back4(const P& p, int pos, int i, float* y) {
+  const float* row = p.x.turn + static_cast<long>(pos < 0 ? 0 : pos >= p.x.turn_rows ? p.x.turn_rows - 1 : pos) * p.x.out_dim + i;
+  const float4 c4 = *reinterpret_cast<const float4*>(row), s4 = *reinterpret_cast<const float4*>(row + p.x.out_dim / 2);
+  const float c[4] = {c4.x, c4.y, c4.z, c4.w}, s[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float u = y[2 * e], v = y[2 * e + 1];
+    y[2 * e] = u * c[e] + v * s[e];
+    y[2 * e + 1] = v * c[e] - u * s[e];
+  }
+}
 #endif
 
 }  // namespace fi

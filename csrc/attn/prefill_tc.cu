@@ -347,16 +347,20 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       const int k0 = (tile_begin + j) * kTile + half * 64;   // first key of this thread's 64
       float alpha = 1.f;
       if constexpr (SIG) {
-        // weights 1 / (1 + e^-s), two at a time with one reciprocal; exponents are held where the product of two sums
-        // stays finite (a weight that small is zero beside any other)
+        // weights 1 / (1 + e^-s), four at a time with one reciprocal; exponents are held where the product of four sums
+        // stays finite (thousands of weights that small are nothing beside the rounding of one)
 #pragma unroll
         for (int e = 0; e < 64; ++e)
-          sr[e] = __float_as_uint(1.f + fast_exp2(fminf(fmaf(__uint_as_float(sr[e]), -sl2, nb), 60.f)));
+          sr[e] = __float_as_uint(1.f + fast_exp2(fminf(fmaf(__uint_as_float(sr[e]), -sl2, nb), 31.f)));
 #pragma unroll
-        for (int e = 0; e < 64; e += 2) {
-          const float a = __uint_as_float(sr[e]), c = __uint_as_float(sr[e + 1]), inv = __fdividef(1.f, a * c);
-          sr[e] = __float_as_uint(inv * c);
-          sr[e + 1] = __float_as_uint(inv * a);
+        for (int e = 0; e < 64; e += 4) {
+          const float a0 = __uint_as_float(sr[e]), a1 = __uint_as_float(sr[e + 1]), a2 = __uint_as_float(sr[e + 2]),
+                      a3 = __uint_as_float(sr[e + 3]);
+          const float lo = a0 * a1, hi = a2 * a3, inv = __fdividef(1.f, lo * hi), il = inv * hi, ih = inv * lo;
+          sr[e] = __float_as_uint(il * a1);
+          sr[e + 1] = __float_as_uint(il * a0);
+          sr[e + 2] = __float_as_uint(ih * a3);
+          sr[e + 3] = __float_as_uint(ih * a2);
         }
         if ((k0 + 63 > first_pos) || k0 < edge_lo) {
           const int vis_hi = qpos - k0 + 1, vis_lo = row_lo - k0;
@@ -496,9 +500,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 #pragma unroll
           for (int e = 0; e < 8; ++e) y[e] = o[c * 8 + e] * inv;
           if constexpr (SIG) {
-            if (p.x.turn != nullptr)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) fi::turn_back(p, qpos, (half * HH + c * 8) / 2 + e, y[2 * e], y[2 * e + 1]);
+            if (p.x.turn != nullptr) fi::turn_back4(p, qpos, (half * HH + c * 8) / 2, y);       // out_dim is a multiple of 8
           }
           if (p.x.gate != nullptr && !p.x.gate_per_head) {
             const uint4 raw = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.x.gate) +
@@ -599,6 +601,7 @@ extern "C" int fi_paged_prefill_tc(const void* q, long q_stride, const void* k_c
   p.max_blocks = max_blocks; p.block_size = block_size; p.nh = nh; p.nkv = nkv; p.window = window;
   p.sm_scale = sm_scale; p.softcap = softcap; p.is_fp16 = dtype == 1;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (p.x.turn != nullptr && (reinterpret_cast<uintptr_t>(p.x.turn) & 15) != 0) return -12;
   if (p.x.bias != nullptr)
     return hd == 64 ? launch_tc<64, 6, 1, true>(qm, km, vm, p, B, max_q_len, s) : launch_tc<128, 3, 1, true>(qm, km, vm, p, B, max_q_len, s);
   if (hd == 64)

@@ -20,6 +20,10 @@ __device__ __forceinline__ void pdl_launch_dependents() {
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
 }
 
+// Ask for a line in L2.  A hint without effect on results, so it may come ahead of pdl_wait() for weights and for memory
+// that other kernels still write.
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 // On by default (measured 1.58 -> 1.38 ms per TinyLlama decode step at batch 32); the environment
 // variable FI_USE_PDL=0, read once when the library is first used, restores fully serialised launches.
 inline bool use_pdl() {

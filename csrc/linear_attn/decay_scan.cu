@@ -334,6 +334,13 @@ __device__ __forceinline__ float block_sum(float v, float* red) {      // 256 th
 template <int VEC, int KIND>
 __global__ void __launch_bounds__(256, 3) decay_step_kernel(const ScanParams p) {
   fi::pdl_launch_dependents();
+  {                                        // the state comes from memory: ask for it while the predecessor ends
+    const int s = p.slots[blockIdx.y];
+    if (p.seq_lens[blockIdx.y] > 1 && s >= 0 && s < p.num_slots) {
+      const float* S = p.pool + (static_cast<long>(s) * p.H + blockIdx.x) * p.d * p.dv;
+      for (int i = threadIdx.x * 32; i < p.d * p.dv; i += 256 * 32) fi::prefetch_l2(S + i);
+    }
+  }
   fi::pdl_wait();
   extern __shared__ __align__(16) float smem[];
   __shared__ float red[2][8];
@@ -396,14 +403,21 @@ __global__ void __launch_bounds__(256, 3) decay_step_kernel(const ScanParams p) 
     g = p.u[head];
     const int pos = len - 1, taps = p.taps;
     float* ring = p.ring + static_cast<long>(slot) * taps * p.C;
-    const int inner = p.H * dv;
+    const int inner = p.H * dv, at = pos % taps;
+#pragma unroll 2
     for (int c = tid; c < 2 * d + dv; c += 256) {
       const int ch = c < d ? inner + (p.G + group) * d + c : (c < 2 * d ? inner + group * d + c - d : head * dv + c - 2 * d);
       const float now = ld_any(p.xbc, b * p.ldq + ch, p.type);
       float y = fmaf(p.conv[static_cast<long>(taps - 1) * p.C + ch], now, p.conv_b[ch]);
-      for (int j = 1; j < taps; ++j)
-        if (pos - j >= 0) y = fmaf(p.conv[static_cast<long>(taps - 1 - j) * p.C + ch], ring[static_cast<long>((pos - j) % taps) * p.C + ch], y);
-      if (c >= 2 * d || head % per == 0) ring[static_cast<long>(pos % taps) * p.C + ch] = now;
+      auto back = [&](int j) {             // j tokens back
+        if (j >= taps || pos - j < 0) return;
+        const int row = at >= j ? at - j : at - j + taps;
+        y = fmaf(p.conv[static_cast<long>(taps - 1 - j) * p.C + ch], ring[static_cast<long>(row) * p.C + ch], y);
+      };
+#pragma unroll
+      for (int j = 1; j < 4; ++j) back(j);
+      for (int j = 4; j < taps; ++j) back(j);
+      if (c >= 2 * d || head % per == 0) ring[static_cast<long>(at) * p.C + ch] = now;
       y *= sigmoidf(y);
       if (c < d) sq[c] = y;
       else if (c < 2 * d) sk[c - d] = dt * y;
@@ -481,20 +495,43 @@ struct ConvParams {
   int B, C, taps, tile, num_slots, type, out_type;
 };
 
-template <int VEC, typename T>
-__device__ __forceinline__ void load_x(const T* p, int type, float* v) {
-  if constexpr (VEC == 4) {
-    expand4(load4(p, 4, 1), type, v);
-  } else if constexpr (sizeof(T) == 4) {
-    v[0] = p[0];
+// VEC values of type TYPE (known at compile time: the convolution is bound by its instructions).
+template <int VEC, int TYPE>
+__device__ __forceinline__ void load_as(const void* p, long i, float* v) {
+  if constexpr (TYPE == kFp32) {
+    const float* f = reinterpret_cast<const float*>(p) + i;
+    if constexpr (VEC == 4) expand4(load4(f, 4, 1), kFp32, v); else v[0] = f[0];
+  } else if constexpr (VEC == 4) {
+    expand4(load4(reinterpret_cast<const uint16_t*>(p) + i, 4, 1), TYPE, v);
   } else {
-    v[0] = ld_any(p, 0, type);
+    v[0] = ld_any(p, i, TYPE);
+  }
+}
+template <int VEC, int TYPE>
+__device__ __forceinline__ void store_as(void* p, long i, const float* v) {
+  if constexpr (VEC == 1) {
+    st_any(p, i, TYPE, v[0]);
+  } else if constexpr (TYPE == kFp32) {
+    *reinterpret_cast<float4*>(reinterpret_cast<float*>(p) + i) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    uint32_t w[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      if constexpr (TYPE == kBf16) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+        w[e] = *reinterpret_cast<const uint32_t*>(&h);
+      } else {
+        const __half2 h = __floats2half2_rn(v[2 * e], v[2 * e + 1]);
+        w[e] = *reinterpret_cast<const uint32_t*>(&h);
+      }
+    }
+    *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p) + i) = make_uint2(w[0], w[1]);
   }
 }
 
-// KT >= taps: registers of the sliding window (leading taps of weight zero).
-template <int KT, int VEC, typename T>
-__global__ void __launch_bounds__(128) conv_silu_kernel(const ConvParams p) {
+// KT >= taps: registers of the sliding window (leading taps of weight zero).  IN, OUT: types of x and out.
+template <int KT, int VEC, int IN, int OUT>
+__global__ void __launch_bounds__(128, KT > 4 ? 1 : 8) conv_silu_kernel(const ConvParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   int lo = 0, hi = p.B - 1;
@@ -509,73 +546,66 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvParams p) {
   if (i0 < 0 || i0 >= n || slot < 0 || slot >= p.num_slots || c >= p.C) return;
   const int taps = p.taps;
   float* ring = p.ring + static_cast<long>(slot) * taps * p.C + c;
-  const T* x = reinterpret_cast<const T*>(p.x) + t_begin * p.ld + c;
-  float a[KT][VEC], win[KT][VEC], bias[VEC];
+  const long x0 = t_begin * p.ld + c;
+  float a[KT][VEC], seq[KT + 3][VEC], bias[VEC];             // seq: the KT - 1 inputs before the present four, then those
 #pragma unroll
   for (int j = 0; j < KT; ++j) {
-    const int tap = j - (KT - taps), i = i0 - KT + 1 + j;     // the window before this tile's first token, in places 0 .. KT - 2
+    const int tap = j - (KT - taps), i = i0 - KT + 1 + j;
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) a[j][e] = win[j][e] = 0.f;
+    for (int e = 0; e < VEC; ++e) a[j][e] = seq[j][e] = 0.f;
     if (tap >= 0) {
-      load_x<VEC>(p.w + static_cast<long>(tap) * p.C + c, kFp32, a[j]);
+      load_as<VEC, kFp32>(p.w, static_cast<long>(tap) * p.C + c, a[j]);
       if (j + 1 < KT) {
-        if (i >= 0) load_x<VEC>(x + i * p.ld, p.type, win[j]);
-        else if (pos0 + i >= 0) load_x<VEC>(ring + static_cast<long>((pos0 + i) % taps) * p.C, kFp32, win[j]);
+        if (i >= 0) load_as<VEC, IN>(p.x, x0 + i * p.ld, seq[j]);
+        else if (pos0 + i >= 0) load_as<VEC, kFp32>(ring, static_cast<long>((pos0 + i) % taps) * p.C, seq[j]);
       }
     }
   }
-  load_x<VEC>(p.bias + c, kFp32, bias);
+  load_as<VEC, kFp32>(p.bias, c, bias);
   const int i_end = min(n, i0 + p.tile);
   for (int i = i0; i < i_end; i += 4) {
-    float xn[4][VEC];
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) xn[u][e] = 0.f;
-      if (i + u < i_end) load_x<VEC>(x + (i + u) * p.ld, p.type, xn[u]);
+      for (int e = 0; e < VEC; ++e) seq[KT - 1 + u][e] = 0.f;
+      if (i + u < i_end) load_as<VEC, IN>(p.x, x0 + (i + u) * p.ld, seq[KT - 1 + u]);
     }
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       if (i + u >= i_end) break;
       float y[VEC];
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) {
-        win[KT - 1][e] = xn[u][e];
-        y[e] = bias[e];
-      }
+      for (int e = 0; e < VEC; ++e) y[e] = bias[e];
 #pragma unroll
       for (int j = 0; j < KT; ++j)
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) y[e] = fmaf(a[j][e], win[j][e], y[e]);
+        for (int e = 0; e < VEC; ++e) y[e] = fmaf(a[j][e], seq[j + u][e], y[e]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) y[e] *= sigmoidf(y[e]);
-      const long at = static_cast<long>(t_begin + i + u) * p.C + c;
-      if constexpr (VEC == 4) {
-        if (p.out_type == kFp32) {
-          *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + at) = make_float4(y[0], y[1], y[2], y[3]);
-        } else {
-          alignas(8) uint16_t h[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e)
-            h[e] = p.out_type == kBf16 ? __bfloat16_as_ushort(__float2bfloat16_rn(y[e])) : __half_as_ushort(__float2half_rn(y[e]));
-          *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p.out) + at) = *reinterpret_cast<const uint2*>(h);
-        }
-      } else {
-        st_any(p.out, at, p.out_type, y[0]);
-      }
-#pragma unroll
-      for (int j = 0; j + 1 < KT; ++j)
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) win[j][e] = win[j + 1][e];
+      store_as<VEC, OUT>(p.out, static_cast<long>(t_begin + i + u) * p.C + c, y);
     }
+#pragma unroll
+    for (int j = 0; j + 1 < KT; ++j)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) seq[j][e] = seq[j + 4][e];
   }
   if (i0 == 0)
     for (int i = max(0, n - taps); i < n; ++i) {
       float v[VEC];
-      load_x<VEC>(x + i * p.ld, p.type, v);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) ring[static_cast<long>((pos0 + i) % taps) * p.C + e] = v[e];
+      load_as<VEC, IN>(p.x, x0 + i * p.ld, v);
+      store_as<VEC, kFp32>(ring, static_cast<long>((pos0 + i) % taps) * p.C, v);
     }
+}
+
+template <int KT, int VEC>
+int launch_conv(const ConvParams& p, int tiles, cudaStream_t s) {
+  const dim3 g(tiles, (p.C + 128 * VEC - 1) / (128 * VEC));
+  auto kern = p.type == kFp32 ? (p.out_type == kFp32   ? conv_silu_kernel<KT, VEC, kFp32, kFp32>
+                                 : p.out_type == kBf16 ? conv_silu_kernel<KT, VEC, kFp32, kBf16>
+                                                       : conv_silu_kernel<KT, VEC, kFp32, kFp16>)
+              : p.type == kBf16 ? conv_silu_kernel<KT, VEC, kBf16, kBf16>
+                                : conv_silu_kernel<KT, VEC, kFp16, kFp16>;
+  return static_cast<int>(fi::launch_kernel(kern, g, dim3(128), 0, s, 0, p));
 }
 
 struct NormParams {
@@ -779,31 +809,25 @@ extern "C" int fi_decay_step_conv(const void* xbc, long ld, const float* z, long
   return dispatch_step<kScalar>(p, B, reinterpret_cast<cudaStream_t>(stream));
 }
 
-// Convolution with bias and SiLU over portions: x [T, ld] (type) -> out [T, C] (out_type); w fp32 [taps, C]; ring as above;
+// Convolution with bias and SiLU over portions: x [T, ld] (type) -> out [T, C] (out_type; the same or, from 32-bit, any); w fp32 [taps, C]; ring as above;
 // tile_base int32 [B + 1] counts tiles of `tile` tokens (at least taps), n_tiles its last entry.
 extern "C" int fi_conv_silu(const void* x, long ld, const float* w, const float* bias, int taps, float* ring, void* out,
                             const int* slots, const int* cu_q, const int* seq_lens, const int* tile_base, int n_tiles, int tile,
                             int B, int C, int num_slots, int type, int out_type, void* stream) {
   if (n_tiles <= 0 || B <= 0) return 0;
-  if (C <= 0 || taps <= 0 || taps > 16 || tile < taps || type < 0 || type > 2 || out_type < 0 || out_type > 2) return -10;
+  if (C <= 0 || taps <= 0 || taps > 16 || tile < taps || type < 0 || type > 2 || out_type < 0 || out_type > 2 ||
+      (type != kFp32 && out_type != type))
+    return -10;
   ConvParams p = {};
   p.x = x; p.ld = ld; p.w = w; p.bias = bias; p.taps = taps; p.ring = ring; p.out = out; p.slots = slots; p.cu_q = cu_q;
   p.seq_lens = seq_lens; p.tile_base = tile_base; p.tile = tile; p.B = B; p.C = C; p.num_slots = num_slots; p.type = type;
   p.out_type = out_type;
   const bool vec4 = C % 4 == 0 && ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(w) |
                                                    reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(ring)) & 15) == 0;
-  const dim3 g(n_tiles, (C + (vec4 ? 512 : 128) - 1) / (vec4 ? 512 : 128));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-#define FI_CONV(KT)                                                                                                   \
-  do {                                                                                                                \
-    auto kern = type == kFp32 ? (vec4 ? conv_silu_kernel<KT, 4, float> : conv_silu_kernel<KT, 1, float>)               \
-                              : (vec4 ? conv_silu_kernel<KT, 4, uint16_t> : conv_silu_kernel<KT, 1, uint16_t>);        \
-    return static_cast<int>(fi::launch_kernel(kern, g, dim3(128), 0, s, 0, p));                                        \
-  } while (0)
-  if (taps <= 4) FI_CONV(4);
-  if (taps <= 8) FI_CONV(8);
-  FI_CONV(16);
-#undef FI_CONV
+  if (taps <= 4) return vec4 ? launch_conv<4, 4>(p, n_tiles, s) : launch_conv<4, 1>(p, n_tiles, s);
+  if (taps <= 8) return vec4 ? launch_conv<8, 4>(p, n_tiles, s) : launch_conv<8, 1>(p, n_tiles, s);
+  return launch_conv<16, 1>(p, n_tiles, s);
 }
 
 // out [T, parts * n] = norm over each part of n values of x fp32 [T, parts * n], times w, with a SiLU gate [T, ldg] (or null)

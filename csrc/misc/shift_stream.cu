@@ -142,6 +142,18 @@ constexpr int block_threads(int tpr) { return tpr > 256 ? tpr : 256; }
 template <int TPR, int VEC, int NV, bool H16, bool TOKEN>
 __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const ShiftParams p) {
   fi::pdl_launch_dependents();
+  if constexpr (TOKEN) {                   // weights of a decode step come from memory: ask for them while the predecessor ends
+    for (int c = static_cast<int>(threadIdx.x) % TPR * VEC; c < p.W; c += TPR * VEC) {
+      if (p.w_y != nullptr) fi::prefetch_l2(p.w_y + c);
+      if (p.w_y2 != nullptr) fi::prefetch_l2(p.w_y2 + c);
+      for (int j = 0; j < p.taps; ++j) {
+        fi::prefetch_l2(p.a1 + static_cast<long>(j) * p.W + c);
+        if (p.a2 != nullptr) fi::prefetch_l2(p.a2 + static_cast<long>(j) * p.W + c);
+      }
+      if (p.mu != nullptr)
+        for (int k = 0; k < kBlends; ++k) fi::prefetch_l2(p.mu + static_cast<long>(k) * p.W + c);
+    }
+  }
   fi::pdl_wait();
   __shared__ float red[2][16];
   constexpr int kRowsPerBlock = block_threads(TPR) / TPR, N = NV * VEC;
@@ -387,9 +399,23 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
   }
 }
 
-// KT >= taps: registers of the sliding window (leading taps of weight zero).
-template <int KT, int VEC, bool H16>
-__global__ void __launch_bounds__(128) shift_conv_kernel(const ShiftParams p) {
+// Stores in a type known at compile time (the convolution is bound by its instructions).
+template <int VEC, int H>
+__device__ __forceinline__ void store_as(void* p, long i, const float* v) {
+  if constexpr (H == kFp32) {
+    store_h<VEC, false>(p, i, kFp32, v);
+  } else if constexpr (VEC == 4 && H == kBf16) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+    *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p) + i) =
+        make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    store_h<VEC, true>(p, i, H, v);
+  }
+}
+
+// KT >= taps: registers of the sliding window (leading taps of weight zero).  MU: blends are formed.
+template <int KT, int VEC, int H, bool MU>
+__global__ void __launch_bounds__(128, KT > 4 ? 1 : MU ? 4 : 6) shift_conv_kernel(const ShiftParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   const int W = p.W, taps = p.taps, R = taps + 1;
@@ -410,76 +436,89 @@ __global__ void __launch_bounds__(128) shift_conv_kernel(const ShiftParams p) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v[e] *= inv;
   };
-  float a1[KT][VEC], a2[KT][VEC], mu[kBlends][VEC], win[KT][VEC], prev[VEC];
+  constexpr int HIST = MU ? KT : KT - 1;   // tokens before the present four; the blends also need the convolution one token back
+  float a1[KT][VEC], a2[KT][VEC], mu[MU ? kBlends : 1][VEC], seq[HIST + 4][VEC], prev[VEC];
 #pragma unroll
   for (int j = 0; j < KT; ++j) {
-    const int tap = j - (KT - taps), i = i0 - KT + j;
+    const int tap = j - (KT - taps);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) a1[j][e] = a2[j][e] = win[j][e] = 0.f;
+    for (int e = 0; e < VEC; ++e) a1[j][e] = a2[j][e] = 0.f;
     if (tap >= 0) {
       load_f<VEC>(p.a1, static_cast<long>(tap) * W + c, a1[j]);
       if (p.a2 != nullptr) load_f<VEC>(p.a2, static_cast<long>(tap) * W + c, a2[j]);
-      if (i >= 0) unit(i, win[j]);
-      else if (pos0 + i >= 0) load_f<VEC>(ring, static_cast<long>((pos0 + i) % R) * W, win[j]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < HIST; ++j) {
+    const int i = i0 - HIST + j;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) seq[j][e] = 0.f;
+    if (HIST - j <= taps) {                // the ring holds the last taps + 1 tokens
+      if (i >= 0) unit(i, seq[j]);
+      else if (pos0 + i >= 0) load_f<VEC>(ring, static_cast<long>((pos0 + i) % R) * W, seq[j]);
     }
   }
 #pragma unroll
   for (int e = 0; e < VEC; ++e) prev[e] = 0.f;
-  if (p.mu != nullptr) {
+  if constexpr (MU) {
 #pragma unroll
     for (int k = 0; k < kBlends; ++k) load_f<VEC>(p.mu, static_cast<long>(k) * W + c, mu[k]);
 #pragma unroll
     for (int j = 0; j < KT; ++j)
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) prev[e] = fmaf(a1[j][e], win[j][e], prev[e]);
+      for (int e = 0; e < VEC; ++e) prev[e] = fmaf(a1[j][e], seq[j][e], prev[e]);
   }
   const int i_end = min(n, i0 + p.tile);
   for (int i = i0; i < i_end; i += 4) {
-    float x[4][VEC];
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) x[u][e] = 0.f;
-      if (i + u < i_end) unit(i + u, x[u]);
+      for (int e = 0; e < VEC; ++e) seq[HIST + u][e] = 0.f;
+      if (i + u < i_end) unit(i + u, seq[HIST + u]);
     }
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       if (i + u >= i_end) break;
+      constexpr int kFirst = HIST - KT + 1;                  // seq[kFirst + u + KT - 1] is token i + u
+      float h[VEC];
 #pragma unroll
-      for (int j = 0; j + 1 < KT; ++j)
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) win[j][e] = win[j + 1][e];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) win[KT - 1][e] = x[u][e];
-      float h[VEC], g[VEC];
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) h[e] = g[e] = 0.f;
+      for (int e = 0; e < VEC; ++e) h[e] = 0.f;
 #pragma unroll
       for (int j = 0; j < KT; ++j)
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-          h[e] = fmaf(a1[j][e], win[j][e], h[e]);
-          g[e] = fmaf(a2[j][e], win[j][e], g[e]);
-        }
+        for (int e = 0; e < VEC; ++e) h[e] = fmaf(a1[j][e], seq[kFirst + u + j][e], h[e]);
       long at = static_cast<long>(t_begin + i + u) * p.ldo + c;
-      store_h<VEC, H16>(p.out, at, p.h_type, h);
+      store_as<VEC, H>(p.out, at, h);
       if (p.a2 != nullptr) {
+        float g[VEC];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) g[e] = 0.f;
+#pragma unroll
+        for (int j = 0; j < KT; ++j)
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) g[e] = fmaf(a2[j][e], seq[kFirst + u + j][e], g[e]);
         at += p.out_stride;
-        store_h<VEC, H16>(p.out, at, p.h_type, g);
+        store_as<VEC, H>(p.out, at, g);
       }
-      if (p.mu != nullptr) {
+      if constexpr (MU) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) prev[e] -= h[e];
 #pragma unroll
         for (int k = 0; k < kBlends; ++k) {
           float m[VEC];
 #pragma unroll
-          for (int e = 0; e < VEC; ++e) m[e] = fmaf(prev[e] - h[e], mu[k][e], h[e]);
+          for (int e = 0; e < VEC; ++e) m[e] = fmaf(prev[e], mu[k][e], h[e]);
           at += p.out_stride;
-          store_h<VEC, H16>(p.out, at, p.h_type, m);
+          store_as<VEC, H>(p.out, at, m);
         }
 #pragma unroll
         for (int e = 0; e < VEC; ++e) prev[e] = h[e];
       }
     }
+#pragma unroll
+    for (int j = 0; j < HIST; ++j)
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) seq[j][e] = seq[j + 4][e];
   }
   if (i0 == 0)                              // what the next step of this sequence looks back at
     for (int i = max(0, n - taps); i < n; ++i) {
@@ -498,13 +537,12 @@ int launch_rows(const ShiftParams& p, cudaStream_t s) {
   return static_cast<int>(fi::launch_kernel(kern, g, dim3(threads), 0, s, 0, p));
 }
 
-template <int KT>
-int launch_conv(const ShiftParams& p, int tiles, bool vec4, cudaStream_t s) {
-  const int per = 128 * (vec4 ? 4 : 1);
-  const dim3 g(tiles, (p.W + per - 1) / per);
-  const bool h16 = p.h_type != kFp32;
-  auto kern = vec4 ? (h16 ? shift_conv_kernel<KT, 4, true> : shift_conv_kernel<KT, 4, false>)
-                   : (h16 ? shift_conv_kernel<KT, 1, true> : shift_conv_kernel<KT, 1, false>);
+template <int KT, int VEC>
+int launch_conv(const ShiftParams& p, int tiles, cudaStream_t s) {
+  const dim3 g(tiles, (p.W + 128 * VEC - 1) / (128 * VEC));
+  auto kern = p.h_type == kBf16   ? (p.mu != nullptr ? shift_conv_kernel<KT, VEC, kBf16, true> : shift_conv_kernel<KT, VEC, kBf16, false>)
+              : p.h_type == kFp16 ? (p.mu != nullptr ? shift_conv_kernel<KT, VEC, kFp16, true> : shift_conv_kernel<KT, VEC, kFp16, false>)
+                                  : (p.mu != nullptr ? shift_conv_kernel<KT, VEC, kFp32, true> : shift_conv_kernel<KT, VEC, kFp32, false>);
   return static_cast<int>(fi::launch_kernel(kern, g, dim3(128), 0, s, 0, p));
 }
 
@@ -587,7 +625,7 @@ extern "C" int fi_shift_conv(const float* x, const float* inv, const float* a1, 
   const bool vec4 = W % 4 == 0 && (ldo | out_stride) % 4 == 0 && aligned(x) && aligned(a1) && aligned(a2) && aligned(mu) &&
                     aligned(ring) && aligned(out);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  if (taps <= 4) return launch_conv<4>(p, n_tiles, vec4, s);
-  if (taps <= 8) return launch_conv<8>(p, n_tiles, vec4, s);
-  return launch_conv<16>(p, n_tiles, vec4, s);
+  if (taps <= 4) return vec4 ? launch_conv<4, 4>(p, n_tiles, s) : launch_conv<4, 1>(p, n_tiles, s);
+  if (taps <= 8) return vec4 ? launch_conv<8, 4>(p, n_tiles, s) : launch_conv<8, 1>(p, n_tiles, s);
+  return launch_conv<16, 1>(p, n_tiles, s);
 }

@@ -386,7 +386,7 @@ def test_weights_reach_from_nothing_to_one():
     got = ops.paged_attention_prefill(q.view(n, -1).cuda(), pages.k, pages.v, pages.table.cuda(), i32("cuda", n), i32("cuda", 0, n), n, 1, 1, 64, 1.0,
                                       sigmoid=sig)[-1, :9].float().cpu()
     want = torch.sigmoid(score.bfloat16().float() - 1.0)
-    assert float(((got - want).abs() / want.clamp(min=1e-12)).max()) < 1e-2
+    assert float(((got - want).abs() / want.clamp(min=1e-7)).max()) < 1e-2
 
 
 def test_sigmoid_weights_go_with_nothing_else():
