@@ -53,27 +53,29 @@ struct QkParams {
   const float* v_cs;        // [max_pos, vdim] or null
 };
 
+constexpr int kThreads = 128;
+
 // VEC: every head, row and table starts on 16-byte groups.  A thread then keeps its place inside a head (and the angles of its
 // channels) while it walks over heads.
 template <typename T, bool VEC>
-__global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
+__global__ void __launch_bounds__(kThreads) qk_prepare_kernel(const QkParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
   constexpr int V = 16 / sizeof(T);
-  __shared__ float red[2][8];
+  __shared__ float red[2][kThreads / 32];
   const int t = blockIdx.x, tid = threadIdx.x;
   const T* row = reinterpret_cast<const T*>(p.proj) + t * p.ld;
   const int nq = p.H * p.dim, nk = p.G * p.dim;
   const int per = VEC ? p.hd / V : p.hd;                   // groups (or channels) of a padded head
-  const int step = VEC ? (per <= 256 ? 256 / per : 0) : 0; // heads that the block handles at a time
-  const int h0 = VEC ? tid / per : 0, c0 = VEC ? (tid % per) * V : 0;
+  const int step = VEC ? kThreads / per : 0;               // heads that the block handles at a time
+  const int h0 = VEC ? tid / per : 0, c0 = VEC ? (tid - h0 * per) * V : 0;
   const bool mine = h0 < step && c0 < p.dim;
   const int pos = min(max(p.positions[t], 0), p.max_pos - 1), half = p.dims / 2, slot = p.slot_mapping[t];
   const float* cs = p.cos_sin + static_cast<long>(pos) * p.dims;
   float sq = 0.f, sk = 0.f;
   if constexpr (VEC) {
     if (mine) {
-#pragma unroll 2
+#pragma unroll 4
       for (int h = h0; h < p.H + p.G; h += step) {
         alignas(16) T x[V];
         *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(row + h * p.dim + c0);
@@ -84,7 +86,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
       }
     }
   } else {
-    for (int i = tid; i < nq + nk; i += 256) {
+    for (int i = tid; i < nq + nk; i += kThreads) {
       const float f = to_f(row[i]);
       if (i < nq) sq = fmaf(f, f, sq); else sk = fmaf(f, f, sk);
     }
@@ -97,10 +99,11 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
   __syncthreads();
   sq = sk = 0.f;
 #pragma unroll
-  for (int w = 0; w < 8; ++w) { sq += red[0][w]; sk += red[1][w]; }
+  for (int w = 0; w < kThreads / 32; ++w) { sq += red[0][w]; sk += red[1][w]; }
   const float iq = 1.f / sqrtf(sq / static_cast<float>(nq) + p.eps), ik = 1.f / sqrtf(sk / static_cast<float>(nk) + p.eps);
   const int heads = slot >= 0 ? p.H + p.G : p.H;
-  const long blk = slot >= 0 ? slot / p.block_size : 0, off = slot >= 0 ? slot % p.block_size : 0;
+  const int blk_i = slot >= 0 ? slot / p.block_size : 0;
+  const long blk = blk_i, off = slot >= 0 ? slot - blk_i * p.block_size : 0;
   T* const q_out = reinterpret_cast<T*>(p.q_out) + static_cast<long>(t) * p.H * p.hd;
   if constexpr (VEC) {
     const bool turns = mine && c0 < p.dims, first = c0 < half;
@@ -116,7 +119,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
         for (int e = 0; e < V; ++e) ss[e] = -ss[e];
     }
     if (h0 < step) {
-#pragma unroll 2
+#pragma unroll 4
       for (int h = h0; h < heads; h += step) {
         const bool is_k = h >= p.H;
         const int g = h - p.H;
@@ -152,7 +155,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
       }
     }
   } else {
-    for (int i = tid; i < heads * per; i += 256) {
+    for (int i = tid; i < heads * per; i += kThreads) {
       const int h = i / per, c = i % per;
       const bool is_k = h >= p.H;
       const T* src = row + h * p.dim;
@@ -184,7 +187,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
   T* v0 = reinterpret_cast<T*>(p.v_cache);
   if constexpr (VEC) {
     const int vper = p.vp / V;
-    for (int i = tid; i < p.G * vper; i += 256) {
+    for (int i = tid; i < p.G * vper; i += kThreads) {
       const int g = i / vper, c = (i % vper) * V;
       alignas(16) T x[V];
       *reinterpret_cast<uint4*>(x) = make_uint4(0, 0, 0, 0);
@@ -210,7 +213,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
       *reinterpret_cast<uint4*>(v0 + ((blk * p.G + g) * p.block_size + off) * p.vp + c) = *reinterpret_cast<const uint4*>(x);
     }
   } else {
-    for (int i = tid; i < p.G * p.vp; i += 256) {
+    for (int i = tid; i < p.G * p.vp; i += kThreads) {
       const int g = i / p.vp, c = i % p.vp;
       float a = 0.f;
       if (c < p.vdim) {
@@ -228,7 +231,7 @@ __global__ void __launch_bounds__(256) qk_prepare_kernel(const QkParams p) {
 
 template <typename T>
 int launch(const QkParams& p, bool vec, int tokens, cudaStream_t s) {
-  return static_cast<int>(fi::launch_kernel(vec ? qk_prepare_kernel<T, true> : qk_prepare_kernel<T, false>, dim3(tokens), dim3(256), 0, s, 0, p));
+  return static_cast<int>(fi::launch_kernel(vec ? qk_prepare_kernel<T, true> : qk_prepare_kernel<T, false>, dim3(tokens), dim3(kThreads), 0, s, 0, p));
 }
 
 }  // namespace
@@ -253,7 +256,7 @@ extern "C" int fi_qk_prepare(const void* proj, long ld, const float* wq, const f
   const uintptr_t at = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(wq) |
                        reinterpret_cast<uintptr_t>(wk) | reinterpret_cast<uintptr_t>(cos_sin) | reinterpret_cast<uintptr_t>(v_cs) |
                        reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
-  const bool vec = dim % v == 0 && hd / v <= 256 && hd % v == 0 && (dims / 2) % v == 0 && ld % v == 0 && (at & 15) == 0 &&
+  const bool vec = dim % v == 0 && hd / v <= kThreads && hd % v == 0 && (dims / 2) % v == 0 && ld % v == 0 && (at & 15) == 0 &&
           (v_off == 0 || (v_off % v == 0 && vdim % v == 0 && vp % v == 0));
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
   if (dtype == 0) return launch<__nv_bfloat16>(p, vec, T, s);

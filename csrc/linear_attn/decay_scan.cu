@@ -550,26 +550,30 @@ __global__ void __launch_bounds__(128, KT > 4 ? 1 : 8) conv_silu_kernel(const Co
   float a[KT][VEC], seq[KT + 3][VEC], bias[VEC];             // seq: the KT - 1 inputs before the present four, then those
 #pragma unroll
   for (int j = 0; j < KT; ++j) {
-    const int tap = j - (KT - taps), i = i0 - KT + 1 + j;
+    const int tap = j - (KT - taps);
+    load_as<VEC, kFp32>(p.w, static_cast<long>(max(tap, 0)) * p.C + c, a[j]);
+    if (tap < 0)
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) a[j][e] = seq[j][e] = 0.f;
-    if (tap >= 0) {
-      load_as<VEC, kFp32>(p.w, static_cast<long>(tap) * p.C + c, a[j]);
-      if (j + 1 < KT) {
-        if (i >= 0) load_as<VEC, IN>(p.x, x0 + i * p.ld, seq[j]);
-        else if (pos0 + i >= 0) load_as<VEC, kFp32>(ring, static_cast<long>((pos0 + i) % taps) * p.C, seq[j]);
-      }
+      for (int e = 0; e < VEC; ++e) a[j][e] = 0.f;
+  }
+  // loads take no branches, so that they are in flight together
+  if (i0 > 0) {                            // a tile holds at least taps tokens
+#pragma unroll
+    for (int j = 0; j + 1 < KT; ++j) load_as<VEC, IN>(p.x, x0 + max(i0 - KT + 1 + j, 0) * p.ld, seq[j]);
+  } else {
+#pragma unroll
+    for (int j = 0; j + 1 < KT; ++j) {
+      const int i = j - KT + 1;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) seq[j][e] = 0.f;
+      if (-i < taps && pos0 + i >= 0) load_as<VEC, kFp32>(ring, static_cast<long>((pos0 + i) % taps) * p.C, seq[j]);
     }
   }
   load_as<VEC, kFp32>(p.bias, c, bias);
   const int i_end = min(n, i0 + p.tile);
   for (int i = i0; i < i_end; i += 4) {
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) seq[KT - 1 + u][e] = 0.f;
-      if (i + u < i_end) load_as<VEC, IN>(p.x, x0 + (i + u) * p.ld, seq[KT - 1 + u]);
-    }
+    for (int u = 0; u < 4; ++u) load_as<VEC, IN>(p.x, x0 + min(i + u, i_end - 1) * p.ld, seq[KT - 1 + u]);
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       if (i + u >= i_end) break;

@@ -436,26 +436,29 @@ __global__ void __launch_bounds__(128, KT > 4 ? 1 : MU ? 4 : 6) shift_conv_kerne
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v[e] *= inv;
   };
+  const float* second = p.a2 != nullptr ? p.a2 : p.a1;
   constexpr int HIST = MU ? KT : KT - 1;   // tokens before the present four; the blends also need the convolution one token back
   float a1[KT][VEC], a2[KT][VEC], mu[MU ? kBlends : 1][VEC], seq[HIST + 4][VEC], prev[VEC];
 #pragma unroll
   for (int j = 0; j < KT; ++j) {
     const int tap = j - (KT - taps);
+    load_f<VEC>(p.a1, static_cast<long>(max(tap, 0)) * W + c, a1[j]);
+    load_f<VEC>(second, static_cast<long>(max(tap, 0)) * W + c, a2[j]);
+    if (tap < 0)
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) a1[j][e] = a2[j][e] = 0.f;
-    if (tap >= 0) {
-      load_f<VEC>(p.a1, static_cast<long>(tap) * W + c, a1[j]);
-      if (p.a2 != nullptr) load_f<VEC>(p.a2, static_cast<long>(tap) * W + c, a2[j]);
-    }
+      for (int e = 0; e < VEC; ++e) a1[j][e] = a2[j][e] = 0.f;
   }
+  // loads take no branches, so that they are in flight together
+  if (i0 > 0) {                            // a tile holds at least taps tokens
 #pragma unroll
-  for (int j = 0; j < HIST; ++j) {
-    const int i = i0 - HIST + j;
+    for (int j = 0; j < HIST; ++j) unit(max(i0 - HIST + j, 0), seq[j]);
+  } else {
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) seq[j][e] = 0.f;
-    if (HIST - j <= taps) {                // the ring holds the last taps + 1 tokens
-      if (i >= 0) unit(i, seq[j]);
-      else if (pos0 + i >= 0) load_f<VEC>(ring, static_cast<long>((pos0 + i) % R) * W, seq[j]);
+    for (int j = 0; j < HIST; ++j) {
+      const int i = j - HIST;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) seq[j][e] = 0.f;
+      if (-i <= taps && pos0 + i >= 0) load_f<VEC>(ring, static_cast<long>((pos0 + i) % R) * W, seq[j]);
     }
   }
 #pragma unroll
@@ -471,11 +474,7 @@ __global__ void __launch_bounds__(128, KT > 4 ? 1 : MU ? 4 : 6) shift_conv_kerne
   const int i_end = min(n, i0 + p.tile);
   for (int i = i0; i < i_end; i += 4) {
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) seq[HIST + u][e] = 0.f;
-      if (i + u < i_end) unit(i + u, seq[HIST + u]);
-    }
+    for (int u = 0; u < 4; ++u) unit(min(i + u, i_end - 1), seq[HIST + u]);
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       if (i + u >= i_end) break;
