@@ -196,12 +196,12 @@ def kernel_rows(width: int, iters: int = 10, only: str = "") -> list[dict]:
     nb = B * ctx // 16 + 1
     kc, vc = rnd(nb, G, 16, dim, std=0.5), rnd(nb, G, 16, vdim, std=0.5)
     table = i32([[1 + s * (ctx // 16) + j for j in range(ctx // 16)] for s in range(B)])
-    qd, ln = rnd(B, H * dim), i32([ctx] * B)
     seen = min(chunk, ctx)
+    qd, ln, short_ln = rnd(B, H * dim), i32([ctx] * B), i32([seen] * B)
     case(f"sigmoid attention, decode batch {B}, {seen} keys",
          lambda: ops.paged_attention_decode(qd, kc, vc, table, ln, H, G, dim, 0.1, max_kv_len=ctx, v_dim=vdim, sigmoid=sig), B * seen * G * dim * 4,
          4.0 * B * seen * H * dim,
-         likes=[("attention", lambda: ops.paged_attention_decode(qd, kc, vc, table, i32([seen] * B), H, G, dim, 0.1, max_kv_len=seen),
+         likes=[("attention", lambda: ops.paged_attention_decode(qd, kc, vc, table, short_ln, H, G, dim, 0.1, max_kv_len=seen),
                  B * seen * G * dim * 4, 4.0 * B * seen * H * dim, tensor)])
     projd, posd, slotd = rnd(B, (H + 2 * G) * dim), i32([ctx - 1] * B), i32([16 + i * ctx for i in range(B)])
     case("queries, keys, values, decode", lambda: qk_attn.prepare(projd, wq, wk, 1e-6, posd, cs, slotd, kc, vc, H, G, dim, vdim, vcs),
@@ -222,14 +222,12 @@ def kernel_rows(width: int, iters: int = 10, only: str = "") -> list[dict]:
     tab = torch.rand(32000, E, generator=g, device="cuda").topk(top, -1).indices.to(torch.int32)
     for n, tag in ((T, f"{T} tokens"), (B, f"decode batch {B}")):
         x, z, ids = rnd(n, W), rnd(n, E, dtype=f32), torch.randint(0, 32000, (n,), device="cuda")
-        e, a = moe.lookup(tab, ids, 1.0 / top)
-        used = int(e.unique().numel())
+        e = moe.Assigned(tab, ids)
+        used = int(e.ids().unique().numel())
         nb, fl = used * 3 * eff * W * 2 + n * W * 2 + n * top * W * 2, 6.0 * n * top * eff * W
         re, ra = moe.route(z, top)
-        case(f"assigned experts, {tag} (sort .. down product)", lambda: moe.expert_rows(x, w1, w2, e, a), nb, fl,
-             likes=[("routed experts", lambda: moe.expert_rows(x, w1, w2, re, ra), nb, fl, tensor)])
-        case(f"assignment of experts, {tag}", lambda: moe.lookup(tab, ids, 1.0 / top), n * 8 + n * top * 12,
-             likes=[("softmax choice of experts", lambda: moe.route(z, top), n * E * 4 + n * top * 8, 0, tensor)])
+        case(f"assigned experts, {tag} (assignment, sort .. down product)", lambda: moe.expert_rows(x, w1, w2, e, 1.0 / top), nb, fl,
+             likes=[("routed experts (sort .. down product)", lambda: moe.expert_rows(x, w1, w2, re, ra), nb, fl, tensor)])
     return rows
 
 

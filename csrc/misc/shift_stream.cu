@@ -50,7 +50,8 @@ struct ShiftParams {
   const void* f;             // [T, ldf] or null
   const void* routed;        // expert rows of pitch ldr, or null
   const int* slot_of;        // [T, top]; null: row = token * top + choice
-  const float* route_w;      // [T, top]
+  const float* route_w;      // [T, top]; null: route_c for every choice
+  float route_c;
   float* x_out;              // [T, W] or null
   long ldy, ldy2, ldf, ldr;
   int top;
@@ -258,7 +259,7 @@ __global__ void __launch_bounds__(block_threads(TPR)) shift_rows_kernel(const Sh
       for (int k = 0; k < p.top; ++k) {
         const long at = t * p.top + k;
         const long s = p.slot_of != nullptr ? p.slot_of[at] : at;
-        const float w = s >= 0 ? p.route_w[at] : 0.f;
+        const float w = s < 0 ? 0.f : p.route_w != nullptr ? p.route_w[at] : p.route_c;
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
           const int c = (i * TPR + tid) * VEC;
@@ -581,7 +582,7 @@ int dispatch_rows(const ShiftParams& p, cudaStream_t s) {
 extern "C" int fi_shift_rows(int src_mode, int out_kind, const long long* ids, const void* table, int vocab, const void* pairs,
                              int buckets, long mul_prev, long mul_cur, int* last_token, const float* x, const void* y,
                              long ldy, const void* y2, long ldy2, const float* w_y, const float* w_y2, const void* f, long ldf,
-                             const void* routed, long ldr, const int* slot_of, const float* route_w, int top, float* x_out,
+                             const void* routed, long ldr, const int* slot_of, const float* route_w, float route_c, int top, float* x_out,
                              float* inv, const float* w_pre, const long long* sel, const float* a1, const float* a2,
                              const float* mu, int taps, float* ring, void* out, long ldo, long out_stride, const int* slots,
                              const int* seq_lens, const int* cu_q, int B, int num_slots, int rows, int W, float eps, int h_type,
@@ -593,7 +594,7 @@ extern "C" int fi_shift_rows(int src_mode, int out_kind, const long long* ids, c
     return -10;
   if (src_mode != kStart && (x == nullptr || y == nullptr)) return -10;
   if (src_mode == kPair && (y2 == nullptr || w_y == nullptr || w_y2 == nullptr)) return -10;
-  if (routed != nullptr && (route_w == nullptr || top <= 0)) return -10;
+  if (routed != nullptr && top <= 0) return -10;
   if (out_kind == kInv && inv == nullptr) return -10;
   if (out_kind == kNorm && (w_pre == nullptr || out == nullptr)) return -10;
   if (out_kind == kToken && (a1 == nullptr || ring == nullptr || out == nullptr || slots == nullptr || seq_lens == nullptr || taps <= 0))
@@ -603,7 +604,7 @@ extern "C" int fi_shift_rows(int src_mode, int out_kind, const long long* ids, c
   p.mode = src_mode; p.out_kind = out_kind; p.h_type = h_type; p.ids = ids; p.table = table; p.vocab = vocab; p.pairs = pairs;
   p.buckets = buckets; p.mul_prev = mul_prev; p.mul_cur = mul_cur; p.last_token = last_token; p.x = x; p.y = y; p.ldy = ldy;
   p.y2 = y2; p.ldy2 = ldy2; p.w_y = w_y; p.w_y2 = w_y2; p.f = f; p.ldf = ldf; p.routed = routed; p.ldr = ldr;
-  p.slot_of = slot_of; p.route_w = route_w; p.top = top; p.x_out = x_out; p.inv = inv; p.w_pre = w_pre; p.sel = sel; p.a1 = a1;
+  p.slot_of = slot_of; p.route_w = route_w; p.route_c = route_c; p.top = top; p.x_out = x_out; p.inv = inv; p.w_pre = w_pre; p.sel = sel; p.a1 = a1;
   p.a2 = a2; p.mu = mu; p.taps = taps; p.ring = ring; p.out = out; p.ldo = ldo; p.out_stride = out_stride; p.slots = slots;
   p.seq_lens = seq_lens; p.cu_q = cu_q; p.B = B; p.num_slots = num_slots; p.rows = rows; p.W = W; p.eps = eps;
   return dispatch_rows(p, reinterpret_cast<cudaStream_t>(stream));

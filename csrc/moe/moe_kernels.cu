@@ -193,7 +193,21 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
 }
 
 // One CTA.  Routes to experts outside [e_lo, e_hi) are dropped (slot_of = -1).
-__global__ void moe_align_kernel(const int* __restrict__ topk_ids, int n_routes, int e_lo, int e_hi,
+// Expert of route i: topk_ids[i], or (assigned) row ids[i / top] of a table [vocab, top].
+struct RouteIds {
+  const int* topk_ids;
+  const int* table;
+  const long long* ids;
+  int vocab, top;
+  __device__ __forceinline__ int operator[](int i) const {
+    if (table == nullptr) return topk_ids[i];
+    const int t = i / top;
+    const long long id = ids[t];
+    return table[(id < 0 || id >= vocab ? 0 : id) * top + i - t * top];      // padded rows of a decode bucket carry stale ids
+  }
+};
+
+__global__ void moe_align_kernel(const RouteIds routes, int n_routes, int e_lo, int e_hi,
                                  int bn, int* __restrict__ sorted_route, int* __restrict__ slot_of,
                                  int* __restrict__ expert_offsets, int* __restrict__ tile_expert,
                                  int* __restrict__ tile_row0, int* __restrict__ tile_rows,
@@ -208,7 +222,7 @@ __global__ void moe_align_kernel(const int* __restrict__ topk_ids, int n_routes,
   for (int i = threadIdx.x; i < EL; i += blockDim.x) { counts[i] = 0; cursor[i] = 0; }
   __syncthreads();
   for (int i = threadIdx.x; i < n_routes; i += blockDim.x) {
-    const int e = topk_ids[i];
+    const int e = routes[i];
     if (e >= e_lo && e < e_hi) atomicAdd(&counts[e - e_lo], 1);
   }
   __syncthreads();
@@ -243,7 +257,7 @@ __global__ void moe_align_kernel(const int* __restrict__ topk_ids, int n_routes,
   __syncthreads();
   for (int i = threadIdx.x; i <= EL; i += blockDim.x) expert_offsets[i] = offs[i];
   for (int i = threadIdx.x; i < n_routes; i += blockDim.x) {
-    const int e = topk_ids[i];
+    const int e = routes[i];
     if (e >= e_lo && e < e_hi) {
       const int slot = offs[e - e_lo] + atomicAdd(&cursor[e - e_lo], 1);
       sorted_route[slot] = i;
@@ -252,19 +266,6 @@ __global__ void moe_align_kernel(const int* __restrict__ topk_ids, int n_routes,
       slot_of[i] = -1;
     }
   }
-}
-
-// Experts that a table assigns to token ids, all with the same weight.
-__global__ void __launch_bounds__(256) moe_lookup_kernel(const int* __restrict__ table, const long long* __restrict__ ids, int vocab,
-                                                         int n, int top, float weight, int* __restrict__ topk_ids,
-                                                         float* __restrict__ topk_w) {
-  fi::pdl_launch_dependents();
-  fi::pdl_wait();
-  const int i = blockIdx.x * 256 + threadIdx.x;
-  if (i >= n) return;
-  const long long id = ids[i / top];
-  topk_ids[i] = table[(id < 0 || id >= vocab ? 0 : id) * top + i % top];     // padded rows of a decode bucket carry stale ids
-  topk_w[i] = weight;
 }
 
 // Tile table of E stacked matrices of T rows each.
@@ -571,15 +572,6 @@ extern "C" int fi_moe_route(const float* logits, const float* bias, const float*
   return static_cast<int>(cudaGetLastError());
 }
 
-// topk_ids, topk_w [T, top] = table [vocab, top] rows of the token ids, each choice with `weight`.
-extern "C" int fi_moe_lookup(const int* table, const long long* ids, int vocab, int T, int top, float weight, int* topk_ids,
-                             float* topk_w, void* stream) {
-  if (T <= 0) return 0;
-  if (vocab <= 0 || top <= 0 || static_cast<long>(T) * top > 2147483647l) return -10;
-  return static_cast<int>(fi::launch_kernel(moe_lookup_kernel, dim3((T * top + 255) / 256), dim3(256), 0, FI_STREAM(stream), 0, table,
-                                            ids, vocab, T * top, top, weight, topk_ids, topk_w));
-}
-
 // Tile table (as of fi_moe_align) of E stacked matrices of T rows: E * ceil(T / bn) tiles.
 extern "C" int fi_stack_tiles(int E, int T, int bn, int* tile_expert, int* tile_row0, int* tile_rows, int* n_tiles, void* stream) {
   if (E <= 0 || T <= 0) return 0;
@@ -589,17 +581,32 @@ extern "C" int fi_stack_tiles(int E, int T, int bn, int* tile_expert, int* tile_
                                             per, tile_expert, tile_row0, tile_rows, n_tiles));
 }
 
-extern "C" int fi_moe_align(const int* topk_ids, int n_routes, int e_lo, int e_hi, int bn,
-                            int* sorted_route, int* slot_of, int* expert_offsets, int* tile_expert,
-                            int* tile_row0, int* tile_rows, int* n_tiles, void* stream) {
+static int launch_align(const RouteIds& routes, int n_routes, int e_lo, int e_hi, int bn, int* sorted_route, int* slot_of,
+                        int* expert_offsets, int* tile_expert, int* tile_row0, int* tile_rows, int* n_tiles, void* stream) {
   if (n_routes <= 0) return 0;
   const int EL = e_hi - e_lo;
   if (EL <= 0 || EL > 4096) return -10;
   const size_t smem = (3 * EL + 1) * sizeof(int);
-  fi::launch_kernel(moe_align_kernel, dim3(1), dim3(1024), smem, FI_STREAM(stream), 0, topk_ids, n_routes,
+  fi::launch_kernel(moe_align_kernel, dim3(1), dim3(1024), smem, FI_STREAM(stream), 0, routes, n_routes,
                     e_lo, e_hi, bn, sorted_route, slot_of, expert_offsets, tile_expert, tile_row0, tile_rows,
                     n_tiles);
   return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int fi_moe_align(const int* topk_ids, int n_routes, int e_lo, int e_hi, int bn,
+                            int* sorted_route, int* slot_of, int* expert_offsets, int* tile_expert,
+                            int* tile_row0, int* tile_rows, int* n_tiles, void* stream) {
+  return launch_align({topk_ids, nullptr, nullptr, 0, 1}, n_routes, e_lo, e_hi, bn, sorted_route, slot_of, expert_offsets, tile_expert,
+                      tile_row0, tile_rows, n_tiles, stream);
+}
+
+// The same for experts assigned to token ids: route i is choice i % top of token ids[i / top] in table [vocab, top].
+extern "C" int fi_moe_align_assigned(const int* table, const long long* ids, int vocab, int top, int n_routes, int e_hi, int bn,
+                                     int* sorted_route, int* slot_of, int* expert_offsets, int* tile_expert, int* tile_row0,
+                                     int* tile_rows, int* n_tiles, void* stream) {
+  if (table == nullptr || ids == nullptr || vocab <= 0 || top <= 0) return -10;
+  return launch_align({nullptr, table, ids, vocab, top}, n_routes, 0, e_hi, bn, sorted_route, slot_of, expert_offsets, tile_expert,
+                      tile_row0, tile_rows, n_tiles, stream);
 }
 
 extern "C" int fi_moe_gather(const void* x, const int* sorted_route, const int* expert_offsets, int EL,

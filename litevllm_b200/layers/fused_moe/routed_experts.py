@@ -75,5 +75,4 @@ class AssignedExperts(nn.Module):
 
     def forward(self, x, token_ids) -> moe.RoutedRows:
         """x [T, hidden], token_ids int64 [T]."""
-        ids, w = moe.lookup(self.table, token_ids, 1.0 / self.top)
-        return moe.expert_rows(x, self.w_gate_up, self.w_down, ids, w, self.act)
+        return moe.expert_rows(x, self.w_gate_up, self.w_down, moe.Assigned(self.table.data, token_ids), 1.0 / self.top, self.act)

@@ -67,40 +67,40 @@ def route(logits: torch.Tensor, top_k: int, mode: str = "softmax", bias: torch.T
     return ids, w
 
 
-def lookup(table: torch.Tensor, token_ids: torch.Tensor, weight: float):
-    """Experts that a table int32 [vocab, k] assigns to token ids (int64 [T]), each with ``weight``: (ids int32 [T, k],
-    weights float32 [T, k])."""
-    T, (V, K) = token_ids.shape[0], table.shape
-    if not table.is_cuda:
-        return table.index_select(0, token_ids), torch.full((T, K), float(weight))
-    ids = torch.empty(T, K, dtype=torch.int32, device=table.device)
-    w = torch.empty(T, K, dtype=torch.float32, device=table.device)
-    assert table.dtype == torch.int32 and table.is_contiguous() and token_ids.dtype == torch.int64 and token_ids.is_contiguous()
-    rc = _lib.kernels().fi_moe_lookup(_p(table), _p(token_ids), V, T, K, float(weight), _p(ids), _p(w), _stream())
-    _lib.check(rc, "fi_moe_lookup")
-    _count()
-    return ids, w
+@dataclass(frozen=True)
+class Assigned:
+    """Choices without a router: token t takes the experts ``table[token_ids[t]]`` (table int32 [vocab, K], ids int64 [T])."""
+    table: torch.Tensor
+    token_ids: torch.Tensor
+
+    @property
+    def shape(self) -> tuple[int, int]:
+        return self.token_ids.shape[0], self.table.shape[1]
+
+    def ids(self) -> torch.Tensor:
+        return self.table.index_select(0, self.token_ids)
 
 
 @dataclass
 class RoutedRows:
     """Outputs of the chosen experts before their weighted sum: choice k of token t is row ``slot_of[t, k]`` of ``rows``
-    (row t * K + k without a map), its weight ``weights[t, k]``.  A choice whose slot is negative has no row: it adds nothing,
+    (row t * K + k without a map), its weight ``weights[t, k]`` (a number: of every choice).  A choice whose slot is negative has no row: it adds nothing,
     or with ``pass_through`` the experts' input itself."""
     rows: torch.Tensor               # [T * K, H]
-    weights: torch.Tensor            # fp32 [T, K]
+    weights: torch.Tensor | float    # fp32 [T, K]
     slot_of: torch.Tensor | None = None
     pass_through: bool = False
 
     def combined(self, x: torch.Tensor | None = None) -> torch.Tensor:
         """fp32 [T, H]; PyTorch form (the kernels fold the sum into the residual add).  ``x``: the experts' input."""
-        T, K = self.weights.shape
+        w = self.weights if isinstance(self.weights, torch.Tensor) else torch.full(self.slot_of.shape, self.weights)
+        T, K = w.shape
         if self.slot_of is None:
-            return (self.rows.float().view(T, K, -1) * self.weights[..., None]).sum(1)
+            return (self.rows.float().view(T, K, -1) * w[..., None]).sum(1)
         none = (self.slot_of < 0)[..., None]
         r = self.rows.index_select(0, self.slot_of.clamp(min=0).reshape(-1).long()).float().view(T, K, -1)
         r = torch.where(none, x.float()[:, None] if self.pass_through else torch.zeros_like(r), r)
-        return (r * self.weights[..., None]).sum(1)
+        return (r * w[..., None]).sum(1)
 
 
 _stack_tables: dict[tuple, torch.Tensor] = {}
@@ -160,16 +160,22 @@ def _tile_table(ids, n: int, E: int, bn: int, dev, scratch_name: str):
     for size in (n, n, E + 1, bound, bound, bound, 1):
         out.append(ints[o:o + size])
         o += size
-    rc = _lib.kernels().fi_moe_align(_p(ids), n, 0, E, bn, *[_p(t) for t in out], _stream())
+    if isinstance(ids, Assigned):
+        assert ids.table.dtype == torch.int32 and ids.table.is_contiguous() and ids.token_ids.dtype == torch.int64
+        assert ids.token_ids.is_contiguous()
+        rc = _lib.kernels().fi_moe_align_assigned(_p(ids.table), _p(ids.token_ids), *ids.table.shape, n, E, bn, *[_p(t) for t in out],
+                                                  _stream())
+    else:
+        rc = _lib.kernels().fi_moe_align(_p(ids), n, 0, E, bn, *[_p(t) for t in out], _stream())
     _lib.check(rc, "fi_moe_align")
     _count()
     return (*out, bound)
 
 
-def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
-                weights: torch.Tensor, act: str = "silu", act_limit: float = 0.0, pass_through: bool = False) -> RoutedRows:
+def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor | Assigned,
+                weights: torch.Tensor | float, act: str = "silu", act_limit: float = 0.0, pass_through: bool = False) -> RoutedRows:
     """Unquantised experts: x [T, H], ``w_gate_up`` [E, 2 I, H] (gate | up), ``w_down`` [E, H, I], ids / weights of
-    :func:`route`; ids from E on have no row (``pass_through``: they stand for x itself).  ``act`` and ``act_limit`` as in
+    :func:`route` (or :class:`Assigned` choices of one weight); ids from E on have no row (``pass_through``: they stand for x itself).  ``act`` and ``act_limit`` as in
     :func:`ops.gated_linear`.  No host synchronisation.  16-bit weights whose rows are whole 16-byte groups run grouped tcgen05
     products (persistent tiles when an expert sees many rows), everything else the general 32-bit kernel."""
     T, H = x.shape
@@ -177,7 +183,7 @@ def expert_rows(x: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, 
     inter, K = two_i // 2, ids.shape[1]
     if not x.is_cuda:
         rows = torch.zeros(T * K, H, dtype=x.dtype)
-        flat = ids.reshape(-1).long()
+        flat = (ids.ids() if isinstance(ids, Assigned) else ids).reshape(-1).long()
         for e in flat[flat < E].unique().tolist():
             at = torch.nonzero(flat == e).view(-1)
             h = x[at // K].float() @ w_gate_up[e].float().t()

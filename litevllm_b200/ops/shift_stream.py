@@ -145,17 +145,21 @@ def _source_args(src, x, x_out, h_dtype):
         if _ops._BOUNDS_CHECK:
             _check_index("shift_stream.ids", src.ids, 0, src.table.shape[0], "rows of the embedding table")
         return (_p(src.ids), _p(src.table), src.table.shape[0], _p(src.pairs), src.pairs.shape[0] - 1, src.mul_prev, src.mul_cur,
-                _p(src.last_token), None, None, 0, None, 0, _p(src.weight), None, None, 0, None, 0, None, None, 0, _p(x_out))
+                _p(src.last_token), None, None, 0, None, 0, _p(src.weight), None, None, 0, None, 0, None, None, 0.0, 0, _p(x_out))
     pair, r, f = isinstance(src, Paired), src.routed, src.f
     assert x.is_contiguous() and x.dtype == torch.float32 and src.y.stride(1) == 1 and src.y.dtype == h_dtype
     assert f is None or (f.stride(1) == 1 and f.dtype == h_dtype)
     assert not pair or (src.y2.stride(1) == 1 and src.y2.dtype == h_dtype)
     if r is not None:
-        assert r.rows.dtype == h_dtype and r.rows.stride(1) == 1 and r.weights.is_contiguous() and not r.pass_through
+        assert r.rows.dtype == h_dtype and r.rows.stride(1) == 1 and not r.pass_through
+    w = r.weights if r is not None else 0.0
+    one = not isinstance(w, torch.Tensor)               # a weight for all choices
+    assert one or w.is_contiguous()
     return (None, None, 0, None, 0, 0, 0, None, _p(x), _p(src.y), src.y.stride(0), _p(src.y2) if pair else None,
             src.y2.stride(0) if pair else 0, _p(src.w) if pair else None, _p(src.w2) if pair else None, _p(f),
             f.stride(0) if f is not None else 0, _p(r.rows) if r else None, r.rows.stride(0) if r else 0,
-            _p(r.slot_of) if r else None, _p(r.weights) if r else None, r.weights.shape[1] if r else 0, _p(x_out))
+            _p(r.slot_of) if r else None, None if one else _p(w), float(w) if one else 0.0,
+            (r.slot_of if one else w).shape[1] if r else 0, _p(x_out))
 
 
 def _mode(src) -> int:

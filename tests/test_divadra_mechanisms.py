@@ -124,6 +124,9 @@ def test_two_normed_outputs_and_experts_join_the_stream(W, top, dtype, device):
         order = torch.randperm(T * top, generator=torch.Generator().manual_seed(6)).to(torch.int32).view(T, top)
         want = want + (rows.float()[order.long().view(-1)].view(T, top, W) * a[..., None]).sum(1)
         routed = moe.RoutedRows(d(rows), d(a), d(order))
+        if top == 2:                                        # one weight for all choices
+            want = want - (rows.float()[order.long().view(-1)].view(T, top, W) * (a[..., None] - 0.5)).sum(1)
+            routed = moe.RoutedRows(d(rows), 0.5, d(order))
     src = stream.Paired(d(y), d(w), d(y2), d(w2), None, routed)
     buf, tol = d(x).clone(), 3e-6 if dtype == "f32" else 6e-3
     h = stream.normed(src, buf, d(wf), None, eps, dt, keep=True)
@@ -427,6 +430,25 @@ def test_time_mixing(H, d, dtype, device):
             close(pool[slots[s]], S, 2e-5)
 
 
+@pytest.mark.parametrize("device", DEV)
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("H, d, rank", [(2, 12, 8), (3, 5, 16), (4, 64, 64), (1, 130, 24), (2, 72, 200)])
+def test_decays_of_low_rank_in_decoding(H, d, rank, dtype, device):
+    dt, n, B = DT[dtype], H * d, 7
+    r, k, v, g = rnd(4, B, n, seed=1).to(dt).to(device)
+    low, w2 = rnd(B, rank, seed=2).to(dt), rnd(n, rank, seed=3, std=rank ** -0.5).to(dt)
+    w0, u, norm, pool = rnd(n, seed=4) - 1, rnd(H, d, seed=5), rnd(n, seed=6), rnd(B, H, d, d, seed=7)
+    d_ = lambda t: t.to(device)
+    out, states = [], []
+    for z, expand in ((d_(low), d_(w2)), (d_(low.float() @ w2.float().t()), None)):
+        p = d_(pool).clone()
+        out.append(lin.time_mix(r, k, v, g, z, d_(w0), d_(u), p, make_batch(device, list(range(B)), [1] * B, [5, 0, 9, 1, 2, 3, 4], True), d_(norm),
+                                1e-3, dt, expand))
+        states.append(p)
+    close(out[0].float(), out[1].float().cpu(), 1e-5 if dtype == "f32" else 8e-3)
+    close(states[0], states[1].cpu(), 1e-5)
+
+
 SSD = [(4, 20, 12, 2, 5, 3), (3, 7, 5, 3, 1, 1), (6, 64, 64, 1, 4, 4), (2, 130, 130, 2, 2, 2), (8, 32, 128, 4, 32, 4), (2, 48, 300, 1, 3, 9)]
 
 
@@ -565,7 +587,7 @@ def test_experts_assigned_by_token(T, W, ff, E, top, V, dtype, device):
         where(w[name]) if callable(where) and not isinstance(where, torch.Tensor) else where.data.copy_(w[name])
     layer, ids, x = layer.to(device), torch.randint(0, V, (T,), generator=gen), torch.randn(T, W, generator=gen).to(dt)
     got = layer(x.to(device), ids.to(device))
-    routed = moe.RoutedRows(got.rows.cpu(), got.weights.cpu(), got.slot_of.cpu())
+    routed = moe.RoutedRows(got.rows.cpu(), got.weights, got.slot_of.cpu())
     close(routed.combined(), O.experts(x.float(), w, "", ids.tolist()), 1e-5 if dtype == "f32" else 2e-2)
 
 
