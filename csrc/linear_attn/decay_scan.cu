@@ -54,11 +54,8 @@ struct ScanParams {
   float* ring;            // [slots, taps, C]
   const float* norm_w;    // kChannel: [H * dv]
   const void* gate;       // kChannel: [B, ldg]
-  const void* low;        // kChannel: [B, ldl] the decay's low-rank half (then z is unused), or null
-  const void* w2;         // [H * d, rank] what expands it
   void* out;              // kChannel: [B, H * dv]
-  long ldq, ldk, ldv, ldz, ldg, ldl;
-  int rank;
+  long ldq, ldk, ldv, ldz, ldg;
   int vec4, H, G, d, dv, C, taps, type, out_type, num_slots;
   float eps;
 };
@@ -389,35 +386,13 @@ __global__ void __launch_bounds__(256, 3) decay_step_kernel(const ScanParams p) 
   if (ry < ry_n) fetch(ry);
   float decay = 1.f, g = 0.f;       // kScalar: decay and skip; kChannel: g is the bonus
   if constexpr (KIND == kChannel) {
-    if (p.low != nullptr) {         // z = w2 low: four lanes share a channel's row
-      float* low = so;              // [rank]; free until the partial outputs
-      for (int j = tid; j < p.rank; j += 256) low[j] = ld_any(p.low, b * p.ldl + j, p.type);
-      __syncthreads();
-      for (int c4 = 0; c4 < d; c4 += 64) {
-        const int c = c4 + (tid >> 2);
-        float z = 0.f;
-        if (c < d) {
-          const long row = (static_cast<long>(head) * d + c) * p.rank;
-          for (int j = (tid & 3) * 4; j < p.rank; j += 16) {
-            float w[4];
-            if (p.type == kFp32) expand4(load4(reinterpret_cast<const float*>(p.w2) + row + j, 4, 1), kFp32, w);
-            else expand4(load4(reinterpret_cast<const uint16_t*>(p.w2) + row + j, 4, 1), p.type, w);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) z = fmaf(w[e], low[j + e], z);
-          }
-        }
-        z += __shfl_xor_sync(0xffffffffu, z, 1);
-        z += __shfl_xor_sync(0xffffffffu, z, 2);
-        if (c < d && (tid & 3) == 0) sw[c] = decay_exp(-__expf(z + p.zb[head * d + c]));
-      }
-    }
     for (int c = tid; c < d; c += 256) {
       const long at = static_cast<long>(group) * d + c;
       const float r = ld_any(p.q, b * p.ldq + at, p.type), k = ld_any(p.k, b * p.ldk + at, p.type);
       const int hc = head * d + c;
       sq[c] = r;
       sk[c] = k;
-      if (p.low == nullptr) sw[c] = decay_exp(-__expf(p.z[b * p.ldz + hc] + p.zb[hc]));
+      sw[c] = decay_exp(-__expf(p.z[b * p.ldz + hc] + p.zb[hc]));
       g = fmaf(r * p.u[hc], k, g);
     }
     for (int c = tid; c < dv; c += 256) sv[c] = ld_any(p.v, b * p.ldv + static_cast<long>(head) * dv + c, p.type);
@@ -773,8 +748,7 @@ int dispatch_step(const ScanParams& p, int B, cudaStream_t s) {
   const bool vec4 = p.dv % 4 == 0 && (reinterpret_cast<uintptr_t>(p.pool) & 15) == 0;
   const int nx = vec4 ? p.dv / 4 : p.dv;
   if (nx > 256) return -11;
-  const int part = (256 / nx) * p.dv;
-  const int smem = (3 * p.d + p.dv + (part > p.rank ? part : p.rank)) * 4;
+  const int smem = (3 * p.d + p.dv + (256 / nx) * p.dv) * 4;
   if (smem > 48 * 1024) return -11;
   auto kern = vec4 ? decay_step_kernel<4, KIND> : decay_step_kernel<1, KIND>;
   return static_cast<int>(fi::launch_kernel(kern, dim3(p.H, B), dim3(256), smem, s, 0, p));
@@ -810,9 +784,8 @@ extern "C" int fi_decay_scan(int kind, const void* q, long ldq, const void* k, l
 
 // One token per sequence, channel decays: operands of fi_decay_scan with B rows, then per head norm(o) * norm_w [H * dv] *
 // silu(gate) (gate [B, ldg] of `type`, or null) into out [B, H * dv] of out_type.  Rows with seq_lens <= 0 are padding.
-// z null: the decays are w2 [H * d, rank] times the rows low [B, ldl] (both of `type`; rank a multiple of four).
 extern "C" int fi_decay_step(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* z, long ldz,
-                             const void* low, long ldl, const void* w2, int rank, const float* w0, const float* u, const void* gate, long ldg, const float* norm_w, float eps, float* pool,
+                             const float* w0, const float* u, const void* gate, long ldg, const float* norm_w, float eps, float* pool,
                              const int* slots, const int* seq_lens, void* out, int B, int H, int d, int dv, int num_slots, int type,
                              int out_type, void* stream) {
   if (B <= 0) return 0;
@@ -821,10 +794,6 @@ extern "C" int fi_decay_step(const void* q, long ldq, const void* k, long ldk, c
   p.q = q; p.k = k; p.v = v; p.ldq = ldq; p.ldk = ldk; p.ldv = ldv; p.z = z; p.ldz = ldz; p.zb = w0; p.u = u; p.gate = gate;
   p.ldg = ldg; p.norm_w = norm_w; p.eps = eps; p.pool = pool; p.slots = slots; p.seq_lens = seq_lens; p.out = out; p.H = H;
   p.G = H; p.d = d; p.dv = dv; p.num_slots = num_slots; p.type = type; p.out_type = out_type;
-  if (z == nullptr) {
-    if (low == nullptr || w2 == nullptr || rank <= 0 || rank % 4 != 0 || (reinterpret_cast<uintptr_t>(w2) & 15) != 0) return -10;
-    p.low = low; p.ldl = ldl; p.w2 = w2; p.rank = rank;
-  }
   return dispatch_step<kChannel>(p, B, reinterpret_cast<cudaStream_t>(stream));
 }
 

@@ -20,8 +20,6 @@ from ..ops import linear_attn, moe
 from .linear import LiteLinear
 
 BLENDS = "rkvgw"
-# up to this many decoded tokens the step kernel expands the low-rank decays itself
-_FOLD_TOKENS = 64
 
 
 def _vec(*shape: int) -> nn.Parameter:
@@ -67,7 +65,5 @@ class TimeMix(nn.Module):
     def forward(self, blends, batch, pool):
         """blends [5, T, hidden] -> [T, hidden]; pool: fp32 [slots, heads, dim, dim]."""
         r, k, v, gate = moe.stacked_linear(blends[:4], self.proj)
-        z, expand = ops.linear(blends[4], self.w1, act="tanh"), self.w2
-        if not batch.is_decode or blends.shape[1] > _FOLD_TOKENS:
-            z, expand = ops.linear(z, expand, out_dtype=torch.float32), None
-        return self.o_proj(linear_attn.time_mix(r, k, v, gate, z, self.w0, self.u, pool, batch, self.norm, self.eps, blends.dtype, expand))
+        z = ops.linear(ops.linear(blends[4], self.w1, act="tanh"), self.w2, out_dtype=torch.float32)
+        return self.o_proj(linear_attn.time_mix(r, k, v, gate, z, self.w0, self.u, pool, batch, self.norm, self.eps, blends.dtype))

@@ -397,19 +397,15 @@ def _scan(kind: int, q, k, v, z, zb, u, rate, pool, batch, G: int):
     return o
 
 
-def time_mix(r, k, v, gate, z, w0, u, pool, batch, norm_w, eps: float, out_dtype, expand=None):
+def time_mix(r, k, v, gate, z, w0, u, pool, batch, norm_w, eps: float, out_dtype):
     """Time mixing of a step: ``o_t = (S + diag(u) k_t v_t^T)^T r_t``, ``S = diag(exp(-exp(z_t + w0))) S + k_t v_t^T``, then per
     head norm, ``norm_w`` and ``silu(gate)``.
 
     r, k, v, gate [T, H * d] (any row pitch, one type), z fp32 [T, H * d], w0 [H * d], u [H, d], norm_w [H * d] fp32; pool fp32
-    [slots, H, d, d], updated in place.  A sequence whose first position is 0 starts from zero.  ``expand`` [H * d, rank] (one
-    token per sequence only): z is low-rank, [T, rank] of the type of r, and stands for ``z @ expand.T``.  Returns [T, H * d]."""
+    [slots, H, d, d], updated in place.  A sequence whose first position is 0 starts from zero.  Returns [T, H * d]."""
     slots_n, H, d, dv = pool.shape
     T = r.shape[0]
-    assert expand is None or batch.is_decode
     if not r.is_cuda:
-        if expand is not None:
-            z = z.float() @ expand.float().t()
         from .shift_stream import sequences
         o = torch.zeros(T, H * dv)
         for slot, lo, hi, pos0 in sequences(batch):
@@ -421,14 +417,12 @@ def time_mix(r, k, v, gate, z, w0, u, pool, batch, norm_w, eps: float, out_dtype
         return part_norm(o, norm_w, H, eps, out_dtype, gate)
     if not batch.is_decode:
         return part_norm(_scan(0, r, k, v, z, w0, u, None, pool, batch, H), norm_w, H, eps, out_dtype, gate)
-    assert r.dtype == k.dtype == v.dtype == gate.dtype
-    assert z.dtype == (torch.float32 if expand is None else r.dtype) and (expand is None or (expand.is_contiguous() and expand.dtype == r.dtype))
-    full, low = (z, None) if expand is None else (None, z)
+    assert r.dtype == k.dtype == v.dtype == gate.dtype and z.dtype == torch.float32
     assert r.stride(1) == k.stride(1) == v.stride(1) == gate.stride(1) == z.stride(1) == 1
     _check_pool(pool, batch)
     out = torch.empty(T, H * dv, dtype=out_dtype, device=r.device)
-    rc = _lib.kernels().fi_decay_step(_p(r), r.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(full), z.stride(0), _p(low),
-                                      z.stride(0), _p(expand), 0 if expand is None else expand.shape[1], _p(w0), _p(u), _p(gate), gate.stride(0), _p(norm_w), eps, _p(pool), _p(batch.extras["slot_ids"]),
+    rc = _lib.kernels().fi_decay_step(_p(r), r.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), z.stride(0), _p(w0), _p(u),
+                                      _p(gate), gate.stride(0), _p(norm_w), eps, _p(pool), _p(batch.extras["slot_ids"]),
                                       _p(batch.seq_lens), _p(out), T, H, d, dv, slots_n, _DT[r.dtype], _DT[out_dtype], _stream())
     _lib.check(rc, "fi_decay_step")
     _count()

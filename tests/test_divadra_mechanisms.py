@@ -430,25 +430,6 @@ def test_time_mixing(H, d, dtype, device):
             close(pool[slots[s]], S, 2e-5)
 
 
-@pytest.mark.parametrize("device", DEV)
-@pytest.mark.parametrize("dtype", ["f32", "bf16"])
-@pytest.mark.parametrize("H, d, rank", [(2, 12, 8), (3, 5, 16), (4, 64, 64), (1, 130, 24), (2, 72, 200)])
-def test_decays_of_low_rank_in_decoding(H, d, rank, dtype, device):
-    dt, n, B = DT[dtype], H * d, 7
-    r, k, v, g = rnd(4, B, n, seed=1).to(dt).to(device)
-    low, w2 = rnd(B, rank, seed=2).to(dt), rnd(n, rank, seed=3, std=rank ** -0.5).to(dt)
-    w0, u, norm, pool = rnd(n, seed=4) - 1, rnd(H, d, seed=5), rnd(n, seed=6), rnd(B, H, d, d, seed=7)
-    d_ = lambda t: t.to(device)
-    out, states = [], []
-    for z, expand in ((d_(low), d_(w2)), (d_(low.float() @ w2.float().t()), None)):
-        p = d_(pool).clone()
-        out.append(lin.time_mix(r, k, v, g, z, d_(w0), d_(u), p, make_batch(device, list(range(B)), [1] * B, [5, 0, 9, 1, 2, 3, 4], True), d_(norm),
-                                1e-3, dt, expand))
-        states.append(p)
-    close(out[0].float(), out[1].float().cpu(), 1e-5 if dtype == "f32" else 8e-3)
-    close(states[0], states[1].cpu(), 1e-5)
-
-
 SSD = [(4, 20, 12, 2, 5, 3), (3, 7, 5, 3, 1, 1), (6, 64, 64, 1, 4, 4), (2, 130, 130, 2, 2, 2), (8, 32, 128, 4, 32, 4), (2, 48, 300, 1, 3, 9)]
 
 
