@@ -13,6 +13,9 @@
 //                       outputs of four tokens are reduced together.  Operands of the next tokens are fetched as raw values
 //                       while the present ones are processed, then turned into what the recurrence reads and staged in
 //                       shared memory.  Products run as packed pairs (fma.rn.f32x2).
+//                       Few long sequences are cut into segments that run side by side: a first pass leaves every segment's end
+//                       state from a zero start and the product of its decays, decay_chain_kernel turns those into start states
+//                       (and the sequence's last state), and a second pass computes the outputs.
 //   decay_step_kernel   one token per sequence (decode): reads and writes the state once; the first form ends with the
 //                       per-head norm, weight and gate, the second starts with its convolution.
 //   conv_silu_kernel    the convolution of portions: a thread owns channels and slides along a tile of tokens
@@ -47,6 +50,10 @@ struct ScanParams {
   const int* cu_q;        // [B + 1] (scan)
   const int* seq_lens;    // [B] length after this step
   float* o;               // [T, H, dv] (scan; step of kScalar)
+  const int* seg_base;    // [B + 1] segments before each sequence, or null: sequences in one piece
+  float* seg_state;       // [segments, H, d, dv] end states from zero, then start states
+  float* seg_decay;       // [segments, H, d] products of decays (kScalar: the first of each row)
+  int seg_len, B;
   // step
   const void* xbc;        // kScalar: [B, ldq] raw x (H * dv) | B (G * d) | C (G * d)
   const float* conv;      // [taps, C]
@@ -72,8 +79,19 @@ struct ScanShape {
   static constexpr int kFloats = 2 * kTok * (kRows * D + COLS + 4) + 2 * D;
 };
 
+// The sequence (or segment) that index i of a running count belongs to.
+__device__ __forceinline__ int find_seq(const int* base, int B, int i) {
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (base[mid] <= i) lo = mid; else hi = mid - 1;
+  }
+  return lo;
+}
+
 // R rows per lane (16 R >= d), C columns per lane (a warp: 2 C columns, a block: 16 C); T: storage of q, k and v.
-template <int R, int C, int KIND, typename T>
+// OUT: outputs are computed; otherwise (first pass over segments) only states and products of decays.
+template <int R, int C, int KIND, typename T, bool OUT>
 __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParams p) {
   fi::pdl_launch_dependents();
   fi::pdl_wait();
@@ -92,16 +110,19 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
   float* c1 = c0 + D;                                        // [D] u
   const int slices = (p.dv + COLS - 1) / COLS;
   const int head = blockIdx.x / slices, slice = blockIdx.x % slices;
-  const int b = blockIdx.y;
-  const int t_begin = p.cu_q[b], n = p.cu_q[b + 1] - t_begin;
+  const bool cut = p.seg_base != nullptr;
+  const int b = cut ? find_seq(p.seg_base, p.B, blockIdx.y) : blockIdx.y;
+  const int s0 = cut ? (static_cast<int>(blockIdx.y) - p.seg_base[b]) * p.seg_len : 0;
+  const int t_begin = p.cu_q[b] + s0, n = cut ? min(p.cu_q[b + 1] - t_begin, p.seg_len) : p.cu_q[b + 1] - t_begin;
   if (n <= 0) return;
   const int slot = p.slots[b];
   if (slot < 0 || slot >= p.num_slots) return;
-  const bool fresh = p.seq_lens[b] == n;    // the portion starts at position 0
+  const bool fresh = !OUT || (!cut && p.seq_lens[b] == n);      // starts from zero
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rg = lane & 15, cg = lane >> 4;
   const int col0 = slice * COLS + (warp * 2 + cg) * C;     // first of this lane's columns
-  float* S0 = p.pool + (static_cast<long>(slot) * p.H + head) * p.d * p.dv;
+  const long piece = static_cast<long>(cut ? blockIdx.y : slot) * p.H + head;
+  float* S0 = (cut ? p.seg_state : p.pool) + piece * p.d * p.dv;
   const int group = head / (p.H / p.G);
 
   // rows of this lane: 64 i4 + 4 rg + e, pairs (e = 0, 1) and (2, 3)
@@ -133,7 +154,7 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
       const int e = (i * 256 + threadIdx.x) * 4, tok = e / D, ch = e % D;
       const int left = t0 + tok < n ? p.d - ch : 0;
       const long t = t_begin + t0 + tok;
-      rq[i] = load4(gq + t * p.ldq + ch, left, p.vec4);
+      if constexpr (OUT) rq[i] = load4(gq + t * p.ldq + ch, left, p.vec4);
       rk[i] = load4(gk + t * p.ldk + ch, left, p.vec4);
       if constexpr (KIND == kChannel) rz[i] = load4(gz + t * p.ldz + ch, left, p.vec4);
       else rdt[i] = t0 + tok < n ? gz[t * p.ldz] : 0.f;
@@ -154,7 +175,7 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
       const int e = (i * 256 + threadIdx.x) * 4, tok = e / D, ch = e % D;
       const bool live = t0 + tok < n;
       float qa[4], ka[4];
-      expand4(rq[i], p.type, qa);           // zeros beyond the last channel and the last token
+      if constexpr (OUT) expand4(rq[i], p.type, qa);          // zeros beyond the last channel and the last token
       expand4(rk[i], p.type, ka);
       const int at = (buf * kTok + tok) * D + ch;
       if constexpr (KIND == kChannel) {
@@ -163,20 +184,22 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           wa[j] = live && ch + j < p.d ? decay_exp(-__expf(za[j] + c0[ch + j])) : 1.f;
-          bonus = fmaf(qa[j] * c1[ch + j], ka[j], bonus);
+          if constexpr (OUT) bonus = fmaf(qa[j] * c1[ch + j], ka[j], bonus);
         }
         *reinterpret_cast<float4*>(sw + at) = make_float4(wa[0], wa[1], wa[2], wa[3]);
-        constexpr int kLanes = D / 4 < 32 ? D / 4 : 32;        // neighbouring lanes that hold one token
+        if constexpr (OUT) {
+          constexpr int kLanes = D / 4 < 32 ? D / 4 : 32;      // neighbouring lanes that hold one token
 #pragma unroll
-        for (int m = kLanes / 2; m > 0; m >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, m);
-        if ((lane & (kLanes - 1)) == 0) sx[(buf * kTok + tok) * 4 + ch / 128] = bonus;
+          for (int m = kLanes / 2; m > 0; m >>= 1) bonus += __shfl_xor_sync(0xffffffffu, bonus, m);
+          if ((lane & (kLanes - 1)) == 0) sx[(buf * kTok + tok) * 4 + ch / 128] = bonus;
+        }
       } else {
         const float dt = softplusf(rdt[i] + dt_bias);
 #pragma unroll
         for (int j = 0; j < 4; ++j) ka[j] *= dt;
         if (ch == 0) sx[(buf * kTok + tok) * 4] = live ? decay_exp(-rate * dt) : 1.f;
       }
-      *reinterpret_cast<float4*>(sq + at) = make_float4(qa[0], qa[1], qa[2], qa[3]);
+      if constexpr (OUT) *reinterpret_cast<float4*>(sq + at) = make_float4(qa[0], qa[1], qa[2], qa[3]);
       *reinterpret_cast<float4*>(sk + at) = make_float4(ka[0], ka[1], ka[2], ka[3]);
     }
 #pragma unroll
@@ -195,6 +218,9 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
       c0[c] = c < p.d ? p.zb[head * p.d + c] : 0.f;
       c1[c] = c < p.d ? p.u[head * p.d + c] : 0.f;
     }
+  f2 prod[!OUT && KIND == kChannel ? R / 2 : 1];             // products of decays: rows of this lane, or one number
+#pragma unroll
+  for (int i = 0; i < (!OUT && KIND == kChannel ? R / 2 : 1); ++i) prod[i] = pack2(1.f, 1.f);
   fetch(0);
   __syncthreads();
   stage(0, 0);
@@ -214,6 +240,7 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
         if constexpr (KIND == kScalar) {
           const float a = sx[tok * 4];
           dec = pack2(a, a);
+          if constexpr (!OUT) prod[0] = mul2(prod[0], dec);
         }
 #pragma unroll
         for (int c = 0; c < C; ++c) {
@@ -224,7 +251,7 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
 #pragma unroll
         for (int i4 = 0; i4 < R / 4; ++i4) {
           const int at = tok * D + i4 * 64 + rg * 4;
-          const float4 q4 = *reinterpret_cast<const float4*>(sq + at);
+          const float4 q4 = OUT ? *reinterpret_cast<const float4*>(sq + at) : make_float4(0.f, 0.f, 0.f, 0.f);
           const float4 k4 = *reinterpret_cast<const float4*>(sk + at);
           const f2 qp[2] = {pack2(q4.x, q4.y), pack2(q4.z, q4.w)};
           const f2 kp[2] = {pack2(k4.x, k4.y), pack2(k4.z, k4.w)};
@@ -233,6 +260,10 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
             const float4 w4 = *reinterpret_cast<const float4*>(sw + at);
             wp[0] = pack2(w4.x, w4.y);
             wp[1] = pack2(w4.z, w4.w);
+            if constexpr (!OUT) {
+              prod[i4 * 2] = mul2(prod[i4 * 2], wp[0]);
+              prod[i4 * 2 + 1] = mul2(prod[i4 * 2 + 1], wp[1]);
+            }
           }
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
@@ -241,7 +272,7 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
               const f2 old = S[i4 * 2 + j][c];
               const f2 s = fma2(wp[j], old, mul2(kp[j], vv[c]));
               S[i4 * 2 + j][c] = s;
-              acc[c] = fma2(qp[j], KIND == kChannel ? old : s, acc[c]);
+              if constexpr (OUT) acc[c] = fma2(qp[j], KIND == kChannel ? old : s, acc[c]);
             }
           }
         }
@@ -252,6 +283,7 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
           part[u * C + c] = lo + hi;
         }
       }
+      if constexpr (!OUT) return;
       // sum over the 16 row lanes; each halving step keeps half of the values on either side
       int base = 0, width = 4 * C;
 #pragma unroll
@@ -305,6 +337,25 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
     __syncthreads();
   }
 
+  if (OUT && cut) return;                   // decay_chain_kernel has stored the sequence's state
+  if constexpr (!OUT) {
+    if (slice == 0 && warp == 0 && cg == 0) {
+      float* dst = p.seg_decay + piece * p.d;
+      float a, bb;
+      if constexpr (KIND == kScalar) {
+        unpack2(prod[0], a, bb);
+        if (rg == 0) dst[0] = a;
+      } else {
+#pragma unroll
+        for (int i = 0; i < R / 2; ++i) {
+          const int row = (i >> 1) * 64 + rg * 4 + (i & 1) * 2;
+          unpack2(prod[i], a, bb);
+          if (row < p.d) dst[row] = a;
+          if (row + 1 < p.d) dst[row + 1] = bb;
+        }
+      }
+    }
+  }
 #pragma unroll
   for (int i = 0; i < R / 2; ++i) {
     const int row = (i >> 1) * 64 + rg * 4 + (i & 1) * 2;
@@ -318,6 +369,49 @@ __global__ void __launch_bounds__(kWarps * 32) decay_scan_kernel(const ScanParam
       }
     }
   }
+}
+
+// Start states of segments from their end states and decays, and the sequences' last states.  Block: (256 groups of VEC state
+// values, head, sequence).
+template <int VEC, int KIND>
+__global__ void __launch_bounds__(256) decay_chain_kernel(const ScanParams p) {
+  fi::pdl_launch_dependents();
+  fi::pdl_wait();
+  const int head = blockIdx.y, b = blockIdx.z, slot = p.slots[b];
+  const int at = (blockIdx.x * 256 + threadIdx.x) * VEC, size = p.d * p.dv;
+  const int n = p.cu_q[b + 1] - p.cu_q[b];
+  if (at >= size || n <= 0 || slot < 0 || slot >= p.num_slots) return;
+  float* pool = p.pool + (static_cast<long>(slot) * p.H + head) * size + at;
+  const int row = KIND == kChannel ? at / p.dv : 0;          // a group lies in one row
+  float S[VEC];
+  auto load = [](const float* src, float* v) {
+    if constexpr (VEC == 4) expand4(load4(src, 4, 1), kFp32, v); else v[0] = src[0];
+  };
+  auto store = [](float* dst, const float* v) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]); else dst[0] = v[0];
+  };
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) S[e] = 0.f;
+  if (p.seq_lens[b] != n) load(pool, S);
+  const int end = p.seg_base[b + 1];
+  constexpr int U = 4;                      // segments whose values are in flight together
+  for (int g0 = p.seg_base[b]; g0 < end; g0 += U) {
+    float u[U][VEC], w[U];
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+      const long piece = static_cast<long>(min(g0 + i, end - 1)) * p.H + head;
+      load(p.seg_state + piece * size + at, u[i]);
+      w[i] = p.seg_decay[piece * p.d + row];
+    }
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+      if (g0 + i >= end) break;
+      store(p.seg_state + (static_cast<long>(g0 + i) * p.H + head) * size + at, S);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) S[e] = fmaf(w[i], S[e], u[i][e]);
+    }
+  }
+  store(pool, S);
 }
 
 __device__ __forceinline__ float block_sum(float v, float* red) {      // 256 threads; red[8] is free again after the next barrier
@@ -712,35 +806,47 @@ __global__ void __launch_bounds__(256) part_norm_kernel(const NormParams p) {
   }
 }
 
-template <int R, int C, int KIND>
-int launch_scan(const ScanParams& p, int B, cudaStream_t s) {
+template <int R, int C, int KIND, bool OUT>
+int launch_scan(const ScanParams& p, int pieces, cudaStream_t s) {
   using L = ScanShape<R, C, KIND>;
-  const dim3 grid(p.H * ((p.dv + L::COLS - 1) / L::COLS), B), block(kWarps * 32);
+  const dim3 grid(p.H * ((p.dv + L::COLS - 1) / L::COLS), pieces), block(kWarps * 32);
   constexpr int smem = L::kFloats * 4;
-  auto kern = p.type == kFp32 ? decay_scan_kernel<R, C, KIND, float> : decay_scan_kernel<R, C, KIND, uint16_t>;
+  auto kern = p.type == kFp32 ? decay_scan_kernel<R, C, KIND, float, OUT> : decay_scan_kernel<R, C, KIND, uint16_t, OUT>;
   const cudaError_t e = fi::ensure_dynamic_smem(kern, smem);
   if (e != cudaSuccess) return static_cast<int>(e);
   return static_cast<int>(fi::launch_kernel(kern, grid, block, smem, s, 0, p));
 }
 
-template <int R, int KIND>
+template <int R, int KIND, bool OUT>
 int pick_cols(const ScanParams& p, int B, cudaStream_t s) {
   // wide tiles spend the fewest instructions per element, narrow ones fill the device when there are few sequences
   const long ctas4 = static_cast<long>(B) * p.H * ((p.dv + 63) / 64);
   if constexpr (R <= 8) {
-    if (ctas4 >= 192) return launch_scan<R, 4, KIND>(p, B, s);
+    if (ctas4 >= 192) return launch_scan<R, 4, KIND, OUT>(p, B, s);
   }
-  if (ctas4 >= 120) return launch_scan<R, 2, KIND>(p, B, s);
-  return launch_scan<R, 1, KIND>(p, B, s);
+  if (ctas4 >= 120) return launch_scan<R, 2, KIND, OUT>(p, B, s);
+  return launch_scan<R, 1, KIND, OUT>(p, B, s);
+}
+
+template <int KIND, bool OUT>
+int dispatch_pass(const ScanParams& p, int pieces, cudaStream_t s) {
+  if (p.d <= 64) return pick_cols<4, KIND, OUT>(p, pieces, s);
+  if (p.d <= 128) return pick_cols<8, KIND, OUT>(p, pieces, s);
+  if (p.d <= 256) return pick_cols<16, KIND, OUT>(p, pieces, s);
+  if (p.d <= 512) return launch_scan<32, 1, KIND, OUT>(p, pieces, s);
+  return -11;
 }
 
 template <int KIND>
-int dispatch_scan(const ScanParams& p, int B, cudaStream_t s) {
-  if (p.d <= 64) return pick_cols<4, KIND>(p, B, s);
-  if (p.d <= 128) return pick_cols<8, KIND>(p, B, s);
-  if (p.d <= 256) return pick_cols<16, KIND>(p, B, s);
-  if (p.d <= 512) return launch_scan<32, 1, KIND>(p, B, s);
-  return -11;
+int dispatch_scan(const ScanParams& p, int segments, cudaStream_t s) {
+  if (p.seg_base == nullptr) return dispatch_pass<KIND, true>(p, p.B, s);
+  int rc = dispatch_pass<KIND, false>(p, segments, s);
+  if (rc != 0) return rc;
+  const bool vec4 = p.dv % 4 == 0 && ((reinterpret_cast<uintptr_t>(p.pool) | reinterpret_cast<uintptr_t>(p.seg_state)) & 15) == 0;
+  const int per = 256 * (vec4 ? 4 : 1);
+  auto kern = vec4 ? decay_chain_kernel<4, KIND> : decay_chain_kernel<1, KIND>;
+  rc = static_cast<int>(fi::launch_kernel(kern, dim3((p.d * p.dv + per - 1) / per, p.H, p.B), dim3(256), 0, s, 0, p));
+  return rc != 0 ? rc : dispatch_pass<KIND, true>(p, segments, s);
 }
 
 template <int KIND>
@@ -766,20 +872,24 @@ bool vec_rows(const ScanParams& p, bool z_rows) {
 // Portions.  kind 0 (channel decays, bonus): q = r, k, v rows of H heads (G = H), z fp32 [T, ldz] (H * d), zb = w0 [H * d],
 // u = bonus [H * d], rate unused.  kind 1 (scalar decays, skip): q = C and k = B rows of G groups, v = x of H heads, z fp32
 // [T, ldz] (H step sizes), zb = their bias [H], u = D [H], rate [H].  type (0 bf16, 1 fp16, 2 fp32): q, k and v.  pool fp32
-// [num_slots, H, d, dv]; o fp32 [T, H, dv].  d <= 512.
+// [num_slots, H, d, dv]; o fp32 [T, H, dv].  d <= 512.  seg_base (or null) int32 [B + 1] counts segments of seg_len tokens,
+// `segments` its last entry; seg_state fp32 [segments, H, d, dv] and seg_decay fp32 [segments, H, d] are scratch.
 extern "C" int fi_decay_scan(int kind, const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* z,
                              long ldz, const float* zb, const float* u, const float* rate, float* pool, const int* slots,
-                             const int* cu_q, const int* seq_lens, float* o, int B, int H, int G, int d, int dv, int num_slots,
-                             int type, void* stream) {
+                             const int* cu_q, const int* seq_lens, float* o, const int* seg_base, int seg_len, int segments,
+                             float* seg_state, float* seg_decay, int B, int H, int G, int d, int dv, int num_slots, int type,
+                             void* stream) {
   if (B <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || d <= 0 || dv <= 0 || B > 65535 || type < 0 || type > 2 || (kind != 0 && kind != 1)) return -10;
+  if (seg_base != nullptr && (seg_len <= 0 || segments <= 0 || segments > 65535 || seg_state == nullptr || seg_decay == nullptr)) return -10;
   ScanParams p = {};
   p.q = q; p.k = k; p.v = v; p.ldq = ldq; p.ldk = ldk; p.ldv = ldv; p.z = z; p.ldz = ldz; p.zb = zb; p.u = u; p.rate = rate;
   p.pool = pool; p.slots = slots; p.cu_q = cu_q; p.seq_lens = seq_lens; p.o = o; p.H = H; p.G = G; p.d = d; p.dv = dv;
-  p.num_slots = num_slots; p.type = type;
+  p.num_slots = num_slots; p.type = type; p.B = B; p.seg_base = seg_base; p.seg_len = seg_len; p.seg_state = seg_state;
+  p.seg_decay = seg_decay;
   p.vec4 = vec_rows(p, kind == 0);
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
-  return kind == 0 ? dispatch_scan<kChannel>(p, B, s) : dispatch_scan<kScalar>(p, B, s);
+  return kind == 0 ? dispatch_scan<kChannel>(p, segments, s) : dispatch_scan<kScalar>(p, segments, s);
 }
 
 // One token per sequence, channel decays: operands of fi_decay_scan with B rows, then per head norm(o) * norm_w [H * dv] *

@@ -384,16 +384,41 @@ def _check_pool(pool, batch) -> None:
     assert pool.dtype == torch.float32 and pool.is_contiguous() and batch.extras["slot_ids"].dtype == batch.seq_lens.dtype == torch.int32
 
 
-def _scan(kind: int, q, k, v, z, zb, u, rate, pool, batch, G: int):
+# segments are worth their second pass when one portion is at least this long
+_SEGMENT_FROM = 512
+
+
+def _segments(batch, heads: int, dv: int, length: int = 0):
+    """(running count of segments per portion int32 [B + 1], tokens per segment, number of segments) for a step of few long
+    portions, or None: the portions fill the device as they are.  ``length``: tokens per segment (0: chosen)."""
+    T, blocks = sum(batch.q_lens_cpu), heads * -(-dv // 64)
+    if length == 0:
+        longest = max(batch.q_lens_cpu)
+        if longest < _SEGMENT_FROM or T * blocks > 64 * longest:       # twice the work must pay for the parallelism
+            return None
+        length = min(512, max(64, -(-T * blocks // 592) + 15 & ~15))
+    key = f"segments{length}"
+    if key not in batch.extras:
+        n = (batch.cu_q[1:] - batch.cu_q[:-1] + length - 1) // length
+        batch.extras[key] = (F.pad(torch.cumsum(n, 0), (1, 0)).to(torch.int32), length, sum(-(-m // length) for m in batch.q_lens_cpu))
+    return batch.extras[key]
+
+
+def _scan(kind: int, q, k, v, z, zb, u, rate, pool, batch, G: int, segment: int = 0):
     T, (slots, H, d, dv) = v.shape[0], pool.shape
     o = torch.empty(T, H * dv, dtype=torch.float32, device=v.device)
     assert q.dtype == k.dtype == v.dtype and z.dtype == torch.float32 and q.stride(1) == k.stride(1) == v.stride(1) == z.stride(1) == 1
     _check_pool(pool, batch)
+    seg, cut = (None, 0, 0, None, None), _segments(batch, H, dv, segment)
+    if cut is not None:
+        base, length, n = cut
+        work = scratch("decay_segments", n * H * d * (dv + 1) * 4, v.device)
+        seg = (_p(base), length, n, _p(work), work.data_ptr() + n * H * d * dv * 4)
     rc = _lib.kernels().fi_decay_scan(kind, _p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), z.stride(0), _p(zb),
                                       _p(u), _p(rate), _p(pool), _p(batch.extras["slot_ids"]), _p(batch.cu_q), _p(batch.seq_lens),
-                                      _p(o), batch.seq_lens.shape[0], H, G, d, dv, slots, _DT[v.dtype], _stream())
+                                      _p(o), *seg, batch.seq_lens.shape[0], H, G, d, dv, slots, _DT[v.dtype], _stream())
     _lib.check(rc, "fi_decay_scan")
-    _count()
+    _count(1 if cut is None else 3)
     return o
 
 

@@ -538,6 +538,28 @@ def test_every_column_width_of_the_scans(B, n):
         close(b[i * n:(i + 1) * n], a.cpu(), 1e-5)
 
 
+@gpu
+@pytest.mark.parametrize("H, G, d, dv", [(4, 2, 64, 64), (2, 1, 12, 20), (2, 2, 130, 66), (3, 1, 5, 7), (1, 1, 300, 40)])
+@pytest.mark.parametrize("segment", [16, 48, 100])
+def test_segments_of_long_portions(H, G, d, dv, segment):
+    """Portions cut into segments that run side by side: new and continued sequences, portions of any length."""
+    lens, done, slots = [500, 1, 97, 48], [0, 30, 65, 0], [3, 0, 2, 1]
+    n = sum(lens)
+    q, k, v, z = rnd(n, H * d, seed=1), rnd(n, H * d, seed=2), rnd(n, H * dv, seed=3), rnd(n, H * d, seed=4)
+    w0, u, rate, pool = rnd(H * d, seed=5, std=2.0) - 3, rnd(H * d, seed=6), torch.exp(rnd(H, seed=7)), rnd(4, H, d, dv, seed=8)
+    cuda = lambda *ts: [t.cuda() for t in ts]
+    for kind, args in ((0, (q, k, v, z, w0, u, rate)), (1, (q[:, :G * d], k[:, :G * d], v, z[:, :H].contiguous(), w0[:H].contiguous(), u[:H].contiguous(), rate))):
+        got = []
+        for cut in (segment, 10 ** 6):                      # one segment: the plain walk, up to the chain of one
+            p, b = pool.cuda(), make_batch("cuda", slots, lens, done)
+            got.append((lin._scan(kind, *cuda(*args), p, b, H if kind == 0 else G, cut), p))
+        p, b = pool.cuda(), make_batch("cuda", slots, lens, done)
+        plain = (lin._scan(kind, *cuda(*args), p, b, H if kind == 0 else G), p)
+        for o, s in got:
+            close(o, plain[0].cpu(), 2e-5)
+            close(s, plain[1].cpu(), 2e-5)
+
+
 @pytest.mark.parametrize("device", DEV)
 @pytest.mark.parametrize("n, parts", [(7, 3), (64, 4), (200, 1), (512, 2), (1000, 3), (2048, 1), (4096, 2), (8192, 1), (9000, 1)])
 def test_norm_of_parts_with_a_gate_on_either_side(n, parts, device):
