@@ -1,9 +1,9 @@
 // Linear attention with decays, in two forms.  Per head, with state S [d, dv] (32-bit, one slot per sequence):
 //
-//   channel decays, bonus    o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t      S_t = diag(w_t) S_(t-1) + k_t v_t^T
-//                            w = exp(-exp(z + w0)) per key channel
-//   scalar decays, skip      S_t = a_t S_(t-1) + dt_t B_t x_t^T             o_t = S_t^T C_t + D x_t
-//                            dt = softplus(z + bias), a = exp(-rate dt) per head; B and C belong to groups of heads, and
+//   channel decays, bonus    y = q S + (sum_i q_i u_i k_i) v,  then  S[i, :] <- w_i S[i, :] + k_i v      (q: the projection r)
+//                            ln w_i = -e^(z_i + w0_i) for every key channel i
+//   scalar decays, skip      S <- a S + (h k) v (outer product),  then  y = q S + D v                    (q: C, k: B, v: x)
+//                            h = softplus(z + bias), ln a = -rate h for every head; B and C belong to groups of heads, and
 //                            x, B and C come out of a short causal convolution with bias and SiLU
 //
 // All arithmetic is 32-bit.

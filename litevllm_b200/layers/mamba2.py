@@ -1,7 +1,7 @@
 """Mamba-2: a state-space layer with one scalar decay per head.
 
     [z | x | B | C | dt] = W_in h,   x, B, C <- silu(conv([x | B | C]) + b)       (short causal convolution per channel)
-    dt <- softplus(dt + bias),   S_t = exp(-exp(A) dt) S_(t-1) + dt B_t x_t^T,   y_t = S_t^T C_t + D x_t
+    dt <- softplus(dt + bias),   S[i, :] <- a S[i, :] + dt B_i x  with  ln a = -dt e^A,   then  y = C S + D x     (per head)
     out = W_o [rms over equal parts of (y silu(z))] * norm
 
 B and C [groups, state] are shared by groups of heads.  The state S [heads, state, vdim] is 32-bit and lives, with the last

@@ -2,8 +2,8 @@
 and the decay each read their own blend of the present and the previous input:
 
     x_i = x_t + (x_(t-1) - x_t) mu_i                                    (i of r, k, v, g, w; formed with the layer's input)
-    r, k, v = W_r x_r, W_k x_k, W_v x_v,   gate = silu(W_g x_g),   w = exp(-exp(W_2 tanh(W_1 x_w) + w0))
-    o_t = (S + diag(u) k_t v_t^T)^T r_t,   S <- diag(w_t) S + k_t v_t^T
+    r, k, v = W_r x_r, W_k x_k, W_v x_v,   gate = silu(W_g x_g),   ln w = -e^z,  z = W_2 tanh(W_1 x_w) + w0
+    o = r S + (sum_i r_i u_i k_i) v,   then  S[i, :] <- w_i S[i, :] + k_i v        (per head; i: key channels)
     y = W_o [rms(o_h) norm_h gate_h]
 
 The state S [heads, dim, dim] is 32-bit and lives in a per-layer pool of the cache manager with one slot per request.  The

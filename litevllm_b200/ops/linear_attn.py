@@ -423,7 +423,7 @@ def _scan(kind: int, q, k, v, z, zb, u, rate, pool, batch, G: int, segment: int 
 
 
 def time_mix(r, k, v, gate, z, w0, u, pool, batch, norm_w, eps: float, out_dtype):
-    """Time mixing of a step: ``o_t = (S + diag(u) k_t v_t^T)^T r_t``, ``S = diag(exp(-exp(z_t + w0))) S + k_t v_t^T``, then per
+    """Time mixing of a step: ``o = r S + (r . (u * k)) v``, ``S[i, :] = w_i S[i, :] + k_i v`` with ``ln w = -e^(z + w0)``, then per
     head norm, ``norm_w`` and ``silu(gate)``.
 
     r, k, v, gate [T, H * d] (any row pitch, one type), z fp32 [T, H * d], w0 [H * d], u [H, d], norm_w [H * d] fp32; pool fp32
